@@ -8,7 +8,7 @@
 #include <stddef.h>
 #include <stdint.h>
 
-#define XP_ABI_VERSION 21
+#define XP_ABI_VERSION 22
 
 #ifdef __cplusplus
 extern "C" {
@@ -27,8 +27,8 @@ typedef struct XpGemmArgs {
   size_t ws_bytes;
   size_t counter_bytes;
   int w_rows_total;    /* 0: derived from n_out / up_offset */
-  int n_out;           /* features produced, multiple of 128 */
-  int k;               /* multiple of 64 */
+  int n_out;           /* features produced (multiple of 128 in the dual, tiled, grouped and fp8 forms) */
+  int k;               /* row pitches are multiples of 16 bytes (multiple of 64 elements in the forms above) */
   int rows;
   int ldw, ldx, ld_out, ld_resid; /* element strides; 0 = dense */
   int epilogue;        /* 0 store bf16, 1 swiglu (dual), 2 residual add, 3 store fp32 */
@@ -50,6 +50,10 @@ typedef struct XpGemmArgs {
   const float* w_scale;
   const float* x_scale;
   int ld_xscale;
+  /* batched form, batch > 1: group g multiplies x rows [g * x_group_rows, + rows) with w rows
+   * [g * w_rows_per_group, + n_out) into out + g * out_group_stride (elements) */
+  int batch, x_group_rows, out_group_stride;
+  float out_scale;     /* multiplies the accumulator of epilogues 0 and 3; 0 = 1 */
 } XpGemmArgs;
 
 typedef struct XpGemmPlan {
@@ -292,6 +296,14 @@ typedef struct XpPrefillAttnArgs {
   uint32_t* status;           /* optional, FOUR words: [0] set non-zero when a bounded wait ran out (7: tcgen05 kernel),
                                  [1..3] detail of the first such CTA (wait site, block, tiles) */
   int total_q;                /* rows of q / out (bound of the query tensor map); 0: no tcgen05 kernel */
+  /* tcgen05 kernel only */
+  int v_dim;                  /* value width; 0: head_dim */
+  int v_valid;                /* columns of a head stored to out (multiple of 8); 0: v_dim */
+  int ld_out;                 /* elements of an out row (multiple of 8); 0: q_heads * v_valid */
+  const int* seq_starts;      /* [num_seqs] first K/V row of each sequence when its rows lie densely (no block table) */
+  const void* gate;           /* optional bf16 [total_q, ld_gate] logits: head h's output is multiplied by sigmoid */
+  int ld_gate;
+  int p_pair;                 /* probabilities as a bf16 pair in the second product */
 } XpPrefillAttnArgs;
 
 int xp_rope_kv(const XpRopeArgs* a, void* stream);

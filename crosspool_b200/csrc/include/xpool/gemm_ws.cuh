@@ -60,8 +60,8 @@ struct Problem {
   const float* bias;          // [n_out] or null
   float* ws;                  // split-K workspace or null
   uint32_t* counters;         // one per (m, n) tile, zero between calls
-  int n_out;                  // features produced (multiple of 128)
-  int k;                      // multiple of 64
+  int n_out;                  // features produced; a last partial 128-row tile reads zeros and stores nothing past n_out
+  int k;                      // a last partial K block reads zeros on both operands
   int rows;                   // live activation rows
   int ld_out;
   int ld_resid;
@@ -89,6 +89,13 @@ struct Problem {
   const float* w_scale;
   const float* x_scale;
   int ld_xscale;
+  // Batched form (batch > 1, e.g. one small matrix per attention head): group g multiplies activation rows
+  // [g * x_group_rows, + rows) with weight rows [g * w_rows_per_group, + n_out) and stores row r at
+  // out + g * out_group_stride + r * ld_out.
+  int batch;
+  int x_group_rows;
+  int out_group_stride;
+  float out_scale;         // multiplies the accumulator of the two plain store epilogues; 0 = 1
 };
 
 struct SmemLayout {
@@ -162,17 +169,21 @@ struct TileCoord {
   int kbn;    // number of K blocks
   int w_row0; // first weight row in the weight tensor (differs from m0 for grouped problems)
   int row_end;  // activation rows >= row_end are not stored
+  int64_t out_off;  // element offset added to the row-major output address (batched problems)
 };
 
-__device__ __forceinline__ int tiles_m(const Problem& p) { return p.n_out / kTileM; }
+__device__ __forceinline__ int tiles_m(const Problem& p) { return (p.n_out + kTileM - 1) / kTileM; }
 __device__ __forceinline__ int tiles_n(const Problem& p) { return (p.rows + p.bn - 1) / p.bn; }
 __device__ __forceinline__ int tile_count(const Problem& p) {
   if (p.tile_table != nullptr) return *p.n_tiles;
-  return tiles_m(p) * tiles_n(p) * p.splits;
+  return tiles_m(p) * tiles_n(p) * p.splits * (p.batch > 1 ? p.batch : 1);
 }
+
+__device__ __forceinline__ int k_blocks(const Problem& p) { return (p.k + p.kblk - 1) / p.kblk; }
 
 __device__ __forceinline__ TileCoord tile_coord(const Problem& p, int t) {
   TileCoord c;
+  c.out_off = 0;
   if (p.tile_table != nullptr) {
     const int4 e = p.tile_table[t];
     c.m0 = e.y;
@@ -182,7 +193,7 @@ __device__ __forceinline__ TileCoord tile_coord(const Problem& p, int t) {
     c.split = 0;
     c.mn = t;
     c.kb0 = 0;
-    c.kbn = p.k / p.kblk;
+    c.kbn = k_blocks(p);
     return c;
   }
   int tm = tiles_m(p);
@@ -191,7 +202,7 @@ __device__ __forceinline__ TileCoord tile_coord(const Problem& p, int t) {
   c.mn = mn;
   c.m0 = (mn % tm) * kTileM;
   c.n0 = (mn / tm) * p.bn;
-  int kb_total = p.k / p.kblk;
+  int kb_total = k_blocks(p);
   int per = (kb_total + p.splits - 1) / p.splits;
   c.kb0 = c.split * per;
   int end = c.kb0 + per;
@@ -199,6 +210,16 @@ __device__ __forceinline__ TileCoord tile_coord(const Problem& p, int t) {
   c.kbn = end > c.kb0 ? end - c.kb0 : 0;
   c.w_row0 = c.m0;
   c.row_end = p.rows;
+  if (p.batch > 1) {
+    const int per_group = tm * tiles_n(p);
+    const int g = mn / per_group;
+    mn -= g * per_group;
+    c.m0 = (mn % tm) * kTileM;
+    c.n0 = g * p.x_group_rows + (mn / tm) * p.bn;
+    c.w_row0 = g * p.w_rows_per_group + c.m0;
+    c.row_end = g * p.x_group_rows + p.rows;
+    c.out_off = static_cast<int64_t>(g) * (p.out_group_stride - static_cast<int64_t>(p.x_group_rows) * p.ld_out);
+  }
   return c;
 }
 
@@ -226,7 +247,7 @@ __device__ __forceinline__ bool produce_tile(const Problem& p, const TileCoord& 
   const uint64_t tx_map = reinterpret_cast<uint64_t>(p.tmap_x);
   // Row-major weights: box at (k, row). Tiled weights: every 128x64 tile is one
   // contiguous 16 KB run, tile index = m_tile * k_tiles + k_tile.
-  const int kb_total = p.k / p.kblk;
+  const int kb_total = k_blocks(p);
   int wc0, wc1, uc1, dwc0, dwc1;
   if (p.w_tiled) {
     wc0 = 0;
@@ -416,10 +437,11 @@ __device__ __forceinline__ void epi_bar_sync() {
 // independent chains (fully unrolled, no early exit) and stored with
 // predicates, the epilogue kind is tested once per call.
 __device__ __forceinline__ void epilogue_store16(const Problem& p, int f, int fb, int n_first, int row_end,
-                                                 const float* g, const float* u) {
-  const float bias = p.bias != nullptr ? p.bias[fb] : 0.f;
-  const int valid = row_end - n_first;  // > 0 by the callers' checks
-  const size_t o0 = static_cast<size_t>(n_first) * p.ld_out + f;
+                                                 const float* g, const float* u, int64_t out_off = 0) {
+  const bool live = f < p.n_out;        // false in the padding rows of a last partial weight tile
+  const float bias = (p.bias != nullptr && live) ? p.bias[fb] : 0.f;
+  const int valid = live ? row_end - n_first : 0;  // live: > 0 by the callers' checks
+  const int64_t o0 = static_cast<int64_t>(n_first) * p.ld_out + f + out_off;
   float v[16];
   if (p.epilogue == kEpiSwiglu) {
     const float bias_u = (p.bias != nullptr && p.dual) ? p.bias[p.up_offset + fb] : 0.f;
@@ -439,8 +461,9 @@ __device__ __forceinline__ void epilogue_store16(const Problem& p, int f, int fb
 #pragma unroll
     for (int j = 0; j < 16; ++j) v[j] = round_bf16(g[j] + bias) + rr[j];
   } else {
+    const float sc = p.out_scale == 0.f ? 1.f : p.out_scale;
 #pragma unroll
-    for (int j = 0; j < 16; ++j) v[j] = g[j] + bias;
+    for (int j = 0; j < 16; ++j) v[j] = fmaf(g[j], sc, bias);
   }
   if (p.epilogue == kEpiStoreF32) {
     float* o = reinterpret_cast<float*>(p.out) + o0;
@@ -530,7 +553,7 @@ __device__ __forceinline__ bool epilogue_tile(const Problem& p, const TileCoord&
     if (p.splits == 1) {
 #pragma unroll
       for (int cc = 0; cc < kMaxBnF8 / 16; ++cc)
-        if (cc * 16 < p.bn && c.n0 + cc * 16 < c.row_end) epilogue_store16(p, f, fb, c.n0 + cc * 16, c.row_end, &acc[cc * 16], u);
+        if (cc * 16 < p.bn && c.n0 + cc * 16 < c.row_end) epilogue_store16(p, f, fb, c.n0 + cc * 16, c.row_end, &acc[cc * 16], u, c.out_off);
     } else {
       float* ws = p.ws + (static_cast<size_t>(c.mn) * p.splits + c.split) * acc_cols * kTileM;
 #pragma unroll
@@ -559,7 +582,7 @@ __device__ __forceinline__ bool epilogue_tile(const Problem& p, const TileCoord&
         g[j] = __uint_as_float(ga[j]);
         u[j] = __uint_as_float(ua[j]);
       }
-      epilogue_store16(p, f, fb, c.n0 + col, c.row_end, g, u);
+      epilogue_store16(p, f, fb, c.n0 + col, c.row_end, g, u, c.out_off);
       if (more) {
         sm100::tmem_ld_wait32(gb, ub);
         if (col + 32 < ncol) {
@@ -571,7 +594,7 @@ __device__ __forceinline__ bool epilogue_tile(const Problem& p, const TileCoord&
           g[j] = __uint_as_float(gb[j]);
           u[j] = __uint_as_float(ub[j]);
         }
-        epilogue_store16(p, f, fb, c.n0 + col + 16, c.row_end, g, u);
+        epilogue_store16(p, f, fb, c.n0 + col + 16, c.row_end, g, u, c.out_off);
       }
     }
   } else {
@@ -629,7 +652,7 @@ __device__ __forceinline__ bool epilogue_tile(const Problem& p, const TileCoord&
             }
           }
         }
-        epilogue_store16(p, f, fb, c.n0 + col, c.row_end, g, u);
+        epilogue_store16(p, f, fb, c.n0 + col, c.row_end, g, u, c.out_off);
       }
       if (ew == 0 && lane == 0) p.counters[c.mn] = 0;  // ready for the next call
     }

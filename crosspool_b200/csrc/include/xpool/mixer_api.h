@@ -1,0 +1,137 @@
+/* C ABI of the row-wise and mixer kernels of layered (hybrid) decoders: per-layer mixers over a latent KV cache or a
+ * recurrent state, gated 32-bit residual streams, norms without statistics, row-normalised activations. Mirrored by
+ * ctypes.Structures in crosspool_b200/native/__init__.py; XP_ABI_VERSION covers these structs too.
+ *
+ * `f32` selects the element type of activations, caches and weights: 0 bf16, 1 fp32. */
+#ifndef XPOOL_MIXER_API_H_
+#define XPOOL_MIXER_API_H_
+
+#include <stdint.h>
+
+#ifdef __cplusplus
+extern "C" {
+#endif
+
+/* resid[r] = ids ? table[ids[r]] : resid[r] + (sum of parts)[r] * sigmoid(gate[r]);  out[i] = norm(resid[r]),
+ * with r = sel ? sel[i] : i. With sel the residual is read only. */
+typedef struct XpResidNormArgs {
+  float* resid;          /* [*, hidden] */
+  const void* parts[8];  /* activations [*, ld_part] */
+  const void* gate;      /* optional logits [*, ld_gate]; null: no gate */
+  const int* ids;        /* optional: start the residual from the embedding table */
+  const void* table;     /* [vocab, hidden] */
+  const int* sel;        /* optional row selection */
+  const float* weight;   /* [hidden] */
+  const float* bias;     /* optional [hidden] */
+  const float* alpha;    /* dynamic tanh: one device float */
+  void* out;             /* [rows, ld_out]; null: residual update only */
+  int rows, hidden, nparts, ld_part, ld_gate, ld_out, vocab;
+  int kind;              /* 0 rms, 1 layernorm, 2 dynamic tanh */
+  float eps;
+  int f32;
+} XpResidNormArgs;
+
+/* out = coef0 N(z) + coef1 N(z^2) + coef2 N(z^3) + coef3 over each row, N dividing by the root mean square. */
+typedef struct XpPolyNormArgs {
+  const void* z;
+  const float* coef;     /* 4 device floats */
+  void* out;
+  int rows, cols, ld_z, ld_out;
+  float eps;
+  int f32;
+} XpPolyNormArgs;
+
+/* out = rmsnorm(o) * weight * sigmoid(gate), o in fp32. */
+typedef struct XpGatedRmsArgs {
+  const float* o;
+  const float* weight;
+  const void* gate;      /* logits [rows, ld_gate] */
+  void* out;
+  int rows, cols, ld_o, ld_gate, ld_out;
+  float eps;
+  int f32;
+} XpGatedRmsArgs;
+
+/* Latent attention, per token row: normalise the latent, rotate the shared key part, write both to the cache row of the
+ * token; rotate the rotary part of every query head and lay the queries out for the absorbed form
+ * (q_plain head-major, q_abs columns [kv_rank, +rot)) and/or the expanded form (q_exp). */
+typedef struct XpLatentPrepArgs {
+  const void* proj;      /* [rows, ld_proj]: q at q_off (heads x (dim + rot)), latent + key at kv_off (kv_rank + rot) */
+  const float* norm_w;   /* [kv_rank] */
+  const double* freq;    /* [rot_dims / 2] rotary frequencies */
+  const int* positions;  /* [rows] */
+  const int* slots;      /* [rows] cache row, -1: none */
+  void* cache;           /* [tokens, ld_cache] */
+  void* q_plain;         /* [heads, qp_rows, dim_p], or null */
+  void* q_abs;           /* [heads, qp_rows, ld_abs], or null */
+  void* q_exp;           /* [rows, heads, dq_pad] zero-padded, or null */
+  int rows, heads, dim, rot, rot_dims, kv_rank, ld_proj, q_off, kv_off, ld_cache, qp_rows, dim_p, ld_abs, dq_pad;
+  int abs_rows;          /* rows < abs_rows are laid out for the absorbed form, the others for the expanded one */
+  float eps;
+  int f32;
+} XpLatentPrepArgs;
+
+/* Attention of single rows against the latent cache (keys: the first kv_rank + rot columns of a cache row shared by
+ * every head; values: its first kv_rank columns). Row r attends to positions[r] + 1 tokens of table row row_seq[r]. */
+typedef struct XpLatentAttnArgs {
+  const void* q;         /* [heads, q_rows, ld_q] (kv_rank + rot columns) */
+  const void* cache;     /* [pages, page_size, ld_cache] */
+  void* out;             /* [heads, q_rows, ld_out] (kv_rank columns) */
+  const void* gate;      /* optional per-head output gate logits [rows, ld_gate] */
+  const int* row_seq;    /* [rows] block-table row, or null: row r uses table row r */
+  const int* positions;  /* [rows] */
+  const int* slots;      /* [rows] < 0: padding row (zeros are stored) */
+  const int* block_table;
+  float* ws;             /* split partials */
+  int rows, heads, kv_rank, rot, q_rows, ld_q, ld_cache, ld_out, ld_gate, page_size, max_blocks;
+  int num_splits, chunk_tokens;
+  float scale;
+  int f32;
+  int force_simt;
+} XpLatentAttnArgs;
+
+/* Copies the cached latents of each sequence to a dense workspace: sequence i's ctx + q tokens start at row starts[i]. */
+typedef struct XpLatentGatherArgs {
+  const void* cache;
+  void* out;             /* [*, ld_cache] */
+  const int* block_table;
+  const int* ctx_lens;
+  const int* q_lens;
+  const int* starts;     /* [n_seqs] first workspace row */
+  int n_seqs, max_len, page_size, max_blocks, ld_cache, elem_bytes;
+} XpLatentGatherArgs;
+
+/* Decayed linear attention S = decay S + k v^T, o = S^T q with silu on q, k, v; the state of sequence slot s is
+ * state[s][heads][dim][vdim] in fp32. A sequence whose first row sits at position 0 starts from a zero state. */
+typedef struct XpLinearAttnArgs {
+  const void* proj;      /* [rows, ld_proj]: q, k (heads x dim) and v (heads x vdim) at the three offsets */
+  float* state;
+  const float* decay;    /* [heads] */
+  const float* decay_pow;/* [heads, kChunk + 1]: decay^0 .. decay^kChunk */
+  float* out;            /* [rows, heads * vdim] fp32 */
+  const int* positions;  /* [rows] */
+  const int* slots;      /* [rows] KV slot of the row, < 0: padding row */
+  const int* state_slots;/* [seqs] */
+  const int* q_starts;   /* [seqs] prefill: first row */
+  const int* q_lens;     /* [seqs] prefill: rows */
+  float* ws;             /* chunked prefill: chunk states */
+  int rows, seqs, seq0, max_q_len, heads, dim, vdim, ld_proj, q_off, k_off, v_off, ws_chunks;
+  int f32;
+} XpLinearAttnArgs;
+
+int xp_resid_norm(const XpResidNormArgs* a, void* stream);
+int xp_polynorm(const XpPolyNormArgs* a, void* stream);
+int xp_gated_rms(const XpGatedRmsArgs* a, void* stream);
+int xp_latent_prep(const XpLatentPrepArgs* a, void* stream);
+int xp_latent_attn(const XpLatentAttnArgs* a, void* stream);
+int xp_latent_gather(const XpLatentGatherArgs* a, void* stream);
+int xp_linear_attn_decode(const XpLinearAttnArgs* a, void* stream);
+int xp_linear_attn_prefill(const XpLinearAttnArgs* a, void* stream);
+/* out[b][r][n] = sum_k x[b][r][k] w[b][n][k] (* out_scale) (+ bias) in true fp32 (no reduced-precision product). */
+int xp_gemm_f32(const float* x, const float* w, const float* bias, float* out, int rows, int n, int k, int ldx, int ldw, int ldo,
+                int batch, int64_t sx, int64_t sw, int64_t so, float out_scale, void* stream);
+
+#ifdef __cplusplus
+}
+#endif
+#endif /* XPOOL_MIXER_API_H_ */

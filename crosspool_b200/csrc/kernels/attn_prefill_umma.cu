@@ -19,6 +19,10 @@
 //   warp 9      allocates tensor memory and issues every tcgen05.mma from one thread. S is double-buffered per
 //               tile and issued one K/V tile ahead, in the order S_A(t+1), PV_A(t), S_B(t+1), PV_B(t).
 //
+// Keys and values may differ in width (DQ, DV; latent attention in its expanded form: keys are [plain | rotary] columns),
+// their rows may lie densely per sequence instead of in pages, every head's output may be gated by a sigmoid, and the
+// probabilities may enter the second product as a bf16 pair (high and low part: two products, 16 mantissa bits).
+//
 // V is used where it lands (token-major rows of 64 dims) through an MN-major operand descriptor; no transpose.
 // Tensor memory: S buffers 4 x 64 columns, O 2 x D columns (512 columns with D = 128).
 // Every wait is bounded; a wait that runs out sets the abort word, the status word (7) and ends the CTA after a
@@ -80,21 +84,23 @@ __device__ __forceinline__ uint32_t pack2(float lo, float hi) {
   return *reinterpret_cast<uint32_t*>(&v);
 }
 
-template <int D, bool kTS>
+template <int DQ, int DV, bool kTS, bool kPair>
 __global__ void __launch_bounds__(kThreads, 1)
 prefill_attn_umma_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
                          const __grid_constant__ CUtensorMap tmap_v, const __grid_constant__ CUtensorMap tmap_k3,
                          const __grid_constant__ CUtensorMap tmap_v3, XpPrefillAttnArgs a, int G, int g_shift,
                          int box_tokens) {
-  constexpr int kHalves = D / 64;                 // 64-dim (128-byte) column blocks of a row
+  static_assert(kTS || !kPair, "the low parts live beside the high parts in tensor memory");
+  constexpr int kHalves = DQ / 64;                // 64-dim (128-byte) column blocks of a query or key row
+  constexpr int kVHalves = DV / 64;               // ... of a value row
   constexpr int kQHalf = kRows * 128;             // one 64-dim block of a query tile
   constexpr int kQTile = kHalves * kQHalf;
   constexpr int kKVHalf = kBN * 128;              // one 64-dim block of a K (or V) tile
-  constexpr int kKVTile = kHalves * kKVHalf;
-  constexpr int kStage = 2 * kKVTile;             // K then V
+  constexpr int kKTile = kHalves * kKVHalf;
+  constexpr int kStage = kKTile + kVHalves * kKVHalf;   // K then V
   constexpr int kPTile = kRows * 128;             // P: 128 rows x 64 tokens bf16
-  constexpr uint32_t kTmemCols = (4 * kBN + 2 * D) <= 256 ? 256 : 512;
-  constexpr uint32_t kOCol = 4 * kBN;             // O_A at 256, O_B at 256 + D
+  constexpr uint32_t kTmemCols = (4 * kBN + 2 * DV) <= 256 ? 256 : 512;
+  constexpr uint32_t kOCol = 4 * kBN;             // O_A at 256, O_B at 256 + DV
   extern __shared__ uint8_t smem_dyn[];
   __shared__ Bars bars;
 
@@ -172,16 +178,16 @@ prefill_attn_umma_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gri
         if (lane < 2) {
           int tk = t * kBN;
           if (tk >= kv_end) tk = (kv_end - 1) & ~(kBN - 1);
-          const int tok = (table[tk >> page_shift] << page_shift) + (tk & page_mask);
-          sm100::tma_load_4d_addr(kv_s + s * kStage + lane * kKVTile, lane ? &tmap_v : &tmap_k,
+          const int tok = a.seq_starts != nullptr ? a.seq_starts[seq] + tk : (table[tk >> page_shift] << page_shift) + (tk & page_mask);
+          sm100::tma_load_4d_addr(kv_s + s * kStage + lane * kKTile, lane ? &tmap_v : &tmap_k,
                                   sm100::smem_u32(&bars.kv_full[s]), 0, tok, 0, hk);
         }
-      } else if (lane < 2 * boxes * kHalves) {
+      } else if (lane < 2 * boxes * kHalves) {       // small pages: DQ == DV (checked by the host)
         const int h = lane % kHalves, is_v = (lane / kHalves) & 1, j = lane / (2 * kHalves);
         int tk = t * kBN + j * box_tokens;
         if (tk >= kv_end) tk = (kv_end - 1) & ~(box_tokens - 1);   // boxes past the end repeat the last valid one (masked)
         const int tok = (table[tk >> page_shift] << page_shift) + (tk & page_mask);
-        sm100::tma_load_3d_addr(kv_s + s * kStage + is_v * kKVTile + h * kKVHalf + j * box_bytes, is_v ? &tmap_v3 : &tmap_k3,
+        sm100::tma_load_3d_addr(kv_s + s * kStage + is_v * kKTile + h * kKVHalf + j * box_bytes, is_v ? &tmap_v3 : &tmap_k3,
                                 sm100::smem_u32(&bars.kv_full[s]), h * 64, hk, tok);
       }
     }
@@ -189,12 +195,12 @@ prefill_attn_umma_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gri
     // ------------------------------------------------------------------ MMA issuer
     if (lane == 0) {
       const uint32_t idesc_s = sm100::umma_idesc_bf16(kRows, kBN);
-      const uint32_t idesc_o = sm100::umma_idesc_bf16_bmn(kRows, D);
+      const uint32_t idesc_o = sm100::umma_idesc_bf16_bmn(kRows, DV);
       auto issue_s = [&](int x, int t) {       // S_x(t) = Q_x K(t)^T into buffer t & 1
         const int s = t % kStages, bf = t & 1;
         const uint32_t d = tmem + static_cast<uint32_t>((x * 2 + bf) * kBN);
 #pragma unroll
-        for (int ks = 0; ks < D / 16; ++ks) {
+        for (int ks = 0; ks < DQ / 16; ++ks) {
           const uint64_t da = sm100::umma_desc_sw128(q_s + x * kQTile + (ks >> 2) * kQHalf) + (ks & 3) * 2;
           const uint64_t db = sm100::umma_desc_sw128(kv_s + s * kStage + (ks >> 2) * kKVHalf) + (ks & 3) * 2;
           sm100::umma_bf16(d, da, db, idesc_s, ks > 0 ? 1u : 0u);
@@ -203,15 +209,17 @@ prefill_attn_umma_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gri
       };
       auto issue_pv = [&](int x, int t) {      // O_x (+)= P_x V(t)
         const int s = t % kStages;
-        const uint32_t d = tmem + kOCol + static_cast<uint32_t>(x * D);
+        const uint32_t d = tmem + kOCol + static_cast<uint32_t>(x * DV);
 #pragma unroll
         for (int kk = 0; kk < kBN / 16; ++kk) {
           const uint64_t da = sm100::umma_desc_sw128(p_s + x * kPTile) + kk * 2;
-          const uint64_t db = sm100::umma_desc_mn_sw128(kv_s + s * kStage + kKVTile + kk * 2048, kKVHalf, 1024);
+          const uint64_t db = sm100::umma_desc_mn_sw128(kv_s + s * kStage + kKTile + kk * 2048, kKVHalf, 1024);
           if constexpr (kTS) {
             // P(t) sits in the first 32 columns of the S buffer it was computed from, 8 columns per K step
             sm100::umma_bf16_ts(d, tmem + static_cast<uint32_t>((x * 2 + (t & 1)) * kBN + kk * 8), db, idesc_o,
                                 (t > 0 || kk > 0) ? 1u : 0u);
+            if constexpr (kPair)     // low parts: the other 32 columns of the buffer
+              sm100::umma_bf16_ts(d, tmem + static_cast<uint32_t>((x * 2 + (t & 1)) * kBN + kBN / 2 + kk * 8), db, idesc_o, 1u);
           } else {
             sm100::umma_bf16(d, da, db, idesc_o, (t > 0 || kk > 0) ? 1u : 0u);
           }
@@ -271,7 +279,7 @@ prefill_attn_umma_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gri
     const int my_tiles = x == 0 ? n_a : n_tiles;
     const int limit = min(ctx + pos, kv_end - 1);     // last visible cache position of this row
     const uint32_t lane_off = static_cast<uint32_t>((warp & 3) * 32) << 16;
-    const uint32_t o_t = tmem + lane_off + kOCol + static_cast<uint32_t>(x * D);
+    const uint32_t o_t = tmem + lane_off + kOCol + static_cast<uint32_t>(x * DV);
     const uint32_t p_row = p_s + x * kPTile + row * 128;
     const float sc2 = a.scale * 1.4426950408889634f;
     float m_used = -CUDART_INF_F, l = 0.f;
@@ -325,6 +333,10 @@ prefill_attn_umma_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gri
           const float p1 = sm100::ex2_approx(fmaf(__uint_as_float(sv[j + 1]), sc2, -m_sub));
           sum4[(j >> 1) & 3] += p0 + p1;
           pk[j >> 1] = pack2(p0, p1);
+          if constexpr (kPair) {
+            const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&pk[j >> 1]));
+            sv[j >> 1] = pack2(p0 - hi.x, p1 - hi.y);     // over scores already consumed
+          }
         }
         l = l * factor + ((sum4[0] + sum4[1]) + (sum4[2] + sum4[3]));
         const bool rescale = __any_sync(0xffffffffu, factor != 1.f);
@@ -335,7 +347,7 @@ prefill_attn_umma_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gri
           if (rescale) {
             sm100::tc_fence_after_sync();
 #pragma unroll 1
-            for (int c = 0; c < D; c += 32) {
+            for (int c = 0; c < DV; c += 32) {
               uint32_t ov[32];
               sm100::tmem_ld32_issue(o_t + c, ov);
               sm100::tmem_ld_wait_all(ov);
@@ -350,6 +362,7 @@ prefill_attn_umma_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gri
         if constexpr (kTS) {
           // P row as the tensor core's A operand: 32 columns of two bf16 each, over the start of the S buffer
           sm100::tmem_st32(s_t, pk);
+          if constexpr (kPair) sm100::tmem_st32(s_t + kBN / 2, sv);
         }
         // P row: 8 chunks of 8 tokens, 16-byte chunks XOR-swizzled by the row like a TMA-written tile
 #pragma unroll
@@ -363,10 +376,10 @@ prefill_attn_umma_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gri
           // cache slots past the sequence end may hold anything: zero those V rows (probability 0 x NaN).
           // Tile A's PV product is issued before tile B's and both read this stage, so tile A's threads do it
           // on the tiles that tile A visits, tile B's on the rest.
-          const uint32_t v_s = kv_s + (t % kStages) * kStage + kKVTile;
+          const uint32_t v_s = kv_s + (t % kStages) * kStage + kKTile;
           const int first = kv_end - t * kBN;
-          for (int i = row; i < (kBN - first) * (D / 8); i += kRows) {
-            const int R = first + i / (D / 8), cc = i % (D / 8);
+          for (int i = row; i < (kBN - first) * (DV / 8); i += kRows) {
+            const int R = first + i / (DV / 8), cc = i % (DV / 8);
             const uint32_t off = (cc >> 3) * kKVHalf + R * 128 + (((cc & 7) ^ (R & 7)) << 4);
             asm volatile("st.shared.v4.u32 [%0], {%1, %1, %1, %1};" ::"r"(v_s + off), "r"(0u) : "memory");
           }
@@ -389,16 +402,20 @@ prefill_attn_umma_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gri
       if (ok && my_tiles > 0) ok = __all_sync(0xffffffffu, wait_bar(&bars.pv_done[x], (my_tiles - 1) & 1, &bars, 11));
       if (ok) {
         sm100::tc_fence_after_sync();
-        const float inv = l > 0.f ? 1.f / l : 0.f;
-        __nv_bfloat16* og = reinterpret_cast<__nv_bfloat16*>(a.out) + (static_cast<size_t>(q_base + pos) * a.q_heads + hq) * D;
+        float inv = l > 0.f ? 1.f / l : 0.f;
+        if (a.gate != nullptr && pos < q_len)
+          inv *= 1.f / (1.f + expf(-__bfloat162float(reinterpret_cast<const __nv_bfloat16*>(a.gate)[static_cast<size_t>(q_base + pos) * a.ld_gate + hq])));
+        const int v_valid = a.v_valid;                    // stored columns of a head (a multiple of 8)
+        __nv_bfloat16* og = reinterpret_cast<__nv_bfloat16*>(a.out) + static_cast<size_t>(q_base + pos) * a.ld_out + hq * v_valid;
 #pragma unroll 1
-        for (int c = 0; c < D; c += 32) {
+        for (int c = 0; c < DV; c += 32) {
           uint32_t ov[32];
           sm100::tmem_ld32_issue(o_t + c, ov);
           sm100::tmem_ld_wait_all(ov);
           if (pos < q_len) {
 #pragma unroll
             for (int j = 0; j < 32; j += 8) {
+              if (c + j >= v_valid) break;
               uint4 v;
               v.x = pack2(__uint_as_float(ov[j]) * inv, __uint_as_float(ov[j + 1]) * inv);
               v.y = pack2(__uint_as_float(ov[j + 2]) * inv, __uint_as_float(ov[j + 3]) * inv);
@@ -429,29 +446,36 @@ prefill_attn_umma_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gri
   }
 }
 
-template <int D, bool kTS>
+template <int DQ, int DV, bool kTS, bool kPair>
 static int launch(const XpPrefillAttnArgs& a, int G, cudaStream_t s) {
   CUtensorMap mq, mk, mv, mk3, mv3;
   const uint64_t tokens = static_cast<uint64_t>(a.num_pages) * a.page_size;
   int g_shift = 0;
   while ((1 << g_shift) < G) ++g_shift;
   const int np = kRows >> g_shift;
-  // pages of 64 tokens or more: one copy brings a whole K (or V) tile; smaller pages: one copy per page and 64 dims
-  const int box_tokens = a.page_size >= kBN ? kBN : 16;
-  if (tmap::cache().get_kv4(&mk, a.k_cache, tokens, a.kv_heads, D, kBN) != 0) return -20;
-  if (tmap::cache().get_kv4(&mv, a.v_cache, tokens, a.kv_heads, D, kBN) != 0) return -20;
-  if (tmap::cache().get_kv(&mk3, a.k_cache, tokens, a.kv_heads, D) != 0) return -20;
-  if (tmap::cache().get_kv(&mv3, a.v_cache, tokens, a.kv_heads, D) != 0) return -20;
-  if (tmap::cache().get_q(&mq, a.q, static_cast<uint64_t>(a.total_q), a.q_heads, D, G, np) != 0) return -20;
-  constexpr int kSmem = 2 * (D / 64) * kRows * 128 + kStages * 2 * (D / 64) * kBN * 128 + 2 * kRows * 128 + 1024;
+  // dense rows or pages of 64 tokens and more: one copy brings a whole K (or V) tile; smaller pages: one copy per page
+  // and 64 dims
+  const int box_tokens = a.page_size >= kBN || a.seq_starts != nullptr ? kBN : 16;
+  if (DQ != DV && box_tokens != kBN) return 1;
+  if (tmap::cache().get_kv4(&mk, a.k_cache, tokens, a.kv_heads, DQ, kBN) != 0) return -20;
+  if (tmap::cache().get_kv4(&mv, a.v_cache, tokens, a.kv_heads, DV, kBN) != 0) return -20;
+  if (tmap::cache().get_kv(&mk3, a.k_cache, tokens, a.kv_heads, DQ) != 0) return -20;
+  if (tmap::cache().get_kv(&mv3, a.v_cache, tokens, a.kv_heads, DV) != 0) return -20;
+  if (tmap::cache().get_q(&mq, a.q, static_cast<uint64_t>(a.total_q), a.q_heads, DQ, G, np) != 0) return -20;
+  // the shared-memory tiles of the probabilities exist only in the form that stages them there
+  constexpr int kSmem = 2 * (DQ / 64) * kRows * 128 + kStages * ((DQ + DV) / 64) * kBN * 128 + (kTS ? 0 : 2 * kRows * 128) + 1024;
+  static_assert(kSmem <= 227 * 1024, "tiles exceed the shared memory of an SM");
   static bool attr_set = false;
   if (!attr_set) {
-    if (cudaFuncSetAttribute(prefill_attn_umma_kernel<D, kTS>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem) != cudaSuccess)
+    if (cudaFuncSetAttribute(prefill_attn_umma_kernel<DQ, DV, kTS, kPair>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem) != cudaSuccess)
       return -21;
     attr_set = true;
   }
-  dim3 grid(a.kv_heads, a.num_seqs, (a.max_q_len + 2 * np - 1) / (2 * np));
-  prefill_attn_umma_kernel<D, kTS><<<grid, kThreads, kSmem, s>>>(mq, mk, mv, mk3, mv3, a, G, g_shift, box_tokens);
+  XpPrefillAttnArgs b = a;
+  if (b.v_valid <= 0) b.v_valid = DV;
+  if (b.ld_out <= 0) b.ld_out = b.q_heads * b.v_valid;
+  dim3 grid(b.kv_heads, b.num_seqs, (b.max_q_len + 2 * np - 1) / (2 * np));
+  prefill_attn_umma_kernel<DQ, DV, kTS, kPair><<<grid, kThreads, kSmem, s>>>(mq, mk, mv, mk3, mv3, b, G, g_shift, box_tokens);
   cudaError_t e = cudaGetLastError();
   return e == cudaSuccess ? 0 : -100 - static_cast<int>(e);
 }
@@ -468,13 +492,22 @@ extern "C" int xp_prefill_attn_umma(const XpPrefillAttnArgs* a, void* stream) {
   const int G = a->q_heads / a->kv_heads;
   const bool ok = a->num_pages > 0 && a->total_q > 0 && a->page_size >= 16 && (a->page_size & (a->page_size - 1)) == 0 &&
                   (G == 1 || G == 2 || G == 4 || G == 8 || G == 16) && (reinterpret_cast<uintptr_t>(a->q) & 15) == 0 &&
-                  (reinterpret_cast<uintptr_t>(a->out) & 15) == 0;
+                  (reinterpret_cast<uintptr_t>(a->out) & 15) == 0 && a->ld_out % 8 == 0 && a->v_valid % 8 == 0;
   if (!ok) return 1;
   // P (the probabilities) reaches the second product through tensor memory; bit 8 of force_simple selects the
   // form that stages P in shared memory instead
   const bool ts = ((a->force_simple >> 8) & 1) != kDefaultTS;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
-  if (a->head_dim == 128) return ts ? launch<128, true>(*a, G, s) : launch<128, false>(*a, G, s);
-  if (a->head_dim == 64) return ts ? launch<64, true>(*a, G, s) : launch<64, false>(*a, G, s);
+  const int dv = a->v_dim > 0 ? a->v_dim : a->head_dim;
+  if (a->p_pair) {
+    if (a->head_dim == 64 && dv == 64) return launch<64, 64, true, true>(*a, G, s);
+    if (a->head_dim == 128 && dv == 64) return launch<128, 64, true, true>(*a, G, s);
+    if (a->head_dim == 128 && dv == 128) return launch<128, 128, true, true>(*a, G, s);
+    if (a->head_dim == 192 && dv == 128) return launch<192, 128, true, true>(*a, G, s);
+    return 1;
+  }
+  if (dv != a->head_dim) return 1;
+  if (a->head_dim == 128) return ts ? launch<128, 128, true, false>(*a, G, s) : launch<128, 128, false, false>(*a, G, s);
+  if (a->head_dim == 64) return ts ? launch<64, 64, true, false>(*a, G, s) : launch<64, 64, false, false>(*a, G, s);
   return 1;
 }

@@ -280,7 +280,12 @@ static inline int kblk_of(const XpGemmArgs* a) { return a->fp8 ? 128 : gemm::kTi
 
 extern "C" int xp_gemm_plan(const XpGemmArgs* a, XpGemmPlan* plan) {
   const int kblk = a->fp8 ? 128 : gemm::kTileK;
-  if (a->n_out <= 0 || a->n_out % gemm::kTileM != 0 || a->k <= 0 || a->k % kblk != 0 || a->rows <= 0) return -10;
+  if (a->n_out <= 0 || a->k <= 0 || a->rows <= 0) return -10;
+  // plain bf16 problems may end in partial tiles (TMA fills them with zeros); the other forms address whole tiles
+  const bool whole = a->fp8 || a->dual || a->w_tiled || a->tile_table != nullptr;
+  if (whole && (a->n_out % gemm::kTileM != 0 || a->k % kblk != 0)) return -10;
+  const int batch = a->batch > 1 ? a->batch : 1;
+  if (batch > 1 && (whole || a->epilogue == gemm::kEpiResidual || a->bias != nullptr || a->x_group_rows < a->rows)) return -16;
   if (a->fp8 && (a->dual || a->w_tiled || a->tile_table != nullptr || a->w_scale == nullptr || a->x_scale == nullptr ||
                  a->ld_xscale % 4 != 0 || a->bn > gemm::kMaxBnF8))
     return -14;
@@ -291,10 +296,10 @@ extern "C" int xp_gemm_plan(const XpGemmArgs* a, XpGemmPlan* plan) {
     cudaDeviceGetAttribute(&sm_count_cache[dev], cudaDevAttrMultiProcessorCount, dev);
   int sms = a->num_sms > 0 ? a->num_sms : (dev < 64 ? sm_count_cache[dev] : 148);
   if (sms <= 0) sms = 148;
-  const int tm = a->n_out / gemm::kTileM;
-  const int kb = a->k / kblk;
+  const int tm = (a->n_out + gemm::kTileM - 1) / gemm::kTileM * batch;
+  const int kb = (a->k + kblk - 1) / kblk;
   if (a->bn > 0 && a->bn != 16 && a->bn != 32 && a->bn != 64 && a->bn != 128 && a->bn != 256) return -11;
-  int fixed_splits = a->splits;
+  int fixed_splits = batch > 1 ? 1 : a->splits;
   if (fixed_splits > kb) fixed_splits = kb;
   while (fixed_splits > 1 && (fixed_splits - 1) * ((kb + fixed_splits - 1) / fixed_splits) >= kb) --fixed_splits;
   const size_t ws_avail = (a->ws != nullptr && a->counters != nullptr) ? a->ws_bytes : 0;
@@ -348,7 +353,8 @@ extern "C" int xp_gemm(const XpGemmArgs* a) {
   if (rc != 0) return -20;
   {
     const int eb = a->fp8 ? 1 : 2;
-    rc = tmap::cache().get(&tx, a->x, a->rows, a->k, static_cast<uint64_t>(a->ldx > 0 ? a->ldx : a->k) * eb, plan.bn, eb);
+    const uint64_t x_rows = a->batch > 1 ? static_cast<uint64_t>(a->batch) * a->x_group_rows : a->rows;
+    rc = tmap::cache().get(&tx, a->x, x_rows, a->k, static_cast<uint64_t>(a->ldx > 0 ? a->ldx : a->k) * eb, plan.bn, eb);
   }
   if (rc != 0) return -21;
   if (a->fp8 && a->ld_xscale < (a->rows + plan.bn - 1) / plan.bn * plan.bn) return -15;  // scales padded to whole tiles
@@ -382,6 +388,10 @@ extern "C" int xp_gemm(const XpGemmArgs* a) {
   p.w_scale = a->w_scale;
   p.x_scale = a->x_scale;
   p.ld_xscale = a->ld_xscale;
+  p.batch = a->batch;
+  p.x_group_rows = a->x_group_rows;
+  p.out_group_stride = a->out_group_stride;
+  p.out_scale = a->out_scale;
   if (a->tile_table != nullptr) {
     if (plan.splits != 1) return -13;
     plan.grid = plan.smem_bytes > 0 ? 148 : 148;

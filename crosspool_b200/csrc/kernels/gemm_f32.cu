@@ -1,0 +1,66 @@
+// Plain fp32 matrix product y = x w^T (+ bias) for models served in 32-bit: FFMA only, no reduced-precision tensor mode.
+// One CTA computes a 64 x 64 tile from 16-deep slices staged in shared memory; a thread owns 4 x 4 outputs.
+#include <cuda_runtime.h>
+#include <stdint.h>
+
+#include "xpool/mixer_api.h"
+
+namespace {
+
+constexpr int kBM = 64, kBN = 64, kBK = 16;
+
+__global__ void __launch_bounds__(256)
+gemm_f32_kernel(const float* __restrict__ x, const float* __restrict__ w, const float* __restrict__ bias, float* __restrict__ out,
+                int rows, int n, int k, int ldx, int ldw, int ldo, int64_t sx, int64_t sw, int64_t so, float scale) {
+  __shared__ float xs[kBK][kBM + 4];
+  __shared__ float ws[kBK][kBN + 4];
+  x += blockIdx.z * sx;
+  w += blockIdx.z * sw;
+  out += blockIdx.z * so;
+  const int r0 = blockIdx.y * kBM, n0 = blockIdx.x * kBN;
+  const int tr = threadIdx.x >> 4, tc = threadIdx.x & 15;
+  float acc[4][4] = {};
+  for (int k0 = 0; k0 < k; k0 += kBK) {
+    for (int i = threadIdx.x; i < kBM * kBK; i += 256) {
+      const int kk = i & (kBK - 1), m = i / kBK;
+      const bool kin = k0 + kk < k;
+      xs[kk][m] = kin && r0 + m < rows ? x[static_cast<int64_t>(r0 + m) * ldx + k0 + kk] : 0.f;
+      ws[kk][m] = kin && n0 + m < n ? w[static_cast<int64_t>(n0 + m) * ldw + k0 + kk] : 0.f;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int kk = 0; kk < kBK; ++kk) {
+      float a[4], b[4];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) a[j] = xs[kk][tr * 4 + j], b[j] = ws[kk][tc * 4 + j];
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(a[i], b[j], acc[i][j]);
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const int r = r0 + tr * 4 + i;
+    if (r >= rows) continue;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int c = n0 + tc * 4 + j;
+      if (c < n) out[static_cast<int64_t>(r) * ldo + c] = fmaf(acc[i][j], scale, bias != nullptr ? bias[c] : 0.f);
+    }
+  }
+}
+
+}  // namespace
+
+extern "C" int xp_gemm_f32(const float* x, const float* w, const float* bias, float* out, int rows, int n, int k, int ldx, int ldw,
+                           int ldo, int batch, int64_t sx, int64_t sw, int64_t so, float out_scale, void* stream) {
+  if (rows <= 0 || n <= 0 || batch <= 0) return 0;
+  if (k <= 0) return -10;
+  dim3 grid((n + kBN - 1) / kBN, (rows + kBM - 1) / kBM, batch);
+  gemm_f32_kernel<<<grid, 256, 0, reinterpret_cast<cudaStream_t>(stream)>>>(x, w, bias, out, rows, n, k, ldx, ldw, ldo, sx, sw, so,
+                                                                           out_scale == 0.f ? 1.f : out_scale);
+  cudaError_t e = cudaGetLastError();
+  return e == cudaSuccess ? 0 : -100 - static_cast<int>(e);
+}

@@ -1,0 +1,491 @@
+// Latent attention over a paged cache of [latent | rotated shared key] rows: one cache row per token serves every head,
+// as key (all of it) and as value (its latent columns). Kernels:
+//   latent_prep       per token: latent RMS norm, rotary on the shared key part and on every query head, cache write,
+//                     query layouts of the two forms below
+//   latent_attn_tc    absorbed form (queries already multiplied into the latent space), one token row and up to 16 heads
+//                     per CTA, split over the sequence: cp.async ring of 64-token tiles, ldmatrix + mma.m16n8k16, the
+//                     probabilities carried as a bf16 pair (high and low part). Bound by reading the cache once.
+//   latent_attn_simt  the same in plain FMAs for any sizes and for fp32
+//   latent_gather     dense copy of a sequence's cached rows, the input of the expanded form (keys and values per head,
+//                     chunked prefill on the tcgen05 kernel of attn_prefill_umma.cu)
+//
+// mma.sync rather than tcgen05 in the absorbed decode kernel: 16 query rows per cache row are 4 * 16 flop per loaded
+// element, far below the tensor roofline, and a UMMA tile needs 64 or 128 query rows.
+#include <math_constants.h>
+
+#include "xpool/elem.cuh"
+#include "xpool/mixer_api.h"
+#include "xpool/sm100.cuh"
+
+namespace xpool {
+namespace latent {
+
+constexpr float kLog2e = 1.4426950408889634f;
+
+// ------------------------------------------------------------------------------------------ prep
+constexpr int kPrepThreads = 256;
+
+template <typename T>
+__global__ void __launch_bounds__(kPrepThreads)
+latent_prep_kernel(XpLatentPrepArgs a) {
+  extern __shared__ float cs[];            // cos | sin, rot_dims / 2 each
+  __shared__ float red[kPrepThreads / 32];
+  const int row = blockIdx.x;
+  const int half = a.rot_dims / 2;
+  const T* proj = reinterpret_cast<const T*>(a.proj) + static_cast<size_t>(row) * a.ld_proj;
+  const double pos = static_cast<double>(a.positions[row]);
+  for (int i = threadIdx.x; i < half; i += kPrepThreads) {
+    // the angle is reduced to one turn in double, so its fp32 sine and cosine are exact to fp32 at any position
+    const double turns = pos * a.freq[i] * 0.15915494309189535;
+    float s, c;
+    sincospif(2.f * static_cast<float>(turns - rint(turns)), &s, &c);
+    cs[i] = c;
+    cs[half + i] = s;
+  }
+  __syncthreads();
+  // element j of a vector x whose first rot_dims elements are rotated in pairs (j, j + half)
+  auto rotated = [&](const T* x, int j) -> float {
+    const float v = elem::ld(x + j);
+    if (j >= a.rot_dims) return v;
+    const int i = j < half ? j : j - half;
+    const float o = elem::ld(x + (j < half ? j + half : i));
+    return j < half ? v * cs[i] - o * cs[half + i] : v * cs[i] + o * cs[half + i];
+  };
+
+  const int slot = a.slots[row];
+  if (slot >= 0) {
+    const T* kv = proj + a.kv_off;
+    float ss = 0.f;
+    for (int c = threadIdx.x; c < a.kv_rank; c += kPrepThreads) {
+      const float v = elem::ld(kv + c);
+      ss += v * v;
+    }
+    const float inv = rsqrtf(elem::block_sum<kPrepThreads>(ss, red) / static_cast<float>(a.kv_rank) + a.eps);
+    T* dst = reinterpret_cast<T*>(a.cache) + static_cast<size_t>(slot) * a.ld_cache;
+    for (int c = threadIdx.x; c < a.ld_cache; c += kPrepThreads) {
+      float v = 0.f;                        // the pitch's padding columns hold zeros
+      if (c < a.kv_rank) v = elem::ld(kv + c) * inv * a.norm_w[c];
+      else if (c < a.kv_rank + a.rot) v = rotated(kv + a.kv_rank, c - a.kv_rank);
+      elem::st(dst + c, v);
+    }
+  }
+
+  const int dh = a.dim + a.rot;
+  const T* q = proj + a.q_off;
+  if (row < a.abs_rows) {
+    T* qp = reinterpret_cast<T*>(a.q_plain);
+    for (int i = threadIdx.x; i < a.heads * a.dim_p; i += kPrepThreads) {
+      const int h = i / a.dim_p, c = i - h * a.dim_p;
+      elem::st(qp + (static_cast<size_t>(h) * a.qp_rows + row) * a.dim_p + c, c < a.dim ? elem::ld(q + h * dh + c) : 0.f);
+    }
+    T* qa = reinterpret_cast<T*>(a.q_abs);
+    const int tail = a.ld_abs - a.kv_rank;
+    for (int i = threadIdx.x; i < a.heads * tail; i += kPrepThreads) {
+      const int h = i / tail, c = i - h * tail;
+      elem::st(qa + (static_cast<size_t>(h) * a.qp_rows + row) * a.ld_abs + a.kv_rank + c, c < a.rot ? rotated(q + h * dh + a.dim, c) : 0.f);
+    }
+  } else {
+    T* qe = reinterpret_cast<T*>(a.q_exp) + static_cast<size_t>(row) * a.heads * a.dq_pad;
+    for (int i = threadIdx.x; i < a.heads * a.dq_pad; i += kPrepThreads) {
+      const int h = i / a.dq_pad, c = i - h * a.dq_pad;
+      float v = 0.f;
+      if (c < a.dim) v = elem::ld(q + h * dh + c);
+      else if (c < dh) v = rotated(q + h * dh + a.dim, c - a.dim);
+      elem::st(qe + i, v);
+    }
+  }
+}
+
+// ------------------------------------------------------------------------------------------ plain kernel
+constexpr int kSimtThreads = 128;
+constexpr int kSimtTile = 32;
+constexpr int kSimtAcc = 8;              // latent columns per thread: kv_rank <= 1024
+
+template <typename T>
+__global__ void __launch_bounds__(kSimtThreads)
+latent_attn_simt_kernel(XpLatentAttnArgs a) {
+  extern __shared__ float q_s[];         // kv_rank + rot
+  __shared__ float sc[kSimtTile];
+  const int h = blockIdx.x, row = blockIdx.y;
+  const int dk = a.kv_rank + a.rot;
+  T* out = reinterpret_cast<T*>(a.out) + (static_cast<size_t>(h) * a.q_rows + row) * a.ld_out;
+  if (a.slots[row] < 0) {
+    for (int c = threadIdx.x; c < a.kv_rank; c += kSimtThreads) elem::st(out + c, 0.f);
+    return;
+  }
+  const T* q = reinterpret_cast<const T*>(a.q) + (static_cast<size_t>(h) * a.q_rows + row) * a.ld_q;
+  for (int c = threadIdx.x; c < dk; c += kSimtThreads) q_s[c] = elem::ld(q + c) * a.scale * kLog2e;
+  __syncthreads();
+  const int* table = a.block_table + static_cast<size_t>(a.row_seq != nullptr ? a.row_seq[row] : row) * a.max_blocks;
+  const T* cache = reinterpret_cast<const T*>(a.cache);
+  const int len = a.positions[row] + 1;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  auto token_row = [&](int t) {
+    return cache + (static_cast<size_t>(table[t / a.page_size]) * a.page_size + t % a.page_size) * a.ld_cache;
+  };
+  float m = -CUDART_INF_F, l = 0.f, acc[kSimtAcc];
+#pragma unroll
+  for (int j = 0; j < kSimtAcc; ++j) acc[j] = 0.f;
+  for (int t0 = 0; t0 < len; t0 += kSimtTile) {
+    const int n = min(kSimtTile, len - t0);
+    for (int j = warp; j < n; j += kSimtThreads / 32) {
+      const T* k = token_row(t0 + j);
+      float s = 0.f;
+      for (int c = lane; c < dk; c += 32) s = fmaf(q_s[c], elem::ld(k + c), s);
+      s = elem::warp_sum(s);
+      if (lane == 0) sc[j] = s;
+    }
+    __syncthreads();
+    float mn = m;
+    for (int j = 0; j < n; ++j) mn = fmaxf(mn, sc[j]);
+    const float f = exp2f(m - mn);       // 0 on the first tile (m = -inf)
+    m = mn;
+    l *= f;
+#pragma unroll
+    for (int j = 0; j < kSimtAcc; ++j) acc[j] *= f;
+    for (int j = 0; j < n; ++j) {
+      const float p = exp2f(sc[j] - m);
+      l += p;
+      const T* v = token_row(t0 + j);
+#pragma unroll
+      for (int u = 0; u < kSimtAcc; ++u) {
+        const int c = threadIdx.x + u * kSimtThreads;
+        if (c < a.kv_rank) acc[u] = fmaf(p, elem::ld(v + c), acc[u]);
+      }
+    }
+    __syncthreads();
+  }
+  float g = 1.f / l;
+  if (a.gate != nullptr) g *= elem::sigmoid(elem::ld(reinterpret_cast<const T*>(a.gate) + static_cast<size_t>(row) * a.ld_gate + h));
+#pragma unroll
+  for (int u = 0; u < kSimtAcc; ++u) {
+    const int c = threadIdx.x + u * kSimtThreads;
+    if (c < a.kv_rank) elem::st(out + c, acc[u] * g);
+  }
+}
+
+// ------------------------------------------------------------------------------------------ tensor-core kernel
+constexpr int kTcThreads = 256;          // 8 warps: 4 token groups x 2 halves of the key columns, then 8 column groups
+constexpr int kTile = 64;                // tokens per tile
+constexpr int kPPitch = kTile + 8;
+
+__device__ __forceinline__ void ldsm_x4(uint32_t addr, uint32_t (&r)[4]) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
+               : "r"(addr));
+}
+__device__ __forceinline__ void ldsm_x4_trans(uint32_t addr, uint32_t (&r)[4]) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
+               : "r"(addr));
+}
+__device__ __forceinline__ void mma16816(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile(
+      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+
+struct TcLayout {
+  int pitch;        // elements of one shared-memory row (an odd multiple of 16 bytes: conflict-free ldmatrix)
+  int stage_bytes;
+  int q_bytes;
+  int stages;
+  int total;
+};
+
+__host__ __device__ inline TcLayout tc_layout(int dk16, int vcols) {
+  TcLayout L;
+  const int w = dk16 > vcols ? dk16 : vcols;
+  L.pitch = w + 8;
+  L.stage_bytes = kTile * L.pitch * 2;
+  L.q_bytes = 16 * L.pitch * 2;
+  const int fixed = L.q_bytes + 2 * 16 * kPPitch * 2 + 2 * 16 * kTile * 4 + 3 * 16 * 4;
+  int st = (100 * 1024 - fixed) / L.stage_bytes;     // two CTAs per SM when the rows are short
+  if (st < 2) st = 2;
+  if (st > 4) st = 4;
+  L.stages = st;
+  L.total = fixed + st * L.stage_bytes;
+  return L;
+}
+
+// NT: 8-column tiles of the latent per warp (kv_rank <= 64 * NT).
+template <int NT>
+__global__ void __launch_bounds__(kTcThreads)
+latent_attn_tc_kernel(XpLatentAttnArgs a) {
+  extern __shared__ __align__(16) uint8_t smem[];
+  const int split = blockIdx.x, h0 = blockIdx.y * 16, row = blockIdx.z;
+  const int nh = min(16, a.heads - h0);
+  const int dk16 = a.ld_cache;
+  const TcLayout L = tc_layout(dk16, 64 * NT);
+  __nv_bfloat16* q_s = reinterpret_cast<__nv_bfloat16*>(smem);
+  __nv_bfloat16* p_s = reinterpret_cast<__nv_bfloat16*>(smem + L.q_bytes);            // high parts, then low parts
+  float* s_s = reinterpret_cast<float*>(smem + L.q_bytes + 2 * 16 * kPPitch * 2);     // [2][16][kTile]
+  float* m_s = s_s + 2 * 16 * kTile;                                                   // running maximum, sum, factor
+  float* l_s = m_s + 16;
+  float* f_s = l_s + 16;
+  uint8_t* ring = smem + L.total - L.stages * L.stage_bytes;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const bool pad = a.slots[row] < 0;
+  const int len = pad ? 0 : a.positions[row] + 1;
+  int chunk = a.chunk_tokens > 0 ? a.chunk_tokens : len;
+  const int t0 = split * chunk, t1 = a.num_splits > 1 ? min(len, t0 + chunk) : len;
+  if (a.num_splits > 1 && t0 >= len) return;         // the merge kernel skips this slice
+  const int tiles = (t1 - t0 + kTile - 1) / kTile;
+  const int* table = a.block_table + static_cast<size_t>(a.row_seq != nullptr ? a.row_seq[row] : row) * a.max_blocks;
+  const __nv_bfloat16* cache = reinterpret_cast<const __nv_bfloat16*>(a.cache);
+  const int chunks_row = dk16 / 8;                   // 16-byte pieces of a row
+
+  auto issue = [&](int it) {
+    if (it < tiles) {
+      uint8_t* st = ring + (it % L.stages) * L.stage_bytes;
+      // four threads walk one token row: the page lookup is shared by its pieces
+      const int tok = threadIdx.x >> 2;
+      const int t = t0 + it * kTile + tok;
+      const bool ok = t < t1;
+      const int tt = ok ? t : t0;
+      const __nv_bfloat16* src = cache + (static_cast<size_t>(table[tt / a.page_size]) * a.page_size + tt % a.page_size) * dk16;
+      const uint32_t dst = sm100::smem_u32(st + tok * L.pitch * 2);
+      const int sz = ok ? 16 : 0;                    // rows past the slice read as zero
+      for (int c = threadIdx.x & 3; c < chunks_row; c += 4)
+        asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst + c * 16), "l"(src + c * 8), "r"(sz));
+    }
+    asm volatile("cp.async.commit_group;");
+  };
+  for (int i = 0; i < L.stages - 1; ++i) issue(i);
+
+  // queries of the head group; absent heads and the pitch's padding columns read as zero
+  for (int i = threadIdx.x; i < 16 * (dk16 / 8); i += kTcThreads) {
+    const int h = i / (dk16 / 8), c = (i - h * (dk16 / 8)) * 8;
+    uint4 v = make_uint4(0, 0, 0, 0);
+    if (h < nh)
+      v = *reinterpret_cast<const uint4*>(reinterpret_cast<const __nv_bfloat16*>(a.q) +
+                                          (static_cast<size_t>(h0 + h) * a.q_rows + row) * a.ld_q + c);
+    *reinterpret_cast<uint4*>(q_s + h * L.pitch + c) = v;
+  }
+  if (threadIdx.x < 16) {
+    m_s[threadIdx.x] = -CUDART_INF_F;
+    l_s[threadIdx.x] = 0.f;
+  }
+  const float qscale = a.scale * kLog2e;
+  const int tg = warp & 3, kh = warp >> 2;           // token group (16 tokens), half of the key columns
+  const int ksteps = dk16 / 16, ks0 = kh ? (ksteps + 1) / 2 : 0, ks1 = kh ? ksteps : (ksteps + 1) / 2;
+  const int g = lane >> 2, q4 = lane & 3;
+  const uint32_t q_addr = sm100::smem_u32(q_s) + ((lane & 15) * L.pitch + (lane >> 4) * 8) * 2;
+  const uint32_t k_lane = ((tg * 16 + (lane & 7) + ((lane >> 4) << 3)) * L.pitch + ((lane >> 3) & 1) * 8) * 2;
+  const uint32_t p_addr = sm100::smem_u32(p_s) + ((lane & 15) * kPPitch + (lane >> 4) * 8) * 2;
+  const uint32_t v_lane = (((lane & 7) + ((lane >> 3) & 1) * 8) * L.pitch + warp * NT * 8 + (lane >> 4) * 8) * 2;
+  float acc[NT][4];
+#pragma unroll
+  for (int j = 0; j < NT; ++j)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) acc[j][e] = 0.f;
+
+  for (int it = 0; it < tiles; ++it) {
+    if (L.stages == 2) asm volatile("cp.async.wait_group 0;" ::: "memory");
+    else if (L.stages == 3) asm volatile("cp.async.wait_group 1;" ::: "memory");
+    else asm volatile("cp.async.wait_group 2;" ::: "memory");
+    __syncthreads();                                 // tile it landed; everyone is done with the tile before it
+    issue(it + L.stages - 1);
+    const uint32_t st = sm100::smem_u32(ring + (it % L.stages) * L.stage_bytes);
+    // scores of 16 tokens over this warp's half of the columns
+    float s0[4] = {0.f, 0.f, 0.f, 0.f}, s1[4] = {0.f, 0.f, 0.f, 0.f};
+    for (int ks = ks0; ks < ks1; ++ks) {
+      uint32_t qa[4], kb[4];
+      ldsm_x4(q_addr + ks * 32, qa);
+      ldsm_x4(st + k_lane + ks * 32, kb);
+      mma16816(s0, qa, kb[0], kb[1]);
+      mma16816(s1, qa, kb[2], kb[3]);
+    }
+    float* sp = s_s + kh * 16 * kTile + tg * 16 + q4 * 2;
+    *reinterpret_cast<float2*>(sp + g * kTile) = make_float2(s0[0], s0[1]);
+    *reinterpret_cast<float2*>(sp + (g + 8) * kTile) = make_float2(s0[2], s0[3]);
+    *reinterpret_cast<float2*>(sp + g * kTile + 8) = make_float2(s1[0], s1[1]);
+    *reinterpret_cast<float2*>(sp + (g + 8) * kTile + 8) = make_float2(s1[2], s1[3]);
+    __syncthreads();
+    // softmax: two heads per warp, two tokens per lane
+    const int tok0 = t0 + it * kTile + lane * 2;
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      const int h = warp * 2 + r;
+      const float2 x = *reinterpret_cast<const float2*>(s_s + h * kTile + lane * 2);
+      const float2 y = *reinterpret_cast<const float2*>(s_s + 16 * kTile + h * kTile + lane * 2);
+      const float v0 = tok0 < t1 ? (x.x + y.x) * qscale : -CUDART_INF_F;
+      const float v1 = tok0 + 1 < t1 ? (x.y + y.y) * qscale : -CUDART_INF_F;
+      float mx = fmaxf(v0, v1);
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+      const float m_old = m_s[h], m_new = fmaxf(m_old, mx);
+      const float p0 = exp2f(v0 - m_new), p1 = exp2f(v1 - m_new);
+      const float sum = elem::warp_sum(p0 + p1);
+      const __nv_bfloat162 hi = __floats2bfloat162_rn(p0, p1);
+      const float2 hf = __bfloat1622float2(hi);
+      *reinterpret_cast<__nv_bfloat162*>(p_s + h * kPPitch + lane * 2) = hi;
+      *reinterpret_cast<__nv_bfloat162*>(p_s + (16 + h) * kPPitch + lane * 2) = __floats2bfloat162_rn(p0 - hf.x, p1 - hf.y);
+      __syncwarp();
+      if (lane == 0) {
+        const float f = exp2f(m_old - m_new);
+        f_s[h] = f;
+        m_s[h] = m_new;
+        l_s[h] = l_s[h] * f + sum;
+      }
+    }
+    __syncthreads();
+    const float fa = f_s[g], fb = f_s[g + 8];
+#pragma unroll
+    for (int j = 0; j < NT; ++j) acc[j][0] *= fa, acc[j][1] *= fa, acc[j][2] *= fb, acc[j][3] *= fb;
+#pragma unroll
+    for (int kk = 0; kk < kTile / 16; ++kk) {
+      uint32_t ph[4], pl[4];
+      ldsm_x4(p_addr + kk * 32, ph);
+      ldsm_x4(p_addr + 16 * kPPitch * 2 + kk * 32, pl);
+#pragma unroll
+      for (int j = 0; j < NT; j += 2) {
+        uint32_t vb[4];
+        ldsm_x4_trans(st + v_lane + kk * 16 * L.pitch * 2 + j * 16, vb);
+        mma16816(acc[j], ph, vb[0], vb[1]);
+        mma16816(acc[j + 1], ph, vb[2], vb[3]);
+        mma16816(acc[j], pl, vb[0], vb[1]);
+        mma16816(acc[j + 1], pl, vb[2], vb[3]);
+      }
+    }
+  }
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
+  __syncthreads();
+#pragma unroll
+  for (int e = 0; e < 2; ++e) {
+    const int h = g + e * 8;
+    if (h >= nh) continue;
+    if (a.num_splits > 1) {
+      float* w = a.ws + ((static_cast<size_t>(row) * a.heads + h0 + h) * a.num_splits + split) * (a.kv_rank + 2);
+      for (int j = 0; j < NT; ++j) {
+        const int c = (warp * NT + j) * 8 + q4 * 2;
+#pragma unroll
+        for (int u = 0; u < 2; ++u)
+          if (c + u < a.kv_rank) w[c + u] = acc[j][e * 2 + u];
+      }
+      if (warp == 0 && q4 == 0) {
+        w[a.kv_rank] = m_s[h];
+        w[a.kv_rank + 1] = l_s[h];
+      }
+    } else {
+      float f = pad ? 0.f : 1.f / l_s[h];
+      if (a.gate != nullptr)
+        f *= elem::sigmoid(elem::ld(reinterpret_cast<const __nv_bfloat16*>(a.gate) + static_cast<size_t>(row) * a.ld_gate + h0 + h));
+      __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(a.out) + (static_cast<size_t>(h0 + h) * a.q_rows + row) * a.ld_out;
+      for (int j = 0; j < NT; ++j) {
+        const int c = (warp * NT + j) * 8 + q4 * 2;
+        if (c + 1 < a.kv_rank && a.ld_out % 2 == 0)
+          *reinterpret_cast<__nv_bfloat162*>(out + c) = __floats2bfloat162_rn(acc[j][e * 2] * f, acc[j][e * 2 + 1] * f);
+        else
+          for (int u = 0; u < 2; ++u)
+            if (c + u < a.kv_rank) out[c + u] = __float2bfloat16_rn(acc[j][e * 2 + u] * f);
+      }
+    }
+  }
+}
+
+// One CTA per (head, row): folds the slices in order.
+__global__ void __launch_bounds__(128)
+latent_merge_kernel(XpLatentAttnArgs a) {
+  const int h = blockIdx.x, row = blockIdx.y;
+  const bool pad = a.slots[row] < 0;
+  const int len = pad ? 0 : a.positions[row] + 1;
+  const int n = min(a.num_splits, (len + a.chunk_tokens - 1) / a.chunk_tokens);
+  const float* w = a.ws + (static_cast<size_t>(row) * a.heads + h) * a.num_splits * (a.kv_rank + 2);
+  float m = -CUDART_INF_F, l = 0.f;
+  for (int s = 0; s < n; ++s) m = fmaxf(m, w[s * (a.kv_rank + 2) + a.kv_rank]);
+  for (int s = 0; s < n; ++s) l += w[s * (a.kv_rank + 2) + a.kv_rank + 1] * exp2f(w[s * (a.kv_rank + 2) + a.kv_rank] - m);
+  float f = pad ? 0.f : 1.f / l;
+  if (a.gate != nullptr)
+    f *= elem::sigmoid(elem::ld(reinterpret_cast<const __nv_bfloat16*>(a.gate) + static_cast<size_t>(row) * a.ld_gate + h));
+  __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(a.out) + (static_cast<size_t>(h) * a.q_rows + row) * a.ld_out;
+  for (int c = threadIdx.x; c < a.kv_rank; c += 128) {
+    float v = 0.f;
+    for (int s = 0; s < n; ++s) v += w[s * (a.kv_rank + 2) + c] * exp2f(w[s * (a.kv_rank + 2) + a.kv_rank] - m);
+    out[c] = __float2bfloat16_rn(v * f);
+  }
+}
+
+// ------------------------------------------------------------------------------------------ gather
+__global__ void __launch_bounds__(128)
+latent_gather_kernel(XpLatentGatherArgs a) {
+  const int seq = blockIdx.y;
+  const int len = a.ctx_lens[seq] + a.q_lens[seq];
+  const int row_bytes = a.ld_cache * a.elem_bytes;   // a multiple of 16
+  const int* table = a.block_table + static_cast<size_t>(seq) * a.max_blocks;
+  const uint8_t* cache = static_cast<const uint8_t*>(a.cache);
+  uint8_t* out = static_cast<uint8_t*>(a.out) + static_cast<size_t>(a.starts[seq]) * row_bytes;
+  const int per = row_bytes / 16;
+  const int t0 = blockIdx.x * 16, n = min(16, len - t0);
+  for (int u = threadIdx.x; u < n * per; u += 128) {
+    const int t = t0 + u / per, c = u % per;
+    const size_t src = (static_cast<size_t>(table[t / a.page_size]) * a.page_size + t % a.page_size) * row_bytes;
+    *reinterpret_cast<uint4*>(out + static_cast<size_t>(t) * row_bytes + c * 16) =
+        __ldg(reinterpret_cast<const uint4*>(cache + src + c * 16));
+  }
+}
+
+inline int done() {
+  cudaError_t e = cudaGetLastError();
+  return e == cudaSuccess ? 0 : -100 - static_cast<int>(e);
+}
+
+template <int NT>
+int launch_tc(const XpLatentAttnArgs& a, cudaStream_t s) {
+  const TcLayout L = tc_layout(a.ld_cache, 64 * NT);
+  if (L.total > 227 * 1024) return 1;
+  static bool set = false;
+  if (!set) {
+    if (cudaFuncSetAttribute(latent_attn_tc_kernel<NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024) != cudaSuccess) return -21;
+    set = true;
+  }
+  dim3 grid(a.num_splits > 1 ? a.num_splits : 1, (a.heads + 15) / 16, a.rows);
+  latent_attn_tc_kernel<NT><<<grid, kTcThreads, L.total, s>>>(a);
+  if (a.num_splits > 1) latent_merge_kernel<<<dim3(a.heads, a.rows), 128, 0, s>>>(a);
+  return done();
+}
+
+}  // namespace latent
+}  // namespace xpool
+
+using namespace xpool::latent;
+
+extern "C" int xp_latent_prep(const XpLatentPrepArgs* a, void* stream) {
+  if (a->rows <= 0) return 0;
+  if (a->rot_dims % 2 != 0 || a->rot_dims > a->rot || a->rot_dims > 2048 || a->ld_cache < a->kv_rank + a->rot) return -10;
+  if (a->abs_rows > 0 && (a->q_plain == nullptr || a->q_abs == nullptr || a->ld_abs < a->kv_rank + a->rot || a->abs_rows > a->qp_rows ||
+                          a->dim_p < a->dim))
+    return -11;
+  if (a->abs_rows < a->rows && (a->q_exp == nullptr || a->dq_pad < a->dim + a->rot)) return -12;
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  const size_t sm = static_cast<size_t>(a->rot_dims > 0 ? a->rot_dims : 1) * 4;
+  if (a->f32) latent_prep_kernel<float><<<a->rows, kPrepThreads, sm, s>>>(*a);
+  else latent_prep_kernel<__nv_bfloat16><<<a->rows, kPrepThreads, sm, s>>>(*a);
+  return done();
+}
+
+extern "C" int xp_latent_attn(const XpLatentAttnArgs* a, void* stream) {
+  if (a->rows <= 0) return 0;
+  if (a->heads <= 0 || a->kv_rank <= 0 || a->page_size <= 0 || a->rows > a->q_rows || a->ld_q < a->kv_rank + a->rot) return -10;
+  if (a->num_splits > 1 && (a->ws == nullptr || a->chunk_tokens <= 0)) return -11;
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  if (!a->f32 && !a->force_simt && a->kv_rank <= 512 && a->ld_cache % 16 == 0 && a->ld_q % 8 == 0 && a->ld_q >= a->ld_cache) {
+    int rc = a->kv_rank <= 128 ? launch_tc<2>(*a, s) : a->kv_rank <= 256 ? launch_tc<4>(*a, s) : launch_tc<8>(*a, s);
+    if (rc <= 0) return rc;
+  }
+  if (a->kv_rank > kSimtAcc * kSimtThreads || a->kv_rank + a->rot > 12000) return -12;
+  dim3 grid(a->heads, a->rows);
+  const size_t sm = static_cast<size_t>(a->kv_rank + a->rot) * 4;
+  if (a->f32) latent_attn_simt_kernel<float><<<grid, kSimtThreads, sm, s>>>(*a);
+  else latent_attn_simt_kernel<__nv_bfloat16><<<grid, kSimtThreads, sm, s>>>(*a);
+  return done();
+}
+
+extern "C" int xp_latent_gather(const XpLatentGatherArgs* a, void* stream) {
+  if (a->n_seqs <= 0 || a->max_len <= 0) return 0;
+  if ((a->ld_cache * a->elem_bytes) % 16 != 0) return -10;
+  dim3 grid((a->max_len + 15) / 16, a->n_seqs);
+  latent_gather_kernel<<<grid, 128, 0, reinterpret_cast<cudaStream_t>(stream)>>>(*a);
+  return done();
+}

@@ -13,8 +13,10 @@ overlap on the GPU(s): while one model's step waits for its FFN, another model's
 
 from __future__ import annotations
 
+import json
 import time
 from dataclasses import dataclass, field
+from pathlib import Path
 
 import torch
 
@@ -22,7 +24,8 @@ from .engine.atn_engine import AttentionEngine, EngineConfig, Sequence
 from .engine.ffn_local import LocalFfnPort
 from .models import config as model_config
 from .models.config import ModelConfig
-from .models.weights import random_attention_weights, random_ffn_weights
+from .models.weights import load_attention_from_safetensors, random_attention_weights, random_ffn_weights
+from .utils.dtype import decode_dtype
 
 
 @dataclass
@@ -128,19 +131,47 @@ class Deployment:
         return out
 
 
+def has_checkpoint(preset) -> bool:
+    if isinstance(preset, ModelConfig):
+        return False
+    p = Path(preset)
+    return p.is_dir() and (p / "config.json").exists() and any(p.glob("*.safetensors"))
+
+
+def load_ffn_weights(cfg: ModelConfig, model_dir, device, dtype: torch.dtype) -> list:
+    """Every layer's whole FFN from a checkpoint directory (None where a layered decoder has none), after checking that
+    its tensors are exactly those the architecture's FFN description names."""
+    from .engine import loader
+    from .engine.checkpoint import read_checkpoint_key_view, validate_ffn_coverage
+    from .models.adapters import compile_ffn_spec
+
+    view = read_checkpoint_key_view(model_dir)
+    spec = compile_ffn_spec(cfg.name, json.loads((Path(model_dir) / "config.json").read_text()), view.keys())
+    validate_ffn_coverage(spec, view)
+    have = {l.layer for l in spec.layers}
+    return [loader.materialize_layer_weights(spec, view, i, device=device, dtype=dtype) if i in have else None
+            for i in range(cfg.num_layers)]
+
+
 def build_loopback(models: list[tuple[str, str | ModelConfig, int]], ecfg: EngineConfig | None = None,
                    device: str | torch.device = "cuda", tile_weights: bool = False) -> Deployment:
-    """``models`` = [(instance id, preset name or ModelConfig, seed)]; random-init weights."""
+    """``models`` = [(instance id, preset name, checkpoint directory or ModelConfig, seed)]; a directory with safetensors
+    files is loaded, everything else gets random-init weights."""
     from .ops import gemm
 
     handles = []
+    dtype = decode_dtype((ecfg or EngineConfig()).dtype)
     for model_id, preset, seed in models:
         cfg = preset if isinstance(preset, ModelConfig) else model_config.load(preset)
-        aw = random_attention_weights(cfg, seed, device, torch.bfloat16)
-        fw = random_ffn_weights(cfg, seed, device, torch.bfloat16)
+        if has_checkpoint(preset):
+            aw = load_attention_from_safetensors(cfg, preset, device, dtype)
+            fw = load_ffn_weights(cfg, preset, device, dtype)
+        else:
+            aw = random_attention_weights(cfg, seed, device, dtype)
+            fw = random_ffn_weights(cfg, seed, device, dtype)
         if tile_weights:
             for l in fw:
-                if not l.is_moe:
+                if l is not None and not l.is_moe and not cfg.layered:
                     l.gate_up, l.down = gemm.tile_weight(l.gate_up), gemm.tile_weight(l.down)
         eng = AttentionEngine(cfg, aw, LocalFfnPort(cfg, fw), ecfg, device)
         handles.append(InstanceHandle(model_id, cfg, eng))

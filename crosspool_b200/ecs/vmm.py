@@ -173,6 +173,8 @@ def elastic_kv_cache(cfg: ModelConfig, max_pages: int, page_size: int, device, d
     fewer driver calls per byte at the price of coarser lending."""
     from ..parallel.fabric import tensor_from_ptr
 
+    if cfg.layered:
+        raise NotImplementedError("elastic KV lends bundles of equal per-layer buffers; layered decoders run on a fixed pool")
     dev_index = torch.device(device).index or 0
     ppb, chunk = bundle_geometry(cfg, page_size, granularity)
     n_bundles = (max_pages + ppb - 1) // ppb

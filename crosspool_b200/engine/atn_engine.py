@@ -25,6 +25,7 @@ from ..models.weights import AttentionWeights
 from ..ops import attention as A
 from ..ops import gemm, norm
 from ..utils import nvtx
+from ..utils.dtype import decode_dtype
 from .kv_cache import OutOfPages, PagedKvCache
 
 MODE_PREFILL, MODE_DECODE = 1, 2
@@ -55,6 +56,8 @@ class EngineConfig:
     use_cuda_graph: bool = True
     decode_buckets: list[int] | None = None
     prefix_cache: bool = False  # keep full prompt pages and share them with later requests
+    dtype: str = "bfloat16"     # activations, weights and cache; "float32" (layered decoders only) runs true 32-bit products
+    mixed_batches: bool = False  # a prefill chunk takes the running sequences' next tokens along in the same forward pass
     sampling: bool = False      # per-request temperature sampling (Gumbel-max kernel) instead of greedy argmax
 
 
@@ -141,23 +144,34 @@ class AttentionEngine:
                 f"{cfg.architecture}: this engine runs rotary grouped-query attention with RMSNorm; LayerNorm with learned "
                 "positions, sliding windows, attention sinks, scaled rotary embeddings and latent attention run in the "
                 "PyTorch oracle and the CPU deployment only (engine/cpu_plumbing.py). The FFN tier serves this architecture.")
+        e = ecfg or EngineConfig()
+        if cfg.layered:
+            if tp is not None or type(port).publish_targets is not FfnPort.publish_targets:
+                raise UnsupportedAttention(f"{cfg.architecture}: layered decoders run their FFNs in-stream (LocalFfnPort), without attention TP")
+            if e.prefix_cache and cfg.recurrent:
+                raise ValueError("prefix sharing needs a cache of pages; this model carries a recurrent state per sequence")
+        elif e.dtype != "bfloat16":
+            raise ValueError(f"{cfg.architecture} runs in bfloat16 on the GPU engine")
         self.cfg, self.w, self.port = cfg, weights, port
         self.tp = tp
-        self.ecfg = ecfg or EngineConfig()
+        self.ecfg = e
         self.device = torch.device(device)
-        e = self.ecfg
+        self.dtype = decode_dtype(e.dtype)
         self.max_blocks = (e.max_seq_len + e.page_size - 1) // e.page_size
         if kv is None:
             pages = e.num_pages or e.max_batch * self.max_blocks
-            kv = PagedKvCache.fixed(cfg, pages, e.page_size, self.device)
+            kv = PagedKvCache.fixed(cfg, pages, e.page_size, self.device, self.dtype, state_slots=e.max_batch)
         self.kv = kv
         self.cap = max(e.max_batch, e.prefill_chunk)
+        # sequences of one ragged pass: portions of prompts and, in mixed batches, every running sequence
+        self.max_seqs = e.max_prefill_seqs + (e.max_batch if e.mixed_batches else 0)
+        self._buckets = e.decode_buckets or capacity_buckets(e.max_batch)
+        self.body = None              # layered decoders: engine/layered.py
         self._alloc_buffers()
         self.waiting: deque[Sequence] = deque()
         self.running: list[Sequence] = []
         self.prefilling: list[Sequence] = []
         self._graphs: dict[int, torch.cuda.CUDAGraph] = {}
-        self._buckets = e.decode_buckets or capacity_buckets(e.max_batch)
         self._next_id = 0
         self._last_was_prefill = False
         self.stats = {"prefill_steps": 0, "decode_steps": 0, "h2d_bytes": 0, "d2h_bytes": 0, "launches": 0}
@@ -168,6 +182,7 @@ class AttentionEngine:
         self._inflight = None
         self._pending: list[tuple[Sequence, int]] | None = None
         self._pre_inflight: list[tuple[Sequence, int]] | None = None
+        self._riding: list[Sequence] = []     # running sequences in the prefill chunk in flight
         self._step_event = torch.cuda.Event() if torch.cuda.is_available() else None
         self._graph_launches: dict[int, int] = {}
         self.prefix = None
@@ -234,6 +249,16 @@ class AttentionEngine:
         cfg, e, dev = self.cfg, self.ecfg, self.device
         bf = torch.bfloat16
         cap, B = self.cap, e.max_batch
+        self._alloc_metadata()
+        if cfg.layered:
+            from .layered import LayeredForward
+
+            n = max(B, self.max_seqs)
+            self.body = LayeredForward(self)
+            h8 = (cfg.hidden_size + 7) // 8 * 8
+            self.sel = torch.zeros(n, h8, dtype=self.dtype, device=dev)[:, :cfg.hidden_size]
+            self.logits = torch.zeros(n, cfg.vocab_size, dtype=torch.float32, device=dev)
+            return
         self.resid = torch.zeros(cap, cfg.hidden_size, dtype=bf, device=dev)
         self.x = torch.zeros(cap, cfg.hidden_size, dtype=bf, device=dev)
         self.x2 = torch.zeros(cap, cfg.hidden_size, dtype=bf, device=dev)
@@ -241,27 +266,31 @@ class AttentionEngine:
         self.q = torch.zeros(cap, cfg.num_q_heads, cfg.head_dim, dtype=bf, device=dev)
         self.attn_out = torch.zeros(cap, cfg.num_q_heads, cfg.head_dim, dtype=bf, device=dev)
         self.o = torch.zeros(cap, cfg.hidden_size, dtype=bf, device=dev)
-        self.sel = torch.zeros(max(B, e.max_prefill_seqs), cfg.hidden_size, dtype=bf, device=dev)
-        self.logits = torch.zeros(max(B, e.max_prefill_seqs), cfg.vocab_size, dtype=bf, device=dev)
-        self.tokens = torch.zeros(max(B, e.max_prefill_seqs), dtype=torch.int32, device=dev)
-        if e.sampling:
-            n = max(B, e.max_prefill_seqs)
-            self.samp_temps = torch.zeros(n, dtype=torch.float32, device=dev)
-            self.samp_seeds = torch.zeros(n, 2, dtype=torch.int32, device=dev)
-            self._samp_host = torch.zeros(n, 3, dtype=torch.float32).pin_memory()   # temperature | seed, step as int bits
-        self.tokens_host = torch.zeros(max(B, e.max_prefill_seqs), dtype=torch.int32).pin_memory()
-        # decode metadata: ids | positions | slots | seq_lens | block_table, one pinned mirror
-        self._dec_words = 4 * B + B * self.max_blocks
-        self.dec_meta = torch.zeros(self._dec_words, dtype=torch.int32, device=dev)
-        self.dec_meta_host = torch.zeros(self._dec_words, dtype=torch.int32).pin_memory()
-        # prefill metadata: ids | positions | slots (chunk) + q_starts | q_lens | ctx_lens | last_idx + table
-        P, S = e.prefill_chunk, e.max_prefill_seqs
-        self._pre_words = 3 * P + 4 * S + S * self.max_blocks
-        self.pre_meta = torch.zeros(self._pre_words, dtype=torch.int32, device=dev)
-        self.pre_meta_host = torch.zeros(self._pre_words, dtype=torch.int32).pin_memory()
+        self.sel = torch.zeros(max(B, self.max_seqs), cfg.hidden_size, dtype=bf, device=dev)
+        self.logits = torch.zeros(max(B, self.max_seqs), cfg.vocab_size, dtype=bf, device=dev)
         buckets = e.decode_buckets or capacity_buckets(B)
         ws_rows = max(b * A.decode_plan(b, cfg.num_kv_heads, e.max_seq_len)[0] for b in buckets)
         self.attn_ws = torch.zeros(ws_rows * cfg.num_q_heads * (cfg.head_dim + 2), dtype=torch.float32, device=dev)
+
+    def _alloc_metadata(self) -> None:
+        e, dev, B = self.ecfg, self.device, self.ecfg.max_batch
+        n = max(B, self.max_seqs)
+        self.tokens = torch.zeros(n, dtype=torch.int32, device=dev)
+        if e.sampling:
+            self.samp_temps = torch.zeros(n, dtype=torch.float32, device=dev)
+            self.samp_seeds = torch.zeros(n, 2, dtype=torch.int32, device=dev)
+            self._samp_host = torch.zeros(n, 3, dtype=torch.float32).pin_memory()   # temperature | seed, step as int bits
+        self.tokens_host = torch.zeros(n, dtype=torch.int32).pin_memory()
+        # decode metadata: ids | positions | slots | seq_lens | block_table | state slots, one pinned mirror
+        self._dec_words = 4 * B + B * self.max_blocks + B
+        self.dec_meta = torch.zeros(self._dec_words, dtype=torch.int32, device=dev)
+        self.dec_meta_host = torch.zeros(self._dec_words, dtype=torch.int32).pin_memory()
+        # prefill metadata: ids | positions | slots (chunk) + q_starts | q_lens | ctx_lens | last_idx + table, and for
+        # layered decoders row_seq (chunk) + state_slots | starts
+        P, S = e.prefill_chunk, self.max_seqs
+        self._pre_words = 3 * P + 4 * S + S * self.max_blocks + (P + 2 * S if self.cfg.layered else 0)
+        self.pre_meta = torch.zeros(self._pre_words, dtype=torch.int32, device=dev)
+        self.pre_meta_host = torch.zeros(self._pre_words, dtype=torch.int32).pin_memory()
 
     def _dec_views(self, B: int):
         m, cap = self.dec_meta, self.ecfg.max_batch
@@ -350,6 +379,9 @@ class AttentionEngine:
         else:
             hsel = A.embedding(sel_idx, self.x[:rows], out=self.sel[:n_sel])
         gemm.linear(hsel, self.w.lm_head, out=self.logits[:n_sel])
+        self._sample(n_sel)
+
+    def _sample(self, n_sel: int) -> None:
         if self.ecfg.sampling:
             A.sample(self.logits[:n_sel], self.samp_temps[:n_sel], self.samp_seeds[:n_sel], out=self.tokens[:n_sel])
         else:
@@ -358,6 +390,15 @@ class AttentionEngine:
     def _decode_forward(self, B: int) -> None:
         cfg = self.cfg
         ids, pos, slots, lens, table = self._dec_views(B)
+        if self.body is not None:
+            from .layered import RowBatch
+
+            at = 4 * self.ecfg.max_batch + self.ecfg.max_batch * self.max_blocks
+            b = RowBatch(B, B, B, B, 1, self.ecfg.max_seq_len, pos, slots, table, self.dec_meta[at:at + B])
+            self.body.forward(ids, b, MODE_DECODE)
+            self.body.head(B, None, B, self.sel, self.logits)
+            self._sample(B)
+            return
         A.embedding(ids, self.w.embed, out=self.resid[:B])
         splits, chunk = A.decode_plan(B, cfg.num_kv_heads, self.ecfg.max_seq_len)
 
@@ -372,7 +413,7 @@ class AttentionEngine:
         self._head(B, B, None)
 
     def _prefill_forward(self, rows: int, n_seqs: int, max_q: int) -> None:
-        cfg, P, S = self.cfg, self.ecfg.prefill_chunk, self.ecfg.max_prefill_seqs
+        cfg, P, S = self.cfg, self.ecfg.prefill_chunk, self.max_seqs
         m = self.pre_meta
         ids, pos, slots = m[0:rows], m[P:P + rows], m[2 * P:2 * P + rows]
         b = 3 * P
@@ -390,6 +431,55 @@ class AttentionEngine:
 
         self._layers(rows, MODE_PREFILL, attn)
         self._head(rows, n_seqs, last_idx)
+
+    def _ragged_forward(self, chosen: list[tuple[Sequence, int]], rows: int) -> None:
+        """The layered form of the prefill pass, up to the residual stream of every row: single tokens first (``chosen``
+        is ordered so), then short portions, then long ones."""
+        from .layered import SHORT_PORTION, ExpandGroup, RowBatch
+
+        P, S, n = self.ecfg.prefill_chunk, self.max_seqs, len(chosen)
+        m, b = self.pre_meta, 3 * P
+        t = b + 4 * S
+        r = t + S * self.max_blocks
+        n_dec = sum(1 for _, c in chosen if c == 1)
+        short = [i for i, (_, c) in enumerate(chosen) if c <= SHORT_PORTION]
+        n_abs = sum(chosen[i][1] for i in short)
+        groups, room, start = [], self.body.ws_tokens, len(short)
+        while start < n and room:
+            used, i = 0, start
+            while i < n:
+                need = (chosen[i][0].computed + chosen[i][1] + 63) // 64 * 64
+                if used + need > room:
+                    break
+                used += need
+                i += 1
+            part = chosen[start:i]
+            groups.append(ExpandGroup(start, i - start, max(s.computed + c for s, c in part), max(c for _, c in part), used))
+            start = i
+        batch = RowBatch(
+            rows, n, n_dec, n_abs, max((c for _, c in chosen[n_dec:]), default=0),
+            max(s.computed + c for s, c in (chosen[:len(short)] if self.body.all_expand and short else chosen)),
+            m[P:P + rows], m[2 * P:2 * P + rows], m[t:t + n * self.max_blocks].view(n, self.max_blocks), m[r + P:r + P + n],
+            m[r:r + rows], m[b:b + n], m[b + S:b + S + n], m[b + 2 * S:b + 2 * S + n], m[r + P + S:r + P + S + n], tuple(groups))
+        self.body.forward(m[0:rows], batch, MODE_PREFILL)
+
+    def _fill_ragged(self, hv, chosen: list[tuple[Sequence, int]]) -> None:
+        """Layered part of the chunk's pinned metadata: sequence of every row, state slots, workspace rows."""
+        P, S = self.ecfg.prefill_chunk, self.max_seqs
+        r = 3 * P + 4 * S + S * self.max_blocks
+        from .layered import SHORT_PORTION
+
+        row, used = 0, 0
+        for i, (s, n) in enumerate(chosen):
+            hv[r + row:r + row + n] = i
+            row += n
+            hv[r + P + i] = self.kv.seq_slots.get(s.seq_id, 0)
+            if n > SHORT_PORTION:
+                need = (s.computed + n + 63) // 64 * 64
+                if used + need > self.body.ws_tokens:
+                    used = 0                       # the next group reuses the workspace from its start
+                hv[r + P + S + i] = used
+                used += need
 
     # ------------------------------------------------------------------ stepping
     def _bucket(self, n: int) -> int:
@@ -451,10 +541,27 @@ class AttentionEngine:
         else:
             self._decode_forward(B)
 
-    def _admit_prefill(self) -> tuple[list[tuple[Sequence, int]], int]:
-        """Chooses the sequences (and token counts) of the next prefill chunk."""
+    def _riders(self) -> list[Sequence]:
+        """Running sequences whose next token joins the prefill chunk (``mixed_batches``), with their pages reserved."""
+        if not self.ecfg.mixed_batches:
+            return []
+        out = []
+        for s in list(self.running[:self.ecfg.max_batch]):
+            if len(out) + 1 >= self.ecfg.prefill_chunk:
+                break
+            try:
+                self.kv.ensure(s.seq_id, s.total_len)
+            except OutOfPages:
+                self._retract(s)
+                continue
+            s.computed = s.total_len - 1
+            out.append(s)
+        return out
+
+    def _admit_prefill(self, reserved: int = 0) -> tuple[list[tuple[Sequence, int]], int]:
+        """Chooses the sequences (and token counts) of the next prefill chunk, ``reserved`` of its rows being taken."""
         e = self.ecfg
-        budget, chosen = e.prefill_chunk, []
+        budget, chosen = e.prefill_chunk - reserved, []
         for s in list(self.prefilling):
             if budget <= 0 or len(chosen) >= e.max_prefill_seqs:
                 break
@@ -488,7 +595,7 @@ class AttentionEngine:
             n = min(s.fill_len - s.computed, budget)
             chosen.append((s, n))
             budget -= n
-        return chosen, e.prefill_chunk - budget
+        return chosen, e.prefill_chunk - reserved - budget
 
     def _step_prefill(self, chosen: list[tuple[Sequence, int]], rows: int) -> list[tuple[Sequence, int]]:
         self._launch_prefill(chosen, rows)
@@ -510,7 +617,38 @@ class AttentionEngine:
 
     def _launch_prefill(self, chosen: list[tuple[Sequence, int]], rows: int) -> None:
         """Fills the chunk's pinned metadata and enqueues the chunk; ``_collect_prefill`` finishes it."""
-        e, P, S = self.ecfg, self.ecfg.prefill_chunk, self.ecfg.max_prefill_seqs
+        e, P, S = self.ecfg, self.ecfg.prefill_chunk, self.max_seqs
+        if self.body is not None:
+            chosen = self._order_portions(chosen)
+        self._fill_portions(chosen)
+        with torch.cuda.stream(self.stream):
+            self.pre_meta.copy_(self.pre_meta_host, non_blocking=True)
+            self._stage_sampling([s for s, _ in chosen])
+            self._announce(rows, MODE_PREFILL)
+            if self.body is not None:
+                n = len(chosen)
+                self._ragged_forward(chosen, rows)
+                self.body.head(rows, self.pre_meta[3 * P + 3 * S:3 * P + 3 * S + n], n, self.sel, self.logits)
+                self._sample(n)
+            else:
+                self._prefill_forward(rows, len(chosen), max(n for _, n in chosen))
+            self.tokens_host[:len(chosen)].copy_(self.tokens[:len(chosen)], non_blocking=True)
+            self._step_event.record(self.stream)
+        self._pre_inflight = chosen
+        self.stats["prefill_steps"] += 1
+        self.stats["h2d_bytes"] += self._pre_words * 4
+        self.stats["d2h_bytes"] += len(chosen) * 4
+
+    @staticmethod
+    def _order_portions(chosen: list[tuple[Sequence, int]]) -> list[tuple[Sequence, int]]:
+        """Single tokens, then short portions, then long ones: the row order the layered forward pass works in."""
+        from .layered import SHORT_PORTION
+
+        return sorted(chosen, key=lambda c: 0 if c[1] == 1 else 1 if c[1] <= SHORT_PORTION else 2)
+
+    def _fill_portions(self, chosen: list[tuple[Sequence, int]]) -> None:
+        """Writes the pinned metadata of a ragged pass over ``chosen`` portions."""
+        e, P, S = self.ecfg, self.ecfg.prefill_chunk, self.max_seqs
         hv = self.pre_meta_host.numpy()
         b = 3 * P
         r = 0
@@ -525,17 +663,71 @@ class AttentionEngine:
             tb = b + 4 * S + i * self.max_blocks
             hv[tb:tb + len(t)] = t
             r += n
+        if self.body is not None:
+            self._fill_ragged(hv, chosen)
+
+    # ------------------------------------------------------------------ replaying given tokens
+    def open_sequence(self) -> Sequence:
+        """A sequence whose tokens the caller supplies (:meth:`run_given`) instead of the sampler; it never enters the
+        scheduler's queues. :meth:`close_sequence` gives its pages and slot back."""
+        s = Sequence(self._next_id, [], self.ecfg.max_seq_len)
+        self._next_id += 1
+        return s
+
+    def close_sequence(self, s: Sequence) -> None:
+        self._release_pages(s)
+
+    def run_given(self, portions: list[tuple[Sequence, list[int]]], want: list[list[int]]) -> torch.Tensor:
+        """Runs the next tokens of several open sequences as one batch and returns the logits (fp32, ``[wanted, vocab]``)
+        after the tokens at the places ``want[i]`` of portion i. Batches of single tokens that continue their sequences
+        replay the captured decode graph, all others run the ragged pass: the kernels and the cache of generation."""
+        if self.body is None:
+            raise UnsupportedAttention("given tokens are replayed for layered decoders only")
+        if self.has_work or self.step_in_flight:
+            raise RuntimeError("the engine is generating")
+        for s, toks in portions:
+            if not toks or min(toks) < 0 or max(toks) >= self.cfg.vocab_size:
+                raise ValueError("empty portion or token id outside the vocabulary")
+            if s.total_len + len(toks) > self.ecfg.max_seq_len:
+                raise ValueError("sequence exceeds max_seq_len")
+        rows = sum(len(t) for _, t in portions)
+        if rows > self.ecfg.prefill_chunk or len(portions) > self.max_seqs:
+            raise ValueError("the batch exceeds the engine's row or sequence limit")
+        for s, toks in portions:
+            s.prompt.extend(toks)
+            self.kv.ensure(s.seq_id, s.total_len)
+        picked: list[torch.Tensor] = []
+        n_want = sum(len(w) for w in want)
+        if len(portions) <= self.ecfg.max_batch and all(len(t) == 1 and s.computed > 0 for s, t in portions):
+            batch = [s for s, _ in portions]
+            B = self._fill_decode(batch)
+            self._b_key = None
+            with torch.cuda.stream(self.stream):
+                self.dec_meta.copy_(self.dec_meta_host, non_blocking=True)
+                self._replay_decode(B)
+                picked = [self.logits[i:i + 1].clone() for i, w in enumerate(want) for _ in w]
+        else:
+            order = self._order_portions([((i, s), len(t)) for i, (s, t) in enumerate(portions)])
+            first, at = {}, 0
+            for (i, _), n in order:
+                first[i], at = at, at + n
+            self._fill_portions([(s, n) for (_, s), n in order])
+            sel_rows = [first[i] + j for i, w in enumerate(want) for j in w]
+            with torch.cuda.stream(self.stream):
+                self.pre_meta.copy_(self.pre_meta_host, non_blocking=True)
+                self._ragged_forward([(s, n) for (_, s), n in order], rows)
+                step = self.logits.shape[0]
+                for lo in range(0, n_want, step):
+                    sel = torch.tensor(sel_rows[lo:lo + step], dtype=torch.int32, device=self.device)
+                    self.body.head(rows, sel, sel.numel(), self.sel, self.logits)
+                    picked.append(self.logits[:sel.numel()].clone())
         with torch.cuda.stream(self.stream):
-            self.pre_meta.copy_(self.pre_meta_host, non_blocking=True)
-            self._stage_sampling([s for s, _ in chosen])
-            self._announce(rows, MODE_PREFILL)
-            self._prefill_forward(rows, len(chosen), max(n for _, n in chosen))
-            self.tokens_host[:len(chosen)].copy_(self.tokens[:len(chosen)], non_blocking=True)
-            self._step_event.record(self.stream)
-        self._pre_inflight = chosen
-        self.stats["prefill_steps"] += 1
-        self.stats["h2d_bytes"] += self._pre_words * 4
-        self.stats["d2h_bytes"] += len(chosen) * 4
+            out = torch.cat(picked) if picked else self.logits[:0].clone()
+        self.stream.synchronize()
+        gemm.check_status(self.device)
+        for s, toks in portions:
+            s.computed += len(toks)
+        return out
 
     def _collect_prefill(self) -> list[tuple[Sequence, int]]:
         """Finishes the prefill chunk in flight: waits for its sampled tokens and does the bookkeeping."""
@@ -545,6 +737,16 @@ class AttentionEngine:
         out = []
         th = self.tokens_host.numpy()
         for i, (s, n) in enumerate(chosen):
+            if s in self._riding:                  # a running sequence that took its next token along
+                tok = int(th[i])
+                s.computed = s.total_len
+                s.generated.append(tok)
+                s.token_times.append(now)
+                out.append((s, tok))
+                if s.finished:
+                    self.running.remove(s)
+                    self._finish(s, now)
+                continue
             s.computed += n
             if s.prefill_done:
                 if self.prefix is not None:
@@ -562,6 +764,7 @@ class AttentionEngine:
                     self._finish(s, now)
                 else:
                     self.running.append(s)
+        self._riding = []
         return out
 
     def _release_pages(self, s: Sequence) -> None:
@@ -620,10 +823,18 @@ class AttentionEngine:
             except OutOfPages:
                 self._retract(s)
         batch = kept
-        n = len(batch)
-        if n == 0:
+        if not batch:
             self._b_key = None
             return None
+        return batch, self._fill_decode(batch)
+
+    def _fill_decode(self, batch: list[Sequence]) -> int:
+        """Writes the whole pinned decode metadata for ``batch``; returns the row bucket."""
+        import numpy as np
+
+        cap, ps = self.ecfg.max_batch, self.ecfg.page_size
+        hv = self.dec_meta_host.numpy()
+        n = len(batch)
         B = self._bucket(n)
         hv[0:B] = 0
         hv[cap:cap + B] = 0
@@ -634,15 +845,17 @@ class AttentionEngine:
             p = s.total_len - 1  # position of the token fed in
             t = self.kv.tables[s.seq_id]
             pos[i] = p
-            hv[i] = s.generated[-1]
+            hv[i] = s.generated[-1] if s.generated else s.prompt[-1]
             hv[cap + i] = p
             hv[2 * cap + i] = t[p // ps] * ps + p % ps
             hv[3 * cap + i] = p + 1
             tb = 4 * cap + i * self.max_blocks
             hv[tb:tb + len(t)] = t
+            if self.kv.slots is not None:
+                hv[4 * cap + cap * self.max_blocks + i] = self.kv.seq_slots[s.seq_id]
         self._b_key = tuple(s.seq_id for s in batch)
         self._b_pos = pos
-        return batch, B
+        return B
 
     def _decode_launch(self) -> bool:
         prep = self._decode_prepare()
@@ -711,9 +924,12 @@ class AttentionEngine:
             with torch.cuda.stream(self.stream):
                 begin()
         want_prefill = bool(self.waiting or self.prefilling)
-        if want_prefill and (not self.running or not self._last_was_prefill):
-            chosen, rows = self._admit_prefill()
+        if want_prefill and (not self.running or not self._last_was_prefill or self.ecfg.mixed_batches):
+            riders = self._riders()
+            chosen, rows = self._admit_prefill(len(riders))
             if chosen:
+                self._riding = [s for s in riders if s in self.running]
+                chosen, rows = chosen + [(s, 1) for s in self._riding], rows + len(self._riding)
                 self._last_was_prefill = True
                 self._b_key = None
                 with nvtx.range(f"{self.cfg.name} prefill {rows}"):

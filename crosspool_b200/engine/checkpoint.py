@@ -15,7 +15,7 @@ from pathlib import Path
 import torch
 
 from ..ffn import FfnModelSpec
-from ..models.weights import FFN_KEY
+from ..models.weights import FFN_KEY, LAYERED_FFN_KEY
 
 
 class CheckpointError(ValueError):
@@ -31,7 +31,8 @@ class CheckpointKeyView:
         return sorted(self.key_to_file)
 
     def ffn_keys(self) -> list[str]:
-        return sorted(k for k in self.key_to_file if FFN_KEY.match(k) or ".decoder.layers." in k and (".fc1." in k or ".fc2." in k))
+        return sorted(k for k in self.key_to_file if FFN_KEY.match(k) or LAYERED_FFN_KEY.match(k)
+                      or ".decoder.layers." in k and (".fc1." in k or ".fc2." in k))
 
 
 def read_checkpoint_key_view(model_dir: str | Path) -> CheckpointKeyView:

@@ -2,7 +2,8 @@
 
 Used when one GPU hosts both roles (kernels that wait on one another must never be separate
 launches on one GPU, so the loopback path is stream-ordered and flag-free). Dense layers are two
-launches: gate/up GEMM with the SwiGLU epilogue, then the down projection.
+launches: gate/up GEMM with the SwiGLU epilogue, then the down projection. Ungated layers with a
+row-normalised activation (PolyNorm) put the activation kernel between the two products.
 """
 
 from __future__ import annotations
@@ -10,18 +11,21 @@ from __future__ import annotations
 import torch
 
 from ..models.config import ModelConfig
+from ..models.layered import ceil8, pad_pitch
 from ..models.weights import FfnLayerWeights
 from ..ops import gemm
 from .atn_engine import FfnPort
 
 
 class LocalFfnPort(FfnPort):
-    def __init__(self, cfg: ModelConfig, weights: list[FfnLayerWeights]):
+    def __init__(self, cfg: ModelConfig, weights: list[FfnLayerWeights | None]):
         self.cfg, self.weights = cfg, weights
         self.act = None
         self.y = None
 
     def attach(self, engine) -> None:
+        if self.cfg.layered:
+            return self._attach_layered(engine)
         inter = max(w.gate_up.shape[-2] // 2 for w in self.weights)
         self.act = torch.zeros(engine.cap, inter, dtype=torch.bfloat16, device=engine.device)
         self.y = torch.zeros(engine.cap, self.cfg.hidden_size, dtype=torch.bfloat16, device=engine.device)
@@ -33,8 +37,29 @@ class LocalFfnPort(FfnPort):
             w = moe_layers[0]  # one scratch set sized for the engine's row capacity serves every layer and bucket
             self.moe_ws = moe.workspace(engine.device, engine.cap, self.cfg, w.gate_up.shape[1] // 2, w.gate_up.shape[0])
 
+    def _attach_layered(self, engine) -> None:
+        for w in self.weights:
+            if w is not None:
+                w.gate_up, w.down = pad_pitch(w.gate_up), pad_pitch(w.down)
+        inter = max((ceil8(w.gate_up.shape[0]) for w in self.weights if w is not None), default=8)
+        self.act = torch.zeros(engine.cap * inter, dtype=engine.dtype, device=engine.device)
+        self.y = torch.zeros(engine.cap, ceil8(self.cfg.hidden_size), dtype=engine.dtype, device=engine.device)[:, :self.cfg.hidden_size]
+
+    def _run_polynorm(self, w: FfnLayerWeights, x: torch.Tensor, rows: int) -> list[torch.Tensor]:
+        from ..ops import mixers
+
+        ff = w.gate_up.shape[0]
+        z = self.act[:rows * ceil8(ff)].view(rows, ceil8(ff))[:, :ff]
+        gemm.linear(x, w.gate_up, out=z)
+        coef, eps = w.extra["polynorm"]
+        mixers.polynorm(z, coef, eps, z)
+        gemm.linear(z, w.down, out=self.y[:rows])
+        return [self.y[:rows]]
+
     def run(self, layer: int, x: torch.Tensor, rows: int, mode: int) -> list[torch.Tensor]:
         w = self.weights[layer]
+        if "polynorm" in w.extra:
+            return self._run_polynorm(w, x, rows)
         if w.is_moe:
             from ..ops import moe
 

@@ -1,4 +1,4 @@
-"""Paged KV cache of one Instance on one attention device.
+"""Paged KV cache (and recurrent states) of one Instance on one attention device.
 
 Logical layer: fixed-size pages handed out by :class:`PageAllocator`; a sequence owns a list of
 pages (its block table row). Physical layer: per-layer K and V buffers ``[pages, page_size,
@@ -8,6 +8,9 @@ VMM address ranges whose physical backing is mapped and unmapped in *bundles*
 tensors' addresses — and therefore captured CUDA graphs — stay valid. The allocator only hands out
 pages whose bundle is mapped, like the reference's ``ElasticPageAllocator``
 (src/xpool/integrations/sglang/ecs/allocator.py:61-104).
+
+Layered decoders cache one row per token in the layers that have a cache at all, and keep one recurrent state per live
+sequence (:class:`StateSlots`) in the others; both follow the sequence through the same ``ensure`` / ``release``.
 """
 
 from __future__ import annotations
@@ -100,6 +103,27 @@ class PageAllocator:
                 self._free[b].append(p)
 
 
+class StateSlots:
+    """Hands out the slots of per-sequence recurrent states. A slot is not cleared when it changes hands: the kernels start
+    a sequence whose first token sits at position 0 from a zero state."""
+
+    def __init__(self, n: int):
+        self.total = n
+        self._free = list(range(n - 1, -1, -1))
+
+    @property
+    def free_slots(self) -> int:
+        return len(self._free)
+
+    def alloc(self) -> int:
+        if not self._free:
+            raise OutOfPages("no free state slot")
+        return self._free.pop()
+
+    def free(self, slot: int) -> None:
+        self._free.append(slot)
+
+
 @dataclass
 class KvLayout:
     page_size: int
@@ -108,6 +132,7 @@ class KvLayout:
     head_dim: int
     num_layers: int
     elem_bytes: int = 2
+    row_widths: tuple[int, ...] = ()   # layered decoders: elements of one token's row per layer (0: the layer caches none)
 
     @property
     def page_bytes_per_buffer(self) -> int:
@@ -119,6 +144,8 @@ class KvLayout:
 
     @property
     def bytes_per_page_all_layers(self) -> int:
+        if self.row_widths:
+            return self.page_size * sum(self.row_widths) * self.elem_bytes
         return 2 * self.num_layers * self.page_bytes_per_buffer
 
 
@@ -130,15 +157,33 @@ class PagedKvCache:
     allocator: PageAllocator
     backing: object | None = None  # ecs.vmm.KvVmmBacking when elastic
     tables: dict[int, list[int]] = field(default_factory=dict)
+    # recurrent layers: fp32 [slots, heads, dim, vdim] per layer (None elsewhere), and the slot of every live sequence
+    states: list[torch.Tensor | None] = field(default_factory=list)
+    slots: StateSlots | None = None
+    seq_slots: dict[int, int] = field(default_factory=dict)
 
     @classmethod
     def fixed(cls, cfg: ModelConfig, num_pages: int, page_size: int = 16, device="cuda",
-              dtype: torch.dtype = torch.bfloat16) -> "PagedKvCache":
+              dtype: torch.dtype = torch.bfloat16, state_slots: int = 0) -> "PagedKvCache":
+        if cfg.layered:
+            return cls._layered(cfg, num_pages, page_size, device, dtype, state_slots)
         lay = KvLayout(page_size, num_pages, cfg.num_kv_heads, cfg.head_dim, cfg.num_layers, dtype.itemsize)
         shape = (num_pages, page_size, cfg.num_kv_heads, cfg.head_dim)
         k = [torch.zeros(shape, dtype=dtype, device=device) for _ in range(cfg.num_layers)]
         v = [torch.zeros(shape, dtype=dtype, device=device) for _ in range(cfg.num_layers)]
         return cls(lay, k, v, PageAllocator(num_pages))
+
+    @classmethod
+    def _layered(cls, cfg: ModelConfig, num_pages: int, page_size: int, device, dtype: torch.dtype, state_slots: int) -> "PagedKvCache":
+        """Pages hold one row per token in the layers that cache one (a latent row that is key and value at once);
+        recurrent layers hold one state per slot."""
+        mixers = [s.mixer for s in cfg.layer_specs]
+        lay = KvLayout(page_size, num_pages, 1, 0, cfg.num_layers, dtype.itemsize, tuple(m.cache_width for m in mixers))
+        k = [torch.zeros(num_pages, page_size, 1, m.cache_width, dtype=dtype, device=device) if m.cache_width else None for m in mixers]
+        states = [torch.zeros(state_slots, m.heads, m.dim, m.vdim, dtype=torch.float32, device=device) if m.state_elems else None
+                  for m in mixers]
+        return cls(lay, k, [None] * len(k), PageAllocator(num_pages), states=states,
+                   slots=StateSlots(state_slots) if cfg.recurrent else None)
 
     # -- per-sequence page tables --------------------------------------------------------------
     def pages_needed(self, seq_id: int, new_len: int) -> int:
@@ -149,6 +194,10 @@ class PagedKvCache:
     def ensure(self, seq_id: int, new_len: int) -> list[int]:
         """Grows the sequence's table to cover ``new_len`` tokens."""
         n = self.pages_needed(seq_id, new_len)
+        if n and n > self.allocator.free_pages:
+            raise OutOfPages(f"need {n} pages, {self.allocator.free_pages} free")
+        if self.slots is not None and seq_id not in self.seq_slots:
+            self.seq_slots[seq_id] = self.slots.alloc()
         t = self.tables.setdefault(seq_id, [])
         if n:
             t.extend(self.allocator.alloc(n))
@@ -158,6 +207,9 @@ class PagedKvCache:
         t = self.tables.pop(seq_id, None)
         if t:
             self.allocator.free(t)
+        slot = self.seq_slots.pop(seq_id, None)
+        if slot is not None:
+            self.slots.free(slot)
 
     def slot(self, seq_id: int, pos: int) -> int:
         t = self.tables[seq_id]

@@ -1,0 +1,184 @@
+"""Forward pass of layered decoders inside :class:`AttentionEngine`: every layer brings its own mixer.
+
+One batch (:class:`RowBatch`) holds single decoded tokens first, then portions of prompts. The products and row kernels run
+over all rows together; a mixer splits the rows where its decode and prefill kernels differ:
+
+* latent attention: decoded tokens and short portions run in the absorbed form (queries multiplied into the latent space,
+  one pass over the cached rows); long portions in the expanded form (the sequence's latents are expanded to per-head keys
+  and values with one product each, then the tcgen05 prefill kernel);
+* decayed linear attention: one kernel advances the states of the decoded tokens, another those of the portions.
+
+The residual stream is fp32; each sublayer's output is gated, added and normalised for the next sublayer in one kernel.
+"""
+
+from __future__ import annotations
+
+from dataclasses import dataclass
+
+import torch
+
+from ..models.config import LatentMixer, LinearMixer
+from ..models.layered import LayeredLayerWeights, ceil8
+from ..ops import gemm
+from ..ops import mixers as M
+
+# Portions of at most this many tokens run as rows of the absorbed form: expanding the whole context costs more.
+SHORT_PORTION = 16
+
+
+@dataclass
+class ExpandGroup:
+    """Consecutive sequences whose contexts are expanded together: ``seq0 .. seq0 + n``."""
+
+    seq0: int
+    n: int
+    max_len: int
+    max_q: int
+    tokens: int       # workspace rows, every sequence starting on a multiple of 64
+
+
+@dataclass
+class RowBatch:
+    rows: int
+    n_seqs: int
+    n_dec: int                           # leading rows that are one token each (= leading sequences)
+    n_abs: int                           # leading rows of the absorbed form (decoded tokens, then short portions)
+    max_q: int                           # longest portion behind the decoded tokens
+    max_len: int                         # bound on positions + 1 of the absorbed rows
+    positions: torch.Tensor              # [rows]
+    slots: torch.Tensor                  # [rows] cache row, -1: padding
+    table: torch.Tensor                  # [seqs, max_blocks]
+    state_slots: torch.Tensor            # [seqs]
+    row_seq: torch.Tensor | None = None  # [rows]; None: row r is sequence r
+    q_starts: torch.Tensor | None = None
+    q_lens: torch.Tensor | None = None
+    ctx_lens: torch.Tensor | None = None
+    starts: torch.Tensor | None = None   # [seqs] first workspace row of an expanded context
+    groups: tuple[ExpandGroup, ...] = ()
+
+
+class LayeredForward:
+    def __init__(self, engine):
+        self.e = engine
+        cfg, dev, dt, cap = engine.cfg, engine.device, engine.dtype, engine.cap
+        self.dtype = dt
+        h8 = ceil8(cfg.hidden_size)
+        layers: list[LayeredLayerWeights] = engine.w.layers
+        self.layers = layers
+
+        def buf(n, dtype=dt):
+            return torch.zeros(n, dtype=dtype, device=dev)
+
+        self.resid = torch.zeros(cap, cfg.hidden_size, dtype=torch.float32, device=dev)
+        self.x, self.x2, self.y, self.rg2 = (torch.zeros(cap, h8, dtype=dt, device=dev)[:, :cfg.hidden_size] for _ in range(4))
+        self.proj = buf(cap * max(lw.offs["end"] for lw in layers))
+        self.mix_out = torch.zeros(cap * max(ceil8(lw.spec.mixer.out_features) for lw in layers), dtype=dt, device=dev)
+        lat = [lw.spec.mixer for lw in layers if isinstance(lw.spec.mixer, LatentMixer)]
+        lin = [lw.spec.mixer for lw in layers if isinstance(lw.spec.mixer, LinearMixer)]
+        self.expands = [("exp_k" in lw.mix) for lw in layers]
+        # every latent layer has an expanded form: only decoded tokens and short portions run absorbed
+        self.all_expand = all(ex for lw, ex in zip(layers, self.expands) if isinstance(lw.spec.mixer, LatentMixer))
+        if lat:
+            self.q_plain = buf(cap * max(m.heads * ceil8(m.dim) for m in lat))
+            self.q_abs = buf(cap * max(m.heads * m.cache_width for m in lat))
+            self.o_lat = buf(cap * max(m.heads * ceil8(m.kv_rank) for m in lat))
+            buckets = engine._buckets
+            need = max(b * M.latent_attn_plan(b, m.heads, engine.ecfg.max_seq_len)[0] * m.heads * (m.kv_rank + 2)
+                       for b in buckets for m in lat)
+            self.attn_ws = buf(max(need, 1 << 20), torch.float32)
+        self.ws_tokens = 0
+        if any(self.expands):
+            shapes = [(m.heads, *M.expanded_shape(m.dim, m.rot_dim, m.vdim), m.cache_width)
+                      for m, ex in ((lw.spec.mixer, ex) for lw, ex in zip(layers, self.expands)) if ex]
+            self.ws_tokens = (max(engine.ecfg.max_seq_len, cap) + 63) // 64 * 64 + 64
+            self.q_exp = buf(cap * max(H * dq for H, dq, _, _ in shapes))
+            self.lat_ws = buf(self.ws_tokens * max(w for *_, w in shapes))
+            self.k_exp = buf(self.ws_tokens * max(H * dq for H, dq, _, _ in shapes))
+            self.v_exp = buf(self.ws_tokens * max(H * dv for H, _, dv, _ in shapes))
+        if lin:
+            self.o_lin = buf(cap * max(m.out_features for m in lin), torch.float32)
+        self.lin_ws = None
+
+    # ------------------------------------------------------------------ mixers
+    def _latent(self, l: int, lw: LayeredLayerWeights, m: LatentMixer, proj: torch.Tensor, out: torch.Tensor, b: RowBatch) -> None:
+        rows, H, R, W = b.rows, m.heads, m.kv_rank, m.cache_width
+        n_abs = b.n_abs if self.expands[l] else rows
+        dp, rp = ceil8(m.dim), ceil8(R)
+        cache = self.e.kv.k[l]
+        q_plain = self.q_plain[:H * n_abs * dp].view(H, n_abs, dp) if n_abs else None
+        q_abs = self.q_abs[:H * n_abs * W].view(H, n_abs, W) if n_abs else None
+        q_exp = None
+        if n_abs < rows:
+            dq, dv = M.expanded_shape(m.dim, m.rot_dim, m.vdim)
+            q_exp = self.q_exp[:rows * H * dq].view(rows, H, dq)
+        gate = proj[:, lw.offs["g"]:lw.offs["g"] + H]
+        M.latent_prep(proj, lw.mix["norm"], lw.mix["freq"], b.positions, b.slots, cache, heads=H, dim=m.dim, rot=m.rot_dim, kv_rank=R,
+                      q_off=lw.offs["q"], kv_off=lw.offs["kv"], eps=self.e.cfg.rms_norm_eps, abs_rows=n_abs, q_plain=q_plain,
+                      q_abs=q_abs, q_exp=q_exp)
+        if n_abs:
+            gemm.linear_batched(q_plain[:, :, :m.dim], lw.mix["uk_t"], q_abs, n_abs * W)
+            splits, chunk = M.latent_attn_plan(n_abs, H, b.max_len)
+            if splits > 1 and n_abs * H * splits * (R + 2) > self.attn_ws.numel():
+                splits, chunk = 1, 0
+            o_lat = self.o_lat[:H * n_abs * rp].view(H, n_abs, rp)
+            M.latent_attn(q_abs, cache, o_lat, b.table, b.positions, b.slots, kv_rank=R, rot=m.rot_dim, scale=m.scale, gate=gate,
+                          row_seq=b.row_seq, num_splits=splits, chunk_tokens=chunk, ws=self.attn_ws)
+            gemm.linear_batched(o_lat[:, :, :R], lw.mix["uv"], out[:n_abs], m.vdim)
+        if n_abs < rows:
+            for g in b.groups:
+                s = slice(g.seq0, g.seq0 + g.n)
+                starts = b.starts[s]
+                lat = self.lat_ws[:g.tokens * W].view(g.tokens, W)
+                M.latent_gather(cache, lat, b.table[s], b.ctx_lens[s], b.q_lens[s], starts, g.max_len)
+                k = self.k_exp[:g.tokens * H * dq].view(g.tokens, H, dq)
+                v = self.v_exp[:g.tokens * H * dv].view(g.tokens, H, dv)
+                gemm.linear(lat[:, :R + m.rot_dim], lw.mix["exp_k"], out=k.view(g.tokens, H * dq))
+                gemm.linear(lat[:, :R], lw.mix["exp_v"], out=v.view(g.tokens, H * dv))
+                M.expanded_prefill(q_exp, k, v, out, b.q_starts[s], b.q_lens[s], b.ctx_lens[s], starts, g.max_q, scale=m.scale,
+                                   vdim=m.vdim, gate=gate)
+
+    def _linear(self, l: int, lw: LayeredLayerWeights, m: LinearMixer, proj: torch.Tensor, out: torch.Tensor, b: RowBatch) -> None:
+        n = m.out_features
+        o = self.o_lin[:b.rows * n].view(b.rows, n)
+        kw = dict(heads=m.heads, dim=m.dim, vdim=m.vdim, offs=(lw.offs["q"], lw.offs["k"], lw.offs["v"]))
+        state, dec, pw = self.e.kv.states[l], lw.mix["decay"], lw.mix["decay_pow"]
+        if b.n_dec:
+            M.linear_attn_decode(proj[:b.n_dec], state, dec, pw, o[:b.n_dec], b.positions, b.slots, b.state_slots, **kw)
+        if b.n_dec < b.n_seqs:
+            s = slice(b.n_dec, b.n_seqs)
+            M.linear_attn_prefill(proj, state, dec, pw, o, b.positions, b.slots, b.state_slots[s], b.q_starts[s], b.q_lens[s], b.max_q,
+                                  ws=self.lin_ws, **kw)
+        M.gated_rms(o, lw.mix["norm"], proj[:, lw.offs["g"]:lw.offs["g"] + n], self.e.cfg.rms_norm_eps, out)
+
+    # ------------------------------------------------------------------ layers
+    def forward(self, ids: torch.Tensor, b: RowBatch, mode: int) -> None:
+        """Embedding and all layers over the batch's rows; the last sublayer's output stays pending for :meth:`head`."""
+        rows, hid = b.rows, self.e.cfg.hidden_size
+        resid, x, x2, y = self.resid[:rows], self.x[:rows], self.x2[:rows], self.y[:rows]
+        pending: dict = dict(ids=ids, table=self.e.w.embed)
+        for l, lw in enumerate(self.layers):
+            M.resid_norm(resid, lw.norm1, x, **pending)
+            proj = self.proj[:rows * lw.offs["end"]].view(rows, lw.offs["end"])
+            gemm.linear(x, lw.proj, out=proj, bias=lw.proj_bias)
+            m = lw.spec.mixer
+            n = m.out_features
+            out = self.mix_out[:rows * ceil8(n)].view(rows, ceil8(n))[:, :n]
+            (self._latent if isinstance(m, LatentMixer) else self._linear)(l, lw, m, proj, out, b)
+            gemm.linear(out, lw.o, out=y)
+            pending = dict(parts=[y], gate=proj[:, lw.offs["rg"]:lw.offs["rg"] + hid])
+            if lw.norm2 is not None:
+                M.resid_norm(resid, lw.norm2, x2, **pending)
+                rg2 = self.rg2[:rows]
+                gemm.linear(x2, lw.rg2, out=rg2, bias=lw.rg2_bias)
+                pending = dict(parts=self.e.port.run(l, x2, rows, mode), gate=rg2)
+            self.tap(l, rows, pending)
+        self._pending = pending
+
+    def tap(self, layer: int, rows: int, pending: dict) -> None:
+        """Called after every layer with its output still pending; a debugging subclass or test may look at it."""
+
+    def head(self, rows: int, sel: torch.Tensor | None, n_sel: int, out: torch.Tensor, logits: torch.Tensor) -> None:
+        """Final norm of the selected rows (all of the first ``n_sel`` without ``sel``) and their scaled logits (fp32)."""
+        e = self.e
+        M.resid_norm(self.resid[:rows], e.w.final_norm, out[:n_sel], sel=sel, rows=n_sel, **self._pending)
+        gemm.linear(out[:n_sel], e.w.lm_head, out=logits[:n_sel], out_scale=e.cfg.logit_scale)

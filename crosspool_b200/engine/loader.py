@@ -17,7 +17,7 @@ from dataclasses import dataclass
 
 import torch
 
-from ..ffn import DenseFfnSpec, FfnModelSpec, GateUpOrder, MoeFfnSpec, RouterProjectionPrecision, TopKWeightRounding
+from ..ffn import ActivationKind, DenseFfnSpec, FfnModelSpec, GateUpOrder, MoeFfnSpec, RouterProjectionPrecision, TopKWeightRounding
 from ..models.weights import FfnLayerWeights
 from .checkpoint import CheckpointKeyView
 
@@ -111,6 +111,8 @@ class PinnedStager:
 
 
 def _dense_reads(l: DenseFfnSpec, rank: int, size: int):
+    if l.activation == ActivationKind.POLYNORM and size > 1:
+        raise NotImplementedError("a row-normalised activation needs the whole FFN row on one rank (FFN TP 1)")
     rows = _local(l.intermediate_size, rank, size)
     ip = l.i_proj
     reads = {}
@@ -132,6 +134,8 @@ def _dense_reads(l: DenseFfnSpec, rank: int, size: int):
     reads["down"] = TensorRead(l.o_proj.weight_key, cols=rows)
     if l.o_proj.bias_key and rank == 0:
         reads["down_bias"] = TensorRead(l.o_proj.bias_key)
+    if l.activation_key:
+        reads["act_coef"] = TensorRead(l.activation_key)
     return reads
 
 
@@ -250,7 +254,7 @@ def materialize_layer_weights(spec: FfnModelSpec, view: CheckpointKeyView, layer
     """Loads one layer's local shard. ``experts`` restricts a MoE layer to a range (expert parallelism)."""
     if spec.quantization not in ("none", "mxfp4", "fp8_block"):
         raise NotImplementedError(f"checkpoints quantised with {spec.quantization} are not loadable")
-    l = spec.layers[layer]
+    l = spec.layer(layer)
     if spec.quantization == "fp8_block":
         if not isinstance(l, DenseFfnSpec) or l.i_proj.gate is None or l.i_proj.gate.scales_key is None:
             raise NotImplementedError("block-scaled fp8 checkpoints are loadable for gated dense layers only")
@@ -265,7 +269,7 @@ def materialize_layer_weights(spec: FfnModelSpec, view: CheckpointKeyView, layer
 
     def fetch(item):
         name, r = item
-        wide = "bias" in name or name == "router_fp32"   # biases stay fp32: the GEMM epilogue adds them to the fp32 accumulator
+        wide = "bias" in name or name in ("router_fp32", "act_coef")   # biases stay fp32: the GEMM epilogue adds them to the fp32 accumulator
         return name, stager.to_device(reader.read(r), torch.float32 if wide else dtype)
 
     with ThreadPoolExecutor(max_workers=max(1, parallelism)) as pool:
@@ -280,6 +284,8 @@ def materialize_layer_weights(spec: FfnModelSpec, view: CheckpointKeyView, layer
             gub = torch.cat([got["gate_bias"], got["up_bias"]], 0) if "gate_bias" in got else got["up_bias"]
         w = FfnLayerWeights(gate_up, got["down"], gate_up_bias=gub, down_bias=got.get("down_bias"))
         w.extra["gated"] = gated
+        if l.activation == ActivationKind.POLYNORM:
+            w.extra["polynorm"] = (got["act_coef"].contiguous(), l.activation_eps)
         t = l.gate_transform
         if t is not None and (t.limit > 0 or t.up_offset != 0 or t.alpha != 1.0):
             w.extra["gate_transform"] = (float(t.limit), float(t.up_offset), float(t.alpha))

@@ -19,6 +19,7 @@ class ActivationKind(str, Enum):
     SILU = "silu"
     RELU = "relu"
     GELU = "gelu"
+    POLYNORM = "polynorm"          # a N(z) + b N(z^2) + c N(z^3) + e, N = row RMS normalisation: needs the whole row
 
 
 class GateUpOrder(str, Enum):
@@ -92,6 +93,8 @@ class DenseFfnSpec:
     o_proj: ProjectionSpec
     gate_transform: GateTransform = GateTransform()
     kind: LayerKind = LayerKind.DENSE
+    activation_key: str | None = None   # checkpoint tensor of the activation's coefficients (PolyNorm)
+    activation_eps: float = 0.0
 
 
 @dataclass(frozen=True)
@@ -155,6 +158,13 @@ class FfnModelSpec:
     def num_layers(self) -> int:
         return len(self.layers)
 
+    def layer(self, ordinal: int) -> DenseFfnSpec | MoeFfnSpec:
+        """The FFN of decoder layer ``ordinal`` (layers of layered decoders may have none)."""
+        for l in self.layers:
+            if l.layer == ordinal:
+                return l
+        raise KeyError(f"decoder layer {ordinal} has no FFN")
+
     def required_keys(self) -> set[str]:
         """Every checkpoint key the FFN side must find (used for exact coverage validation)."""
         keys: set[str] = set()
@@ -172,6 +182,8 @@ class FfnModelSpec:
             if isinstance(l, DenseFfnSpec):
                 add(l.i_proj.gate), add(l.i_proj.up if l.i_proj.packed is None else None), add(l.i_proj.packed)
                 add(l.o_proj)
+                if l.activation_key:
+                    keys.add(l.activation_key)
             else:
                 keys.add(l.router_weight_key)
                 for k in (l.router_bias_key, l.correction_bias_key, l.shared_gate_key, l.shared_up_key,

@@ -1,7 +1,7 @@
 """Architecture adapters: Hugging Face ``config.json`` + checkpoint keys → :class:`FfnModelSpec`.
 
-One adapter per supported architecture, discovered by ``architectures[0]`` — the same eight
-families the reference serves (src/xpool/runtime/ffnagent/models/*.py, discovery in
+One adapter per supported architecture, discovered by ``architectures[0]`` (``architecture`` in the
+configuration files of layered decoders) — Segirax and the same eight families the reference serves (src/xpool/runtime/ffnagent/models/*.py, discovery in
 src/xpool/runtime/ffnagent/architecture.py:175-215): Qwen2, Qwen3, Qwen3-MoE, Llama, OPT,
 DeepSeek-V2, GLM-4 MoE Lite and GPT-OSS. Adapters only read the configuration and the *names* of
 checkpoint tensors; no weight is opened here.
@@ -60,6 +60,8 @@ class FfnSourceConfig:
     @property
     def architecture(self) -> str:
         a = self.cfg.get("architectures") or []
+        if isinstance(self.cfg.get("architecture"), str):
+            return self.cfg["architecture"]
         if not a:
             raise UnsupportedModel("config.json has no architectures")
         return a[0]
@@ -209,6 +211,22 @@ def _gpt_oss(model_id: str, src: FfnSourceConfig, keys: Iterable[str]) -> FfnMod
     return FfnModelSpec(model_id, src.architecture, src.payload_dtype, hidden, quant, tuple(layers))
 
 
+def _segirax(model_id: str, src: FfnSourceConfig, keys: Iterable[str]) -> FfnModelSpec:
+    from .config import segirax_config
+
+    c = segirax_config(dict(src.cfg), model_id)
+    layers = []
+    for i, s in enumerate(c.layer_specs):
+        if s.ff == 0:
+            continue
+        p = f"l{i}.mlp"
+        layers.append(DenseFfnSpec(i, c.hidden_size, s.ff, ActivationKind.POLYNORM,
+                                   GatedProjectionSpec(None, ProjectionSpec(f"{p}.up", s.ff, c.hidden_size)),
+                                   ProjectionSpec(f"{p}.down", c.hidden_size, s.ff), activation_key=f"{p}.act",
+                                   activation_eps=c.rms_norm_eps))
+    return FfnModelSpec(model_id, src.architecture, src.payload_dtype, c.hidden_size, src.quantization, tuple(layers))
+
+
 ADAPTERS: dict[str, Callable[[str, FfnSourceConfig, Iterable[str]], FfnModelSpec]] = {
     "Qwen2ForCausalLM": _llama_like,
     "Qwen3ForCausalLM": _llama_like,
@@ -219,6 +237,7 @@ ADAPTERS: dict[str, Callable[[str, FfnSourceConfig, Iterable[str]], FfnModelSpec
     "DeepseekV2ForCausalLM": lambda m, s, k: _deepseek_like(m, s, k, sigmoid=False),
     "Glm4MoeLiteForCausalLM": lambda m, s, k: _deepseek_like(m, s, k, sigmoid=True),
     "GptOssForCausalLM": _gpt_oss,
+    "Segirax": _segirax,
 }
 
 

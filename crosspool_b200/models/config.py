@@ -33,6 +33,83 @@ class MlaShape:
 
 
 @dataclass(frozen=True)
+class RotarySpec:
+    """Rotary positions on the first ``dims`` dimensions of a vector, paired (i, i + dims / 2): the pair at position p
+    turns by ``p * base ** (-2 i / dims)``."""
+
+    dims: int
+    base: float
+
+
+@dataclass(frozen=True)
+class LatentMixer:
+    """Latent attention as a layer's mixer: per-head keys and values are linear maps of one cached ``kv_rank`` latent,
+    plus one rotary key part of ``rot_dim`` shared by the heads. The output of every head is gated by a sigmoid."""
+
+    heads: int
+    dim: int                    # unrotated query/key dimensions per head
+    rot_dim: int                # rotated query/key dimensions per head
+    vdim: int
+    kv_rank: int
+    rot: RotarySpec
+    scale: float
+    kind: str = "latent_attention"
+
+    @property
+    def cache_width(self) -> int:
+        """Elements of one token's cache row: latent and rotated key, padded to whole 16-element tensor-core steps."""
+        return (self.kv_rank + self.rot_dim + 15) // 16 * 16
+
+    @property
+    def state_elems(self) -> int:
+        return 0
+
+    @property
+    def out_features(self) -> int:
+        return self.heads * self.vdim
+
+    def param_count(self, hidden: int) -> int:
+        q = self.heads * (self.dim + self.rot_dim)
+        return (hidden * (q + self.kv_rank + self.rot_dim + self.heads + self.out_features) + self.kv_rank
+                + self.kv_rank * self.heads * (self.dim + self.vdim))
+
+
+@dataclass(frozen=True)
+class LinearMixer:
+    """Decayed linear attention (one fp32 ``dim x vdim`` state per head and sequence, a fixed decay per head), its heads
+    normalised together and gated."""
+
+    heads: int
+    dim: int
+    vdim: int
+    decay: tuple[float, ...]
+    kind: str = "lightning"
+
+    @property
+    def cache_width(self) -> int:
+        return 0
+
+    @property
+    def state_elems(self) -> int:
+        return self.heads * self.dim * self.vdim
+
+    @property
+    def out_features(self) -> int:
+        return self.heads * self.vdim
+
+    def param_count(self, hidden: int) -> int:
+        return hidden * self.heads * (2 * self.dim + 3 * self.vdim) + self.out_features
+
+
+@dataclass(frozen=True)
+class LayerSpec:
+    """One layer of a layered (hybrid) decoder: its mixer and the width of its ungated FFN (0: no FFN)."""
+
+    mixer: LatentMixer | LinearMixer
+    ff: int = 0
+
+
+@dataclass(frozen=True)
 class ModelConfig:
     name: str
     architecture: str  # HF ``architectures[0]``
@@ -70,10 +147,26 @@ class ModelConfig:
     attention_sinks: bool = False    # one learned logit per head joins every softmax and takes no value: GPT-OSS
     o_bias: bool = False
     mla: MlaShape | None = None
+    # Layered decoders: every layer names its own mixer and FFN. norm "dyt" is dynamic tanh (elementwise, no statistics);
+    # ``residual_gate``: each sublayer's result is multiplied by sigmoid(W h + b) of its input and summed in fp32.
+    layer_specs: tuple[LayerSpec, ...] = ()
+    residual_gate: bool = False
+    logit_scale: float = 1.0
     extra: dict[str, Any] = field(default_factory=dict, compare=False, hash=False)
 
     @property
+    def layered(self) -> bool:
+        return bool(self.layer_specs)
+
+    @property
+    def recurrent(self) -> bool:
+        """Some layer carries a per-sequence state, which cannot be shared between sequences like a cache page."""
+        return any(s.mixer.state_elems for s in self.layer_specs)
+
+    @property
     def gpu_attention_supported(self) -> bool:
+        if self.layered:
+            return True
         return (self.norm == "rmsnorm" and self.positions == "rope" and self.mla is None and not self.attention_sinks
                 and not self.sliding_window and not self.o_bias and not self.extra.get("rope_scaling"))
 
@@ -100,12 +193,22 @@ class ModelConfig:
         return self.is_moe and layer >= self.first_k_dense
 
     def attention_param_bytes(self) -> int:
+        if self.layered:
+            n = self.hidden_size * (self.vocab_size * (1 if self.tie_word_embeddings else 2) + 2) + 1
+            for s in self.layer_specs:
+                subs = 1 + (s.ff > 0)
+                n += s.mixer.param_count(self.hidden_size) + subs * (2 * self.hidden_size + 1)
+                if self.residual_gate:
+                    n += subs * self.hidden_size * (self.hidden_size + 1)
+            return 2 * n
         per_layer = (self.q_size + 2 * self.kv_size) * self.hidden_size + self.hidden_size * self.q_size
         per_layer += 2 * self.hidden_size + 2 * self.head_dim
         emb = self.vocab_size * self.hidden_size * (1 if self.tie_word_embeddings else 2)
         return 2 * (per_layer * self.num_layers + emb + self.hidden_size)
 
     def ffn_param_bytes_per_layer(self, layer: int = 0) -> int:
+        if self.layered:
+            return 2 * 2 * self.hidden_size * self.layer_specs[layer].ff
         if self.layer_is_moe(layer):
             e = self.num_experts * 3 * self.hidden_size * self.moe_intermediate_size
             e += self.num_experts * self.hidden_size
@@ -114,9 +217,17 @@ class ModelConfig:
         return 2 * 3 * self.hidden_size * self.intermediate_size
 
     def kv_bytes_per_token(self) -> int:
+        if self.layered:
+            return 2 * sum(s.mixer.cache_width for s in self.layer_specs)
         return 2 * self.num_layers * self.kv_size * 2
 
+    def state_bytes_per_sequence(self) -> int:
+        """fp32 recurrent state of one running sequence over all layers."""
+        return 4 * sum(s.mixer.state_elems for s in self.layer_specs)
+
     def with_layers(self, n: int) -> "ModelConfig":
+        if self.layered:
+            return replace(self, num_layers=n, layer_specs=tuple(self.layer_specs[i % len(self.layer_specs)] for i in range(n)))
         return replace(self, num_layers=n)
 
 
@@ -158,8 +269,43 @@ def preset(name: str) -> ModelConfig:
         raise KeyError(f"unknown model preset {name!r}; known: {sorted(PRESETS)}") from None
 
 
+def _mixer_from_config(kind: str, m: dict[str, Any]) -> LatentMixer | LinearMixer:
+    if kind == "latent_attention":
+        rot = RotarySpec(int(m["rot"]["dims"]), float(m["rot"]["base"]))
+        mixer = LatentMixer(int(m["heads"]), int(m["dim"]), int(m["rot_dim"]), int(m["vdim"]), int(m["kv_rank"]), rot, float(m["scale"]))
+        if rot.dims % 2 or rot.dims > mixer.rot_dim:
+            raise ValueError(f"rotary dims {rot.dims} do not fit the {mixer.rot_dim}-wide rotary part")
+        return mixer
+    if kind == "lightning":
+        decay = tuple(float(d) for d in m["decay"])
+        if len(decay) != int(m["heads"]):
+            raise ValueError(f"{len(decay)} decays for {m['heads']} heads")
+        return LinearMixer(int(m["heads"]), int(m["dim"]), int(m["vdim"]), decay)
+    raise ValueError(f"unsupported mixer {kind!r}")
+
+
+def segirax_config(cfg: dict[str, Any], name: str = "") -> ModelConfig:
+    """Segirax: dynamic-tanh norms, gated fp32 residual stream, latent-attention and lightning mixers in any order, and
+    ungated PolyNorm FFNs; its ``config.json`` lists every layer."""
+    specs = []
+    for l in cfg["layers"]:
+        mlp = l.get("mlp")
+        if mlp is not None and mlp.get("kind", "dense") != "dense":
+            raise ValueError(f"unsupported feed-forward kind {mlp['kind']!r}")
+        specs.append(LayerSpec(_mixer_from_config(l["type"], l["mixer"]), int(mlp["ff"]) if mlp is not None else 0))
+    first = specs[0].mixer
+    return ModelConfig(
+        name=name or cfg["architecture"], architecture=cfg["architecture"], hidden_size=int(cfg["width"]), num_layers=len(specs),
+        num_q_heads=first.heads, num_kv_heads=1, head_dim=first.dim, intermediate_size=max(s.ff for s in specs),
+        vocab_size=int(cfg["vocab"]), rms_norm_eps=float(cfg["norm"]["eps"]), qk_norm=False, tie_word_embeddings=True,
+        hidden_act="polynorm", max_position_embeddings=1 << 30, norm="dyt", layer_specs=tuple(specs), residual_gate=True,
+        logit_scale=float(cfg["logit_scale"]))
+
+
 def from_hf_config(cfg: dict[str, Any], name: str = "") -> ModelConfig:
     """Builds a :class:`ModelConfig` from a parsed ``config.json``."""
+    if cfg.get("architecture") == "Segirax":
+        return segirax_config(cfg, name)
     arch = (cfg.get("architectures") or ["Qwen3ForCausalLM"])[0]
     hidden = int(cfg["hidden_size"])
     heads = int(cfg["num_attention_heads"])

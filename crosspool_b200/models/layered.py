@@ -1,0 +1,137 @@
+"""Attention-side weights of layered decoders in the layout the kernels want.
+
+Every layer's linear maps of the same input become one matrix: the mixer's input projections and the residual gate
+(``[projections | gate | residual gate]``), each section padded to eight rows so that its columns in the product start on a
+16-byte boundary. Latent attention keeps its up-projections twice: per head for the absorbed form (decode), and with the
+shared rotary key folded in as identity rows for the expanded form (prefill), so that one product writes complete per-head
+keys. Norm parameters, gates' biases and decays are fp32.
+"""
+
+from __future__ import annotations
+
+from dataclasses import dataclass, field
+from typing import Callable
+
+import torch
+
+from ..ops.mixers import NormParams, decay_powers, expanded_shape
+from .config import LatentMixer, LayerSpec, LinearMixer, ModelConfig
+
+# get(name, shape): the checkpoint tensor (or a random one) of that name
+Getter = Callable[[str, tuple[int, ...]], torch.Tensor]
+
+
+def ceil8(n: int) -> int:
+    return (n + 7) // 8 * 8
+
+
+def pad_pitch(w: torch.Tensor) -> torch.Tensor:
+    """``[n, k]`` with a row pitch of whole 16-byte units (zeros behind the k columns)."""
+    n, k = w.shape
+    if k % 8 == 0:
+        return w.contiguous()
+    out = torch.zeros(n, ceil8(k), dtype=w.dtype, device=w.device)
+    out[:, :k] = w
+    return out[:, :k]
+
+
+@dataclass
+class LayeredLayerWeights:
+    spec: LayerSpec
+    norm1: NormParams
+    proj: torch.Tensor                      # every linear map of norm1's output
+    proj_bias: torch.Tensor                 # fp32, zero outside the residual gate
+    offs: dict[str, int]                    # first column of each section of the product
+    o: torch.Tensor                         # [hidden, mixer outputs]
+    mix: dict[str, torch.Tensor] = field(default_factory=dict)
+    norm2: NormParams | None = None
+    rg2: torch.Tensor | None = None         # residual gate of the FFN
+    rg2_bias: torch.Tensor | None = None
+
+
+def _fuse(sections: list[tuple[str, torch.Tensor]]) -> tuple[torch.Tensor, dict[str, int]]:
+    rows, offs, at = [], {}, 0
+    for name, w in sections:
+        offs[name] = at
+        rows.append(w)
+        pad = ceil8(w.shape[0]) - w.shape[0]
+        if pad:
+            rows.append(torch.zeros(pad, w.shape[1], dtype=w.dtype, device=w.device))
+        at += w.shape[0] + pad
+    offs["end"] = at
+    return pad_pitch(torch.cat(rows, 0)), offs
+
+
+def _norm(get: Getter, name: str, cfg: ModelConfig) -> NormParams:
+    h = cfg.hidden_size
+    return NormParams("dyt", get(name, (h,)).float().contiguous(), get(name + ".b", (h,)).float().contiguous(),
+                      get(name + ".alpha", ()).float().reshape(1).contiguous(), cfg.rms_norm_eps)
+
+
+def rotary_frequencies(dims: int, base: float) -> torch.Tensor:
+    return float(base) ** (-2.0 * torch.arange(dims // 2, dtype=torch.float64) / dims)
+
+
+def _latent(m: LatentMixer, get: Getter, p: str, hidden: int, dtype: torch.dtype, device) -> tuple[list, dict]:
+    H, R, d, r, vd = m.heads, m.kv_rank, m.dim, m.rot_dim, m.vdim
+    q, dkv, g = get(p + "q", (H * (d + r), hidden)), get(p + "dkv", (R + r, hidden)), get(p + "g", (H, hidden))
+    uk, uv = get(p + "uk", (H * d, R)), get(p + "uv", (H * vd, R))
+    mix = {"norm": get(p + "dkv.norm", (R,)).float().contiguous(), "freq": rotary_frequencies(m.rot.dims, m.rot.base).to(device),
+           "uk_t": pad_pitch(uk.view(H, d, R).transpose(1, 2).reshape(H * R, d)), "uv": pad_pitch(uv)}
+    shape = expanded_shape(d, r, vd) if dtype == torch.bfloat16 else None
+    if shape is not None:
+        dq, dv = shape
+        ek = torch.zeros(H, dq, R + r, dtype=uk.dtype, device=uk.device)
+        ek[:, :d, :R] = uk.view(H, d, R)
+        ek[:, torch.arange(d, d + r), torch.arange(R, R + r)] = 1
+        ev = torch.zeros(H, dv, R, dtype=uv.dtype, device=uv.device)
+        ev[:, :vd] = uv.view(H, vd, R)
+        mix["exp_k"], mix["exp_v"] = pad_pitch(ek.view(H * dq, R + r)), pad_pitch(ev.view(H * dv, R))
+    return [("q", q), ("kv", dkv), ("g", g)], mix
+
+
+def _linear(m: LinearMixer, get: Getter, p: str, hidden: int, device) -> tuple[list, dict]:
+    H, d, vd = m.heads, m.dim, m.vdim
+    sections = [(n, get(p + n, (H * w, hidden))) for n, w in (("q", d), ("k", d), ("v", vd), ("g", vd))]
+    return sections, {"norm": get(p + "norm", (H * vd,)).float().contiguous(),
+                      "decay": torch.tensor(m.decay, dtype=torch.float32, device=device),
+                      "decay_pow": decay_powers(m.decay).to(device)}
+
+
+def layered_attention_weights(cfg: ModelConfig, get: Getter, device, dtype: torch.dtype):
+    """Everything but the FFNs of a layered decoder, from its named tensors (``l<i>.norm1``, ``l<i>.mix.*``,
+    ``l<i>.rg1``, ...)."""
+    from .weights import AttentionWeights
+
+    h = cfg.hidden_size
+    layers = []
+    for i, spec in enumerate(cfg.layer_specs):
+        p, m = f"l{i}", spec.mixer
+        if isinstance(m, LatentMixer):
+            sections, mix = _latent(m, get, p + ".mix.", h, dtype, device)
+        else:
+            sections, mix = _linear(m, get, p + ".mix.", h, device)
+        sections.append(("rg", get(p + ".rg1", (h, h))))
+        proj, offs = _fuse(sections)
+        bias = torch.zeros(offs["end"], dtype=torch.float32, device=device)
+        bias[offs["rg"]:offs["rg"] + h] = get(p + ".rg1.b", (h,)).float()
+        lw = LayeredLayerWeights(spec, _norm(get, p + ".norm1", cfg), proj, bias, offs, pad_pitch(get(p + ".mix.o", (h, m.out_features))),
+                                 mix)
+        if spec.ff:
+            lw.norm2 = _norm(get, p + ".norm2", cfg)
+            lw.rg2, lw.rg2_bias = pad_pitch(get(p + ".rg2", (h, h))), get(p + ".rg2.b", (h,)).float().contiguous()
+        layers.append(lw)
+    embed = get("embed", (cfg.vocab_size, h)).contiguous()
+    return AttentionWeights(embed, layers, _norm(get, "final.norm", cfg), pad_pitch(embed))
+
+
+def random_getter(gen: torch.Generator, dtype: torch.dtype, device) -> Getter:
+    """Random tensors by name: linear maps N(0, 0.02), norm weights one, biases zero, dynamic-tanh scalars one."""
+    from .weights import _randn
+
+    def get(name: str, shape: tuple[int, ...]) -> torch.Tensor:
+        if len(shape) == 2:
+            return _randn(gen, shape, dtype, device)
+        return (torch.zeros if name.endswith(".b") else torch.ones)(shape, dtype=dtype, device=device)
+
+    return get

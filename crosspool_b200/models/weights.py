@@ -21,6 +21,7 @@ from .config import ModelConfig
 from ..utils.dtype import decode_dtype
 
 FFN_KEY = re.compile(r"^model\.layers\.(\d+)\.mlp\.")
+LAYERED_FFN_KEY = re.compile(r"^l(\d+)\.mlp\.")
 OPT_FFN_KEY = re.compile(r"^model\.decoder\.layers\.(\d+)\.fc[12]\.")
 
 
@@ -96,6 +97,10 @@ def random_attention_weights(cfg: ModelConfig, seed: int = 0, device="cpu", dtyp
                              ) -> AttentionWeights:
     dt = _dtype(cfg, dtype)
     gen = _generator(seed * 1000003 + 1, device)
+    if cfg.layered:
+        from .layered import layered_attention_weights, random_getter
+
+        return layered_attention_weights(cfg, random_getter(gen, dt, device), device, dt)
     embed = _randn(gen, (cfg.vocab_size, cfg.hidden_size), dt, device)
     layers = []
     if not cfg.gpu_attention_supported:
@@ -219,6 +224,13 @@ def random_ffn_layer(cfg: ModelConfig, layer: int, seed: int = 0, device="cpu", 
                                           ).contiguous()
                 w.router = w.extra["router_fp32"].to(dt)
         return w
+    if cfg.layered:
+        inter = cfg.layer_specs[layer].ff
+        if tp_size > 1:
+            raise NotImplementedError("a row-normalised activation needs the whole FFN row on one rank (FFN TP 1)")
+        w = FfnLayerWeights(_randn(gen, (inter, h), dt, device), _randn(gen, (h, inter), dt, device))
+        w.extra.update(gated=False, polynorm=(torch.tensor([1.0, 1.0, 1.0, 0.0], device=device) / 3, cfg.rms_norm_eps))
+        return w
     inter = cfg.intermediate_size
     gate_up = _randn(gen, (2 * inter, h), dt, device)
     down = _randn(gen, (h, inter), dt, device)
@@ -242,16 +254,18 @@ def quantize_ffn_layer_fp8(w: FfnLayerWeights) -> FfnLayerWeights:
 
 
 def random_ffn_weights(cfg: ModelConfig, seed: int = 0, device="cpu", dtype: torch.dtype | None = None,
-                       tp_rank: int = 0, tp_size: int = 1) -> list[FfnLayerWeights]:
-    return [random_ffn_layer(cfg, l, seed, device, dtype, tp_rank, tp_size) for l in range(cfg.num_layers)]
+                       tp_rank: int = 0, tp_size: int = 1) -> list[FfnLayerWeights | None]:
+    """One entry per layer; None for the layers of a layered decoder that have no FFN."""
+    return [None if cfg.layered and not cfg.layer_specs[l].ff else random_ffn_layer(cfg, l, seed, device, dtype, tp_rank, tp_size)
+            for l in range(cfg.num_layers)]
 
 
 # ------------------------------------------------------------------ safetensors (attention side)
 
 def attention_keys_filter(key: str) -> bool:
     """True for tensors the attention side loads: everything except the decoder FFNs (``model.layers.N.mlp.*``; for
-    OPT ``model.decoder.layers.N.fc1/fc2.*``)."""
-    return FFN_KEY.match(key) is None and OPT_FFN_KEY.match(key) is None
+    OPT ``model.decoder.layers.N.fc1/fc2.*``; for layered decoders ``lN.mlp.*``)."""
+    return FFN_KEY.match(key) is None and OPT_FFN_KEY.match(key) is None and LAYERED_FFN_KEY.match(key) is None
 
 
 def load_attention_from_safetensors(cfg: ModelConfig, model_dir: str | Path, device="cpu",
@@ -281,6 +295,16 @@ def load_attention_from_safetensors(cfg: ModelConfig, model_dir: str | Path, dev
     def opt(key: str) -> torch.Tensor | None:
         return get(key) if key in view.key_to_file else None
 
+    if cfg.layered:
+        from .layered import layered_attention_weights
+
+        def named(key: str, shape: tuple[int, ...]) -> torch.Tensor:
+            t = get(key)
+            if tuple(t.shape) != shape:
+                raise ValueError(f"{key} has shape {tuple(t.shape)}, the configuration gives {shape}")
+            return t
+
+        return layered_attention_weights(cfg, named, device, dt)
     if cfg.positions == "learned":
         return _load_opt_attention(cfg, get, opt)
     layers = []

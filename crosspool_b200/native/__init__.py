@@ -15,7 +15,7 @@ import ctypes as C
 import functools
 from pathlib import Path
 
-EXPECTED_ABI = 21
+EXPECTED_ABI = 22
 HERE = Path(__file__).resolve().parent
 
 
@@ -63,6 +63,10 @@ class GemmArgs(C.Structure):
         ("w_scale", C.c_void_p),
         ("x_scale", C.c_void_p),
         ("ld_xscale", C.c_int),
+        ("batch", C.c_int),
+        ("x_group_rows", C.c_int),
+        ("out_group_stride", C.c_int),
+        ("out_scale", C.c_float),
     ]
 
 
@@ -145,6 +149,7 @@ def kernels() -> C.CDLL:
     lib.xp_encode_tmap_2d.argtypes = [C.c_void_p, C.c_void_p, C.c_uint64, C.c_uint64, C.c_uint64, C.c_uint32,
                                       C.c_uint32]
     _declare_attention(lib)
+    _declare_mixers(lib)
     _declare_lane(lib)
     _declare_moe(lib)
     return lib
@@ -237,7 +242,52 @@ class PrefillAttnArgs(C.Structure):
         ("force_simple", C.c_int),
         ("status", C.c_void_p),
         ("total_q", C.c_int),
+        ("v_dim", C.c_int),
+        ("v_valid", C.c_int),
+        ("ld_out", C.c_int),
+        ("seq_starts", C.c_void_p),
+        ("gate", C.c_void_p),
+        ("ld_gate", C.c_int),
+        ("p_pair", C.c_int),
     ]
+
+
+def _struct(name: str, doc: str, **fields):
+    """A ctypes.Structure whose fields are given as ``ctype="space separated names"`` groups in ABI order, keyed
+    ``group_index_ctype``."""
+    types = {"ptr": C.c_void_p, "int": C.c_int, "float": C.c_float, "ptr8": C.c_void_p * 8}
+    decl = [(n, types[key.split("_", 1)[1]]) for key, names in fields.items() for n in names.split()]
+    return type(name, (C.Structure,), {"_fields_": decl, "__doc__": doc})
+
+
+# mixer_api.h
+ResidNormArgs = _struct("ResidNormArgs", "XpResidNormArgs", a_ptr="resid", b_ptr8="parts",
+                        c_ptr="gate ids table sel weight bias alpha out",
+                        d_int="rows hidden nparts ld_part ld_gate ld_out vocab kind", e_float="eps", f_int="f32")
+PolyNormArgs = _struct("PolyNormArgs", "XpPolyNormArgs", a_ptr="z coef out", b_int="rows cols ld_z ld_out", c_float="eps", d_int="f32")
+GatedRmsArgs = _struct("GatedRmsArgs", "XpGatedRmsArgs", a_ptr="o weight gate out", b_int="rows cols ld_o ld_gate ld_out", c_float="eps",
+                       d_int="f32")
+LatentPrepArgs = _struct("LatentPrepArgs", "XpLatentPrepArgs", a_ptr="proj norm_w freq positions slots cache q_plain q_abs q_exp",
+                         b_int="rows heads dim rot rot_dims kv_rank ld_proj q_off kv_off ld_cache qp_rows dim_p ld_abs dq_pad abs_rows",
+                         c_float="eps", d_int="f32")
+LatentAttnArgs = _struct("LatentAttnArgs", "XpLatentAttnArgs", a_ptr="q cache out gate row_seq positions slots block_table ws",
+                         b_int="rows heads kv_rank rot q_rows ld_q ld_cache ld_out ld_gate page_size max_blocks num_splits chunk_tokens",
+                         c_float="scale", d_int="f32 force_simt")
+LatentGatherArgs = _struct("LatentGatherArgs", "XpLatentGatherArgs", a_ptr="cache out block_table ctx_lens q_lens starts",
+                           b_int="n_seqs max_len page_size max_blocks ld_cache elem_bytes")
+LinearAttnArgs = _struct("LinearAttnArgs", "XpLinearAttnArgs",
+                         a_ptr="proj state decay decay_pow out positions slots state_slots q_starts q_lens ws",
+                         b_int="rows seqs seq0 max_q_len heads dim vdim ld_proj q_off k_off v_off ws_chunks f32")
+
+
+def _declare_mixers(lib: C.CDLL) -> None:
+    for fn, args in (("xp_resid_norm", ResidNormArgs), ("xp_polynorm", PolyNormArgs), ("xp_gated_rms", GatedRmsArgs),
+                     ("xp_latent_prep", LatentPrepArgs), ("xp_latent_attn", LatentAttnArgs), ("xp_latent_gather", LatentGatherArgs),
+                     ("xp_linear_attn_decode", LinearAttnArgs), ("xp_linear_attn_prefill", LinearAttnArgs)):
+        getattr(lib, fn).restype = C.c_int
+        getattr(lib, fn).argtypes = [C.POINTER(args), C.c_void_p]
+    lib.xp_gemm_f32.restype = C.c_int
+    lib.xp_gemm_f32.argtypes = [C.c_void_p] * 4 + [C.c_int] * 7 + [C.c_int64] * 3 + [C.c_float, C.c_void_p]
 
 
 def _declare_attention(lib: C.CDLL) -> None:
