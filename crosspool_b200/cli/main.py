@@ -3,6 +3,8 @@
     xpool daemon serve | check     control plane (exit 20 if a failure was recorded, else 0)
     xpool atnagent --device N      attention role for one GPU (hosts the Instances placed on it)
     xpool ffnagent --device N      FFN role for one GPU
+    xpool serve --model M          one GPU serves a model whole: engine, FFN in-stream, POST /generate
+    xpool generate --model M       the same engine, a few prompts of token ids, tokens on standard output
     xpool exec -- <cmd ...>        normalise device visibility, export daemon endpoint, exec the command
     xpool config dump              print the effective configuration
     xpool memory-profile           print the analytic device memory estimate per FFN device
@@ -38,6 +40,23 @@ def _parser() -> argparse.ArgumentParser:
     r.add_argument("--host", default="127.0.0.1")
     r.add_argument("--port", type=int, required=True)
     r.add_argument("--model", action="append", default=None, help="restrict to these models (default: every model with a listener)")
+    for name, what in (("serve", "serve one model whole on one GPU (FFN in-stream): POST /generate"),
+                       ("generate", "generate from prompts of token ids on one GPU and print the tokens as JSON lines")):
+        g = sub.add_parser(name, help=what)
+        g.add_argument("--model", required=True, help="checkpoint directory (config.json + safetensors) or preset name (random weights)")
+        g.add_argument("--dtype", default="bfloat16", choices=("bfloat16", "float32"))
+        g.add_argument("--device", type=int, default=0, dest="gpu")
+        g.add_argument("--max-batch", type=int, default=64)
+        g.add_argument("--max-seq-len", type=int, default=8192)
+        g.add_argument("--kv-tokens", type=int, default=0, help="cache capacity (default: max-batch sequences of max-seq-len)")
+        if name == "serve":
+            g.add_argument("--host", default="127.0.0.1")
+            g.add_argument("--port", type=int, required=True)
+        else:
+            g.add_argument("--ids", action="append", required=True, help="one prompt: token ids with commas between them (repeatable)")
+            g.add_argument("--max-new-tokens", type=int, default=16)
+            g.add_argument("--temperature", type=float, default=0.0)
+            g.add_argument("--seed", type=int, default=0)
     e = sub.add_parser("exec", help="run a command in the deployment's environment")
     e.add_argument("argv", nargs=argparse.REMAINDER)
     c = sub.add_parser("config", help="dump the resolved configuration; print the settings and supported-model references")
@@ -206,6 +225,10 @@ def main(argv: list[str] | None = None) -> int:
             return cmd_daemon_serve(ns) if ns.daemon_command == "serve" else cmd_daemon_check(ns)
         if ns.command == "exec":
             return cmd_exec(ns)
+        if ns.command in ("serve", "generate"):
+            from ..runtime import local_serving
+
+            return local_serving.serve(ns) if ns.command == "serve" else local_serving.generate(ns)
         if ns.command == "router":
             from ..runtime.dp_router import serve_router
 

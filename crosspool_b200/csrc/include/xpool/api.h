@@ -54,6 +54,7 @@ typedef struct XpGemmArgs {
    * [g * w_rows_per_group, + n_out) into out + g * out_group_stride (elements) */
   int batch, x_group_rows, out_group_stride;
   float out_scale;     /* multiplies the accumulator of epilogues 0 and 3; 0 = 1 */
+  int silu_cols;       /* epilogues 0 and 3: features below this are stored as silu(value) */
 } XpGemmArgs;
 
 typedef struct XpGemmPlan {

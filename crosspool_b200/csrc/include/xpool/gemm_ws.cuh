@@ -95,6 +95,7 @@ struct Problem {
   int batch;
   int x_group_rows;
   int out_group_stride;
+  int silu_cols;           // plain stores: features below this are stored as silu(value)
   float out_scale;         // multiplies the accumulator of the two plain store epilogues; 0 = 1
 };
 
@@ -464,6 +465,10 @@ __device__ __forceinline__ void epilogue_store16(const Problem& p, int f, int fb
     const float sc = p.out_scale == 0.f ? 1.f : p.out_scale;
 #pragma unroll
     for (int j = 0; j < 16; ++j) v[j] = fmaf(g[j], sc, bias);
+    if (f < p.silu_cols) {
+#pragma unroll
+      for (int j = 0; j < 16; ++j) v[j] = __fdividef(v[j], 1.f + __expf(-v[j]));
+    }
   }
   if (p.epilogue == kEpiStoreF32) {
     float* o = reinterpret_cast<float*>(p.out) + o0;
@@ -553,7 +558,7 @@ __device__ __forceinline__ bool epilogue_tile(const Problem& p, const TileCoord&
     if (p.splits == 1) {
 #pragma unroll
       for (int cc = 0; cc < kMaxBnF8 / 16; ++cc)
-        if (cc * 16 < p.bn && c.n0 + cc * 16 < c.row_end) epilogue_store16(p, f, fb, c.n0 + cc * 16, c.row_end, &acc[cc * 16], u, c.out_off);
+        if (cc * 16 < p.bn && c.n0 + cc * 16 < c.row_end) epilogue_store16(p, f, fb, c.n0 + cc * 16, c.row_end, &acc[cc * 16], u);
     } else {
       float* ws = p.ws + (static_cast<size_t>(c.mn) * p.splits + c.split) * acc_cols * kTileM;
 #pragma unroll
@@ -652,7 +657,7 @@ __device__ __forceinline__ bool epilogue_tile(const Problem& p, const TileCoord&
             }
           }
         }
-        epilogue_store16(p, f, fb, c.n0 + col, c.row_end, g, u, c.out_off);
+        epilogue_store16(p, f, fb, c.n0 + col, c.row_end, g, u);
       }
       if (ew == 0 && lane == 0) p.counters[c.mn] = 0;  // ready for the next call
     }

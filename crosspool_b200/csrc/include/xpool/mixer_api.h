@@ -101,21 +101,21 @@ typedef struct XpLatentGatherArgs {
   int n_seqs, max_len, page_size, max_blocks, ld_cache, elem_bytes;
 } XpLatentGatherArgs;
 
-/* Decayed linear attention S = decay S + k v^T, o = S^T q with silu on q, k, v; the state of sequence slot s is
+/* Decayed linear attention S = decay S + k v^T, o = S^T q; the state of sequence slot s is
  * state[s][heads][dim][vdim] in fp32. A sequence whose first row sits at position 0 starts from a zero state. */
 typedef struct XpLinearAttnArgs {
   const void* proj;      /* [rows, ld_proj]: q, k (heads x dim) and v (heads x vdim) at the three offsets */
   float* state;
   const float* decay;    /* [heads] */
-  const float* decay_pow;/* [heads, kChunk + 1]: decay^0 .. decay^kChunk */
+  const float* decay_pow;/* [heads, 65]: decay^0 .. decay^64 */
   float* out;            /* [rows, heads * vdim] fp32 */
   const int* positions;  /* [rows] */
   const int* slots;      /* [rows] KV slot of the row, < 0: padding row */
   const int* state_slots;/* [seqs] */
   const int* q_starts;   /* [seqs] prefill: first row */
   const int* q_lens;     /* [seqs] prefill: rows */
-  float* ws;             /* chunked prefill: chunk states */
-  int rows, seqs, seq0, max_q_len, heads, dim, vdim, ld_proj, q_off, k_off, v_off, ws_chunks;
+  int rows, seqs, heads, dim, vdim, ld_proj, q_off, k_off, v_off;
+  int force_sequential;
   int f32;
 } XpLinearAttnArgs;
 
@@ -127,9 +127,10 @@ int xp_latent_attn(const XpLatentAttnArgs* a, void* stream);
 int xp_latent_gather(const XpLatentGatherArgs* a, void* stream);
 int xp_linear_attn_decode(const XpLinearAttnArgs* a, void* stream);
 int xp_linear_attn_prefill(const XpLinearAttnArgs* a, void* stream);
-/* out[b][r][n] = sum_k x[b][r][k] w[b][n][k] (* out_scale) (+ bias) in true fp32 (no reduced-precision product). */
+/* out[b][r][n] = sum_k x[b][r][k] w[b][n][k] (* out_scale) (+ bias), silu below column silu_cols, in true fp32 (no
+ * reduced-precision product). */
 int xp_gemm_f32(const float* x, const float* w, const float* bias, float* out, int rows, int n, int k, int ldx, int ldw, int ldo,
-                int batch, int64_t sx, int64_t sw, int64_t so, float out_scale, void* stream);
+                int batch, int64_t sx, int64_t sw, int64_t so, float out_scale, int silu_cols, void* stream);
 
 #ifdef __cplusplus
 }

@@ -392,6 +392,7 @@ extern "C" int xp_gemm(const XpGemmArgs* a) {
   p.x_group_rows = a->x_group_rows;
   p.out_group_stride = a->out_group_stride;
   p.out_scale = a->out_scale;
+  p.silu_cols = a->silu_cols;
   if (a->tile_table != nullptr) {
     if (plan.splits != 1) return -13;
     plan.grid = plan.smem_bytes > 0 ? 148 : 148;

@@ -11,7 +11,7 @@ constexpr int kBM = 64, kBN = 64, kBK = 16;
 
 __global__ void __launch_bounds__(256)
 gemm_f32_kernel(const float* __restrict__ x, const float* __restrict__ w, const float* __restrict__ bias, float* __restrict__ out,
-                int rows, int n, int k, int ldx, int ldw, int ldo, int64_t sx, int64_t sw, int64_t so, float scale) {
+                int rows, int n, int k, int ldx, int ldw, int ldo, int64_t sx, int64_t sw, int64_t so, float scale, int silu_cols) {
   __shared__ float xs[kBK][kBM + 4];
   __shared__ float ws[kBK][kBN + 4];
   x += blockIdx.z * sx;
@@ -47,7 +47,10 @@ gemm_f32_kernel(const float* __restrict__ x, const float* __restrict__ w, const 
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int c = n0 + tc * 4 + j;
-      if (c < n) out[static_cast<int64_t>(r) * ldo + c] = fmaf(acc[i][j], scale, bias != nullptr ? bias[c] : 0.f);
+      if (c >= n) continue;
+      float v = fmaf(acc[i][j], scale, bias != nullptr ? bias[c] : 0.f);
+      if (c < silu_cols) v = v / (1.f + expf(-v));
+      out[static_cast<int64_t>(r) * ldo + c] = v;
     }
   }
 }
@@ -55,12 +58,12 @@ gemm_f32_kernel(const float* __restrict__ x, const float* __restrict__ w, const 
 }  // namespace
 
 extern "C" int xp_gemm_f32(const float* x, const float* w, const float* bias, float* out, int rows, int n, int k, int ldx, int ldw,
-                           int ldo, int batch, int64_t sx, int64_t sw, int64_t so, float out_scale, void* stream) {
+                           int ldo, int batch, int64_t sx, int64_t sw, int64_t so, float out_scale, int silu_cols, void* stream) {
   if (rows <= 0 || n <= 0 || batch <= 0) return 0;
   if (k <= 0) return -10;
   dim3 grid((n + kBN - 1) / kBN, (rows + kBM - 1) / kBM, batch);
   gemm_f32_kernel<<<grid, 256, 0, reinterpret_cast<cudaStream_t>(stream)>>>(x, w, bias, out, rows, n, k, ldx, ldw, ldo, sx, sw, so,
-                                                                           out_scale == 0.f ? 1.f : out_scale);
+                                                                           out_scale == 0.f ? 1.f : out_scale, silu_cols);
   cudaError_t e = cudaGetLastError();
   return e == cudaSuccess ? 0 : -100 - static_cast<int>(e);
 }

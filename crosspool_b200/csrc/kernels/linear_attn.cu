@@ -1,7 +1,8 @@
-// Decayed linear attention with a recurrent state per sequence and head: S <- decay S + k v^T, o = S^T q, with silu on the
-// projected q, k and v. The state is fp32 and lives in the sequence's slot, [dim][vdim] per head; a sequence whose first
+// Decayed linear attention with a recurrent state per sequence and head: S <- decay S + k v^T, o = S^T q (the projection's
+// epilogue has put q, k and v through silu). The state is fp32 and lives in the sequence's slot, [dim][vdim] per head; a sequence whose first
 // row sits at position 0 starts from zero, so slots are handed out without clearing them.
 //   linear_decode      one token per sequence: bound by reading and writing the state once
+//   linear_chunked     prefill in chunks of 64 tokens on the tensor cores, bf16 inputs
 //   linear_sequential  prefill as a loop over tokens, any sizes, fp32 or bf16 inputs
 #include "xpool/elem.cuh"
 #include "xpool/mixer_api.h"
@@ -9,8 +10,6 @@
 
 namespace xpool {
 namespace linear {
-
-using elem::silu;
 
 constexpr int kThreads = 256;
 
@@ -31,8 +30,8 @@ linear_decode_kernel(XpLinearAttnArgs a) {
   float* part = sm + 2 * a.dim;
   const T* proj = reinterpret_cast<const T*>(a.proj) + static_cast<size_t>(row) * a.ld_proj;
   for (int c = threadIdx.x; c < a.dim; c += kThreads) {
-    q_s[c] = silu(elem::ld(proj + a.q_off + h * a.dim + c));
-    k_s[c] = silu(elem::ld(proj + a.k_off + h * a.dim + c));
+    q_s[c] = elem::ld(proj + a.q_off + h * a.dim + c);
+    k_s[c] = elem::ld(proj + a.k_off + h * a.dim + c);
   }
   __syncthreads();
   const bool fresh = a.positions[row] == 0;
@@ -48,7 +47,7 @@ linear_decode_kernel(XpLinearAttnArgs a) {
       float v[N], acc[N];
       elem::ldv<N>(proj + a.v_off + h * a.vdim + c, v);
 #pragma unroll
-      for (int j = 0; j < N; ++j) v[j] = silu(v[j]), acc[j] = 0.f;
+      for (int j = 0; j < N; ++j) acc[j] = 0.f;
 #pragma unroll 8
       for (int i = gi; i < a.dim; i += groups) {
         float s[N];
@@ -87,7 +86,7 @@ template <typename T, int PER>
 __global__ void __launch_bounds__(kThreads)
 linear_sequential_kernel(XpLinearAttnArgs a) {
   extern __shared__ float sm[];            // q, k [kBatch][dim]; v [kBatch][32]; partial [kBatch][8][32]
-  const int h = blockIdx.y, seq = a.seq0 + blockIdx.z;
+  const int h = blockIdx.y, seq = blockIdx.z;
   const int n = a.q_lens[seq];
   if (n <= 0) return;
   const int r0 = a.q_starts[seq];
@@ -112,13 +111,13 @@ linear_sequential_kernel(XpLinearAttnArgs a) {
     for (int i = threadIdx.x; i < m * a.dim; i += kThreads) {
       const int t = i / a.dim, d = i - t * a.dim;
       const T* p = reinterpret_cast<const T*>(a.proj) + static_cast<size_t>(r0 + t0 + t) * a.ld_proj + h * a.dim + d;
-      q_s[i] = silu(elem::ld(p + a.q_off));
-      k_s[i] = silu(elem::ld(p + a.k_off));
+      q_s[i] = elem::ld(p + a.q_off);
+      k_s[i] = elem::ld(p + a.k_off);
     }
     for (int i = threadIdx.x; i < m * 32; i += kThreads) {
       const int t = i >> 5, cc = blockIdx.x * 32 + (i & 31);
-      v_s[i] = cc < a.vdim ? silu(elem::ld(reinterpret_cast<const T*>(a.proj) + static_cast<size_t>(r0 + t0 + t) * a.ld_proj + a.v_off +
-                                           h * a.vdim + cc))
+      v_s[i] = cc < a.vdim ? elem::ld(reinterpret_cast<const T*>(a.proj) + static_cast<size_t>(r0 + t0 + t) * a.ld_proj + a.v_off +
+                                      h * a.vdim + cc)
                            : 0.f;
     }
     __syncthreads();
@@ -155,6 +154,275 @@ linear_sequential_kernel(XpLinearAttnArgs a) {
   }
 }
 
+// ------------------------------------------------------------------------------------------ chunked prefill
+// CTA = (VS state columns, head, sequence); it walks the sequence in chunks of 64 tokens with the state in registers.
+// With p(n) = decay^n, for row i of a chunk of n tokens and the state S before it:
+//   o_i = sum_{j <= i} p(i - j) (q_i . k_j) v_j + p(i + 1) S^T q_i          (four warps, 16 rows each)
+//   S   <- p(n) S + sum_j k_j (p(n - 1 - j) v_j)^T                          (four warps, D / 4 rows of S each)
+// Decayed scores, decayed values and the state enter their products as bf16 pairs (high and low part), so everything
+// that belongs to the recurrence keeps at least 16 mantissa bits; the sums are fp32.
+//
+// mma.sync rather than tcgen05: the state has to be scaled and re-split between chunks, which from tensor memory costs a
+// round trip per chunk, and the kernel is bound by that dependency chain.
+constexpr int kChunk = 64;
+constexpr int kChunkThreads = 128;
+
+__device__ __forceinline__ void ldsm4(uint32_t addr, uint32_t (&r)[4]) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
+               : "r"(addr));
+}
+__device__ __forceinline__ void ldsm4t(uint32_t addr, uint32_t (&r)[4]) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
+               : "r"(addr));
+}
+__device__ __forceinline__ void mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile(
+      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+// (x, y) as a bf16 pair of packed values: hi + lo carries 16 mantissa bits
+__device__ __forceinline__ void split2(float x, float y, uint32_t& hi, uint32_t& lo) {
+  const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
+  const float2 f = __bfloat1622float2(h);
+  const __nv_bfloat162 l = __floats2bfloat162_rn(x - f.x, y - f.y);
+  hi = *reinterpret_cast<const uint32_t*>(&h);
+  lo = *reinterpret_cast<const uint32_t*>(&l);
+}
+
+template <int D, int VS>
+constexpr int chunk_smem_bytes() {
+  // q, k [2][64][D + 8]; v [2][64][VS + 8]; decayed v pair [2][64][VS + 8]; state pair [2][D][VS + 8]; powers
+  return (4 * kChunk * (D + 8) + 2 * kChunk * (VS + 8) + 2 * kChunk * (VS + 8) + 2 * D * (VS + 8)) * 2 + (kChunk + 1 + 3) * 4;
+}
+
+template <int D, int VS>
+__global__ void __launch_bounds__(kChunkThreads)
+linear_chunked_kernel(XpLinearAttnArgs a) {
+  extern __shared__ __align__(16) uint8_t smem[];
+  constexpr int PD = D + 8, PV = VS + 8;             // pitches: odd multiples of 16 bytes
+  constexpr int NV = VS / 8, MT = D / 64;            // value tiles; 16-row state tiles per warp
+  __nv_bfloat16* q_s = reinterpret_cast<__nv_bfloat16*>(smem);
+  __nv_bfloat16* k_s = q_s + 2 * kChunk * PD;
+  __nv_bfloat16* v_s = k_s + 2 * kChunk * PD;
+  __nv_bfloat16* vd_s = v_s + 2 * kChunk * PV;       // decayed values: high parts, low parts
+  __nv_bfloat16* st_s = vd_s + 2 * kChunk * PV;      // state: high parts, low parts
+  float* pw = reinterpret_cast<float*>(st_s + 2 * D * PV);
+  const int h = blockIdx.y, seq = blockIdx.z, c0 = blockIdx.x * VS;
+  const int n = a.q_lens[seq];
+  if (n <= 0) return;
+  const int r0 = a.q_starts[seq];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int g = lane >> 2, q4 = lane & 3;
+  const int chunks = (n + kChunk - 1) / kChunk;
+  const __nv_bfloat16* proj = reinterpret_cast<const __nv_bfloat16*>(a.proj);
+
+  // columns behind dim stay zero; nothing below writes them
+  if (a.dim < D) {
+    const int gap = (D - a.dim) / 8;
+    for (int i = threadIdx.x; i < 4 * kChunk * gap; i += kChunkThreads)
+      *reinterpret_cast<uint4*>(q_s + (i / gap) * PD + a.dim + (i % gap) * 8) = make_uint4(0, 0, 0, 0);
+  }
+  for (int i = threadIdx.x; i <= kChunk; i += kChunkThreads) pw[i] = a.decay_pow[h * (kChunk + 1) + i];
+
+  auto copy = [&](__nv_bfloat16* dst, const __nv_bfloat16* src, bool ok) {
+    const int sz = ok ? 16 : 0;
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(sm100::smem_u32(dst)), "l"(src), "r"(sz));
+  };
+  auto issue = [&](int c) {
+    if (c < chunks) {
+      const int b = c & 1, m = min(kChunk, n - c * kChunk);
+      const int per = a.dim / 8;
+      for (int i = threadIdx.x; i < kChunk * per; i += kChunkThreads) {
+        const int t = i / per, e = (i - t * per) * 8;
+        const bool ok = t < m;
+        const __nv_bfloat16* row = proj + static_cast<size_t>(r0 + c * kChunk + (ok ? t : 0)) * a.ld_proj + h * a.dim + e;
+        copy(q_s + (b * kChunk + t) * PD + e, row + a.q_off, ok);
+        copy(k_s + (b * kChunk + t) * PD + e, row + a.k_off, ok);
+      }
+      for (int i = threadIdx.x; i < kChunk * NV; i += kChunkThreads) {
+        const int t = i / NV, e = (i % NV) * 8;
+        const bool ok = t < m && c0 + e < a.vdim;
+        copy(v_s + (b * kChunk + t) * PV + e,
+             proj + static_cast<size_t>(r0 + c * kChunk + (t < m ? t : 0)) * a.ld_proj + a.v_off + h * a.vdim + (ok ? c0 + e : 0), ok);
+      }
+    }
+    asm volatile("cp.async.commit_group;");
+  };
+  issue(0);
+
+  // state: this warp's rows [warp * D / 4, + D / 4), columns c0 .. c0 + VS
+  float* S = a.state + (static_cast<size_t>(a.state_slots[seq]) * a.heads + h) * a.dim * a.vdim;
+  const bool fresh = a.positions[r0] == 0;
+  float s[MT][NV][4];
+  auto state_at = [&](int mt, int j, int e, int& d, int& c) {
+    d = warp * (D / 4) + mt * 16 + g + (e >> 1) * 8;
+    c = c0 + j * 8 + q4 * 2 + (e & 1);
+    return d < a.dim && c < a.vdim;
+  };
+#pragma unroll
+  for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+    for (int j = 0; j < NV; ++j)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        int d, c;
+        s[mt][j][e] = state_at(mt, j, e, d, c) && !fresh ? S[static_cast<size_t>(d) * a.vdim + c] : 0.f;
+      }
+  auto publish_state = [&]() {
+#pragma unroll
+    for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+      for (int j = 0; j < NV; ++j)
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+          uint32_t hi, lo;
+          split2(s[mt][j][2 * r], s[mt][j][2 * r + 1], hi, lo);
+          __nv_bfloat16* p = st_s + (warp * (D / 4) + mt * 16 + g + r * 8) * PV + j * 8 + q4 * 2;
+          *reinterpret_cast<uint32_t*>(p) = hi;
+          *reinterpret_cast<uint32_t*>(p + D * PV) = lo;
+        }
+  };
+  publish_state();
+
+  const uint32_t a_off = ((warp * 16 + (lane & 15)) * PD + (lane >> 4) * 8) * 2;                        // Q rows of this warp
+  const uint32_t b_off = (((lane & 7) + ((lane >> 4) << 3)) * PD + ((lane >> 3) & 1) * 8) * 2;          // K as [tokens][dims]
+  const uint32_t t_off = (((lane & 7) + ((lane >> 3) & 1) * 8) * PV + (lane >> 4) * 8) * 2;             // [k][n] operands, transposed
+  const uint32_t kt_off = (((lane & 7) + (lane >> 4) * 8) * PD + warp * (D / 4) + ((lane >> 3) & 1) * 8) * 2;  // K^T rows of this warp
+
+  for (int c = 0; c < chunks; ++c) {
+    const int b = c & 1, m = min(kChunk, n - c * kChunk);
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();                                 // chunk c landed, state published, buffers of chunk c - 1 free
+    issue(c + 1);
+    // decayed values of the state update
+    for (int i = threadIdx.x; i < kChunk * (VS / 2); i += kChunkThreads) {
+      const int t = i / (VS / 2), e = (i % (VS / 2)) * 2;
+      const float w = t < m ? pw[m - 1 - t] : 0.f;
+      const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(v_s + (b * kChunk + t) * PV + e));
+      uint32_t hi, lo;
+      split2(v.x * w, v.y * w, hi, lo);
+      *reinterpret_cast<uint32_t*>(vd_s + t * PV + e) = hi;
+      *reinterpret_cast<uint32_t*>(vd_s + (kChunk + t) * PV + e) = lo;
+    }
+    const uint32_t qb = sm100::smem_u32(q_s + b * kChunk * PD) + a_off;
+    const uint32_t kb = sm100::smem_u32(k_s + b * kChunk * PD);
+    const uint32_t vb = sm100::smem_u32(v_s + b * kChunk * PV) + t_off;
+    const uint32_t sb = sm100::smem_u32(st_s) + t_off;
+    float o[NV][4], os[NV][4], p[8][4];
+#pragma unroll
+    for (int j = 0; j < NV; ++j)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) o[j][e] = os[j][e] = 0.f;
+#pragma unroll
+    for (int j = 0; j < 8; ++j)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) p[j][e] = 0.f;
+    // scores of this warp's rows against tokens up to its own, and S^T q
+#pragma unroll 2
+    for (int ks = 0; ks < D / 16; ++ks) {
+      uint32_t qa[4];
+      ldsm4(qb + ks * 32, qa);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {                  // 16 tokens each
+        if (j <= warp) {
+          uint32_t kf[4];
+          ldsm4(kb + b_off + (j * 16 * PD + ks * 16) * 2, kf);
+          mma(p[2 * j], qa, kf[0], kf[1]);
+          mma(p[2 * j + 1], qa, kf[2], kf[3]);
+        }
+      }
+#pragma unroll
+      for (int j = 0; j < NV; j += 2) {
+        uint32_t hi[4], lo[4];
+        ldsm4t(sb + (ks * 16 * PV + j * 8) * 2, hi);
+        ldsm4t(sb + ((D + ks * 16) * PV + j * 8) * 2, lo);
+        mma(os[j], qa, hi[0], hi[1]);
+        mma(os[j + 1], qa, hi[2], hi[3]);
+        mma(os[j], qa, lo[0], lo[1]);
+        mma(os[j + 1], qa, lo[2], lo[3]);
+      }
+    }
+    const int i0 = warp * 16 + g;                    // rows i0 and i0 + 8 of the chunk
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      if (j <= warp) {
+        uint32_t ph[4], pl[4];
+#pragma unroll
+        for (int u = 0; u < 2; ++u) {
+          const int t = j * 16 + u * 8 + q4 * 2;
+          auto w = [&](int i, int tok) { return tok <= i ? pw[i - tok] : 0.f; };
+          split2(p[2 * j + u][0] * w(i0, t), p[2 * j + u][1] * w(i0, t + 1), ph[2 * u], pl[2 * u]);
+          split2(p[2 * j + u][2] * w(i0 + 8, t), p[2 * j + u][3] * w(i0 + 8, t + 1), ph[2 * u + 1], pl[2 * u + 1]);
+        }
+#pragma unroll
+        for (int v = 0; v < NV; v += 2) {
+          uint32_t vf[4];
+          ldsm4t(vb + (j * 16 * PV + v * 8) * 2, vf);
+          mma(o[v], ph, vf[0], vf[1]);
+          mma(o[v + 1], ph, vf[2], vf[3]);
+          mma(o[v], pl, vf[0], vf[1]);
+          mma(o[v + 1], pl, vf[2], vf[3]);
+        }
+      }
+    }
+    const float f0 = pw[i0 + 1], f1 = pw[i0 + 9 <= kChunk ? i0 + 9 : kChunk];
+#pragma unroll
+    for (int v = 0; v < NV; ++v) {
+      const int col = c0 + v * 8 + q4 * 2;
+#pragma unroll
+      for (int r = 0; r < 2; ++r) {
+        const int i = i0 + r * 8;
+        if (i < m && col < a.vdim) {                 // vdim is even
+          const float f = r ? f1 : f0;
+          *reinterpret_cast<float2*>(a.out + static_cast<size_t>(r0 + c * kChunk + i) * a.heads * a.vdim + h * a.vdim + col) =
+              make_float2(fmaf(f, os[v][2 * r], o[v][2 * r]), fmaf(f, os[v][2 * r + 1], o[v][2 * r + 1]));
+        }
+      }
+    }
+    __syncthreads();                                 // decayed values written; everyone is done with the published state
+    const float pn = pw[m];
+    const uint32_t db = sm100::smem_u32(vd_s) + t_off;
+#pragma unroll
+    for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+      for (int j = 0; j < NV; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) s[mt][j][e] *= pn;
+#pragma unroll
+    for (int kk = 0; kk < kChunk / 16; ++kk) {
+      uint32_t ka[MT][4];
+#pragma unroll
+      for (int mt = 0; mt < MT; ++mt) ldsm4t(kb + kt_off + (kk * 16 * PD + mt * 16) * 2, ka[mt]);
+#pragma unroll
+      for (int j = 0; j < NV; j += 2) {
+        uint32_t hi[4], lo[4];
+        ldsm4t(db + (kk * 16 * PV + j * 8) * 2, hi);
+        ldsm4t(db + ((kChunk + kk * 16) * PV + j * 8) * 2, lo);
+#pragma unroll
+        for (int mt = 0; mt < MT; ++mt) {
+          mma(s[mt][j], ka[mt], hi[0], hi[1]);
+          mma(s[mt][j + 1], ka[mt], hi[2], hi[3]);
+          mma(s[mt][j], ka[mt], lo[0], lo[1]);
+          mma(s[mt][j + 1], ka[mt], lo[2], lo[3]);
+        }
+      }
+    }
+    if (c + 1 < chunks) publish_state();
+  }
+#pragma unroll
+  for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+    for (int j = 0; j < NV; ++j)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        int d, c;
+        if (state_at(mt, j, e, d, c)) S[static_cast<size_t>(d) * a.vdim + c] = s[mt][j][e];
+      }
+}
+
 inline int done() {
   cudaError_t e = cudaGetLastError();
   return e == cudaSuccess ? 0 : -100 - static_cast<int>(e);
@@ -187,6 +455,23 @@ int launch_sequential(const XpLinearAttnArgs& a, cudaStream_t s) {
   return done();
 }
 
+template <int D, int VS>
+int launch_chunked(const XpLinearAttnArgs& a, cudaStream_t s) {
+  constexpr int kSmem = chunk_smem_bytes<D, VS>();
+  static_assert(kSmem <= 227 * 1024, "chunk buffers exceed the shared memory of an SM");
+  int rc = big_smem(linear_chunked_kernel<D, VS>, kSmem);
+  if (rc != 0) return rc;
+  linear_chunked_kernel<D, VS><<<dim3((a.vdim + VS - 1) / VS, a.heads, a.seqs), kChunkThreads, kSmem, s>>>(a);
+  return done();
+}
+
+template <int D>
+int launch_chunked_any(const XpLinearAttnArgs& a, cudaStream_t s) {
+  // narrow state slices while there are too few CTAs for the 148 SMs: the scores are recomputed per slice
+  if (a.heads * a.seqs * ((a.vdim + 31) / 32) < 148) return launch_chunked<D, 16>(a, s);
+  return launch_chunked<D, 32>(a, s);
+}
+
 template <typename T>
 int launch_sequential_any(const XpLinearAttnArgs& a, cudaStream_t s) {
   if (a.dim <= 64) return launch_sequential<T, 8>(a, s);
@@ -213,10 +498,17 @@ extern "C" int xp_linear_attn_decode(const XpLinearAttnArgs* a, void* stream) {
   return v ? launch_decode<__nv_bfloat16, 4>(*a, s) : launch_decode<__nv_bfloat16, 1>(*a, s);
 }
 
-// Sequences [seq0, seq0 + seqs) with q_lens[s] rows from q_starts[s].
+// Portion s: q_lens[s] rows from row q_starts[s].
 extern "C" int xp_linear_attn_prefill(const XpLinearAttnArgs* a, void* stream) {
   if (a->seqs <= 0) return 0;
   if (a->heads <= 0 || a->dim <= 0 || a->vdim <= 0) return -10;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
-  return a->f32 ? launch_sequential_any<float>(*a, s) : launch_sequential_any<__nv_bfloat16>(*a, s);
+  if (a->f32) return launch_sequential_any<float>(*a, s);
+  const bool chunked = !a->force_sequential && a->dim <= 256 && a->dim % 8 == 0 && a->vdim % 8 == 0 && a->ld_proj % 8 == 0 &&
+                       a->q_off % 8 == 0 && a->k_off % 8 == 0 && a->v_off % 8 == 0 && reinterpret_cast<uintptr_t>(a->proj) % 16 == 0 &&
+                       reinterpret_cast<uintptr_t>(a->out) % 8 == 0;
+  if (!chunked) return launch_sequential_any<__nv_bfloat16>(*a, s);
+  if (a->dim <= 64) return launch_chunked_any<64>(*a, s);
+  if (a->dim <= 128) return launch_chunked_any<128>(*a, s);
+  return launch_chunked<256, 16>(*a, s);
 }

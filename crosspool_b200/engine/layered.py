@@ -43,7 +43,6 @@ class RowBatch:
     n_seqs: int
     n_dec: int                           # leading rows that are one token each (= leading sequences)
     n_abs: int                           # leading rows of the absorbed form (decoded tokens, then short portions)
-    max_q: int                           # longest portion behind the decoded tokens
     max_len: int                         # bound on positions + 1 of the absorbed rows
     positions: torch.Tensor              # [rows]
     slots: torch.Tensor                  # [rows] cache row, -1: padding
@@ -97,7 +96,6 @@ class LayeredForward:
             self.v_exp = buf(self.ws_tokens * max(H * dv for H, _, dv, _ in shapes))
         if lin:
             self.o_lin = buf(cap * max(m.out_features for m in lin), torch.float32)
-        self.lin_ws = None
 
     # ------------------------------------------------------------------ mixers
     def _latent(self, l: int, lw: LayeredLayerWeights, m: LatentMixer, proj: torch.Tensor, out: torch.Tensor, b: RowBatch) -> None:
@@ -146,8 +144,7 @@ class LayeredForward:
             M.linear_attn_decode(proj[:b.n_dec], state, dec, pw, o[:b.n_dec], b.positions, b.slots, b.state_slots, **kw)
         if b.n_dec < b.n_seqs:
             s = slice(b.n_dec, b.n_seqs)
-            M.linear_attn_prefill(proj, state, dec, pw, o, b.positions, b.slots, b.state_slots[s], b.q_starts[s], b.q_lens[s], b.max_q,
-                                  ws=self.lin_ws, **kw)
+            M.linear_attn_prefill(proj, state, dec, pw, o, b.positions, b.slots, b.state_slots[s], b.q_starts[s], b.q_lens[s], **kw)
         M.gated_rms(o, lw.mix["norm"], proj[:, lw.offs["g"]:lw.offs["g"] + n], self.e.cfg.rms_norm_eps, out)
 
     # ------------------------------------------------------------------ layers
@@ -159,7 +156,7 @@ class LayeredForward:
         for l, lw in enumerate(self.layers):
             M.resid_norm(resid, lw.norm1, x, **pending)
             proj = self.proj[:rows * lw.offs["end"]].view(rows, lw.offs["end"])
-            gemm.linear(x, lw.proj, out=proj, bias=lw.proj_bias)
+            gemm.linear(x, lw.proj, out=proj, bias=lw.proj_bias, silu_cols=lw.silu_cols)
             m = lw.spec.mixer
             n = m.out_features
             out = self.mix_out[:rows * ceil8(n)].view(rows, ceil8(n))[:, :n]

@@ -47,6 +47,7 @@ class LayeredLayerWeights:
     norm2: NormParams | None = None
     rg2: torch.Tensor | None = None         # residual gate of the FFN
     rg2_bias: torch.Tensor | None = None
+    silu_cols: int = 0                      # leading columns of the product that are stored through silu
 
 
 def _fuse(sections: list[tuple[str, torch.Tensor]]) -> tuple[torch.Tensor, dict[str, int]]:
@@ -120,6 +121,8 @@ def layered_attention_weights(cfg: ModelConfig, get: Getter, device, dtype: torc
         if spec.ff:
             lw.norm2 = _norm(get, p + ".norm2", cfg)
             lw.rg2, lw.rg2_bias = pad_pitch(get(p + ".rg2", (h, h))), get(p + ".rg2.b", (h,)).float().contiguous()
+        if isinstance(m, LinearMixer):
+            lw.silu_cols = offs["g"]            # q, k and v
         layers.append(lw)
     embed = get("embed", (cfg.vocab_size, h)).contiguous()
     return AttentionWeights(embed, layers, _norm(get, "final.norm", cfg), pad_pitch(embed))

@@ -27,9 +27,20 @@ class ArchitectureSupport:
     gpu_attention: bool                # the repository's own GPU attention engine runs it
     engine_adapter: bool               # a serving-engine shim adapter exists (attention in the external engine)
     quantization: tuple[str, ...]
+    ffn_tier: bool = True              # FFN devices (Lanes) serve it; False: one GPU, the FFN in the engine's own stream
+    library: bool = True               # a model class of the transformers library exists (engine processes, CPU oracle parity)
+
+
+_SEGIRAX_PROBE = {
+    "architecture": "Segirax", "vocab": 256, "width": 64, "norm": {"eps": 1e-6}, "logit_scale": 1.0,
+    "layers": [{"type": "lightning", "mixer": {"heads": 1, "dim": 16, "vdim": 16, "decay": [0.9]}, "mlp": {"kind": "dense", "ff": 128}},
+               {"type": "latent_attention", "mlp": None,
+                "mixer": {"heads": 2, "dim": 16, "rot_dim": 8, "vdim": 16, "kv_rank": 32, "scale": 0.2, "rot": {"dims": 8, "base": 1e4}}}]}
 
 
 def _probe(arch: str) -> dict:
+    if arch == "Segirax":
+        return _SEGIRAX_PROBE
     cfg = {k: v for k, v in _PROBE.items() if arch in _LATENT or not k.startswith(("kv_lora", "qk_", "v_head"))}
     if not arch.startswith("GptOss"):
         cfg.pop("sliding_window")
@@ -39,6 +50,9 @@ def _probe(arch: str) -> dict:
 
 
 def _attention_form(c: mc.ModelConfig) -> str:
+    if c.layered:
+        return ("per layer: latent attention (rotate-half rotary, output gate) or decayed linear attention; dynamic tanh norms, "
+                "gated fp32 residual")
     if c.mla is not None:
         return "latent attention (MLA), interleaved rotary pairs, YaRN"
     parts = ["grouped-query" if c.num_kv_heads != c.num_q_heads else "multi-head"]
@@ -102,7 +116,7 @@ def supported_architectures() -> list[ArchitectureSupport]:
             (("block fp8 checkpoints (expanded to bf16 for the Lanes; stored codes feed the decode-size fp8 GEMM)",)
              if kinds == ("dense",) and c.hidden_act == "silu" else ())
         rows.append(ArchitectureSupport(arch, kinds, _ffn_features(spec), _attention_form(c), c.gpu_attention_supported,
-                                        arch in with_adapter, quant))
+                                        arch in with_adapter, quant, ffn_tier=not c.layered, library=not c.layered))
     return rows
 
 
@@ -111,6 +125,7 @@ def support_markdown() -> str:
              "library-attention engine process | CPU deployment and oracle | weight formats |",
              "| --- | --- | --- | --- | --- | --- | --- | --- | --- |"]
     for r in supported_architectures():
-        lines.append(f"| `{r.architecture}` | {' + '.join(r.ffn_kinds)} | {r.ffn_features} | {r.attention_form} | "
-                     f"{'yes' if r.gpu_attention else 'no'} | {'yes' if r.engine_adapter else 'no'} | yes | yes | {', '.join(r.quantization)} |")
+        lib, tier = "yes" if r.library else "no", "" if r.ffn_tier else " (in-stream, one GPU: `xpool serve`)"
+        lines.append(f"| `{r.architecture}` | {' + '.join(r.ffn_kinds)}{tier} | {r.ffn_features} | {r.attention_form} | "
+                     f"{'yes' if r.gpu_attention else 'no'} | {'yes' if r.engine_adapter else 'no'} | {lib} | {lib} | {', '.join(r.quantization)} |")
     return "\n".join(lines) + "\n"

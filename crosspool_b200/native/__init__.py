@@ -67,6 +67,7 @@ class GemmArgs(C.Structure):
         ("x_group_rows", C.c_int),
         ("out_group_stride", C.c_int),
         ("out_scale", C.c_float),
+        ("silu_cols", C.c_int),
     ]
 
 
@@ -276,8 +277,8 @@ LatentAttnArgs = _struct("LatentAttnArgs", "XpLatentAttnArgs", a_ptr="q cache ou
 LatentGatherArgs = _struct("LatentGatherArgs", "XpLatentGatherArgs", a_ptr="cache out block_table ctx_lens q_lens starts",
                            b_int="n_seqs max_len page_size max_blocks ld_cache elem_bytes")
 LinearAttnArgs = _struct("LinearAttnArgs", "XpLinearAttnArgs",
-                         a_ptr="proj state decay decay_pow out positions slots state_slots q_starts q_lens ws",
-                         b_int="rows seqs seq0 max_q_len heads dim vdim ld_proj q_off k_off v_off ws_chunks f32")
+                         a_ptr="proj state decay decay_pow out positions slots state_slots q_starts q_lens",
+                         b_int="rows seqs heads dim vdim ld_proj q_off k_off v_off force_sequential f32")
 
 
 def _declare_mixers(lib: C.CDLL) -> None:
@@ -287,7 +288,7 @@ def _declare_mixers(lib: C.CDLL) -> None:
         getattr(lib, fn).restype = C.c_int
         getattr(lib, fn).argtypes = [C.POINTER(args), C.c_void_p]
     lib.xp_gemm_f32.restype = C.c_int
-    lib.xp_gemm_f32.argtypes = [C.c_void_p] * 4 + [C.c_int] * 7 + [C.c_int64] * 3 + [C.c_float, C.c_void_p]
+    lib.xp_gemm_f32.argtypes = [C.c_void_p] * 4 + [C.c_int] * 7 + [C.c_int64] * 3 + [C.c_float, C.c_int, C.c_void_p]
 
 
 def _declare_attention(lib: C.CDLL) -> None:

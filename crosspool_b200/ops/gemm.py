@@ -120,7 +120,7 @@ def tile_weight(w: torch.Tensor) -> TiledWeight:
 
 
 def _args(x, w, out, *, n_out, rows, epilogue, dual=0, up_offset=0, bias=None, resid=None, splits=0, bn=0,
-          num_sms=0, evict_first=None, gate_limit=0.0, up_add=0.0, act_alpha=0.0, out_scale=0.0) -> native.GemmArgs:
+          num_sms=0, evict_first=None, gate_limit=0.0, up_add=0.0, act_alpha=0.0, out_scale=0.0, silu_cols=0) -> native.GemmArgs:
     tiled = isinstance(w, TiledWeight)
     assert x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16
     assert x.stride(-1) == 1 and out.stride(-1) == 1 and (tiled or w.stride(-1) == 1)
@@ -160,6 +160,7 @@ def _args(x, w, out, *, n_out, rows, epilogue, dual=0, up_offset=0, bias=None, r
     a.up_add = up_add
     a.act_alpha = act_alpha
     a.out_scale = out_scale
+    a.silu_cols = silu_cols
     # decode-size calls leave room for a second kernel on the SM (the co-located Instance's attention)
     small = w.shape[0] * k * 2 <= DECODE_SMALL_WEIGHT_BYTES
     a.smem_limit = DECODE_SMEM_LIMIT if rows <= DECODE_ROWS and small else 0
@@ -183,9 +184,9 @@ def plan_shape(n_out: int, k: int, rows: int, dual: int = 0, num_sms: int = 148,
 
 def linear(x: torch.Tensor, w: torch.Tensor, *, out: torch.Tensor | None = None, bias: torch.Tensor | None = None,
            resid: torch.Tensor | None = None, out_fp32: bool = False, splits: int = 0, bn: int = 0,
-           num_sms: int = 0, evict_first: bool | None = None, out_scale: float = 0.0) -> torch.Tensor:
+           num_sms: int = 0, evict_first: bool | None = None, out_scale: float = 0.0, silu_cols: int = 0) -> torch.Tensor:
     """``x[rows, k] @ w[n, k].T`` (* ``out_scale`` unless 0) (+ fp32 ``bias``) (+ ``resid``) on the tcgen05 kernel; fp32
-    operands run the plain fp32 kernel. Any ``n`` and ``k``; bf16 row pitches must be multiples of 16 bytes."""
+    operands run the plain fp32 kernel. The first ``silu_cols`` features are stored as ``silu(value)``. Any ``n`` and ``k``; bf16 row pitches must be multiples of 16 bytes."""
     x2 = x.reshape(-1, x.shape[-1])
     rows, n = x2.shape[0], w.shape[0]
     if x.dtype == torch.float32:
@@ -193,23 +194,23 @@ def linear(x: torch.Tensor, w: torch.Tensor, *, out: torch.Tensor | None = None,
             raise ValueError("the fp32 product has no residual epilogue")
         if out is None:
             out = torch.empty(rows, n, dtype=torch.float32, device=x.device)
-        _linear_f32(x2, w, out, bias, out_scale)
+        _linear_f32(x2, w, out, bias, out_scale, silu_cols)
         return out.reshape(*x.shape[:-1], n) if x.dim() != 2 else out
     if out is None:
         out = torch.empty(rows, n, dtype=torch.float32 if out_fp32 else torch.bfloat16, device=x.device)
     epi = EPI_STORE_F32 if out.dtype == torch.float32 else (EPI_RESIDUAL if resid is not None else EPI_STORE)
     a = _args(x2, w, out, n_out=n, rows=rows, epilogue=epi, bias=bias, resid=resid, splits=splits, bn=bn,
-              num_sms=num_sms, evict_first=evict_first, out_scale=out_scale)
+              num_sms=num_sms, evict_first=evict_first, out_scale=out_scale, silu_cols=silu_cols)
     native.check(native.kernels().xp_gemm(C.byref(a)), "xp_gemm")
     return out.reshape(*x.shape[:-1], n) if x.dim() != 2 else out
 
 
-def _linear_f32(x, w, out, bias, out_scale=0.0, rows=None, n=None, batch=1, sx=0, sw=0, so=0) -> None:
+def _linear_f32(x, w, out, bias, out_scale=0.0, silu_cols=0, rows=None, n=None, batch=1, sx=0, sw=0, so=0) -> None:
     assert w.dtype == torch.float32 and out.dtype == torch.float32 and x.stride(-1) == w.stride(-1) == out.stride(-1) == 1
     native.check(native.kernels().xp_gemm_f32(
         x.data_ptr(), w.data_ptr(), bias.data_ptr() if bias is not None else None, out.data_ptr(),
         x.shape[0] if rows is None else rows, w.shape[0] if n is None else n, x.shape[-1], x.stride(-2), w.stride(-2), out.stride(-2),
-        batch, sx, sw, so, out_scale, torch.cuda.current_stream(x.device).cuda_stream), "xp_gemm_f32")
+        batch, sx, sw, so, out_scale, silu_cols, torch.cuda.current_stream(x.device).cuda_stream), "xp_gemm_f32")
 
 
 def linear_batched(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, out_group_stride: int) -> torch.Tensor:

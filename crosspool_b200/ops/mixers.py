@@ -218,10 +218,10 @@ def linear_attn_decode(proj, state, decay, decay_pow, out, positions, slots, sta
     native.check(native.kernels().xp_linear_attn_decode(C.byref(a), _stream(proj)), "xp_linear_attn_decode")
 
 
-def linear_attn_prefill(proj, state, decay, decay_pow, out, positions, slots, state_slots, q_starts, q_lens, max_q: int, *, heads: int,
-                        dim: int, vdim: int, offs: tuple[int, int, int], ws: torch.Tensor | None = None) -> None:
+def linear_attn_prefill(proj, state, decay, decay_pow, out, positions, slots, state_slots, q_starts, q_lens, *, heads: int,
+                        dim: int, vdim: int, offs: tuple[int, int, int], force_sequential: bool = False) -> None:
     """Portions of sequences: portion i covers rows ``q_starts[i] .. + q_lens[i]`` and continues state ``state_slots[i]``."""
     a = _linear_args(proj, state, decay, decay_pow, out, positions, slots, state_slots, heads, dim, vdim, offs)
-    a.q_starts, a.q_lens, a.seqs, a.max_q_len = q_starts.data_ptr(), q_lens.data_ptr(), q_lens.shape[0], max_q
-    a.rows, a.ws = proj.shape[0], _ptr(ws)
+    a.q_starts, a.q_lens, a.seqs = q_starts.data_ptr(), q_lens.data_ptr(), q_lens.shape[0]
+    a.rows, a.force_sequential = proj.shape[0], int(force_sequential)
     native.check(native.kernels().xp_linear_attn_prefill(C.byref(a), _stream(proj)), "xp_linear_attn_prefill")

@@ -412,6 +412,8 @@ class FfnRankRuntime:
     def add_instance(self, place: InstancePlacement, tp_rank: int, layers: tuple[int, int] | None = None) -> FfnInstanceState:
         """``layers``: the half-open layer range this rank holds (layer-split placements); other layers get no
         weights and an invocation naming them is refused."""
+        if place.cfg.layered:
+            raise NotImplementedError(f"{place.cfg.architecture}: Lanes run gated and MoE FFNs; a layered decoder's FFNs run in-stream (xpool serve)")
         lay = ffn_slot_layout(place)
         slot = PeerBuffer(lay.total_bytes)
         cfg = place.cfg

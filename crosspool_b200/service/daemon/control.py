@@ -218,6 +218,8 @@ class ControlPlane:
             return self._model_demand(model_id)
         m = self.config.model(model_id)
         cfg = self.config.model_shape(model_id)
+        if cfg.layered:
+            raise DaemonError("invalid", f"{model_id}: {cfg.architecture} is served whole on one GPU (xpool serve), not by an FFN tier")
         regs = [r.payload for (mid, _), r in self.instances.items() if mid == model_id]
         rows = max([max(p.ffn_profile.max_prefill_rows, p.ffn_profile.max_decode_rows) for p in regs] or [1])
         inter = cfg.moe_intermediate_size * max(1, cfg.num_experts_per_tok) if cfg.is_moe else cfg.intermediate_size

@@ -28,7 +28,8 @@ def test_supported_models_page_is_what_the_adapters_and_engines_implement():
     rows = {r.architecture: r for r in supported_architectures()}
     assert set(rows) == set(adapters.ADAPTERS)
     assert rows["Qwen3ForCausalLM"].gpu_attention and not rows["DeepseekV2ForCausalLM"].gpu_attention
-    assert all(r.engine_adapter for r in rows.values())
+    assert all(r.engine_adapter for r in rows.values() if r.library)
+    assert rows["Segirax"].gpu_attention and not rows["Segirax"].ffn_tier
 
 
 def test_every_page_of_the_index_exists_and_commands_named_in_the_docs_parse():
@@ -39,7 +40,7 @@ def test_every_page_of_the_index_exists_and_commands_named_in_the_docs_parse():
 
     p = _parser()
     for argv in (["config", "dump"], ["config", "reference"], ["config", "models"], ["daemon", "check"], ["daemon", "serve"],
-                 ["atnagent", "--device", "0"], ["ffnagent", "--device", "1"], ["memory-profile", "--calibrate", "--out", "p.json"]):
+                 ["serve", "--model", "m", "--port", "1"], ["generate", "--model", "m", "--ids", "1,2"], ["atnagent", "--device", "0"], ["ffnagent", "--device", "1"], ["memory-profile", "--calibrate", "--out", "p.json"]):
         p.parse_args(argv)
 
 
