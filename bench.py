@@ -25,7 +25,8 @@ when an SLO is missed or the correctness gate (logits against an oracle engine) 
 ``--impl baseline`` runs the same deployment and workload with the FFN tier built from library calls (NCCL
 broadcast / reduce, cuBLAS GEMMs, unfused SwiGLU). ``--impl reference`` reports why the reference itself cannot
 run here. ``--decode-only`` runs the steady-state decode replay benchmark instead (every Instance at a full
-running batch, no arrivals), a kernel-level figure.
+running batch, no arrivals), a kernel-level figure. ``--layered`` measures layered decoders (per-layer mixers:
+latent attention, decayed linear attention) beside the closest classic model of equal size.
 """
 
 from __future__ import annotations
@@ -54,6 +55,8 @@ def parse_args(argv=None):
     ap.add_argument("--layers", type=int, default=0, help="debug only: truncate the models (marks the result invalid)")
     ap.add_argument("--lanes", type=int, default=2, help="Executor Lanes per FFN device (multi-GPU only)")
     ap.add_argument("--policy", default="fifo", choices=["fifo", "random", "slo"], help="Lane scheduling policy")
+    ap.add_argument("--layered", action="store_true",
+                    help="layered decoders beside the closest classic model of equal size, rates and kernels (one GPU)")
     # steady-state decode replay (kernel-level)
     ap.add_argument("--decode-only", action="store_true")
     ap.add_argument("--batch", type=int, default=256, help="decode-only: in-flight requests per Instance")
@@ -103,6 +106,11 @@ def main(argv=None) -> int:
             print(json.dumps({"impl": "reference", "unavailable": REFERENCE_UNAVAILABLE}), flush=True)
         return 0
     world = int(os.environ.get("WORLD_SIZE", "1"))
+    if args.layered:
+        from crosspool_b200.bench import layered
+
+        print(json.dumps(layered.run(args.steps, max(3, args.warmup), args.layers or 8)))
+        return 0
     if args.decode_only:
         if args.gpus == 1 and world == 1:
             print(json.dumps(run_decode_only_single_gpu(args)))
