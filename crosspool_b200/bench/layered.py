@@ -127,7 +127,7 @@ def kernel_table(classic: ModelConfig, cfg: ModelConfig, timer: Timer, batch: in
     cache = rnd(batch * blocks, 64, 1, lat.cache_width)
     q, o = rnd(H, batch, lat.cache_width), torch.empty(H, batch, R, dtype=bf, device=dev)
     gate = rnd(batch, H)
-    splits, chunk = M.latent_attn_plan(batch, H, CONTEXT)
+    splits, chunk = M.latent_attn_plan(batch, H, CONTEXT, lat.cache_width)
     ws = torch.empty(batch * H * splits * (R + 2), device=dev)
     add(f"latent decode b{batch}", lambda: M.latent_attn(q, cache, o, table, pos, slots, kv_rank=R, rot=r, scale=lat.scale, gate=gate,
                                                         num_splits=splits, chunk_tokens=chunk, ws=ws),
@@ -152,7 +152,10 @@ def kernel_table(classic: ModelConfig, cfg: ModelConfig, timer: Timer, batch: in
     # ---- attention and recurrence, one prefill chunk of one sequence
     T = CHUNK
     p0, one, st = torch.arange(T, dtype=torch.int32, device=dev), i32([0]), i32([T])
-    add(f"linear prefill {T}", lambda: M.linear_attn_prefill(pl, state, dec, pw, ol, p0, p0, one, one, st, **kw),
+    segs, seg_tokens = M.linear_attn_plan(1, Hl, dl, vl, T)
+    lws = torch.empty(M.linear_attn_ws_elems(dl, vl), device=dev)
+    add(f"linear prefill {T}", lambda: M.linear_attn_prefill(pl, state, dec, pw, ol, p0, p0, one, one, st, segs=segs, seg_tokens=seg_tokens,
+                                                            ws=lws, **kw),
         T * Hl * (2 * dl + vl) * 2 + ol.numel() * 4, 2.0 * T * Hl * (2 * dl * vl + 64 / 2 * (dl + vl)), "paged prefill")
     dq, dv = M.expanded_shape(lat.dim, r, lat.vdim)
     qe, ke, ve = rnd(T, H, dq), rnd(T, H, dq), rnd(T, H, dv)

@@ -114,8 +114,10 @@ typedef struct XpLinearAttnArgs {
   const int* state_slots;/* [seqs] */
   const int* q_starts;   /* [seqs] prefill: first row */
   const int* q_lens;     /* [seqs] prefill: rows */
+  float* ws;             /* [seqs, heads, segs, dim, vdim] states between segments, segs > 1 */
   int rows, seqs, heads, dim, vdim, ld_proj, q_off, k_off, v_off;
   int force_sequential;
+  int segs, seg_tokens;  /* chunked prefill: segments of a portion that run at the same time (multiples of 64 tokens) */
   int f32;
 } XpLinearAttnArgs;
 

@@ -2,14 +2,14 @@
 // as key (all of it) and as value (its latent columns). Kernels:
 //   latent_prep       per token: latent RMS norm, rotary on the shared key part and on every query head, cache write,
 //                     query layouts of the two forms below
-//   latent_attn_tc    absorbed form (queries already multiplied into the latent space), one token row and up to 16 heads
+//   latent_attn_tc    absorbed form (queries already multiplied into the latent space), one token row and up to 32 heads
 //                     per CTA, split over the sequence: cp.async ring of 64-token tiles, ldmatrix + mma.m16n8k16, the
 //                     probabilities carried as a bf16 pair (high and low part). Bound by reading the cache once.
 //   latent_attn_simt  the same in plain FMAs for any sizes and for fp32
 //   latent_gather     dense copy of a sequence's cached rows, the input of the expanded form (keys and values per head,
 //                     chunked prefill on the tcgen05 kernel of attn_prefill_umma.cu)
 //
-// mma.sync rather than tcgen05 in the absorbed decode kernel: 16 query rows per cache row are 4 * 16 flop per loaded
+// mma.sync rather than tcgen05 in the absorbed decode kernel: 16 or 32 query rows per cache row are 64 or 128 flop per loaded
 // element, far below the tensor roofline, and a UMMA tile needs 64 or 128 query rows.
 #include <math_constants.h>
 
@@ -24,8 +24,9 @@ constexpr float kLog2e = 1.4426950408889634f;
 
 // ------------------------------------------------------------------------------------------ prep
 constexpr int kPrepThreads = 256;
+constexpr int kPrepHeads = 8;              // heads per CTA (grid y): one per warp
 
-template <typename T>
+template <typename T, int VEC>
 __global__ void __launch_bounds__(kPrepThreads)
 latent_prep_kernel(XpLatentPrepArgs a) {
   extern __shared__ float cs[];            // cos | sin, rot_dims / 2 each
@@ -53,7 +54,7 @@ latent_prep_kernel(XpLatentPrepArgs a) {
   };
 
   const int slot = a.slots[row];
-  if (slot >= 0) {
+  if (slot >= 0 && blockIdx.y == 0) {
     const T* kv = proj + a.kv_off;
     float ss = 0.f;
     for (int c = threadIdx.x; c < a.kv_rank; c += kPrepThreads) {
@@ -70,29 +71,36 @@ latent_prep_kernel(XpLatentPrepArgs a) {
     }
   }
 
+  // queries: one warp per head
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int dh = a.dim + a.rot;
-  const T* q = proj + a.q_off;
-  if (row < a.abs_rows) {
-    T* qp = reinterpret_cast<T*>(a.q_plain);
-    for (int i = threadIdx.x; i < a.heads * a.dim_p; i += kPrepThreads) {
-      const int h = i / a.dim_p, c = i - h * a.dim_p;
-      elem::st(qp + (static_cast<size_t>(h) * a.qp_rows + row) * a.dim_p + c, c < a.dim ? elem::ld(q + h * dh + c) : 0.f);
+  for (int h = blockIdx.y * kPrepHeads + warp; h < min(a.heads, static_cast<int>(blockIdx.y + 1) * kPrepHeads); h += kPrepThreads / 32) {
+    const T* q = proj + a.q_off + h * dh;
+    T *plain, *rot;
+    int plain_end, rot_end;                 // columns past the vector's own hold zeros
+    if (row < a.abs_rows) {
+      const size_t r = static_cast<size_t>(h) * a.qp_rows + row;
+      plain = reinterpret_cast<T*>(a.q_plain) + r * a.dim_p;
+      rot = reinterpret_cast<T*>(a.q_abs) + r * a.ld_abs + a.kv_rank;
+      plain_end = a.dim_p;
+      rot_end = a.ld_abs - a.kv_rank;
+    } else {
+      plain = reinterpret_cast<T*>(a.q_exp) + (static_cast<size_t>(row) * a.heads + h) * a.dq_pad;
+      rot = plain + a.dim;
+      plain_end = a.dim;
+      rot_end = a.dq_pad - a.dim;
     }
-    T* qa = reinterpret_cast<T*>(a.q_abs);
-    const int tail = a.ld_abs - a.kv_rank;
-    for (int i = threadIdx.x; i < a.heads * tail; i += kPrepThreads) {
-      const int h = i / tail, c = i - h * tail;
-      elem::st(qa + (static_cast<size_t>(h) * a.qp_rows + row) * a.ld_abs + a.kv_rank + c, c < a.rot ? rotated(q + h * dh + a.dim, c) : 0.f);
+    if (VEC == 4) {
+      for (int c = lane * 4; c < a.dim; c += 128) {
+        float v[4];
+        elem::ldv<4>(q + c, v);
+        elem::stv<4>(plain + c, v);
+      }
+      for (int c = a.dim + lane; c < plain_end; c += 32) elem::st(plain + c, 0.f);
+    } else {
+      for (int c = lane; c < plain_end; c += 32) elem::st(plain + c, c < a.dim ? elem::ld(q + c) : 0.f);
     }
-  } else {
-    T* qe = reinterpret_cast<T*>(a.q_exp) + static_cast<size_t>(row) * a.heads * a.dq_pad;
-    for (int i = threadIdx.x; i < a.heads * a.dq_pad; i += kPrepThreads) {
-      const int h = i / a.dq_pad, c = i - h * a.dq_pad;
-      float v = 0.f;
-      if (c < a.dim) v = elem::ld(q + h * dh + c);
-      else if (c < dh) v = rotated(q + h * dh + a.dim, c - a.dim);
-      elem::st(qe + i, v);
-    }
+    for (int c = lane; c < rot_end; c += 32) elem::st(rot + c, c < a.rot ? rotated(q + a.dim, c) : 0.f);
   }
 }
 
@@ -194,13 +202,14 @@ struct TcLayout {
   int total;
 };
 
-__host__ __device__ inline TcLayout tc_layout(int dk16, int vcols) {
+__host__ __device__ inline TcLayout tc_layout(int dk16, int vcols, int hg) {
   TcLayout L;
   const int w = dk16 > vcols ? dk16 : vcols;
   L.pitch = w + 8;
   L.stage_bytes = kTile * L.pitch * 2;
-  L.q_bytes = 16 * L.pitch * 2;
-  const int fixed = L.q_bytes + 2 * 16 * kPPitch * 2 + 2 * 16 * kTile * 4 + 3 * 16 * 4;
+  const int m = 16 * hg;
+  L.q_bytes = m * L.pitch * 2;
+  const int fixed = L.q_bytes + 2 * m * kPPitch * 2 + 2 * m * kTile * 4 + 3 * m * 4;
   int st = (100 * 1024 - fixed) / L.stage_bytes;     // two CTAs per SM when the rows are short
   if (st < 2) st = 2;
   if (st > 4) st = 4;
@@ -209,26 +218,27 @@ __host__ __device__ inline TcLayout tc_layout(int dk16, int vcols) {
   return L;
 }
 
-// NT: 8-column tiles of the latent per warp (kv_rank <= 64 * NT).
-template <int NT>
+// NT: 8-column tiles of the latent per warp (kv_rank <= 64 * NT). HG: groups of 16 heads that share a CTA's tiles.
+template <int NT, int HG>
 __global__ void __launch_bounds__(kTcThreads)
 latent_attn_tc_kernel(XpLatentAttnArgs a) {
   extern __shared__ __align__(16) uint8_t smem[];
-  const int split = blockIdx.x, h0 = blockIdx.y * 16, row = blockIdx.z;
-  const int nh = min(16, a.heads - h0);
+  constexpr int MH = 16 * HG;                        // heads of the CTA
+  const int split = blockIdx.x, h0 = blockIdx.y * MH, row = blockIdx.z;
+  const int nh = min(MH, a.heads - h0);
   const int dk16 = a.ld_cache;
-  const TcLayout L = tc_layout(dk16, 64 * NT);
+  const TcLayout L = tc_layout(dk16, 64 * NT, HG);
   __nv_bfloat16* q_s = reinterpret_cast<__nv_bfloat16*>(smem);
   __nv_bfloat16* p_s = reinterpret_cast<__nv_bfloat16*>(smem + L.q_bytes);            // high parts, then low parts
-  float* s_s = reinterpret_cast<float*>(smem + L.q_bytes + 2 * 16 * kPPitch * 2);     // [2][16][kTile]
-  float* m_s = s_s + 2 * 16 * kTile;                                                   // running maximum, sum, factor
-  float* l_s = m_s + 16;
-  float* f_s = l_s + 16;
+  float* s_s = reinterpret_cast<float*>(smem + L.q_bytes + 2 * MH * kPPitch * 2);     // [2][MH][kTile]
+  float* m_s = s_s + 2 * MH * kTile;                                                   // final maximum and sum, tile's factor
+  float* l_s = m_s + MH;
+  float* f_s = l_s + MH;
   uint8_t* ring = smem + L.total - L.stages * L.stage_bytes;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const bool pad = a.slots[row] < 0;
   const int len = pad ? 0 : a.positions[row] + 1;
-  int chunk = a.chunk_tokens > 0 ? a.chunk_tokens : len;
+  const int chunk = a.chunk_tokens > 0 ? a.chunk_tokens : len;
   const int t0 = split * chunk, t1 = a.num_splits > 1 ? min(len, t0 + chunk) : len;
   if (a.num_splits > 1 && t0 >= len) return;         // the merge kernel skips this slice
   const int tiles = (t1 - t0 + kTile - 1) / kTile;
@@ -247,6 +257,7 @@ latent_attn_tc_kernel(XpLatentAttnArgs a) {
       const __nv_bfloat16* src = cache + (static_cast<size_t>(table[tt / a.page_size]) * a.page_size + tt % a.page_size) * dk16;
       const uint32_t dst = sm100::smem_u32(st + tok * L.pitch * 2);
       const int sz = ok ? 16 : 0;                    // rows past the slice read as zero
+#pragma unroll 6
       for (int c = threadIdx.x & 3; c < chunks_row; c += 4)
         asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst + c * 16), "l"(src + c * 8), "r"(sz));
     }
@@ -254,32 +265,35 @@ latent_attn_tc_kernel(XpLatentAttnArgs a) {
   };
   for (int i = 0; i < L.stages - 1; ++i) issue(i);
 
-  // queries of the head group; absent heads and the pitch's padding columns read as zero
-  for (int i = threadIdx.x; i < 16 * (dk16 / 8); i += kTcThreads) {
-    const int h = i / (dk16 / 8), c = (i - h * (dk16 / 8)) * 8;
+  // queries of the head groups; absent heads read as zero
+  for (int i = threadIdx.x; i < MH * chunks_row; i += kTcThreads) {
+    const int h = i / chunks_row, c = (i - h * chunks_row) * 8;
     uint4 v = make_uint4(0, 0, 0, 0);
     if (h < nh)
       v = *reinterpret_cast<const uint4*>(reinterpret_cast<const __nv_bfloat16*>(a.q) +
                                           (static_cast<size_t>(h0 + h) * a.q_rows + row) * a.ld_q + c);
     *reinterpret_cast<uint4*>(q_s + h * L.pitch + c) = v;
   }
-  if (threadIdx.x < 16) {
-    m_s[threadIdx.x] = -CUDART_INF_F;
-    l_s[threadIdx.x] = 0.f;
-  }
   const float qscale = a.scale * kLog2e;
   const int tg = warp & 3, kh = warp >> 2;           // token group (16 tokens), half of the key columns
   const int ksteps = dk16 / 16, ks0 = kh ? (ksteps + 1) / 2 : 0, ks1 = kh ? ksteps : (ksteps + 1) / 2;
   const int g = lane >> 2, q4 = lane & 3;
   const uint32_t q_addr = sm100::smem_u32(q_s) + ((lane & 15) * L.pitch + (lane >> 4) * 8) * 2;
+  const uint32_t q_group = 16 * L.pitch * 2;
   const uint32_t k_lane = ((tg * 16 + (lane & 7) + ((lane >> 4) << 3)) * L.pitch + ((lane >> 3) & 1) * 8) * 2;
   const uint32_t p_addr = sm100::smem_u32(p_s) + ((lane & 15) * kPPitch + (lane >> 4) * 8) * 2;
   const uint32_t v_lane = (((lane & 7) + ((lane >> 3) & 1) * 8) * L.pitch + warp * NT * 8 + (lane >> 4) * 8) * 2;
-  float acc[NT][4];
+  constexpr int MW = MH / 8;                         // heads whose softmax this warp does: warp * MW ..
+  float m_run[MW], l_run[MW];
 #pragma unroll
-  for (int j = 0; j < NT; ++j)
+  for (int r = 0; r < MW; ++r) m_run[r] = -CUDART_INF_F, l_run[r] = 0.f;
+  float acc[HG][NT][4];
 #pragma unroll
-    for (int e = 0; e < 4; ++e) acc[j][e] = 0.f;
+  for (int hg = 0; hg < HG; ++hg)
+#pragma unroll
+    for (int j = 0; j < NT; ++j)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) acc[hg][j][e] = 0.f;
 
   for (int it = 0; it < tiles; ++it) {
     if (L.stages == 2) asm volatile("cp.async.wait_group 0;" ::: "memory");
@@ -288,101 +302,149 @@ latent_attn_tc_kernel(XpLatentAttnArgs a) {
     __syncthreads();                                 // tile it landed; everyone is done with the tile before it
     issue(it + L.stages - 1);
     const uint32_t st = sm100::smem_u32(ring + (it % L.stages) * L.stage_bytes);
-    // scores of 16 tokens over this warp's half of the columns
-    float s0[4] = {0.f, 0.f, 0.f, 0.f}, s1[4] = {0.f, 0.f, 0.f, 0.f};
-    for (int ks = ks0; ks < ks1; ++ks) {
-      uint32_t qa[4], kb[4];
-      ldsm_x4(q_addr + ks * 32, qa);
+    // scores of 16 tokens over this warp's half of the columns; even and odd steps in chains of their own
+    float sc[2][HG][2][4];
+#pragma unroll
+    for (int i = 0; i < 2 * HG * 2 * 4; ++i) (&sc[0][0][0][0])[i] = 0.f;
+    auto score_step = [&](int ks, float (&c)[HG][2][4]) {
+      uint32_t kb[4];
       ldsm_x4(st + k_lane + ks * 32, kb);
-      mma16816(s0, qa, kb[0], kb[1]);
-      mma16816(s1, qa, kb[2], kb[3]);
+#pragma unroll
+      for (int hg = 0; hg < HG; ++hg) {
+        uint32_t qa[4];
+        ldsm_x4(q_addr + hg * q_group + ks * 32, qa);
+        mma16816(c[hg][0], qa, kb[0], kb[1]);
+        mma16816(c[hg][1], qa, kb[2], kb[3]);
+      }
+    };
+    int ks = ks0;
+#pragma unroll 3
+    for (; ks + 1 < ks1; ks += 2) {
+      score_step(ks, sc[0]);
+      score_step(ks + 1, sc[1]);
     }
-    float* sp = s_s + kh * 16 * kTile + tg * 16 + q4 * 2;
-    *reinterpret_cast<float2*>(sp + g * kTile) = make_float2(s0[0], s0[1]);
-    *reinterpret_cast<float2*>(sp + (g + 8) * kTile) = make_float2(s0[2], s0[3]);
-    *reinterpret_cast<float2*>(sp + g * kTile + 8) = make_float2(s1[0], s1[1]);
-    *reinterpret_cast<float2*>(sp + (g + 8) * kTile + 8) = make_float2(s1[2], s1[3]);
+    if (ks < ks1) score_step(ks, sc[0]);
+#pragma unroll
+    for (int hg = 0; hg < HG; ++hg)
+#pragma unroll
+      for (int u = 0; u < 2; ++u)
+#pragma unroll
+        for (int r = 0; r < 2; ++r)
+          *reinterpret_cast<float2*>(s_s + (kh * MH + hg * 16 + g + r * 8) * kTile + tg * 16 + u * 8 + q4 * 2) =
+              make_float2(sc[0][hg][u][2 * r] + sc[1][hg][u][2 * r], sc[0][hg][u][2 * r + 1] + sc[1][hg][u][2 * r + 1]);
     __syncthreads();
-    // softmax: two heads per warp, two tokens per lane
+    // softmax: MW heads per warp (independent chains), two tokens per lane
     const int tok0 = t0 + it * kTile + lane * 2;
+    float v[MW][2], mx[MW], sum[MW];
 #pragma unroll
-    for (int r = 0; r < 2; ++r) {
-      const int h = warp * 2 + r;
+    for (int r = 0; r < MW; ++r) {
+      const int h = warp * MW + r;
       const float2 x = *reinterpret_cast<const float2*>(s_s + h * kTile + lane * 2);
-      const float2 y = *reinterpret_cast<const float2*>(s_s + 16 * kTile + h * kTile + lane * 2);
-      const float v0 = tok0 < t1 ? (x.x + y.x) * qscale : -CUDART_INF_F;
-      const float v1 = tok0 + 1 < t1 ? (x.y + y.y) * qscale : -CUDART_INF_F;
-      float mx = fmaxf(v0, v1);
+      const float2 y = *reinterpret_cast<const float2*>(s_s + (MH + h) * kTile + lane * 2);
+      v[r][0] = tok0 < t1 ? (x.x + y.x) * qscale : -CUDART_INF_F;
+      v[r][1] = tok0 + 1 < t1 ? (x.y + y.y) * qscale : -CUDART_INF_F;
+      mx[r] = fmaxf(v[r][0], v[r][1]);
+    }
 #pragma unroll
-      for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
-      const float m_old = m_s[h], m_new = fmaxf(m_old, mx);
-      const float p0 = exp2f(v0 - m_new), p1 = exp2f(v1 - m_new);
-      const float sum = elem::warp_sum(p0 + p1);
+    for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+      for (int r = 0; r < MW; ++r) mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], o));
+#pragma unroll
+    for (int r = 0; r < MW; ++r) {
+      const int h = warp * MW + r;
+      const float m_new = fmaxf(m_run[r], mx[r]);
+      const float p0 = exp2f(v[r][0] - m_new), p1 = exp2f(v[r][1] - m_new);
+      const float f = exp2f(m_run[r] - m_new);
+      m_run[r] = m_new;
+      l_run[r] *= f;
+      sum[r] = p0 + p1;
       const __nv_bfloat162 hi = __floats2bfloat162_rn(p0, p1);
       const float2 hf = __bfloat1622float2(hi);
       *reinterpret_cast<__nv_bfloat162*>(p_s + h * kPPitch + lane * 2) = hi;
-      *reinterpret_cast<__nv_bfloat162*>(p_s + (16 + h) * kPPitch + lane * 2) = __floats2bfloat162_rn(p0 - hf.x, p1 - hf.y);
-      __syncwarp();
-      if (lane == 0) {
-        const float f = exp2f(m_old - m_new);
-        f_s[h] = f;
-        m_s[h] = m_new;
-        l_s[h] = l_s[h] * f + sum;
-      }
+      *reinterpret_cast<__nv_bfloat162*>(p_s + (MH + h) * kPPitch + lane * 2) = __floats2bfloat162_rn(p0 - hf.x, p1 - hf.y);
+      if (lane == 0) f_s[h] = f;
     }
     __syncthreads();
-    const float fa = f_s[g], fb = f_s[g + 8];
+    // the sums are off the critical path: their shuffles overlap the second product
 #pragma unroll
-    for (int j = 0; j < NT; ++j) acc[j][0] *= fa, acc[j][1] *= fa, acc[j][2] *= fb, acc[j][3] *= fb;
+    for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+      for (int r = 0; r < MW; ++r) sum[r] += __shfl_xor_sync(0xffffffffu, sum[r], o);
+#pragma unroll
+    for (int r = 0; r < MW; ++r) l_run[r] += sum[r];
+#pragma unroll
+    for (int hg = 0; hg < HG; ++hg) {
+      const float fa = f_s[hg * 16 + g], fb = f_s[hg * 16 + g + 8];
+#pragma unroll
+      for (int j = 0; j < NT; ++j) acc[hg][j][0] *= fa, acc[hg][j][1] *= fa, acc[hg][j][2] *= fb, acc[hg][j][3] *= fb;
+    }
 #pragma unroll
     for (int kk = 0; kk < kTile / 16; ++kk) {
-      uint32_t ph[4], pl[4];
-      ldsm_x4(p_addr + kk * 32, ph);
-      ldsm_x4(p_addr + 16 * kPPitch * 2 + kk * 32, pl);
+      uint32_t ph[HG][4], pl[HG][4];
+#pragma unroll
+      for (int hg = 0; hg < HG; ++hg) {
+        ldsm_x4(p_addr + hg * 16 * kPPitch * 2 + kk * 32, ph[hg]);
+        ldsm_x4(p_addr + (MH + hg * 16) * kPPitch * 2 + kk * 32, pl[hg]);
+      }
 #pragma unroll
       for (int j = 0; j < NT; j += 2) {
         uint32_t vb[4];
         ldsm_x4_trans(st + v_lane + kk * 16 * L.pitch * 2 + j * 16, vb);
-        mma16816(acc[j], ph, vb[0], vb[1]);
-        mma16816(acc[j + 1], ph, vb[2], vb[3]);
-        mma16816(acc[j], pl, vb[0], vb[1]);
-        mma16816(acc[j + 1], pl, vb[2], vb[3]);
+#pragma unroll
+        for (int hg = 0; hg < HG; ++hg) {
+          mma16816(acc[hg][j], ph[hg], vb[0], vb[1]);
+          mma16816(acc[hg][j + 1], ph[hg], vb[2], vb[3]);
+          mma16816(acc[hg][j], pl[hg], vb[0], vb[1]);
+          mma16816(acc[hg][j + 1], pl[hg], vb[2], vb[3]);
+        }
       }
     }
   }
   asm volatile("cp.async.wait_group 0;" ::: "memory");
+#pragma unroll
+  for (int r = 0; r < MW; ++r)
+    if (lane == 0) {
+      m_s[warp * MW + r] = m_run[r];
+      l_s[warp * MW + r] = l_run[r];
+    }
   __syncthreads();
 #pragma unroll
-  for (int e = 0; e < 2; ++e) {
-    const int h = g + e * 8;
-    if (h >= nh) continue;
-    if (a.num_splits > 1) {
-      float* w = a.ws + ((static_cast<size_t>(row) * a.heads + h0 + h) * a.num_splits + split) * (a.kv_rank + 2);
-      for (int j = 0; j < NT; ++j) {
-        const int c = (warp * NT + j) * 8 + q4 * 2;
+  for (int hg = 0; hg < HG; ++hg)
 #pragma unroll
-        for (int u = 0; u < 2; ++u)
-          if (c + u < a.kv_rank) w[c + u] = acc[j][e * 2 + u];
-      }
-      if (warp == 0 && q4 == 0) {
-        w[a.kv_rank] = m_s[h];
-        w[a.kv_rank + 1] = l_s[h];
-      }
-    } else {
-      float f = pad ? 0.f : 1.f / l_s[h];
-      if (a.gate != nullptr)
-        f *= elem::sigmoid(elem::ld(reinterpret_cast<const __nv_bfloat16*>(a.gate) + static_cast<size_t>(row) * a.ld_gate + h0 + h));
-      __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(a.out) + (static_cast<size_t>(h0 + h) * a.q_rows + row) * a.ld_out;
-      for (int j = 0; j < NT; ++j) {
-        const int c = (warp * NT + j) * 8 + q4 * 2;
-        if (c + 1 < a.kv_rank && a.ld_out % 2 == 0)
-          *reinterpret_cast<__nv_bfloat162*>(out + c) = __floats2bfloat162_rn(acc[j][e * 2] * f, acc[j][e * 2 + 1] * f);
-        else
+    for (int e = 0; e < 2; ++e) {
+      const int h = hg * 16 + g + e * 8;
+      if (h >= nh) continue;
+      if (a.num_splits > 1) {
+        float* w = a.ws + ((static_cast<size_t>(row) * a.heads + h0 + h) * a.num_splits + split) * (a.kv_rank + 2);
+#pragma unroll
+        for (int j = 0; j < NT; ++j) {
+          const int c = (warp * NT + j) * 8 + q4 * 2;
+#pragma unroll
           for (int u = 0; u < 2; ++u)
-            if (c + u < a.kv_rank) out[c + u] = __float2bfloat16_rn(acc[j][e * 2 + u] * f);
+            if (c + u < a.kv_rank) w[c + u] = acc[hg][j][e * 2 + u];
+        }
+        if (warp == 0 && q4 == 0) {
+          w[a.kv_rank] = m_s[h];
+          w[a.kv_rank + 1] = l_s[h];
+        }
+      } else {
+        float f = pad ? 0.f : 1.f / l_s[h];
+        if (a.gate != nullptr)
+          f *= elem::sigmoid(elem::ld(reinterpret_cast<const __nv_bfloat16*>(a.gate) + static_cast<size_t>(row) * a.ld_gate + h0 + h));
+        __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(a.out) + (static_cast<size_t>(h0 + h) * a.q_rows + row) * a.ld_out;
+#pragma unroll
+        for (int j = 0; j < NT; ++j) {
+          const int c = (warp * NT + j) * 8 + q4 * 2;
+          if (c + 1 < a.kv_rank && a.ld_out % 2 == 0) {
+            *reinterpret_cast<__nv_bfloat162*>(out + c) = __floats2bfloat162_rn(acc[hg][j][e * 2] * f, acc[hg][j][e * 2 + 1] * f);
+          } else {
+#pragma unroll
+            for (int u = 0; u < 2; ++u)
+              if (c + u < a.kv_rank) out[c + u] = __float2bfloat16_rn(acc[hg][j][e * 2 + u] * f);
+          }
+        }
       }
     }
-  }
 }
 
 // One CTA per (head, row): folds the slices in order.
@@ -408,6 +470,8 @@ latent_merge_kernel(XpLatentAttnArgs a) {
 }
 
 // ------------------------------------------------------------------------------------------ gather
+constexpr int kGatherTokens = 4;
+
 __global__ void __launch_bounds__(128)
 latent_gather_kernel(XpLatentGatherArgs a) {
   const int seq = blockIdx.y;
@@ -417,7 +481,7 @@ latent_gather_kernel(XpLatentGatherArgs a) {
   const uint8_t* cache = static_cast<const uint8_t*>(a.cache);
   uint8_t* out = static_cast<uint8_t*>(a.out) + static_cast<size_t>(a.starts[seq]) * row_bytes;
   const int per = row_bytes / 16;
-  const int t0 = blockIdx.x * 16, n = min(16, len - t0);
+  const int t0 = blockIdx.x * kGatherTokens, n = min(kGatherTokens, len - t0);
   for (int u = threadIdx.x; u < n * per; u += 128) {
     const int t = t0 + u / per, c = u % per;
     const size_t src = (static_cast<size_t>(table[t / a.page_size]) * a.page_size + t % a.page_size) * row_bytes;
@@ -431,17 +495,17 @@ inline int done() {
   return e == cudaSuccess ? 0 : -100 - static_cast<int>(e);
 }
 
-template <int NT>
+template <int NT, int HG>
 int launch_tc(const XpLatentAttnArgs& a, cudaStream_t s) {
-  const TcLayout L = tc_layout(a.ld_cache, 64 * NT);
+  const TcLayout L = tc_layout(a.ld_cache, 64 * NT, HG);
   if (L.total > 227 * 1024) return 1;
   static bool set = false;
   if (!set) {
-    if (cudaFuncSetAttribute(latent_attn_tc_kernel<NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024) != cudaSuccess) return -21;
+    if (cudaFuncSetAttribute(latent_attn_tc_kernel<NT, HG>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024) != cudaSuccess) return -21;
     set = true;
   }
-  dim3 grid(a.num_splits > 1 ? a.num_splits : 1, (a.heads + 15) / 16, a.rows);
-  latent_attn_tc_kernel<NT><<<grid, kTcThreads, L.total, s>>>(a);
+  dim3 grid(a.num_splits > 1 ? a.num_splits : 1, (a.heads + 16 * HG - 1) / (16 * HG), a.rows);
+  latent_attn_tc_kernel<NT, HG><<<grid, kTcThreads, L.total, s>>>(a);
   if (a.num_splits > 1) latent_merge_kernel<<<dim3(a.heads, a.rows), 128, 0, s>>>(a);
   return done();
 }
@@ -460,8 +524,19 @@ extern "C" int xp_latent_prep(const XpLatentPrepArgs* a, void* stream) {
   if (a->abs_rows < a->rows && (a->q_exp == nullptr || a->dq_pad < a->dim + a->rot)) return -12;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   const size_t sm = static_cast<size_t>(a->rot_dims > 0 ? a->rot_dims : 1) * 4;
-  if (a->f32) latent_prep_kernel<float><<<a->rows, kPrepThreads, sm, s>>>(*a);
-  else latent_prep_kernel<__nv_bfloat16><<<a->rows, kPrepThreads, sm, s>>>(*a);
+  // four elements at a time where every head's plain part starts on a 4-element boundary in all layouts
+  const int eb = a->f32 ? 4 : 2;
+  auto al = [&](const void* p) { return reinterpret_cast<uintptr_t>(p) % (4 * eb) == 0; };
+  const bool v = a->dim % 4 == 0 && a->rot % 4 == 0 && a->ld_proj % 4 == 0 && a->q_off % 4 == 0 && a->dim_p % 4 == 0 && a->dq_pad % 4 == 0 &&
+                 al(a->proj) && al(a->q_plain) && al(a->q_exp);
+  dim3 grid(a->rows, (a->heads + kPrepHeads - 1) / kPrepHeads);
+  if (a->f32) {
+    if (v) latent_prep_kernel<float, 4><<<grid, kPrepThreads, sm, s>>>(*a);
+    else latent_prep_kernel<float, 1><<<grid, kPrepThreads, sm, s>>>(*a);
+  } else {
+    if (v) latent_prep_kernel<__nv_bfloat16, 4><<<grid, kPrepThreads, sm, s>>>(*a);
+    else latent_prep_kernel<__nv_bfloat16, 1><<<grid, kPrepThreads, sm, s>>>(*a);
+  }
   return done();
 }
 
@@ -471,7 +546,9 @@ extern "C" int xp_latent_attn(const XpLatentAttnArgs* a, void* stream) {
   if (a->num_splits > 1 && (a->ws == nullptr || a->chunk_tokens <= 0)) return -11;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   if (!a->f32 && !a->force_simt && a->kv_rank <= 512 && a->ld_cache % 16 == 0 && a->ld_q % 8 == 0 && a->ld_q >= a->ld_cache) {
-    int rc = a->kv_rank <= 128 ? launch_tc<2>(*a, s) : a->kv_rank <= 256 ? launch_tc<4>(*a, s) : launch_tc<8>(*a, s);
+    int rc;
+    if (a->heads > 16) rc = a->kv_rank <= 128 ? launch_tc<2, 2>(*a, s) : a->kv_rank <= 256 ? launch_tc<4, 2>(*a, s) : launch_tc<8, 2>(*a, s);
+    else rc = a->kv_rank <= 128 ? launch_tc<2, 1>(*a, s) : a->kv_rank <= 256 ? launch_tc<4, 1>(*a, s) : launch_tc<8, 1>(*a, s);
     if (rc <= 0) return rc;
   }
   if (a->kv_rank > kSimtAcc * kSimtThreads || a->kv_rank + a->rot > 12000) return -12;
@@ -485,7 +562,7 @@ extern "C" int xp_latent_attn(const XpLatentAttnArgs* a, void* stream) {
 extern "C" int xp_latent_gather(const XpLatentGatherArgs* a, void* stream) {
   if (a->n_seqs <= 0 || a->max_len <= 0) return 0;
   if ((a->ld_cache * a->elem_bytes) % 16 != 0) return -10;
-  dim3 grid((a->max_len + 15) / 16, a->n_seqs);
+  dim3 grid((a->max_len + kGatherTokens - 1) / kGatherTokens, a->n_seqs);
   latent_gather_kernel<<<grid, 128, 0, reinterpret_cast<cudaStream_t>(stream)>>>(*a);
   return done();
 }

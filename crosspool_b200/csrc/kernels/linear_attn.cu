@@ -155,17 +155,21 @@ linear_sequential_kernel(XpLinearAttnArgs a) {
 }
 
 // ------------------------------------------------------------------------------------------ chunked prefill
-// CTA = (VS state columns, head, sequence); it walks the sequence in chunks of 64 tokens with the state in registers.
-// With p(n) = decay^n, for row i of a chunk of n tokens and the state S before it:
-//   o_i = sum_{j <= i} p(i - j) (q_i . k_j) v_j + p(i + 1) S^T q_i          (four warps, 16 rows each)
-//   S   <- p(n) S + sum_j k_j (p(n - 1 - j) v_j)^T                          (four warps, D / 4 rows of S each)
+// CTA = (segment of a portion, VS state columns, head, sequence); it walks its segment in chunks of 64 tokens with the
+// state in registers. With p(n) = decay^n, for row i of a chunk of n tokens and the state S before it:
+//   o_i = p(i + 1) S^T q_i + sum_{j <= i} p(i - j) (q_i . k_j) v_j          (warp: 16 rows, half of the columns)
+//   S   <- p(n) S + sum_j k_j (p(n - 1 - j) v_j)^T                          (warp: its 16-row tiles of S)
 // Decayed scores, decayed values and the state enter their products as bf16 pairs (high and low part), so everything
 // that belongs to the recurrence keeps at least 16 mantissa bits; the sums are fp32.
 //
+// A long portion with few heads is cut into segments that run at the same time: a first pass computes what each segment
+// adds to the state (the second line alone, from zero), a scan over the segments turns that into the state before each of
+// them, and the full pass starts every segment from there.
+//
 // mma.sync rather than tcgen05: the state has to be scaled and re-split between chunks, which from tensor memory costs a
-// round trip per chunk, and the kernel is bound by that dependency chain.
+// round trip per chunk.
 constexpr int kChunk = 64;
-constexpr int kChunkThreads = 128;
+constexpr int kChunkThreads = 256;
 
 __device__ __forceinline__ void ldsm4(uint32_t addr, uint32_t (&r)[4]) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
@@ -198,22 +202,31 @@ constexpr int chunk_smem_bytes() {
   return (4 * kChunk * (D + 8) + 2 * kChunk * (VS + 8) + 2 * kChunk * (VS + 8) + 2 * D * (VS + 8)) * 2 + (kChunk + 1 + 3) * 4;
 }
 
-template <int D, int VS>
-__global__ void __launch_bounds__(kChunkThreads)
+// kFull: outputs and the state; otherwise only what the segment adds to the state.
+template <int D, int VS, bool kFull>
+__global__ void __launch_bounds__(kChunkThreads, 1)
 linear_chunked_kernel(XpLinearAttnArgs a) {
   extern __shared__ __align__(16) uint8_t smem[];
   constexpr int PD = D + 8, PV = VS + 8;             // pitches: odd multiples of 16 bytes
-  constexpr int NV = VS / 8, MT = D / 64;            // value tiles; 16-row state tiles per warp
+  constexpr int NO = VS / 16;                        // output tiles of a warp (8 columns each)
+  constexpr int MT = D > 128 ? D / 128 : 1;          // state row tiles of a warp
+  constexpr int NS = D >= 128 ? VS / 8 : VS / 16;    // state column tiles of a warp
   __nv_bfloat16* q_s = reinterpret_cast<__nv_bfloat16*>(smem);
   __nv_bfloat16* k_s = q_s + 2 * kChunk * PD;
   __nv_bfloat16* v_s = k_s + 2 * kChunk * PD;
   __nv_bfloat16* vd_s = v_s + 2 * kChunk * PV;       // decayed values: high parts, low parts
   __nv_bfloat16* st_s = vd_s + 2 * kChunk * PV;      // state: high parts, low parts
   float* pw = reinterpret_cast<float*>(st_s + 2 * D * PV);
-  const int h = blockIdx.y, seq = blockIdx.z, c0 = blockIdx.x * VS;
-  const int n = a.q_lens[seq];
-  if (n <= 0) return;
-  const int r0 = a.q_starts[seq];
+  const int slices = (a.vdim + VS - 1) / VS;
+  const int seg = blockIdx.x / slices, c0 = (blockIdx.x % slices) * VS;
+  const int h = blockIdx.y, seq = blockIdx.z;
+  const int total = a.q_lens[seq];
+  const int first = seg * a.seg_tokens;              // segments are whole chunks long
+  if (first >= total) return;
+  const bool last = first + a.seg_tokens >= total;
+  if (!kFull && last) return;                        // nobody starts behind the last segment
+  const int n = min(a.seg_tokens, total - first);
+  const int r0 = a.q_starts[seq] + first;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int g = lane >> 2, q4 = lane & 3;
   const int chunks = (n + kChunk - 1) / kChunk;
@@ -239,11 +252,11 @@ linear_chunked_kernel(XpLinearAttnArgs a) {
         const int t = i / per, e = (i - t * per) * 8;
         const bool ok = t < m;
         const __nv_bfloat16* row = proj + static_cast<size_t>(r0 + c * kChunk + (ok ? t : 0)) * a.ld_proj + h * a.dim + e;
-        copy(q_s + (b * kChunk + t) * PD + e, row + a.q_off, ok);
+        if (kFull) copy(q_s + (b * kChunk + t) * PD + e, row + a.q_off, ok);
         copy(k_s + (b * kChunk + t) * PD + e, row + a.k_off, ok);
       }
-      for (int i = threadIdx.x; i < kChunk * NV; i += kChunkThreads) {
-        const int t = i / NV, e = (i % NV) * 8;
+      for (int i = threadIdx.x; i < kChunk * (VS / 8); i += kChunkThreads) {
+        const int t = i / (VS / 8), e = (i % (VS / 8)) * 8;
         const bool ok = t < m && c0 + e < a.vdim;
         copy(v_s + (b * kChunk + t) * PV + e,
              proj + static_cast<size_t>(r0 + c * kChunk + (t < m ? t : 0)) * a.ld_proj + a.v_off + h * a.vdim + (ok ? c0 + e : 0), ok);
@@ -253,44 +266,48 @@ linear_chunked_kernel(XpLinearAttnArgs a) {
   };
   issue(0);
 
-  // state: this warp's rows [warp * D / 4, + D / 4), columns c0 .. c0 + VS
-  float* S = a.state + (static_cast<size_t>(a.state_slots[seq]) * a.heads + h) * a.dim * a.vdim;
-  const bool fresh = a.positions[r0] == 0;
-  float s[MT][NV][4];
-  auto state_at = [&](int mt, int j, int e, int& d, int& c) {
-    d = warp * (D / 4) + mt * 16 + g + (e >> 1) * 8;
-    c = c0 + j * 8 + q4 * 2 + (e & 1);
-    return d < a.dim && c < a.vdim;
-  };
+  // the warp's part of the state
+  const int d0 = D >= 128 ? warp * MT * 16 : (warp & 3) * 16;
+  const int s0 = D >= 128 ? 0 : (warp >> 2) * (VS / 2);
+  const size_t state_elems = static_cast<size_t>(a.dim) * a.vdim;
+  float* slot = a.state + (static_cast<size_t>(a.state_slots[seq]) * a.heads + h) * state_elems;
+  float* mid = a.ws + ((static_cast<size_t>(seq) * a.heads + h) * a.segs + seg) * state_elems;   // used when segs > 1
+  const float* from = kFull && a.segs > 1 ? mid : slot;
+  const bool zero = !kFull || (a.segs == 1 && a.positions[r0] == 0);
+  float s[MT][NS][4];
 #pragma unroll
   for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
-    for (int j = 0; j < NV; ++j)
+    for (int j = 0; j < NS; ++j)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        int d, c;
-        s[mt][j][e] = state_at(mt, j, e, d, c) && !fresh ? S[static_cast<size_t>(d) * a.vdim + c] : 0.f;
+      for (int r = 0; r < 2; ++r) {
+        const int d = d0 + mt * 16 + g + r * 8, c = c0 + s0 + j * 8 + q4 * 2;
+        float2 x = make_float2(0.f, 0.f);
+        if (!zero && d < a.dim && c < a.vdim) x = *reinterpret_cast<const float2*>(from + static_cast<size_t>(d) * a.vdim + c);
+        s[mt][j][2 * r] = x.x;
+        s[mt][j][2 * r + 1] = x.y;
       }
   auto publish_state = [&]() {
 #pragma unroll
     for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
-      for (int j = 0; j < NV; ++j)
+      for (int j = 0; j < NS; ++j)
 #pragma unroll
         for (int r = 0; r < 2; ++r) {
           uint32_t hi, lo;
           split2(s[mt][j][2 * r], s[mt][j][2 * r + 1], hi, lo);
-          __nv_bfloat16* p = st_s + (warp * (D / 4) + mt * 16 + g + r * 8) * PV + j * 8 + q4 * 2;
+          __nv_bfloat16* p = st_s + (d0 + mt * 16 + g + r * 8) * PV + s0 + j * 8 + q4 * 2;
           *reinterpret_cast<uint32_t*>(p) = hi;
           *reinterpret_cast<uint32_t*>(p + D * PV) = lo;
         }
   };
-  publish_state();
+  if (kFull) publish_state();
 
-  const uint32_t a_off = ((warp * 16 + (lane & 15)) * PD + (lane >> 4) * 8) * 2;                        // Q rows of this warp
+  const int rw = warp & 3, o0 = (warp >> 2) * (VS / 2);   // output rows and columns of the warp
+  const uint32_t a_off = ((rw * 16 + (lane & 15)) * PD + (lane >> 4) * 8) * 2;                          // Q rows of this warp
   const uint32_t b_off = (((lane & 7) + ((lane >> 4) << 3)) * PD + ((lane >> 3) & 1) * 8) * 2;          // K as [tokens][dims]
   const uint32_t t_off = (((lane & 7) + ((lane >> 3) & 1) * 8) * PV + (lane >> 4) * 8) * 2;             // [k][n] operands, transposed
-  const uint32_t kt_off = (((lane & 7) + (lane >> 4) * 8) * PD + warp * (D / 4) + ((lane >> 3) & 1) * 8) * 2;  // K^T rows of this warp
+  const uint32_t kt_off = (((lane & 7) + (lane >> 4) * 8) * PD + d0 + ((lane >> 3) & 1) * 8) * 2;       // K^T rows of this warp
 
   for (int c = 0; c < chunks; ++c) {
     const int b = c & 1, m = min(kChunk, n - c * kChunk);
@@ -298,97 +315,102 @@ linear_chunked_kernel(XpLinearAttnArgs a) {
     __syncthreads();                                 // chunk c landed, state published, buffers of chunk c - 1 free
     issue(c + 1);
     // decayed values of the state update
-    for (int i = threadIdx.x; i < kChunk * (VS / 2); i += kChunkThreads) {
-      const int t = i / (VS / 2), e = (i % (VS / 2)) * 2;
+    for (int i = threadIdx.x; i < kChunk * (VS / 4); i += kChunkThreads) {
+      const int t = i / (VS / 4), e = (i % (VS / 4)) * 4;
       const float w = t < m ? pw[m - 1 - t] : 0.f;
-      const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(v_s + (b * kChunk + t) * PV + e));
-      uint32_t hi, lo;
-      split2(v.x * w, v.y * w, hi, lo);
-      *reinterpret_cast<uint32_t*>(vd_s + t * PV + e) = hi;
-      *reinterpret_cast<uint32_t*>(vd_s + (kChunk + t) * PV + e) = lo;
+      float v[4];
+      elem::ldv<4>(v_s + (b * kChunk + t) * PV + e, v);
+      uint2 hi, lo;
+      split2(v[0] * w, v[1] * w, hi.x, lo.x);
+      split2(v[2] * w, v[3] * w, hi.y, lo.y);
+      *reinterpret_cast<uint2*>(vd_s + t * PV + e) = hi;
+      *reinterpret_cast<uint2*>(vd_s + (kChunk + t) * PV + e) = lo;
     }
-    const uint32_t qb = sm100::smem_u32(q_s + b * kChunk * PD) + a_off;
     const uint32_t kb = sm100::smem_u32(k_s + b * kChunk * PD);
-    const uint32_t vb = sm100::smem_u32(v_s + b * kChunk * PV) + t_off;
-    const uint32_t sb = sm100::smem_u32(st_s) + t_off;
-    float o[NV][4], os[NV][4], p[8][4];
+    if constexpr (kFull) {
+      const uint32_t qb = sm100::smem_u32(q_s + b * kChunk * PD) + a_off;
+      const uint32_t vb = sm100::smem_u32(v_s + b * kChunk * PV) + t_off + o0 * 2;
+      const uint32_t sb = sm100::smem_u32(st_s) + t_off + o0 * 2;
+      float o[NO][4], p[8][4];
 #pragma unroll
-    for (int j = 0; j < NV; ++j)
+      for (int j = 0; j < NO; ++j)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) o[j][e] = os[j][e] = 0.f;
+        for (int e = 0; e < 4; ++e) o[j][e] = 0.f;
 #pragma unroll
-    for (int j = 0; j < 8; ++j)
+      for (int j = 0; j < 8; ++j)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) p[j][e] = 0.f;
-    // scores of this warp's rows against tokens up to its own, and S^T q
+        for (int e = 0; e < 4; ++e) p[j][e] = 0.f;
+      // S^T q, and the scores of this warp's rows against tokens up to its own
 #pragma unroll 2
-    for (int ks = 0; ks < D / 16; ++ks) {
-      uint32_t qa[4];
-      ldsm4(qb + ks * 32, qa);
+      for (int ks = 0; ks < D / 16; ++ks) {
+        uint32_t qa[4];
+        ldsm4(qb + ks * 32, qa);
 #pragma unroll
-      for (int j = 0; j < 4; ++j) {                  // 16 tokens each
-        if (j <= warp) {
-          uint32_t kf[4];
-          ldsm4(kb + b_off + (j * 16 * PD + ks * 16) * 2, kf);
-          mma(p[2 * j], qa, kf[0], kf[1]);
-          mma(p[2 * j + 1], qa, kf[2], kf[3]);
+        for (int j = 0; j < 4; ++j) {                // 16 tokens each
+          if (j <= rw) {
+            uint32_t kf[4];
+            ldsm4(kb + b_off + (j * 16 * PD + ks * 16) * 2, kf);
+            mma(p[2 * j], qa, kf[0], kf[1]);
+            mma(p[2 * j + 1], qa, kf[2], kf[3]);
+          }
+        }
+#pragma unroll
+        for (int j = 0; j < NO; j += 2) {
+          uint32_t hi[4], lo[4];
+          ldsm4t(sb + (ks * 16 * PV + j * 8) * 2, hi);
+          ldsm4t(sb + ((D + ks * 16) * PV + j * 8) * 2, lo);
+          mma(o[j], qa, hi[0], hi[1]);
+          mma(o[j + 1], qa, hi[2], hi[3]);
+          mma(o[j], qa, lo[0], lo[1]);
+          mma(o[j + 1], qa, lo[2], lo[3]);
+        }
+      }
+      const int i0 = rw * 16 + g;                    // rows i0 and i0 + 8 of the chunk
+      const float f0 = pw[i0 + 1], f1 = pw[i0 + 9];
+#pragma unroll
+      for (int j = 0; j < NO; ++j) o[j][0] *= f0, o[j][1] *= f0, o[j][2] *= f1, o[j][3] *= f1;
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        if (j <= rw) {
+          uint32_t ph[4], pl[4];
+#pragma unroll
+          for (int u = 0; u < 2; ++u) {
+            const int t = j * 16 + u * 8 + q4 * 2;
+            auto w = [&](int i, int tok) { return tok <= i ? pw[i - tok] : 0.f; };
+            split2(p[2 * j + u][0] * w(i0, t), p[2 * j + u][1] * w(i0, t + 1), ph[2 * u], pl[2 * u]);
+            split2(p[2 * j + u][2] * w(i0 + 8, t), p[2 * j + u][3] * w(i0 + 8, t + 1), ph[2 * u + 1], pl[2 * u + 1]);
+          }
+#pragma unroll
+          for (int v = 0; v < NO; v += 2) {
+            uint32_t vf[4];
+            ldsm4t(vb + (j * 16 * PV + v * 8) * 2, vf);
+            mma(o[v], ph, vf[0], vf[1]);
+            mma(o[v + 1], ph, vf[2], vf[3]);
+            mma(o[v], pl, vf[0], vf[1]);
+            mma(o[v + 1], pl, vf[2], vf[3]);
+          }
         }
       }
 #pragma unroll
-      for (int j = 0; j < NV; j += 2) {
-        uint32_t hi[4], lo[4];
-        ldsm4t(sb + (ks * 16 * PV + j * 8) * 2, hi);
-        ldsm4t(sb + ((D + ks * 16) * PV + j * 8) * 2, lo);
-        mma(os[j], qa, hi[0], hi[1]);
-        mma(os[j + 1], qa, hi[2], hi[3]);
-        mma(os[j], qa, lo[0], lo[1]);
-        mma(os[j + 1], qa, lo[2], lo[3]);
-      }
-    }
-    const int i0 = warp * 16 + g;                    // rows i0 and i0 + 8 of the chunk
+      for (int v = 0; v < NO; ++v) {
+        const int col = c0 + o0 + v * 8 + q4 * 2;
 #pragma unroll
-    for (int j = 0; j < 4; ++j) {
-      if (j <= warp) {
-        uint32_t ph[4], pl[4];
-#pragma unroll
-        for (int u = 0; u < 2; ++u) {
-          const int t = j * 16 + u * 8 + q4 * 2;
-          auto w = [&](int i, int tok) { return tok <= i ? pw[i - tok] : 0.f; };
-          split2(p[2 * j + u][0] * w(i0, t), p[2 * j + u][1] * w(i0, t + 1), ph[2 * u], pl[2 * u]);
-          split2(p[2 * j + u][2] * w(i0 + 8, t), p[2 * j + u][3] * w(i0 + 8, t + 1), ph[2 * u + 1], pl[2 * u + 1]);
-        }
-#pragma unroll
-        for (int v = 0; v < NV; v += 2) {
-          uint32_t vf[4];
-          ldsm4t(vb + (j * 16 * PV + v * 8) * 2, vf);
-          mma(o[v], ph, vf[0], vf[1]);
-          mma(o[v + 1], ph, vf[2], vf[3]);
-          mma(o[v], pl, vf[0], vf[1]);
-          mma(o[v + 1], pl, vf[2], vf[3]);
+        for (int r = 0; r < 2; ++r) {
+          const int i = i0 + r * 8;
+          if (i < m && col < a.vdim)                 // vdim is even
+            *reinterpret_cast<float2*>(a.out + static_cast<size_t>(r0 + c * kChunk + i) * a.heads * a.vdim + h * a.vdim + col) =
+                make_float2(o[v][2 * r], o[v][2 * r + 1]);
         }
       }
-    }
-    const float f0 = pw[i0 + 1], f1 = pw[i0 + 9 <= kChunk ? i0 + 9 : kChunk];
-#pragma unroll
-    for (int v = 0; v < NV; ++v) {
-      const int col = c0 + v * 8 + q4 * 2;
-#pragma unroll
-      for (int r = 0; r < 2; ++r) {
-        const int i = i0 + r * 8;
-        if (i < m && col < a.vdim) {                 // vdim is even
-          const float f = r ? f1 : f0;
-          *reinterpret_cast<float2*>(a.out + static_cast<size_t>(r0 + c * kChunk + i) * a.heads * a.vdim + h * a.vdim + col) =
-              make_float2(fmaf(f, os[v][2 * r], o[v][2 * r]), fmaf(f, os[v][2 * r + 1], o[v][2 * r + 1]));
-        }
-      }
+      if (c + 1 == chunks && !last) break;           // the next segment has its own start state
     }
     __syncthreads();                                 // decayed values written; everyone is done with the published state
     const float pn = pw[m];
-    const uint32_t db = sm100::smem_u32(vd_s) + t_off;
+    const uint32_t db = sm100::smem_u32(vd_s) + t_off + s0 * 2;
 #pragma unroll
     for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
-      for (int j = 0; j < NV; ++j)
+      for (int j = 0; j < NS; ++j)
 #pragma unroll
         for (int e = 0; e < 4; ++e) s[mt][j][e] *= pn;
 #pragma unroll
@@ -397,7 +419,7 @@ linear_chunked_kernel(XpLinearAttnArgs a) {
 #pragma unroll
       for (int mt = 0; mt < MT; ++mt) ldsm4t(kb + kt_off + (kk * 16 * PD + mt * 16) * 2, ka[mt]);
 #pragma unroll
-      for (int j = 0; j < NV; j += 2) {
+      for (int j = 0; j < NS; j += 2) {
         uint32_t hi[4], lo[4];
         ldsm4t(db + (kk * 16 * PV + j * 8) * 2, hi);
         ldsm4t(db + ((kChunk + kk * 16) * PV + j * 8) * 2, lo);
@@ -410,17 +432,41 @@ linear_chunked_kernel(XpLinearAttnArgs a) {
         }
       }
     }
-    if (c + 1 < chunks) publish_state();
+    if (kFull && c + 1 < chunks) publish_state();
   }
+  if (kFull && !last) return;
+  float* to = kFull ? slot : mid;
 #pragma unroll
   for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
-    for (int j = 0; j < NV; ++j)
+    for (int j = 0; j < NS; ++j)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        int d, c;
-        if (state_at(mt, j, e, d, c)) S[static_cast<size_t>(d) * a.vdim + c] = s[mt][j][e];
+      for (int r = 0; r < 2; ++r) {
+        const int d = d0 + mt * 16 + g + r * 8, c = c0 + s0 + j * 8 + q4 * 2;
+        if (d < a.dim && c < a.vdim)
+          *reinterpret_cast<float2*>(to + static_cast<size_t>(d) * a.vdim + c) = make_float2(s[mt][j][2 * r], s[mt][j][2 * r + 1]);
       }
+}
+
+// What each segment adds -> the state before each segment, in place.
+__global__ void __launch_bounds__(256)
+linear_scan_kernel(XpLinearAttnArgs a) {
+  const int h = blockIdx.y, seq = blockIdx.z;
+  const int total = a.q_lens[seq];
+  if (total <= 0) return;
+  const size_t state_elems = static_cast<size_t>(a.dim) * a.vdim;
+  const size_t i = blockIdx.x * 256ull + threadIdx.x;
+  if (i >= state_elems) return;
+  float* mid = a.ws + (static_cast<size_t>(seq) * a.heads + h) * a.segs * state_elems + i;
+  float x = a.positions[a.q_starts[seq]] == 0 ? 0.f : a.state[(static_cast<size_t>(a.state_slots[seq]) * a.heads + h) * state_elems + i];
+  const float p64 = a.decay_pow[h * (kChunk + 1) + kChunk];
+  float f = 1.f;                                     // decay over one whole segment
+  for (int c = 0; c < a.seg_tokens / kChunk; ++c) f *= p64;
+  for (int s = 0; s * a.seg_tokens < total; ++s) {
+    const float add = (s + 1) * a.seg_tokens < total ? mid[s * state_elems] : 0.f;   // the last segment adds to nobody
+    mid[s * state_elems] = x;
+    x = fmaf(f, x, add);
+  }
 }
 
 inline int done() {
@@ -459,17 +505,30 @@ template <int D, int VS>
 int launch_chunked(const XpLinearAttnArgs& a, cudaStream_t s) {
   constexpr int kSmem = chunk_smem_bytes<D, VS>();
   static_assert(kSmem <= 227 * 1024, "chunk buffers exceed the shared memory of an SM");
-  int rc = big_smem(linear_chunked_kernel<D, VS>, kSmem);
+  int rc = big_smem(linear_chunked_kernel<D, VS, true>, kSmem);
+  if (rc == 0) rc = big_smem(linear_chunked_kernel<D, VS, false>, kSmem);
   if (rc != 0) return rc;
-  linear_chunked_kernel<D, VS><<<dim3((a.vdim + VS - 1) / VS, a.heads, a.seqs), kChunkThreads, kSmem, s>>>(a);
+  XpLinearAttnArgs b = a;
+  if (b.segs <= 1) {
+    b.segs = 1;
+    b.seg_tokens = 0x40000000;
+  } else if (b.ws == nullptr || b.seg_tokens <= 0 || b.seg_tokens % kChunk != 0) {
+    return -13;
+  }
+  const dim3 grid((a.vdim + VS - 1) / VS * b.segs, a.heads, a.seqs);
+  if (b.segs > 1) {
+    linear_chunked_kernel<D, VS, false><<<grid, kChunkThreads, kSmem, s>>>(b);
+    linear_scan_kernel<<<dim3((a.dim * a.vdim + 255) / 256, a.heads, a.seqs), 256, 0, s>>>(b);
+  }
+  linear_chunked_kernel<D, VS, true><<<grid, kChunkThreads, kSmem, s>>>(b);
   return done();
 }
 
 template <int D>
 int launch_chunked_any(const XpLinearAttnArgs& a, cudaStream_t s) {
-  // narrow state slices while there are too few CTAs for the 148 SMs: the scores are recomputed per slice
-  if (a.heads * a.seqs * ((a.vdim + 31) / 32) < 148) return launch_chunked<D, 16>(a, s);
-  return launch_chunked<D, 32>(a, s);
+  if (a.vdim <= 32) return launch_chunked<D, 32>(a, s);
+  if (a.vdim <= 64) return launch_chunked<D, 64>(a, s);
+  return launch_chunked<D, 128>(a, s);
 }
 
 template <typename T>
@@ -498,7 +557,7 @@ extern "C" int xp_linear_attn_decode(const XpLinearAttnArgs* a, void* stream) {
   return v ? launch_decode<__nv_bfloat16, 4>(*a, s) : launch_decode<__nv_bfloat16, 1>(*a, s);
 }
 
-// Portion s: q_lens[s] rows from row q_starts[s].
+// Portion s: q_lens[s] rows from row q_starts[s]. segs > 1: every portion has at most segs * seg_tokens rows.
 extern "C" int xp_linear_attn_prefill(const XpLinearAttnArgs* a, void* stream) {
   if (a->seqs <= 0) return 0;
   if (a->heads <= 0 || a->dim <= 0 || a->vdim <= 0) return -10;
@@ -510,5 +569,5 @@ extern "C" int xp_linear_attn_prefill(const XpLinearAttnArgs* a, void* stream) {
   if (!chunked) return launch_sequential_any<__nv_bfloat16>(*a, s);
   if (a->dim <= 64) return launch_chunked_any<64>(*a, s);
   if (a->dim <= 128) return launch_chunked_any<128>(*a, s);
-  return launch_chunked<256, 16>(*a, s);
+  return launch_chunked<256, 32>(*a, s);
 }

@@ -43,6 +43,7 @@ class RowBatch:
     n_seqs: int
     n_dec: int                           # leading rows that are one token each (= leading sequences)
     n_abs: int                           # leading rows of the absorbed form (decoded tokens, then short portions)
+    max_q: int                           # longest portion behind the decoded tokens
     max_len: int                         # bound on positions + 1 of the absorbed rows
     positions: torch.Tensor              # [rows]
     slots: torch.Tensor                  # [rows] cache row, -1: padding
@@ -82,7 +83,7 @@ class LayeredForward:
             self.q_abs = buf(cap * max(m.heads * m.cache_width for m in lat))
             self.o_lat = buf(cap * max(m.heads * ceil8(m.kv_rank) for m in lat))
             buckets = engine._buckets
-            need = max(b * M.latent_attn_plan(b, m.heads, engine.ecfg.max_seq_len)[0] * m.heads * (m.kv_rank + 2)
+            need = max(b * M.latent_attn_plan(b, m.heads, engine.ecfg.max_seq_len, m.cache_width)[0] * m.heads * (m.kv_rank + 2)
                        for b in buckets for m in lat)
             self.attn_ws = buf(max(need, 1 << 20), torch.float32)
         self.ws_tokens = 0
@@ -96,6 +97,7 @@ class LayeredForward:
             self.v_exp = buf(self.ws_tokens * max(H * dv for H, _, dv, _ in shapes))
         if lin:
             self.o_lin = buf(cap * max(m.out_features for m in lin), torch.float32)
+            self.lin_ws = buf(max(M.linear_attn_ws_elems(m.dim, m.vdim) for m in lin) if dt == torch.bfloat16 else 1, torch.float32)
 
     # ------------------------------------------------------------------ mixers
     def _latent(self, l: int, lw: LayeredLayerWeights, m: LatentMixer, proj: torch.Tensor, out: torch.Tensor, b: RowBatch) -> None:
@@ -115,7 +117,7 @@ class LayeredForward:
                       q_abs=q_abs, q_exp=q_exp)
         if n_abs:
             gemm.linear_batched(q_plain[:, :, :m.dim], lw.mix["uk_t"], q_abs, n_abs * W)
-            splits, chunk = M.latent_attn_plan(n_abs, H, b.max_len)
+            splits, chunk = M.latent_attn_plan(n_abs, H, b.max_len, W)
             if splits > 1 and n_abs * H * splits * (R + 2) > self.attn_ws.numel():
                 splits, chunk = 1, 0
             o_lat = self.o_lat[:H * n_abs * rp].view(H, n_abs, rp)
@@ -144,7 +146,9 @@ class LayeredForward:
             M.linear_attn_decode(proj[:b.n_dec], state, dec, pw, o[:b.n_dec], b.positions, b.slots, b.state_slots, **kw)
         if b.n_dec < b.n_seqs:
             s = slice(b.n_dec, b.n_seqs)
-            M.linear_attn_prefill(proj, state, dec, pw, o, b.positions, b.slots, b.state_slots[s], b.q_starts[s], b.q_lens[s], **kw)
+            segs, seg_tokens = M.linear_attn_plan(b.n_seqs - b.n_dec, m.heads, m.dim, m.vdim, b.max_q)
+            M.linear_attn_prefill(proj, state, dec, pw, o, b.positions, b.slots, b.state_slots[s], b.q_starts[s], b.q_lens[s], segs=segs,
+                                  seg_tokens=seg_tokens, ws=self.lin_ws, **kw)
         M.gated_rms(o, lw.mix["norm"], proj[:, lw.offs["g"]:lw.offs["g"] + n], self.e.cfg.rms_norm_eps, out)
 
     # ------------------------------------------------------------------ layers

@@ -277,8 +277,8 @@ LatentAttnArgs = _struct("LatentAttnArgs", "XpLatentAttnArgs", a_ptr="q cache ou
 LatentGatherArgs = _struct("LatentGatherArgs", "XpLatentGatherArgs", a_ptr="cache out block_table ctx_lens q_lens starts",
                            b_int="n_seqs max_len page_size max_blocks ld_cache elem_bytes")
 LinearAttnArgs = _struct("LinearAttnArgs", "XpLinearAttnArgs",
-                         a_ptr="proj state decay decay_pow out positions slots state_slots q_starts q_lens",
-                         b_int="rows seqs heads dim vdim ld_proj q_off k_off v_off force_sequential f32")
+                         a_ptr="proj state decay decay_pow out positions slots state_slots q_starts q_lens ws",
+                         b_int="rows seqs heads dim vdim ld_proj q_off k_off v_off force_sequential segs seg_tokens f32")
 
 
 def _declare_mixers(lib: C.CDLL) -> None:

@@ -187,7 +187,7 @@ def linear(x: torch.Tensor, w: torch.Tensor, *, out: torch.Tensor | None = None,
            num_sms: int = 0, evict_first: bool | None = None, out_scale: float = 0.0, silu_cols: int = 0) -> torch.Tensor:
     """``x[rows, k] @ w[n, k].T`` (* ``out_scale`` unless 0) (+ fp32 ``bias``) (+ ``resid``) on the tcgen05 kernel; fp32
     operands run the plain fp32 kernel. The first ``silu_cols`` features are stored as ``silu(value)``. Any ``n`` and ``k``; bf16 row pitches must be multiples of 16 bytes."""
-    x2 = x.reshape(-1, x.shape[-1])
+    x2 = x if x.dim() == 2 else x.reshape(-1, x.shape[-1])   # reshape would forget the row pitch of a single row
     rows, n = x2.shape[0], w.shape[0]
     if x.dtype == torch.float32:
         if resid is not None:

@@ -113,15 +113,21 @@ def latent_prep(proj: torch.Tensor, norm_w: torch.Tensor, freq: torch.Tensor, po
     native.check(native.kernels().xp_latent_prep(C.byref(a), _stream(proj)), "xp_latent_prep")
 
 
-def latent_attn_plan(rows: int, heads: int, max_len: int) -> tuple[int, int]:
-    """(num_splits, chunk_tokens): slices long enough to amortise a CTA's start, enough CTAs to fill the 148 SMs."""
-    ctas = rows * ((heads + 15) // 16)
-    if ctas >= 592 or max_len <= 256:
-        return 1, 0
-    want = max(1, (296 + ctas - 1) // ctas)
-    chunk = max(128, ((max_len + want - 1) // want + 63) // 64 * 64)
-    splits = (max_len + chunk - 1) // chunk
-    return (splits, chunk) if splits > 1 else (1, 0)
+def latent_attn_plan(rows: int, heads: int, max_len: int, width: int = 576) -> tuple[int, int]:
+    """(num_splits, chunk_tokens) of the absorbed decode kernel: the split count that finishes first, counting a CTA as its
+    64-token tiles plus three for start and merge, with one CTA per SM for wide cache rows and two for narrow ones."""
+    ctas = rows * ((heads + 15) // 16 if heads <= 16 else (heads + 31) // 32)
+    slots = 148 if width > 288 else 296
+    tiles = (max_len + 63) // 64
+    best, best_cost = 1, None
+    for s in range(1, min(64, max(1, tiles // 2)) + 1):
+        per = (tiles + s - 1) // s
+        if s > 1 and (s - 1) * per >= tiles:
+            continue
+        cost = ((ctas * s + slots - 1) // slots) * (per + 3) + (2 if s > 1 else 0)
+        if best_cost is None or cost < best_cost:
+            best, best_cost = s, cost
+    return (best, (tiles + best - 1) // best * 64) if best > 1 else (1, 0)
 
 
 def latent_attn(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, block_table: torch.Tensor, positions: torch.Tensor,
@@ -218,10 +224,37 @@ def linear_attn_decode(proj, state, decay, decay_pow, out, positions, slots, sta
     native.check(native.kernels().xp_linear_attn_decode(C.byref(a), _stream(proj)), "xp_linear_attn_decode")
 
 
+def linear_attn_plan(seqs: int, heads: int, dim: int, vdim: int, max_q: int) -> tuple[int, int]:
+    """(segments, tokens per segment) of the chunked prefill: enough CTAs for the 148 SMs when sequences and heads are few.
+    A segmented run reads keys and values twice and passes its states through memory."""
+    slices = (vdim + 127) // 128 if dim <= 128 else (vdim + 31) // 32
+    ctas, chunks = seqs * heads * slices, (max_q + LINEAR_CHUNK - 1) // LINEAR_CHUNK
+    best, best_cost = 1, None
+    for s in range(1, min(chunks, 64) + 1):
+        per = (chunks + s - 1) // s
+        if s > 1 and (ctas * s > 2 * 148 or (s - 1) * per >= chunks):
+            continue
+        cost = ((ctas * s + 147) // 148) * per * (1.0 if s == 1 else 1.4) + (0 if s == 1 else 4)
+        if best_cost is None or cost < best_cost:
+            best, best_cost = s, cost
+    return best, (chunks + best - 1) // best * LINEAR_CHUNK
+
+
+def linear_attn_ws_elems(dim: int, vdim: int) -> int:
+    """Bound on the workspace of any plan (fp32 elements)."""
+    return 2 * 148 * dim * vdim
+
+
 def linear_attn_prefill(proj, state, decay, decay_pow, out, positions, slots, state_slots, q_starts, q_lens, *, heads: int,
-                        dim: int, vdim: int, offs: tuple[int, int, int], force_sequential: bool = False) -> None:
-    """Portions of sequences: portion i covers rows ``q_starts[i] .. + q_lens[i]`` and continues state ``state_slots[i]``."""
+                        dim: int, vdim: int, offs: tuple[int, int, int], force_sequential: bool = False, segs: int = 1, seg_tokens: int = 0,
+                        ws: torch.Tensor | None = None) -> None:
+    """Portions of sequences: portion i covers rows ``q_starts[i] .. + q_lens[i]`` and continues state ``state_slots[i]``.
+    ``segs`` and ``seg_tokens`` as planned for the longest portion (:func:`linear_attn_plan`), with ``ws`` of
+    ``seqs * heads * segs * dim * vdim`` fp32 elements when ``segs`` > 1."""
     a = _linear_args(proj, state, decay, decay_pow, out, positions, slots, state_slots, heads, dim, vdim, offs)
     a.q_starts, a.q_lens, a.seqs = q_starts.data_ptr(), q_lens.data_ptr(), q_lens.shape[0]
     a.rows, a.force_sequential = proj.shape[0], int(force_sequential)
-    native.check(native.kernels().xp_linear_attn_prefill(C.byref(a), _stream(proj)), "xp_linear_attn_prefill")
+    if segs > 1 and a.f32 == 0 and not force_sequential:
+        assert ws is not None and ws.numel() >= q_lens.shape[0] * heads * segs * dim * vdim
+        a.segs, a.seg_tokens, a.ws = segs, seg_tokens, ws.data_ptr()
+    native.check(native.kernels().xp_linear_attn_prefill(C.byref(a), _stream(proj)), "xp_linear_attn_prefill", 3 if a.segs > 1 else 1)

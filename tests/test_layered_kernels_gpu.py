@@ -263,7 +263,7 @@ def test_expanded_prefill_over_gathered_latents(dim, rot, vdim, heads, page):
 # ------------------------------------------------------------------ linear attention
 
 @pytest.mark.parametrize("heads,dim,vdim", [(2, 48, 24), (3, 20, 7), (1, 200, 136), (4, 128, 128), (2, 64, 32), (1, 8, 16)])
-@pytest.mark.parametrize("form", ["f32", "bf16", "bf16-sequential"])
+@pytest.mark.parametrize("form", ["f32", "bf16", "bf16-sequential", "bf16-segments"])
 def test_linear_attention_portions_and_single_tokens(heads, dim, vdim, form):
     """Three sequences of unequal length in unequal portions, some of two tokens, with single tokens at the end; slots are
     shuffled and hold garbage before."""
@@ -280,14 +280,17 @@ def test_linear_attention_portions_and_single_tokens(heads, dim, vdim, form):
     dec, pw = torch.tensor(decay, device="cuda"), M.decay_powers(decay).cuda()
     kw = dict(heads=heads, dim=dim, vdim=vdim, offs=offs)
     slot, done, got = [2, 0, 3], [0, 0, 0], [[], [], []]
-    for portions in ([2, 64, 0], [64, 0, 63], [67, 2, 0], [65, 0, 0]):
+    for portions in ([2, 64, 0], [64, 0, 63], [130, 2, 0], [5, 0, 0]):
         live = [i for i in range(3) if portions[i]]
         rows = torch.cat([x[i][done[i]:done[i] + portions[i]] for i in live])
         pos = _i32([done[i] + j for i in live for j in range(portions[i])])
         lens = [portions[i] for i in live]
         out = torch.full((len(rows), heads * vdim), 5.0, device="cuda")
+        # segments of one chunk: portions of 64 tokens end with their first segment, longer ones do not
+        segs = dict(segs=3, seg_tokens=64, ws=torch.full((len(live) * 3 * heads * dim * vdim,), float("nan"), device="cuda")) \
+            if form == "bf16-segments" else {}
         M.linear_attn_prefill(rows, state, dec, pw, out, pos, pos, _i32([slot[i] for i in live]), _i32([sum(lens[:j]) for j in range(len(lens))]),
-                              _i32(lens), force_sequential=form == "bf16-sequential", **kw)
+                              _i32(lens), force_sequential=form == "bf16-sequential", **segs, **kw)
         for i, o in zip(live, out.split(lens)):
             got[i].append(o)
             done[i] += portions[i]
@@ -310,3 +313,12 @@ def test_linear_attention_portions_and_single_tokens(heads, dim, vdim, form):
         scale = want.pow(2).mean().sqrt().item()
         assert (torch.cat(got[i]).double().cpu().view_as(want) - want).abs().max().item() < 2e-4 * scale
         assert (state[slot[i]].double().cpu() - S).abs().max().item() < 2e-4 * S.pow(2).mean().sqrt().item()
+
+
+def test_segment_plans_cover_the_portion_and_fit_the_workspace():
+    from crosspool_b200.ops import mixers as M
+
+    for seqs, heads, dim, vdim, q in [(1, 16, 128, 128, 4096), (1, 1, 64, 32, 64), (3, 2, 200, 136, 1000), (40, 16, 128, 128, 100), (1, 1, 256, 256, 9000)]:
+        segs, tokens = M.linear_attn_plan(seqs, heads, dim, vdim, q)
+        assert tokens % 64 == 0 and segs * tokens >= q and (segs - 1) * tokens < q
+        assert segs == 1 or seqs * heads * segs * dim * vdim <= M.linear_attn_ws_elems(dim, vdim)
