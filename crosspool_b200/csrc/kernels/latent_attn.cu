@@ -545,7 +545,15 @@ extern "C" int xp_latent_attn(const XpLatentAttnArgs* a, void* stream) {
   if (a->heads <= 0 || a->kv_rank <= 0 || a->page_size <= 0 || a->rows > a->q_rows || a->ld_q < a->kv_rank + a->rot) return -10;
   if (a->num_splits > 1 && (a->ws == nullptr || a->chunk_tokens <= 0)) return -11;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
-  if (!a->f32 && !a->force_simt && a->kv_rank <= 512 && a->ld_cache % 16 == 0 && a->ld_q % 8 == 0 && a->ld_q >= a->ld_cache) {
+  if (!a->f32 && a->force == 0) {
+    const int rc = xp_latent_attn_umma(a, stream);
+    if (rc < 0) return rc;
+    if (rc == 0) {
+      if (a->num_splits > 1) latent_merge_kernel<<<dim3(a->heads, a->rows), 128, 0, s>>>(*a);
+      return done();
+    }
+  }
+  if (!a->f32 && a->force != 1 && a->kv_rank <= 512 && a->ld_cache % 16 == 0 && a->ld_q % 8 == 0 && a->ld_q >= a->ld_cache) {
     int rc;
     if (a->heads > 16) rc = a->kv_rank <= 128 ? launch_tc<2, 2>(*a, s) : a->kv_rank <= 256 ? launch_tc<4, 2>(*a, s) : launch_tc<8, 2>(*a, s);
     else rc = a->kv_rank <= 128 ? launch_tc<2, 1>(*a, s) : a->kv_rank <= 256 ? launch_tc<4, 1>(*a, s) : launch_tc<8, 1>(*a, s);

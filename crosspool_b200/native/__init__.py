@@ -271,9 +271,9 @@ GatedRmsArgs = _struct("GatedRmsArgs", "XpGatedRmsArgs", a_ptr="o weight gate ou
 LatentPrepArgs = _struct("LatentPrepArgs", "XpLatentPrepArgs", a_ptr="proj norm_w freq positions slots cache q_plain q_abs q_exp",
                          b_int="rows heads dim rot rot_dims kv_rank ld_proj q_off kv_off ld_cache qp_rows dim_p ld_abs dq_pad abs_rows",
                          c_float="eps", d_int="f32")
-LatentAttnArgs = _struct("LatentAttnArgs", "XpLatentAttnArgs", a_ptr="q cache out gate row_seq positions slots block_table ws",
+LatentAttnArgs = _struct("LatentAttnArgs", "XpLatentAttnArgs", a_ptr="q cache out gate row_seq positions slots block_table ws status",
                          b_int="rows heads kv_rank rot q_rows ld_q ld_cache ld_out ld_gate page_size max_blocks num_splits chunk_tokens",
-                         c_float="scale", d_int="f32 force_simt")
+                         c_float="scale", d_int="f32 force num_pages")
 LatentGatherArgs = _struct("LatentGatherArgs", "XpLatentGatherArgs", a_ptr="cache out block_table ctx_lens q_lens starts",
                            b_int="n_seqs max_len page_size max_blocks ld_cache elem_bytes")
 LinearAttnArgs = _struct("LinearAttnArgs", "XpLinearAttnArgs",

@@ -144,7 +144,7 @@ def _paged(lens, page, width, dtype, seed):
 
 @pytest.mark.parametrize("heads,rank,rot", [(1, 30, 6), (3, 56, 16), (17, 200, 32), (16, 512, 64), (2, 120, 8)])
 @pytest.mark.parametrize("page", [16, 64])
-@pytest.mark.parametrize("form", ["f32", "bf16", "bf16-plain", "bf16-split"])
+@pytest.mark.parametrize("form", ["f32", "bf16-umma", "bf16-mma", "bf16-simt", "bf16-umma-split", "bf16-mma-split"])
 def test_latent_attention_of_single_rows(heads, rank, rot, page, form):
     from crosspool_b200.ops import mixers as M
 
@@ -164,10 +164,13 @@ def test_latent_attention_of_single_rows(heads, rank, rot, page, form):
     seq, slots = _i32(list(range(8)) + [6, 0]), _i32([0] * 9 + [-1])
     gate = _rnd(rows, heads + 5, seed=3, dtype=dtype)
     out = torch.full((heads, rows, (rank + 7) // 8 * 8), 5.0, dtype=dtype, device="cuda")
-    splits, chunk = (6, 64) if form == "bf16-split" else (1, 0)
+    splits, chunk = (6, 64) if form.endswith("split") else (1, 0)
     ws = torch.empty(rows * heads * splits * (rank + 2), device="cuda")
     M.latent_attn(q, cache, out, table, pos, slots, kv_rank=rank, rot=rot, scale=0.11, gate=gate, row_seq=seq, num_splits=splits,
-                  chunk_tokens=chunk, ws=ws, force_simt=form == "bf16-plain")
+                  chunk_tokens=chunk, ws=ws, kernel=(form + "-umma").split("-")[1])
+    from crosspool_b200.ops import gemm
+
+    gemm.check_status(torch.device("cuda"))
     for r in range(9):
         k = kv[int(seq[r])][:int(pos[r]) + 1].double()
         s = q[:, r, :rank + rot].double().cpu() @ k[:, :rank + rot].T * 0.11
