@@ -173,7 +173,9 @@ latent_attn_simt_kernel(XpLatentAttnArgs a) {
 }
 
 // ------------------------------------------------------------------------------------------ tensor-core kernel
-constexpr int kTcThreads = 256;          // 8 warps: 4 token groups x 2 halves of the key columns, then 8 column groups
+constexpr int kTcWarps = 8;              // compute warps: 4 token groups x 2 halves of the key columns, then 8 column groups
+constexpr int kTcThreads = kTcWarps * 32 + 32;   // and a producer warp
+constexpr int kTablePages = 512;         // page-table entries of a slice kept in shared memory
 constexpr int kTile = 64;                // tokens per tile
 constexpr int kPPitch = kTile + 8;
 
@@ -209,7 +211,7 @@ __host__ __device__ inline TcLayout tc_layout(int dk16, int vcols, int hg) {
   L.stage_bytes = kTile * L.pitch * 2;
   const int m = 16 * hg;
   L.q_bytes = m * L.pitch * 2;
-  const int fixed = L.q_bytes + 2 * m * kPPitch * 2 + 2 * m * kTile * 4 + 3 * m * 4;
+  const int fixed = 128 + L.q_bytes + 2 * m * kPPitch * 2 + 2 * m * kTile * 4 + 3 * m * 4 + kTablePages * 4;
   int st = (100 * 1024 - fixed) / L.stage_bytes;     // two CTAs per SM when the rows are short
   if (st < 2) st = 2;
   if (st > 4) st = 4;
@@ -218,7 +220,31 @@ __host__ __device__ inline TcLayout tc_layout(int dk16, int vcols, int hg) {
   return L;
 }
 
+__device__ __forceinline__ void bulk_load(uint32_t dst, const void* src, uint32_t bytes, uint32_t bar) {
+  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(dst), "l"(src), "r"(bytes),
+               "r"(bar)
+               : "memory");
+}
+
+// Barrier of the compute warps; true when any of their threads passes true.
+__device__ __forceinline__ bool compute_any(bool p) {
+  uint32_t r;
+  asm volatile(
+      "{\n\t"
+      ".reg .pred a, b;\n\t"
+      "setp.ne.u32 a, %1, 0;\n\t"
+      "barrier.cta.red.or.pred b, 1, %2, a;\n\t"
+      "selp.u32 %0, 1, 0, b;\n\t"
+      "}"
+      : "=r"(r)
+      : "r"(p ? 1u : 0u), "n"(kTcWarps * 32)
+      : "memory");
+  return r != 0;
+}
+
 // NT: 8-column tiles of the latent per warp (kv_rank <= 64 * NT). HG: groups of 16 heads that share a CTA's tiles.
+// A producer warp keeps the ring of tiles full (one bulk copy per cached row), so that the compute warps meet at two
+// barriers per tile only: behind the scores and behind the probabilities.
 template <int NT, int HG>
 __global__ void __launch_bounds__(kTcThreads)
 latent_attn_tc_kernel(XpLatentAttnArgs a) {
@@ -228,12 +254,15 @@ latent_attn_tc_kernel(XpLatentAttnArgs a) {
   const int nh = min(MH, a.heads - h0);
   const int dk16 = a.ld_cache;
   const TcLayout L = tc_layout(dk16, 64 * NT, HG);
-  __nv_bfloat16* q_s = reinterpret_cast<__nv_bfloat16*>(smem);
-  __nv_bfloat16* p_s = reinterpret_cast<__nv_bfloat16*>(smem + L.q_bytes);            // high parts, then low parts
-  float* s_s = reinterpret_cast<float*>(smem + L.q_bytes + 2 * MH * kPPitch * 2);     // [2][MH][kTile]
+  uint64_t* full = reinterpret_cast<uint64_t*>(smem);                                  // [4] tile landed
+  uint64_t* empty = full + 4;                                                          // [4] tile consumed
+  __nv_bfloat16* q_s = reinterpret_cast<__nv_bfloat16*>(smem + 128);
+  __nv_bfloat16* p_s = q_s + L.q_bytes / 2;                                            // high parts, then low parts
+  float* s_s = reinterpret_cast<float*>(p_s + 2 * MH * kPPitch);                       // [2][MH][kTile]
   float* m_s = s_s + 2 * MH * kTile;                                                   // final maximum and sum, tile's factor
   float* l_s = m_s + MH;
   float* f_s = l_s + MH;
+  int* table_s = reinterpret_cast<int*>(f_s + MH);
   uint8_t* ring = smem + L.total - L.stages * L.stage_bytes;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const bool pad = a.slots[row] < 0;
@@ -246,27 +275,50 @@ latent_attn_tc_kernel(XpLatentAttnArgs a) {
   const __nv_bfloat16* cache = reinterpret_cast<const __nv_bfloat16*>(a.cache);
   const int chunks_row = dk16 / 8;                   // 16-byte pieces of a row
 
-  auto issue = [&](int it) {
-    if (it < tiles) {
-      uint8_t* st = ring + (it % L.stages) * L.stage_bytes;
-      // four threads walk one token row: the page lookup is shared by its pieces
-      const int tok = threadIdx.x >> 2;
-      const int t = t0 + it * kTile + tok;
-      const bool ok = t < t1;
-      const int tt = ok ? t : t0;
-      const __nv_bfloat16* src = cache + (static_cast<size_t>(table[tt / a.page_size]) * a.page_size + tt % a.page_size) * dk16;
-      const uint32_t dst = sm100::smem_u32(st + tok * L.pitch * 2);
-      const int sz = ok ? 16 : 0;                    // rows past the slice read as zero
-#pragma unroll 6
-      for (int c = threadIdx.x & 3; c < chunks_row; c += 4)
-        asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst + c * 16), "l"(src + c * 8), "r"(sz));
+  if (threadIdx.x == 0) {
+    for (int i = 0; i < L.stages; ++i) {
+      sm100::mbar_init(&full[i], 1);
+      sm100::mbar_init(&empty[i], kTcWarps);
     }
-    asm volatile("cp.async.commit_group;");
-  };
-  for (int i = 0; i < L.stages - 1; ++i) issue(i);
+    sm100::mbar_fence_init();
+    sm100::fence_proxy_async_smem();
+  }
+  // the slice's page table, so that no copy waits for a lookup in memory
+  const int page0 = t0 / a.page_size, pages = tiles > 0 ? (t1 - 1) / a.page_size - page0 + 1 : 0;
+  const bool cached = pages <= kTablePages;
+  if (cached)
+    for (int i = threadIdx.x; i < pages; i += kTcThreads) table_s[i] = table[page0 + i];
+  __syncthreads();
+
+  if (warp == kTcWarps) {
+    for (int it = 0; it < tiles; ++it) {
+      const int b = it % L.stages, n = min(kTile, t1 - t0 - it * kTile);
+      if (it >= L.stages) {
+        const uint32_t parity = ((it / L.stages) - 1) & 1;
+        const bool ok = sm100::mbar_try_wait(&empty[b], parity) ||
+                        sm100::mbar_wait(&empty[b], parity, sm100::global_timer_ns() + sm100::kPipelineWaitNs);
+        if (!__all_sync(0xffffffffu, ok)) break;       // the compute warps' own wait runs out and reports it
+      }
+      uint8_t* st = ring + b * L.stage_bytes;
+      // rows past the slice: zeros (their probability is zero, but not their memory); this is the last tile
+      for (int i = lane; i < (kTile - n) * chunks_row; i += 32)
+        *reinterpret_cast<uint4*>(st + (n + i / chunks_row) * L.pitch * 2 + (i % chunks_row) * 16) = make_uint4(0, 0, 0, 0);
+      __syncwarp();
+      const uint32_t bar = sm100::smem_u32(&full[b]);
+      if (lane == 0) sm100::mbar_arrive_expect_tx_addr(bar, static_cast<uint32_t>(n * dk16 * 2));
+      __syncwarp();
+      for (int tok = lane; tok < n; tok += 32) {
+        const int t = t0 + it * kTile + tok, page = t / a.page_size;
+        const __nv_bfloat16* src =
+            cache + (static_cast<size_t>(cached ? table_s[page - page0] : table[page]) * a.page_size + (t - page * a.page_size)) * dk16;
+        bulk_load(sm100::smem_u32(st + tok * L.pitch * 2), src, static_cast<uint32_t>(dk16 * 2), bar);
+      }
+    }
+    return;
+  }
 
   // queries of the head groups; absent heads read as zero
-  for (int i = threadIdx.x; i < MH * chunks_row; i += kTcThreads) {
+  for (int i = threadIdx.x; i < MH * chunks_row; i += kTcWarps * 32) {
     const int h = i / chunks_row, c = (i - h * chunks_row) * 8;
     uint4 v = make_uint4(0, 0, 0, 0);
     if (h < nh)
@@ -295,13 +347,14 @@ latent_attn_tc_kernel(XpLatentAttnArgs a) {
 #pragma unroll
       for (int e = 0; e < 4; ++e) acc[hg][j][e] = 0.f;
 
+  bool failed = false;
+  compute_any(false);                                // queries are in place
   for (int it = 0; it < tiles; ++it) {
-    if (L.stages == 2) asm volatile("cp.async.wait_group 0;" ::: "memory");
-    else if (L.stages == 3) asm volatile("cp.async.wait_group 1;" ::: "memory");
-    else asm volatile("cp.async.wait_group 2;" ::: "memory");
-    __syncthreads();                                 // tile it landed; everyone is done with the tile before it
-    issue(it + L.stages - 1);
-    const uint32_t st = sm100::smem_u32(ring + (it % L.stages) * L.stage_bytes);
+    const int b = it % L.stages;
+    const uint32_t parity = (it / L.stages) & 1;
+    const bool ok = sm100::mbar_try_wait(&full[b], parity) ||
+                    sm100::mbar_wait(&full[b], parity, sm100::global_timer_ns() + sm100::kPipelineWaitNs);
+    const uint32_t st = sm100::smem_u32(ring + b * L.stage_bytes);
     // scores of 16 tokens over this warp's half of the columns; even and odd steps in chains of their own
     float sc[2][HG][2][4];
 #pragma unroll
@@ -332,7 +385,8 @@ latent_attn_tc_kernel(XpLatentAttnArgs a) {
         for (int r = 0; r < 2; ++r)
           *reinterpret_cast<float2*>(s_s + (kh * MH + hg * 16 + g + r * 8) * kTile + tg * 16 + u * 8 + q4 * 2) =
               make_float2(sc[0][hg][u][2 * r] + sc[1][hg][u][2 * r], sc[0][hg][u][2 * r + 1] + sc[1][hg][u][2 * r + 1]);
-    __syncthreads();
+    failed = compute_any(!ok);
+    if (failed) break;
     // softmax: MW heads per warp (independent chains), two tokens per lane
     const int tok0 = t0 + it * kTile + lane * 2;
     float v[MW][2], mx[MW], sum[MW];
@@ -364,7 +418,7 @@ latent_attn_tc_kernel(XpLatentAttnArgs a) {
       *reinterpret_cast<__nv_bfloat162*>(p_s + (MH + h) * kPPitch + lane * 2) = __floats2bfloat162_rn(p0 - hf.x, p1 - hf.y);
       if (lane == 0) f_s[h] = f;
     }
-    __syncthreads();
+    compute_any(false);
     // the sums are off the critical path: their shuffles overlap the second product
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1)
@@ -399,15 +453,21 @@ latent_attn_tc_kernel(XpLatentAttnArgs a) {
         }
       }
     }
+    __syncwarp();
+    if (lane == 0) sm100::mbar_arrive(&empty[b]);
   }
-  asm volatile("cp.async.wait_group 0;" ::: "memory");
+  if (failed) {
+    if (threadIdx.x == 0 && a.status != nullptr) atomicCAS(a.status, 0u, 8u);
+    __nanosleep(1000000);   // copies still in flight get a bounded chance to land before the CTA retires
+    return;
+  }
 #pragma unroll
   for (int r = 0; r < MW; ++r)
     if (lane == 0) {
       m_s[warp * MW + r] = m_run[r];
       l_s[warp * MW + r] = l_run[r];
     }
-  __syncthreads();
+  compute_any(false);
 #pragma unroll
   for (int hg = 0; hg < HG; ++hg)
 #pragma unroll
