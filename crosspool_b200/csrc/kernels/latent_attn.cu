@@ -190,11 +190,16 @@ __device__ __forceinline__ void ldsm_x4_trans(uint32_t addr, uint32_t (&r)[4]) {
                : "r"(addr));
 }
 __device__ __forceinline__ void mma16816(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile(
+  asm(
       "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
       : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
       : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
+
+template <int V>
+struct Count {
+  static constexpr int value = V;
+};
 
 struct TcLayout {
   int pitch;        // elements of one shared-memory row (an odd multiple of 16 bytes: conflict-free ldmatrix)
@@ -359,24 +364,28 @@ latent_attn_tc_kernel(XpLatentAttnArgs a) {
     float sc[2][HG][2][4];
 #pragma unroll
     for (int i = 0; i < 2 * HG * 2 * 4; ++i) (&sc[0][0][0][0])[i] = 0.f;
-    auto score_step = [&](int ks, float (&c)[HG][2][4]) {
-      uint32_t kb[4];
-      ldsm_x4(st + k_lane + ks * 32, kb);
+    // kGroup steps at a time: all their fragments are requested before the first product
+    auto score_steps = [&](int ks, auto count) {
+      constexpr int kGroup = decltype(count)::value;
+      uint32_t kb[kGroup][4], qa[kGroup][HG][4];
 #pragma unroll
-      for (int hg = 0; hg < HG; ++hg) {
-        uint32_t qa[4];
-        ldsm_x4(q_addr + hg * q_group + ks * 32, qa);
-        mma16816(c[hg][0], qa, kb[0], kb[1]);
-        mma16816(c[hg][1], qa, kb[2], kb[3]);
+      for (int i = 0; i < kGroup; ++i) {
+        ldsm_x4(st + k_lane + (ks + i) * 32, kb[i]);
+#pragma unroll
+        for (int hg = 0; hg < HG; ++hg) ldsm_x4(q_addr + hg * q_group + (ks + i) * 32, qa[i][hg]);
       }
+#pragma unroll
+      for (int i = 0; i < kGroup; ++i)
+#pragma unroll
+        for (int hg = 0; hg < HG; ++hg) {
+          mma16816(sc[i & 1][hg][0], qa[i][hg], kb[i][0], kb[i][1]);
+          mma16816(sc[i & 1][hg][1], qa[i][hg], kb[i][2], kb[i][3]);
+        }
     };
     int ks = ks0;
-#pragma unroll 3
-    for (; ks + 1 < ks1; ks += 2) {
-      score_step(ks, sc[0]);
-      score_step(ks + 1, sc[1]);
-    }
-    if (ks < ks1) score_step(ks, sc[0]);
+    for (; ks + 6 <= ks1; ks += 6) score_steps(ks, Count<6>{});
+    for (; ks + 2 <= ks1; ks += 2) score_steps(ks, Count<2>{});
+    if (ks < ks1) score_steps(ks, Count<1>{});
 #pragma unroll
     for (int hg = 0; hg < HG; ++hg)
 #pragma unroll
@@ -440,18 +449,18 @@ latent_attn_tc_kernel(XpLatentAttnArgs a) {
         ldsm_x4(p_addr + hg * 16 * kPPitch * 2 + kk * 32, ph[hg]);
         ldsm_x4(p_addr + (MH + hg * 16) * kPPitch * 2 + kk * 32, pl[hg]);
       }
+      uint32_t vb[NT / 2][4];
 #pragma unroll
-      for (int j = 0; j < NT; j += 2) {
-        uint32_t vb[4];
-        ldsm_x4_trans(st + v_lane + kk * 16 * L.pitch * 2 + j * 16, vb);
+      for (int j = 0; j < NT / 2; ++j) ldsm_x4_trans(st + v_lane + kk * 16 * L.pitch * 2 + j * 32, vb[j]);
+      // high parts of every column tile, then low parts: products on one accumulator stay far apart
 #pragma unroll
-        for (int hg = 0; hg < HG; ++hg) {
-          mma16816(acc[hg][j], ph[hg], vb[0], vb[1]);
-          mma16816(acc[hg][j + 1], ph[hg], vb[2], vb[3]);
-          mma16816(acc[hg][j], pl[hg], vb[0], vb[1]);
-          mma16816(acc[hg][j + 1], pl[hg], vb[2], vb[3]);
-        }
-      }
+      for (int hg = 0; hg < HG; ++hg)
+#pragma unroll
+        for (int j = 0; j < NT; ++j) mma16816(acc[hg][j], ph[hg], vb[j / 2][(j & 1) * 2], vb[j / 2][(j & 1) * 2 + 1]);
+#pragma unroll
+      for (int hg = 0; hg < HG; ++hg)
+#pragma unroll
+        for (int j = 0; j < NT; ++j) mma16816(acc[hg][j], pl[hg], vb[j / 2][(j & 1) * 2], vb[j / 2][(j & 1) * 2 + 1]);
     }
     __syncwarp();
     if (lane == 0) sm100::mbar_arrive(&empty[b]);
