@@ -158,8 +158,8 @@ linear_sequential_kernel(XpLinearAttnArgs a) {
 // CTA = (segment of a portion, VS state columns, head, sequence); it walks its segment in chunks of 64 tokens with the
 // state in registers. With p(n) = decay^n, for row i of a chunk of n tokens and the state S before it:
 //   o_i = p(i + 1) S^T q_i + sum_{j <= i} p(i - j) (q_i . k_j) v_j          (warp: 16 rows, half of the columns)
-//   S   <- p(n) S + sum_j k_j (p(n - 1 - j) v_j)^T                          (warp: its 16-row tiles of S)
-// Decayed scores, decayed values and the state enter their products as bf16 pairs (high and low part), so everything
+//   S   <- p(n) S + sum_j (p(n - 1 - j) k_j) v_j^T                          (warp: its 16-row tiles of S)
+// Decayed scores, decayed keys and the state enter their products as bf16 pairs (high and low part), so everything
 // that belongs to the recurrence keeps at least 16 mantissa bits; the sums are fp32.
 //
 // A long portion with few heads is cut into segments that run at the same time: a first pass computes what each segment
@@ -182,7 +182,7 @@ __device__ __forceinline__ void ldsm4t(uint32_t addr, uint32_t (&r)[4]) {
                : "r"(addr));
 }
 __device__ __forceinline__ void mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile(
+  asm(
       "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
       : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
       : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
@@ -198,8 +198,8 @@ __device__ __forceinline__ void split2(float x, float y, uint32_t& hi, uint32_t&
 
 template <int D, int VS>
 constexpr int chunk_smem_bytes() {
-  // q, k [2][64][D + 8]; v [2][64][VS + 8]; decayed v pair [2][64][VS + 8]; state pair [2][D][VS + 8]; powers
-  return (4 * kChunk * (D + 8) + 2 * kChunk * (VS + 8) + 2 * kChunk * (VS + 8) + 2 * D * (VS + 8)) * 2 + (kChunk + 1 + 3) * 4;
+  // q, k [2][64][D + 8]; v [2][64][VS + 8]; state pair [2][D][VS + 8]; powers
+  return (4 * kChunk * (D + 8) + 2 * kChunk * (VS + 8) + 2 * D * (VS + 8)) * 2 + (kChunk + 1 + 3) * 4;
 }
 
 // kFull: outputs and the state; otherwise only what the segment adds to the state.
@@ -214,8 +214,7 @@ linear_chunked_kernel(XpLinearAttnArgs a) {
   __nv_bfloat16* q_s = reinterpret_cast<__nv_bfloat16*>(smem);
   __nv_bfloat16* k_s = q_s + 2 * kChunk * PD;
   __nv_bfloat16* v_s = k_s + 2 * kChunk * PD;
-  __nv_bfloat16* vd_s = v_s + 2 * kChunk * PV;       // decayed values: high parts, low parts
-  __nv_bfloat16* st_s = vd_s + 2 * kChunk * PV;      // state: high parts, low parts
+  __nv_bfloat16* st_s = v_s + 2 * kChunk * PV;       // state: high parts, low parts
   float* pw = reinterpret_cast<float*>(st_s + 2 * D * PV);
   const int slices = (a.vdim + VS - 1) / VS;
   const int seg = blockIdx.x / slices, c0 = (blockIdx.x % slices) * VS;
@@ -241,25 +240,30 @@ linear_chunked_kernel(XpLinearAttnArgs a) {
   for (int i = threadIdx.x; i <= kChunk; i += kChunkThreads) pw[i] = a.decay_pow[h * (kChunk + 1) + i];
 
   auto copy = [&](__nv_bfloat16* dst, const __nv_bfloat16* src, bool ok) {
-    const int sz = ok ? 16 : 0;
+    const int sz = ok ? 16 : 0;                      // rows and columns out of range read as zero
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(sm100::smem_u32(dst)), "l"(src), "r"(sz));
   };
   auto issue = [&](int c) {
     if (c < chunks) {
       const int b = c & 1, m = min(kChunk, n - c * kChunk);
-      const int per = a.dim / 8;
-      for (int i = threadIdx.x; i < kChunk * per; i += kChunkThreads) {
-        const int t = i / per, e = (i - t * per) * 8;
-        const bool ok = t < m;
-        const __nv_bfloat16* row = proj + static_cast<size_t>(r0 + c * kChunk + (ok ? t : 0)) * a.ld_proj + h * a.dim + e;
-        if (kFull) copy(q_s + (b * kChunk + t) * PD + e, row + a.q_off, ok);
-        copy(k_s + (b * kChunk + t) * PD + e, row + a.k_off, ok);
+      const __nv_bfloat16* rows = proj + static_cast<size_t>(r0 + c * kChunk) * a.ld_proj;
+      constexpr int kPieces = D / 8, kRows = kChunkThreads / kPieces;       // a row's 16-byte pieces; rows covered at a time
+      const int e = (threadIdx.x % kPieces) * 8;
+      if (e < a.dim) {
+#pragma unroll
+        for (int t = threadIdx.x / kPieces; t < kChunk; t += kRows) {
+          const bool ok = t < m;
+          const __nv_bfloat16* row = rows + static_cast<size_t>(ok ? t : 0) * a.ld_proj + h * a.dim + e;
+          if (kFull) copy(q_s + (b * kChunk + t) * PD + e, row + a.q_off, ok);
+          copy(k_s + (b * kChunk + t) * PD + e, row + a.k_off, ok);
+        }
       }
-      for (int i = threadIdx.x; i < kChunk * (VS / 8); i += kChunkThreads) {
-        const int t = i / (VS / 8), e = (i % (VS / 8)) * 8;
-        const bool ok = t < m && c0 + e < a.vdim;
-        copy(v_s + (b * kChunk + t) * PV + e,
-             proj + static_cast<size_t>(r0 + c * kChunk + (t < m ? t : 0)) * a.ld_proj + a.v_off + h * a.vdim + (ok ? c0 + e : 0), ok);
+      constexpr int kVPieces = VS / 8, kVRows = kChunkThreads / kVPieces;
+      const int ev = (threadIdx.x % kVPieces) * 8;
+#pragma unroll
+      for (int t = threadIdx.x / kVPieces; t < kChunk; t += kVRows) {
+        const bool ok = t < m && c0 + ev < a.vdim;
+        copy(v_s + (b * kChunk + t) * PV + ev, rows + static_cast<size_t>(t < m ? t : 0) * a.ld_proj + a.v_off + h * a.vdim + (ok ? c0 + ev : 0), ok);
       }
     }
     asm volatile("cp.async.commit_group;");
@@ -314,18 +318,6 @@ linear_chunked_kernel(XpLinearAttnArgs a) {
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();                                 // chunk c landed, state published, buffers of chunk c - 1 free
     issue(c + 1);
-    // decayed values of the state update
-    for (int i = threadIdx.x; i < kChunk * (VS / 4); i += kChunkThreads) {
-      const int t = i / (VS / 4), e = (i % (VS / 4)) * 4;
-      const float w = t < m ? pw[m - 1 - t] : 0.f;
-      float v[4];
-      elem::ldv<4>(v_s + (b * kChunk + t) * PV + e, v);
-      uint2 hi, lo;
-      split2(v[0] * w, v[1] * w, hi.x, lo.x);
-      split2(v[2] * w, v[3] * w, hi.y, lo.y);
-      *reinterpret_cast<uint2*>(vd_s + t * PV + e) = hi;
-      *reinterpret_cast<uint2*>(vd_s + (kChunk + t) * PV + e) = lo;
-    }
     const uint32_t kb = sm100::smem_u32(k_s + b * kChunk * PD);
     if constexpr (kFull) {
       const uint32_t qb = sm100::smem_u32(q_s + b * kChunk * PD) + a_off;
@@ -404,9 +396,9 @@ linear_chunked_kernel(XpLinearAttnArgs a) {
       }
       if (c + 1 == chunks && !last) break;           // the next segment has its own start state
     }
-    __syncthreads();                                 // decayed values written; everyone is done with the published state
+    if (kFull) __syncthreads();                      // everyone is done with the published state
     const float pn = pw[m];
-    const uint32_t db = sm100::smem_u32(vd_s) + t_off + s0 * 2;
+    const uint32_t vt = sm100::smem_u32(v_s + b * kChunk * PV) + t_off + s0 * 2;
 #pragma unroll
     for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
@@ -415,20 +407,33 @@ linear_chunked_kernel(XpLinearAttnArgs a) {
         for (int e = 0; e < 4; ++e) s[mt][j][e] *= pn;
 #pragma unroll
     for (int kk = 0; kk < kChunk / 16; ++kk) {
-      uint32_t ka[MT][4];
+      // keys of 16 tokens with their decay, as a bf16 pair
+      const int t = kk * 16 + q4 * 2;
+      auto w = [&](int tok) { return tok < m ? pw[m - 1 - tok] : 0.f; };
+      const float w0 = w(t), w1 = w(t + 1), w8 = w(t + 8), w9 = w(t + 9);
+      uint32_t hi[MT][4], lo[MT][4];
 #pragma unroll
-      for (int mt = 0; mt < MT; ++mt) ldsm4t(kb + kt_off + (kk * 16 * PD + mt * 16) * 2, ka[mt]);
+      for (int mt = 0; mt < MT; ++mt) {
+        uint32_t ka[4];
+        ldsm4t(kb + kt_off + (kk * 16 * PD + mt * 16) * 2, ka);
 #pragma unroll
-      for (int j = 0; j < NS; j += 2) {
-        uint32_t hi[4], lo[4];
-        ldsm4t(db + (kk * 16 * PV + j * 8) * 2, hi);
-        ldsm4t(db + ((kChunk + kk * 16) * PV + j * 8) * 2, lo);
+        for (int i = 0; i < 4; ++i) {
+          const float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&ka[i]));
+          split2(x.x * (i < 2 ? w0 : w8), x.y * (i < 2 ? w1 : w9), hi[mt][i], lo[mt][i]);
+        }
+      }
+      constexpr int kGroup = NS < 8 ? NS : 8;        // value tiles whose fragments are live at a time
+#pragma unroll
+      for (int j0 = 0; j0 < NS; j0 += kGroup) {
+        uint32_t vf[kGroup / 2][4];
+#pragma unroll
+        for (int j = 0; j < kGroup / 2; ++j) ldsm4t(vt + (kk * 16 * PV + (j0 + 2 * j) * 8) * 2, vf[j]);
 #pragma unroll
         for (int mt = 0; mt < MT; ++mt) {
-          mma(s[mt][j], ka[mt], hi[0], hi[1]);
-          mma(s[mt][j + 1], ka[mt], hi[2], hi[3]);
-          mma(s[mt][j], ka[mt], lo[0], lo[1]);
-          mma(s[mt][j + 1], ka[mt], lo[2], lo[3]);
+#pragma unroll
+          for (int j = 0; j < kGroup; ++j) mma(s[mt][j0 + j], hi[mt], vf[j / 2][(j & 1) * 2], vf[j / 2][(j & 1) * 2 + 1]);
+#pragma unroll
+          for (int j = 0; j < kGroup; ++j) mma(s[mt][j0 + j], lo[mt], vf[j / 2][(j & 1) * 2], vf[j / 2][(j & 1) * 2 + 1]);
         }
       }
     }
