@@ -83,13 +83,12 @@ typedef struct XpLatentAttnArgs {
   const int* slots;      /* [rows] < 0: padding row (zeros are stored) */
   const int* block_table;
   float* ws;             /* split partials */
-  uint32_t* status;      /* optional, FOUR words: [0] set to 8 when a bounded wait ran out, [1..3] its detail */
+  uint32_t* status;      /* optional: set to 8 when a bounded wait ran out */
   int rows, heads, kv_rank, rot, q_rows, ld_q, ld_cache, ld_out, ld_gate, page_size, max_blocks;
   int num_splits, chunk_tokens;
   float scale;
   int f32;
-  int force;             /* 0 tcgen05 kernel (falls back when the shape is outside it), 1 plain kernel, 2 mma.sync kernel */
-  int num_pages;         /* pages in the cache (bound of the tensor map); 0: no tcgen05 kernel */
+  int force_simt;        /* plain kernel */
 } XpLatentAttnArgs;
 
 /* Copies the cached latents of each sequence to a dense workspace: sequence i's ctx + q tokens start at row starts[i]. */
@@ -128,7 +127,6 @@ int xp_polynorm(const XpPolyNormArgs* a, void* stream);
 int xp_gated_rms(const XpGatedRmsArgs* a, void* stream);
 int xp_latent_prep(const XpLatentPrepArgs* a, void* stream);
 int xp_latent_attn(const XpLatentAttnArgs* a, void* stream);
-int xp_latent_attn_umma(const XpLatentAttnArgs* a, void* stream);
 int xp_latent_gather(const XpLatentGatherArgs* a, void* stream);
 int xp_linear_attn_decode(const XpLinearAttnArgs* a, void* stream);
 int xp_linear_attn_prefill(const XpLinearAttnArgs* a, void* stream);

@@ -108,22 +108,6 @@ inline int encode_q_3d(CUtensorMap* out, const void* base, uint64_t rows, uint32
   return r == CUDA_SUCCESS ? 0 : static_cast<int>(r);
 }
 
-// Head-major rows [heads, rows, cols] (bf16) as a 3-D map whose box is 64 columns of `box_heads` heads of one row: it lands
-// in shared memory as box_heads rows of 128 bytes. Columns, rows and heads out of range read as zero.
-inline int encode_heads_3d(CUtensorMap* out, const void* base, uint64_t cols, uint64_t rows, uint64_t heads, uint32_t box_heads) {
-  EncodeFn fn = encode_fn();
-  if (fn == nullptr) return -1;
-  if ((reinterpret_cast<uintptr_t>(base) & 15) != 0 || cols % 8 != 0 || box_heads == 0 || box_heads > 256) return -2;
-  cuuint64_t dims[3] = {cols, rows, heads};
-  cuuint64_t strides[2] = {cols * 2, cols * 2 * rows};
-  cuuint32_t box[3] = {64, 1, box_heads};
-  cuuint32_t estr[3] = {1, 1, 1};
-  CUresult r = fn(out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(base), dims, strides, box, estr,
-                  CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
-                  CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
-  return r == CUDA_SUCCESS ? 0 : static_cast<int>(r);
-}
-
 // Small cache: encoding costs a few microseconds and serving reuses the same
 // (pointer, shape) pairs on every step.
 class Cache {
@@ -192,23 +176,6 @@ class Cache {
     }
     CUtensorMap m;
     int rc = encode_q_3d(&m, base, rows, q_heads, head_dim, heads, positions);
-    if (rc != 0) return rc;
-    if (map_.size() > 8192) map_.clear();
-    map_.emplace(k, m);
-    *out = m;
-    return 0;
-  }
-
-  int get_heads(CUtensorMap* out, const void* base, uint64_t cols, uint64_t rows, uint32_t heads, uint32_t box_heads) {
-    Key k{base, cols, rows, heads, box_heads, 6};
-    std::lock_guard<std::mutex> g(mu_);
-    auto it = map_.find(k);
-    if (it != map_.end()) {
-      *out = it->second;
-      return 0;
-    }
-    CUtensorMap m;
-    int rc = encode_heads_3d(&m, base, cols, rows, heads, box_heads);
     if (rc != 0) return rc;
     if (map_.size() > 8192) map_.clear();
     map_.emplace(k, m);

@@ -3,14 +3,15 @@
 //   latent_prep       per token: latent RMS norm, rotary on the shared key part and on every query head, cache write,
 //                     query layouts of the two forms below
 //   latent_attn_tc    absorbed form (queries already multiplied into the latent space), one token row and up to 32 heads
-//                     per CTA, split over the sequence: cp.async ring of 64-token tiles, ldmatrix + mma.m16n8k16, the
+//                     per CTA, split over the sequence: a producer warp fills a ring of 64-token tiles; ldmatrix + mma.m16n8k16, the
 //                     probabilities carried as a bf16 pair (high and low part). Bound by reading the cache once.
 //   latent_attn_simt  the same in plain FMAs for any sizes and for fp32
 //   latent_gather     dense copy of a sequence's cached rows, the input of the expanded form (keys and values per head,
 //                     chunked prefill on the tcgen05 kernel of attn_prefill_umma.cu)
 //
-// mma.sync rather than tcgen05 in the absorbed decode kernel: 16 or 32 query rows per cache row are 64 or 128 flop per loaded
-// element, far below the tensor roofline, and a UMMA tile needs 64 or 128 query rows.
+// mma.sync rather than tcgen05 in the absorbed decode kernel: a UMMA tile needs 64 or 128 query rows where there are 16 or 32.
+// With tokens and latent columns on the M axis instead (heads on N), the fixed cost of the small-N instructions and the
+// round trip of the scores through tensor memory made a tcgen05 form a third slower than this one.
 #include <math_constants.h>
 
 #include "xpool/elem.cuh"
@@ -614,15 +615,7 @@ extern "C" int xp_latent_attn(const XpLatentAttnArgs* a, void* stream) {
   if (a->heads <= 0 || a->kv_rank <= 0 || a->page_size <= 0 || a->rows > a->q_rows || a->ld_q < a->kv_rank + a->rot) return -10;
   if (a->num_splits > 1 && (a->ws == nullptr || a->chunk_tokens <= 0)) return -11;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
-  if (!a->f32 && a->force == 0) {
-    const int rc = xp_latent_attn_umma(a, stream);
-    if (rc < 0) return rc;
-    if (rc == 0) {
-      if (a->num_splits > 1) latent_merge_kernel<<<dim3(a->heads, a->rows), 128, 0, s>>>(*a);
-      return done();
-    }
-  }
-  if (!a->f32 && a->force != 1 && a->kv_rank <= 512 && a->ld_cache % 16 == 0 && a->ld_q % 8 == 0 && a->ld_q >= a->ld_cache) {
+  if (!a->f32 && !a->force_simt && a->kv_rank <= 512 && a->ld_cache % 16 == 0 && a->ld_q % 8 == 0 && a->ld_q >= a->ld_cache) {
     int rc;
     if (a->heads > 16) rc = a->kv_rank <= 128 ? launch_tc<2, 2>(*a, s) : a->kv_rank <= 256 ? launch_tc<4, 2>(*a, s) : launch_tc<8, 2>(*a, s);
     else rc = a->kv_rank <= 128 ? launch_tc<2, 1>(*a, s) : a->kv_rank <= 256 ? launch_tc<4, 1>(*a, s) : launch_tc<8, 1>(*a, s);

@@ -273,7 +273,7 @@ LatentPrepArgs = _struct("LatentPrepArgs", "XpLatentPrepArgs", a_ptr="proj norm_
                          c_float="eps", d_int="f32")
 LatentAttnArgs = _struct("LatentAttnArgs", "XpLatentAttnArgs", a_ptr="q cache out gate row_seq positions slots block_table ws status",
                          b_int="rows heads kv_rank rot q_rows ld_q ld_cache ld_out ld_gate page_size max_blocks num_splits chunk_tokens",
-                         c_float="scale", d_int="f32 force num_pages")
+                         c_float="scale", d_int="f32 force_simt")
 LatentGatherArgs = _struct("LatentGatherArgs", "XpLatentGatherArgs", a_ptr="cache out block_table ctx_lens q_lens starts",
                            b_int="n_seqs max_len page_size max_blocks ld_cache elem_bytes")
 LinearAttnArgs = _struct("LinearAttnArgs", "XpLinearAttnArgs",

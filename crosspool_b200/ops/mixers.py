@@ -133,10 +133,9 @@ def latent_attn_plan(rows: int, heads: int, max_len: int, width: int = 576) -> t
 def latent_attn(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, block_table: torch.Tensor, positions: torch.Tensor,
                 slots: torch.Tensor, *, kv_rank: int, rot: int, scale: float, gate: torch.Tensor | None = None,
                 row_seq: torch.Tensor | None = None, num_splits: int = 1, chunk_tokens: int = 0, ws: torch.Tensor | None = None,
-                kernel: str = "umma") -> torch.Tensor:
+                force_simt: bool = False) -> torch.Tensor:
     """Rows of latent-space queries ``q`` ``[heads, rows, width]`` against the latent cache; ``out`` ``[heads, rows, >= kv_rank]``.
-    Row ``r`` attends to the first ``positions[r] + 1`` tokens of its sequence. ``kernel``: "umma" (tcgen05; shapes it does
-    not cover fall back), "mma" (mma.sync) or "simt"."""
+    Row ``r`` attends to the first ``positions[r] + 1`` tokens of its sequence. ``force_simt`` selects the plain kernel."""
     a = native.LatentAttnArgs()
     heads, rows = q.shape[0], q.shape[1]
     a.q, a.cache, a.out, a.gate, a.row_seq = q.data_ptr(), cache.data_ptr(), out.data_ptr(), _ptr(gate), _ptr(row_seq)
@@ -146,8 +145,7 @@ def latent_attn(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, block_t
     a.ld_gate = gate.stride(0) if gate is not None else 0
     a.page_size, a.max_blocks, a.num_splits, a.chunk_tokens = cache.shape[1], block_table.stride(0), num_splits, chunk_tokens
     assert num_splits == 1 or ws.numel() >= rows * heads * num_splits * (kv_rank + 2)
-    a.scale, a.f32, a.force = scale, _f32(q), {"umma": 0, "simt": 1, "mma": 2}[kernel]
-    a.num_pages = cache.shape[0] if cache.is_contiguous() else 0
+    a.scale, a.f32, a.force_simt = scale, _f32(q), int(force_simt)
     from .gemm import status_words
 
     a.status = status_words(q.device).data_ptr()

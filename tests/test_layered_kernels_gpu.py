@@ -144,7 +144,7 @@ def _paged(lens, page, width, dtype, seed):
 
 @pytest.mark.parametrize("heads,rank,rot", [(1, 30, 6), (3, 56, 16), (17, 200, 32), (16, 512, 64), (2, 120, 8)])
 @pytest.mark.parametrize("page", [16, 64])
-@pytest.mark.parametrize("form", ["f32", "bf16-umma", "bf16-mma", "bf16-simt", "bf16-umma-split", "bf16-mma-split"])
+@pytest.mark.parametrize("form", ["f32", "bf16", "bf16-plain", "bf16-split"])
 def test_latent_attention_of_single_rows(heads, rank, rot, page, form):
     from crosspool_b200.ops import mixers as M
 
@@ -167,7 +167,7 @@ def test_latent_attention_of_single_rows(heads, rank, rot, page, form):
     splits, chunk = (6, 64) if form.endswith("split") else (1, 0)
     ws = torch.empty(rows * heads * splits * (rank + 2), device="cuda")
     M.latent_attn(q, cache, out, table, pos, slots, kv_rank=rank, rot=rot, scale=0.11, gate=gate, row_seq=seq, num_splits=splits,
-                  chunk_tokens=chunk, ws=ws, kernel=(form + "-umma").split("-")[1])
+                  chunk_tokens=chunk, ws=ws, force_simt=form == "bf16-plain")
     from crosspool_b200.ops import gemm
 
     gemm.check_status(torch.device("cuda"))
