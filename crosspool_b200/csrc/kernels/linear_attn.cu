@@ -48,23 +48,28 @@ linear_decode_kernel(XpLinearAttnArgs a) {
       elem::ldv<N>(proj + a.v_off + h * a.vdim + c, v);
 #pragma unroll
       for (int j = 0; j < N; ++j) acc[j] = 0.f;
-#pragma unroll 8
-      for (int i = gi; i < a.dim; i += groups) {
-        float s[N];
-        float* p = S + static_cast<size_t>(i) * a.vdim + c;
-        if (fresh) {
+      // kAhead rows are requested before the first of them is stored back (a store would hold back later loads)
+      constexpr int kAhead = 8;
+      for (int i0 = gi; i0 < a.dim; i0 += groups * kAhead) {
+        float s[kAhead][N];
 #pragma unroll
-          for (int j = 0; j < N; ++j) s[j] = 0.f;
-        } else {
-          elem::ldv<N>(p, s);
-        }
-        const float ki = k_s[i], qi = q_s[i];
+        for (int u = 0; u < kAhead; ++u) {
 #pragma unroll
-        for (int j = 0; j < N; ++j) {
-          s[j] = fmaf(ki, v[j], decay * s[j]);
-          acc[j] = fmaf(qi, s[j], acc[j]);
+          for (int j = 0; j < N; ++j) s[u][j] = 0.f;
+          if (!fresh && i0 + u * groups < a.dim) elem::ldv<N>(S + static_cast<size_t>(i0 + u * groups) * a.vdim + c, s[u]);
         }
-        elem::stv<N>(p, s);
+#pragma unroll
+        for (int u = 0; u < kAhead; ++u) {
+          const int i = i0 + u * groups;
+          if (i >= a.dim) break;
+          const float ki = k_s[i], qi = q_s[i];
+#pragma unroll
+          for (int j = 0; j < N; ++j) {
+            s[u][j] = fmaf(ki, v[j], decay * s[u][j]);
+            acc[j] = fmaf(qi, s[u][j], acc[j]);
+          }
+          elem::stv<N>(S + static_cast<size_t>(i) * a.vdim + c, s[u]);
+        }
       }
 #pragma unroll
       for (int j = 0; j < N; ++j) part[gi * a.vdim + c + j] = acc[j];
