@@ -144,7 +144,7 @@ def _paged(lens, page, width, dtype, seed):
 
 @pytest.mark.parametrize("heads,rank,rot", [(1, 30, 6), (3, 56, 16), (17, 200, 32), (16, 512, 64), (2, 120, 8)])
 @pytest.mark.parametrize("page", [16, 64])
-@pytest.mark.parametrize("form", ["f32", "bf16", "bf16-plain", "bf16-split"])
+@pytest.mark.parametrize("form", ["f32", "bf16", "bf16-plain", "bf16-split6", "bf16-split3"])
 def test_latent_attention_of_single_rows(heads, rank, rot, page, form):
     from crosspool_b200.ops import mixers as M
 
@@ -164,7 +164,7 @@ def test_latent_attention_of_single_rows(heads, rank, rot, page, form):
     seq, slots = _i32(list(range(8)) + [6, 0]), _i32([0] * 9 + [-1])
     gate = _rnd(rows, heads + 5, seed=3, dtype=dtype)
     out = torch.full((heads, rows, (rank + 7) // 8 * 8), 5.0, dtype=dtype, device="cuda")
-    splits, chunk = (6, 64) if form.endswith("split") else (1, 0)
+    splits, chunk = {"6": (6, 64), "3": (3, 128)}.get(form[-1], (1, 0)) if "split" in form else (1, 0)
     ws = torch.empty(rows * heads * splits * (rank + 2), device="cuda")
     M.latent_attn(q, cache, out, table, pos, slots, kv_rank=rank, rot=rot, scale=0.11, gate=gate, row_seq=seq, num_splits=splits,
                   chunk_tokens=chunk, ws=ws, force_simt=form == "bf16-plain")
