@@ -8,7 +8,7 @@
 #include <stddef.h>
 #include <stdint.h>
 
-#define XP_ABI_VERSION 22
+#define XP_ABI_VERSION 23
 
 #ifdef __cplusplus
 extern "C" {

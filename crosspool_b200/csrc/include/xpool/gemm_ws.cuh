@@ -445,7 +445,7 @@ __device__ __forceinline__ void epilogue_store16(const Problem& p, int f, int fb
   const int64_t o0 = static_cast<int64_t>(n_first) * p.ld_out + f + out_off;
   float v[16];
   if (p.epilogue == kEpiSwiglu) {
-    const float bias_u = (p.bias != nullptr && p.dual) ? p.bias[p.up_offset + fb] : 0.f;
+    const float bias_u = (p.bias != nullptr && p.dual && live) ? p.bias[p.up_offset + fb] : 0.f;
     const float lim = p.gate_limit > 0.f ? p.gate_limit : 3.0e38f;
     const float a = p.act_alpha == 0.f ? 1.f : p.act_alpha;
 #pragma unroll

@@ -52,6 +52,127 @@ typedef struct XpGatedRmsArgs {
   int f32;
 } XpGatedRmsArgs;
 
+/* Norms behind a sublayer: y = branches[0], or with branch weights the mean over the branches of rmsnorm(b_i) * branch_w[i];
+ * v = resid[r] + rmsnorm(y) * weight (or v = table[ids[r]]), stored to resid[r];
+ * out[i] = out_weight ? rmsnorm(v) * out_weight : v,  with r = sel ? sel[i] : i. With sel the residual is read only. */
+typedef struct XpPostNormArgs {
+  float* resid;            /* [*, hidden] */
+  const void* branches[2]; /* activations [*, ld_branch[i]] */
+  const float* branch_w[2];/* [hidden], or null: a single branch is taken as it is */
+  const int* ids;          /* optional: start the residual from the embedding table */
+  const void* table;       /* [vocab, hidden] */
+  const int* sel;          /* optional row selection */
+  const float* weight;     /* [hidden] */
+  const float* out_weight; /* optional [hidden] */
+  void* out;               /* [rows, ld_out]; null: residual update only */
+  int rows, hidden, nbranches;
+  int ld_branch[2];
+  int ld_out, vocab;
+  float eps;
+  int f32;
+} XpPostNormArgs;
+
+/* out = rmsnorm(o) * weight * silu(gate), o in fp32, the norm over each head of `dim` columns; weight shared by the heads. */
+typedef struct XpHeadGateArgs {
+  const float* o;        /* [rows, heads * dim] */
+  const float* weight;   /* [dim] */
+  const void* gate;      /* logits [rows, ld_gate] */
+  void* out;             /* [rows, ld_out] */
+  int rows, heads, dim, ld_o, ld_gate, ld_out;
+  float eps;
+  int f32;
+} XpHeadGateArgs;
+
+/* out = min(g, limit) sigmoid(alpha min(g, limit)) (clamp(u, +-limit) + up_add), g and u the halves of z's rows, in fp32. */
+typedef struct XpGluArgs {
+  const float* z;        /* [rows, ld_z]: g (cols), u (cols) */
+  float* out;            /* [rows, ld_out] */
+  int rows, cols, ld_z, ld_out;
+  float limit, up_add, alpha;
+} XpGluArgs;
+
+/* Grouped-query attention without rotation, per token row: RMS norm of query and key heads, queries laid out
+ * [rows, kv_heads, group_pad, dq], keys and values written to the cache row of the token, everything zero-padded. */
+typedef struct XpGroupedPrepArgs {
+  const void* proj;      /* [rows, ld_proj]: q (heads x dim), k (kv_heads x dim), v (kv_heads x vdim) at the offsets */
+  const float* q_norm;   /* [dim], or null: no norm */
+  const float* k_norm;
+  const int* slots;      /* [rows] cache row, -1: none */
+  void* k_cache;         /* [tokens, kv_heads, dq] */
+  void* v_cache;         /* [tokens, kv_heads, dv] */
+  void* q_out;
+  int rows, heads, kv_heads, group_pad, dim, vdim, dq, dv, ld_proj, q_off, k_off, v_off;
+  float eps;
+  int f32;
+} XpGroupedPrepArgs;
+
+/* Attention of single rows against the paged cache of grouped keys and values, plain form for any sizes. Row r attends to
+ * positions[r] + 1 tokens of block-table row row_seq[r]; softcap > 0: scores become softcap tanh(score / softcap). */
+typedef struct XpGroupedAttnArgs {
+  const void* q;         /* [rows, kv_heads, group_pad, dq] */
+  const void* k_cache;   /* [pages, page_size, kv_heads, dq] */
+  const void* v_cache;   /* [pages, page_size, kv_heads, dv] */
+  void* out;             /* [rows, ld_out]: heads x vdim */
+  const void* gate;      /* optional per-head output gate logits [rows, ld_gate] */
+  const int* row_seq;    /* [rows], or null: row r uses table row r */
+  const int* positions;  /* [rows] */
+  const int* slots;      /* [rows] < 0: padding row (zeros are stored) */
+  const int* block_table;
+  int rows, heads, kv_heads, group_pad, dim, vdim, dq, dv, ld_gate, ld_out, page_size, max_blocks;
+  float scale, softcap;
+  int f32;
+} XpGroupedAttnArgs;
+
+/* Linear attention with a decay per key channel: S = diag(alpha) S + k v^T, o = S^T q qscale, log alpha = -softplus(-z) / tau.
+ * Decode computes z itself (z = a2 a1 + a2_bias) and stores rmsnorm(o) * norm * silu(gate); prefill reads z and stores o. */
+typedef struct XpGatedLinearArgs {
+  const void* proj;      /* [rows, ld_proj]: q, k (heads x dim), v, gate (heads x vdim), a1 (rank) at the offsets */
+  const float* z;        /* prefill: [rows, heads * dim] */
+  const void* a2;        /* decode: [heads * dim, ld_a2] */
+  const float* a2_bias;  /* decode: [heads * dim] */
+  const float* norm;     /* decode: [vdim] */
+  float* state;          /* [slots, heads, dim, vdim] */
+  void* out;             /* decode: activations [rows, ld_out]; prefill: fp32 [rows, ld_out] */
+  const int* positions;
+  const int* slots;      /* [rows] KV slot of the row, < 0: padding row */
+  const int* state_slots;
+  const int* q_starts;
+  const int* q_lens;
+  float* ws;             /* chunked prefill: states and decays of segments */
+  int rows, seqs, heads, dim, vdim, ld_proj, ld_out, q_off, k_off, v_off, g_off, a_off, rank, ld_a2;
+  int segs, seg_tokens, force_sequential;
+  float inv_tau, qscale, eps;
+  int f32;
+} XpGatedLinearArgs;
+
+/* Gated delta rule: S = g S; u = beta (v - S^T k); S = S + k u^T; o = S^T q. The convolution's inputs are kept per slot as a
+ * ring, position p in entry p % taps. Decode does everything from the projection to rmsnorm(o) * norm * silu(gate); prefill
+ * convolves into qkv (activations behind silu, unnormalised), writes the factors that make queries and keys unit vectors
+ * (queries times qscale), beta and log g, and runs the recurrence on those. */
+typedef struct XpDeltaArgs {
+  const void* proj;      /* [rows, ld_proj] at the offsets: q, k (kv_heads x dim), v (heads x vdim), gate, b, a (heads) */
+  const float* conv_w;   /* [channels, taps], channels = q, k, v */
+  void* conv_state;      /* [slots, taps, channels] activations */
+  const float* neg_a;    /* [heads] -exp(A_log) */
+  const float* dt_bias;  /* [heads] */
+  const float* norm;     /* decode: [vdim] */
+  float* state;          /* [slots, heads, dim, vdim] */
+  void* out;             /* decode: activations [rows, ld_out]; prefill: fp32 [rows, ld_out] */
+  void* qkv;             /* prefill: [rows, channels] */
+  float* qk_scale;       /* prefill: [rows, 2, kv_heads] */
+  float* beta_g;         /* prefill: [rows, 2, heads]: beta, log g */
+  void* ws;              /* chunked prefill */
+  const int* positions;
+  const int* slots;
+  const int* state_slots;
+  const int* q_starts;
+  const int* q_lens;
+  int rows, seqs, max_q, heads, kv_heads, dim, vdim, taps, ld_proj, ld_out, q_off, k_off, v_off, g_off, b_off, a_off;
+  int force_sequential;
+  float qscale, eps;
+  int f32;
+} XpDeltaArgs;
+
 /* Latent attention, per token row: normalise the latent, rotate the shared key part, write both to the cache row of the
  * token; rotate the rotary part of every query head and lay the queries out for the absorbed form
  * (q_plain head-major, q_abs columns [kv_rank, +rot)) and/or the expanded form (q_exp). */
@@ -125,6 +246,16 @@ typedef struct XpLinearAttnArgs {
 int xp_resid_norm(const XpResidNormArgs* a, void* stream);
 int xp_polynorm(const XpPolyNormArgs* a, void* stream);
 int xp_gated_rms(const XpGatedRmsArgs* a, void* stream);
+int xp_post_norm(const XpPostNormArgs* a, void* stream);
+int xp_head_gate(const XpHeadGateArgs* a, void* stream);
+int xp_glu_f32(const XpGluArgs* a, void* stream);
+int xp_grouped_prep(const XpGroupedPrepArgs* a, void* stream);
+int xp_grouped_attn(const XpGroupedAttnArgs* a, void* stream);
+int xp_gated_linear_decode(const XpGatedLinearArgs* a, void* stream);
+int xp_gated_linear_prefill(const XpGatedLinearArgs* a, void* stream);
+int xp_delta_decode(const XpDeltaArgs* a, void* stream);
+int xp_delta_prep(const XpDeltaArgs* a, void* stream);
+int xp_delta_prefill(const XpDeltaArgs* a, void* stream);
 int xp_latent_prep(const XpLatentPrepArgs* a, void* stream);
 int xp_latent_attn(const XpLatentAttnArgs* a, void* stream);
 int xp_latent_gather(const XpLatentGatherArgs* a, void* stream);

@@ -281,11 +281,12 @@ static inline int kblk_of(const XpGemmArgs* a) { return a->fp8 ? 128 : gemm::kTi
 extern "C" int xp_gemm_plan(const XpGemmArgs* a, XpGemmPlan* plan) {
   const int kblk = a->fp8 ? 128 : gemm::kTileK;
   if (a->n_out <= 0 || a->k <= 0 || a->rows <= 0) return -10;
-  // plain bf16 problems may end in partial tiles (TMA fills them with zeros); the other forms address whole tiles
-  const bool whole = a->fp8 || a->dual || a->w_tiled || a->tile_table != nullptr;
+  // bf16 problems over row-major weights may end in partial tiles (TMA fills them with zeros; a partial gate tile computes
+  // rows of the up matrix that nobody stores); the other forms address whole tiles
+  const bool whole = a->fp8 || a->w_tiled || a->tile_table != nullptr;
   if (whole && (a->n_out % gemm::kTileM != 0 || a->k % kblk != 0)) return -10;
   const int batch = a->batch > 1 ? a->batch : 1;
-  if (batch > 1 && (whole || a->epilogue == gemm::kEpiResidual || a->bias != nullptr || a->x_group_rows < a->rows)) return -16;
+  if (batch > 1 && (whole || a->dual || a->epilogue == gemm::kEpiResidual || a->bias != nullptr || a->x_group_rows < a->rows)) return -16;
   if (a->fp8 && (a->dual || a->w_tiled || a->tile_table != nullptr || a->w_scale == nullptr || a->x_scale == nullptr ||
                  a->ld_xscale % 4 != 0 || a->bn > gemm::kMaxBnF8))
     return -14;

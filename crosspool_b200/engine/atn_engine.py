@@ -394,7 +394,7 @@ class AttentionEngine:
             from .layered import RowBatch
 
             at = 4 * self.ecfg.max_batch + self.ecfg.max_batch * self.max_blocks
-            b = RowBatch(B, B, B, B, 1, self.ecfg.max_seq_len, pos, slots, table, self.dec_meta[at:at + B])
+            b = RowBatch(B, B, B, B, B, 1, self.ecfg.max_seq_len, pos, slots, table, self.dec_meta[at:at + B])
             self.body.forward(ids, b, MODE_DECODE)
             self.body.head(B, None, B, self.sel, self.logits)
             self._sample(B)
@@ -457,7 +457,7 @@ class AttentionEngine:
             groups.append(ExpandGroup(start, i - start, max(s.computed + c for s, c in part), max(c for _, c in part), used))
             start = i
         batch = RowBatch(
-            rows, n, n_dec, n_abs, max((c for _, c in chosen[n_dec:]), default=0),
+            rows, n, n_dec, n_abs, len(short), max((c for _, c in chosen[n_dec:]), default=0),
             max(s.computed + c for s, c in (chosen[:len(short)] if self.body.all_expand and short else chosen)),
             m[P:P + rows], m[2 * P:2 * P + rows], m[t:t + n * self.max_blocks].view(n, self.max_blocks), m[r + P:r + P + n],
             m[r:r + rows], m[b:b + n], m[b + S:b + S + n], m[b + 2 * S:b + 2 * S + n], m[r + P + S:r + P + S + n], tuple(groups))

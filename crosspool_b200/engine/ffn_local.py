@@ -3,7 +3,8 @@
 Used when one GPU hosts both roles (kernels that wait on one another must never be separate
 launches on one GPU, so the loopback path is stream-ordered and flag-free). Dense layers are two
 launches: gate/up GEMM with the SwiGLU epilogue, then the down projection. Ungated layers with a
-row-normalised activation (PolyNorm) put the activation kernel between the two products.
+row-normalised activation (PolyNorm) put the activation kernel between the two products, and so do
+gated layers in fp32.
 """
 
 from __future__ import annotations
@@ -41,7 +42,8 @@ class LocalFfnPort(FfnPort):
         for w in self.weights:
             if w is not None:
                 w.gate_up, w.down = pad_pitch(w.gate_up), pad_pitch(w.down)
-        inter = max((ceil8(w.gate_up.shape[0]) for w in self.weights if w is not None), default=8)
+        # widest activation row; fp32 gated layers keep gate and up columns, then the activations behind them
+        inter = max((ceil8(w.gate_up.shape[0]) + ceil8(w.down.shape[1]) for w in self.weights if w is not None), default=8)
         self.act = torch.zeros(engine.cap * inter, dtype=engine.dtype, device=engine.device)
         self.y = torch.zeros(engine.cap, ceil8(self.cfg.hidden_size), dtype=engine.dtype, device=engine.device)[:, :self.cfg.hidden_size]
 
@@ -56,10 +58,28 @@ class LocalFfnPort(FfnPort):
         gemm.linear(z, w.down, out=self.y[:rows])
         return [self.y[:rows]]
 
+    def _run_gated(self, w: FfnLayerWeights, x: torch.Tensor, rows: int) -> list[torch.Tensor]:
+        """Gated FFN of any width in the engine's element type."""
+        ff = w.down.shape[1]
+        act = self.act[:rows * ceil8(ff)].view(rows, ceil8(ff))[:, :ff]
+        limit, up_add, alpha = w.extra.get("gate_transform", (0.0, 0.0, 1.0))
+        if x.dtype == torch.float32:
+            from ..ops import mixers
+
+            z = self.act[rows * ceil8(ff):][:rows * 2 * ff].view(rows, 2 * ff)
+            gemm.linear(x, w.gate_up, out=z)
+            mixers.glu_f32(z, limit, up_add, alpha, act)
+        else:
+            gemm.gateup_swiglu(x, w.gate_up, out=act, gate_limit=limit, up_add=up_add, act_alpha=alpha)
+        gemm.linear(act, w.down, out=self.y[:rows])
+        return [self.y[:rows]]
+
     def run(self, layer: int, x: torch.Tensor, rows: int, mode: int) -> list[torch.Tensor]:
         w = self.weights[layer]
         if "polynorm" in w.extra:
             return self._run_polynorm(w, x, rows)
+        if self.cfg.layered:
+            return self._run_gated(w, x, rows)
         if w.is_moe:
             from ..ops import moe
 

@@ -9,8 +9,8 @@ tensors' addresses — and therefore captured CUDA graphs — stay valid. The al
 pages whose bundle is mapped, like the reference's ``ElasticPageAllocator``
 (src/xpool/integrations/sglang/ecs/allocator.py:61-104).
 
-Layered decoders cache one row per token in the layers that have a cache at all, and keep one recurrent state per live
-sequence (:class:`StateSlots`) in the others; both follow the sequence through the same ``ensure`` / ``release``.
+Layered decoders cache rows per token in the layers that have a cache at all, and keep one recurrent state per live
+sequence (:class:`StateSlots`) in those with a recurrence (a layer can have both); they follow the sequence through the same ``ensure`` / ``release``.
 """
 
 from __future__ import annotations
@@ -19,7 +19,7 @@ from dataclasses import dataclass, field
 
 import torch
 
-from ..models.config import ModelConfig
+from ..models.config import DeltaMixer, ModelConfig, sub_mixers
 
 
 class OutOfPages(RuntimeError):
@@ -159,6 +159,8 @@ class PagedKvCache:
     tables: dict[int, list[int]] = field(default_factory=dict)
     # recurrent layers: fp32 [slots, heads, dim, vdim] per layer (None elsewhere), and the slot of every live sequence
     states: list[torch.Tensor | None] = field(default_factory=list)
+    # convolution inputs behind every live sequence, [slots, taps, channels] per layer: the input at position p is entry p % taps
+    conv: list[torch.Tensor | None] = field(default_factory=list)
     slots: StateSlots | None = None
     seq_slots: dict[int, int] = field(default_factory=dict)
 
@@ -175,14 +177,24 @@ class PagedKvCache:
 
     @classmethod
     def _layered(cls, cfg: ModelConfig, num_pages: int, page_size: int, device, dtype: torch.dtype, state_slots: int) -> "PagedKvCache":
-        """Pages hold one row per token in the layers that cache one (a latent row that is key and value at once);
-        recurrent layers hold one state per slot."""
+        """Pages hold a key row and a value row per token in the layers that cache any (or one latent row that is both);
+        recurrent mixers hold one state per slot, and those with a convolution its latest inputs."""
         mixers = [s.mixer for s in cfg.layer_specs]
         lay = KvLayout(page_size, num_pages, 1, 0, cfg.num_layers, dtype.itemsize, tuple(m.cache_width for m in mixers))
-        k = [torch.zeros(num_pages, page_size, 1, m.cache_width, dtype=dtype, device=device) if m.cache_width else None for m in mixers]
-        states = [torch.zeros(state_slots, m.heads, m.dim, m.vdim, dtype=torch.float32, device=device) if m.state_elems else None
-                  for m in mixers]
-        return cls(lay, k, [None] * len(k), PageAllocator(num_pages), states=states,
+
+        def rows(m, i: int) -> torch.Tensor | None:
+            if len(m.cache_rows) <= i:
+                return None
+            return torch.zeros(num_pages, page_size, *m.cache_rows[i], dtype=dtype, device=device)
+
+        states, conv = [None] * len(mixers), [None] * len(mixers)
+        for l, m in enumerate(mixers):
+            for sub in sub_mixers(m):
+                if sub.state_elems:
+                    states[l] = torch.zeros(state_slots, sub.heads, sub.dim, sub.vdim, dtype=torch.float32, device=device)
+                if isinstance(sub, DeltaMixer):
+                    conv[l] = torch.zeros(state_slots, sub.conv, sub.conv_channels, dtype=dtype, device=device)
+        return cls(lay, [rows(m, 0) for m in mixers], [rows(m, 1) for m in mixers], PageAllocator(num_pages), states=states, conv=conv,
                    slots=StateSlots(state_slots) if cfg.recurrent else None)
 
     # -- per-sequence page tables --------------------------------------------------------------

@@ -6,9 +6,14 @@ over all rows together; a mixer splits the rows where its decode and prefill ker
 * latent attention: decoded tokens and short portions run in the absorbed form (queries multiplied into the latent space,
   one pass over the cached rows); long portions in the expanded form (the sequence's latents are expanded to per-head keys
   and values with one product each, then the tcgen05 prefill kernel);
-* decayed linear attention: one kernel advances the states of the decoded tokens, another those of the portions.
+* grouped-query attention: decoded tokens and short portions as single rows, long portions in the tcgen05 prefill kernel;
+* recurrences (decayed linear attention, gated linear attention, gated delta rule): one kernel advances the states of the
+  decoded tokens, others those of the portions;
+* a parallel pair runs both of its sides on the columns of one projection.
 
-The residual stream is fp32; each sublayer's output is gated, added and normalised for the next sublayer in one kernel.
+The residual stream is fp32. Where a norm stands in front of a sublayer, one kernel gates and adds the previous sublayer's
+output and normalises for the next; where it stands behind, one kernel norms the output (of both sides of a pair), adds it and
+hands the residual itself on.
 """
 
 from __future__ import annotations
@@ -17,12 +22,14 @@ from dataclasses import dataclass
 
 import torch
 
-from ..models.config import LatentMixer, LinearMixer
-from ..models.layered import LayeredLayerWeights, ceil8
+from ..models.config import (DeltaMixer, GatedLinearMixer, GroupedMixer, LatentMixer, LinearMixer, ParallelMixer, attention_shape,
+                             ceil8, sub_mixers)
+from ..models.layered import LayeredLayerWeights
 from ..ops import gemm
 from ..ops import mixers as M
 
-# Portions of at most this many tokens run as rows of the absorbed form: expanding the whole context costs more.
+# Portions of at most this many tokens run as single rows (latent attention: in the absorbed form, expanding the whole context
+# costs more).
 SHORT_PORTION = 16
 
 
@@ -42,9 +49,10 @@ class RowBatch:
     rows: int
     n_seqs: int
     n_dec: int                           # leading rows that are one token each (= leading sequences)
-    n_abs: int                           # leading rows of the absorbed form (decoded tokens, then short portions)
+    n_abs: int                           # leading rows that attend as single rows (decoded tokens, then short portions)
+    n_short: int                         # leading sequences that do
     max_q: int                           # longest portion behind the decoded tokens
-    max_len: int                         # bound on positions + 1 of the absorbed rows
+    max_len: int                         # bound on positions + 1 of those rows
     positions: torch.Tensor              # [rows]
     slots: torch.Tensor                  # [rows] cache row, -1: padding
     table: torch.Tensor                  # [seqs, max_blocks]
@@ -72,12 +80,20 @@ class LayeredForward:
         self.resid = torch.zeros(cap, cfg.hidden_size, dtype=torch.float32, device=dev)
         self.x, self.x2, self.y, self.rg2 = (torch.zeros(cap, h8, dtype=dt, device=dev)[:, :cfg.hidden_size] for _ in range(4))
         self.proj = buf(cap * max(lw.offs["end"] for lw in layers))
-        self.mix_out = torch.zeros(cap * max(ceil8(lw.spec.mixer.out_features) for lw in layers), dtype=dt, device=dev)
-        lat = [lw.spec.mixer for lw in layers if isinstance(lw.spec.mixer, LatentMixer)]
-        lin = [lw.spec.mixer for lw in layers if isinstance(lw.spec.mixer, LinearMixer)]
+        self.mix_out = torch.zeros(cap * max(sum(ceil8(m.out_features) for m in sub_mixers(lw.spec.mixer)) for lw in layers),
+                                   dtype=dt, device=dev)
+        mixers = [m for lw in layers for m in sub_mixers(lw.spec.mixer)]
+
+        def of(kind):
+            return [m for m in mixers if isinstance(m, kind)]
+
+        lat, lin, grp, gla, delta = of(LatentMixer), of(LinearMixer), of(GroupedMixer), of(GatedLinearMixer), of(DeltaMixer)
         self.expands = [("exp_k" in lw.mix) for lw in layers]
-        # every latent layer has an expanded form: only decoded tokens and short portions run absorbed
-        self.all_expand = all(ex for lw, ex in zip(layers, self.expands) if isinstance(lw.spec.mixer, LatentMixer))
+        # only decoded tokens and short portions attend as single rows, in every layer
+        self.all_expand = all(ex for lw, ex in zip(layers, self.expands) if isinstance(lw.spec.mixer, LatentMixer)) and \
+            all(self._tiled(m) for m in grp)
+        if cfg.output_norm:
+            self.y2 = torch.zeros(cap, h8, dtype=dt, device=dev)[:, :cfg.hidden_size]
         if lat:
             self.q_plain = buf(cap * max(m.heads * ceil8(m.dim) for m in lat))
             self.q_abs = buf(cap * max(m.heads * m.cache_width for m in lat))
@@ -95,8 +111,16 @@ class LayeredForward:
             self.lat_ws = buf(self.ws_tokens * max(w for *_, w in shapes))
             self.k_exp = buf(self.ws_tokens * max(H * dq for H, dq, _, _ in shapes))
             self.v_exp = buf(self.ws_tokens * max(H * dv for H, _, dv, _ in shapes))
+        if grp:
+            self.q_grp = buf(cap * max(m.kv_heads * M.group_pad(m.heads, m.kv_heads) * m.cache_rows[0][1] for m in grp))
+        if gla:
+            self.z = buf(cap * max(m.heads * m.dim for m in gla), torch.float32)
+        if delta:
+            self.delta_ws = M.DeltaScratch(buf(cap * max(m.conv_channels for m in delta)), buf(cap * max(2 * m.kv_heads for m in delta), torch.float32),
+                                           buf(cap * max(2 * m.heads for m in delta), torch.float32))
+        if lin or gla or delta:
+            self.o_lin = buf(cap * max(m.out_features for m in lin + gla + delta), torch.float32)
         if lin:
-            self.o_lin = buf(cap * max(m.out_features for m in lin), torch.float32)
             self.lin_ws = buf(max(M.linear_attn_ws_elems(m.dim, m.vdim) for m in lin) if dt == torch.bfloat16 else 1, torch.float32)
 
     # ------------------------------------------------------------------ mixers
@@ -151,27 +175,97 @@ class LayeredForward:
                                   seg_tokens=seg_tokens, ws=self.lin_ws, **kw)
         M.gated_rms(o, lw.mix["norm"], proj[:, lw.offs["g"]:lw.offs["g"] + n], self.e.cfg.rms_norm_eps, out)
 
+    def _tiled(self, m: GroupedMixer) -> bool:
+        """Whether the tensor-core attention kernels cover the mixer."""
+        shape, page = attention_shape(m.dim, m.vdim), self.e.ecfg.page_size
+        return False
+
+    def _grouped(self, l: int, lw: LayeredLayerWeights, m: GroupedMixer, proj: torch.Tensor, out: torch.Tensor, b: RowBatch) -> None:
+        rows, o, kv = b.rows, lw.offs, self.e.kv
+        k, v = kv.k[l], kv.v[l]
+        gp = M.group_pad(m.heads, m.kv_heads)
+        q = self.q_grp[:rows * m.kv_heads * gp * k.shape[3]].view(rows, m.kv_heads, gp, k.shape[3])
+        M.grouped_prep(proj, lw.mix["q_norm"], lw.mix["k_norm"], b.slots, k, v, q, heads=m.heads, dim=m.dim, vdim=m.vdim,
+                       offs=(o["q"], o["k"], o["v"]), eps=self.e.cfg.rms_norm_eps)
+        gate = proj[:, o["hg"]:o["hg"] + m.heads]
+        M.grouped_attn(q, k, v, out, b.table, b.positions, b.slots, heads=m.heads, dim=m.dim, vdim=m.vdim, scale=m.scale,
+                       softcap=m.softcap, gate=gate, row_seq=b.row_seq)
+
+    def _gated_linear(self, l: int, lw: LayeredLayerWeights, m: GatedLinearMixer, proj: torch.Tensor, out: torch.Tensor, b: RowBatch) -> None:
+        o, w, n, nd, eps = lw.offs, lw.mix, m.out_features, b.n_dec, self.e.cfg.rms_norm_eps
+        state = self.e.kv.states[l]
+        kw = dict(heads=m.heads, dim=m.dim, vdim=m.vdim, tau=m.tau)
+        qkv = (o["lin_q"], o["lin_k"], o["lin_v"])
+        if nd:
+            M.gated_linear_decode(proj[:nd], state, w["a2"], w["a2_bias"], w["norm"], out[:nd], b.positions, b.slots, b.state_slots,
+                                  offs=(*qkv, o["lin_g"], o["lin_a"]), eps=eps, **kw)
+        if nd < b.n_seqs:
+            s = slice(nd, b.n_seqs)
+            z = self.z[:b.rows * m.heads * m.dim].view(b.rows, m.heads * m.dim)
+            gemm.linear(proj[nd:, o["lin_a"]:o["lin_a"] + w["a2"].shape[1]], w["a2"], out=z[nd:], bias=w["a2_bias"])
+            y = self.o_lin[:b.rows * n].view(b.rows, n)
+            M.gated_linear_prefill(proj, z, state, y, b.positions, b.slots, b.state_slots[s], b.q_starts[s], b.q_lens[s], offs=qkv, **kw)
+            M.head_gate(y[nd:], w["norm"], proj[nd:, o["lin_g"]:o["lin_g"] + n], eps, out[nd:])
+
+    def _delta(self, l: int, lw: LayeredLayerWeights, m: DeltaMixer, proj: torch.Tensor, out: torch.Tensor, b: RowBatch) -> None:
+        o, w, n, nd, eps = lw.offs, lw.mix["delta"], m.out_features, b.n_dec, self.e.cfg.rms_norm_eps
+        state, conv = self.e.kv.states[l], self.e.kv.conv[l]
+        kw = dict(heads=m.heads, kv_heads=m.kv_heads, dim=m.dim, vdim=m.vdim, offs=tuple(o[c] for c in "qkvgba"), eps=eps)
+        if nd:
+            M.delta_decode(proj[:nd], conv, w, state, out[:nd], b.positions, b.slots, b.state_slots, **kw)
+        if nd < b.n_seqs:
+            s = slice(nd, b.n_seqs)
+            y = self.o_lin[:b.rows * n].view(b.rows, n)
+            M.delta_prefill(proj, conv, w, state, y, b.positions, b.slots, b.state_slots[s], b.q_starts[s], b.q_lens[s], b.max_q, self.delta_ws, **kw)
+            M.head_gate(y[nd:], w.norm, proj[nd:, o["g"]:o["g"] + n], eps, out[nd:])
+
+    _RUN = {LatentMixer: _latent, LinearMixer: _linear, GroupedMixer: _grouped, GatedLinearMixer: _gated_linear, DeltaMixer: _delta}
+
     # ------------------------------------------------------------------ layers
+    def _mix(self, l: int, lw: LayeredLayerWeights, x: torch.Tensor, b: RowBatch) -> tuple[torch.Tensor, list[torch.Tensor]]:
+        """The layer's projection, and the outputs of its mixer (of both sides of a pair) behind their output products."""
+        rows = b.rows
+        proj = self.proj[:rows * lw.offs["end"]].view(rows, lw.offs["end"])
+        gemm.linear(x, lw.proj, out=proj, bias=lw.proj_bias, silu_cols=lw.silu_cols)
+        ys, at = [], 0
+        for i, m in enumerate(sub_mixers(lw.spec.mixer)):
+            n = m.out_features
+            out = self.mix_out[at:][:rows * ceil8(n)].view(rows, ceil8(n))[:, :n]
+            at += rows * ceil8(n)
+            self._RUN[type(m)](self, l, lw, m, proj, out, b)
+            y = (self.y2 if i else self.y)[:rows]
+            gemm.linear(out, lw.o_right if i else lw.o, out=y, bias=None if i else lw.o_bias)
+            ys.append(y)
+        return proj, ys
+
+    def _enter(self, resid: torch.Tensor, norm, x: torch.Tensor, pending: dict) -> None:
+        """Adds the pending sublayer output to the residual and prepares the next sublayer's input."""
+        if self.e.cfg.output_norm:
+            M.post_norm(resid, x, **pending)
+        else:
+            M.resid_norm(resid, norm, x, **pending)
+
     def forward(self, ids: torch.Tensor, b: RowBatch, mode: int) -> None:
         """Embedding and all layers over the batch's rows; the last sublayer's output stays pending for :meth:`head`."""
         rows, hid = b.rows, self.e.cfg.hidden_size
-        resid, x, x2, y = self.resid[:rows], self.x[:rows], self.x2[:rows], self.y[:rows]
+        resid, x, x2 = self.resid[:rows], self.x[:rows], self.x2[:rows]
+        post = self.e.cfg.output_norm
         pending: dict = dict(ids=ids, table=self.e.w.embed)
         for l, lw in enumerate(self.layers):
-            M.resid_norm(resid, lw.norm1, x, **pending)
-            proj = self.proj[:rows * lw.offs["end"]].view(rows, lw.offs["end"])
-            gemm.linear(x, lw.proj, out=proj, bias=lw.proj_bias, silu_cols=lw.silu_cols)
-            m = lw.spec.mixer
-            n = m.out_features
-            out = self.mix_out[:rows * ceil8(n)].view(rows, ceil8(n))[:, :n]
-            (self._latent if isinstance(m, LatentMixer) else self._linear)(l, lw, m, proj, out, b)
-            gemm.linear(out, lw.o, out=y)
-            pending = dict(parts=[y], gate=proj[:, lw.offs["rg"]:lw.offs["rg"] + hid])
+            self._enter(resid, lw.norm1, x, pending)
+            proj, ys = self._mix(l, lw, x, b)
+            if post:
+                pending = dict(branches=ys, branch_norms=lw.branch_norms, norm=lw.norm1)
+            else:
+                pending = dict(parts=ys, gate=proj[:, lw.offs["rg"]:lw.offs["rg"] + hid])
             if lw.norm2 is not None:
-                M.resid_norm(resid, lw.norm2, x2, **pending)
-                rg2 = self.rg2[:rows]
-                gemm.linear(x2, lw.rg2, out=rg2, bias=lw.rg2_bias)
-                pending = dict(parts=self.e.port.run(l, x2, rows, mode), gate=rg2)
+                self._enter(resid, lw.norm2, x2, pending)
+                if post:
+                    pending = dict(branches=self.e.port.run(l, x2, rows, mode), norm=lw.norm2)
+                else:
+                    rg2 = self.rg2[:rows]
+                    gemm.linear(x2, lw.rg2, out=rg2, bias=lw.rg2_bias)
+                    pending = dict(parts=self.e.port.run(l, x2, rows, mode), gate=rg2)
             self.tap(l, rows, pending)
         self._pending = pending
 
@@ -181,5 +275,9 @@ class LayeredForward:
     def head(self, rows: int, sel: torch.Tensor | None, n_sel: int, out: torch.Tensor, logits: torch.Tensor) -> None:
         """Final norm of the selected rows (all of the first ``n_sel`` without ``sel``) and their scaled logits (fp32)."""
         e = self.e
-        M.resid_norm(self.resid[:rows], e.w.final_norm, out[:n_sel], sel=sel, rows=n_sel, **self._pending)
+        if e.cfg.output_norm:
+            # (without a selection the rows are their own; a selection leaves the residual of the others alone)
+            M.post_norm(self.resid[:rows], out[:n_sel], out_norm=e.w.final_norm, sel=sel, rows=n_sel, **self._pending)
+        else:
+            M.resid_norm(self.resid[:rows], e.w.final_norm, out[:n_sel], sel=sel, rows=n_sel, **self._pending)
         gemm.linear(out[:n_sel], e.w.lm_head, out=logits[:n_sel], out_scale=e.cfg.logit_scale)

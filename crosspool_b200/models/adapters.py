@@ -1,7 +1,7 @@
 """Architecture adapters: Hugging Face ``config.json`` + checkpoint keys → :class:`FfnModelSpec`.
 
 One adapter per supported architecture, discovered by ``architectures[0]`` (``architecture`` in the
-configuration files of layered decoders) — Segirax and the same eight families the reference serves (src/xpool/runtime/ffnagent/models/*.py, discovery in
+configuration files of layered decoders) — Saninex, Segirax and the same eight families the reference serves (src/xpool/runtime/ffnagent/models/*.py, discovery in
 src/xpool/runtime/ffnagent/architecture.py:175-215): Qwen2, Qwen3, Qwen3-MoE, Llama, OPT,
 DeepSeek-V2, GLM-4 MoE Lite and GPT-OSS. Adapters only read the configuration and the *names* of
 checkpoint tensors; no weight is opened here.
@@ -227,6 +227,21 @@ def _segirax(model_id: str, src: FfnSourceConfig, keys: Iterable[str]) -> FfnMod
     return FfnModelSpec(model_id, src.architecture, src.payload_dtype, c.hidden_size, src.quantization, tuple(layers))
 
 
+def _saninex(model_id: str, src: FfnSourceConfig, keys: Iterable[str]) -> FfnModelSpec:
+    from .config import GLU_ALPHA, saninex_config
+
+    c = saninex_config(dict(src.cfg), model_id)
+    layers = []
+    for i, s in enumerate(c.layer_specs):
+        if s.ff == 0:
+            continue
+        p, h = f"l{i}.mlp", c.hidden_size
+        layers.append(DenseFfnSpec(i, h, s.ff, ActivationKind.SILU,
+                                   GatedProjectionSpec(ProjectionSpec(f"{p}.gate", s.ff, h), ProjectionSpec(f"{p}.up", s.ff, h)),
+                                   ProjectionSpec(f"{p}.down", h, s.ff), GateTransform(s.gate_limit, 1.0, GLU_ALPHA)))
+    return FfnModelSpec(model_id, src.architecture, src.payload_dtype, c.hidden_size, src.quantization, tuple(layers))
+
+
 ADAPTERS: dict[str, Callable[[str, FfnSourceConfig, Iterable[str]], FfnModelSpec]] = {
     "Qwen2ForCausalLM": _llama_like,
     "Qwen3ForCausalLM": _llama_like,
@@ -237,6 +252,7 @@ ADAPTERS: dict[str, Callable[[str, FfnSourceConfig, Iterable[str]], FfnModelSpec
     "DeepseekV2ForCausalLM": lambda m, s, k: _deepseek_like(m, s, k, sigmoid=False),
     "Glm4MoeLiteForCausalLM": lambda m, s, k: _deepseek_like(m, s, k, sigmoid=True),
     "GptOssForCausalLM": _gpt_oss,
+    "Saninex": _saninex,
     "Segirax": _segirax,
 }
 

@@ -41,6 +41,24 @@ class RotarySpec:
     base: float
 
 
+def ceil8(n: int) -> int:
+    return (n + 7) // 8 * 8
+
+
+# (query/key width, value width) of the tensor-core attention kernels, narrowest first
+ATTENTION_SHAPES = ((64, 64), (128, 64), (128, 128), (192, 128))
+
+
+def attention_shape(dim: int, vdim: int) -> tuple[int, int] | None:
+    """Padded head widths of the tensor-core attention kernels, None when no kernel covers the sizes."""
+    if vdim % 8:
+        return None
+    for dq, dv in ATTENTION_SHAPES:
+        if dim <= dq and vdim <= dv:
+            return dq, dv
+    return None
+
+
 @dataclass(frozen=True)
 class LatentMixer:
     """Latent attention as a layer's mixer: per-head keys and values are linear maps of one cached ``kv_rank`` latent,
@@ -61,6 +79,10 @@ class LatentMixer:
         return (self.kv_rank + self.rot_dim + 15) // 16 * 16
 
     @property
+    def cache_rows(self) -> tuple[tuple[int, int], ...]:
+        return ((1, self.cache_width),)
+
+    @property
     def state_elems(self) -> int:
         return 0
 
@@ -74,16 +96,10 @@ class LatentMixer:
                 + self.kv_rank * self.heads * (self.dim + self.vdim))
 
 
-@dataclass(frozen=True)
-class LinearMixer:
-    """Decayed linear attention (one fp32 ``dim x vdim`` state per head and sequence, a fixed decay per head), its heads
-    normalised together and gated."""
+class _RecurrentMixer:
+    """Common part of mixers that keep one fp32 ``dim x vdim`` state per head and sequence instead of cached tokens."""
 
-    heads: int
-    dim: int
-    vdim: int
-    decay: tuple[float, ...]
-    kind: str = "lightning"
+    cache_rows: tuple[tuple[int, int], ...] = ()
 
     @property
     def cache_width(self) -> int:
@@ -97,16 +113,156 @@ class LinearMixer:
     def out_features(self) -> int:
         return self.heads * self.vdim
 
+
+@dataclass(frozen=True)
+class LinearMixer(_RecurrentMixer):
+    """Decayed linear attention (one fp32 ``dim x vdim`` state per head and sequence, a fixed decay per head), its heads
+    normalised together and gated."""
+
+    heads: int
+    dim: int
+    vdim: int
+    decay: tuple[float, ...]
+    kind: str = "lightning"
+
     def param_count(self, hidden: int) -> int:
         return hidden * self.heads * (2 * self.dim + 3 * self.vdim) + self.out_features
 
 
 @dataclass(frozen=True)
-class LayerSpec:
-    """One layer of a layered (hybrid) decoder: its mixer and the width of its ungated FFN (0: no FFN)."""
+class GroupedMixer:
+    """Grouped-query softmax attention without positions: ``heads`` query heads share ``kv_heads`` cached keys and values,
+    queries and keys are RMS-normed per head, scores saturate at +-``softcap`` (0: they do not), and a sigmoid per head
+    gates the output."""
 
-    mixer: LatentMixer | LinearMixer
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    softcap: float = 0.0
+    kind: str = "grouped_attention"
+
+    @property
+    def cache_rows(self) -> tuple[tuple[int, int], ...]:
+        """(heads, elements per head) of a token's key and value rows, padded to the widths of the tensor-core kernels
+        where one covers the sizes."""
+        return tuple((self.kv_heads, n) for n in attention_shape(self.dim, self.vdim) or (ceil8(self.dim), ceil8(self.vdim)))
+
+    @property
+    def cache_width(self) -> int:
+        return sum(h * n for h, n in self.cache_rows)
+
+    @property
+    def state_elems(self) -> int:
+        return 0
+
+    @property
+    def out_features(self) -> int:
+        return self.heads * self.vdim
+
+    def param_count(self, hidden: int) -> int:
+        kv = self.kv_heads * (self.dim + self.vdim)
+        return ((hidden + 1) * (self.heads * self.dim + kv) + 2 * self.dim + hidden * (self.heads + self.out_features + 1))
+
+
+@dataclass(frozen=True)
+class GatedLinearMixer(_RecurrentMixer):
+    """Linear attention whose state decays per key channel, ``sigmoid(z) ** (1 / tau)`` with ``z`` a low-rank map of the
+    input; every head's output is RMS-normed and gated. ``rank`` of the map belongs to the checkpoint (0: unknown)."""
+
+    heads: int
+    dim: int
+    vdim: int
+    tau: float
+    rank: int = 0
+    kind: str = "gated_linear"
+
+    def param_count(self, hidden: int) -> int:
+        return (hidden * self.heads * (2 * self.dim + 3 * self.vdim) + self.vdim + self.rank * (hidden + self.heads * self.dim)
+                + self.heads * self.dim)
+
+
+@dataclass(frozen=True)
+class DeltaMixer(_RecurrentMixer):
+    """Gated delta rule: the state decays by one factor per head and token, and a write replaces the share ``beta`` of what
+    it holds under the key. Queries, keys and values pass a causal convolution of ``conv`` taps; ``kv_heads`` queries and
+    keys (unit vectors) are shared by the ``heads`` values."""
+
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    conv: int
+    kind: str = "delta"
+
+    @property
+    def conv_channels(self) -> int:
+        """Channels that pass the convolution: queries, keys, values."""
+        return 2 * self.kv_heads * self.dim + self.heads * self.vdim
+
+    @property
+    def conv_state_elems(self) -> int:
+        """Convolution inputs a sequence carries (a ring of ``conv`` tokens: the ones behind, and the token at hand)."""
+        return self.conv * self.conv_channels
+
+    def param_count(self, hidden: int) -> int:
+        return (hidden * (self.conv_channels + 2 * self.heads + 2 * self.out_features) + self.conv * self.conv_channels
+                + 2 * self.heads + self.vdim)
+
+
+@dataclass(frozen=True)
+class ParallelMixer:
+    """Two mixers that read the same input; half the sum of their outputs, each RMS-normed over the model width first."""
+
+    left: GroupedMixer
+    right: GatedLinearMixer
+    kind: str = "parallel"
+
+    @property
+    def cache_rows(self) -> tuple[tuple[int, int], ...]:
+        return self.left.cache_rows
+
+    @property
+    def cache_width(self) -> int:
+        return self.left.cache_width
+
+    @property
+    def state_elems(self) -> int:
+        return self.right.state_elems
+
+    @property
+    def out_features(self) -> int:
+        return self.left.out_features + self.right.out_features
+
+    def param_count(self, hidden: int) -> int:
+        return self.left.param_count(hidden) + self.right.param_count(hidden) + 2 * hidden
+
+
+def sub_mixers(m) -> tuple:
+    """The mixers that do the work: both sides of a parallel pair, else the mixer itself."""
+    return (m.left, m.right) if isinstance(m, ParallelMixer) else (m,)
+
+
+Mixer = LatentMixer | LinearMixer | GroupedMixer | GatedLinearMixer | DeltaMixer | ParallelMixer
+
+
+GLU_ALPHA = 1.702    # slope of the sigmoid in the clamped gated activation
+
+
+@dataclass(frozen=True)
+class LayerSpec:
+    """One layer of a layered (hybrid) decoder: its mixer and the width of its FFN (0: no FFN). ``gate_limit`` > 0: the FFN
+    is gated and clamped, ``min(g, limit) sigmoid(1.702 g) (clamp(u, +-limit) + 1)``; otherwise it is ungated."""
+
+    mixer: Mixer
     ff: int = 0
+    gate_limit: float = 0.0
+
+    @property
+    def ffn_maps(self) -> int:
+        """Matrices of ``hidden x ff`` elements."""
+        return 3 if self.gate_limit > 0 else 2
 
 
 @dataclass(frozen=True)
@@ -149,8 +305,10 @@ class ModelConfig:
     mla: MlaShape | None = None
     # Layered decoders: every layer names its own mixer and FFN. norm "dyt" is dynamic tanh (elementwise, no statistics);
     # ``residual_gate``: each sublayer's result is multiplied by sigmoid(W h + b) of its input and summed in fp32.
+    # ``output_norm``: sublayers read the residual itself, and their results are normed before they are added to it.
     layer_specs: tuple[LayerSpec, ...] = ()
     residual_gate: bool = False
+    output_norm: bool = False
     logit_scale: float = 1.0
     extra: dict[str, Any] = field(default_factory=dict, compare=False, hash=False)
 
@@ -194,10 +352,11 @@ class ModelConfig:
 
     def attention_param_bytes(self) -> int:
         if self.layered:
-            n = self.hidden_size * (self.vocab_size * (1 if self.tie_word_embeddings else 2) + 2) + 1
+            norm = 2 * self.hidden_size + 1 if self.norm == "dyt" else self.hidden_size
+            n = self.hidden_size * self.vocab_size * (1 if self.tie_word_embeddings else 2) + norm
             for s in self.layer_specs:
                 subs = 1 + (s.ff > 0)
-                n += s.mixer.param_count(self.hidden_size) + subs * (2 * self.hidden_size + 1)
+                n += s.mixer.param_count(self.hidden_size) + subs * norm
                 if self.residual_gate:
                     n += subs * self.hidden_size * (self.hidden_size + 1)
             return 2 * n
@@ -208,7 +367,7 @@ class ModelConfig:
 
     def ffn_param_bytes_per_layer(self, layer: int = 0) -> int:
         if self.layered:
-            return 2 * 2 * self.hidden_size * self.layer_specs[layer].ff
+            return 2 * self.layer_specs[layer].ffn_maps * self.hidden_size * self.layer_specs[layer].ff
         if self.layer_is_moe(layer):
             e = self.num_experts * 3 * self.hidden_size * self.moe_intermediate_size
             e += self.num_experts * self.hidden_size
@@ -222,8 +381,8 @@ class ModelConfig:
         return 2 * self.num_layers * self.kv_size * 2
 
     def state_bytes_per_sequence(self) -> int:
-        """fp32 recurrent state of one running sequence over all layers."""
-        return 4 * sum(s.mixer.state_elems for s in self.layer_specs)
+        """State of one running sequence over all layers: fp32 recurrences, convolution inputs in the activation type."""
+        return sum(4 * s.mixer.state_elems + 2 * getattr(s.mixer, "conv_state_elems", 0) for s in self.layer_specs)
 
     def with_layers(self, n: int) -> "ModelConfig":
         if self.layered:
@@ -269,7 +428,25 @@ def preset(name: str) -> ModelConfig:
         raise KeyError(f"unknown model preset {name!r}; known: {sorted(PRESETS)}") from None
 
 
-def _mixer_from_config(kind: str, m: dict[str, Any]) -> LatentMixer | LinearMixer:
+def _ints(m: dict[str, Any], *names: str) -> dict[str, int]:
+    return {n: int(m[n]) for n in names}
+
+
+def _grouped_heads(m: dict[str, Any]) -> None:
+    if int(m["heads"]) % int(m["kv_heads"]):
+        raise ValueError(f"{m['heads']} heads do not share {m['kv_heads']} key heads evenly")
+
+
+def _mixer_from_config(kind: str, m: dict[str, Any]) -> Mixer:
+    if kind == "delta":
+        _grouped_heads(m)
+        return DeltaMixer(**_ints(m, "heads", "kv_heads", "dim", "vdim", "conv"))
+    if kind == "parallel":
+        left, right = m["left"], m["right"]
+        _grouped_heads(left)
+        return ParallelMixer(
+            GroupedMixer(**_ints(left, "heads", "kv_heads", "dim", "vdim"), scale=float(left["scale"]), softcap=float(left["softcap"])),
+            GatedLinearMixer(**_ints(right, "heads", "dim", "vdim"), tau=float(right["tau"])))
     if kind == "latent_attention":
         rot = RotarySpec(int(m["rot"]["dims"]), float(m["rot"]["base"]))
         mixer = LatentMixer(int(m["heads"]), int(m["dim"]), int(m["rot_dim"]), int(m["vdim"]), int(m["kv_rank"]), rot, float(m["scale"]))
@@ -284,15 +461,21 @@ def _mixer_from_config(kind: str, m: dict[str, Any]) -> LatentMixer | LinearMixe
     raise ValueError(f"unsupported mixer {kind!r}")
 
 
+def _dense_mlp(layer: dict[str, Any]) -> dict[str, Any]:
+    mlp = layer.get("mlp")
+    if mlp is not None and mlp.get("kind", "dense") != "dense":
+        raise ValueError(f"unsupported feed-forward kind {mlp['kind']!r}")
+    return mlp or {"ff": 0}
+
+
 def segirax_config(cfg: dict[str, Any], name: str = "") -> ModelConfig:
     """Segirax: dynamic-tanh norms, gated fp32 residual stream, latent-attention and lightning mixers in any order, and
     ungated PolyNorm FFNs; its ``config.json`` lists every layer."""
     specs = []
     for l in cfg["layers"]:
-        mlp = l.get("mlp")
-        if mlp is not None and mlp.get("kind", "dense") != "dense":
-            raise ValueError(f"unsupported feed-forward kind {mlp['kind']!r}")
-        specs.append(LayerSpec(_mixer_from_config(l["type"], l["mixer"]), int(mlp["ff"]) if mlp is not None else 0))
+        if l["type"] not in ("latent_attention", "lightning"):
+            raise ValueError(f"unsupported mixer {l['type']!r}")
+        specs.append(LayerSpec(_mixer_from_config(l["type"], l["mixer"]), int(_dense_mlp(l)["ff"])))
     first = specs[0].mixer
     return ModelConfig(
         name=name or cfg["architecture"], architecture=cfg["architecture"], hidden_size=int(cfg["width"]), num_layers=len(specs),
@@ -302,10 +485,33 @@ def segirax_config(cfg: dict[str, Any], name: str = "") -> ModelConfig:
         logit_scale=float(cfg["logit_scale"]))
 
 
+def saninex_config(cfg: dict[str, Any], name: str = "") -> ModelConfig:
+    """Saninex: no norm before a sublayer and an RMS norm (weight stored as its distance from one) behind it, gated delta
+    rule mixers and parallel pairs of capped softmax attention and gated linear attention in any order, clamped gated FFNs;
+    its ``config.json`` lists every layer."""
+    specs = []
+    for l in cfg["layers"]:
+        if l["type"] not in ("delta", "parallel"):
+            raise ValueError(f"unsupported mixer {l['type']!r}")
+        mlp = _dense_mlp(l)
+        if mlp["ff"] and not float(mlp["limit"]) > 0:
+            raise ValueError(f"feed-forward limit {mlp['limit']!r} is not positive")
+        specs.append(LayerSpec(_mixer_from_config(l["type"], l["mixer"]), int(mlp["ff"]), float(mlp.get("limit", 0.0))))
+    first = sub_mixers(specs[0].mixer)[0]
+    return ModelConfig(
+        name=name or cfg["architecture"], architecture=cfg["architecture"], hidden_size=int(cfg["width"]), num_layers=len(specs),
+        num_q_heads=first.heads, num_kv_heads=first.kv_heads, head_dim=first.dim, intermediate_size=max(s.ff for s in specs),
+        vocab_size=int(cfg["vocab"]), rms_norm_eps=float(cfg["norm"]["eps"]), qk_norm=True, tie_word_embeddings=True,
+        hidden_act="clamped_glu", max_position_embeddings=1 << 30, norm="rmsnorm", layer_specs=tuple(specs), output_norm=True)
+
+
+LAYERED_CONFIGS = {"Segirax": segirax_config, "Saninex": saninex_config}
+
+
 def from_hf_config(cfg: dict[str, Any], name: str = "") -> ModelConfig:
     """Builds a :class:`ModelConfig` from a parsed ``config.json``."""
-    if cfg.get("architecture") == "Segirax":
-        return segirax_config(cfg, name)
+    if cfg.get("architecture") in LAYERED_CONFIGS:
+        return LAYERED_CONFIGS[cfg["architecture"]](cfg, name)
     arch = (cfg.get("architectures") or ["Qwen3ForCausalLM"])[0]
     hidden = int(cfg["hidden_size"])
     heads = int(cfg["num_attention_heads"])

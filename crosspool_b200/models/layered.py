@@ -1,8 +1,8 @@
 """Attention-side weights of layered decoders in the layout the kernels want.
 
-Every layer's linear maps of the same input become one matrix: the mixer's input projections and the residual gate
-(``[projections | gate | residual gate]``), each section padded to eight rows so that its columns in the product start on a
-16-byte boundary. Latent attention keeps its up-projections twice: per head for the absorbed form (decode), and with the
+Every layer's linear maps of the same input become one matrix: the mixer's input projections (those of both sides of a
+parallel pair) and the residual gate (``[projections | gate | residual gate]``), each section padded to eight rows so that its
+columns in the product start on a 16-byte boundary. Latent attention keeps its up-projections twice: per head for the absorbed form (decode), and with the
 shared rotary key folded in as identity rows for the expanded form (prefill), so that one product writes complete per-head
 keys. Norm parameters, gates' biases and decays are fp32.
 """
@@ -14,15 +14,11 @@ from typing import Callable
 
 import torch
 
-from ..ops.mixers import NormParams, decay_powers, expanded_shape
-from .config import LatentMixer, LayerSpec, LinearMixer, ModelConfig
+from ..ops.mixers import DeltaWeights, NormParams, decay_powers, expanded_shape
+from .config import DeltaMixer, GatedLinearMixer, GroupedMixer, LatentMixer, LayerSpec, LinearMixer, ModelConfig, ParallelMixer, ceil8
 
-# get(name, shape): the checkpoint tensor (or a random one) of that name
+# get(name, shape): the checkpoint tensor (or a random one) of that name; a size of 0 is whatever the checkpoint has
 Getter = Callable[[str, tuple[int, ...]], torch.Tensor]
-
-
-def ceil8(n: int) -> int:
-    return (n + 7) // 8 * 8
 
 
 def pad_pitch(w: torch.Tensor) -> torch.Tensor:
@@ -38,12 +34,15 @@ def pad_pitch(w: torch.Tensor) -> torch.Tensor:
 @dataclass
 class LayeredLayerWeights:
     spec: LayerSpec
-    norm1: NormParams
-    proj: torch.Tensor                      # every linear map of norm1's output
-    proj_bias: torch.Tensor                 # fp32, zero outside the residual gate
+    norm1: NormParams                       # in front of the mixer, or behind it (ModelConfig.output_norm)
+    proj: torch.Tensor                      # every linear map of the mixer's input
+    proj_bias: torch.Tensor | None          # fp32
     offs: dict[str, int]                    # first column of each section of the product
-    o: torch.Tensor                         # [hidden, mixer outputs]
-    mix: dict[str, torch.Tensor] = field(default_factory=dict)
+    o: torch.Tensor                         # [hidden, mixer outputs] (left side of a parallel pair)
+    mix: dict = field(default_factory=dict)
+    o_bias: torch.Tensor | None = None
+    o_right: torch.Tensor | None = None     # right side of a parallel pair
+    branch_norms: tuple[NormParams, ...] = ()   # of both sides' outputs
     norm2: NormParams | None = None
     rg2: torch.Tensor | None = None         # residual gate of the FFN
     rg2_bias: torch.Tensor | None = None
@@ -99,6 +98,62 @@ def _linear(m: LinearMixer, get: Getter, p: str, hidden: int, device) -> tuple[l
                       "decay_pow": decay_powers(m.decay).to(device)}
 
 
+def _grouped(m: GroupedMixer, get: Getter, p: str, hidden: int) -> tuple[list, dict, dict]:
+    """Projection sections, their biases, and what else the mixer has."""
+    rows = {"q": m.heads * m.dim, "k": m.kv_heads * m.dim, "v": m.kv_heads * m.vdim}
+    sections = [(n, get(p + n, (r, hidden))) for n, r in rows.items()] + [("hg", get(p + "g", (m.heads, hidden)))]
+    biases = {n: get(f"{p}{n}.b", (r,)).float() for n, r in rows.items()}
+    return sections, biases, {n: get(f"{p}{n[0]}.norm", (m.dim,)).float().contiguous() for n in ("q_norm", "k_norm")}
+
+
+def _gated_linear(m: GatedLinearMixer, get: Getter, p: str, hidden: int) -> tuple[list, dict]:
+    H, d, vd = m.heads, m.dim, m.vdim
+    sections = [("lin_" + n, get(p + n, (H * w, hidden))) for n, w in (("q", d), ("k", d), ("v", vd), ("g", vd))]
+    a1 = get(p + "a1", (m.rank, hidden))
+    return sections + [("lin_a", a1)], {"norm": get(p + "norm", (vd,)).float().contiguous(), "a2": pad_pitch(get(p + "a2", (H * d, a1.shape[0]))),
+                                     "a2_bias": get(p + "a2.b", (H * d,)).float().contiguous()}
+
+
+def _delta(m: DeltaMixer, get: Getter, p: str, hidden: int) -> tuple[list, dict]:
+    H, G, d, vd = m.heads, m.kv_heads, m.dim, m.vdim
+    rows = {"q": G * d, "k": G * d, "v": H * vd, "g": H * vd, "b": H, "a": H}
+    conv = torch.cat([get(f"{p}{n}.conv", (rows[n], m.conv)).float() for n in "qkv"], 0)
+    w = DeltaWeights(conv.contiguous(), -get(p + "A_log", (H,)).float().exp(), get(p + "dt_bias", (H,)).float().contiguous(),
+                     get(p + "norm", (vd,)).float().contiguous())
+    return [(n, get(p + n, (r, hidden))) for n, r in rows.items()], {"delta": w}
+
+
+def _centred_norm(get: Getter, name: str, cfg: ModelConfig) -> NormParams:
+    """An RMS norm whose weight is stored as its distance from one."""
+    return NormParams("rmsnorm", 1.0 + get(name, (cfg.hidden_size,)).float(), eps=cfg.rms_norm_eps)
+
+
+def _output_norm_layer(cfg: ModelConfig, i: int, spec: LayerSpec, get: Getter, device) -> LayeredLayerWeights:
+    """A layer whose sublayers read the residual itself and are normed behind."""
+    h, m, p = cfg.hidden_size, spec.mixer, f"l{i}.mix."
+    biases: dict = {}
+    extra: dict = {}
+    if isinstance(m, ParallelMixer):
+        left, biases, mix = _grouped(m.left, get, p + "left.", h)
+        right, mix_r = _gated_linear(m.right, get, p + "right.", h)
+        sections, mix = left + right, {**mix, **mix_r}
+        o = get(p + "left.o", (h, m.left.out_features))
+        extra = dict(o_bias=get(p + "left.o.b", (h,)).float().contiguous(), o_right=pad_pitch(get(p + "right.o", (h, m.right.out_features))),
+                     branch_norms=tuple(NormParams("rmsnorm", get(f"{p}{side}.out", (h,)).float().contiguous(), eps=cfg.rms_norm_eps)
+                                        for side in ("left", "right")))
+    else:
+        sections, mix = _delta(m, get, p, h)
+        o = get(p + "o", (h, m.out_features))
+    proj, offs = _fuse(sections)
+    bias = torch.zeros(offs["end"], dtype=torch.float32, device=device) if biases else None
+    for n, b in biases.items():
+        bias[offs[n]:offs[n] + b.shape[0]] = b
+    lw = LayeredLayerWeights(spec, _centred_norm(get, f"l{i}.norm1", cfg), proj, bias, offs, pad_pitch(o), mix, **extra)
+    if spec.ff:
+        lw.norm2 = _centred_norm(get, f"l{i}.norm2", cfg)
+    return lw
+
+
 def layered_attention_weights(cfg: ModelConfig, get: Getter, device, dtype: torch.dtype):
     """Everything but the FFNs of a layered decoder, from its named tensors (``l<i>.norm1``, ``l<i>.mix.*``,
     ``l<i>.rg1``, ...)."""
@@ -107,6 +162,9 @@ def layered_attention_weights(cfg: ModelConfig, get: Getter, device, dtype: torc
     h = cfg.hidden_size
     layers = []
     for i, spec in enumerate(cfg.layer_specs):
+        if cfg.output_norm:
+            layers.append(_output_norm_layer(cfg, i, spec, get, device))
+            continue
         p, m = f"l{i}", spec.mixer
         if isinstance(m, LatentMixer):
             sections, mix = _latent(m, get, p + ".mix.", h, dtype, device)
@@ -125,16 +183,24 @@ def layered_attention_weights(cfg: ModelConfig, get: Getter, device, dtype: torc
             lw.silu_cols = offs["g"]            # q, k and v
         layers.append(lw)
     embed = get("embed", (cfg.vocab_size, h)).contiguous()
-    return AttentionWeights(embed, layers, _norm(get, "final.norm", cfg), pad_pitch(embed))
+    final = (_centred_norm if cfg.output_norm else _norm)(get, "final.norm", cfg)
+    return AttentionWeights(embed, layers, final, pad_pitch(embed))
 
 
-def random_getter(gen: torch.Generator, dtype: torch.dtype, device) -> Getter:
-    """Random tensors by name: linear maps N(0, 0.02), norm weights one, biases zero, dynamic-tanh scalars one."""
+# stored around zero: norms behind sublayers; biases and decays of random models are zero too
+_ZERO = (".b", "A_log", "dt_bias")
+
+
+def random_getter(gen: torch.Generator, dtype: torch.dtype, device, centred_norms: bool = False) -> Getter:
+    """Random tensors by name: linear maps N(0, 0.02), norm weights one (``centred_norms``: layer norms are stored as zero),
+    biases and decay parameters zero, dynamic-tanh scalars one, 16 rows where the checkpoint would say how many."""
     from .weights import _randn
 
     def get(name: str, shape: tuple[int, ...]) -> torch.Tensor:
+        shape = tuple(n or 16 for n in shape)
         if len(shape) == 2:
             return _randn(gen, shape, dtype, device)
-        return (torch.zeros if name.endswith(".b") else torch.ones)(shape, dtype=dtype, device=device)
+        zero = name.endswith(_ZERO) or centred_norms and name.rsplit(".", 1)[-1] in ("norm1", "norm2") or centred_norms and name == "final.norm"
+        return (torch.zeros if zero else torch.ones)(shape, dtype=dtype, device=device)
 
     return get

@@ -38,9 +38,24 @@ _SEGIRAX_PROBE = {
                 "mixer": {"heads": 2, "dim": 16, "rot_dim": 8, "vdim": 16, "kv_rank": 32, "scale": 0.2, "rot": {"dims": 8, "base": 1e4}}}]}
 
 
+_SANINEX_PROBE = {
+    "architecture": "Saninex", "vocab": 256, "width": 64, "norm": {"eps": 1e-6},
+    "layers": [{"type": "delta", "mixer": {"heads": 2, "kv_heads": 1, "dim": 16, "vdim": 16, "conv": 3}, "mlp": None},
+               {"type": "parallel", "mlp": {"kind": "dense", "ff": 128, "limit": 5.0},
+                "mixer": {"left": {"heads": 2, "kv_heads": 1, "dim": 16, "vdim": 16, "scale": 0.2, "softcap": 30.0},
+                          "right": {"heads": 1, "dim": 16, "vdim": 16, "tau": 8.0}}}]}
+
+_LAYERED = {
+    "Segirax": (_SEGIRAX_PROBE, "per layer: latent attention (rotate-half rotary, output gate) or decayed linear attention; dynamic tanh "
+                                "norms, gated fp32 residual"),
+    "Saninex": (_SANINEX_PROBE, "per layer: gated delta rule (short convolutions) or, side by side, grouped-query attention (q/k RMSNorm, "
+                                "capped scores, output gate, no positions) and gated linear attention; norms behind the sublayers"),
+}
+
+
 def _probe(arch: str) -> dict:
-    if arch == "Segirax":
-        return _SEGIRAX_PROBE
+    if arch in _LAYERED:
+        return _LAYERED[arch][0]
     cfg = {k: v for k, v in _PROBE.items() if arch in _LATENT or not k.startswith(("kv_lora", "qk_", "v_head"))}
     if not arch.startswith("GptOss"):
         cfg.pop("sliding_window")
@@ -51,8 +66,7 @@ def _probe(arch: str) -> dict:
 
 def _attention_form(c: mc.ModelConfig) -> str:
     if c.layered:
-        return ("per layer: latent attention (rotate-half rotary, output gate) or decayed linear attention; dynamic tanh norms, "
-                "gated fp32 residual")
+        return _LAYERED[c.architecture][1]
     if c.mla is not None:
         return "latent attention (MLA), interleaved rotary pairs, YaRN"
     parts = ["grouped-query" if c.num_kv_heads != c.num_q_heads else "multi-head"]
@@ -78,6 +92,8 @@ def _ffn_features(spec) -> str:
             out.append(l.activation.value)
             if l.o_proj.bias_key:
                 out.append("biases")
+            if l.gate_transform.limit > 0:
+                out.append("clamped activation")
         elif isinstance(l, MoeFfnSpec):
             out.append(f"top-k {'sigmoid' if l.router_algorithm == RouterAlgorithm.SIGMOID else 'softmax'} router")
             if l.router_precision != RouterProjectionPrecision.PAYLOAD:

@@ -17,7 +17,7 @@ from pathlib import Path
 
 import torch
 
-from .config import ModelConfig
+from .config import GLU_ALPHA, ModelConfig
 from ..utils.dtype import decode_dtype
 
 FFN_KEY = re.compile(r"^model\.layers\.(\d+)\.mlp\.")
@@ -100,7 +100,7 @@ def random_attention_weights(cfg: ModelConfig, seed: int = 0, device="cpu", dtyp
     if cfg.layered:
         from .layered import layered_attention_weights, random_getter
 
-        return layered_attention_weights(cfg, random_getter(gen, dt, device), device, dt)
+        return layered_attention_weights(cfg, random_getter(gen, dt, device, cfg.output_norm), device, dt)
     embed = _randn(gen, (cfg.vocab_size, cfg.hidden_size), dt, device)
     layers = []
     if not cfg.gpu_attention_supported:
@@ -225,9 +225,13 @@ def random_ffn_layer(cfg: ModelConfig, layer: int, seed: int = 0, device="cpu", 
                 w.router = w.extra["router_fp32"].to(dt)
         return w
     if cfg.layered:
-        inter = cfg.layer_specs[layer].ff
+        inter, limit = cfg.layer_specs[layer].ff, cfg.layer_specs[layer].gate_limit
         if tp_size > 1:
-            raise NotImplementedError("a row-normalised activation needs the whole FFN row on one rank (FFN TP 1)")
+            raise NotImplementedError("the FFNs of layered decoders run whole on one GPU (FFN TP 1)")
+        if limit > 0:
+            w = FfnLayerWeights(_randn(gen, (2 * inter, h), dt, device), _randn(gen, (h, inter), dt, device))
+            w.extra.update(gated=True, gate_transform=(limit, 1.0, GLU_ALPHA))
+            return w
         w = FfnLayerWeights(_randn(gen, (inter, h), dt, device), _randn(gen, (h, inter), dt, device))
         w.extra.update(gated=False, polynorm=(torch.tensor([1.0, 1.0, 1.0, 0.0], device=device) / 3, cfg.rms_norm_eps))
         return w
@@ -300,7 +304,7 @@ def load_attention_from_safetensors(cfg: ModelConfig, model_dir: str | Path, dev
 
         def named(key: str, shape: tuple[int, ...]) -> torch.Tensor:
             t = get(key)
-            if tuple(t.shape) != shape:
+            if len(t.shape) != len(shape) or any(n not in (m, 0) for m, n in zip(t.shape, shape)):
                 raise ValueError(f"{key} has shape {tuple(t.shape)}, the configuration gives {shape}")
             return t
 

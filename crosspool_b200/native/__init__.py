@@ -15,7 +15,7 @@ import ctypes as C
 import functools
 from pathlib import Path
 
-EXPECTED_ABI = 22
+EXPECTED_ABI = 23
 HERE = Path(__file__).resolve().parent
 
 
@@ -256,7 +256,7 @@ class PrefillAttnArgs(C.Structure):
 def _struct(name: str, doc: str, **fields):
     """A ctypes.Structure whose fields are given as ``ctype="space separated names"`` groups in ABI order, keyed
     ``group_index_ctype``."""
-    types = {"ptr": C.c_void_p, "int": C.c_int, "float": C.c_float, "ptr8": C.c_void_p * 8}
+    types = {"ptr": C.c_void_p, "int": C.c_int, "float": C.c_float, "ptr8": C.c_void_p * 8, "ptr2": C.c_void_p * 2, "int2": C.c_int * 2}
     decl = [(n, types[key.split("_", 1)[1]]) for key, names in fields.items() for n in names.split()]
     return type(name, (C.Structure,), {"_fields_": decl, "__doc__": doc})
 
@@ -268,6 +268,24 @@ ResidNormArgs = _struct("ResidNormArgs", "XpResidNormArgs", a_ptr="resid", b_ptr
 PolyNormArgs = _struct("PolyNormArgs", "XpPolyNormArgs", a_ptr="z coef out", b_int="rows cols ld_z ld_out", c_float="eps", d_int="f32")
 GatedRmsArgs = _struct("GatedRmsArgs", "XpGatedRmsArgs", a_ptr="o weight gate out", b_int="rows cols ld_o ld_gate ld_out", c_float="eps",
                        d_int="f32")
+PostNormArgs = _struct("PostNormArgs", "XpPostNormArgs", a_ptr="resid", b_ptr2="branches branch_w", c_ptr="ids table sel weight out_weight out",
+                       d_int="rows hidden nbranches", e_int2="ld_branch", f_int="ld_out vocab", g_float="eps", h_int="f32")
+HeadGateArgs = _struct("HeadGateArgs", "XpHeadGateArgs", a_ptr="o weight gate out", b_int="rows heads dim ld_o ld_gate ld_out", c_float="eps",
+                       d_int="f32")
+GluArgs = _struct("GluArgs", "XpGluArgs", a_ptr="z out", b_int="rows cols ld_z ld_out", c_float="limit up_add alpha")
+GroupedPrepArgs = _struct("GroupedPrepArgs", "XpGroupedPrepArgs", a_ptr="proj q_norm k_norm slots k_cache v_cache q_out",
+                          b_int="rows heads kv_heads group_pad dim vdim dq dv ld_proj q_off k_off v_off", c_float="eps", d_int="f32")
+GroupedAttnArgs = _struct("GroupedAttnArgs", "XpGroupedAttnArgs", a_ptr="q k_cache v_cache out gate row_seq positions slots block_table",
+                          b_int="rows heads kv_heads group_pad dim vdim dq dv ld_gate ld_out page_size max_blocks", c_float="scale softcap",
+                          d_int="f32")
+GatedLinearArgs = _struct("GatedLinearArgs", "XpGatedLinearArgs",
+                          a_ptr="proj z a2 a2_bias norm state out positions slots state_slots q_starts q_lens ws",
+                          b_int="rows seqs heads dim vdim ld_proj ld_out q_off k_off v_off g_off a_off rank ld_a2 segs seg_tokens force_sequential",
+                          c_float="inv_tau qscale eps", d_int="f32")
+DeltaArgs = _struct("DeltaArgs", "XpDeltaArgs",
+                    a_ptr="proj conv_w conv_state neg_a dt_bias norm state out qkv qk_scale beta_g ws positions slots state_slots q_starts q_lens",
+                    b_int="rows seqs max_q heads kv_heads dim vdim taps ld_proj ld_out q_off k_off v_off g_off b_off a_off force_sequential",
+                    c_float="qscale eps", d_int="f32")
 LatentPrepArgs = _struct("LatentPrepArgs", "XpLatentPrepArgs", a_ptr="proj norm_w freq positions slots cache q_plain q_abs q_exp",
                          b_int="rows heads dim rot rot_dims kv_rank ld_proj q_off kv_off ld_cache qp_rows dim_p ld_abs dq_pad abs_rows",
                          c_float="eps", d_int="f32")
@@ -284,7 +302,11 @@ LinearAttnArgs = _struct("LinearAttnArgs", "XpLinearAttnArgs",
 def _declare_mixers(lib: C.CDLL) -> None:
     for fn, args in (("xp_resid_norm", ResidNormArgs), ("xp_polynorm", PolyNormArgs), ("xp_gated_rms", GatedRmsArgs),
                      ("xp_latent_prep", LatentPrepArgs), ("xp_latent_attn", LatentAttnArgs), ("xp_latent_gather", LatentGatherArgs),
-                     ("xp_linear_attn_decode", LinearAttnArgs), ("xp_linear_attn_prefill", LinearAttnArgs)):
+                     ("xp_linear_attn_decode", LinearAttnArgs), ("xp_linear_attn_prefill", LinearAttnArgs),
+                     ("xp_post_norm", PostNormArgs), ("xp_head_gate", HeadGateArgs), ("xp_glu_f32", GluArgs),
+                     ("xp_grouped_prep", GroupedPrepArgs), ("xp_grouped_attn", GroupedAttnArgs),
+                     ("xp_gated_linear_decode", GatedLinearArgs), ("xp_gated_linear_prefill", GatedLinearArgs),
+                     ("xp_delta_decode", DeltaArgs), ("xp_delta_prep", DeltaArgs), ("xp_delta_prefill", DeltaArgs)):
         getattr(lib, fn).restype = C.c_int
         getattr(lib, fn).argtypes = [C.POINTER(args), C.c_void_p]
     lib.xp_gemm_f32.restype = C.c_int

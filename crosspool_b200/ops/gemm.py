@@ -234,7 +234,7 @@ def gateup_swiglu(x: torch.Tensor, w_gate_up: torch.Tensor, *, out: torch.Tensor
                   bias: torch.Tensor | None = None, gate_limit: float = 0.0, up_add: float = 0.0,
                   act_alpha: float = 0.0, splits: int = 0, bn: int = 0, num_sms: int = 0) -> torch.Tensor:
     """``silu(x @ Wg.T) * (x @ Wu.T)`` with ``w_gate_up = cat([Wg, Wu])`` of shape ``[2*I, k]``."""
-    x2 = x.reshape(-1, x.shape[-1])
+    x2 = x if x.dim() == 2 else x.reshape(-1, x.shape[-1])
     rows = x2.shape[0]
     inter = w_gate_up.shape[0] // 2
     if out is None:

@@ -1,6 +1,7 @@
-"""Row-wise and mixer operators of layered decoders (``csrc/kernels/{row_ops,latent_attn,linear_attn}.cu``): gated fp32
-residual streams with a fused norm, PolyNorm, latent attention over a paged latent cache, decayed linear attention with
-per-sequence states. Every operator exists for bf16 and for fp32 activations; norms, scores, gates and states are fp32 in
+"""Row-wise and mixer operators of layered decoders (``csrc/kernels/{row_ops,latent_attn,linear_attn,grouped_attn,
+recurrence,...}.cu``): fp32 residual streams with gates or norms behind the sublayers, PolyNorm, latent attention over a paged
+latent cache, grouped-query attention with capped scores, and recurrences with per-sequence states (decayed linear attention,
+per-channel decays, the gated delta rule). Every operator exists for bf16 and for fp32 activations; norms, scores, gates and states are fp32 in
 both. The reference borrows such layers from its serving engine (pyproject.toml:17-35).
 """
 
@@ -13,6 +14,7 @@ from typing import Sequence
 import torch
 
 from .. import native
+from ..models.config import attention_shape
 
 NORM_KINDS = {"rmsnorm": 0, "layernorm": 1, "dyt": 2}
 # Rows of a recurrence computed with one set of matrix products (decay powers are tabulated up to this).
@@ -69,6 +71,53 @@ def resid_norm(resid: torch.Tensor, norm: NormParams | None, out: torch.Tensor |
         a.weight, a.bias, a.alpha, a.kind, a.eps = norm.weight.data_ptr(), _ptr(norm.bias), _ptr(norm.alpha), NORM_KINDS[norm.kind], norm.eps
     a.f32 = _f32(act)
     native.check(native.kernels().xp_resid_norm(C.byref(a), _stream(resid)), "xp_resid_norm")
+
+
+def post_norm(resid: torch.Tensor, out: torch.Tensor | None, *, norm: NormParams | None = None, branches: Sequence[torch.Tensor] = (),
+              branch_norms: Sequence[NormParams] = (), ids: torch.Tensor | None = None, table: torch.Tensor | None = None,
+              out_norm: NormParams | None = None, sel: torch.Tensor | None = None, rows: int | None = None, eps: float = 1e-6) -> None:
+    """``resid += norm(branch)`` (``branch_norms``: of the mean of the normed branches; ``ids``: ``resid = table[ids]``) in
+    fp32, then ``out = resid``, or ``out_norm(resid)``. All norms are RMS norms with ``eps``. With ``sel`` (int32) only the
+    selected rows are computed and the residual is left alone."""
+    a = native.PostNormArgs()
+    act = branches[0] if branches else table
+    assert resid.dtype == torch.float32 and resid.is_contiguous() and len(branch_norms) in (0, len(branches))
+    a.resid = resid.data_ptr()
+    for i, b in enumerate(branches):
+        assert b.dtype == act.dtype and b.stride(1) == 1
+        a.branches[i], a.ld_branch[i] = b.data_ptr(), b.stride(0)
+    for i, n in enumerate(branch_norms):
+        a.branch_w[i] = n.weight.data_ptr()
+    a.ids, a.table, a.sel, a.out = _ptr(ids), _ptr(table), _ptr(sel), _ptr(out)
+    a.weight = norm.weight.data_ptr() if norm is not None else None
+    a.out_weight = out_norm.weight.data_ptr() if out_norm is not None else None
+    a.rows = rows if rows is not None else (sel.shape[0] if sel is not None else resid.shape[0])
+    a.hidden, a.nbranches = resid.shape[1], len(branches)
+    a.ld_out = out.stride(0) if out is not None else 0
+    a.vocab = table.shape[0] if table is not None else 0
+    a.eps, a.f32 = norm.eps if norm is not None else eps, _f32(act)
+    native.check(native.kernels().xp_post_norm(C.byref(a), _stream(resid)), "xp_post_norm")
+
+
+def head_gate(o: torch.Tensor, weight: torch.Tensor, gate: torch.Tensor, eps: float, out: torch.Tensor) -> torch.Tensor:
+    """``rmsnorm(o) * weight * silu(gate)`` with the norm over every head of ``len(weight)`` columns; ``o`` fp32."""
+    assert o.dtype == torch.float32 and weight.dtype == torch.float32 and gate.dtype == out.dtype
+    a = native.HeadGateArgs()
+    a.o, a.weight, a.gate, a.out = o.data_ptr(), weight.data_ptr(), gate.data_ptr(), out.data_ptr()
+    a.rows, a.heads, a.dim = o.shape[0], o.shape[1] // weight.numel(), weight.numel()
+    a.ld_o, a.ld_gate, a.ld_out, a.eps, a.f32 = o.stride(0), gate.stride(0), out.stride(0), eps, _f32(out)
+    native.check(native.kernels().xp_head_gate(C.byref(a), _stream(o)), "xp_head_gate")
+    return out
+
+
+def glu_f32(z: torch.Tensor, limit: float, up_add: float, alpha: float, out: torch.Tensor) -> torch.Tensor:
+    """Clamped gated activation of fp32 rows ``[g, u]`` (the bf16 product applies it in its epilogue)."""
+    assert z.dtype == out.dtype == torch.float32
+    a = native.GluArgs()
+    a.z, a.out, a.rows, a.cols, a.ld_z, a.ld_out = z.data_ptr(), out.data_ptr(), z.shape[0], z.shape[1] // 2, z.stride(0), out.stride(0)
+    a.limit, a.up_add, a.alpha = limit, up_add, alpha
+    native.check(native.kernels().xp_glu_f32(C.byref(a), _stream(z)), "xp_glu_f32")
+    return out
 
 
 def polynorm(z: torch.Tensor, coef: torch.Tensor, eps: float, out: torch.Tensor) -> torch.Tensor:
@@ -164,18 +213,9 @@ def latent_gather(cache: torch.Tensor, out: torch.Tensor, block_table: torch.Ten
     native.check(native.kernels().xp_latent_gather(C.byref(a), _stream(cache)), "xp_latent_gather")
 
 
-# tcgen05 prefill shapes (query/key width, value width), narrowest first
-EXPANDED_SHAPES = ((64, 64), (128, 64), (128, 128), (192, 128))
-
-
 def expanded_shape(dim: int, rot: int, vdim: int) -> tuple[int, int] | None:
     """Padded widths of the expanded (per-head keys and values) prefill form, None when no kernel covers the sizes."""
-    if vdim % 8:
-        return None
-    for dq, dv in EXPANDED_SHAPES:
-        if dim + rot <= dq and vdim <= dv:
-            return dq, dv
-    return None
+    return attention_shape(dim + rot, vdim)
 
 
 def expanded_prefill(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, out: torch.Tensor, q_starts: torch.Tensor, q_lens: torch.Tensor,
@@ -261,3 +301,133 @@ def linear_attn_prefill(proj, state, decay, decay_pow, out, positions, slots, st
         assert ws is not None and ws.numel() >= q_lens.shape[0] * heads * segs * dim * vdim
         a.segs, a.seg_tokens, a.ws = segs, seg_tokens, ws.data_ptr()
     native.check(native.kernels().xp_linear_attn_prefill(C.byref(a), _stream(proj)), "xp_linear_attn_prefill", 3 if a.segs > 1 else 1)
+
+
+# ------------------------------------------------------------------------------------------ grouped-query attention
+
+def group_pad(heads: int, kv_heads: int) -> int:
+    """Query heads of a group rounded up to a power of two (the tiles of the prefill kernel)."""
+    n = 1
+    while n < heads // kv_heads:
+        n *= 2
+    return n
+
+
+def grouped_prep(proj: torch.Tensor, q_norm: torch.Tensor | None, k_norm: torch.Tensor | None, slots: torch.Tensor, k_cache: torch.Tensor,
+                 v_cache: torch.Tensor, q_out: torch.Tensor, *, heads: int, dim: int, vdim: int, offs: tuple[int, int, int], eps: float) -> None:
+    """Query and key norms, cache write and the padded query layout ``q_out`` ``[rows, kv_heads, group_pad, dq]``; caches
+    ``[pages, page, kv_heads, dq]`` and ``[..., dv]``."""
+    assert k_cache.dtype == proj.dtype == q_out.dtype and (q_norm is None or q_norm.dtype == torch.float32)
+    a = native.GroupedPrepArgs()
+    a.proj, a.q_norm, a.k_norm, a.slots = proj.data_ptr(), _ptr(q_norm), _ptr(k_norm), slots.data_ptr()
+    a.k_cache, a.v_cache, a.q_out = k_cache.data_ptr(), v_cache.data_ptr(), q_out.data_ptr()
+    a.rows, a.heads, a.kv_heads, a.group_pad = proj.shape[0], heads, k_cache.shape[2], q_out.shape[2]
+    a.dim, a.vdim, a.dq, a.dv, a.ld_proj = dim, vdim, k_cache.shape[3], v_cache.shape[3], proj.stride(0)
+    a.q_off, a.k_off, a.v_off = offs
+    a.eps, a.f32 = eps, _f32(proj)
+    native.check(native.kernels().xp_grouped_prep(C.byref(a), _stream(proj)), "xp_grouped_prep")
+
+
+def grouped_attn(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, out: torch.Tensor, block_table: torch.Tensor,
+                 positions: torch.Tensor, slots: torch.Tensor, *, heads: int, dim: int, vdim: int, scale: float, softcap: float = 0.0,
+                 gate: torch.Tensor | None = None, row_seq: torch.Tensor | None = None) -> torch.Tensor:
+    """Rows of queries ``[rows, kv_heads, group_pad, dq]`` against the first ``positions[r] + 1`` cached tokens of their
+    sequences, any sizes and types; ``out`` ``[rows, heads * vdim]``, head h multiplied by ``sigmoid(gate[:, h])``."""
+    step = 32768
+    for lo in range(0, q.shape[0], step):
+        n = min(step, q.shape[0] - lo)
+        a = native.GroupedAttnArgs()
+        a.q, a.k_cache, a.v_cache, a.out = q[lo:].data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), out[lo:].data_ptr()
+        a.gate = gate[lo:].data_ptr() if gate is not None else None
+        a.row_seq = row_seq[lo:].data_ptr() if row_seq is not None else None
+        a.positions, a.slots = positions[lo:].data_ptr(), slots[lo:].data_ptr()
+        a.block_table = block_table[lo:].data_ptr() if row_seq is None else block_table.data_ptr()
+        a.rows, a.heads, a.kv_heads, a.group_pad, a.dim, a.vdim = n, heads, q.shape[1], q.shape[2], dim, vdim
+        a.dq, a.dv, a.ld_gate, a.ld_out = q.shape[3], v_cache.shape[3], gate.stride(0) if gate is not None else 0, out.stride(0)
+        a.page_size, a.max_blocks, a.scale, a.softcap, a.f32 = k_cache.shape[1], block_table.stride(0), scale, softcap, _f32(q)
+        native.check(native.kernels().xp_grouped_attn(C.byref(a), _stream(q)), "xp_grouped_attn")
+    return out
+
+
+# ------------------------------------------------------------------------------------------ input-dependent recurrences
+
+def _recurrent(a, proj, state, out, positions, slots, state_slots, heads, dim, vdim):
+    assert state.dtype == torch.float32
+    a.proj, a.state, a.out, a.positions, a.slots, a.state_slots = (t.data_ptr() for t in (proj, state, out, positions, slots, state_slots))
+    a.heads, a.dim, a.vdim, a.ld_proj, a.ld_out, a.f32, a.rows = heads, dim, vdim, proj.stride(0), out.stride(0), _f32(proj), proj.shape[0]
+    return a
+
+
+def gated_linear_decode(proj, state, a2, a2_bias, norm, out, positions, slots, state_slots, *, heads: int, dim: int, vdim: int,
+                        offs: tuple[int, int, int, int, int], tau: float, eps: float) -> None:
+    """One token per row from the projection (q, k, v, gate and the decay's first map at ``offs``) to the gated heads
+    ``out`` ``[rows, heads * vdim]``; row r updates state slot ``state_slots[r]``."""
+    a = _recurrent(native.GatedLinearArgs(), proj, state, out, positions, slots, state_slots, heads, dim, vdim)
+    assert a2.dtype == proj.dtype == out.dtype and a2_bias.dtype == norm.dtype == torch.float32
+    a.a2, a.a2_bias, a.norm = a2.data_ptr(), a2_bias.data_ptr(), norm.data_ptr()
+    a.q_off, a.k_off, a.v_off, a.g_off, a.a_off = offs
+    a.rank, a.ld_a2, a.inv_tau, a.qscale, a.eps = a2.shape[1], a2.stride(0), 1.0 / tau, dim ** -0.5, eps
+    native.check(native.kernels().xp_gated_linear_decode(C.byref(a), _stream(proj)), "xp_gated_linear_decode")
+
+
+def gated_linear_prefill(proj, z, state, out, positions, slots, state_slots, q_starts, q_lens, *, heads: int, dim: int, vdim: int,
+                         offs: tuple[int, int, int], tau: float, force_sequential: bool = False) -> None:
+    """Portions of sequences: portion i covers rows ``q_starts[i] .. + q_lens[i]`` and continues state ``state_slots[i]``;
+    ``z`` fp32 ``[rows, heads * dim]`` is the decay map's value, ``out`` fp32 ``[rows, heads * vdim]``."""
+    a = _recurrent(native.GatedLinearArgs(), proj, state, out, positions, slots, state_slots, heads, dim, vdim)
+    assert z.dtype == out.dtype == torch.float32 and z.is_contiguous()
+    a.z, a.q_starts, a.q_lens, a.seqs = z.data_ptr(), q_starts.data_ptr(), q_lens.data_ptr(), q_lens.shape[0]
+    a.q_off, a.k_off, a.v_off = offs
+    a.inv_tau, a.qscale, a.force_sequential = 1.0 / tau, dim ** -0.5, int(force_sequential)
+    native.check(native.kernels().xp_gated_linear_prefill(C.byref(a), _stream(proj)), "xp_gated_linear_prefill")
+
+
+@dataclass
+class DeltaWeights:
+    """Parameters of the gated delta rule around its projections, fp32: convolution ``[channels, taps]`` over queries, keys
+    and values, ``-exp(A_log)`` and the step bias per head, the output norm ``[vdim]``."""
+
+    conv: torch.Tensor
+    neg_a: torch.Tensor
+    dt_bias: torch.Tensor
+    norm: torch.Tensor
+
+
+@dataclass
+class DeltaScratch:
+    """What the prefill kernels hand on: convolved rows, unit-vector factors, ``beta`` and ``log g``."""
+
+    qkv: torch.Tensor
+    qk_scale: torch.Tensor
+    beta_g: torch.Tensor
+
+
+def _delta(proj, conv_state, w: DeltaWeights, state, out, positions, slots, state_slots, heads, kv_heads, dim, vdim, offs, eps):
+    a = _recurrent(native.DeltaArgs(), proj, state, out, positions, slots, state_slots, heads, dim, vdim)
+    assert conv_state.dtype == proj.dtype and w.conv.dtype == torch.float32
+    a.conv_w, a.conv_state, a.neg_a, a.dt_bias, a.norm = (t.data_ptr() for t in (w.conv, conv_state, w.neg_a, w.dt_bias, w.norm))
+    a.kv_heads, a.taps, a.qscale, a.eps = kv_heads, w.conv.shape[1], dim ** -0.5, eps
+    a.q_off, a.k_off, a.v_off, a.g_off, a.b_off, a.a_off = offs
+    return a
+
+
+def delta_decode(proj, conv_state, w: DeltaWeights, state, out, positions, slots, state_slots, *, heads: int, kv_heads: int, dim: int,
+                 vdim: int, offs: tuple[int, int, int, int, int, int], eps: float) -> None:
+    """One token per row from the projection (q, k, v, gate, b, a at ``offs``) to the gated heads ``out``; row r updates
+    state and convolution slot ``state_slots[r]``."""
+    a = _delta(proj, conv_state, w, state, out, positions, slots, state_slots, heads, kv_heads, dim, vdim, offs, eps)
+    assert out.dtype == proj.dtype
+    native.check(native.kernels().xp_delta_decode(C.byref(a), _stream(proj)), "xp_delta_decode")
+
+
+def delta_prefill(proj, conv_state, w: DeltaWeights, state, out, positions, slots, state_slots, q_starts, q_lens, max_q: int,
+                  scratch: DeltaScratch, *, heads: int, kv_heads: int, dim: int, vdim: int, offs: tuple[int, int, int, int, int, int],
+                  eps: float, force_sequential: bool = False) -> None:
+    """Portions of sequences (the longest has ``max_q`` rows): convolution and recurrence; ``out`` fp32 ``[rows, heads * vdim]``."""
+    a = _delta(proj, conv_state, w, state, out, positions, slots, state_slots, heads, kv_heads, dim, vdim, offs, eps)
+    assert out.dtype == torch.float32 and scratch.qkv.dtype == proj.dtype
+    a.qkv, a.qk_scale, a.beta_g = scratch.qkv.data_ptr(), scratch.qk_scale.data_ptr(), scratch.beta_g.data_ptr()
+    a.q_starts, a.q_lens, a.seqs, a.max_q, a.force_sequential = q_starts.data_ptr(), q_lens.data_ptr(), q_lens.shape[0], max_q, int(force_sequential)
+    lib = native.kernels()
+    native.check(lib.xp_delta_prep(C.byref(a), _stream(proj)), "xp_delta_prep")
+    native.check(lib.xp_delta_prefill(C.byref(a), _stream(proj)), "xp_delta_prefill")
