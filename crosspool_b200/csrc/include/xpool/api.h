@@ -279,6 +279,18 @@ typedef struct XpDecodeAttnArgs {
   int reserved;
 } XpDecodeAttnArgs;
 
+/* Tensor-core decode attention of single rows: padded query groups, keys and values of different widths, capped scores,
+ * output gates, rows that belong to any sequence. */
+typedef struct XpDecodeRowsArgs {
+  XpDecodeAttnArgs a;         /* q [rows, kv_heads, group_pad, head_dim]; q_heads without the padding; seq_lens unused */
+  const int* row_seq;         /* [rows] block-table row, or null: row r uses table row r */
+  const int* positions;       /* [rows] row r attends to positions[r] + 1 tokens */
+  const int* slots;           /* [rows] < 0: padding row (zeros are stored) */
+  const void* gate;           /* optional bf16 logits [rows, ld_gate]: head h's output is multiplied by sigmoid */
+  int group_pad, v_dim, v_valid, ld_out, ld_gate;
+  float softcap;              /* > 0: scores become softcap tanh(score / softcap) */
+} XpDecodeRowsArgs;
+
 typedef struct XpPrefillAttnArgs {
   const void* q;              /* bf16 [total_q, q_heads, head_dim], sequences packed */
   const void* k_cache;
@@ -305,11 +317,14 @@ typedef struct XpPrefillAttnArgs {
   const void* gate;           /* optional bf16 [total_q, ld_gate] logits: head h's output is multiplied by sigmoid */
   int ld_gate;
   int p_pair;                 /* probabilities as a bf16 pair in the second product */
+  int group_valid;            /* > 0: query heads of a group that exist (the others are padding of q, q_heads counts them) */
+  float softcap;              /* > 0: scores become softcap tanh(score / softcap) */
 } XpPrefillAttnArgs;
 
 int xp_rope_kv(const XpRopeArgs* a, void* stream);
 int xp_decode_attn_splits(int batch, int kv_heads, int max_len);
 int xp_decode_attn(const XpDecodeAttnArgs* a, void* stream);
+int xp_decode_rows(const XpDecodeRowsArgs* a, void* stream);
 int xp_prefill_attn(const XpPrefillAttnArgs* a, void* stream);
 int xp_prefill_attn_umma(const XpPrefillAttnArgs* a, void* stream);
 

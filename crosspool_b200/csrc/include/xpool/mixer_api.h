@@ -6,6 +6,7 @@
 #ifndef XPOOL_MIXER_API_H_
 #define XPOOL_MIXER_API_H_
 
+#include <stddef.h>
 #include <stdint.h>
 
 #ifdef __cplusplus
@@ -138,8 +139,9 @@ typedef struct XpGatedLinearArgs {
   const int* state_slots;
   const int* q_starts;
   const int* q_lens;
-  float* ws;             /* chunked prefill: states and decays of segments */
-  int rows, seqs, heads, dim, vdim, ld_proj, ld_out, q_off, k_off, v_off, g_off, a_off, rank, ld_a2;
+  float* ws;             /* chunked prefill, segs > 1: [seqs, heads, segs, dim * vdim + dim] */
+  void* records;         /* chunked prefill: xp_gated_linear_record_bytes(); z is overwritten */
+  int rows, seqs, max_q, heads, dim, vdim, ld_proj, ld_out, q_off, k_off, v_off, g_off, a_off, rank, ld_a2;
   int segs, seg_tokens, force_sequential;
   float inv_tau, qscale, eps;
   int f32;
@@ -161,7 +163,7 @@ typedef struct XpDeltaArgs {
   void* qkv;             /* prefill: [rows, channels] */
   float* qk_scale;       /* prefill: [rows, 2, kv_heads] */
   float* beta_g;         /* prefill: [rows, 2, heads]: beta, log g */
-  void* ws;              /* chunked prefill */
+  void* ws;              /* chunked prefill: xp_delta_ws_bytes() */
   const int* positions;
   const int* slots;
   const int* state_slots;
@@ -256,6 +258,10 @@ int xp_gated_linear_prefill(const XpGatedLinearArgs* a, void* stream);
 int xp_delta_decode(const XpDeltaArgs* a, void* stream);
 int xp_delta_prep(const XpDeltaArgs* a, void* stream);
 int xp_delta_prefill(const XpDeltaArgs* a, void* stream);
+int xp_delta_chunked(const XpDeltaArgs* a, void* stream);           /* 1: sizes not covered */
+int xp_gated_linear_chunked(const XpGatedLinearArgs* a, void* stream);
+size_t xp_delta_ws_bytes(int rows, int seqs, int heads);
+size_t xp_gated_linear_record_bytes(int rows, int seqs, int heads);
 int xp_latent_prep(const XpLatentPrepArgs* a, void* stream);
 int xp_latent_attn(const XpLatentAttnArgs* a, void* stream);
 int xp_latent_gather(const XpLatentGatherArgs* a, void* stream);

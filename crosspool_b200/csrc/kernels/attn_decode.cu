@@ -9,6 +9,8 @@
 // it, pyproject.toml:17-35); the oracle is a plain fp32 softmax(QK^T)V.
 #include <math_constants.h>
 
+#include <type_traits>
+
 #include "xpool/api.h"
 #include "xpool/sm100.cuh"
 #include "xpool/tensormap.hpp"
@@ -271,6 +273,10 @@ decode_attn_kernel(XpDecodeAttnArgs a) {
 // mma.sync rather than tcgen05: the op moves 2 x D x 2 bytes per token for 4 x G x D flops, i.e.
 // at most 16 flop/byte with 8 heads per group -- two orders below the tensor roofline -- and a
 // UMMA tile needs 64 or 128 query rows where there are 16 at most.
+//
+// kRows: the form of layered decoders (XpDecodeRowsArgs): rows name their sequence, query groups are padded, keys and values
+// differ in width, scores may be capped, outputs gated, and the probabilities enter the second product as a bf16 pair (high
+// and low part), so that they keep 16 mantissa bits.
 constexpr int kTcStages = 3;
 
 __device__ __forceinline__ void tma_load_kv(uint32_t dst, const CUtensorMap* m, uint32_t bar, int d0, int head, int token) {
@@ -301,20 +307,50 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
   return *reinterpret_cast<uint32_t*>(&h);
 }
 
-template <int D>
+// (low, high) packed as bf16, and what the rounding left of them
+__device__ __forceinline__ uint32_t pack_rest(float lo, float hi, uint32_t packed) {
+  const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&packed));
+  return pack_bf16(lo - f.x, hi - f.y);
+}
+
+__device__ __forceinline__ const XpDecodeAttnArgs& base_of(const XpDecodeRowsArgs& a) { return a.a; }
+__device__ __forceinline__ const XpDecodeAttnArgs& base_of(const XpDecodeAttnArgs& a) { return a; }
+
+template <typename A>
+__device__ __forceinline__ int row_len(const A& args, int b) {
+  if constexpr (std::is_same<A, XpDecodeRowsArgs>::value) return args.slots[b] < 0 ? 0 : args.positions[b] + 1;
+  else return args.seq_lens[b];
+}
+
+// Stores one element of a finished head.
+template <int DV, typename A>
+__device__ __forceinline__ void store_out(const A& args, int b, int hq, int d, float v) {
+  if constexpr (std::is_same<A, XpDecodeRowsArgs>::value) {
+    if (d >= args.v_valid) return;
+    if (args.gate != nullptr)
+      v *= 1.f / (1.f + expf(-__bfloat162float(reinterpret_cast<const __nv_bfloat16*>(args.gate)[static_cast<size_t>(b) * args.ld_gate + hq])));
+    reinterpret_cast<__nv_bfloat16*>(args.a.out)[static_cast<size_t>(b) * args.ld_out + hq * args.v_valid + d] = __float2bfloat16_rn(v);
+  } else {
+    reinterpret_cast<__nv_bfloat16*>(args.out)[(static_cast<size_t>(b) * args.q_heads + hq) * DV + d] = __float2bfloat16_rn(v);
+  }
+}
+
+template <int DQ, int DV, typename A>
 __global__ void __launch_bounds__(kDecodeThreads, 2)
-decode_attn_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constant__ CUtensorMap tmap_v,
-                      XpDecodeAttnArgs a) {
-  constexpr int kHalves = D / 64;              // 64-dim boxes per row
+decode_attn_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constant__ CUtensorMap tmap_v, A args) {
+  constexpr bool kRows = std::is_same<A, XpDecodeRowsArgs>::value;
+  const XpDecodeAttnArgs& a = base_of(args);
+  constexpr int kHalves = DQ / 64;             // 64-dim boxes per key row
+  constexpr int kVHalves = DV / 64;            // ... per value row
   constexpr int kBox = 16 * 128;               // bytes of one box: 16 tokens x 64 dims
-  constexpr int kStage = 2 * kHalves * kBox;   // K boxes then V boxes
+  constexpr int kStage = (kHalves + kVHalves) * kBox;   // K boxes then V boxes
   constexpr int kWarpRing = kTcStages * kStage;
   extern __shared__ uint8_t smem_dyn[];
   __shared__ __align__(8) uint64_t full[4][kTcStages];
 
   const int split = blockIdx.x, hk = blockIdx.y, b = blockIdx.z;
   const int G = a.q_heads / a.kv_heads;
-  const int len = a.seq_lens[b];
+  const int len = row_len(args, b);
   const int nsplit = gridDim.x;
   int chunk = a.chunk_tokens;
   if (chunk <= 0) {
@@ -342,7 +378,11 @@ decode_attn_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_c
   const int n_it = tiles > warp ? (tiles - warp + 3) >> 2 : 0;
   const int page_shift = 31 - __clz(a.page_size);
   const int page_mask = a.page_size - 1;
-  const int* table = a.block_table + static_cast<size_t>(b) * a.max_blocks;
+  int table_row = b;
+  if constexpr (kRows) {
+    if (args.row_seq != nullptr) table_row = args.row_seq[b];
+  }
+  const int* table = a.block_table + static_cast<size_t>(table_row) * a.max_blocks;
   // lane i looks up the cache position of the tile of iteration (base + i)
   auto lookup = [&](int it) -> int {
     if (it >= n_it) return 0;
@@ -356,9 +396,9 @@ decode_attn_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_c
     const uint32_t dst = ring + s * kStage;
     sm100::mbar_arrive_expect_tx(&full[warp][s], kStage);
 #pragma unroll
-    for (int h = 0; h < kHalves; ++h) {
-      tma_load_kv(dst + h * kBox, &tmap_k, bar, h * 64, hk, tok);
-      tma_load_kv(dst + (kHalves + h) * kBox, &tmap_v, bar, h * 64, hk, tok);
+    for (int h = 0; h < (kHalves > kVHalves ? kHalves : kVHalves); ++h) {
+      if (h < kHalves) tma_load_kv(dst + h * kBox, &tmap_k, bar, h * 64, hk, tok);
+      if (h < kVHalves) tma_load_kv(dst + (kHalves + h) * kBox, &tmap_v, bar, h * 64, hk, tok);
     }
   };
 #pragma unroll
@@ -368,23 +408,29 @@ decode_attn_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_c
   }
 
   // Q fragments (A operand), unscaled; rows >= G are zero
-  uint32_t qf[D / 16][4];
+  uint32_t qf[DQ / 16][4];
   {
-    const __nv_bfloat16* qb = reinterpret_cast<const __nv_bfloat16*>(a.q) + (static_cast<size_t>(b) * a.q_heads + hk * G) * D;
+    size_t q_row = static_cast<size_t>(b) * a.q_heads + hk * G;
+    if constexpr (kRows) q_row = (static_cast<size_t>(b) * a.kv_heads + hk) * args.group_pad;
+    const __nv_bfloat16* qb = reinterpret_cast<const __nv_bfloat16*>(a.q) + q_row * DQ;
 #pragma unroll
-    for (int ks = 0; ks < D / 16; ++ks) {
+    for (int ks = 0; ks < DQ / 16; ++ks) {
       const int c = ks * 16 + q4 * 2;
-      qf[ks][0] = g < G ? *reinterpret_cast<const uint32_t*>(qb + g * D + c) : 0u;
-      qf[ks][1] = g + 8 < G ? *reinterpret_cast<const uint32_t*>(qb + (g + 8) * D + c) : 0u;
-      qf[ks][2] = g < G ? *reinterpret_cast<const uint32_t*>(qb + g * D + c + 8) : 0u;
-      qf[ks][3] = g + 8 < G ? *reinterpret_cast<const uint32_t*>(qb + (g + 8) * D + c + 8) : 0u;
+      qf[ks][0] = g < G ? *reinterpret_cast<const uint32_t*>(qb + g * DQ + c) : 0u;
+      qf[ks][1] = g + 8 < G ? *reinterpret_cast<const uint32_t*>(qb + (g + 8) * DQ + c) : 0u;
+      qf[ks][2] = g < G ? *reinterpret_cast<const uint32_t*>(qb + g * DQ + c + 8) : 0u;
+      qf[ks][3] = g + 8 < G ? *reinterpret_cast<const uint32_t*>(qb + (g + 8) * DQ + c + 8) : 0u;
     }
   }
   const float sscale = a.scale * 1.4426950408889634f;  // scores in the exp2 domain
+  float cap2 = 0.f, capx = 0.f;                        // cap tanh(s) = cap - 2 cap / (1 + 2 ** (2 log2(e) s))
+  if constexpr (kRows) {
+    if (args.softcap > 0.f) cap2 = args.softcap * 1.4426950408889634f, capx = 2.f * sscale / args.softcap;
+  }
   float m0 = -CUDART_INF_F, m1 = -CUDART_INF_F, l0 = 0.f, l1 = 0.f;
-  float acc[D / 8][4];
+  float acc[DV / 8][4];
 #pragma unroll
-  for (int j = 0; j < D / 8; ++j)
+  for (int j = 0; j < DV / 8; ++j)
 #pragma unroll
     for (int e = 0; e < 4; ++e) acc[j][e] = 0.f;
 
@@ -403,8 +449,8 @@ decode_attn_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_c
     if (nvalid < 16) {
       // cache slots past the sequence end hold whatever was there: zero those V rows so that a
       // probability of exactly zero cannot meet a NaN
-      for (int i = lane; i < (16 - nvalid) * kHalves * 8; i += 32) {
-        const int r = nvalid + i / (kHalves * 8), rest = i % (kHalves * 8);
+      for (int i = lane; i < (16 - nvalid) * kVHalves * 8; i += 32) {
+        const int r = nvalid + i / (kVHalves * 8), rest = i % (kVHalves * 8);
         const uint32_t addr = st + (kHalves + rest / 8) * kBox + r * 128 + (rest % 8) * 16;
         asm volatile("st.shared.v4.u32 [%0], {%1, %1, %1, %1};" ::"r"(addr), "r"(0u) : "memory");
       }
@@ -418,7 +464,7 @@ decode_attn_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_c
       for (int e = 0; e < 4; ++e) sc[nt][e] = 0.f;
       const int r = nt * 8 + lr;
 #pragma unroll
-      for (int j = 0; j < D / 32; ++j) {
+      for (int j = 0; j < DQ / 32; ++j) {
         const int cc = 4 * j + lm;  // 16-byte chunk of the row: dims cc * 8 .. + 7
         const uint32_t addr = st + (cc >> 3) * kBox + r * 128 + (((cc & 7) ^ (r & 7)) << 4);
         uint32_t kb[4];
@@ -434,7 +480,11 @@ decode_attn_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_c
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int col = nt * 8 + q4 * 2 + (e & 1);
-        const float v = col < nvalid ? sc[nt][e] * sscale : -CUDART_INF_F;
+        float v = sc[nt][e] * sscale;
+        if constexpr (kRows) {
+          if (args.softcap > 0.f) v = cap2 - 2.f * cap2 * __frcp_rn(1.f + exp2f(sc[nt][e] * capx));
+        }
+        if (col >= nvalid) v = -CUDART_INF_F;
         sc[nt][e] = v;
         if (e < 2) mx0 = fmaxf(mx0, v);
         else mx1 = fmaxf(mx1, v);
@@ -449,7 +499,7 @@ decode_attn_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_c
       l0 *= c0;
       l1 *= c1;
 #pragma unroll
-      for (int j = 0; j < D / 8; ++j) {
+      for (int j = 0; j < DV / 8; ++j) {
         acc[j][0] *= c0;
         acc[j][1] *= c0;
         acc[j][2] *= c1;
@@ -458,7 +508,7 @@ decode_attn_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_c
       m0 = n0;
       m1 = n1;
     }
-    uint32_t pf[4];
+    uint32_t pf[4], pl[4];
     {
       const float p00 = exp2f(sc[0][0] - m0), p01 = exp2f(sc[0][1] - m0), p02 = exp2f(sc[0][2] - m1), p03 = exp2f(sc[0][3] - m1);
       const float p10 = exp2f(sc[1][0] - m0), p11 = exp2f(sc[1][1] - m0), p12 = exp2f(sc[1][2] - m1), p13 = exp2f(sc[1][3] - m1);
@@ -468,10 +518,16 @@ decode_attn_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_c
       pf[1] = pack_bf16(p02, p03);  // (row g + 8, tokens 2 q4 ..)
       pf[2] = pack_bf16(p10, p11);  // (row g,     tokens 8 + 2 q4 ..)
       pf[3] = pack_bf16(p12, p13);  // (row g + 8, tokens 8 + 2 q4 ..)
+      if constexpr (kRows) {
+        pl[0] = pack_rest(p00, p01, pf[0]);
+        pl[1] = pack_rest(p02, p03, pf[1]);
+        pl[2] = pack_rest(p10, p11, pf[2]);
+        pl[3] = pack_rest(p12, p13, pf[3]);
+      }
     }
     // ---- O += P V
 #pragma unroll
-    for (int jp = 0; jp < D / 16; ++jp) {
+    for (int jp = 0; jp < DV / 16; ++jp) {
       const int r = (lm & 1) * 8 + lr;
       const int cc = 2 * jp + (lm >> 1);
       const uint32_t addr = st + (kHalves + (cc >> 3)) * kBox + r * 128 + (((cc & 7) ^ (r & 7)) << 4);
@@ -479,6 +535,10 @@ decode_attn_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_c
       ldsm_x4_trans(addr, vb);
       mma_bf16_16816(acc[2 * jp], pf, vb[0], vb[1]);
       mma_bf16_16816(acc[2 * jp + 1], pf, vb[2], vb[3]);
+      if constexpr (kRows) {
+        mma_bf16_16816(acc[2 * jp], pl, vb[0], vb[1]);
+        mma_bf16_16816(acc[2 * jp + 1], pl, vb[2], vb[3]);
+      }
     }
     __syncwarp();  // every lane has consumed the stage
     const int nxt = it + kTcStages;
@@ -499,12 +559,12 @@ decode_attn_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_c
   l1 += __shfl_xor_sync(0xffffffffu, l1, 1);
   l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
   __syncthreads();  // all warps are done with their rings: reuse the memory for the merge
-  float* red = reinterpret_cast<float*>(smem_dyn + (ring_base - sm100::smem_u32(smem_dyn)));  // [4][16][D + 2]
+  float* red = reinterpret_cast<float*>(smem_dyn + (ring_base - sm100::smem_u32(smem_dyn)));  // [4][16][DV + 2]
   {
-    float* r0 = red + (warp * 16 + g) * (D + 2);
-    float* r1 = red + (warp * 16 + g + 8) * (D + 2);
+    float* r0 = red + (warp * 16 + g) * (DV + 2);
+    float* r1 = red + (warp * 16 + g + 8) * (DV + 2);
 #pragma unroll
-    for (int j = 0; j < D / 8; ++j) {
+    for (int j = 0; j < DV / 8; ++j) {
       const int c = j * 8 + q4 * 2;
       r0[c] = acc[j][0];
       r0[c + 1] = acc[j][1];
@@ -512,47 +572,47 @@ decode_attn_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_c
       r1[c + 1] = acc[j][3];
     }
     if (q4 == 0) {
-      r0[D] = m0;
-      r0[D + 1] = l0;
-      r1[D] = m1;
-      r1[D + 1] = l1;
+      r0[DV] = m0;
+      r0[DV + 1] = l0;
+      r1[DV] = m1;
+      r1[DV + 1] = l1;
     }
   }
   __syncthreads();
-  for (int i = threadIdx.x; i < G * D; i += kDecodeThreads) {
-    const int gg = i / D, d = i % D;
+  for (int i = threadIdx.x; i < G * DV; i += kDecodeThreads) {
+    const int gg = i / DV, d = i % DV;
     float mm = -CUDART_INF_F;
 #pragma unroll
-    for (int w = 0; w < 4; ++w) mm = fmaxf(mm, red[(w * 16 + gg) * (D + 2) + D]);
+    for (int w = 0; w < 4; ++w) mm = fmaxf(mm, red[(w * 16 + gg) * (DV + 2) + DV]);
     float ll = 0.f, av = 0.f;
 #pragma unroll
     for (int w = 0; w < 4; ++w) {
-      const float* rw = red + (w * 16 + gg) * (D + 2);
-      const float c = (rw[D] == -CUDART_INF_F) ? 0.f : exp2f(rw[D] - mm);
-      ll += rw[D + 1] * c;
+      const float* rw = red + (w * 16 + gg) * (DV + 2);
+      const float c = (rw[DV] == -CUDART_INF_F) ? 0.f : exp2f(rw[DV] - mm);
+      ll += rw[DV + 1] * c;
       av += rw[d] * c;
     }
     const int hq = hk * G + gg;
     if (nsplit == 1) {
-      reinterpret_cast<__nv_bfloat16*>(a.out)[(static_cast<size_t>(b) * a.q_heads + hq) * D + d] =
-          __float2bfloat16_rn(ll > 0.f ? av / ll : 0.f);
+      store_out<DV>(args, b, hq, d, ll > 0.f ? av / ll : 0.f);
     } else {
-      float* ws = a.ws + ((static_cast<size_t>(b) * a.q_heads + hq) * nsplit + split) * (D + 2);
+      float* ws = a.ws + ((static_cast<size_t>(b) * a.q_heads + hq) * nsplit + split) * (DV + 2);
       ws[d] = av;
       if (d == 0) {
-        ws[D] = mm;
-        ws[D + 1] = ll;
+        ws[DV] = mm;
+        ws[DV + 1] = ll;
       }
     }
   }
 }
 
-template <int D>
-__global__ void decode_combine_kernel(XpDecodeAttnArgs a, int nsplit) {
+template <int D, typename A>
+__global__ void decode_combine_kernel(A args, int nsplit) {
+  const XpDecodeAttnArgs& a = base_of(args);
   const int hq = blockIdx.x, b = blockIdx.y, d = threadIdx.x;
   const float* ws = a.ws + (static_cast<size_t>(b) * a.q_heads + hq) * nsplit * (D + 2);
   if (a.chunk_tokens > 0) {
-    const int len = a.seq_lens[b];
+    const int len = row_len(args, b);
     nsplit = min(nsplit, (len + a.chunk_tokens - 1) / a.chunk_tokens);  // slices that ran
   }
   float mm = -CUDART_INF_F;
@@ -564,8 +624,7 @@ __global__ void decode_combine_kernel(XpDecodeAttnArgs a, int nsplit) {
     ll += ws[s * (D + 2) + D + 1] * c;
     av += ws[s * (D + 2) + d] * c;
   }
-  reinterpret_cast<__nv_bfloat16*>(a.out)[(static_cast<size_t>(b) * a.q_heads + hq) * D + d] =
-      __float2bfloat16_rn(ll > 0.f ? av / ll : 0.f);
+  store_out<D>(args, b, hq, d, ll > 0.f ? av / ll : 0.f);
 }
 
 template <int D, int GMAX>
@@ -583,23 +642,24 @@ static int launch_decode(const XpDecodeAttnArgs& a, int nsplit, cudaStream_t s) 
   return e == cudaSuccess ? 0 : -100 - static_cast<int>(e);
 }
 
-template <int D>
-static int launch_decode_tc(const XpDecodeAttnArgs& a, int nsplit, cudaStream_t s) {
+template <int DQ, int DV, typename A>
+static int launch_decode_tc(const A& args, int nsplit, cudaStream_t s) {
+  const XpDecodeAttnArgs& a = reinterpret_cast<const XpDecodeAttnArgs&>(args);   // the first member of the wider form
   CUtensorMap mk, mv;
   const uint64_t tokens = static_cast<uint64_t>(a.num_pages) * a.page_size;
-  if (tmap::cache().get_kv(&mk, a.k_cache, tokens, a.kv_heads, D) != 0) return -20;
-  if (tmap::cache().get_kv(&mv, a.v_cache, tokens, a.kv_heads, D) != 0) return -20;
-  constexpr int kStage = 2 * (D / 64) * 16 * 128;
+  if (tmap::cache().get_kv(&mk, a.k_cache, tokens, a.kv_heads, DQ) != 0) return -20;
+  if (tmap::cache().get_kv(&mv, a.v_cache, tokens, a.kv_heads, DV) != 0) return -20;
+  constexpr int kStage = ((DQ + DV) / 64) * 16 * 128;
   constexpr int kSmem = 4 * kTcStages * kStage + 1024;  // rings of four warps + alignment slack
-  static_assert(4 * 16 * (D + 2) * 4 <= 4 * kTcStages * kStage, "merge scratch must fit in the rings");
+  static_assert(4 * 16 * (DV + 2) * 4 <= 4 * kTcStages * kStage, "merge scratch must fit in the rings");
   static bool attr_set = false;
   if (!attr_set) {
-    if (cudaFuncSetAttribute(decode_attn_tc_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem) != cudaSuccess) return -21;
+    if (cudaFuncSetAttribute(decode_attn_tc_kernel<DQ, DV, A>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem) != cudaSuccess) return -21;
     attr_set = true;
   }
   dim3 grid(nsplit, a.kv_heads, a.batch);
-  decode_attn_tc_kernel<D><<<grid, kDecodeThreads, kSmem, s>>>(mk, mv, a);
-  if (nsplit > 1) decode_combine_kernel<D><<<dim3(a.q_heads, a.batch), D, 0, s>>>(a, nsplit);
+  decode_attn_tc_kernel<DQ, DV, A><<<grid, kDecodeThreads, kSmem, s>>>(mk, mv, args);
+  if (nsplit > 1) decode_combine_kernel<DV><<<dim3(a.q_heads, a.batch), DV, 0, s>>>(args, nsplit);
   cudaError_t e = cudaGetLastError();
   return e == cudaSuccess ? 0 : -100 - static_cast<int>(e);
 }
@@ -628,8 +688,8 @@ extern "C" int xp_decode_attn(const XpDecodeAttnArgs* a, void* stream) {
   // tensor-core kernel: 16-token tiles must not straddle pages, slices must start on a tile
   const bool tc_ok = !a->force_simt && a->num_pages > 0 && a->page_size >= 16 && (a->page_size & (a->page_size - 1)) == 0 &&
                      G <= 16 && a->chunk_tokens % 16 == 0 && (reinterpret_cast<uintptr_t>(a->q) & 3) == 0;
-  if (tc_ok && a->head_dim == 128) return launch_decode_tc<128>(*a, nsplit, s);
-  if (tc_ok && a->head_dim == 64) return launch_decode_tc<64>(*a, nsplit, s);
+  if (tc_ok && a->head_dim == 128) return launch_decode_tc<128, 128>(*a, nsplit, s);
+  if (tc_ok && a->head_dim == 64) return launch_decode_tc<64, 64>(*a, nsplit, s);
   if (a->head_dim == 128) {
     if (G <= 2) return launch_decode<128, 2>(*a, nsplit, s);
     if (G <= 4) return launch_decode<128, 4>(*a, nsplit, s);
@@ -640,4 +700,23 @@ extern "C" int xp_decode_attn(const XpDecodeAttnArgs* a, void* stream) {
     if (G <= 8) return launch_decode<64, 8>(*a, nsplit, s);
   }
   return -12;
+}
+
+extern "C" int xp_decode_rows(const XpDecodeRowsArgs* r, void* stream) {
+  using namespace xpool::attn;
+  const XpDecodeAttnArgs* a = &r->a;
+  if (a->batch <= 0) return 0;
+  if (a->kv_heads <= 0 || a->q_heads % a->kv_heads != 0) return -10;
+  const int G = a->q_heads / a->kv_heads;
+  const int nsplit = a->num_splits > 0 ? a->num_splits : 1;
+  if (nsplit > 1 && a->ws == nullptr) return -11;
+  if (G > r->group_pad || G > 16 || a->num_pages <= 0 || a->page_size < 16 || (a->page_size & (a->page_size - 1)) != 0 ||
+      a->chunk_tokens % 16 != 0 || (reinterpret_cast<uintptr_t>(a->q) & 3) != 0 || a->batch > 65535)
+    return -12;
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  if (a->head_dim == 64 && r->v_dim == 64) return launch_decode_tc<64, 64>(*r, nsplit, s);
+  if (a->head_dim == 128 && r->v_dim == 64) return launch_decode_tc<128, 64>(*r, nsplit, s);
+  if (a->head_dim == 128 && r->v_dim == 128) return launch_decode_tc<128, 128>(*r, nsplit, s);
+  if (a->head_dim == 192 && r->v_dim == 128) return launch_decode_tc<192, 128>(*r, nsplit, s);
+  return -13;
 }

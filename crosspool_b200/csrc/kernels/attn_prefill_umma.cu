@@ -21,7 +21,10 @@
 //
 // Keys and values may differ in width (DQ, DV; latent attention in its expanded form: keys are [plain | rotary] columns),
 // their rows may lie densely per sequence instead of in pages, every head's output may be gated by a sigmoid, and the
-// probabilities may enter the second product as a bf16 pair (high and low part: two products, 16 mantissa bits).
+// probabilities may enter the second product as a bf16 pair (high and low part: two products, 16 mantissa bits). Groups whose
+// number of query heads is no power of two come padded (their padding is computed and not stored). Scores may be capped,
+// cap tanh(s / cap): in a tile whose scores are all far below the cap by a polynomial on the FMA pipe, otherwise through
+// 2 ** x and a reciprocal.
 //
 // V is used where it lands (token-major rows of 64 dims) through an MN-major operand descriptor; no transpose.
 // Tensor memory: S buffers 4 x 64 columns, O 2 x D columns (512 columns with D = 128).
@@ -84,7 +87,46 @@ __device__ __forceinline__ uint32_t pack2(float lo, float hi) {
   return *reinterpret_cast<uint32_t*>(&v);
 }
 
-template <int DQ, int DV, bool kTS, bool kPair>
+// tanh(x) / x as a polynomial in x^2, for x^2 up to kTanhRange (interpolated at Chebyshev nodes; relative error 2e-8)
+constexpr float kTanhRange = 0.49f;
+__device__ __forceinline__ float tanh_poly(float t, const float (&c)[6]) {
+  return fmaf(fmaf(fmaf(fmaf(fmaf(c[5], t, c[4]), t, c[3]), t, c[2]), t, c[1]), t, c[0]);
+}
+
+// Scores of one row (raw products) -> cap tanh(s scale / cap) in log2 units.
+__device__ __forceinline__ void cap_scores(uint32_t (&sv)[kBN], float scale, float cap) {
+  const float x = scale / cap, x2 = x * x;
+  float mx[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+  for (int j = 0; j < kBN; j += 8) {
+#pragma unroll
+    for (int c = 0; c < 4; ++c)
+      mx[c] = max3(mx[c], fabsf(__uint_as_float(sv[j + 2 * c])), fabsf(__uint_as_float(sv[j + 2 * c + 1])));
+  }
+  const float m = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3]));
+  if (__all_sync(0xffffffffu, m * m * x2 <= kTanhRange)) {
+    // coefficients for the raw product's square; the factor that makes the result scale log2(e) s is in all of them
+    float c[6] = {1.0f, -0.3333313465118408f, 0.1332847625017166f, -0.05352945625782013f, 0.020032446831464767f, -0.005094828084111214f};
+    float f = scale * 1.4426950408889634f;
+#pragma unroll
+    for (int i = 0; i < 6; ++i) c[i] *= f, f *= x2;
+#pragma unroll
+    for (int j = 0; j < kBN; ++j) {
+      const float v = __uint_as_float(sv[j]);
+      sv[j] = __float_as_uint(v * tanh_poly(v * v, c));
+    }
+  } else {
+    const float cl = cap * 1.4426950408889634f, e = 2.f * x * 1.4426950408889634f;
+#pragma unroll
+    for (int j = 0; j < kBN; ++j) {
+      float r;
+      asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.f + sm100::ex2_approx(__uint_as_float(sv[j]) * e)));
+      sv[j] = __float_as_uint(fmaf(-2.f * cl, r, cl));
+    }
+  }
+}
+
+template <int DQ, int DV, bool kTS, bool kPair, bool kCap>
 __global__ void __launch_bounds__(kThreads, 1)
 prefill_attn_umma_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
                          const __grid_constant__ CUtensorMap tmap_v, const __grid_constant__ CUtensorMap tmap_k3,
@@ -274,14 +316,16 @@ prefill_attn_umma_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gri
     const int x = warp >> 2;                          // tile
     const int row = (warp & 3) * 32 + lane;           // row of the tile = TMEM lane
     const int pos = q0 + x * np + (row >> g_shift);   // query position inside the chunk
-    const int hq = hk * G + (row & (G - 1));
+    const int heads = a.group_valid;                  // query heads of the group; the rest of G is padding
+    const int hq = hk * heads + (row & (G - 1));
+    const bool stored = pos < q_len && (row & (G - 1)) < heads;
     const bool tile_on = x == 0 || act_b;
     const int my_tiles = x == 0 ? n_a : n_tiles;
     const int limit = min(ctx + pos, kv_end - 1);     // last visible cache position of this row
     const uint32_t lane_off = static_cast<uint32_t>((warp & 3) * 32) << 16;
     const uint32_t o_t = tmem + lane_off + kOCol + static_cast<uint32_t>(x * DV);
     const uint32_t p_row = p_s + x * kPTile + row * 128;
-    const float sc2 = a.scale * 1.4426950408889634f;
+    const float sc2 = kCap ? 1.f : a.scale * 1.4426950408889634f;
     float m_used = -CUDART_INF_F, l = 0.f;
     bool ok = true;
     if (tile_on) {
@@ -302,6 +346,7 @@ prefill_attn_umma_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gri
           if (lane == 0) sm100::mbar_arrive(&bars.s_empty[x][bf]);
         }
 
+        if constexpr (kCap) cap_scores(sv, a.scale, a.softcap);
         const int nvis = min(kBN, max(0, limit - t * kBN + 1));   // visible tokens of this tile for this row
         if (nvis < kBN) {
 #pragma unroll
@@ -403,7 +448,7 @@ prefill_attn_umma_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gri
       if (ok) {
         sm100::tc_fence_after_sync();
         float inv = l > 0.f ? 1.f / l : 0.f;
-        if (a.gate != nullptr && pos < q_len)
+        if (a.gate != nullptr && stored)
           inv *= 1.f / (1.f + expf(-__bfloat162float(reinterpret_cast<const __nv_bfloat16*>(a.gate)[static_cast<size_t>(q_base + pos) * a.ld_gate + hq])));
         const int v_valid = a.v_valid;                    // stored columns of a head (a multiple of 8)
         __nv_bfloat16* og = reinterpret_cast<__nv_bfloat16*>(a.out) + static_cast<size_t>(q_base + pos) * a.ld_out + hq * v_valid;
@@ -412,7 +457,7 @@ prefill_attn_umma_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gri
           uint32_t ov[32];
           sm100::tmem_ld32_issue(o_t + c, ov);
           sm100::tmem_ld_wait_all(ov);
-          if (pos < q_len) {
+          if (stored) {
 #pragma unroll
             for (int j = 0; j < 32; j += 8) {
               if (c + j >= v_valid) break;
@@ -446,7 +491,7 @@ prefill_attn_umma_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gri
   }
 }
 
-template <int DQ, int DV, bool kTS, bool kPair>
+template <int DQ, int DV, bool kTS, bool kPair, bool kCap = false>
 static int launch(const XpPrefillAttnArgs& a, int G, cudaStream_t s) {
   CUtensorMap mq, mk, mv, mk3, mv3;
   const uint64_t tokens = static_cast<uint64_t>(a.num_pages) * a.page_size;
@@ -467,17 +512,23 @@ static int launch(const XpPrefillAttnArgs& a, int G, cudaStream_t s) {
   static_assert(kSmem <= 227 * 1024, "tiles exceed the shared memory of an SM");
   static bool attr_set = false;
   if (!attr_set) {
-    if (cudaFuncSetAttribute(prefill_attn_umma_kernel<DQ, DV, kTS, kPair>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem) != cudaSuccess)
+    if (cudaFuncSetAttribute(prefill_attn_umma_kernel<DQ, DV, kTS, kPair, kCap>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem) != cudaSuccess)
       return -21;
     attr_set = true;
   }
   XpPrefillAttnArgs b = a;
   if (b.v_valid <= 0) b.v_valid = DV;
   if (b.ld_out <= 0) b.ld_out = b.q_heads * b.v_valid;
+  if (b.group_valid <= 0) b.group_valid = G;
   dim3 grid(b.kv_heads, b.num_seqs, (b.max_q_len + 2 * np - 1) / (2 * np));
-  prefill_attn_umma_kernel<DQ, DV, kTS, kPair><<<grid, kThreads, kSmem, s>>>(mq, mk, mv, mk3, mv3, b, G, g_shift, box_tokens);
+  prefill_attn_umma_kernel<DQ, DV, kTS, kPair, kCap><<<grid, kThreads, kSmem, s>>>(mq, mk, mv, mk3, mv3, b, G, g_shift, box_tokens);
   cudaError_t e = cudaGetLastError();
   return e == cudaSuccess ? 0 : -100 - static_cast<int>(e);
+}
+
+template <int DQ, int DV>
+static int launch_pair(const XpPrefillAttnArgs& a, int G, cudaStream_t s) {
+  return a.softcap > 0.f ? launch<DQ, DV, true, true, true>(a, G, s) : launch<DQ, DV, true, true>(a, G, s);
 }
 
 }  // namespace attn5
@@ -500,13 +551,13 @@ extern "C" int xp_prefill_attn_umma(const XpPrefillAttnArgs* a, void* stream) {
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   const int dv = a->v_dim > 0 ? a->v_dim : a->head_dim;
   if (a->p_pair) {
-    if (a->head_dim == 64 && dv == 64) return launch<64, 64, true, true>(*a, G, s);
-    if (a->head_dim == 128 && dv == 64) return launch<128, 64, true, true>(*a, G, s);
-    if (a->head_dim == 128 && dv == 128) return launch<128, 128, true, true>(*a, G, s);
-    if (a->head_dim == 192 && dv == 128) return launch<192, 128, true, true>(*a, G, s);
+    if (a->head_dim == 64 && dv == 64) return launch_pair<64, 64>(*a, G, s);
+    if (a->head_dim == 128 && dv == 64) return launch_pair<128, 64>(*a, G, s);
+    if (a->head_dim == 128 && dv == 128) return launch_pair<128, 128>(*a, G, s);
+    if (a->head_dim == 192 && dv == 128) return launch_pair<192, 128>(*a, G, s);
     return 1;
   }
-  if (dv != a->head_dim) return 1;
+  if (dv != a->head_dim || a->softcap > 0.f) return 1;
   if (a->head_dim == 128) return ts ? launch<128, 128, true, false>(*a, G, s) : launch<128, 128, false, false>(*a, G, s);
   if (a->head_dim == 64) return ts ? launch<64, 64, true, false>(*a, G, s) : launch<64, 64, false, false>(*a, G, s);
   return 1;

@@ -612,6 +612,10 @@ extern "C" int xp_delta_prep(const XpDeltaArgs* a, void* stream) {
 extern "C" int xp_delta_prefill(const XpDeltaArgs* a, void* stream) {
   if (a->seqs <= 0) return 0;
   if (!delta_ok(*a)) return -10;
+  if (!a->force_sequential) {
+    const int rc = xp_delta_chunked(a, stream);
+    if (rc <= 0) return rc;
+  }
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   return a->f32 ? sequential_any<float, true>(*a, s) : sequential_any<__nv_bfloat16, true>(*a, s);
 }
@@ -619,6 +623,10 @@ extern "C" int xp_delta_prefill(const XpDeltaArgs* a, void* stream) {
 extern "C" int xp_gated_linear_prefill(const XpGatedLinearArgs* a, void* stream) {
   if (a->seqs <= 0) return 0;
   if (a->heads <= 0 || a->dim <= 0 || a->vdim <= 0) return -10;
+  if (!a->force_sequential) {
+    const int rc = xp_gated_linear_chunked(a, stream);
+    if (rc <= 0) return rc;
+  }
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   return a->f32 ? sequential_any<float, false>(*a, s) : sequential_any<__nv_bfloat16, false>(*a, s);
 }

@@ -27,6 +27,7 @@ from ..models.config import (DeltaMixer, GatedLinearMixer, GroupedMixer, LatentM
 from ..models.layered import LayeredLayerWeights
 from ..ops import gemm
 from ..ops import mixers as M
+from ..ops.attention import decode_plan
 
 # Portions of at most this many tokens run as single rows (latent attention: in the absorbed form, expanding the whole context
 # costs more).
@@ -113,11 +114,18 @@ class LayeredForward:
             self.v_exp = buf(self.ws_tokens * max(H * dv for H, _, dv, _ in shapes))
         if grp:
             self.q_grp = buf(cap * max(m.kv_heads * M.group_pad(m.heads, m.kv_heads) * m.cache_rows[0][1] for m in grp))
+            need = max(b * m.heads * decode_plan(b, m.kv_heads, engine.ecfg.max_seq_len)[0] * (m.cache_rows[1][1] + 2)
+                       for b in engine._buckets for m in grp)
+            self.grp_ws = buf(max(need, 1 << 20), torch.float32)
         if gla:
             self.z = buf(cap * max(m.heads * m.dim for m in gla), torch.float32)
+            self.gla_ws = None
+            if dt == torch.bfloat16:
+                self.gla_ws = M.GatedLinearScratch.for_rows(cap, engine.max_seqs, max(m.heads for m in gla), max(m.dim for m in gla),
+                                                            max(m.vdim for m in gla), dev)
         if delta:
-            self.delta_ws = M.DeltaScratch(buf(cap * max(m.conv_channels for m in delta)), buf(cap * max(2 * m.kv_heads for m in delta), torch.float32),
-                                           buf(cap * max(2 * m.heads for m in delta), torch.float32))
+            self.delta_ws = M.DeltaScratch.for_rows(cap, engine.max_seqs, max(m.heads for m in delta), max(m.kv_heads for m in delta),
+                                                    max(m.dim for m in delta), max(m.vdim for m in delta), dt, dev)
         if lin or gla or delta:
             self.o_lin = buf(cap * max(m.out_features for m in lin + gla + delta), torch.float32)
         if lin:
@@ -178,7 +186,8 @@ class LayeredForward:
     def _tiled(self, m: GroupedMixer) -> bool:
         """Whether the tensor-core attention kernels cover the mixer."""
         shape, page = attention_shape(m.dim, m.vdim), self.e.ecfg.page_size
-        return False
+        return (self.dtype == torch.bfloat16 and shape is not None and m.heads // m.kv_heads <= 16 and page & (page - 1) == 0
+                and page >= (16 if shape[0] == shape[1] else 64))
 
     def _grouped(self, l: int, lw: LayeredLayerWeights, m: GroupedMixer, proj: torch.Tensor, out: torch.Tensor, b: RowBatch) -> None:
         rows, o, kv = b.rows, lw.offs, self.e.kv
@@ -188,8 +197,20 @@ class LayeredForward:
         M.grouped_prep(proj, lw.mix["q_norm"], lw.mix["k_norm"], b.slots, k, v, q, heads=m.heads, dim=m.dim, vdim=m.vdim,
                        offs=(o["q"], o["k"], o["v"]), eps=self.e.cfg.rms_norm_eps)
         gate = proj[:, o["hg"]:o["hg"] + m.heads]
-        M.grouped_attn(q, k, v, out, b.table, b.positions, b.slots, heads=m.heads, dim=m.dim, vdim=m.vdim, scale=m.scale,
-                       softcap=m.softcap, gate=gate, row_seq=b.row_seq)
+        kw = dict(heads=m.heads, vdim=m.vdim, scale=m.scale, softcap=m.softcap)
+        if not self._tiled(m):
+            M.grouped_attn(q, k, v, out, b.table, b.positions, b.slots, dim=m.dim, gate=gate, row_seq=b.row_seq, **kw)
+            return
+        n = b.n_abs
+        if n:
+            splits, chunk = decode_plan(n, m.kv_heads, b.max_len)
+            if splits > 1 and n * m.heads * splits * (v.shape[3] + 2) > self.grp_ws.numel():
+                splits, chunk = 1, 0
+            M.grouped_decode(q[:n], k, v, out[:n], b.table, b.positions, b.slots, dim=m.dim, gate=gate, row_seq=b.row_seq, num_splits=splits,
+                             chunk_tokens=chunk, ws=self.grp_ws, **kw)
+        if n < rows:
+            s = slice(b.n_short, b.n_seqs)
+            M.grouped_prefill(q, k, v, out, b.table[s], b.q_starts[s], b.q_lens[s], b.ctx_lens[s], b.max_q, gate=gate, **kw)
 
     def _gated_linear(self, l: int, lw: LayeredLayerWeights, m: GatedLinearMixer, proj: torch.Tensor, out: torch.Tensor, b: RowBatch) -> None:
         o, w, n, nd, eps = lw.offs, lw.mix, m.out_features, b.n_dec, self.e.cfg.rms_norm_eps
@@ -204,7 +225,9 @@ class LayeredForward:
             z = self.z[:b.rows * m.heads * m.dim].view(b.rows, m.heads * m.dim)
             gemm.linear(proj[nd:, o["lin_a"]:o["lin_a"] + w["a2"].shape[1]], w["a2"], out=z[nd:], bias=w["a2_bias"])
             y = self.o_lin[:b.rows * n].view(b.rows, n)
-            M.gated_linear_prefill(proj, z, state, y, b.positions, b.slots, b.state_slots[s], b.q_starts[s], b.q_lens[s], offs=qkv, **kw)
+            segs, seg_tokens = M.gated_linear_plan(b.n_seqs - nd, m.heads, m.vdim, b.max_q)
+            M.gated_linear_prefill(proj, z, state, y, b.positions, b.slots, b.state_slots[s], b.q_starts[s], b.q_lens[s], b.max_q, self.gla_ws,
+                                   offs=qkv, segs=segs, seg_tokens=seg_tokens, **kw)
             M.head_gate(y[nd:], w["norm"], proj[nd:, o["lin_g"]:o["lin_g"] + n], eps, out[nd:])
 
     def _delta(self, l: int, lw: LayeredLayerWeights, m: DeltaMixer, proj: torch.Tensor, out: torch.Tensor, b: RowBatch) -> None:

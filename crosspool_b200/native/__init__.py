@@ -221,6 +221,22 @@ class DecodeAttnArgs(C.Structure):
     ]
 
 
+class DecodeRowsArgs(C.Structure):
+    _fields_ = [
+        ("a", DecodeAttnArgs),
+        ("row_seq", C.c_void_p),
+        ("positions", C.c_void_p),
+        ("slots", C.c_void_p),
+        ("gate", C.c_void_p),
+        ("group_pad", C.c_int),
+        ("v_dim", C.c_int),
+        ("v_valid", C.c_int),
+        ("ld_out", C.c_int),
+        ("ld_gate", C.c_int),
+        ("softcap", C.c_float),
+    ]
+
+
 class PrefillAttnArgs(C.Structure):
     _fields_ = [
         ("q", C.c_void_p),
@@ -250,6 +266,8 @@ class PrefillAttnArgs(C.Structure):
         ("gate", C.c_void_p),
         ("ld_gate", C.c_int),
         ("p_pair", C.c_int),
+        ("group_valid", C.c_int),
+        ("softcap", C.c_float),
     ]
 
 
@@ -279,8 +297,8 @@ GroupedAttnArgs = _struct("GroupedAttnArgs", "XpGroupedAttnArgs", a_ptr="q k_cac
                           b_int="rows heads kv_heads group_pad dim vdim dq dv ld_gate ld_out page_size max_blocks", c_float="scale softcap",
                           d_int="f32")
 GatedLinearArgs = _struct("GatedLinearArgs", "XpGatedLinearArgs",
-                          a_ptr="proj z a2 a2_bias norm state out positions slots state_slots q_starts q_lens ws",
-                          b_int="rows seqs heads dim vdim ld_proj ld_out q_off k_off v_off g_off a_off rank ld_a2 segs seg_tokens force_sequential",
+                          a_ptr="proj z a2 a2_bias norm state out positions slots state_slots q_starts q_lens ws records",
+                          b_int="rows seqs max_q heads dim vdim ld_proj ld_out q_off k_off v_off g_off a_off rank ld_a2 segs seg_tokens force_sequential",
                           c_float="inv_tau qscale eps", d_int="f32")
 DeltaArgs = _struct("DeltaArgs", "XpDeltaArgs",
                     a_ptr="proj conv_w conv_state neg_a dt_bias norm state out qkv qk_scale beta_g ws positions slots state_slots q_starts q_lens",
@@ -309,6 +327,9 @@ def _declare_mixers(lib: C.CDLL) -> None:
                      ("xp_delta_decode", DeltaArgs), ("xp_delta_prep", DeltaArgs), ("xp_delta_prefill", DeltaArgs)):
         getattr(lib, fn).restype = C.c_int
         getattr(lib, fn).argtypes = [C.POINTER(args), C.c_void_p]
+    for fn in ("xp_delta_ws_bytes", "xp_gated_linear_record_bytes"):
+        getattr(lib, fn).restype = C.c_size_t
+        getattr(lib, fn).argtypes = [C.c_int] * 3
     lib.xp_gemm_f32.restype = C.c_int
     lib.xp_gemm_f32.argtypes = [C.c_void_p] * 4 + [C.c_int] * 7 + [C.c_int64] * 3 + [C.c_float, C.c_int, C.c_void_p]
 
@@ -319,6 +340,8 @@ def _declare_attention(lib: C.CDLL) -> None:
         getattr(lib, fn).restype = C.c_int
     lib.xp_rope_kv.argtypes = [C.POINTER(RopeArgs), C.c_void_p]
     lib.xp_decode_attn.argtypes = [C.POINTER(DecodeAttnArgs), C.c_void_p]
+    lib.xp_decode_rows.restype = C.c_int
+    lib.xp_decode_rows.argtypes = [C.POINTER(DecodeRowsArgs), C.c_void_p]
     lib.xp_prefill_attn.argtypes = [C.POINTER(PrefillAttnArgs), C.c_void_p]
     lib.xp_decode_attn_splits.argtypes = [C.c_int, C.c_int, C.c_int]
     lib.xp_embedding.argtypes = [C.c_void_p, C.c_void_p, C.c_void_p, C.c_int, C.c_int, C.c_int, C.c_void_p]

@@ -349,6 +349,48 @@ def grouped_attn(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, 
     return out
 
 
+def grouped_decode(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, out: torch.Tensor, block_table: torch.Tensor,
+                   positions: torch.Tensor, slots: torch.Tensor, *, heads: int, dim: int, vdim: int, scale: float, softcap: float = 0.0,
+                   gate: torch.Tensor | None = None, row_seq: torch.Tensor | None = None, num_splits: int = 1, chunk_tokens: int = 0,
+                   ws: torch.Tensor | None = None) -> torch.Tensor:
+    """:func:`grouped_attn` on the tensor cores (bf16, widths of ``ATTENTION_SHAPES``, at most 16 query heads per key head).
+    ``ws``: fp32, ``rows * heads * num_splits * (dv + 2)`` elements when ``num_splits`` > 1."""
+    from .gemm import status_words
+
+    r = native.DecodeRowsArgs()
+    a = r.a
+    a.q, a.k_cache, a.v_cache, a.out, a.ws = q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), out.data_ptr(), _ptr(ws)
+    assert q.dtype == out.dtype == torch.bfloat16 and (num_splits == 1 or ws.numel() >= q.shape[0] * heads * num_splits * (v_cache.shape[3] + 2))
+    a.block_table, a.batch, a.q_heads, a.kv_heads, a.head_dim = block_table.data_ptr(), q.shape[0], heads, q.shape[1], q.shape[3]
+    a.page_size, a.max_blocks, a.num_splits, a.chunk_tokens, a.num_pages = k_cache.shape[1], block_table.stride(0), num_splits, chunk_tokens, k_cache.shape[0]
+    a.scale, a.status = scale, status_words(q.device).data_ptr()
+    r.row_seq, r.positions, r.slots, r.gate = _ptr(row_seq), positions.data_ptr(), slots.data_ptr(), _ptr(gate)
+    r.group_pad, r.v_dim, r.v_valid, r.ld_out, r.softcap = q.shape[2], v_cache.shape[3], vdim, out.stride(0), softcap
+    r.ld_gate = gate.stride(0) if gate is not None else 0
+    native.check(native.kernels().xp_decode_rows(C.byref(r), _stream(q)), "xp_decode_rows", 2 if num_splits > 1 else 1)
+    return out
+
+
+def grouped_prefill(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, out: torch.Tensor, block_table: torch.Tensor,
+                    q_starts: torch.Tensor, q_lens: torch.Tensor, ctx_lens: torch.Tensor, max_q: int, *, heads: int, vdim: int, scale: float,
+                    softcap: float = 0.0, gate: torch.Tensor | None = None) -> torch.Tensor:
+    """Causal attention of portions (rows of ``q`` ``[rows, kv_heads, group_pad, dq]``) over the paged cache, which holds the
+    portions' own tokens already, on tcgen05; ``out`` ``[rows, heads * vdim]``."""
+    from .gemm import status_words
+
+    a = native.PrefillAttnArgs()
+    a.q, a.k_cache, a.v_cache, a.out, a.block_table = (t.data_ptr() for t in (q, k_cache, v_cache, out, block_table))
+    a.q_starts, a.q_lens, a.ctx_lens = q_starts.data_ptr(), q_lens.data_ptr(), ctx_lens.data_ptr()
+    a.num_seqs, a.max_q_len, a.kv_heads, a.q_heads = q_lens.shape[0], max_q, q.shape[1], q.shape[1] * q.shape[2]
+    a.head_dim, a.v_dim, a.v_valid, a.ld_out = q.shape[3], v_cache.shape[3], vdim, out.stride(0)
+    a.page_size, a.max_blocks, a.num_pages = k_cache.shape[1], block_table.stride(0), k_cache.shape[0]
+    a.scale, a.total_q, a.p_pair, a.group_valid, a.softcap = scale, q.shape[0], 1, heads // q.shape[1], softcap
+    a.gate, a.ld_gate = _ptr(gate), gate.stride(0) if gate is not None else 0
+    a.status = status_words(q.device).data_ptr()
+    native.check(native.kernels().xp_prefill_attn_umma(C.byref(a), _stream(q)), "xp_prefill_attn_umma")
+    return out
+
+
 # ------------------------------------------------------------------------------------------ input-dependent recurrences
 
 def _recurrent(a, proj, state, out, positions, slots, state_slots, heads, dim, vdim):
@@ -370,16 +412,54 @@ def gated_linear_decode(proj, state, a2, a2_bias, norm, out, positions, slots, s
     native.check(native.kernels().xp_gated_linear_decode(C.byref(a), _stream(proj)), "xp_gated_linear_decode")
 
 
-def gated_linear_prefill(proj, z, state, out, positions, slots, state_slots, q_starts, q_lens, *, heads: int, dim: int, vdim: int,
-                         offs: tuple[int, int, int], tau: float, force_sequential: bool = False) -> None:
-    """Portions of sequences: portion i covers rows ``q_starts[i] .. + q_lens[i]`` and continues state ``state_slots[i]``;
-    ``z`` fp32 ``[rows, heads * dim]`` is the decay map's value, ``out`` fp32 ``[rows, heads * vdim]``."""
+def gated_linear_plan(seqs: int, heads: int, vdim: int, max_q: int) -> tuple[int, int]:
+    """(segments, tokens per segment) of the chunked prefill: enough CTAs for the 148 SMs when sequences and heads are few. A
+    segmented run walks the chunks twice, the first time without outputs."""
+    slices = (vdim + 63) // 64
+    ctas, chunks = seqs * heads * slices, (max_q + LINEAR_CHUNK - 1) // LINEAR_CHUNK
+    best, best_cost = 1, None
+    for s in range(1, min(chunks, 64) + 1):
+        per = (chunks + s - 1) // s
+        if s > 1 and (ctas * s > 2 * 148 or (s - 1) * per >= chunks):
+            continue
+        cost = ((ctas * s + 147) // 148) * per * (1.0 if s == 1 else 1.6) + (0 if s == 1 else 4)
+        if best_cost is None or cost < best_cost:
+            best, best_cost = s, cost
+    return best, (chunks + best - 1) // best * LINEAR_CHUNK
+
+
+@dataclass
+class GatedLinearScratch:
+    """What the chunked prefill kernels hand on: scores of every (chunk, head), states and decays between segments."""
+
+    records: torch.Tensor
+    ws: torch.Tensor
+
+    @classmethod
+    def for_rows(cls, rows: int, seqs: int, heads: int, dim: int, vdim: int, device) -> "GatedLinearScratch":
+        """For batches of at most ``rows`` rows in ``seqs`` portions; any plan of :func:`gated_linear_plan` fits."""
+        n = native.kernels().xp_gated_linear_record_bytes(rows, seqs, heads)
+        return cls(torch.zeros(n, dtype=torch.uint8, device=device), torch.zeros(2 * 148 * dim * (vdim + 1), dtype=torch.float32, device=device))
+
+
+def gated_linear_prefill(proj, z, state, out, positions, slots, state_slots, q_starts, q_lens, max_q: int, scratch: GatedLinearScratch | None,
+                         *, heads: int, dim: int, vdim: int, offs: tuple[int, int, int], tau: float, segs: int = 1, seg_tokens: int = 0,
+                         force_sequential: bool = False) -> None:
+    """Portions of sequences (the longest has ``max_q`` rows): portion i covers rows ``q_starts[i] .. + q_lens[i]`` and
+    continues state ``state_slots[i]``; ``z`` fp32 ``[rows, heads * dim]`` is the decay map's value and is used up, ``out`` fp32
+    ``[rows, heads * vdim]``. ``segs`` and ``seg_tokens`` as planned. bf16 rows with widths in multiples of 8 and at most 128
+    key dimensions run the chunked tensor-core kernels when there is ``scratch``, everything else the sequential kernel."""
     a = _recurrent(native.GatedLinearArgs(), proj, state, out, positions, slots, state_slots, heads, dim, vdim)
     assert z.dtype == out.dtype == torch.float32 and z.is_contiguous()
-    a.z, a.q_starts, a.q_lens, a.seqs = z.data_ptr(), q_starts.data_ptr(), q_lens.data_ptr(), q_lens.shape[0]
+    a.z, a.q_starts, a.q_lens, a.seqs, a.max_q = z.data_ptr(), q_starts.data_ptr(), q_lens.data_ptr(), q_lens.shape[0], max_q
     a.q_off, a.k_off, a.v_off = offs
     a.inv_tau, a.qscale, a.force_sequential = 1.0 / tau, dim ** -0.5, int(force_sequential)
-    native.check(native.kernels().xp_gated_linear_prefill(C.byref(a), _stream(proj)), "xp_gated_linear_prefill")
+    n = 1
+    if scratch is not None:
+        a.records, a.segs, a.seg_tokens, a.ws = scratch.records.data_ptr(), segs, seg_tokens, scratch.ws.data_ptr()
+        assert segs <= 1 or scratch.ws.numel() >= q_lens.shape[0] * heads * segs * dim * (vdim + 1)
+        n = 4 if segs > 1 else 2
+    native.check(native.kernels().xp_gated_linear_prefill(C.byref(a), _stream(proj)), "xp_gated_linear_prefill", n)
 
 
 @dataclass
@@ -395,11 +475,23 @@ class DeltaWeights:
 
 @dataclass
 class DeltaScratch:
-    """What the prefill kernels hand on: convolved rows, unit-vector factors, ``beta`` and ``log g``."""
+    """What the prefill kernels hand on: convolved rows, unit-vector factors, ``beta`` and ``log g``, and the solved systems
+    of every (chunk, head)."""
 
     qkv: torch.Tensor
     qk_scale: torch.Tensor
     beta_g: torch.Tensor
+    ws: torch.Tensor | None = None
+
+    @classmethod
+    def for_rows(cls, rows: int, seqs: int, heads: int, kv_heads: int, dim: int, vdim: int, dtype: torch.dtype, device) -> "DeltaScratch":
+        """For batches of at most ``rows`` rows in ``seqs`` portions."""
+        def buf(n, dt):
+            return torch.zeros(n, dtype=dt, device=device)
+
+        ws = buf(native.kernels().xp_delta_ws_bytes(rows, seqs, heads), torch.uint8) if dtype == torch.bfloat16 else None
+        return cls(buf(rows * (2 * kv_heads * dim + heads * vdim), dtype), buf(rows * 2 * kv_heads, torch.float32),
+                   buf(rows * 2 * heads, torch.float32), ws)
 
 
 def _delta(proj, conv_state, w: DeltaWeights, state, out, positions, slots, state_slots, heads, kv_heads, dim, vdim, offs, eps):
@@ -423,11 +515,13 @@ def delta_decode(proj, conv_state, w: DeltaWeights, state, out, positions, slots
 def delta_prefill(proj, conv_state, w: DeltaWeights, state, out, positions, slots, state_slots, q_starts, q_lens, max_q: int,
                   scratch: DeltaScratch, *, heads: int, kv_heads: int, dim: int, vdim: int, offs: tuple[int, int, int, int, int, int],
                   eps: float, force_sequential: bool = False) -> None:
-    """Portions of sequences (the longest has ``max_q`` rows): convolution and recurrence; ``out`` fp32 ``[rows, heads * vdim]``."""
+    """Portions of sequences (the longest has ``max_q`` rows): convolution and recurrence; ``out`` fp32 ``[rows, heads * vdim]``.
+    bf16 rows with widths in multiples of 8 and at most 128 key dimensions run the chunked tensor-core kernels."""
     a = _delta(proj, conv_state, w, state, out, positions, slots, state_slots, heads, kv_heads, dim, vdim, offs, eps)
     assert out.dtype == torch.float32 and scratch.qkv.dtype == proj.dtype
     a.qkv, a.qk_scale, a.beta_g = scratch.qkv.data_ptr(), scratch.qk_scale.data_ptr(), scratch.beta_g.data_ptr()
+    a.ws = _ptr(scratch.ws)
     a.q_starts, a.q_lens, a.seqs, a.max_q, a.force_sequential = q_starts.data_ptr(), q_lens.data_ptr(), q_lens.shape[0], max_q, int(force_sequential)
     lib = native.kernels()
     native.check(lib.xp_delta_prep(C.byref(a), _stream(proj)), "xp_delta_prep")
-    native.check(lib.xp_delta_prefill(C.byref(a), _stream(proj)), "xp_delta_prefill")
+    native.check(lib.xp_delta_prefill(C.byref(a), _stream(proj)), "xp_delta_prefill", 1 if scratch.ws is None else 2)

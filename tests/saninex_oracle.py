@@ -152,7 +152,9 @@ def forward(config, tensors, ids, dtype=torch.float64, layer_outputs=None):
 
 
 def random_tensors(config, seed, rank=12):
-    """Random bf16 tensors under the checkpoint's names, sized so that every term matters; ``rank``: of the decay map."""
+    """Random bf16 tensors under the checkpoint's names, sized so that every term matters; ``rank``: of the decay map.
+    Recurrent queries resemble their keys: a first token reads (q . k) v, which is normed, so that its sign would be a matter of
+    rounding where q and k happen to be orthogonal."""
     g = torch.Generator().manual_seed(seed)
     W = config["width"]
 
@@ -161,6 +163,9 @@ def random_tensors(config, seed, rank=12):
 
     def vec(n, mean=0.0, std=0.3):
         return (mean + std * torch.randn(n, generator=g)).bfloat16()
+
+    def alike(w):
+        return (0.8 * w.float() + 0.6 * torch.randn(w.shape, generator=g) * w.float().std()).bfloat16()
 
     t = {"embed": torch.randn(config["vocab"], W, generator=g).bfloat16()}
     for i, layer in enumerate(config["layers"]):
@@ -171,6 +176,7 @@ def random_tensors(config, seed, rank=12):
             q = p + ".mix."
             for n, rows in (("q", G * d), ("k", G * d), ("v", H * e)):
                 t[q + n], t[q + n + ".conv"] = lin(rows, W), lin(rows, c, 1.2)
+            t[q + "k"], t[q + "k.conv"] = alike(t[q + "q"]), alike(t[q + "q.conv"])
             t[q + "b"], t[q + "a"], t[q + "g"], t[q + "o"] = lin(H, W), lin(H, W), lin(H * e, W), lin(W, H * e)
             t[q + "A_log"], t[q + "dt_bias"], t[q + "norm"] = vec(H, -1.0, 1.5), vec(H, -1.0, 1.0), vec(e, 1.0)
         else:
@@ -182,7 +188,8 @@ def random_tensors(config, seed, rank=12):
             t[q + "q.norm"], t[q + "k.norm"], t[q + "g"] = vec(d, 1.3), vec(d, 1.3), lin(H, W)
             r, q = m["right"], p + ".mix.right."
             H, d, e = r["heads"], r["dim"], r["vdim"]
-            t[q + "q"], t[q + "k"], t[q + "v"] = lin(H * d, W), lin(H * d, W), lin(H * e, W)
+            t[q + "q"], t[q + "v"] = lin(H * d, W), lin(H * e, W)
+            t[q + "k"] = alike(t[q + "q"])
             t[q + "g"], t[q + "o"], t[q + "norm"] = lin(H * e, W), lin(W, H * e), vec(e, 1.0)
             t[q + "a1"], t[q + "a2"], t[q + "a2.b"] = lin(rank, W), lin(H * d, rank, 1.5), vec(H * d, 1.0, 1.5)
             t[p + ".mix.left.out"], t[p + ".mix.right.out"] = vec(W, 1.0), vec(W, 1.0)
