@@ -55,8 +55,8 @@ def parse_args(argv=None):
     ap.add_argument("--layers", type=int, default=0, help="debug only: truncate the models (marks the result invalid)")
     ap.add_argument("--lanes", type=int, default=2, help="Executor Lanes per FFN device (multi-GPU only)")
     ap.add_argument("--policy", default="fifo", choices=["fifo", "random", "slo"], help="Lane scheduling policy")
-    ap.add_argument("--layered", action="store_true",
-                    help="layered decoders beside the closest classic model of equal size, rates and kernels (one GPU)")
+    ap.add_argument("--layered", nargs="?", const="segirax", default="", choices=["segirax", "saninex"],
+                    help="a layered decoder beside the closest classic model of equal size, rates and kernels (one GPU)")
     # steady-state decode replay (kernel-level)
     ap.add_argument("--decode-only", action="store_true")
     ap.add_argument("--batch", type=int, default=256, help="decode-only: in-flight requests per Instance")
@@ -109,7 +109,7 @@ def main(argv=None) -> int:
     if args.layered:
         from crosspool_b200.bench import layered
 
-        print(json.dumps(layered.run(args.steps, max(3, args.warmup), args.layers or 8)))
+        print(json.dumps(layered.run(args.steps, max(3, args.warmup), args.layers or 8, design=args.layered)))
         return 0
     if args.decode_only:
         if args.gpus == 1 and world == 1:

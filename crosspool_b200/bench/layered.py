@@ -1,4 +1,5 @@
-"""Layered decoders (Segirax) beside the closest classic model of equal size on one GPU: ``bench.py --layered``.
+"""Layered decoders beside the closest classic model of equal size on one GPU: ``bench.py --layered`` (Segirax) and
+``--layered saninex`` (also beside Segirax; its sizes and kernels are in ``layered_saninex.py``).
 
 Two sizes whose layers resemble a real model's (random weights, a few layers): latent attention and decayed linear attention
 alternate, each with a PolyNorm FFN that holds as many weights as the gated FFN of the classic model. For both models, in
@@ -220,7 +221,8 @@ def kernel_table(classic: ModelConfig, cfg: ModelConfig, timer: Timer, batch: in
     return rows_out
 
 
-def run(steps: int = 20, warmup: int = 5, layers: int = 8, sizes=tuple(SIZES)) -> dict:
+def run(steps: int = 20, warmup: int = 5, layers: int = 8, sizes=tuple(SIZES), design: str = "segirax") -> dict:
+    from . import layered_saninex
     from .decode_bench import ClockSampler
 
     torch.cuda.set_device(0)
@@ -228,14 +230,21 @@ def run(steps: int = 20, warmup: int = 5, layers: int = 8, sizes=tuple(SIZES)) -
     sampler.start()
     out = {"metric": "prefill and decode tok/s of layered decoders beside the closest classic model of equal size", "unit": "tok/s",
            "dtype": "bf16", "data": "synthetic: random-init weights, random token ids", "context": CONTEXT, "chunk": CHUNK,
-           "layers": layers, "sizes": {}}
+           "layers": layers, "design": design, "sizes": {}}
     for size in sizes:
         name, heads = SIZES[size]
         classic = mc_preset(name).with_layers(layers)
-        cfg = layered_twin(classic, heads, layers)
+        segirax = layered_twin(classic, heads, layers)
+        cfg = segirax if design == "segirax" else layered_saninex.twin(classic, heads, layers)
         res = {"classic": name, "layered": throughput(cfg, steps, warmup), "classic_rates": throughput(classic, steps, warmup)}
         torch.cuda.empty_cache()
-        res["kernels"] = kernel_table(classic, cfg, Timer(max(10, steps), max(3, warmup), True))
+        timer = Timer(max(10, steps), max(3, warmup), True)
+        if design == "segirax":
+            res["kernels"] = kernel_table(classic, cfg, timer)
+        else:
+            res["segirax_rates"] = throughput(segirax, steps, warmup)
+            torch.cuda.empty_cache()
+            res["kernels"] = layered_saninex.kernel_table(classic, cfg, timer, CONTEXT, CHUNK, _row)
         torch.cuda.empty_cache()
         out["sizes"][size] = res
     out["clocks"] = sampler.stop()
