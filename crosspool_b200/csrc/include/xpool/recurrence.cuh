@@ -33,6 +33,17 @@ __device__ __forceinline__ void ldx(const __nv_bfloat16* p, float (&x)[VEC]) {
   }
 }
 template <int VEC, typename T>
+__device__ __forceinline__ void ldr(const T* p, T (&x)[VEC]) {
+  if constexpr (VEC * sizeof(T) == 16) {
+    const uint4 v = *reinterpret_cast<const uint4*>(p);
+    const T* e = reinterpret_cast<const T*>(&v);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) x[i] = e[i];
+  } else {
+    x[0] = p[0];
+  }
+}
+template <int VEC, typename T>
 __device__ __forceinline__ void stx(T* p, const T (&x)[VEC]) {
   if constexpr (VEC * sizeof(T) == 16) {
     uint4 v;

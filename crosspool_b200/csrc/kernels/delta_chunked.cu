@@ -6,7 +6,7 @@
 //   o_i = e^(c_i) a_i S^T q_i + sum_{j <= i} M_ij u_j,   M_ij = a_i b_j e^(c_i - c_j) q_i . k_j
 //   S  <- e^(c_n) S + sum_j k_j (b_j e^(c_n - c_j) u_j)^T
 //   delta_chunk_kernel   per (chunk, head), all at once: T = (1 + L)^-1 diag(beta), M and the factors, to the workspace
-//   delta_scan_kernel    per (32 value columns, head, sequence): walks the chunks with its part of the state in registers
+//   delta_scan_kernel    per (16 or 32 value columns, head, sequence): walks the chunks with its part of the state in registers
 // Queries and keys enter their products as the bf16 rows they are, their factors in fp32 afterwards; T, M, U and the state
 // enter as bf16 pairs (high and low part), so that everything of the recurrence keeps at least 16 mantissa bits.
 //
@@ -22,8 +22,6 @@ using namespace xpool::frag;
 
 constexpr int kChunk = 64;
 constexpr int kPC = kChunk + 8;            // pitch of chunk x chunk tiles
-constexpr int kVS = 32;                    // value columns of a scanning CTA
-constexpr int kPV = kVS + 8;
 
 // What the chunk kernel leaves for a (chunk, head).
 struct __align__(16) Record {
@@ -175,27 +173,49 @@ delta_chunk_kernel(XpDeltaArgs a) {
   }
 }
 
-template <int D>
+template <int D, int VS>
 struct ScanSmem {
-  static constexpr int PD = D + 8;
-  __nv_bfloat16 q[2][kChunk * PD], k[2][kChunk * PD], v[2][kChunk * kPV];
+  static constexpr int PD = D + 8, PV = VS + 8;
+  __nv_bfloat16 q[2][kChunk * PD], k[2][kChunk * PD];
   __nv_bfloat16 t[2][2][kChunk * kPC], m[2][2][kChunk * kPC];
-  __nv_bfloat16 s[2][D * kPV];             // state, high and low parts
-  __nv_bfloat16 r[2][kChunk * kPV];        // V - R, then the writes scaled for the state
-  __nv_bfloat16 u[2][kChunk * kPV];
+  __nv_bfloat16 s[2][2][D * PV];           // state before chunk c in buffer c & 1; high and low parts
+  __nv_bfloat16 r[2][kChunk * PV];         // V - R
+  __nv_bfloat16 w[2][kChunk * PV];         // writes, scaled for the state
+  __nv_bfloat16 u[2][2][kChunk * PV];      // writes of chunk c in buffer c & 1
   float f[2][3][kChunk];
   float decay[2];
 };
 
-// Warps 0-3 work on keys (16 rows each), warps 4-7 on queries where the two differ.
-template <int D>
-__global__ void __launch_bounds__(256, 1)
+__device__ __forceinline__ void chain_sync() { asm volatile("bar.sync 1, 256;" ::: "memory"); }
+
+// B operands of one k-step (16 rows of a [k][n] tile of pitch PV) for a warp's NT column tiles. A single column tile takes two
+// k-steps with one ldmatrix: every second call is free.
+template <int NT, int PV>
+struct BTile {
+  uint32_t addr;
+  uint32_t r[4];
+  __device__ __forceinline__ BTile(const __nv_bfloat16* tile, int col, int lane) {
+    addr = sm100::smem_u32(tile + col) + (NT == 2 ? bt_lane(lane, PV) : static_cast<uint32_t>(lane * PV * 2));
+  }
+  __device__ __forceinline__ void load(int ks) {
+    if (NT == 2 || (ks & 1) == 0) ldsm4t(addr + ks * 16 * PV * 2, r);
+  }
+  __device__ __forceinline__ uint32_t b0(int j, int ks) const { return NT == 2 ? r[j * 2] : r[(ks & 1) * 2]; }
+  __device__ __forceinline__ uint32_t b1(int j, int ks) const { return NT == 2 ? r[j * 2 + 1] : r[(ks & 1) * 2 + 1]; }
+};
+
+// Warps 0-7 carry the chain state -> V - R -> U -> state; warps 8-15 compute the outputs beside it: S^T q of the chunk at hand,
+// and M U of the chunk before. In both groups a warp owns 16 tokens and half of the columns (the state: 16 of its rows).
+template <int D, int VS>
+__global__ void __launch_bounds__(512, 1)
 delta_scan_kernel(XpDeltaArgs a) {
-  constexpr int PD = D + 8;
-  constexpr int NS = D >= 128 ? kVS / 8 : kVS / 16;  // state column tiles of a warp; its 16 rows start at d0
+  using Smem = ScanSmem<D, VS>;
+  constexpr int PD = Smem::PD, PV = Smem::PV;
+  constexpr int NT = VS / 16;                        // column tiles of a warp
+  constexpr int NS = D >= 128 ? VS / 8 : VS / 16;    // state column tiles of a warp; its 16 rows start at d0
   extern __shared__ __align__(16) uint8_t smem[];
-  ScanSmem<D>& sm = *reinterpret_cast<ScanSmem<D>*>(smem);
-  const int c0 = blockIdx.x * kVS, h = blockIdx.y, seq = blockIdx.z;
+  Smem& sm = *reinterpret_cast<Smem*>(smem);
+  const int c0 = blockIdx.x * VS, h = blockIdx.y, seq = blockIdx.z;
   const int n = a.q_lens[seq];
   if (n <= 0) return;
   const int r0 = a.q_starts[seq], chunks = (n + kChunk - 1) / kChunk;
@@ -203,211 +223,218 @@ delta_scan_kernel(XpDeltaArgs a) {
   const __nv_bfloat16* qkv = reinterpret_cast<const __nv_bfloat16*>(a.qkv) + static_cast<size_t>(r0) * channels;
   const Record* recs = reinterpret_cast<const Record*>(a.ws) + static_cast<size_t>(first_record(r0, seq)) * a.heads + h;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, q4 = lane & 3;
+  const bool chain = warp < 8;
+  const int rw = warp & 3, col = ((warp >> 2) & 1) * (VS / 2);
+  const int i0 = rw * 16 + g;                        // the lane's rows of a chunk: i0 and i0 + 8
 
+  auto issue_matrix = [&](__nv_bfloat16 (&dst)[2][kChunk * kPC], const __nv_bfloat16 (&src)[2][kChunk * kChunk]) {
+#pragma unroll
+    for (int i = threadIdx.x; i < 2 * kChunk * 8; i += 512) {
+      const int p = i >> 9, t = (i >> 3) & 63, e = (i & 7) * 8;
+      if (e / 16 <= t / 16) copy16(dst[p] + t * kPC + e, src[p] + t * kChunk + e, true);   // blocks above the diagonal are never read
+    }
+  };
+  // rows, T and factors of chunk c, M of the chunk before
   auto issue = [&](int c) {
     if (c < chunks) {
       const int b = c & 1, m = min(kChunk, n - c * kChunk);
-      const __nv_bfloat16* rows = qkv + static_cast<size_t>(c) * kChunk * channels;
+      const __nv_bfloat16* rows = qkv + static_cast<size_t>(c) * kChunk * channels + hk * a.dim;
       constexpr int kPieces = D / 8;
 #pragma unroll
-      for (int i = threadIdx.x; i < kChunk * kPieces; i += 256) {
+      for (int i = threadIdx.x; i < kChunk * kPieces; i += 512) {
         const int t = i / kPieces, e = i % kPieces * 8;
         const bool ok = t < m && e < a.dim;
-        const __nv_bfloat16* src = rows + static_cast<size_t>(ok ? t : 0) * channels + hk * a.dim + (ok ? e : 0);
+        const __nv_bfloat16* src = rows + static_cast<size_t>(ok ? t : 0) * channels + (ok ? e : 0);
         copy16(sm.q[b] + t * PD + e, src, ok);
         copy16(sm.k[b] + t * PD + e, src + nq, ok);
       }
-      {
-        const int t = threadIdx.x >> 2, e = (threadIdx.x & 3) * 8;
-        const bool ok = t < m && c0 + e < a.vdim;
-        copy16(sm.v[b] + t * kPV + e, rows + static_cast<size_t>(ok ? t : 0) * channels + 2 * nq + h * a.vdim + (ok ? c0 + e : 0), ok);
-      }
       const Record* rec = recs + static_cast<size_t>(c) * a.heads;
-#pragma unroll
-      for (int p = 0; p < 2; ++p)
-#pragma unroll
-        for (int i = threadIdx.x; i < kChunk * 8; i += 256) {
-          const int t = i >> 3, e = (i & 7) * 8;
-          const bool ok = e / 16 <= t / 16;                  // blocks above the diagonal are never read
-          if (ok) {
-            copy16(sm.t[b][p] + t * kPC + e, rec->t[p] + t * kChunk + e, true);
-            copy16(sm.m[b][p] + t * kPC + e, rec->m[p] + t * kChunk + e, true);
-          }
-        }
+      issue_matrix(sm.t[b], rec->t);
       if (threadIdx.x < 48) copy16(&sm.f[b][0][0] + threadIdx.x * 4, rec->read_k + threadIdx.x * 4, true);   // three arrays in a row
       if (threadIdx.x == 64) sm.decay[b] = rec->decay[0];
     }
+    if (c > 0 && c <= chunks) issue_matrix(sm.m[(c - 1) & 1], recs[static_cast<size_t>(c - 1) * a.heads].m);
     copies_issued();
   };
   issue(0);
 
-  const int d0 = D >= 128 ? warp * 16 : (warp & 3) * 16, s0 = D >= 128 ? 0 : (warp >> 2) * (kVS / 2);
+  // values of the lane's rows, one chunk ahead
+  uint32_t v[NT][2];
+  auto load_v = [&](int c) {
+#pragma unroll
+    for (int j = 0; j < NT; ++j)
+#pragma unroll
+      for (int r = 0; r < 2; ++r) {
+        const int t = c * kChunk + i0 + r * 8, cc = c0 + col + j * 8 + q4 * 2;
+        v[j][r] = t < n && cc < a.vdim ? *reinterpret_cast<const uint32_t*>(qkv + static_cast<size_t>(t) * channels + 2 * nq + h * a.vdim + cc) : 0u;
+      }
+  };
+  const int d0 = D >= 128 ? (warp & 7) * 16 : rw * 16, s0 = D >= 128 ? 0 : col;
   float* slot = a.state + (static_cast<size_t>(a.state_slots[seq]) * a.heads + h) * a.dim * a.vdim;
-  const bool fresh = a.positions[r0] == 0;
   float s[NS][4];
-#pragma unroll
-  for (int j = 0; j < NS; ++j)
-#pragma unroll
-    for (int r = 0; r < 2; ++r) {
-      const int d = d0 + g + r * 8, c = c0 + s0 + j * 8 + q4 * 2;
-      float2 x = make_float2(0.f, 0.f);
-      if (!fresh && d < a.dim && c < a.vdim) x = *reinterpret_cast<const float2*>(slot + static_cast<size_t>(d) * a.vdim + c);
-      s[j][2 * r] = x.x;
-      s[j][2 * r + 1] = x.y;
-    }
-  auto publish = [&](__nv_bfloat16 (&dst)[2][D * kPV]) {
+  auto publish = [&](int b) {
 #pragma unroll
     for (int j = 0; j < NS; ++j)
 #pragma unroll
       for (int r = 0; r < 2; ++r) {
         uint32_t hi, lo;
         split2(s[j][2 * r], s[j][2 * r + 1], hi, lo);
-        const int at = (d0 + g + r * 8) * kPV + s0 + j * 8 + q4 * 2;
-        *reinterpret_cast<uint32_t*>(dst[0] + at) = hi;
-        *reinterpret_cast<uint32_t*>(dst[1] + at) = lo;
+        const int at = (d0 + g + r * 8) * PV + s0 + j * 8 + q4 * 2;
+        *reinterpret_cast<uint32_t*>(sm.s[b][0] + at) = hi;
+        *reinterpret_cast<uint32_t*>(sm.s[b][1] + at) = lo;
       }
   };
-  publish(sm.s);
+  if (chain) {
+    load_v(0);
+    const bool fresh = a.positions[r0] == 0;
+#pragma unroll
+    for (int j = 0; j < NS; ++j)
+#pragma unroll
+      for (int r = 0; r < 2; ++r) {
+        const int d = d0 + g + r * 8, c = c0 + s0 + j * 8 + q4 * 2;
+        float2 x = make_float2(0.f, 0.f);
+        if (!fresh && d < a.dim && c < a.vdim) x = *reinterpret_cast<const float2*>(slot + static_cast<size_t>(d) * a.vdim + c);
+        s[j][2 * r] = x.x;
+        s[j][2 * r + 1] = x.y;
+      }
+    publish(0);
+  }
 
-  const int rw = warp & 3;
-  const bool on_q = warp >= 4;
-  const uint32_t bt_v = bt_lane(lane, kPV);
-  const uint32_t s_hi = sm100::smem_u32(sm.s[0]) + bt_v, s_lo = sm100::smem_u32(sm.s[1]) + bt_v;
-  const uint32_t r_hi = sm100::smem_u32(sm.r[0]) + bt_v, r_lo = sm100::smem_u32(sm.r[1]) + bt_v;
-  const uint32_t u_hi = sm100::smem_u32(sm.u[0]) + bt_v, u_lo = sm100::smem_u32(sm.u[1]) + bt_v;
-  for (int c = 0; c < chunks; ++c) {
-    const int b = c & 1, m = min(kChunk, n - c * kChunk);
+  float o[NT][4];                                    // outputs of the chunk at hand until its M U joins them
+  for (int c = 0; c <= chunks; ++c) {
+    const int b = c & 1;
     copies_wait<0>();
-    __syncthreads();                       // chunk c landed, state published, buffers of chunk c - 1 free
+    __syncthreads();                                 // chunk c landed, state published, writes of chunk c - 1 there
     issue(c + 1);
-    // ---- S^T k and S^T q: warp = 16 rows, all columns
-    float o[4][4];
+    if (!chain && c > 0) {
+      // ---- o += M U, and out
+      float x[2][NT][4];
 #pragma unroll
-    for (int j = 0; j < 4; ++j)
+      for (int p = 0; p < 2; ++p)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) o[j][e] = 0.f;
-    const uint32_t rows_a = sm100::smem_u32((on_q ? sm.q[b] : sm.k[b]) + rw * 16 * PD) + a_lane(lane, PD);
-#pragma unroll 4
-    for (int ks = 0; ks < D / 16; ++ks) {
-      uint32_t fa[4], h0[4], h1[4], l0[4], l1[4];
-      ldsm4(rows_a + ks * 32, fa);
-      ldsm4t(s_hi + ks * 16 * kPV * 2, h0);
-      ldsm4t(s_hi + (ks * 16 * kPV + 16) * 2, h1);
-      ldsm4t(s_lo + ks * 16 * kPV * 2, l0);
-      ldsm4t(s_lo + (ks * 16 * kPV + 16) * 2, l1);
-      mma(o[0], fa, h0[0], h0[1]);
-      mma(o[1], fa, h0[2], h0[3]);
-      mma(o[2], fa, h1[0], h1[1]);
-      mma(o[3], fa, h1[2], h1[3]);
-      mma(o[0], fa, l0[0], l0[1]);
-      mma(o[1], fa, l0[2], l0[3]);
-      mma(o[2], fa, l1[0], l1[1]);
-      mma(o[3], fa, l1[2], l1[3]);
-    }
-    const int i0 = rw * 16 + g;            // rows i0 and i0 + 8 of the chunk
-    {
-      const float* f = sm.f[b][on_q ? 1 : 0];
-      const float f0 = f[i0], f1 = f[i0 + 8];
+        for (int j = 0; j < NT; ++j)
 #pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        o[j][0] *= f0, o[j][1] *= f0, o[j][2] *= f1, o[j][3] *= f1;
-        if (!on_q) {
-#pragma unroll
-          for (int r = 0; r < 2; ++r) {
-            const int at = (i0 + r * 8) * kPV + j * 8 + q4 * 2;
-            const float2 v = unpack2(*reinterpret_cast<const uint32_t*>(sm.v[b] + at));
-            uint32_t hi, lo;
-            split2(v.x - o[j][2 * r], v.y - o[j][2 * r + 1], hi, lo);
-            *reinterpret_cast<uint32_t*>(sm.r[0] + at) = hi;
-            *reinterpret_cast<uint32_t*>(sm.r[1] + at) = lo;
-          }
-        }
-      }
-    }
-    __syncthreads();
-    // ---- U = T (V - R): warp = 16 rows, half of the columns
-    float u[2][4];
-#pragma unroll
-    for (int j = 0; j < 2; ++j)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) u[j][e] = 0.f;
-    const int uc = (warp >> 2) * 16;
-    const uint32_t ta_hi = sm100::smem_u32(sm.t[b][0] + rw * 16 * kPC) + a_lane(lane, kPC);
-    const uint32_t ta_lo = sm100::smem_u32(sm.t[b][1] + rw * 16 * kPC) + a_lane(lane, kPC);
-#pragma unroll
-    for (int ks = 0; ks < 4; ++ks) {
-      if (ks <= rw) {
-        uint32_t th[4], tl[4], bh[4], bl[4];
-        ldsm4(ta_hi + ks * 32, th);
-        ldsm4(ta_lo + ks * 32, tl);
-        ldsm4t(r_hi + (ks * 16 * kPV + uc) * 2, bh);
-        ldsm4t(r_lo + (ks * 16 * kPV + uc) * 2, bl);
-        mma(u[0], th, bh[0], bh[1]);
-        mma(u[1], th, bh[2], bh[3]);
-        mma(u[0], th, bl[0], bl[1]);
-        mma(u[1], th, bl[2], bl[3]);
-        mma(u[0], tl, bh[0], bh[1]);
-        mma(u[1], tl, bh[2], bh[3]);
-      }
-    }
-    __syncthreads();                       // everyone has read V - R
-    {
-      const float w0 = sm.f[b][2][i0], w1 = sm.f[b][2][i0 + 8];
-#pragma unroll
-      for (int j = 0; j < 2; ++j)
-#pragma unroll
-        for (int r = 0; r < 2; ++r) {
-          const int at = (i0 + r * 8) * kPV + uc + j * 8 + q4 * 2;
-          const float x = u[j][2 * r], y = u[j][2 * r + 1], w = r ? w1 : w0;
-          uint32_t hi, lo;
-          split2(x, y, hi, lo);
-          *reinterpret_cast<uint32_t*>(sm.u[0] + at) = hi;
-          *reinterpret_cast<uint32_t*>(sm.u[1] + at) = lo;
-          split2(x * w, y * w, hi, lo);
-          *reinterpret_cast<uint32_t*>(sm.r[0] + at) = hi;
-          *reinterpret_cast<uint32_t*>(sm.r[1] + at) = lo;
-        }
-    }
-    __syncthreads();
-    // ---- outputs (warps of the queries)
-    if (on_q) {
-      const uint32_t ma_hi = sm100::smem_u32(sm.m[b][0] + rw * 16 * kPC) + a_lane(lane, kPC);
-      const uint32_t ma_lo = sm100::smem_u32(sm.m[b][1] + rw * 16 * kPC) + a_lane(lane, kPC);
+          for (int e = 0; e < 4; ++e) x[p][j][e] = p ? 0.f : o[j][e];
+      const uint32_t m_hi = sm100::smem_u32(sm.m[b ^ 1][0] + rw * 16 * kPC) + a_lane(lane, kPC);
+      const uint32_t m_lo = sm100::smem_u32(sm.m[b ^ 1][1] + rw * 16 * kPC) + a_lane(lane, kPC);
+      BTile<NT, PV> uh(sm.u[b ^ 1][0], col, lane), ul(sm.u[b ^ 1][1], col, lane);
 #pragma unroll
       for (int ks = 0; ks < 4; ++ks) {
         if (ks <= rw) {
           uint32_t mh[4], ml[4];
-          ldsm4(ma_hi + ks * 32, mh);
-          ldsm4(ma_lo + ks * 32, ml);
+          ldsm4(m_hi + ks * 32, mh);
+          ldsm4(m_lo + ks * 32, ml);
+          uh.load(ks), ul.load(ks);
 #pragma unroll
-          for (int j = 0; j < 2; ++j) {
-            uint32_t bh[4], bl[4];
-            ldsm4t(u_hi + (ks * 16 * kPV + j * 16) * 2, bh);
-            ldsm4t(u_lo + (ks * 16 * kPV + j * 16) * 2, bl);
-            mma(o[2 * j], mh, bh[0], bh[1]);
-            mma(o[2 * j + 1], mh, bh[2], bh[3]);
-            mma(o[2 * j], mh, bl[0], bl[1]);
-            mma(o[2 * j + 1], mh, bl[2], bl[3]);
-            mma(o[2 * j], ml, bh[0], bh[1]);
-            mma(o[2 * j + 1], ml, bh[2], bh[3]);
+          for (int j = 0; j < NT; ++j) {
+            mma(x[0][j], mh, uh.b0(j, ks), uh.b1(j, ks));
+            mma(x[1][j], mh, ul.b0(j, ks), ul.b1(j, ks));
+            mma(x[1][j], ml, uh.b0(j, ks), uh.b1(j, ks));
           }
         }
       }
 #pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        const int col = c0 + j * 8 + q4 * 2;
+      for (int j = 0; j < NT; ++j) {
+        const int cc = c0 + col + j * 8 + q4 * 2;
 #pragma unroll
         for (int r = 0; r < 2; ++r) {
-          const int i = i0 + r * 8;
-          if (i < m && col < a.vdim)
-            *reinterpret_cast<float2*>(reinterpret_cast<float*>(a.out) + static_cast<size_t>(r0 + c * kChunk + i) * a.ld_out + h * a.vdim + col) =
-                make_float2(o[j][2 * r], o[j][2 * r + 1]);
+          const int t = (c - 1) * kChunk + i0 + r * 8;
+          if (t < n && cc < a.vdim)
+            *reinterpret_cast<float2*>(reinterpret_cast<float*>(a.out) + static_cast<size_t>(r0 + t) * a.ld_out + h * a.vdim + cc) =
+                make_float2(x[0][j][2 * r] + x[1][j][2 * r], x[0][j][2 * r + 1] + x[1][j][2 * r + 1]);
         }
       }
     }
-    // ---- state: warp = 16 rows of it
+    if (c == chunks) break;
+    // ---- S^T k (chain) and S^T q
+    float y[2][NT][4];
+#pragma unroll
+    for (int p = 0; p < 2; ++p)
+#pragma unroll
+      for (int j = 0; j < NT; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) y[p][j][e] = 0.f;
+    {
+      const uint32_t rows_a = sm100::smem_u32((chain ? sm.k[b] : sm.q[b]) + rw * 16 * PD) + a_lane(lane, PD);
+      BTile<NT, PV> sh(sm.s[b][0], col, lane), sl(sm.s[b][1], col, lane);
+#pragma unroll
+      for (int ks = 0; ks < D / 16; ++ks) {
+        uint32_t fa[4];
+        ldsm4(rows_a + ks * 32, fa);
+        sh.load(ks), sl.load(ks);
+#pragma unroll
+        for (int j = 0; j < NT; ++j) {
+          mma(y[0][j], fa, sh.b0(j, ks), sh.b1(j, ks));
+          mma(y[1][j], fa, sl.b0(j, ks), sl.b1(j, ks));
+        }
+      }
+    }
+    const float f0 = sm.f[b][chain ? 0 : 1][i0], f1 = sm.f[b][chain ? 0 : 1][i0 + 8];
+#pragma unroll
+    for (int j = 0; j < NT; ++j)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) o[j][e] = (y[0][j][e] + y[1][j][e]) * (e < 2 ? f0 : f1);
+    if (!chain) continue;
+#pragma unroll
+    for (int j = 0; j < NT; ++j)
+#pragma unroll
+      for (int r = 0; r < 2; ++r) {
+        const int at = (i0 + r * 8) * PV + col + j * 8 + q4 * 2;
+        const float2 x = unpack2(v[j][r]);
+        uint32_t hi, lo;
+        split2(x.x - o[j][2 * r], x.y - o[j][2 * r + 1], hi, lo);
+        *reinterpret_cast<uint32_t*>(sm.r[0] + at) = hi;
+        *reinterpret_cast<uint32_t*>(sm.r[1] + at) = lo;
+      }
+    load_v(c + 1);
+    chain_sync();
+    // ---- U = T (V - R)
+#pragma unroll
+    for (int p = 0; p < 2; ++p)
+#pragma unroll
+      for (int j = 0; j < NT; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) y[p][j][e] = 0.f;
+    {
+      const uint32_t t_hi = sm100::smem_u32(sm.t[b][0] + rw * 16 * kPC) + a_lane(lane, kPC);
+      const uint32_t t_lo = sm100::smem_u32(sm.t[b][1] + rw * 16 * kPC) + a_lane(lane, kPC);
+      BTile<NT, PV> rh(sm.r[0], col, lane), rl(sm.r[1], col, lane);
+#pragma unroll
+      for (int ks = 0; ks < 4; ++ks) {
+        if (ks <= rw) {
+          uint32_t th[4], tl[4];
+          ldsm4(t_hi + ks * 32, th);
+          ldsm4(t_lo + ks * 32, tl);
+          rh.load(ks), rl.load(ks);
+#pragma unroll
+          for (int j = 0; j < NT; ++j) {
+            mma(y[0][j], th, rh.b0(j, ks), rh.b1(j, ks));
+            mma(y[1][j], th, rl.b0(j, ks), rl.b1(j, ks));
+            mma(y[1][j], tl, rh.b0(j, ks), rh.b1(j, ks));
+          }
+        }
+      }
+    }
+    const float w0 = sm.f[b][2][i0], w1 = sm.f[b][2][i0 + 8];
+#pragma unroll
+    for (int j = 0; j < NT; ++j)
+#pragma unroll
+      for (int r = 0; r < 2; ++r) {
+        const int at = (i0 + r * 8) * PV + col + j * 8 + q4 * 2;
+        const float x0 = y[0][j][2 * r] + y[1][j][2 * r], x1 = y[0][j][2 * r + 1] + y[1][j][2 * r + 1], w = r ? w1 : w0;
+        uint32_t hi, lo;
+        split2(x0 * w, x1 * w, hi, lo);
+        *reinterpret_cast<uint32_t*>(sm.w[0] + at) = hi;
+        *reinterpret_cast<uint32_t*>(sm.w[1] + at) = lo;
+        split2(x0, x1, hi, lo);
+        *reinterpret_cast<uint32_t*>(sm.u[b][0] + at) = hi;
+        *reinterpret_cast<uint32_t*>(sm.u[b][1] + at) = lo;
+      }
+    chain_sync();
+    // ---- state
     const float dec = sm.decay[b];
     const uint32_t kt = sm100::smem_u32(sm.k[b] + d0) + at_lane(lane, PD);
+    const uint32_t w_hi = sm100::smem_u32(sm.w[0] + s0) + bt_lane(lane, PV), w_lo = sm100::smem_u32(sm.w[1] + s0) + bt_lane(lane, PV);
 #pragma unroll
     for (int j = 0; j < NS; ++j)
 #pragma unroll
@@ -416,19 +443,29 @@ delta_scan_kernel(XpDeltaArgs a) {
     for (int ks = 0; ks < 4; ++ks) {
       uint32_t ka[4];
       ldsm4t(kt + ks * 16 * PD * 2, ka);
+      if constexpr (NS == 1) {
+        uint32_t bh[4], bl[4];             // (the second tile belongs to the other half's warp)
+        ldsm4t(w_hi + ks * 16 * PV * 2 - (s0 ? 16 : 0), bh);
+        ldsm4t(w_lo + ks * 16 * PV * 2 - (s0 ? 16 : 0), bl);
+        mma(s[0], ka, s0 ? bh[2] : bh[0], s0 ? bh[3] : bh[1]);
+        mma(s[0], ka, s0 ? bl[2] : bl[0], s0 ? bl[3] : bl[1]);
+      } else {
 #pragma unroll
-      for (int j = 0; j < NS; j += 2) {
-        uint32_t bh[4], bl[4];
-        ldsm4t(r_hi + (ks * 16 * kPV + s0 + j * 8) * 2, bh);
-        ldsm4t(r_lo + (ks * 16 * kPV + s0 + j * 8) * 2, bl);
-        mma(s[j], ka, bh[0], bh[1]);
-        mma(s[j + 1], ka, bh[2], bh[3]);
-        mma(s[j], ka, bl[0], bl[1]);
-        mma(s[j + 1], ka, bl[2], bl[3]);
+        for (int j = 0; j < NS; j += 2) {
+          uint32_t bh[4], bl[4];
+          ldsm4t(w_hi + (ks * 16 * PV + j * 8) * 2, bh);
+          ldsm4t(w_lo + (ks * 16 * PV + j * 8) * 2, bl);
+          mma(s[j], ka, bh[0], bh[1]);
+          mma(s[j + 1], ka, bh[2], bh[3]);
+          mma(s[j], ka, bl[0], bl[1]);
+          mma(s[j + 1], ka, bl[2], bl[3]);
+        }
       }
     }
-    if (c + 1 < chunks) publish(sm.s);     // the reads of the old state lie two barriers back
+    if (c + 1 < chunks) publish(b ^ 1);
   }
+  copies_wait<0>();
+  if (!chain) return;
 #pragma unroll
   for (int j = 0; j < NS; ++j)
 #pragma unroll
@@ -439,18 +476,31 @@ delta_scan_kernel(XpDeltaArgs a) {
     }
 }
 
-template <int D>
-int launch(const XpDeltaArgs& a, cudaStream_t s) {
-  static_assert(sizeof(ScanSmem<D>) <= 227 * 1024, "tiles exceed the shared memory of an SM");
+template <int D, int VS>
+int launch_scan(const XpDeltaArgs& a, cudaStream_t s) {
+  constexpr int kBytes = sizeof(ScanSmem<D, VS>);
+  static_assert(kBytes <= 227 * 1024, "tiles exceed the shared memory of an SM");
   static bool attr_set = false;
   if (!attr_set) {
-    if (cudaFuncSetAttribute(delta_chunk_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, chunk_smem<D>()) != cudaSuccess ||
-        cudaFuncSetAttribute(delta_scan_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, sizeof(ScanSmem<D>)) != cudaSuccess)
-      return -21;
+    if (cudaFuncSetAttribute(delta_scan_kernel<D, VS>, cudaFuncAttributeMaxDynamicSharedMemorySize, kBytes) != cudaSuccess) return -21;
+    attr_set = true;
+  }
+  delta_scan_kernel<D, VS><<<dim3((a.vdim + VS - 1) / VS, a.heads, a.seqs), 512, kBytes, s>>>(a);
+  return 0;
+}
+
+template <int D>
+int launch(const XpDeltaArgs& a, cudaStream_t s) {
+  static bool attr_set = false;
+  if (!attr_set) {
+    if (cudaFuncSetAttribute(delta_chunk_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, chunk_smem<D>()) != cudaSuccess) return -21;
     attr_set = true;
   }
   delta_chunk_kernel<D><<<dim3((a.max_q + kChunk - 1) / kChunk, a.heads, a.seqs), 128, chunk_smem<D>(), s>>>(a);
-  delta_scan_kernel<D><<<dim3((a.vdim + kVS - 1) / kVS, a.heads, a.seqs), 256, sizeof(ScanSmem<D>), s>>>(a);
+  // narrow columns while they still fit on the SMs at the same time
+  const bool narrow = static_cast<int64_t>((a.vdim + 15) / 16) * a.heads * a.seqs <= 148;
+  const int rc = narrow ? launch_scan<D, 16>(a, s) : launch_scan<D, 32>(a, s);
+  if (rc != 0) return rc;
   cudaError_t e = cudaGetLastError();
   return e == cudaSuccess ? 0 : -100 - static_cast<int>(e);
 }

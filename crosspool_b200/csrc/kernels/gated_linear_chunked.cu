@@ -20,6 +20,7 @@ using namespace xpool::frag;
 
 constexpr int kChunk = 64;
 constexpr int kPC = kChunk + 8;
+constexpr int kScan = 512;                 // threads of a scanning CTA
 constexpr float kRange = 80.f;
 constexpr float kLog2e = 1.4426950408889634f;
 
@@ -33,17 +34,25 @@ template <int D>
 struct ChunkSmem {
   static constexpr int PD = D + 8;
   __nv_bfloat16 q[2][kChunk * PD], k[2][kChunk * PD];
-  float c[kChunk * D];                     // running sums
-  float b[4][D];                           // ... before each block
+  float b[5][D];                           // running sums before each block, and behind the last
 };
 
+// log2 of sigmoid(z) ** inv_tau; the logarithm of 1 + e keeps its relative accuracy for small e
+__device__ __forceinline__ float log2_decay(float z, float inv_tau) {
+  const float x = -kLog2e * z, e = sm100::ex2_approx(-fabsf(x));
+  float l;
+  asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(l) : "f"(1.f + e));
+  if (e < 0.03125f) l = kLog2e * e * fmaf(e, fmaf(e, fmaf(e, -0.25f, 0.33333333f), -0.5f), 1.f);
+  return -(fmaxf(x, 0.f) + l) * inv_tau;
+}
+
+// A thread takes two channels of one block: 16 tokens, all loads in flight at once.
 template <int D>
 __global__ void __launch_bounds__(256)
 gated_linear_chunk_kernel(XpGatedLinearArgs a) {
-  constexpr int PD = D + 8;
+  constexpr int PD = D + 8, kPairs = D / 2;
   extern __shared__ __align__(16) uint8_t smem[];
   ChunkSmem<D>& sm = *reinterpret_cast<ChunkSmem<D>*>(smem);
-  __shared__ int wide;
   const int h = blockIdx.y, seq = blockIdx.z, total = a.q_lens[seq];
   const int t0 = blockIdx.x * kChunk;
   if (t0 >= total) return;
@@ -51,81 +60,73 @@ gated_linear_chunk_kernel(XpGatedLinearArgs a) {
   const int width = a.heads * a.dim;
   float* z = const_cast<float*>(a.z) + static_cast<size_t>(r0) * width + h * a.dim;
   const __nv_bfloat16* rows = reinterpret_cast<const __nv_bfloat16*>(a.proj) + static_cast<size_t>(r0) * a.ld_proj + h * a.dim;
-  if (threadIdx.x == 0) wide = 0;
-  for (int i = threadIdx.x; i < kChunk * D; i += 256) {
-    const int t = i / D, d = i % D;
-    sm.c[i] = t < n && d < a.dim ? recur::log_decay(z[static_cast<size_t>(t) * width + d], a.inv_tau) * kLog2e : 0.f;
-  }
-  __syncthreads();
-  // sums inside each block of 16 tokens, then the blocks' starts
-  for (int i = threadIdx.x; i < 4 * D; i += 256) {
-    const int d = i % D, r = i / D;
-    float s = 0.f;
+  const int d = threadIdx.x % kPairs * 2, blk = threadIdx.x / kPairs;
+  const bool mine = blk < 4;
+  float2 c[16];
+  uint32_t q[16], k[16];
+  bool far = false;
+  if (mine) {
 #pragma unroll
     for (int t = 0; t < 16; ++t) {
-      s += sm.c[(r * 16 + t) * D + d];
-      sm.c[(r * 16 + t) * D + d] = s;
+      const int row = blk * 16 + t;
+      const bool ok = row < n && d < a.dim;
+      const __nv_bfloat16* p = rows + static_cast<size_t>(ok ? row : 0) * a.ld_proj + (ok ? d : 0);
+      c[t] = ok ? *reinterpret_cast<const float2*>(z + static_cast<size_t>(row) * width + d) : make_float2(0.f, 0.f);
+      q[t] = ok ? *reinterpret_cast<const uint32_t*>(p + a.q_off) : 0u;
+      k[t] = ok ? *reinterpret_cast<const uint32_t*>(p + a.k_off) : 0u;
     }
-    if (s < -kRange) wide = 1;
+    float2 s = make_float2(0.f, 0.f);
+#pragma unroll
+    for (int t = 0; t < 16; ++t) {
+      if (blk * 16 + t < n && d < a.dim) s.x += log2_decay(c[t].x, a.inv_tau), s.y += log2_decay(c[t].y, a.inv_tau);
+      c[t] = s;
+    }
+    *reinterpret_cast<float2*>(&sm.b[blk + 1][d]) = s;
+    far = s.x < -kRange || s.y < -kRange;
   }
-  __syncthreads();
-  for (int d = threadIdx.x; d < D; d += 256) {
+  const bool direct = __syncthreads_or(far) != 0;
+  // the blocks' starts
+  for (int i = threadIdx.x; i < D; i += 256) {
     float s = 0.f;
+    sm.b[0][i] = 0.f;
 #pragma unroll
-    for (int r = 0; r < 4; ++r) {
-      sm.b[r][d] = s;
-      s += sm.c[(r * 16 + 15) * D + d];
-    }
+    for (int r = 1; r < 5; ++r) sm.b[r][i] = s += sm.b[r][i];
   }
   __syncthreads();
-  // c to the workspace; decayed queries and keys (of both only what their own block adds)
-  const bool direct = wide != 0;
-  constexpr int kPieces = D / 8;
-  for (int i = threadIdx.x; i < kChunk * kPieces; i += 256) {
-    const int t = i / kPieces, e = i % kPieces * 8, r = t >> 4;
-    const bool ok = t < n && e < a.dim;
-    float q[8], k[8];
+  // c to the workspace; queries and keys with what their own block decays them
+  if (mine) {
+    const float2 start = *reinterpret_cast<const float2*>(&sm.b[blk][d]);
 #pragma unroll
-    for (int j = 0; j < 8; ++j) q[j] = k[j] = 0.f;
-    if (ok) {
-      recur::ldx<8>(rows + static_cast<size_t>(t) * a.ld_proj + a.q_off + e, q);
-      recur::ldx<8>(rows + static_cast<size_t>(t) * a.ld_proj + a.k_off + e, k);
-    }
-    float4 c[2];
-#pragma unroll
-    for (int j = 0; j < 8; ++j) {
-      const float x = sm.c[t * D + e + j];
-      reinterpret_cast<float*>(c)[j] = x + sm.b[r][e + j];
-      q[j] *= a.qscale;
+    for (int t = 0; t < 16; ++t) {
+      const int row = blk * 16 + t;
+      if (row < n && d < a.dim) *reinterpret_cast<float2*>(z + static_cast<size_t>(row) * width + d) = make_float2(start.x + c[t].x, start.y + c[t].y);
+      float2 x = unpack2(q[t]), y = unpack2(k[t]);
+      x.x *= a.qscale, x.y *= a.qscale;
       if (!direct) {
-        q[j] *= sm100::ex2_approx(x);
-        k[j] *= sm100::ex2_approx(-x);
+        x.x *= sm100::ex2_approx(c[t].x), x.y *= sm100::ex2_approx(c[t].y);
+        y.x *= sm100::ex2_approx(-c[t].x), y.y *= sm100::ex2_approx(-c[t].y);
       }
+      uint32_t hi, lo;
+      split2(x.x, x.y, hi, lo);
+      *reinterpret_cast<uint32_t*>(sm.q[0] + row * PD + d) = hi;
+      *reinterpret_cast<uint32_t*>(sm.q[1] + row * PD + d) = lo;
+      split2(y.x, y.y, hi, lo);
+      *reinterpret_cast<uint32_t*>(sm.k[0] + row * PD + d) = hi;
+      *reinterpret_cast<uint32_t*>(sm.k[1] + row * PD + d) = lo;
     }
-    if (ok) {
-      *reinterpret_cast<float4*>(z + static_cast<size_t>(t) * width + e) = c[0];
-      *reinterpret_cast<float4*>(z + static_cast<size_t>(t) * width + e + 4) = c[1];
-    }
-    uint4 hi, lo;
-    split2(q[0], q[1], hi.x, lo.x), split2(q[2], q[3], hi.y, lo.y), split2(q[4], q[5], hi.z, lo.z), split2(q[6], q[7], hi.w, lo.w);
-    *reinterpret_cast<uint4*>(sm.q[0] + t * PD + e) = hi;
-    *reinterpret_cast<uint4*>(sm.q[1] + t * PD + e) = lo;
-    split2(k[0], k[1], hi.x, lo.x), split2(k[2], k[3], hi.y, lo.y), split2(k[4], k[5], hi.z, lo.z), split2(k[6], k[7], hi.w, lo.w);
-    *reinterpret_cast<uint4*>(sm.k[0] + t * PD + e) = hi;
-    *reinterpret_cast<uint4*>(sm.k[1] + t * PD + e) = lo;
   }
-  __syncthreads();
+  __syncthreads();                         // also makes c visible to the block
   Record* rec = reinterpret_cast<Record*>(a.records) + static_cast<size_t>(first_record(a.q_starts[seq], seq) + blockIdx.x) * a.heads + h;
   if (direct) {                            // q and k are undecayed here
     for (int p = threadIdx.x; p < kChunk * kChunk; p += 256) {
       const int i = p / kChunk, j = p % kChunk;
       float s = 0.f;
-      if (j <= i) {
-        for (int d = 0; d < a.dim; ++d) {
-          const float x = (sm.c[i * D + d] - sm.c[j * D + d]) + (sm.b[i >> 4][d] - sm.b[j >> 4][d]);
-          const float q = __bfloat162float(sm.q[0][i * PD + d]) + __bfloat162float(sm.q[1][i * PD + d]);
-          const float k = __bfloat162float(sm.k[0][j * PD + d]) + __bfloat162float(sm.k[1][j * PD + d]);
-          s = fmaf(q * k, exp2f(x), s);
+      if (j <= i && i < n) {
+        for (int e = 0; e < a.dim; ++e) {
+          const float x = z[static_cast<size_t>(i) * width + e] - z[static_cast<size_t>(j) * width + e];
+          const float qe = __bfloat162float(sm.q[0][i * PD + e]) + __bfloat162float(sm.q[1][i * PD + e]);
+          const float ke = __bfloat162float(sm.k[0][j * PD + e]) + __bfloat162float(sm.k[1][j * PD + e]);
+          s = fmaf(qe * ke, exp2f(x), s);
         }
       }
       const __nv_bfloat16 hi = __float2bfloat16_rn(s);
@@ -157,8 +158,8 @@ gated_linear_chunk_kernel(XpGatedLinearArgs a) {
       if (j < rw) {                        // what lies between the two blocks
 #pragma unroll
         for (int u = 0; u < 2; ++u) {      // dims d, d + 1 and d + 8, d + 9 of the fragment
-          const int d = ks * 16 + u * 8 + q4 * 2;
-          const float f0 = sm100::ex2_approx(sm.b[rw][d] - sm.b[j][d]), f1 = sm100::ex2_approx(sm.b[rw][d + 1] - sm.b[j][d + 1]);
+          const int e = ks * 16 + u * 8 + q4 * 2;
+          const float f0 = sm100::ex2_approx(sm.b[rw][e] - sm.b[j][e]), f1 = sm100::ex2_approx(sm.b[rw][e + 1] - sm.b[j][e + 1]);
 #pragma unroll
           for (int v = 0; v < 2; ++v) {    // rows g and g + 8
             const float2 x = unpack2(qh[u * 2 + v]), y = unpack2(ql[u * 2 + v]);
@@ -200,11 +201,13 @@ struct ScanSmem {
 
 // kFull: outputs and the state; otherwise only what the segment adds to the state, and its decay.
 template <int D, int VS, bool kFull>
-__global__ void __launch_bounds__(256, 1)
+__global__ void __launch_bounds__(kScan, 1)
 gated_linear_scan_kernel(XpGatedLinearArgs a) {
   constexpr int PD = D + 8, PV = VS + 8;
-  constexpr int NO = VS / 16;                        // output tiles of a warp (half of the columns, 8 each)
-  constexpr int NS = D >= 128 ? VS / 8 : VS / 16;    // state column tiles of a warp
+  constexpr int NO = VS / 32 > 1 ? VS / 32 : 2;      // output tiles of a warp (8 columns each; 16 rows)
+  constexpr int kOut = VS / (8 * NO);                // warps side by side there
+  constexpr int NS = D >= 128 ? VS / 16 : VS / 32 > 1 ? VS / 32 : 2;   // state column tiles of a warp (16 rows)
+  constexpr int kRowWarps = D / 16, kState = VS / (8 * NS);
   extern __shared__ __align__(16) uint8_t smem[];
   ScanSmem<D, VS>& sm = *reinterpret_cast<ScanSmem<D, VS>*>(smem);
   const int slices = (a.vdim + VS - 1) / VS;
@@ -227,7 +230,7 @@ gated_linear_scan_kernel(XpGatedLinearArgs a) {
       const float* cs = a.z + static_cast<size_t>(r0 + c * kChunk) * width + h * a.dim;
       constexpr int kPieces = D / 8;
 #pragma unroll
-      for (int i = threadIdx.x; i < kChunk * kPieces; i += 256) {
+      for (int i = threadIdx.x; i < kChunk * kPieces; i += kScan) {
         const int t = i / kPieces, e = i % kPieces * 8;
         const bool ok = t < m && e < a.dim;
         const __nv_bfloat16* row = rows + static_cast<size_t>(ok ? t : 0) * a.ld_proj + (ok ? e : 0);
@@ -245,7 +248,7 @@ gated_linear_scan_kernel(XpGatedLinearArgs a) {
       const __nv_bfloat16* rows = proj + static_cast<size_t>(r0 + c * kChunk) * a.ld_proj + a.v_off + h * a.vdim;
       constexpr int kVPieces = VS / 8;
 #pragma unroll
-      for (int i = threadIdx.x; i < kChunk * kVPieces; i += 256) {
+      for (int i = threadIdx.x; i < kChunk * kVPieces; i += kScan) {
         const int t = i / kVPieces, e = i % kVPieces * 8;
         const bool ok = t < m && c0 + e < a.vdim;
         copy16(sm.v[b] + t * PV + e, rows + static_cast<size_t>(ok ? t : 0) * a.ld_proj + (ok ? c0 + e : 0), ok);
@@ -255,7 +258,7 @@ gated_linear_scan_kernel(XpGatedLinearArgs a) {
 #pragma unroll
         for (int p = 0; p < 2; ++p)
 #pragma unroll
-          for (int i = threadIdx.x; i < kChunk * 8; i += 256) {
+          for (int i = threadIdx.x; i < kChunk * 8; i += kScan) {
             const int t = i >> 3, e = (i & 7) * 8;
             if (e / 16 <= t / 16) copy16(sm.a[b][p] + t * kPC + e, rec->a[p] + t * kChunk + e, true);   // lower blocks only
           }
@@ -266,7 +269,8 @@ gated_linear_scan_kernel(XpGatedLinearArgs a) {
   issue_tiles(0);
   copies_issued();
 
-  const int d0 = D >= 128 ? warp * 16 : (warp & 3) * 16, s0 = D >= 128 ? 0 : (warp >> 2) * (VS / 2);
+  const int d0 = warp % kRowWarps * 16, s0 = warp / kRowWarps * (NS * 8);
+  const bool has_state = warp / kRowWarps < kState;
   const size_t state_elems = static_cast<size_t>(a.dim) * a.vdim;
   float* slot = a.state + (static_cast<size_t>(a.state_slots[seq]) * a.heads + h) * state_elems;
   // segments: state before (or what is added) [dim][vdim], then log2 of the decay [dim]
@@ -280,11 +284,12 @@ gated_linear_scan_kernel(XpGatedLinearArgs a) {
     for (int r = 0; r < 2; ++r) {
       const int d = d0 + g + r * 8, c = c0 + s0 + j * 8 + q4 * 2;
       float2 x = make_float2(0.f, 0.f);
-      if (!zero && d < a.dim && c < a.vdim) x = make_float2(from[static_cast<size_t>(d) * a.vdim + c], from[static_cast<size_t>(d) * a.vdim + c + 1]);
+      if (has_state && !zero && d < a.dim && c < a.vdim) x = make_float2(from[static_cast<size_t>(d) * a.vdim + c], from[static_cast<size_t>(d) * a.vdim + c + 1]);
       s[j][2 * r] = x.x;
       s[j][2 * r + 1] = x.y;
     }
   auto publish = [&]() {
+    if (!has_state) return;
 #pragma unroll
     for (int j = 0; j < NS; ++j)
 #pragma unroll
@@ -299,34 +304,32 @@ gated_linear_scan_kernel(XpGatedLinearArgs a) {
   if (kFull) publish();
   float log_total = 0.f;                             // thread d: log2 of channel d's decay over the segment
 
-  const int rw = warp & 3, o0 = (warp >> 2) * (VS / 2);
+  const int rw = warp & 3, o0 = (warp >> 2) * (NO * 8);
   for (int c = 0; c < chunks; ++c) {
     const int b = c & 1, m = min(kChunk, n - c * kChunk);
     copies_wait<0>();
     __syncthreads();                                 // chunk c landed, state published, everything of chunk c - 1 used
     // ---- decay queries and keys
-    constexpr int kPieces = D / 8;
-    for (int i = threadIdx.x; i < kChunk * kPieces; i += 256) {
-      const int t = i / kPieces, e = i % kPieces * 8;
-      float x[8];
-      uint4 hi, lo;
-      float cc[8];
-      *reinterpret_cast<float4*>(cc) = *reinterpret_cast<const float4*>(sm.c_in + t * D + e);
-      *reinterpret_cast<float4*>(cc + 4) = *reinterpret_cast<const float4*>(sm.c_in + t * D + e + 4);
-      if (kFull) {
-        recur::ldx<8>(sm.q_in + t * D + e, x);
-#pragma unroll
-        for (int j = 0; j < 8; ++j) x[j] *= a.qscale * sm100::ex2_approx(cc[j]);
-        split2(x[0], x[1], hi.x, lo.x), split2(x[2], x[3], hi.y, lo.y), split2(x[4], x[5], hi.z, lo.z), split2(x[6], x[7], hi.w, lo.w);
-        *reinterpret_cast<uint4*>(sm.q[0] + t * PD + e) = hi;
-        *reinterpret_cast<uint4*>(sm.q[1] + t * PD + e) = lo;
+    {
+      constexpr int kPairs = D / 2, kRows = kScan / kPairs;
+      const int e = threadIdx.x % kPairs * 2;
+      const float2 end = *reinterpret_cast<const float2*>(sm.c_in + (m - 1) * D + e);
+#pragma unroll 4
+      for (int t = threadIdx.x / kPairs; t < kChunk; t += kRows) {
+        const float2 cc = *reinterpret_cast<const float2*>(sm.c_in + t * D + e);
+        uint32_t hi, lo;
+        if (kFull) {
+          const float2 x = unpack2(*reinterpret_cast<const uint32_t*>(sm.q_in + t * D + e));
+          split2(x.x * (a.qscale * sm100::ex2_approx(cc.x)), x.y * (a.qscale * sm100::ex2_approx(cc.y)), hi, lo);
+          *reinterpret_cast<uint32_t*>(sm.q[0] + t * PD + e) = hi;
+          *reinterpret_cast<uint32_t*>(sm.q[1] + t * PD + e) = lo;
+        }
+        const float2 x = unpack2(*reinterpret_cast<const uint32_t*>(sm.k_in + t * D + e));   // zeros behind the portion
+        const bool in = t < m;
+        split2(in ? x.x * sm100::ex2_approx(end.x - cc.x) : 0.f, in ? x.y * sm100::ex2_approx(end.y - cc.y) : 0.f, hi, lo);
+        *reinterpret_cast<uint32_t*>(sm.k[0] + t * PD + e) = hi;
+        *reinterpret_cast<uint32_t*>(sm.k[1] + t * PD + e) = lo;
       }
-      recur::ldx<8>(sm.k_in + t * D + e, x);         // zeros behind the portion
-#pragma unroll
-      for (int j = 0; j < 8; ++j) x[j] *= t < m ? sm100::ex2_approx(sm.c_in[(m - 1) * D + e + j] - cc[j]) : 0.f;
-      split2(x[0], x[1], hi.x, lo.x), split2(x[2], x[3], hi.y, lo.y), split2(x[4], x[5], hi.z, lo.z), split2(x[6], x[7], hi.w, lo.w);
-      *reinterpret_cast<uint4*>(sm.k[0] + t * PD + e) = hi;
-      *reinterpret_cast<uint4*>(sm.k[1] + t * PD + e) = lo;
     }
     if (threadIdx.x < D) {
       const float x = sm.c_in[(m - 1) * D + threadIdx.x];
@@ -339,80 +342,86 @@ gated_linear_scan_kernel(XpGatedLinearArgs a) {
     copies_issued();
     const uint32_t vb = sm100::smem_u32(sm.v[b]) + bt_lane(lane, PV);
     if constexpr (kFull) {
-      float o[NO][4];
+      if (warp >> 2 < kOut) {
+        float o[2][NO][4];                           // two chains of sums
 #pragma unroll
-      for (int j = 0; j < NO; ++j)
+        for (int p = 0; p < 2; ++p)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) o[j][e] = 0.f;
-      const uint32_t qh_a = sm100::smem_u32(sm.q[0] + rw * 16 * PD) + a_lane(lane, PD), ql_a = sm100::smem_u32(sm.q[1] + rw * 16 * PD) + a_lane(lane, PD);
-      const uint32_t sh = sm100::smem_u32(sm.s[0] + o0) + bt_lane(lane, PV), sl = sm100::smem_u32(sm.s[1] + o0) + bt_lane(lane, PV);
-#pragma unroll 2
-      for (int ks = 0; ks < D / 16; ++ks) {
-        uint32_t qh[4], ql[4];
-        ldsm4(qh_a + ks * 32, qh);
-        ldsm4(ql_a + ks * 32, ql);
+          for (int j = 0; j < NO; ++j)
 #pragma unroll
-        for (int j = 0; j < NO; j += 2) {
-          uint32_t hi[4], lo[4];
-          ldsm4t(sh + (ks * 16 * PV + j * 8) * 2, hi);
-          ldsm4t(sl + (ks * 16 * PV + j * 8) * 2, lo);
-          mma(o[j], qh, hi[0], hi[1]);
-          mma(o[j + 1], qh, hi[2], hi[3]);
-          mma(o[j], qh, lo[0], lo[1]);
-          mma(o[j + 1], qh, lo[2], lo[3]);
-          mma(o[j], ql, hi[0], hi[1]);
-          mma(o[j + 1], ql, hi[2], hi[3]);
-        }
-      }
-      const uint32_t ah_a = sm100::smem_u32(sm.a[b][0] + rw * 16 * kPC) + a_lane(lane, kPC), al_a = sm100::smem_u32(sm.a[b][1] + rw * 16 * kPC) + a_lane(lane, kPC);
-#pragma unroll
-      for (int ks = 0; ks < 4; ++ks) {
-        if (ks <= rw) {
-          uint32_t ah[4], al[4];
-          ldsm4(ah_a + ks * 32, ah);
-          ldsm4(al_a + ks * 32, al);
+            for (int e = 0; e < 4; ++e) o[p][j][e] = 0.f;
+        const uint32_t qh_a = sm100::smem_u32(sm.q[0] + rw * 16 * PD) + a_lane(lane, PD), ql_a = sm100::smem_u32(sm.q[1] + rw * 16 * PD) + a_lane(lane, PD);
+        const uint32_t sh = sm100::smem_u32(sm.s[0] + o0) + bt_lane(lane, PV), sl = sm100::smem_u32(sm.s[1] + o0) + bt_lane(lane, PV);
+#pragma unroll 4
+        for (int ks = 0; ks < D / 16; ++ks) {
+          uint32_t qh[4], ql[4];
+          ldsm4(qh_a + ks * 32, qh);
+          ldsm4(ql_a + ks * 32, ql);
 #pragma unroll
           for (int j = 0; j < NO; j += 2) {
-            uint32_t vf[4];
-            ldsm4t(vb + (ks * 16 * PV + o0 + j * 8) * 2, vf);
-            mma(o[j], ah, vf[0], vf[1]);
-            mma(o[j + 1], ah, vf[2], vf[3]);
-            mma(o[j], al, vf[0], vf[1]);
-            mma(o[j + 1], al, vf[2], vf[3]);
+            uint32_t hi[4], lo[4];
+            ldsm4t(sh + (ks * 16 * PV + j * 8) * 2, hi);
+            ldsm4t(sl + (ks * 16 * PV + j * 8) * 2, lo);
+            mma(o[0][j], qh, hi[0], hi[1]);
+            mma(o[0][j + 1], qh, hi[2], hi[3]);
+            mma(o[1][j], qh, lo[0], lo[1]);
+            mma(o[1][j + 1], qh, lo[2], lo[3]);
+            mma(o[1][j], ql, hi[0], hi[1]);
+            mma(o[1][j + 1], ql, hi[2], hi[3]);
           }
         }
-      }
+        const uint32_t ah_a = sm100::smem_u32(sm.a[b][0] + rw * 16 * kPC) + a_lane(lane, kPC), al_a = sm100::smem_u32(sm.a[b][1] + rw * 16 * kPC) + a_lane(lane, kPC);
 #pragma unroll
-      for (int j = 0; j < NO; ++j) {
-        const int col = c0 + o0 + j * 8 + q4 * 2;
+        for (int ks = 0; ks < 4; ++ks) {
+          if (ks <= rw) {
+            uint32_t ah[4], al[4];
+            ldsm4(ah_a + ks * 32, ah);
+            ldsm4(al_a + ks * 32, al);
 #pragma unroll
-        for (int r = 0; r < 2; ++r) {
-          const int i = rw * 16 + g + r * 8;
-          if (i < m && col < a.vdim)
-            *reinterpret_cast<float2*>(reinterpret_cast<float*>(a.out) + static_cast<size_t>(r0 + c * kChunk + i) * a.ld_out + h * a.vdim + col) =
-                make_float2(o[j][2 * r], o[j][2 * r + 1]);
+            for (int j = 0; j < NO; j += 2) {
+              uint32_t vf[4];
+              ldsm4t(vb + (ks * 16 * PV + o0 + j * 8) * 2, vf);
+              mma(o[0][j], ah, vf[0], vf[1]);
+              mma(o[0][j + 1], ah, vf[2], vf[3]);
+              mma(o[1][j], al, vf[0], vf[1]);
+              mma(o[1][j + 1], al, vf[2], vf[3]);
+            }
+          }
+        }
+#pragma unroll
+        for (int j = 0; j < NO; ++j) {
+          const int col = c0 + o0 + j * 8 + q4 * 2;
+#pragma unroll
+          for (int r = 0; r < 2; ++r) {
+            const int i = rw * 16 + g + r * 8;
+            if (i < m && col < a.vdim)
+              *reinterpret_cast<float2*>(reinterpret_cast<float*>(a.out) + static_cast<size_t>(r0 + c * kChunk + i) * a.ld_out + h * a.vdim + col) =
+                  make_float2(o[0][j][2 * r] + o[1][j][2 * r], o[0][j][2 * r + 1] + o[1][j][2 * r + 1]);
+          }
         }
       }
       if (c + 1 == chunks && !last) break;           // the next segment has its own start state
       __syncthreads();                               // everyone is done with the published state
     }
-    const float e0 = sm.dec[d0 + g], e1 = sm.dec[d0 + g + 8];
+    if (has_state) {
+      const float e0 = sm.dec[d0 + g], e1 = sm.dec[d0 + g + 8];
 #pragma unroll
-    for (int j = 0; j < NS; ++j) s[j][0] *= e0, s[j][1] *= e0, s[j][2] *= e1, s[j][3] *= e1;
-    const uint32_t kh_a = sm100::smem_u32(sm.k[0] + d0) + at_lane(lane, PD), kl_a = sm100::smem_u32(sm.k[1] + d0) + at_lane(lane, PD);
+      for (int j = 0; j < NS; ++j) s[j][0] *= e0, s[j][1] *= e0, s[j][2] *= e1, s[j][3] *= e1;
+      const uint32_t kh_a = sm100::smem_u32(sm.k[0] + d0) + at_lane(lane, PD), kl_a = sm100::smem_u32(sm.k[1] + d0) + at_lane(lane, PD);
 #pragma unroll
-    for (int ks = 0; ks < 4; ++ks) {
-      uint32_t kh[4], kl[4];
-      ldsm4t(kh_a + ks * 16 * PD * 2, kh);
-      ldsm4t(kl_a + ks * 16 * PD * 2, kl);
+      for (int ks = 0; ks < 4; ++ks) {
+        uint32_t kh[4], kl[4];
+        ldsm4t(kh_a + ks * 16 * PD * 2, kh);
+        ldsm4t(kl_a + ks * 16 * PD * 2, kl);
 #pragma unroll
-      for (int j = 0; j < NS; j += 2) {
-        uint32_t vf[4];
-        ldsm4t(vb + (ks * 16 * PV + s0 + j * 8) * 2, vf);
-        mma(s[j], kh, vf[0], vf[1]);
-        mma(s[j + 1], kh, vf[2], vf[3]);
-        mma(s[j], kl, vf[0], vf[1]);
-        mma(s[j + 1], kl, vf[2], vf[3]);
+        for (int j = 0; j < NS; j += 2) {
+          uint32_t vf[4];
+          ldsm4t(vb + (ks * 16 * PV + s0 + j * 8) * 2, vf);
+          mma(s[j], kh, vf[0], vf[1]);
+          mma(s[j + 1], kh, vf[2], vf[3]);
+          mma(s[j], kl, vf[0], vf[1]);
+          mma(s[j + 1], kl, vf[2], vf[3]);
+        }
       }
     }
     if (kFull && c + 1 < chunks) publish();
@@ -425,7 +434,7 @@ gated_linear_scan_kernel(XpGatedLinearArgs a) {
 #pragma unroll
     for (int r = 0; r < 2; ++r) {
       const int d = d0 + g + r * 8, c = c0 + s0 + j * 8 + q4 * 2;
-      if (d < a.dim && c < a.vdim) {
+      if (has_state && d < a.dim && c < a.vdim) {
         to[static_cast<size_t>(d) * a.vdim + c] = s[j][2 * r];
         to[static_cast<size_t>(d) * a.vdim + c + 1] = s[j][2 * r + 1];
       }
@@ -473,10 +482,10 @@ int launch(const XpGatedLinearArgs& a, cudaStream_t s) {
   gated_linear_chunk_kernel<D><<<dim3((a.max_q + kChunk - 1) / kChunk, a.heads, a.seqs), 256, kChunkBytes, s>>>(b);
   const dim3 grid((a.vdim + VS - 1) / VS * b.segs, a.heads, a.seqs);
   if (b.segs > 1) {
-    gated_linear_scan_kernel<D, VS, false><<<grid, 256, kScanBytes, s>>>(b);
+    gated_linear_scan_kernel<D, VS, false><<<grid, kScan, kScanBytes, s>>>(b);
     gated_linear_segments_kernel<<<dim3((a.dim * a.vdim + 255) / 256, a.heads, a.seqs), 256, 0, s>>>(b);
   }
-  gated_linear_scan_kernel<D, VS, true><<<grid, 256, kScanBytes, s>>>(b);
+  gated_linear_scan_kernel<D, VS, true><<<grid, kScan, kScanBytes, s>>>(b);
   cudaError_t e = cudaGetLastError();
   return e == cudaSuccess ? 0 : -100 - static_cast<int>(e);
 }

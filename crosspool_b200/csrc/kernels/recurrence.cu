@@ -392,16 +392,20 @@ sequential_kernel(A a) {
 
 // ------------------------------------------------------------------------------------------ delta rule: in front of the recurrence
 // CTA = (kPrepRows rows, one head of queries, keys or values, portion): convolution and silu, and for queries and keys the sum
-// of squares per row. A thread walks kRun rows of VEC channels. The last CTA column computes beta and log g. The CTA of a
-// portion's first rows is the only one that reads the ring (a window reaches back less than kPrepRows rows) and puts the
-// portion's last inputs into it when it is done.
-constexpr int kPrepRows = 64;
+// of squares per row. A thread takes kRun rows of VEC channels, all of its inputs in flight at once. The last CTA column
+// computes beta and log g. The CTA of a portion's first rows is the only one that reads the ring (a window reaches back less
+// than kPrepRows rows) and puts the portion's last inputs into it when it is done.
+constexpr int kPrepRows = 128;
 constexpr int kRun = 8;
 
-template <typename T, int VEC>
-__global__ void __launch_bounds__(kThreads)
+__device__ __forceinline__ void conv_out(float* p, float y) { *p = silu(y); }
+__device__ __forceinline__ void conv_out(__nv_bfloat16* p, float y) { *p = __float2bfloat16_rn(__fdividef(y, 1.f + __expf(-y))); }
+
+// TAPS = 0: any number, inputs read again for every output
+template <typename T, int VEC, int TAPS>
+__global__ void __launch_bounds__(kThreads, 2)
 delta_prep_kernel(XpDeltaArgs a) {
-  extern __shared__ float sm[];            // sums of squares [kPrepRows][vector columns]
+  extern __shared__ float sm[];            // sums of squares [kPrepRows][vector columns + 1]
   const int seq = blockIdx.z, n = a.q_lens[seq], t0 = blockIdx.x * kPrepRows;
   if (t0 >= n) return;
   const int rows = min(kPrepRows, n - t0), r0 = a.q_starts[seq] + t0;
@@ -427,56 +431,66 @@ delta_prep_kernel(XpDeltaArgs a) {
   const int vecs = width / VEC, runs = (rows + kRun - 1) / kRun;
   for (int w = threadIdx.x; w < vecs * runs; w += kThreads) {
     const int c = w % vecs * VEC, first = w / vecs * kRun;
-    const int last = min(first + kRun, rows);
-    auto input = [&](int t, float (&x)[VEC]) {       // row t of the tile, or what came before it
-      if (t0 + t >= 0) {
-        ldx<VEC>(x0 + static_cast<int64_t>(t) * a.ld_proj + c, x);
-      } else if (pos0 + t >= 0) {
-        ldx<VEC>(ring + static_cast<size_t>((pos0 + t) % a.taps) * channels + ch0 + c, x);
+    auto input = [&](int t, T (&x)[VEC]) {           // row t of the tile, or what came before it
+      const T* p = nullptr;
+      if (t0 + t >= 0) p = t < rows ? x0 + static_cast<int64_t>(t) * a.ld_proj : nullptr;
+      else if (pos0 + t >= 0) p = ring + static_cast<size_t>((pos0 + t) % a.taps) * channels + ch0;
+      if (p != nullptr) {
+        ldr<VEC>(p + c, x);
       } else {
 #pragma unroll
-        for (int j = 0; j < VEC; ++j) x[j] = 0.f;
+        for (int j = 0; j < VEC; ++j) st(&x[j], 0.f);
       }
     };
-    auto finish = [&](int t, float (&y)[VEC]) {
+    auto finish = [&](int t, const float (&y)[VEC]) {
+      if (t >= rows) return;
       float ss = 0.f;
       T r[VEC];
 #pragma unroll
       for (int j = 0; j < VEC; ++j) {
-        st(&r[j], silu(y[j]));
+        conv_out(&r[j], y[j]);
         const float f = ld(&r[j]);
         ss += f * f;
       }
       stx<VEC>(qkv + static_cast<size_t>(t) * channels + c, r);
-      if (!is_v) sm[t * vecs + w % vecs] = ss;
+      if (!is_v) sm[t * (vecs + 1) + w % vecs] = ss;
     };
-    if (a.taps == 4) {                               // window and weights in registers
-      float wt[4][VEC], b0[VEC], b1[VEC], b2[VEC], b3[VEC];
+    if constexpr (TAPS > 0) {
+      T x[kRun + TAPS - 1][VEC];
 #pragma unroll
-      for (int j = 0; j < VEC; ++j)
+      for (int i = 0; i < kRun + TAPS - 1; ++i) input(first + i - (TAPS - 1), x[i]);
+      float wt[VEC][TAPS];
 #pragma unroll
-        for (int k = 0; k < 4; ++k) wt[k][j] = a.conv_w[static_cast<size_t>(ch0 + c + j) * 4 + k];
-      input(first - 3, b0), input(first - 2, b1), input(first - 1, b2);
-      for (int t = first; t < last; ++t) {
-        input(t, b3);
+      for (int j = 0; j < VEC; ++j) {
+        if constexpr (TAPS == 4) {
+          const float4 f = *reinterpret_cast<const float4*>(a.conv_w + static_cast<size_t>(ch0 + c + j) * 4);
+          wt[j][0] = f.x, wt[j][1] = f.y, wt[j][2] = f.z, wt[j][3] = f.w;
+        } else {
+#pragma unroll
+          for (int k = 0; k < TAPS; ++k) wt[j][k] = a.conv_w[static_cast<size_t>(ch0 + c + j) * TAPS + k];
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < kRun; ++i) {
         float y[VEC];
 #pragma unroll
         for (int j = 0; j < VEC; ++j) {
-          y[j] = fmaf(wt[0][j], b0[j], fmaf(wt[1][j], b1[j], fmaf(wt[2][j], b2[j], wt[3][j] * b3[j])));
-          b0[j] = b1[j], b1[j] = b2[j], b2[j] = b3[j];
+          y[j] = 0.f;
+#pragma unroll
+          for (int k = 0; k < TAPS; ++k) y[j] = fmaf(wt[j][k], ld(&x[i + k][j]), y[j]);
         }
-        finish(t, y);
+        finish(first + i, y);
       }
     } else {
-      for (int t = first; t < last; ++t) {
+      for (int t = first; t < min(first + kRun, rows); ++t) {
         float y[VEC];
 #pragma unroll
         for (int j = 0; j < VEC; ++j) y[j] = 0.f;
         for (int k = 0; k < a.taps; ++k) {
-          float x[VEC];
+          T x[VEC];
           input(t - k, x);
 #pragma unroll
-          for (int j = 0; j < VEC; ++j) y[j] = fmaf(a.conv_w[static_cast<size_t>(ch0 + c + j) * a.taps + a.taps - 1 - k], x[j], y[j]);
+          for (int j = 0; j < VEC; ++j) y[j] = fmaf(a.conv_w[static_cast<size_t>(ch0 + c + j) * a.taps + a.taps - 1 - k], ld(&x[j]), y[j]);
         }
         finish(t, y);
       }
@@ -487,7 +501,7 @@ delta_prep_kernel(XpDeltaArgs a) {
     const bool is_q = u < a.kv_heads;
     for (int t = threadIdx.x; t < rows; t += kThreads) {
       float ss = 0.f;
-      for (int i = 0; i < vecs; ++i) ss += sm[t * vecs + i];
+      for (int i = 0; i < vecs; ++i) ss += sm[t * (vecs + 1) + i];
       a.qk_scale[static_cast<size_t>(r0 + t) * 2 * a.kv_heads + u] = (is_q ? a.qscale : 1.f) * rsqrtf(ss + kUnitEps);
     }
   }
@@ -564,13 +578,23 @@ int sequential_any(const A& a, cudaStream_t s) {
 
 inline bool aligned(const void* p, size_t n) { return reinterpret_cast<uintptr_t>(p) % n == 0; }
 
+template <typename T, int VEC, int TAPS>
+int launch_prep_taps(const XpDeltaArgs& a, cudaStream_t s) {
+  const size_t sm = static_cast<size_t>(kPrepRows) * (a.dim / VEC + 1) * 4;
+  const int rc = big_smem(delta_prep_kernel<T, VEC, TAPS>, sm);
+  if (rc != 0) return rc;
+  delta_prep_kernel<T, VEC, TAPS><<<dim3((a.max_q + kPrepRows - 1) / kPrepRows, 2 * a.kv_heads + a.heads + 1, a.seqs), kThreads, sm, s>>>(a);
+  return done();
+}
+
 template <typename T, int VEC>
 int launch_prep(const XpDeltaArgs& a, cudaStream_t s) {
-  const size_t sm = static_cast<size_t>(kPrepRows) * (a.dim / VEC) * 4;
-  const int rc = big_smem(delta_prep_kernel<T, VEC>, sm);
-  if (rc != 0) return rc;
-  delta_prep_kernel<T, VEC><<<dim3((a.max_q + kPrepRows - 1) / kPrepRows, 2 * a.kv_heads + a.heads + 1, a.seqs), kThreads, sm, s>>>(a);
-  return done();
+  if constexpr (VEC > 1) {
+    if (a.taps == 4 && aligned(a.conv_w, 16)) return launch_prep_taps<T, VEC, 4>(a, s);
+    if (a.taps == 3) return launch_prep_taps<T, VEC, 3>(a, s);
+    if (a.taps == 2) return launch_prep_taps<T, VEC, 2>(a, s);
+  }
+  return launch_prep_taps<T, VEC, 0>(a, s);
 }
 
 inline bool delta_ok(const XpDeltaArgs& a) {
