@@ -457,8 +457,14 @@ delta_prep_kernel(XpDeltaArgs a) {
     };
     if constexpr (TAPS > 0) {
       T x[kRun + TAPS - 1][VEC];
+      if (t0 + first >= TAPS - 1 && first + kRun <= rows) {      // no branch between the loads
+        const T* p = x0 + static_cast<int64_t>(first - (TAPS - 1)) * a.ld_proj + c;
 #pragma unroll
-      for (int i = 0; i < kRun + TAPS - 1; ++i) input(first + i - (TAPS - 1), x[i]);
+        for (int i = 0; i < kRun + TAPS - 1; ++i) ldr<VEC>(p + static_cast<int64_t>(i) * a.ld_proj, x[i]);
+      } else {
+#pragma unroll
+        for (int i = 0; i < kRun + TAPS - 1; ++i) input(first + i - (TAPS - 1), x[i]);
+      }
       float wt[VEC][TAPS];
 #pragma unroll
       for (int j = 0; j < VEC; ++j) {
