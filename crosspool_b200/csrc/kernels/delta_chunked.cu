@@ -30,7 +30,7 @@ struct __align__(16) Record {
   float read_k[kChunk];                    // e^(c_i) b_i
   float read_q[kChunk];                    // e^(c_i) a_i
   float write[kChunk];                     // b_j e^(c_n - c_j)
-  float decay[4];                          // e^(c_n)
+  float decay[4];                          // e^(c_n), four times
 };
 
 // Records of a sequence start here: distinct for all chunks of a batch of packed portions.
@@ -141,17 +141,19 @@ delta_chunk_kernel(XpDeltaArgs a) {
     rec->read_k[t] = e * fb[t];
     rec->read_q[t] = e * fa[t];
     rec->write[t] = fb[t] * expf(cum[kChunk - 1] - cum[t]);
-    if (t == 0) rec->decay[0] = expf(cum[kChunk - 1]);
+    if (t < 4) rec->decay[t] = expf(cum[kChunk - 1]);
   }
   __syncthreads();
-  // Column t of (1 + L)^-1 by forward substitution, thread = column.
-  if (threadIdx.x < kChunk) {
-    const int t = threadIdx.x;
-    float x[kChunk];
+  // (1 + L)^-1 in halves of 32: the diagonal blocks by forward substitution (thread = column), T21 = -T22 (L21 T11) by all.
+  constexpr int kHalf = 32, PT = kHalf + 1;
+  float (*t_s)[kHalf][PT] = reinterpret_cast<float (*)[kHalf][PT]>(q_s);   // T11, T22, L21 T11, over the queries and keys
+  if (warp < 2) {
+    const float* base = l_s + warp * kHalf * PL + warp * kHalf;
+    float x[kHalf];
 #pragma unroll
-    for (int i = 0; i < kChunk; ++i) {
-      float s[4] = {i == t ? 1.f : 0.f, 0.f, 0.f, 0.f};
-      const float4* row = reinterpret_cast<const float4*>(l_s + i * PL);
+    for (int i = 0; i < kHalf; ++i) {
+      float s[4] = {i == lane ? 1.f : 0.f, 0.f, 0.f, 0.f};
+      const float4* row = reinterpret_cast<const float4*>(base + i * PL);
 #pragma unroll
       for (int m4 = 0; m4 < (i + 3) / 4; ++m4) {     // L is zero on and above the diagonal
         const float4 v = row[m4];
@@ -161,15 +163,45 @@ delta_chunk_kernel(XpDeltaArgs a) {
         s[3] = fmaf(-v.w, m4 * 4 + 3 < i ? x[m4 * 4 + 3] : 0.f, s[3]);
       }
       x[i] = (s[0] + s[1]) + (s[2] + s[3]);
+      t_s[warp][i][lane] = x[i];
     }
-    const float b = beta[t];
+  }
+  __syncthreads();
+  const int i1 = warp * 8;                           // eight rows of the lower left block, column = lane
+  float x[8];
 #pragma unroll
-    for (int i = 0; i < kChunk; ++i) {
-      const float v = x[i] * b;
-      const __nv_bfloat16 hi = __float2bfloat16_rn(v);
-      rec->t[0][i * kChunk + t] = hi;
-      rec->t[1][i * kChunk + t] = __float2bfloat16_rn(v - __bfloat162float(hi));
+  for (int r = 0; r < 8; ++r) x[r] = 0.f;
+#pragma unroll
+  for (int m = 0; m < kHalf; m += 4) {
+    const float y0 = t_s[0][m][lane], y1 = t_s[0][m + 1][lane], y2 = t_s[0][m + 2][lane], y3 = t_s[0][m + 3][lane];
+#pragma unroll
+    for (int r = 0; r < 8; ++r) {
+      const float4 v = *reinterpret_cast<const float4*>(l_s + (kHalf + i1 + r) * PL + m);
+      x[r] = fmaf(v.x, y0, fmaf(v.y, y1, fmaf(v.z, y2, fmaf(v.w, y3, x[r]))));
     }
+  }
+#pragma unroll
+  for (int r = 0; r < 8; ++r) t_s[2][i1 + r][lane] = x[r];
+  __syncthreads();
+#pragma unroll
+  for (int r = 0; r < 8; ++r) x[r] = 0.f;
+#pragma unroll 8
+  for (int m = 0; m < kHalf; ++m) {
+    const float y = t_s[2][m][lane];
+#pragma unroll
+    for (int r = 0; r < 8; ++r) x[r] = fmaf(-t_s[1][i1 + r][m], y, x[r]);
+  }
+  auto store_t = [&](int i, int t, float v) {
+    v *= beta[t];
+    const __nv_bfloat16 hi = __float2bfloat16_rn(v);
+    rec->t[0][i * kChunk + t] = hi;
+    rec->t[1][i * kChunk + t] = __float2bfloat16_rn(v - __bfloat162float(hi));
+  };
+#pragma unroll
+  for (int r = 0; r < 8; ++r) {
+    store_t(i1 + r, lane, t_s[0][i1 + r][lane]);
+    store_t(kHalf + i1 + r, lane, x[r]);
+    store_t(kHalf + i1 + r, kHalf + lane, t_s[1][i1 + r][lane]);
   }
 }
 
@@ -183,7 +215,7 @@ struct ScanSmem {
   __nv_bfloat16 w[2][kChunk * PV];         // writes, scaled for the state
   __nv_bfloat16 u[2][2][kChunk * PV];      // writes of chunk c in buffer c & 1
   float f[2][3][kChunk];
-  float decay[2];
+  float decay[2][4];
 };
 
 __device__ __forceinline__ void chain_sync() { asm volatile("bar.sync 1, 256;" ::: "memory"); }
@@ -229,19 +261,20 @@ delta_scan_kernel(XpDeltaArgs a) {
 
   auto issue_matrix = [&](__nv_bfloat16 (&dst)[2][kChunk * kPC], const __nv_bfloat16 (&src)[2][kChunk * kChunk]) {
 #pragma unroll
-    for (int i = threadIdx.x; i < 2 * kChunk * 8; i += 512) {
+    for (int i = threadIdx.x - 256; i < 2 * kChunk * 8; i += 256) {
       const int p = i >> 9, t = (i >> 3) & 63, e = (i & 7) * 8;
       if (e / 16 <= t / 16) copy16(dst[p] + t * kPC + e, src[p] + t * kChunk + e, true);   // blocks above the diagonal are never read
     }
   };
-  // rows, T and factors of chunk c, M of the chunk before
+  // rows, T and factors of chunk c, M of the chunk before; by the warps off the chain
   auto issue = [&](int c) {
+    if (chain) return;
     if (c < chunks) {
       const int b = c & 1, m = min(kChunk, n - c * kChunk);
       const __nv_bfloat16* rows = qkv + static_cast<size_t>(c) * kChunk * channels + hk * a.dim;
       constexpr int kPieces = D / 8;
 #pragma unroll
-      for (int i = threadIdx.x; i < kChunk * kPieces; i += 512) {
+      for (int i = threadIdx.x - 256; i < kChunk * kPieces; i += 256) {
         const int t = i / kPieces, e = i % kPieces * 8;
         const bool ok = t < m && e < a.dim;
         const __nv_bfloat16* src = rows + static_cast<size_t>(ok ? t : 0) * channels + (ok ? e : 0);
@@ -250,8 +283,9 @@ delta_scan_kernel(XpDeltaArgs a) {
       }
       const Record* rec = recs + static_cast<size_t>(c) * a.heads;
       issue_matrix(sm.t[b], rec->t);
-      if (threadIdx.x < 48) copy16(&sm.f[b][0][0] + threadIdx.x * 4, rec->read_k + threadIdx.x * 4, true);   // three arrays in a row
-      if (threadIdx.x == 64) sm.decay[b] = rec->decay[0];
+      const int i = threadIdx.x - 256;
+      if (i < 48) copy16(&sm.f[b][0][0] + i * 4, rec->read_k + i * 4, true);     // three arrays in a row
+      if (i == 64) copy16(sm.decay[b], rec->decay, true);
     }
     if (c > 0 && c <= chunks) issue_matrix(sm.m[(c - 1) & 1], recs[static_cast<size_t>(c - 1) * a.heads].m);
     copies_issued();
@@ -432,7 +466,7 @@ delta_scan_kernel(XpDeltaArgs a) {
       }
     chain_sync();
     // ---- state
-    const float dec = sm.decay[b];
+    const float dec = sm.decay[b][0];
     const uint32_t kt = sm100::smem_u32(sm.k[b] + d0) + at_lane(lane, PD);
     const uint32_t w_hi = sm100::smem_u32(sm.w[0] + s0) + bt_lane(lane, PV), w_lo = sm100::smem_u32(sm.w[1] + s0) + bt_lane(lane, PV);
 #pragma unroll
