@@ -8,7 +8,7 @@
 #include <stddef.h>
 #include <stdint.h>
 
-#define XP_ABI_VERSION 23
+#define XP_ABI_VERSION 24
 
 #ifdef __cplusplus
 extern "C" {
@@ -27,11 +27,11 @@ typedef struct XpGemmArgs {
   size_t ws_bytes;
   size_t counter_bytes;
   int w_rows_total;    /* 0: derived from n_out / up_offset */
-  int n_out;           /* features produced (multiple of 128 in the dual, tiled, grouped and fp8 forms) */
+  int n_out;           /* features produced (multiple of 128 in the tiled and fp8 forms) */
   int k;               /* row pitches are multiples of 16 bytes (multiple of 64 elements in the forms above) */
   int rows;
   int ldw, ldx, ld_out, ld_resid; /* element strides; 0 = dense */
-  int epilogue;        /* 0 store bf16, 1 swiglu (dual), 2 residual add, 3 store fp32 */
+  int epilogue;        /* 0 store bf16, 1 swiglu (dual), 2 residual add, 3 store fp32, 4 act(value) * resid[ids[row]] */
   int dual;
   int up_offset;       /* first weight row of the up projection */
   int splits;          /* 0 = choose */
@@ -55,6 +55,11 @@ typedef struct XpGemmArgs {
   int batch, x_group_rows, out_group_stride;
   float out_scale;     /* multiplies the accumulator of epilogues 0 and 3; 0 = 1 */
   int silu_cols;       /* epilogues 0 and 3: features below this are stored as silu(value) */
+  float act_cubic;     /* the activation of epilogues 1 and 4: g sigmoid(act_alpha g (1 + act_cubic g^2)) */
+  int ids_limit;       /* epilogue 4: rows of the table; ids outside read row 0 */
+  const int* ids;      /* epilogue 4: [rows] */
+  float* tail;         /* epilogue 0: features from tail_from on are stored here in fp32 instead, [rows, ld_tail] */
+  int tail_from, ld_tail;
 } XpGemmArgs;
 
 typedef struct XpGemmPlan {
@@ -225,6 +230,24 @@ typedef struct XpRouteArgs {
   int tm_gateup, bn_gateup, tm_down, bn_down;
 } XpRouteArgs;
 
+/* out[t] = sum over k (in order) of weights[t, k] * (y[route_pos[t, k]], or x[t] where topk_ids[t, k] >= experts)
+ *          + sigmoid(shared_gate[t]) * shared[t] */
+typedef struct XpMoeMixArgs {
+  const void* y;                /* [routes, ld_y] expert outputs in route order */
+  const void* x;                /* [rows, ld_x] the layer's input */
+  const void* shared;           /* optional [rows, ld_shared] */
+  const float* shared_gate;     /* logits, row t at t * ld_gate */
+  const int* topk_ids;          /* [rows, top_k] */
+  const int* route_pos;         /* [rows, top_k], -1: not an expert */
+  const float* weights;         /* [rows, top_k] */
+  void* out;                    /* [rows, ld_out] */
+  int rows, top_k, hidden, experts, ld_y, ld_x, ld_shared, ld_gate, ld_out;
+  int f32;                      /* element type: 0 bf16, 1 fp32 */
+} XpMoeMixArgs;
+
+int xp_moe_mix(const XpMoeMixArgs* a, void* stream);
+/* xp_router_topk and xp_moe_route in one launch, for few rows (at most 128). */
+int xp_moe_topk_route(const XpRouterArgs* a, const XpRouteArgs* r, void* stream);
 int xp_router_topk(const XpRouterArgs* a, void* stream);
 /* Router projection with IEEE fp32 accumulation: x bf16 [rows, ldx], w [experts, hidden] bf16 (w_fp32 = 0) or fp32. */
 int xp_router_fp32(const void* x, int ldx, const void* w, int w_fp32, float* logits, int ld_logits, int rows, int hidden,
@@ -289,6 +312,9 @@ typedef struct XpDecodeRowsArgs {
   const void* gate;           /* optional bf16 logits [rows, ld_gate]: head h's output is multiplied by sigmoid */
   int group_pad, v_dim, v_valid, ld_out, ld_gate;
   float softcap;              /* > 0: scores become softcap tanh(score / softcap) */
+  int window;                 /* > 0: a row sees the last `window` of its tokens, and the first `keep_first` */
+  int keep_first;
+  int gate_elems;             /* the gate has one logit per output element: [rows, heads * v_valid] */
 } XpDecodeRowsArgs;
 
 typedef struct XpPrefillAttnArgs {
@@ -319,6 +345,9 @@ typedef struct XpPrefillAttnArgs {
   int p_pair;                 /* probabilities as a bf16 pair in the second product */
   int group_valid;            /* > 0: query heads of a group that exist (the others are padding of q, q_heads counts them) */
   float softcap;              /* > 0: scores become softcap tanh(score / softcap) */
+  int window;                 /* > 0: a token sees the `window` tokens that end with itself, and the first `keep_first` */
+  int keep_first;
+  int gate_elems;             /* the gate has one logit per output element: [rows, heads * v_valid], rows of 16-byte units */
 } XpPrefillAttnArgs;
 
 int xp_rope_kv(const XpRopeArgs* a, void* stream);

@@ -38,6 +38,7 @@ enum Epilogue : int {
   kEpiSwiglu = 1,    // dual: out = silu(round(g)) * round(u)
   kEpiResidual = 2,  // out = round(acc) + resid
   kEpiStoreF32 = 3,  // fp32 out = acc (+ bias)
+  kEpiTokenGate = 4, // out = act(acc) * table[ids[row], f], resid being the table
 };
 
 enum Status : uint32_t {
@@ -97,6 +98,12 @@ struct Problem {
   int out_group_stride;
   int silu_cols;           // plain stores: features below this are stored as silu(value)
   float out_scale;         // multiplies the accumulator of the two plain store epilogues; 0 = 1
+  float act_cubic;         // the activation is g * sigmoid(alpha * g * (1 + cubic * g^2))
+  const int* ids;          // token of every row (kEpiTokenGate), below ids_limit
+  int ids_limit;
+  float* tail;             // kEpiStore: features from tail_from on go here in fp32, row r at r * ld_tail
+  int tail_from;
+  int ld_tail;
 };
 
 struct SmemLayout {
@@ -448,11 +455,32 @@ __device__ __forceinline__ void epilogue_store16(const Problem& p, int f, int fb
     const float bias_u = (p.bias != nullptr && p.dual && live) ? p.bias[p.up_offset + fb] : 0.f;
     const float lim = p.gate_limit > 0.f ? p.gate_limit : 3.0e38f;
     const float a = p.act_alpha == 0.f ? 1.f : p.act_alpha;
+    if (p.act_cubic != 0.f) {
+#pragma unroll
+      for (int j = 0; j < 16; ++j) {
+        const float gg = fminf(round_bf16(g[j] + bias), lim);
+        const float uu = fminf(fmaxf(round_bf16(u[j] + bias_u), -lim), lim);
+        v[j] = __fdividef(gg, 1.f + __expf(-a * gg * fmaf(p.act_cubic * gg, gg, 1.f))) * (uu + p.up_add);
+      }
+    } else {
+#pragma unroll
+      for (int j = 0; j < 16; ++j) {
+        const float gg = fminf(round_bf16(g[j] + bias), lim);
+        const float uu = fminf(fmaxf(round_bf16(u[j] + bias_u), -lim), lim);
+        v[j] = __fdividef(gg, 1.f + __expf(-a * gg)) * (uu + p.up_add);
+      }
+    }
+  } else if (p.epilogue == kEpiTokenGate) {
+    const __nv_bfloat16* table = reinterpret_cast<const __nv_bfloat16*>(p.resid) + f;
 #pragma unroll
     for (int j = 0; j < 16; ++j) {
-      const float gg = fminf(round_bf16(g[j] + bias), lim);
-      const float uu = fminf(fmaxf(round_bf16(u[j] + bias_u), -lim), lim);
-      v[j] = __fdividef(gg, 1.f + __expf(-a * gg)) * (uu + p.up_add);
+      v[j] = 0.f;
+      if (j < valid) {
+        const int id = p.ids[n_first + j];
+        const float e = __bfloat162float(table[static_cast<size_t>(id >= 0 && id < p.ids_limit ? id : 0) * p.ld_resid]);
+        const float gg = round_bf16(g[j] + bias);
+        v[j] = __fdividef(gg, 1.f + __expf(-p.act_alpha * gg * fmaf(p.act_cubic * gg, gg, 1.f))) * e;
+      }
     }
   } else if (p.epilogue == kEpiResidual) {
     const __nv_bfloat16* r = reinterpret_cast<const __nv_bfloat16*>(p.resid) + static_cast<size_t>(n_first) * p.ld_resid + f;
@@ -475,6 +503,11 @@ __device__ __forceinline__ void epilogue_store16(const Problem& p, int f, int fb
 #pragma unroll
     for (int j = 0; j < 16; ++j)
       if (j < valid) o[static_cast<size_t>(j) * p.ld_out] = v[j];
+  } else if (p.tail != nullptr && f >= p.tail_from) {
+    float* o = p.tail + static_cast<int64_t>(n_first) * p.ld_tail + (f - p.tail_from);
+#pragma unroll
+    for (int j = 0; j < 16; ++j)
+      if (j < valid) o[static_cast<size_t>(j) * p.ld_tail] = v[j];
   } else {
     __nv_bfloat16* o = reinterpret_cast<__nv_bfloat16*>(p.out) + o0;
 #pragma unroll

@@ -70,27 +70,41 @@ typedef struct XpPostNormArgs {
   int ld_branch[2];
   int ld_out, vocab;
   float eps;
+  float embed_scale;       /* ids: the table's rows are multiplied by this; 0 = 1 */
   int f32;
 } XpPostNormArgs;
 
-/* out = rmsnorm(o) * weight * silu(gate), o in fp32, the norm over each head of `dim` columns; weight shared by the heads. */
+/* out = rmsnorm(o) * weight * silu(gate), o in fp32, the norm over each head of `dim` columns. */
 typedef struct XpHeadGateArgs {
   const float* o;        /* [rows, heads * dim] */
-  const float* weight;   /* [dim] */
+  const float* weight;   /* [dim], or [heads * dim] with per_head_weight */
   const void* gate;      /* logits [rows, ld_gate] */
   void* out;             /* [rows, ld_out] */
   int rows, heads, dim, ld_o, ld_gate, ld_out;
   float eps;
   int f32;
+  int per_head_weight;
+  int sigmoid_gate;      /* sigmoid instead of silu */
 } XpHeadGateArgs;
 
-/* out = min(g, limit) sigmoid(alpha min(g, limit)) (clamp(u, +-limit) + up_add), g and u the halves of z's rows, in fp32. */
+/* out = act(min(g, limit)) (clamp(u, +-limit) + up_add), act(g) = g sigmoid(alpha g (1 + cubic g^2)), g and u the halves of
+ * z's rows, in fp32. */
 typedef struct XpGluArgs {
   const float* z;        /* [rows, ld_z]: g (cols), u (cols) */
   float* out;            /* [rows, ld_out] */
   int rows, cols, ld_z, ld_out;
-  float limit, up_add, alpha;
+  float limit, up_add, alpha, cubic;
 } XpGluArgs;
+
+/* out = act(z) * table[ids[row]], act as above, in fp32. */
+typedef struct XpTokenGateArgs {
+  const float* z;        /* [rows, ld_z] */
+  const float* table;    /* [vocab, ld_table] */
+  const int* ids;        /* [rows] */
+  float* out;            /* [rows, ld_out] */
+  int rows, cols, ld_z, ld_table, ld_out, vocab;
+  float alpha, cubic;
+} XpTokenGateArgs;
 
 /* Grouped-query attention without rotation, per token row: RMS norm of query and key heads, queries laid out
  * [rows, kv_heads, group_pad, dq], keys and values written to the cache row of the token, everything zero-padded. */
@@ -107,14 +121,37 @@ typedef struct XpGroupedPrepArgs {
   int f32;
 } XpGroupedPrepArgs;
 
+/* Between the projection and grouped-query attention: causal convolution over time of every query, key and value channel
+ * (conv_w null: none), rotary positions on the first 2 rot_pairs channels of queries and keys (pairs (i, i + rot_pairs)),
+ * queries laid out [rows, kv_heads, group_pad, dq], keys and values written to the cache row of the token, zero-padded.
+ * own_kv = 0: queries only. The convolution's inputs are kept per slot as a ring, position p in entry p % taps. */
+typedef struct XpConvRopeArgs {
+  const void* proj;      /* [rows, ld_proj]: q (heads x dim), k (kv_heads x dim), v (kv_heads x vdim) at the offsets */
+  const float* conv_w;   /* [taps, channels], channels = q, k, v; the last tap belongs to the token itself */
+  void* ring;            /* [slots, taps, channels] activations */
+  const float* rot;      /* [rot_positions, rot_pairs, 2]: cos, sin */
+  const int* positions;  /* [rows] */
+  const int* slots;      /* [rows] cache row, -1: none */
+  const int* state_slots;/* [seqs] */
+  const int* q_starts;   /* [seqs] prefill: first row */
+  const int* q_lens;     /* [seqs] prefill: rows */
+  void* k_cache;         /* [tokens, kv_heads, dq] */
+  void* v_cache;         /* [tokens, kv_heads, dv] */
+  void* q_out;
+  int rows, seqs, max_q, heads, kv_heads, group_pad, dim, vdim, dq, dv, own_kv, ld_proj, q_off, k_off, v_off, taps, rot_pairs, rot_positions;
+  int row_floats;        /* set by the library */
+  int f32;
+} XpConvRopeArgs;
+
 /* Attention of single rows against the paged cache of grouped keys and values, plain form for any sizes. Row r attends to
- * positions[r] + 1 tokens of block-table row row_seq[r]; softcap > 0: scores become softcap tanh(score / softcap). */
+ * positions[r] + 1 tokens of block-table row row_seq[r]; softcap > 0: scores become softcap tanh(score / softcap); window >
+ * 0: only to the last `window` of them and to the first `keep_first`. */
 typedef struct XpGroupedAttnArgs {
   const void* q;         /* [rows, kv_heads, group_pad, dq] */
   const void* k_cache;   /* [pages, page_size, kv_heads, dq] */
   const void* v_cache;   /* [pages, page_size, kv_heads, dv] */
   void* out;             /* [rows, ld_out]: heads x vdim */
-  const void* gate;      /* optional per-head output gate logits [rows, ld_gate] */
+  const void* gate;      /* optional output gate logits [rows, ld_gate]: one per head, or per output element (gate_elems) */
   const int* row_seq;    /* [rows], or null: row r uses table row r */
   const int* positions;  /* [rows] */
   const int* slots;      /* [rows] < 0: padding row (zeros are stored) */
@@ -122,6 +159,7 @@ typedef struct XpGroupedAttnArgs {
   int rows, heads, kv_heads, group_pad, dim, vdim, dq, dv, ld_gate, ld_out, page_size, max_blocks;
   float scale, softcap;
   int f32;
+  int window, keep_first, gate_elems;
 } XpGroupedAttnArgs;
 
 /* Linear attention with a decay per key channel: S = diag(alpha) S + k v^T, o = S^T q qscale, log alpha = -softplus(-z) / tau.
@@ -174,6 +212,30 @@ typedef struct XpDeltaArgs {
   float qscale, eps;
   int f32;
 } XpDeltaArgs;
+
+/* Matrix memory with exponential gates: i = cap tanh(z_i / cap), f = log sigmoid(cap tanh(z_f / cap)); m' = max(f + m, i);
+ * S' = e^(f + m - m') S + e^(i - m') k v^T, n' likewise with k alone; o = S'^T q / (max(|n' . q|, e^-m') + 1e-6), q scaled by
+ * qscale. A head's state is [dim x vdim | n (dim) | m] in head_state floats. Decode stores rmsnorm(o) * norm * sigmoid(gate);
+ * prefill stores o. */
+typedef struct XpMemoryArgs {
+  const void* proj;      /* [rows, ld_proj]: q, k (heads x dim), v, gate (heads x vdim) at the offsets */
+  const float* gates;    /* [rows, ld_gates]: z_i and z_f (heads) at their offsets, biases added */
+  const float* norm;     /* decode: [heads * vdim] */
+  float* state;          /* [slots, heads, head_state] */
+  void* out;             /* decode: activations [rows, ld_out]; prefill: fp32 [rows, ld_out] */
+  float* planes;         /* prefill: [3, heads, rows] */
+  float* before;         /* prefill: [seqs, heads, dim + 1] */
+  float* ws;             /* chunked prefill, segs > 1: [seqs, heads, segs, head_state] */
+  const int* positions;
+  const int* slots;      /* [rows] KV slot of the row, < 0: padding row */
+  const int* state_slots;
+  const int* q_starts;
+  const int* q_lens;
+  int rows, seqs, max_q, heads, dim, vdim, head_state, ld_proj, ld_gates, ld_out, q_off, k_off, v_off, g_off, i_off, f_off;
+  int segs, seg_tokens, force_sequential;
+  float qscale, cap, eps;
+  int f32;
+} XpMemoryArgs;
 
 /* Latent attention, per token row: normalise the latent, rotate the shared key part, write both to the cache row of the
  * token; rotate the rotary part of every query head and lay the queries out for the absorbed form
@@ -251,8 +313,13 @@ int xp_gated_rms(const XpGatedRmsArgs* a, void* stream);
 int xp_post_norm(const XpPostNormArgs* a, void* stream);
 int xp_head_gate(const XpHeadGateArgs* a, void* stream);
 int xp_glu_f32(const XpGluArgs* a, void* stream);
+int xp_token_gate_f32(const XpTokenGateArgs* a, void* stream);
 int xp_grouped_prep(const XpGroupedPrepArgs* a, void* stream);
+int xp_conv_rope_decode(const XpConvRopeArgs* a, void* stream);
+int xp_conv_rope_prefill(const XpConvRopeArgs* a, void* stream);
 int xp_grouped_attn(const XpGroupedAttnArgs* a, void* stream);
+int xp_memory_decode(const XpMemoryArgs* a, void* stream);
+int xp_memory_prefill(const XpMemoryArgs* a, void* stream);
 int xp_gated_linear_decode(const XpGatedLinearArgs* a, void* stream);
 int xp_gated_linear_prefill(const XpGatedLinearArgs* a, void* stream);
 int xp_delta_decode(const XpDeltaArgs* a, void* stream);
@@ -271,6 +338,10 @@ int xp_linear_attn_prefill(const XpLinearAttnArgs* a, void* stream);
  * reduced-precision product). */
 int xp_gemm_f32(const float* x, const float* w, const float* bias, float* out, int rows, int n, int k, int ldx, int ldw, int ldo,
                 int batch, int64_t sx, int64_t sw, int64_t so, float out_scale, int silu_cols, void* stream);
+/* Grouped form over a device table of int4 {group, first feature (multiples of 128), first row, row end}, tiles of at most 64
+ * rows: group g uses w rows [g * w_rows_per_group, + n). max_tiles bounds *n_tiles. */
+int xp_gemm_f32_grouped(const float* x, const float* w, float* out, const void* tiles, const int* n_tiles, int max_tiles, int n, int k,
+                        int ldx, int ldw, int ldo, int w_rows_per_group, void* stream);
 
 #ifdef __cplusplus
 }

@@ -275,7 +275,8 @@ decode_attn_kernel(XpDecodeAttnArgs a) {
 // UMMA tile needs 64 or 128 query rows where there are 16 at most.
 //
 // kRows: the form of layered decoders (XpDecodeRowsArgs): rows name their sequence, query groups are padded, keys and values
-// differ in width, scores may be capped, outputs gated, and the probabilities enter the second product as a bf16 pair (high
+// differ in width, scores may be capped, rows may see a window of their tokens and the first ones only (the tiles between are
+// left out: slices and tiles count over what remains), outputs gated, and the probabilities enter the second product as a bf16 pair (high
 // and low part), so that they keep 16 mantissa bits.
 constexpr int kTcStages = 3;
 
@@ -316,10 +317,28 @@ __device__ __forceinline__ uint32_t pack_rest(float lo, float hi, uint32_t packe
 __device__ __forceinline__ const XpDecodeAttnArgs& base_of(const XpDecodeRowsArgs& a) { return a.a; }
 __device__ __forceinline__ const XpDecodeAttnArgs& base_of(const XpDecodeAttnArgs& a) { return a; }
 
+// What a row reads of its sequence: tokens [0, head) and [head + skip, len + skip), head and skip whole 16-token tiles. `len`
+// counts both; lo is the first token of the window.
+struct Span {
+  int len, head, skip, lo;
+  __device__ __forceinline__ int token(int v) const { return v < head ? v : v + skip; }
+};
+
 template <typename A>
-__device__ __forceinline__ int row_len(const A& args, int b) {
-  if constexpr (std::is_same<A, XpDecodeRowsArgs>::value) return args.slots[b] < 0 ? 0 : args.positions[b] + 1;
-  else return args.seq_lens[b];
+__device__ __forceinline__ Span row_span(const A& args, int b) {
+  Span s{0, 0, 0, 0};
+  if constexpr (std::is_same<A, XpDecodeRowsArgs>::value) {
+    s.len = args.slots[b] < 0 ? 0 : args.positions[b] + 1;
+    if (args.window > 0 && s.len > args.window) {
+      s.lo = s.len - args.window;
+      s.head = min((args.keep_first + 15) & ~15, s.lo & ~15);
+      s.skip = (s.lo & ~15) - s.head;
+      s.len -= s.skip;
+    }
+  } else {
+    s.len = args.seq_lens[b];
+  }
+  return s;
 }
 
 // Stores one element of a finished head.
@@ -327,8 +346,10 @@ template <int DV, typename A>
 __device__ __forceinline__ void store_out(const A& args, int b, int hq, int d, float v) {
   if constexpr (std::is_same<A, XpDecodeRowsArgs>::value) {
     if (d >= args.v_valid) return;
-    if (args.gate != nullptr)
-      v *= 1.f / (1.f + expf(-__bfloat162float(reinterpret_cast<const __nv_bfloat16*>(args.gate)[static_cast<size_t>(b) * args.ld_gate + hq])));
+    if (args.gate != nullptr) {
+      const int g = args.gate_elems ? hq * args.v_valid + d : hq;
+      v *= 1.f / (1.f + expf(-__bfloat162float(reinterpret_cast<const __nv_bfloat16*>(args.gate)[static_cast<size_t>(b) * args.ld_gate + g])));
+    }
     reinterpret_cast<__nv_bfloat16*>(args.a.out)[static_cast<size_t>(b) * args.ld_out + hq * args.v_valid + d] = __float2bfloat16_rn(v);
   } else {
     reinterpret_cast<__nv_bfloat16*>(args.out)[(static_cast<size_t>(b) * args.q_heads + hq) * DV + d] = __float2bfloat16_rn(v);
@@ -350,7 +371,8 @@ decode_attn_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_c
 
   const int split = blockIdx.x, hk = blockIdx.y, b = blockIdx.z;
   const int G = a.q_heads / a.kv_heads;
-  const int len = row_len(args, b);
+  const Span span = row_span(args, b);
+  const int len = span.len;
   const int nsplit = gridDim.x;
   int chunk = a.chunk_tokens;
   if (chunk <= 0) {
@@ -386,7 +408,7 @@ decode_attn_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_c
   // lane i looks up the cache position of the tile of iteration (base + i)
   auto lookup = [&](int it) -> int {
     if (it >= n_it) return 0;
-    const int ts = t0 + ((it * 4 + warp) << 4);
+    const int ts = span.token(t0 + ((it * 4 + warp) << 4));
     return (table[ts >> page_shift] << page_shift) + (ts & page_mask);
   };
   int my_tok = lookup(lane);
@@ -446,6 +468,12 @@ decode_attn_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_c
     }
     const int tbase = t0 + ((it * 4 + warp) << 4);
     const int nvalid = min(16, t1 - tbase);
+    // tokens [unseen, below) of the tile lie between the first tokens and the window
+    int unseen = 0, below = 0;
+    if constexpr (kRows) {
+      const int first = span.token(tbase);
+      if (first < span.lo) unseen = max(0, args.keep_first - first), below = span.lo - first;
+    }
     if (nvalid < 16) {
       // cache slots past the sequence end hold whatever was there: zero those V rows so that a
       // probability of exactly zero cannot meet a NaN
@@ -484,7 +512,7 @@ decode_attn_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_c
         if constexpr (kRows) {
           if (args.softcap > 0.f) v = cap2 - 2.f * cap2 * __frcp_rn(1.f + exp2f(sc[nt][e] * capx));
         }
-        if (col >= nvalid) v = -CUDART_INF_F;
+        if (col >= nvalid || (kRows && col >= unseen && col < below)) v = -CUDART_INF_F;
         sc[nt][e] = v;
         if (e < 2) mx0 = fmaxf(mx0, v);
         else mx1 = fmaxf(mx1, v);
@@ -612,7 +640,7 @@ __global__ void decode_combine_kernel(A args, int nsplit) {
   const int hq = blockIdx.x, b = blockIdx.y, d = threadIdx.x;
   const float* ws = a.ws + (static_cast<size_t>(b) * a.q_heads + hq) * nsplit * (D + 2);
   if (a.chunk_tokens > 0) {
-    const int len = row_len(args, b);
+    const int len = row_span(args, b).len;
     nsplit = min(nsplit, (len + a.chunk_tokens - 1) / a.chunk_tokens);  // slices that ran
   }
   float mm = -CUDART_INF_F;

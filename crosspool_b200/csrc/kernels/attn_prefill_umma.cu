@@ -24,7 +24,8 @@
 // probabilities may enter the second product as a bf16 pair (high and low part: two products, 16 mantissa bits). Groups whose
 // number of query heads is no power of two come padded (their padding is computed and not stored). Scores may be capped,
 // cap tanh(s / cap): in a tile whose scores are all far below the cap by a polynomial on the FMA pipe, otherwise through
-// 2 ** x and a reciprocal.
+// 2 ** x and a reciprocal. Queries may see a window of tokens and the first ones of the sequence only: the K/V tiles between
+// are left out (the roles count over the tiles that remain), the edges are masked per row.
 //
 // V is used where it lands (token-major rows of 64 dims) through an MN-major operand descriptor; no transpose.
 // Tensor memory: S buffers 4 x 64 columns, O 2 x D columns (512 columns with D = 128).
@@ -160,8 +161,16 @@ prefill_attn_umma_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gri
   const uint32_t q_s = base, kv_s = base + 2 * kQTile, p_s = kv_s + kStages * kStage;
   const bool act_b = q0 + np < q_len;             // tile B holds at least one real row
   const int kv_end = ctx + min(q_len, q0 + 2 * np);            // causal bound of the CTA
-  const int n_tiles = (kv_end + kBN - 1) / kBN;
-  const int n_a = min(n_tiles, (ctx + min(q_len, q0 + np) + kBN - 1) / kBN);   // tiles that tile A can see
+  // tiles [0, head) and those from head + skip on are read
+  int head = 0, skip = 0;
+  if (a.window > 0 && ctx + q0 >= a.window) {
+    const int lo_tile = (ctx + q0 - a.window + 1) / kBN;       // of the first query's window
+    head = min((a.keep_first + kBN - 1) / kBN, lo_tile);
+    skip = lo_tile - head;
+  }
+  const int n_tiles = (kv_end + kBN - 1) / kBN - skip;
+  const int n_a = min(n_tiles, (ctx + min(q_len, q0 + np) + kBN - 1) / kBN - skip);   // tiles that tile A can see
+  auto tile_token = [&](int t) { return (t < head ? t : t + skip) * kBN; };           // first token of a tile
 
   if (threadIdx.x == 0) {
     sm100::mbar_init(&bars.q_full, 1);
@@ -218,7 +227,7 @@ prefill_attn_umma_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gri
       __syncwarp();
       if (boxes == 1) {
         if (lane < 2) {
-          int tk = t * kBN;
+          int tk = tile_token(t);
           if (tk >= kv_end) tk = (kv_end - 1) & ~(kBN - 1);
           const int tok = a.seq_starts != nullptr ? a.seq_starts[seq] + tk : (table[tk >> page_shift] << page_shift) + (tk & page_mask);
           sm100::tma_load_4d_addr(kv_s + s * kStage + lane * kKTile, lane ? &tmap_v : &tmap_k,
@@ -226,7 +235,7 @@ prefill_attn_umma_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gri
         }
       } else if (lane < 2 * boxes * kHalves) {       // small pages: DQ == DV (checked by the host)
         const int h = lane % kHalves, is_v = (lane / kHalves) & 1, j = lane / (2 * kHalves);
-        int tk = t * kBN + j * box_tokens;
+        int tk = tile_token(t) + j * box_tokens;
         if (tk >= kv_end) tk = (kv_end - 1) & ~(box_tokens - 1);   // boxes past the end repeat the last valid one (masked)
         const int tok = (table[tk >> page_shift] << page_shift) + (tk & page_mask);
         sm100::tma_load_3d_addr(kv_s + s * kStage + is_v * kKTile + h * kKVHalf + j * box_bytes, is_v ? &tmap_v3 : &tmap_k3,
@@ -322,6 +331,7 @@ prefill_attn_umma_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gri
     const bool tile_on = x == 0 || act_b;
     const int my_tiles = x == 0 ? n_a : n_tiles;
     const int limit = min(ctx + pos, kv_end - 1);     // last visible cache position of this row
+    const int win_lo = a.window > 0 ? ctx + pos - a.window + 1 : 0;   // first of its window
     const uint32_t lane_off = static_cast<uint32_t>((warp & 3) * 32) << 16;
     const uint32_t o_t = tmem + lane_off + kOCol + static_cast<uint32_t>(x * DV);
     const uint32_t p_row = p_s + x * kPTile + row * 128;
@@ -347,11 +357,18 @@ prefill_attn_umma_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gri
         }
 
         if constexpr (kCap) cap_scores(sv, a.scale, a.softcap);
-        const int nvis = min(kBN, max(0, limit - t * kBN + 1));   // visible tokens of this tile for this row
+        const int tok0 = tile_token(t);
+        const int nvis = min(kBN, max(0, limit - tok0 + 1));      // visible tokens of this tile for this row
         if (nvis < kBN) {
 #pragma unroll
           for (int j = 0; j < kBN; ++j)
             if (j >= nvis) sv[j] = 0xff800000u;       // -inf: selected, never computed with (the slot may hold NaN)
+        }
+        const int below = win_lo - tok0, kept = a.keep_first - tok0;   // tokens [kept, below) of the tile are behind the window
+        if (below > 0 && kept < kBN) {
+#pragma unroll
+          for (int j = 0; j < kBN; ++j)
+            if (j >= kept && j < below) sv[j] = 0xff800000u;
         }
         // four independent chains of three-input maxima: a serial chain over 64 values costs its latency 64 times
         float mx4[4] = {-CUDART_INF_F, -CUDART_INF_F, -CUDART_INF_F, -CUDART_INF_F};
@@ -416,13 +433,13 @@ prefill_attn_umma_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gri
                        "r"(pk[c * 4 + 1]), "r"(pk[c * 4 + 2]), "r"(pk[c * 4 + 3])
                        : "memory");
         }
-        const bool v_tail = (x == 0 || t >= n_a) && t * kBN + kBN > kv_end;
+        const bool v_tail = (x == 0 || t >= n_a) && tok0 + kBN > kv_end;
         if (v_tail) {
           // cache slots past the sequence end may hold anything: zero those V rows (probability 0 x NaN).
           // Tile A's PV product is issued before tile B's and both read this stage, so tile A's threads do it
           // on the tiles that tile A visits, tile B's on the rest.
           const uint32_t v_s = kv_s + (t % kStages) * kStage + kKTile;
-          const int first = kv_end - t * kBN;
+          const int first = kv_end - tok0;
           for (int i = row; i < (kBN - first) * (DV / 8); i += kRows) {
             const int R = first + i / (DV / 8), cc = i % (DV / 8);
             const uint32_t off = (cc >> 3) * kKVHalf + R * 128 + (((cc & 7) ^ (R & 7)) << 4);
@@ -448,7 +465,10 @@ prefill_attn_umma_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gri
       if (ok) {
         sm100::tc_fence_after_sync();
         float inv = l > 0.f ? 1.f / l : 0.f;
-        if (a.gate != nullptr && stored)
+        const __nv_bfloat16* ge = nullptr;                // one gate per element
+        if (a.gate_elems && stored)
+          ge = reinterpret_cast<const __nv_bfloat16*>(a.gate) + static_cast<size_t>(q_base + pos) * a.ld_gate + hq * a.v_valid;
+        else if (a.gate != nullptr && stored)
           inv *= 1.f / (1.f + expf(-__bfloat162float(reinterpret_cast<const __nv_bfloat16*>(a.gate)[static_cast<size_t>(q_base + pos) * a.ld_gate + hq])));
         const int v_valid = a.v_valid;                    // stored columns of a head (a multiple of 8)
         __nv_bfloat16* og = reinterpret_cast<__nv_bfloat16*>(a.out) + static_cast<size_t>(q_base + pos) * a.ld_out + hq * v_valid;
@@ -461,6 +481,16 @@ prefill_attn_umma_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gri
 #pragma unroll
             for (int j = 0; j < 32; j += 8) {
               if (c + j >= v_valid) break;
+              if (ge != nullptr) {
+                const uint4 gr = *reinterpret_cast<const uint4*>(ge + c + j);
+                const uint32_t gw[4] = {gr.x, gr.y, gr.z, gr.w};
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                  const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&gw[i]));
+                  ov[j + 2 * i] = __float_as_uint(__uint_as_float(ov[j + 2 * i]) * (1.f / (1.f + __expf(-f.x))));
+                  ov[j + 2 * i + 1] = __float_as_uint(__uint_as_float(ov[j + 2 * i + 1]) * (1.f / (1.f + __expf(-f.y))));
+                }
+              }
               uint4 v;
               v.x = pack2(__uint_as_float(ov[j]) * inv, __uint_as_float(ov[j + 1]) * inv);
               v.y = pack2(__uint_as_float(ov[j + 2]) * inv, __uint_as_float(ov[j + 3]) * inv);
@@ -543,7 +573,8 @@ extern "C" int xp_prefill_attn_umma(const XpPrefillAttnArgs* a, void* stream) {
   const int G = a->q_heads / a->kv_heads;
   const bool ok = a->num_pages > 0 && a->total_q > 0 && a->page_size >= 16 && (a->page_size & (a->page_size - 1)) == 0 &&
                   (G == 1 || G == 2 || G == 4 || G == 8 || G == 16) && (reinterpret_cast<uintptr_t>(a->q) & 15) == 0 &&
-                  (reinterpret_cast<uintptr_t>(a->out) & 15) == 0 && a->ld_out % 8 == 0 && a->v_valid % 8 == 0;
+                  (reinterpret_cast<uintptr_t>(a->out) & 15) == 0 && a->ld_out % 8 == 0 && a->v_valid % 8 == 0 &&
+                  (!a->gate_elems || (a->gate != nullptr && a->ld_gate % 8 == 0 && (reinterpret_cast<uintptr_t>(a->gate) & 15) == 0));
   if (!ok) return 1;
   // P (the probabilities) reaches the second product through tensor memory; bit 8 of force_simple selects the
   // form that stages P in shared memory instead

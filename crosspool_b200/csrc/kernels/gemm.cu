@@ -283,10 +283,13 @@ extern "C" int xp_gemm_plan(const XpGemmArgs* a, XpGemmPlan* plan) {
   if (a->n_out <= 0 || a->k <= 0 || a->rows <= 0) return -10;
   // bf16 problems over row-major weights may end in partial tiles (TMA fills them with zeros; a partial gate tile computes
   // rows of the up matrix that nobody stores); the other forms address whole tiles
-  const bool whole = a->fp8 || a->w_tiled || a->tile_table != nullptr;
+  const bool whole = a->fp8 || a->w_tiled;
   if (whole && (a->n_out % gemm::kTileM != 0 || a->k % kblk != 0)) return -10;
   const int batch = a->batch > 1 ? a->batch : 1;
-  if (batch > 1 && (whole || a->dual || a->epilogue == gemm::kEpiResidual || a->bias != nullptr || a->x_group_rows < a->rows)) return -16;
+  if (batch > 1 && (whole || a->tile_table != nullptr || a->dual || a->epilogue == gemm::kEpiResidual || a->bias != nullptr || a->x_group_rows < a->rows)) return -16;
+  if (a->epilogue == gemm::kEpiTokenGate && (a->dual || batch > 1 || a->tile_table != nullptr || a->ids == nullptr || a->resid == nullptr || a->ids_limit <= 0))
+    return -17;
+  if (a->tail != nullptr && (a->epilogue != gemm::kEpiStore || batch > 1 || a->tile_table != nullptr)) return -18;
   if (a->fp8 && (a->dual || a->w_tiled || a->tile_table != nullptr || a->w_scale == nullptr || a->x_scale == nullptr ||
                  a->ld_xscale % 4 != 0 || a->bn > gemm::kMaxBnF8))
     return -14;
@@ -394,6 +397,12 @@ extern "C" int xp_gemm(const XpGemmArgs* a) {
   p.out_group_stride = a->out_group_stride;
   p.out_scale = a->out_scale;
   p.silu_cols = a->silu_cols;
+  p.act_cubic = a->act_cubic;
+  p.ids = a->ids;
+  p.ids_limit = a->ids_limit;
+  p.tail = a->tail;
+  p.tail_from = a->tail_from;
+  p.ld_tail = a->ld_tail;
   if (a->tile_table != nullptr) {
     if (plan.splits != 1) return -13;
     plan.grid = plan.smem_bytes > 0 ? 148 : 148;

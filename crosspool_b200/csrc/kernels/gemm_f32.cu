@@ -9,15 +9,12 @@ namespace {
 
 constexpr int kBM = 64, kBN = 64, kBK = 16;
 
-__global__ void __launch_bounds__(256)
-gemm_f32_kernel(const float* __restrict__ x, const float* __restrict__ w, const float* __restrict__ bias, float* __restrict__ out,
-                int rows, int n, int k, int ldx, int ldw, int ldo, int64_t sx, int64_t sw, int64_t so, float scale, int silu_cols) {
+// Rows r0 .. and features n0 .. of one product; rows and n bound both.
+__device__ __forceinline__ void tile_f32(const float* __restrict__ x, const float* __restrict__ w, const float* __restrict__ bias,
+                                         float* __restrict__ out, int r0, int n0, int rows, int n, int k, int ldx, int ldw, int ldo, float scale,
+                                         int silu_cols) {
   __shared__ float xs[kBK][kBM + 4];
   __shared__ float ws[kBK][kBN + 4];
-  x += blockIdx.z * sx;
-  w += blockIdx.z * sw;
-  out += blockIdx.z * so;
-  const int r0 = blockIdx.y * kBM, n0 = blockIdx.x * kBN;
   const int tr = threadIdx.x >> 4, tc = threadIdx.x & 15;
   float acc[4][4] = {};
   for (int k0 = 0; k0 < k; k0 += kBK) {
@@ -55,7 +52,36 @@ gemm_f32_kernel(const float* __restrict__ x, const float* __restrict__ w, const 
   }
 }
 
+__global__ void __launch_bounds__(256)
+gemm_f32_kernel(const float* __restrict__ x, const float* __restrict__ w, const float* __restrict__ bias, float* __restrict__ out,
+                int rows, int n, int k, int ldx, int ldw, int ldo, int64_t sx, int64_t sw, int64_t so, float scale, int silu_cols) {
+  tile_f32(x + blockIdx.z * sx, w + blockIdx.z * sw, bias, out + blockIdx.z * so, blockIdx.y * kBM, blockIdx.x * kBN, rows, n, k, ldx, ldw, ldo,
+           scale, silu_cols);
+}
+
+// Grouped form: tiles {group, first feature of 128, first row, row end} of at most kBM rows from a device table; a CTA takes
+// one half of a tile's features.
+__global__ void __launch_bounds__(256)
+gemm_f32_grouped_kernel(const float* __restrict__ x, const float* __restrict__ w, float* __restrict__ out, const int4* __restrict__ tiles,
+                        const int* __restrict__ n_tiles, int n, int k, int ldx, int ldw, int ldo, int w_rows_per_group) {
+  if (static_cast<int>(blockIdx.x) >= *n_tiles) return;
+  const int4 t = tiles[blockIdx.x];
+  const int n0 = t.y + blockIdx.y * kBN;
+  if (n0 >= n) return;
+  tile_f32(x, w + static_cast<int64_t>(t.x) * w_rows_per_group * ldw, nullptr, out, t.z, n0, min(t.w, t.z + kBM), n, k, ldx, ldw, ldo, 1.f, 0);
+}
+
 }  // namespace
+
+extern "C" int xp_gemm_f32_grouped(const float* x, const float* w, float* out, const void* tiles, const int* n_tiles, int max_tiles, int n, int k,
+                                   int ldx, int ldw, int ldo, int w_rows_per_group, void* stream) {
+  if (max_tiles <= 0 || n <= 0) return 0;
+  if (k <= 0) return -10;
+  gemm_f32_grouped_kernel<<<dim3(max_tiles, 128 / kBN), 256, 0, reinterpret_cast<cudaStream_t>(stream)>>>(
+      x, w, out, static_cast<const int4*>(tiles), n_tiles, n, k, ldx, ldw, ldo, w_rows_per_group);
+  cudaError_t e = cudaGetLastError();
+  return e == cudaSuccess ? 0 : -100 - static_cast<int>(e);
+}
 
 extern "C" int xp_gemm_f32(const float* x, const float* w, const float* bias, float* out, int rows, int n, int k, int ldx, int ldw,
                            int ldo, int batch, int64_t sx, int64_t sw, int64_t so, float out_scale, int silu_cols, void* stream) {

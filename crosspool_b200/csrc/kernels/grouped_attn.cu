@@ -1,4 +1,4 @@
-// Grouped-query attention without rotation: the row kernel between the projection and the attention kernels, and the plain
+// Grouped-query attention: the row kernel of the form without positions between the projection and the attention kernels, and the plain
 // attention kernel for sizes and types that the tensor-core kernels (attn_decode.cu, attn_prefill_umma.cu) do not cover.
 #include <math_constants.h>
 
@@ -87,11 +87,14 @@ grouped_attn_kernel(XpGroupedAttnArgs a) {
   const int len = a.positions[row] + 1;
   const T* kc = reinterpret_cast<const T*>(a.k_cache);
   const T* vc = reinterpret_cast<const T*>(a.v_cache);
+  // the kept first tokens in whole steps of 32, then the step in which the window begins and those behind it
+  const int lo = a.window > 0 && len > a.window ? len - a.window : 0;
+  const int head = min((a.keep_first + 31) / 32, lo / 32) * 32, skip = lo / 32 * 32 - head;
   float m = -CUDART_INF_F, l = 0.f;
-  for (int t0 = warp * 32; t0 < len; t0 += kAttnWarps * 32) {
-    const int t = t0 + lane;
-    const bool on = t < len;
-    const int tt = on ? t : t0;
+  for (int v0 = warp * 32; v0 + (v0 < head ? 0 : skip) < len; v0 += kAttnWarps * 32) {
+    const int t0 = v0 + (v0 < head ? 0 : skip), t = t0 + lane;
+    const bool on = t < len && (t >= lo || t < a.keep_first);
+    const int tt = t < len ? t : t0;
     const size_t tok = (static_cast<size_t>(table[tt / a.page_size]) * a.page_size + tt % a.page_size) * a.kv_heads + hk;
     const T* k = kc + tok * a.dq;
     float s = 0.f;
@@ -127,13 +130,15 @@ grouped_attn_kernel(XpGroupedAttnArgs a) {
     if (mw != -CUDART_INF_F) ll += all[w * step + a.vdim + 1] * expf(mw - mm);
   }
   float f = 1.f / ll;
-  if (a.gate != nullptr) f *= elem::sigmoid(ld(reinterpret_cast<const T*>(a.gate) + static_cast<size_t>(row) * a.ld_gate + h));
+  const T* gate = a.gate != nullptr ? reinterpret_cast<const T*>(a.gate) + static_cast<size_t>(row) * a.ld_gate : nullptr;
+  if (gate != nullptr && !a.gate_elems) f *= elem::sigmoid(ld(gate + h));
   for (int c = threadIdx.x; c < a.vdim; c += kAttnWarps * 32) {
     float v = 0.f;
     for (int w = 0; w < kAttnWarps; ++w) {
       const float mw = all[w * step + a.vdim];
       if (mw != -CUDART_INF_F) v += all[w * step + c] * expf(mw - mm);
     }
+    if (gate != nullptr && a.gate_elems) v *= elem::sigmoid(ld(gate + h * a.vdim + c));
     st(out + c, v * f);
   }
 }

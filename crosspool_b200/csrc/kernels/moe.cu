@@ -14,6 +14,7 @@
 #include <math_constants.h>
 
 #include "xpool/api.h"
+#include "xpool/elem.cuh"
 #include "xpool/lane.cuh"
 #include "xpool/sm100.cuh"
 
@@ -253,6 +254,37 @@ combine_kernel(const __nv_bfloat16* __restrict__ y, const int* __restrict__ rout
   combine_token(y, route_pos, weights, out, top_k, hidden, ld_out, blockIdx.x);
 }
 
+// Weighted experts, identity experts and the gated shared expert of one token.
+template <typename T, int N>
+__global__ void __launch_bounds__(128)
+mix_kernel(XpMoeMixArgs a) {
+  const int t = blockIdx.x;
+  const T* x = reinterpret_cast<const T*>(a.x) + static_cast<size_t>(t) * a.ld_x;
+  const T* sh = a.shared != nullptr ? reinterpret_cast<const T*>(a.shared) + static_cast<size_t>(t) * a.ld_shared : nullptr;
+  const float sg = sh != nullptr ? elem::sigmoid(a.shared_gate[static_cast<size_t>(t) * a.ld_gate]) : 0.f;
+  T* out = reinterpret_cast<T*>(a.out) + static_cast<size_t>(t) * a.ld_out;
+  for (int c = threadIdx.x * N; c < a.hidden; c += 128 * N) {
+    float acc[N], v[N];
+#pragma unroll
+    for (int j = 0; j < N; ++j) acc[j] = 0.f;
+    for (int k = 0; k < a.top_k; ++k) {
+      const int pos = a.route_pos[t * a.top_k + k];
+      const float w = a.weights[t * a.top_k + k];
+      if (pos >= 0) elem::ldv<N>(reinterpret_cast<const T*>(a.y) + static_cast<size_t>(pos) * a.ld_y + c, v);
+      else if (a.topk_ids[t * a.top_k + k] >= a.experts) elem::ldv<N>(x + c, v);
+      else continue;
+#pragma unroll
+      for (int j = 0; j < N; ++j) acc[j] = fmaf(w, v[j], acc[j]);
+    }
+    if (sh != nullptr) {
+      elem::ldv<N>(sh + c, v);
+#pragma unroll
+      for (int j = 0; j < N; ++j) acc[j] = fmaf(sg, v[j], acc[j]);
+    }
+    elem::stv<N>(out + c, acc);
+  }
+}
+
 // ---------------------------------------------------------------------------------------------
 // Lane forms: the same steps with every parameter read from the Lane's current invocation, so
 // that one captured graph serves dense and MoE layers of every model. Each is a no-op unless the
@@ -310,6 +342,50 @@ __device__ __forceinline__ int block_exclusive_scan(int v, int* warp_sums, int* 
   *total = warp_sums[31];
   __syncthreads();
   return base + inc - v;
+}
+
+// Decode-size form of router_topk, route_count, route_offsets_tiles and route_place: one CTA does all of them.
+__global__ void __launch_bounds__(1024)
+topk_route_kernel(XpRouterArgs a, XpRouteArgs r) {
+  __shared__ int hist[1024], cursor[1024], warp_sums[32];
+  const int e = threadIdx.x, lo = r.expert_lo, n_local = r.expert_hi - r.expert_lo;
+  hist[e] = 0;
+  for (int row = e >> 5; row < a.rows; row += 32) router_topk_row(a, row, e & 31);
+  __syncthreads();                                   // the ids below were written by this CTA
+  const int n_routes = a.rows * a.top_k;
+  for (int i = e; i < n_routes; i += 1024) {
+    const int x = a.topk_ids[i] - lo;
+    if (x >= 0 && x < n_local) atomicAdd(&hist[x], 1);
+    else r.route_pos[i] = -1;
+  }
+  __syncthreads();
+  const int c = e < n_local ? hist[e] : 0;
+  const int b_gu = (c + r.bn_gateup - 1) / r.bn_gateup, b_dn = (c + r.bn_down - 1) / r.bn_down;
+  int total, total_gu, total_dn;
+  const int off = block_exclusive_scan(c, warp_sums, &total);
+  const int t_gu = block_exclusive_scan(r.tm_gateup * b_gu, warp_sums, &total_gu);
+  const int t_dn = block_exclusive_scan(r.tm_down * b_dn, warp_sums, &total_dn);
+  cursor[e] = off;
+  if (e <= n_local) r.offsets[e] = off;
+  if (e < n_local) r.counts[e] = c;
+  if (e == 0) *r.n_tiles_gateup = total_gu, *r.n_tiles_down = total_dn;
+  __syncthreads();
+  for (int i = e; i < n_routes; i += 1024) {
+    const int x = a.topk_ids[i] - lo;
+    if (x >= 0 && x < n_local) {
+      const int pos = atomicAdd(&cursor[x], 1);
+      r.perm_token[pos] = i / r.top_k;
+      r.route_pos[i] = pos;
+    }
+  }
+  if (e < n_local) {
+    int idx = t_gu;
+    for (int m = 0; m < r.tm_gateup; ++m)
+      for (int p = off; p < off + c; p += r.bn_gateup) reinterpret_cast<int4*>(r.tiles_gateup)[idx++] = make_int4(e, m * 128, p, off + c);
+    idx = t_dn;
+    for (int m = 0; m < r.tm_down; ++m)
+      for (int p = off; p < off + c; p += r.bn_down) reinterpret_cast<int4*>(r.tiles_down)[idx++] = make_int4(e, m * 128, p, off + c);
+  }
 }
 
 // One CTA orders the routes of this rank's experts and writes both tile tables. Positions inside
@@ -492,6 +568,33 @@ extern "C" int xp_moe_route(const XpRouteArgs* a, void* stream) {
                                                 a->bn_down, reinterpret_cast<int4*>(a->tiles_down), a->n_tiles_down);
   route_place_kernel<<<n_local, 256, 0, s>>>(a->topk_ids, n_routes, a->top_k, a->expert_lo, a->offsets, a->perm_token,
                                              a->route_pos);
+  return last_error();
+}
+
+extern "C" int xp_moe_topk_route(const XpRouterArgs* a, const XpRouteArgs* r, void* stream) {
+  if (a->rows <= 0) return 0;
+  const int n_local = r->expert_hi - r->expert_lo;
+  if (a->num_experts > 32 * kMaxPerLane || a->top_k > 32 || a->top_k > a->num_experts || n_local < 1 || n_local > 1023 || a->rows > 128 ||
+      a->rows != r->rows || a->top_k != r->top_k || a->topk_ids != r->topk_ids)
+    return -10;
+  topk_route_kernel<<<1, 1024, 0, reinterpret_cast<cudaStream_t>(stream)>>>(*a, *r);
+  return last_error();
+}
+
+extern "C" int xp_moe_mix(const XpMoeMixArgs* a, void* stream) {
+  if (a->rows <= 0) return 0;
+  if (a->hidden <= 0 || a->top_k <= 0 || (a->shared != nullptr && a->shared_gate == nullptr)) return -10;
+  const int eb = a->f32 ? 4 : 2;
+  auto fits = [&](const void* p, int ld) { return p == nullptr || (reinterpret_cast<uintptr_t>(p) % (4 * eb) == 0 && ld % 4 == 0); };
+  const bool v = a->hidden % 4 == 0 && fits(a->y, a->ld_y) && fits(a->x, a->ld_x) && fits(a->shared, a->ld_shared) && fits(a->out, a->ld_out);
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  if (a->f32) {
+    if (v) mix_kernel<float, 4><<<a->rows, 128, 0, s>>>(*a);
+    else mix_kernel<float, 1><<<a->rows, 128, 0, s>>>(*a);
+  } else {
+    if (v) mix_kernel<__nv_bfloat16, 4><<<a->rows, 128, 0, s>>>(*a);
+    else mix_kernel<__nv_bfloat16, 1><<<a->rows, 128, 0, s>>>(*a);
+  }
   return last_error();
 }
 

@@ -3,8 +3,9 @@
 //   polynorm     a N(z) + b N(z^2) + c N(z^3) + e, N dividing the row by its root mean square
 //   gated_rms    rmsnorm(o) * w * sigmoid(gate)
 //   post_norm    residual += rmsnorm(sublayer output, or the mean of normed branches) * w [-> norm] -> activation row
-//   head_gate    rmsnorm per head * w * silu(gate), one warp per head
-//   glu_f32      clamped gated activation of fp32 models (bf16 has it in the product's epilogue)
+//   head_gate    rmsnorm per head * w * silu(gate) or sigmoid(gate), one warp per head
+//   glu_f32      gated activation of fp32 models (bf16 has it in the product's epilogue)
+//   token_gate   activation times a row of a token table, fp32 models (bf16: the product's epilogue)
 // Rows whose pitches allow it are moved four elements at a time.
 #include "xpool/elem.cuh"
 #include "xpool/mixer_api.h"
@@ -216,7 +217,12 @@ post_norm_kernel(XpPostNormArgs a) {
     int id = a.ids[r];
     if (id < 0 || id >= a.vocab) id = 0;
     const T* row = reinterpret_cast<const T*>(a.table) + static_cast<size_t>(id) * a.hidden;
-    each([&](int it, int c) { ldv<N>(row + c, y[it]); });
+    const float es = a.embed_scale == 0.f ? 1.f : a.embed_scale;
+    each([&](int it, int c) {
+      ldv<N>(row + c, y[it]);
+#pragma unroll
+      for (int j = 0; j < N; ++j) y[it][j] *= es;
+    });
   } else {
     const T* b0 = reinterpret_cast<const T*>(a.branches[0]) + static_cast<size_t>(r) * a.ld_branch[0];
     float s0 = 0.f, s1 = 0.f;
@@ -292,6 +298,7 @@ head_gate_kernel(XpHeadGateArgs a) {
   const float* o = a.o + static_cast<size_t>(row) * a.ld_o + h * a.dim;
   const T* gate = reinterpret_cast<const T*>(a.gate) + static_cast<size_t>(row) * a.ld_gate + h * a.dim;
   T* out = reinterpret_cast<T*>(a.out) + static_cast<size_t>(row) * a.ld_out + h * a.dim;
+  const float* weight = a.weight + (a.per_head_weight ? h * a.dim : 0);
   float ss = 0.f;
   for (int c = lane * N; c < a.dim; c += 32 * N) {
     float v[N];
@@ -303,13 +310,15 @@ head_gate_kernel(XpHeadGateArgs a) {
   for (int c = lane * N; c < a.dim; c += 32 * N) {
     float v[N], w[N], g[N];
     ldv<N>(o + c, v);
-    ldv<N>(a.weight + c, w);
+    ldv<N>(weight + c, w);
     ldv<N>(gate + c, g);
 #pragma unroll
-    for (int j = 0; j < N; ++j) v[j] = v[j] * inv * w[j] * elem::silu(g[j]);
+    for (int j = 0; j < N; ++j) v[j] = v[j] * inv * w[j] * (a.sigmoid_gate ? sigmoid(g[j]) : elem::silu(g[j]));
     stv<N>(out + c, v);
   }
 }
+
+__device__ __forceinline__ float gated(float g, float alpha, float cubic) { return g / (1.f + expf(-alpha * g * fmaf(cubic * g, g, 1.f))); }
 
 __global__ void __launch_bounds__(kThreads)
 glu_f32_kernel(XpGluArgs a) {
@@ -319,7 +328,19 @@ glu_f32_kernel(XpGluArgs a) {
     const float* z = a.z + static_cast<size_t>(r) * a.ld_z;
     const float lim = a.limit > 0.f ? a.limit : 3.0e38f;
     const float g = fminf(z[c], lim), u = fminf(fmaxf(z[a.cols + c], -lim), lim);
-    a.out[static_cast<size_t>(r) * a.ld_out + c] = g / (1.f + expf(-a.alpha * g)) * (u + a.up_add);
+    a.out[static_cast<size_t>(r) * a.ld_out + c] = gated(g, a.alpha, a.cubic) * (u + a.up_add);
+  }
+}
+
+__global__ void __launch_bounds__(kThreads)
+token_gate_f32_kernel(XpTokenGateArgs a) {
+  const int c = blockIdx.x * kThreads + threadIdx.x;
+  if (c >= a.cols) return;
+  for (int r = blockIdx.y; r < a.rows; r += gridDim.y) {
+    int id = a.ids[r];
+    if (id < 0 || id >= a.vocab) id = 0;
+    a.out[static_cast<size_t>(r) * a.ld_out + c] =
+        gated(a.z[static_cast<size_t>(r) * a.ld_z + c], a.alpha, a.cubic) * a.table[static_cast<size_t>(id) * a.ld_table + c];
   }
 }
 
@@ -439,5 +460,13 @@ extern "C" int xp_glu_f32(const XpGluArgs* a, void* stream) {
   if (a->cols <= 0) return -10;
   const dim3 grid((a->cols + kThreads - 1) / kThreads, a->rows < 65535 ? a->rows : 65535);
   glu_f32_kernel<<<grid, kThreads, 0, reinterpret_cast<cudaStream_t>(stream)>>>(*a);
+  return done();
+}
+
+extern "C" int xp_token_gate_f32(const XpTokenGateArgs* a, void* stream) {
+  if (a->rows <= 0) return 0;
+  if (a->cols <= 0 || a->vocab <= 0) return -10;
+  const dim3 grid((a->cols + kThreads - 1) / kThreads, a->rows < 65535 ? a->rows : 65535);
+  token_gate_f32_kernel<<<grid, kThreads, 0, reinterpret_cast<cudaStream_t>(stream)>>>(*a);
   return done();
 }

@@ -4,7 +4,7 @@ Used when one GPU hosts both roles (kernels that wait on one another must never 
 launches on one GPU, so the loopback path is stream-ordered and flag-free). Dense layers are two
 launches: gate/up GEMM with the SwiGLU epilogue, then the down projection. Ungated layers with a
 row-normalised activation (PolyNorm) put the activation kernel between the two products, and so do
-gated layers in fp32.
+gated layers in fp32. Routed layers run the grouped products of :mod:`crosspool_b200.ops.moe`.
 """
 
 from __future__ import annotations
@@ -39,11 +39,20 @@ class LocalFfnPort(FfnPort):
             self.moe_ws = moe.workspace(engine.device, engine.cap, self.cfg, w.gate_up.shape[1] // 2, w.gate_up.shape[0])
 
     def _attach_layered(self, engine) -> None:
-        for w in self.weights:
-            if w is not None:
-                w.gate_up, w.down = pad_pitch(w.gate_up), pad_pitch(w.down)
+        routed = [s.moe for s in self.cfg.layer_specs if s.moe is not None]
+        plain = [w for w in self.weights if w is not None and not w.is_moe]
+        for w in plain:
+            w.gate_up, w.down = pad_pitch(w.gate_up), pad_pitch(w.down)
         # widest activation row; fp32 gated layers keep gate and up columns, then the activations behind them
-        inter = max((ceil8(w.gate_up.shape[0]) + ceil8(w.down.shape[1]) for w in self.weights if w is not None), default=8)
+        inter = max((ceil8(w.gate_up.shape[0]) + ceil8(w.down.shape[1]) for w in plain), default=8)
+        self.moe_ws = None
+        if routed:
+            from ..ops import moe
+
+            for w in self.weights:
+                if w is not None and w.is_moe:
+                    moe.prepare_routed(w)
+            self.moe_ws = moe.RoutedWorkspace.for_layers(routed, self.cfg.hidden_size, engine.cap, engine.dtype, engine.device)
         self.act = torch.zeros(engine.cap * inter, dtype=engine.dtype, device=engine.device)
         self.y = torch.zeros(engine.cap, ceil8(self.cfg.hidden_size), dtype=engine.dtype, device=engine.device)[:, :self.cfg.hidden_size]
 
@@ -62,15 +71,15 @@ class LocalFfnPort(FfnPort):
         """Gated FFN of any width in the engine's element type."""
         ff = w.down.shape[1]
         act = self.act[:rows * ceil8(ff)].view(rows, ceil8(ff))[:, :ff]
-        limit, up_add, alpha = w.extra.get("gate_transform", (0.0, 0.0, 1.0))
+        limit, up_add, alpha, cubic = (*w.extra.get("gate_transform", (0.0, 0.0, 1.0)), 0.0)[:4]
         if x.dtype == torch.float32:
             from ..ops import mixers
 
             z = self.act[rows * ceil8(ff):][:rows * 2 * ff].view(rows, 2 * ff)
             gemm.linear(x, w.gate_up, out=z)
-            mixers.glu_f32(z, limit, up_add, alpha, act)
+            mixers.glu_f32(z, limit, up_add, alpha, act, cubic)
         else:
-            gemm.gateup_swiglu(x, w.gate_up, out=act, gate_limit=limit, up_add=up_add, act_alpha=alpha)
+            gemm.gateup_swiglu(x, w.gate_up, out=act, gate_limit=limit, up_add=up_add, act_alpha=alpha, act_cubic=cubic)
         gemm.linear(act, w.down, out=self.y[:rows])
         return [self.y[:rows]]
 
@@ -78,6 +87,10 @@ class LocalFfnPort(FfnPort):
         w = self.weights[layer]
         if "polynorm" in w.extra:
             return self._run_polynorm(w, x, rows)
+        if self.cfg.layered and w.is_moe:
+            from ..ops import moe
+
+            return [moe.routed_ffn(x, w, self.cfg.layer_specs[layer].moe, self.y[:rows], self.moe_ws)]
         if self.cfg.layered:
             return self._run_gated(w, x, rows)
         if w.is_moe:

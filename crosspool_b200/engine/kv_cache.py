@@ -19,7 +19,7 @@ from dataclasses import dataclass, field
 
 import torch
 
-from ..models.config import DeltaMixer, ModelConfig, sub_mixers
+from ..models.config import ModelConfig, sub_mixers
 
 
 class OutOfPages(RuntimeError):
@@ -157,7 +157,7 @@ class PagedKvCache:
     allocator: PageAllocator
     backing: object | None = None  # ecs.vmm.KvVmmBacking when elastic
     tables: dict[int, list[int]] = field(default_factory=dict)
-    # recurrent layers: fp32 [slots, heads, dim, vdim] per layer (None elsewhere), and the slot of every live sequence
+    # recurrent layers: fp32 [slots, *state_shape of the mixer] per layer (None elsewhere), and the slot of every live sequence
     states: list[torch.Tensor | None] = field(default_factory=list)
     # convolution inputs behind every live sequence, [slots, taps, channels] per layer: the input at position p is entry p % taps
     conv: list[torch.Tensor | None] = field(default_factory=list)
@@ -177,8 +177,9 @@ class PagedKvCache:
 
     @classmethod
     def _layered(cls, cfg: ModelConfig, num_pages: int, page_size: int, device, dtype: torch.dtype, state_slots: int) -> "PagedKvCache":
-        """Pages hold a key row and a value row per token in the layers that cache any (or one latent row that is both);
-        recurrent mixers hold one state per slot, and those with a convolution its latest inputs."""
+        """Pages hold a key row and a value row per token in the layers that cache any (or one latent row that is both); a layer
+        may read another one's instead. Recurrent mixers hold one state per slot, and mixers with a convolution its latest
+        inputs."""
         mixers = [s.mixer for s in cfg.layer_specs]
         lay = KvLayout(page_size, num_pages, 1, 0, cfg.num_layers, dtype.itemsize, tuple(m.cache_width for m in mixers))
 
@@ -191,10 +192,14 @@ class PagedKvCache:
         for l, m in enumerate(mixers):
             for sub in sub_mixers(m):
                 if sub.state_elems:
-                    states[l] = torch.zeros(state_slots, sub.heads, sub.dim, sub.vdim, dtype=torch.float32, device=device)
-                if isinstance(sub, DeltaMixer):
+                    states[l] = torch.zeros(state_slots, *sub.state_shape, dtype=torch.float32, device=device)
+                if getattr(sub, "conv", 0):
                     conv[l] = torch.zeros(state_slots, sub.conv, sub.conv_channels, dtype=dtype, device=device)
-        return cls(lay, [rows(m, 0) for m in mixers], [rows(m, 1) for m in mixers], PageAllocator(num_pages), states=states, conv=conv,
+        k, v = [rows(m, 0) for m in mixers], [rows(m, 1) for m in mixers]
+        for l, m in enumerate(mixers):
+            if getattr(m, "kv_from", None) is not None:
+                k[l], v[l] = k[m.kv_from], v[m.kv_from]
+        return cls(lay, k, v, PageAllocator(num_pages), states=states, conv=conv,
                    slots=StateSlots(state_slots) if cfg.recurrent else None)
 
     # -- per-sequence page tables --------------------------------------------------------------

@@ -7,13 +7,13 @@ over all rows together; a mixer splits the rows where its decode and prefill ker
   one pass over the cached rows); long portions in the expanded form (the sequence's latents are expanded to per-head keys
   and values with one product each, then the tcgen05 prefill kernel);
 * grouped-query attention: decoded tokens and short portions as single rows, long portions in the tcgen05 prefill kernel;
-* recurrences (decayed linear attention, gated linear attention, gated delta rule): one kernel advances the states of the
-  decoded tokens, others those of the portions;
+* recurrences (decayed linear attention, gated linear attention, gated delta rule, matrix memory): one kernel advances the
+  states of the decoded tokens, others those of the portions;
 * a parallel pair runs both of its sides on the columns of one projection.
 
 The residual stream is fp32. Where a norm stands in front of a sublayer, one kernel gates and adds the previous sublayer's
 output and normalises for the next; where it stands behind, one kernel norms the output (of both sides of a pair), adds it and
-hands the residual itself on.
+hands the residual itself on, or its norm where one stands in front as well.
 """
 
 from __future__ import annotations
@@ -22,9 +22,9 @@ from dataclasses import dataclass
 
 import torch
 
-from ..models.config import (DeltaMixer, GatedLinearMixer, GroupedMixer, LatentMixer, LinearMixer, ParallelMixer, attention_shape,
-                             ceil8, sub_mixers)
-from ..models.layered import LayeredLayerWeights
+from ..models.config import (DeltaMixer, GatedLinearMixer, GroupedMixer, LatentMixer, LinearMixer, MemoryMixer, ParallelMixer,
+                             attention_shape, ceil8, sub_mixers)
+from ..models.layered import LayeredLayerWeights, rotary_table
 from ..ops import gemm
 from ..ops import mixers as M
 from ..ops.attention import decode_plan
@@ -88,7 +88,7 @@ class LayeredForward:
         def of(kind):
             return [m for m in mixers if isinstance(m, kind)]
 
-        lat, lin, grp, gla, delta = of(LatentMixer), of(LinearMixer), of(GroupedMixer), of(GatedLinearMixer), of(DeltaMixer)
+        lat, lin, grp, gla, delta, mem = (of(k) for k in (LatentMixer, LinearMixer, GroupedMixer, GatedLinearMixer, DeltaMixer, MemoryMixer))
         self.expands = [("exp_k" in lw.mix) for lw in layers]
         # only decoded tokens and short portions attend as single rows, in every layer
         self.all_expand = all(ex for lw, ex in zip(layers, self.expands) if isinstance(lw.spec.mixer, LatentMixer)) and \
@@ -112,9 +112,11 @@ class LayeredForward:
             self.lat_ws = buf(self.ws_tokens * max(w for *_, w in shapes))
             self.k_exp = buf(self.ws_tokens * max(H * dq for H, dq, _, _ in shapes))
             self.v_exp = buf(self.ws_tokens * max(H * dv for H, _, dv, _ in shapes))
+        # cos and sin of every position, one table for all layers of the same rotation
+        self.rot_tables = {rot: rotary_table(rot, engine.ecfg.max_seq_len, dev) for rot in {m.rot for m in grp if m.rot is not None}}
         if grp:
-            self.q_grp = buf(cap * max(m.kv_heads * M.group_pad(m.heads, m.kv_heads) * m.cache_rows[0][1] for m in grp))
-            need = max(b * m.heads * decode_plan(b, m.kv_heads, engine.ecfg.max_seq_len)[0] * (m.cache_rows[1][1] + 2)
+            self.q_grp = buf(cap * max(m.kv_heads * M.group_pad(m.heads, m.kv_heads) * m.row_shapes[0][1] for m in grp))
+            need = max(b * m.heads * decode_plan(b, m.kv_heads, engine.ecfg.max_seq_len)[0] * (m.row_shapes[1][1] + 2)
                        for b in engine._buckets for m in grp)
             self.grp_ws = buf(max(need, 1 << 20), torch.float32)
         if gla:
@@ -126,8 +128,15 @@ class LayeredForward:
         if delta:
             self.delta_ws = M.DeltaScratch.for_rows(cap, engine.max_seqs, max(m.heads for m in delta), max(m.kv_heads for m in delta),
                                                     max(m.dim for m in delta), max(m.vdim for m in delta), dt, dev)
-        if lin or gla or delta:
-            self.o_lin = buf(cap * max(m.out_features for m in lin + gla + delta), torch.float32)
+        if mem:
+            self.mem_ws = M.MemoryScratch.for_rows(cap, engine.max_seqs, max(m.heads for m in mem), max(m.dim for m in mem),
+                                                   max(m.vdim for m in mem), dev)
+        self.tails = buf(cap * max((lw.offs["end"] - lw.fp32_from for lw in layers if lw.fp32_from), default=0), torch.float32)
+        if cfg.token_side:
+            self.side = torch.zeros(cap, ceil8(cfg.token_side), dtype=dt, device=dev)[:, :cfg.token_side]
+            self.side_z = self.side if dt == torch.float32 else None
+        if lin or gla or delta or mem:
+            self.o_lin = buf(cap * max(m.out_features for m in lin + gla + delta + mem), torch.float32)
         if lin:
             self.lin_ws = buf(max(M.linear_attn_ws_elems(m.dim, m.vdim) for m in lin) if dt == torch.bfloat16 else 1, torch.float32)
 
@@ -194,16 +203,20 @@ class LayeredForward:
         k, v = kv.k[l], kv.v[l]
         gp = M.group_pad(m.heads, m.kv_heads)
         q = self.q_grp[:rows * m.kv_heads * gp * k.shape[3]].view(rows, m.kv_heads, gp, k.shape[3])
-        M.grouped_prep(proj, lw.mix["q_norm"], lw.mix["k_norm"], b.slots, k, v, q, heads=m.heads, dim=m.dim, vdim=m.vdim,
-                       offs=(o["q"], o["k"], o["v"]), eps=self.e.cfg.rms_norm_eps)
-        gate = proj[:, o["hg"]:o["hg"] + m.heads]
-        kw = dict(heads=m.heads, vdim=m.vdim, scale=m.scale, softcap=m.softcap)
+        if m.head_norms:
+            M.grouped_prep(proj, lw.mix["q_norm"], lw.mix["k_norm"], b.slots, k, v, q, heads=m.heads, dim=m.dim, vdim=m.vdim,
+                           offs=(o["q"], o["k"], o["v"]), eps=self.e.cfg.rms_norm_eps)
+            gate = proj[:, o["hg"]:o["hg"] + m.heads]
+        else:
+            self._conv_rope(l, lw, m, proj, q, b)
+            gate = proj[:, o["g"]:o["g"] + m.out_features]
+        kw = dict(heads=m.heads, vdim=m.vdim, scale=m.scale, softcap=m.softcap, window=m.window, keep_first=m.keep_first)
         if not self._tiled(m):
             M.grouped_attn(q, k, v, out, b.table, b.positions, b.slots, dim=m.dim, gate=gate, row_seq=b.row_seq, **kw)
             return
         n = b.n_abs
         if n:
-            splits, chunk = decode_plan(n, m.kv_heads, b.max_len)
+            splits, chunk = decode_plan(n, m.kv_heads, min(b.max_len, m.visible(b.max_len) + 32))   # a window's edges lie inside tiles
             if splits > 1 and n * m.heads * splits * (v.shape[3] + 2) > self.grp_ws.numel():
                 splits, chunk = 1, 0
             M.grouped_decode(q[:n], k, v, out[:n], b.table, b.positions, b.slots, dim=m.dim, gate=gate, row_seq=b.row_seq, num_splits=splits,
@@ -211,6 +224,34 @@ class LayeredForward:
         if n < rows:
             s = slice(b.n_short, b.n_seqs)
             M.grouped_prefill(q, k, v, out, b.table[s], b.q_starts[s], b.q_lens[s], b.ctx_lens[s], b.max_q, gate=gate, **kw)
+
+    def _conv_rope(self, l: int, lw: LayeredLayerWeights, m: GroupedMixer, proj: torch.Tensor, q: torch.Tensor, b: RowBatch) -> None:
+        o, kv, nd = lw.offs, self.e.kv, b.n_dec
+        offs = (o["q"], o["k"], o["v"]) if m.kv_from is None else (o["q"],)
+        kw = dict(heads=m.heads, dim=m.dim, vdim=m.vdim, offs=offs)
+        args = (lw.mix["conv"], kv.conv[l], self.rot_tables.get(m.rot))
+        if nd:
+            M.conv_rope(proj[:nd], *args, b.positions, b.slots, b.state_slots, kv.k[l], kv.v[l], q, **kw)
+        if nd < b.n_seqs:
+            s = slice(nd, b.n_seqs)
+            M.conv_rope(proj, *args, b.positions, b.slots, b.state_slots[s], kv.k[l], kv.v[l], q, q_starts=b.q_starts[s], q_lens=b.q_lens[s],
+                        max_q=b.max_q, **kw)
+
+    def _memory(self, l: int, lw: LayeredLayerWeights, m: MemoryMixer, proj: torch.Tensor, out: torch.Tensor, b: RowBatch) -> None:
+        o, n, nd, eps = lw.offs, m.out_features, b.n_dec, self.e.cfg.rms_norm_eps
+        state = self.e.kv.states[l]
+        gates = self._tail(lw, proj, b.rows)
+        kw = dict(heads=m.heads, dim=m.dim, vdim=m.vdim, cap=m.gate_cap,
+                  offs=(*(o[c] for c in "qkvg"), o["i"] - lw.fp32_from, o["f"] - lw.fp32_from))
+        if nd:
+            M.memory_decode(proj[:nd], gates, state, lw.mix["norm"], out[:nd], b.positions, b.slots, b.state_slots, eps=eps, **kw)
+        if nd < b.n_seqs:
+            s = slice(nd, b.n_seqs)
+            y = self.o_lin[:b.rows * n].view(b.rows, n)
+            segs, seg_tokens = M.linear_attn_plan(b.n_seqs - nd, m.heads, m.dim, m.vdim, b.max_q)
+            M.memory_prefill(proj, gates, state, y, b.positions, b.slots, b.state_slots[s], b.q_starts[s], b.q_lens[s], b.max_q, self.mem_ws,
+                             segs=segs, seg_tokens=seg_tokens, **kw)
+            M.head_gate(y[nd:], lw.mix["norm"], proj[nd:, o["g"]:o["g"] + n], eps, out[nd:], heads=m.heads)
 
     def _gated_linear(self, l: int, lw: LayeredLayerWeights, m: GatedLinearMixer, proj: torch.Tensor, out: torch.Tensor, b: RowBatch) -> None:
         o, w, n, nd, eps = lw.offs, lw.mix, m.out_features, b.n_dec, self.e.cfg.rms_norm_eps
@@ -242,14 +283,23 @@ class LayeredForward:
             M.delta_prefill(proj, conv, w, state, y, b.positions, b.slots, b.state_slots[s], b.q_starts[s], b.q_lens[s], b.max_q, self.delta_ws, **kw)
             M.head_gate(y[nd:], w.norm, proj[nd:, o["g"]:o["g"] + n], eps, out[nd:])
 
-    _RUN = {LatentMixer: _latent, LinearMixer: _linear, GroupedMixer: _grouped, GatedLinearMixer: _gated_linear, DeltaMixer: _delta}
+    _RUN = {LatentMixer: _latent, LinearMixer: _linear, GroupedMixer: _grouped, GatedLinearMixer: _gated_linear, DeltaMixer: _delta,
+            MemoryMixer: _memory}
 
     # ------------------------------------------------------------------ layers
+    def _tail(self, lw: LayeredLayerWeights, proj: torch.Tensor, rows: int) -> torch.Tensor | None:
+        """Where the layer's fp32 columns of the product are: a buffer of their own, or the product itself in an fp32 model."""
+        if not lw.fp32_from:
+            return None
+        n = lw.offs["end"] - lw.fp32_from
+        return proj[:, lw.fp32_from:] if self.dtype == torch.float32 else self.tails[:rows * n].view(rows, n)
+
     def _mix(self, l: int, lw: LayeredLayerWeights, x: torch.Tensor, b: RowBatch) -> tuple[torch.Tensor, list[torch.Tensor]]:
         """The layer's projection, and the outputs of its mixer (of both sides of a pair) behind their output products."""
         rows = b.rows
         proj = self.proj[:rows * lw.offs["end"]].view(rows, lw.offs["end"])
-        gemm.linear(x, lw.proj, out=proj, bias=lw.proj_bias, silu_cols=lw.silu_cols)
+        tail = self._tail(lw, proj, rows) if self.dtype != torch.float32 else None
+        gemm.linear(x, lw.proj, out=proj, bias=lw.proj_bias, silu_cols=lw.silu_cols, tail=tail)
         ys, at = [], 0
         for i, m in enumerate(sub_mixers(lw.spec.mixer)):
             n = m.out_features
@@ -262,9 +312,10 @@ class LayeredForward:
         return proj, ys
 
     def _enter(self, resid: torch.Tensor, norm, x: torch.Tensor, pending: dict) -> None:
-        """Adds the pending sublayer output to the residual and prepares the next sublayer's input."""
+        """Adds the pending sublayer output to the residual and prepares the next sublayer's input (``norm``: the one in front
+        of it)."""
         if self.e.cfg.output_norm:
-            M.post_norm(resid, x, **pending)
+            M.post_norm(resid, x, out_norm=norm if self.e.cfg.input_norm else None, **pending)
         else:
             M.resid_norm(resid, norm, x, **pending)
 
@@ -272,25 +323,40 @@ class LayeredForward:
         """Embedding and all layers over the batch's rows; the last sublayer's output stays pending for :meth:`head`."""
         rows, hid = b.rows, self.e.cfg.hidden_size
         resid, x, x2 = self.resid[:rows], self.x[:rows], self.x2[:rows]
-        post = self.e.cfg.output_norm
+        cfg = self.e.cfg
+        post = cfg.output_norm
         pending: dict = dict(ids=ids, table=self.e.w.embed)
+        if cfg.embed_scale != 1.0:
+            pending["embed_scale"] = cfg.embed_scale
         for l, lw in enumerate(self.layers):
             self._enter(resid, lw.norm1, x, pending)
             proj, ys = self._mix(l, lw, x, b)
             if post:
-                pending = dict(branches=ys, branch_norms=lw.branch_norms, norm=lw.norm1)
+                pending = dict(branches=ys, branch_norms=lw.branch_norms, norm=lw.norm1b or lw.norm1)
             else:
                 pending = dict(parts=ys, gate=proj[:, lw.offs["rg"]:lw.offs["rg"] + hid])
             if lw.norm2 is not None:
                 self._enter(resid, lw.norm2, x2, pending)
                 if post:
-                    pending = dict(branches=self.e.port.run(l, x2, rows, mode), norm=lw.norm2)
+                    pending = dict(branches=self.e.port.run(l, x2, rows, mode), norm=lw.norm2b or lw.norm2)
                 else:
                     rg2 = self.rg2[:rows]
                     gemm.linear(x2, lw.rg2, out=rg2, bias=lw.rg2_bias)
                     pending = dict(parts=self.e.port.run(l, x2, rows, mode), gate=rg2)
+            if lw.side_gate is not None:
+                pending = self._token_side(l, lw, resid, x, ids, pending)
             self.tap(l, rows, pending)
         self._pending = pending
+
+    def _token_side(self, l: int, lw: LayeredLayerWeights, resid: torch.Tensor, x: torch.Tensor, ids: torch.Tensor, pending: dict) -> dict:
+        """``gelu_tanh(side_gate x)`` times the layer's part of the token's second embedding, mapped back to the model width;
+        ``x`` is the residual itself."""
+        rows, n = x.shape[0], self.e.cfg.token_side
+        M.post_norm(resid, x, **pending)
+        e = self.side[:rows]
+        M.token_gate(x, lw.side_gate, self.e.w.extra["side_embed"][:, l * n:(l + 1) * n], ids, e, self.side_z[:rows] if self.side_z is not None else None)
+        gemm.linear(e, lw.side_proj, out=self.y[:rows])
+        return dict(branches=[self.y[:rows]], norm=lw.side_norm)
 
     def tap(self, layer: int, rows: int, pending: dict) -> None:
         """Called after every layer with its output still pending; a debugging subclass or test may look at it."""

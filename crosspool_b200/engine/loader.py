@@ -245,6 +245,8 @@ def _moe_reads(l: MoeFfnSpec, rank: int, size: int, experts: range, packed_weigh
         reads["shared_gate"] = TensorRead(l.shared_gate_key, rows=srows)
         reads["shared_up"] = TensorRead(l.shared_up_key, rows=srows)
         reads["shared_down"] = TensorRead(l.shared_down_key, cols=srows)
+    if l.shared_scale_key:
+        reads["shared_scale"] = TensorRead(l.shared_scale_key)
     return reads
 
 
@@ -287,8 +289,8 @@ def materialize_layer_weights(spec: FfnModelSpec, view: CheckpointKeyView, layer
         if l.activation == ActivationKind.POLYNORM:
             w.extra["polynorm"] = (got["act_coef"].contiguous(), l.activation_eps)
         t = l.gate_transform
-        if t is not None and (t.limit > 0 or t.up_offset != 0 or t.alpha != 1.0):
-            w.extra["gate_transform"] = (float(t.limit), float(t.up_offset), float(t.alpha))
+        if t is not None and not t.plain:
+            w.extra["gate_transform"] = t.constants()
         return w
     gate_up = torch.stack([torch.cat([got[f"gate{e}"], got[f"up{e}"]], 0) for e in experts])
     down = torch.stack([got[f"down{e}"] for e in experts])
@@ -298,12 +300,12 @@ def materialize_layer_weights(spec: FfnModelSpec, view: CheckpointKeyView, layer
     if f"down_bias{experts[0]}" in got:
         w.down_bias = torch.stack([got[f"down_bias{e}"] for e in experts]).contiguous()
     t = l.gate_transform
-    if t is not None and (t.limit > 0 or t.up_offset != 0 or t.alpha != 1.0):
-        w.extra["gate_transform"] = (float(t.limit), float(t.up_offset), float(t.alpha))
+    if t is not None and not t.plain:
+        w.extra["gate_transform"] = t.constants()
     if "shared_gate" in got:
         w.shared_gate_up = torch.cat([got["shared_gate"], got["shared_up"]], 0)
         w.shared_down = got["shared_down"]
-    for k in ("router_bias", "correction_bias"):
+    for k in ("router_bias", "correction_bias", "shared_scale"):
         if k in got:
             w.extra[k] = got[k]
     w.extra["experts"] = (experts.start, experts.stop)

@@ -51,11 +51,23 @@ class LayerKind(str, Enum):
 @dataclass(frozen=True)
 class GateTransform:
     """``act(min(g, limit)) * (clamp(u, -limit, limit) + up_offset)``; ``limit <= 0`` disables clamping.
-    ``alpha`` generalises SiLU to ``g * sigmoid(alpha * g)`` (GPT-OSS uses 1.702, limit 7, offset 1)."""
+    ``alpha`` and ``cubic`` generalise SiLU to ``g * sigmoid(alpha * g * (1 + cubic * g^2))`` (GPT-OSS uses alpha 1.702, limit
+    7, offset 1; the tanh form of GELU is alpha 2 sqrt(2 / pi), cubic 0.044715)."""
 
     limit: float = 0.0
     up_offset: float = 0.0
     alpha: float = 1.0
+    cubic: float = 0.0
+
+    @property
+    def plain(self) -> bool:
+        """SiLU as it is."""
+        return self.limit <= 0 and self.up_offset == 0 and self.alpha == 1.0 and self.cubic == 0
+
+    def constants(self) -> tuple[float, ...]:
+        """(limit, up offset, alpha), and the cubic term where there is one."""
+        t = (float(self.limit), float(self.up_offset), float(self.alpha))
+        return t + (float(self.cubic),) if self.cubic else t
 
 
 @dataclass(frozen=True)
@@ -139,6 +151,8 @@ class MoeFfnSpec:
     gate_transform: GateTransform = GateTransform()
     source_order: GateUpOrder = GateUpOrder.CONCATENATED
     kind: LayerKind = LayerKind.MOE
+    identity_experts: int = 0            # router outputs behind the experts that stand for the layer's input itself
+    shared_scale_key: str | None = None  # one row: the shared experts' output is multiplied by sigmoid of its product
 
     @property
     def effective_topk(self) -> int:
@@ -187,7 +201,7 @@ class FfnModelSpec:
             else:
                 keys.add(l.router_weight_key)
                 for k in (l.router_bias_key, l.correction_bias_key, l.shared_gate_key, l.shared_up_key,
-                          l.shared_down_key):
+                          l.shared_down_key, l.shared_scale_key):
                     if k:
                         keys.add(k)
                 ex = l.experts

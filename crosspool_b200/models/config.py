@@ -10,6 +10,7 @@ architecture adapters). The reference reads the same fields through ``FfnSourceC
 from __future__ import annotations
 
 import json
+import math
 from dataclasses import dataclass, field, replace
 from pathlib import Path
 from typing import Any
@@ -33,12 +34,24 @@ class MlaShape:
 
 
 @dataclass(frozen=True)
+class RotaryScaling:
+    """Rotary frequencies for contexts beyond ``original`` tokens: wavelengths above ``original / low`` are stretched by
+    ``factor``, those below ``original / high`` are kept, the ones between blend linearly in ``original / wavelength``."""
+
+    factor: float
+    low: float
+    high: float
+    original: float
+
+
+@dataclass(frozen=True)
 class RotarySpec:
     """Rotary positions on the first ``dims`` dimensions of a vector, paired (i, i + dims / 2): the pair at position p
-    turns by ``p * base ** (-2 i / dims)``."""
+    turns by ``p * f_i``, ``f_i = base ** (-2 i / dims)``, scaled where there is a ``scaling``."""
 
     dims: int
     base: float
+    scaling: RotaryScaling | None = None
 
 
 def ceil8(n: int) -> int:
@@ -106,8 +119,12 @@ class _RecurrentMixer:
         return 0
 
     @property
+    def state_shape(self) -> tuple[int, ...]:
+        return (self.heads, self.dim, self.vdim)
+
+    @property
     def state_elems(self) -> int:
-        return self.heads * self.dim * self.vdim
+        return math.prod(self.state_shape)
 
     @property
     def out_features(self) -> int:
@@ -131,9 +148,14 @@ class LinearMixer(_RecurrentMixer):
 
 @dataclass(frozen=True)
 class GroupedMixer:
-    """Grouped-query softmax attention without positions: ``heads`` query heads share ``kv_heads`` cached keys and values,
-    queries and keys are RMS-normed per head, scores saturate at +-``softcap`` (0: they do not), and a sigmoid per head
-    gates the output."""
+    """Grouped-query softmax attention: ``heads`` query heads share ``kv_heads`` cached keys and values, scores saturate at
+    +-``softcap`` (0: they do not), and a sigmoid gates the output.
+
+    ``head_norms``: projections have biases, queries and keys are RMS-normed per head, the gate is one number per head.
+    Without: none of these, and the gate is one number per output element. ``conv``: queries, keys and values pass a causal
+    convolution of that many taps before anything else (0: none). ``window``: a token sees itself and the ``window - 1``
+    tokens before it, and the first ``keep_first`` tokens of the sequence (0: all before it). ``kv_from``: the layer has no
+    keys and values of its own and reads those that layer caches."""
 
     heads: int
     kv_heads: int
@@ -141,13 +163,23 @@ class GroupedMixer:
     vdim: int
     scale: float
     softcap: float = 0.0
+    head_norms: bool = True
+    conv: int = 0
+    rot: RotarySpec | None = None
+    window: int = 0
+    keep_first: int = 0
+    kv_from: int | None = None
     kind: str = "grouped_attention"
 
     @property
-    def cache_rows(self) -> tuple[tuple[int, int], ...]:
+    def row_shapes(self) -> tuple[tuple[int, int], ...]:
         """(heads, elements per head) of a token's key and value rows, padded to the widths of the tensor-core kernels
         where one covers the sizes."""
         return tuple((self.kv_heads, n) for n in attention_shape(self.dim, self.vdim) or (ceil8(self.dim), ceil8(self.vdim)))
+
+    @property
+    def cache_rows(self) -> tuple[tuple[int, int], ...]:
+        return () if self.kv_from is not None else self.row_shapes
 
     @property
     def cache_width(self) -> int:
@@ -158,10 +190,25 @@ class GroupedMixer:
         return 0
 
     @property
+    def conv_channels(self) -> int:
+        """Channels that pass the convolution: queries, and the layer's own keys and values."""
+        return self.heads * self.dim + (0 if self.kv_from is not None else self.kv_heads * (self.dim + self.vdim))
+
+    @property
+    def conv_state_elems(self) -> int:
+        return self.conv * self.conv_channels
+
+    @property
     def out_features(self) -> int:
         return self.heads * self.vdim
 
+    def visible(self, length: int) -> int:
+        """Bound on the tokens a query at the end of ``length`` tokens sees."""
+        return min(length, self.window + self.keep_first) if self.window else length
+
     def param_count(self, hidden: int) -> int:
+        if not self.head_norms:
+            return hidden * (self.conv_channels + 2 * self.out_features) + self.conv_state_elems
         kv = self.kv_heads * (self.dim + self.vdim)
         return ((hidden + 1) * (self.heads * self.dim + kv) + 2 * self.dim + hidden * (self.heads + self.out_features + 1))
 
@@ -212,6 +259,31 @@ class DeltaMixer(_RecurrentMixer):
 
 
 @dataclass(frozen=True)
+class MemoryMixer(_RecurrentMixer):
+    """Matrix memory with exponential gates: the state decays by a forget gate and takes a key's value in by an input gate,
+    both as logarithms that saturate at +-``gate_cap`` before the forget gate's sigmoid; a vector of decayed keys normalises
+    what is read, and a running maximum of the logarithms scales all three."""
+
+    heads: int
+    dim: int
+    vdim: int
+    gate_cap: float
+    kind: str = "mlstm"
+
+    @property
+    def head_state(self) -> int:
+        """fp32 elements of a head: the matrix, the key sum and the maximum, rounded up to whole 16 bytes."""
+        return (self.dim * self.vdim + self.dim + 1 + 3) // 4 * 4
+
+    @property
+    def state_shape(self) -> tuple[int, ...]:
+        return (self.heads, self.head_state)
+
+    def param_count(self, hidden: int) -> int:
+        return hidden * self.heads * (2 * self.dim + 3 * self.vdim + 2) + self.out_features + 2 * self.heads
+
+
+@dataclass(frozen=True)
 class ParallelMixer:
     """Two mixers that read the same input; half the sum of their outputs, each RMS-normed over the model width first."""
 
@@ -244,25 +316,63 @@ def sub_mixers(m) -> tuple:
     return (m.left, m.right) if isinstance(m, ParallelMixer) else (m,)
 
 
-Mixer = LatentMixer | LinearMixer | GroupedMixer | GatedLinearMixer | DeltaMixer | ParallelMixer
+Mixer = LatentMixer | LinearMixer | GroupedMixer | GatedLinearMixer | DeltaMixer | MemoryMixer | ParallelMixer
 
 
 GLU_ALPHA = 1.702    # slope of the sigmoid in the clamped gated activation
 
 
+# g sigmoid(alpha g (1 + cubic g^2)): the tanh form of gelu as a gated activation
+GELU_ALPHA = 2.0 * math.sqrt(2.0 / math.pi)
+GELU_CUBIC = 0.044715
+
+
+@dataclass(frozen=True)
+class MoeSpec:
+    """Routed FFN of a layered decoder: ``experts`` gated (silu) FFNs of ``ff`` features and ``identity`` experts that return
+    their input; a token takes ``top`` of them by softmax score plus a correction, weighted by their scores normalised to
+    ``scale``. ``shared_ff`` > 0: one more expert for every token, its output times a sigmoid per token."""
+
+    experts: int
+    top: int
+    ff: int
+    identity: int = 0
+    scale: float = 1.0
+    shared_ff: int = 0
+
+    @property
+    def routed(self) -> int:
+        """Outputs of the router."""
+        return self.experts + self.identity
+
+
 @dataclass(frozen=True)
 class LayerSpec:
-    """One layer of a layered (hybrid) decoder: its mixer and the width of its FFN (0: no FFN). ``gate_limit`` > 0: the FFN
-    is gated and clamped, ``min(g, limit) sigmoid(1.702 g) (clamp(u, +-limit) + 1)``; otherwise it is ungated."""
+    """One layer of a layered (hybrid) decoder: its mixer and the width of its FFN (0: no FFN, or a routed one, ``moe``).
+    ``gate_limit`` > 0: the FFN is gated and clamped, ``min(g, limit) sigmoid(1.702 g) (clamp(u, +-limit) + 1)``; ``gelu``: it
+    is gated, ``gelu_tanh(g) u``; otherwise it is ungated."""
 
     mixer: Mixer
     ff: int = 0
     gate_limit: float = 0.0
+    gelu: bool = False
+    moe: MoeSpec | None = None
+
+    @property
+    def has_ffn(self) -> bool:
+        return self.ff > 0 or self.moe is not None
 
     @property
     def ffn_maps(self) -> int:
         """Matrices of ``hidden x ff`` elements."""
-        return 3 if self.gate_limit > 0 else 2
+        return 3 if self.gate_limit > 0 or self.gelu else 2
+
+    def ffn_params(self, hidden: int) -> int:
+        m = self.moe
+        if m is None:
+            return self.ffn_maps * hidden * self.ff
+        shared = hidden * (3 * m.shared_ff + 1) if m.shared_ff else 0
+        return 3 * m.experts * hidden * m.ff + m.routed * (hidden + 1) + shared
 
 
 @dataclass(frozen=True)
@@ -305,10 +415,16 @@ class ModelConfig:
     mla: MlaShape | None = None
     # Layered decoders: every layer names its own mixer and FFN. norm "dyt" is dynamic tanh (elementwise, no statistics);
     # ``residual_gate``: each sublayer's result is multiplied by sigmoid(W h + b) of its input and summed in fp32.
-    # ``output_norm``: sublayers read the residual itself, and their results are normed before they are added to it.
+    # ``output_norm``: sublayers' results are normed before they are added to the residual, which the sublayers read as it
+    # is, or with ``input_norm`` through a norm of their own.
+    # ``token_side`` > 0: behind the FFN every layer adds a small gated map of the residual and of a second embedding of its
+    # token (that many dimensions per layer).
     layer_specs: tuple[LayerSpec, ...] = ()
     residual_gate: bool = False
     output_norm: bool = False
+    input_norm: bool = False
+    token_side: int = 0
+    embed_scale: float = 1.0
     logit_scale: float = 1.0
     extra: dict[str, Any] = field(default_factory=dict, compare=False, hash=False)
 
@@ -318,8 +434,9 @@ class ModelConfig:
 
     @property
     def recurrent(self) -> bool:
-        """Some layer carries a per-sequence state, which cannot be shared between sequences like a cache page."""
-        return any(s.mixer.state_elems for s in self.layer_specs)
+        """Some layer carries a per-sequence state (or a convolution's inputs), which cannot be shared between sequences like
+        a cache page."""
+        return any(s.mixer.state_elems or getattr(s.mixer, "conv_state_elems", 0) for s in self.layer_specs)
 
     @property
     def gpu_attention_supported(self) -> bool:
@@ -354,9 +471,11 @@ class ModelConfig:
         if self.layered:
             norm = 2 * self.hidden_size + 1 if self.norm == "dyt" else self.hidden_size
             n = self.hidden_size * self.vocab_size * (1 if self.tie_word_embeddings else 2) + norm
+            if self.token_side:
+                n += self.num_layers * (self.token_side * (self.vocab_size + 2 * self.hidden_size) + norm)
             for s in self.layer_specs:
-                subs = 1 + (s.ff > 0)
-                n += s.mixer.param_count(self.hidden_size) + subs * norm
+                subs = 1 + s.has_ffn
+                n += s.mixer.param_count(self.hidden_size) + subs * norm * (2 if self.input_norm else 1)
                 if self.residual_gate:
                     n += subs * self.hidden_size * (self.hidden_size + 1)
             return 2 * n
@@ -367,7 +486,7 @@ class ModelConfig:
 
     def ffn_param_bytes_per_layer(self, layer: int = 0) -> int:
         if self.layered:
-            return 2 * self.layer_specs[layer].ffn_maps * self.hidden_size * self.layer_specs[layer].ff
+            return 2 * self.layer_specs[layer].ffn_params(self.hidden_size)
         if self.layer_is_moe(layer):
             e = self.num_experts * 3 * self.hidden_size * self.moe_intermediate_size
             e += self.num_experts * self.hidden_size
@@ -505,7 +624,78 @@ def saninex_config(cfg: dict[str, Any], name: str = "") -> ModelConfig:
         hidden_act="clamped_glu", max_position_embeddings=1 << 30, norm="rmsnorm", layer_specs=tuple(specs), output_norm=True)
 
 
-LAYERED_CONFIGS = {"Segirax": segirax_config, "Saninex": saninex_config}
+def _rotary(r: dict[str, Any] | None, dim: int) -> RotarySpec | None:
+    if not r:
+        return None
+    sc = r.get("scaling")
+    rot = RotarySpec(int(r["dims"]), float(r["base"]),
+                     RotaryScaling(*(float(sc[n]) for n in ("factor", "low", "high", "original"))) if sc else None)
+    if rot.dims % 2 or not 0 < rot.dims <= dim:
+        raise ValueError(f"rotary dims {rot.dims} do not fit a head of {dim}")
+    return rot
+
+
+def _kadavik_attention(m: dict[str, Any]) -> GroupedMixer:
+    _grouped_heads(m)
+    mask = m.get("mask") or {}
+    window, keep = int(mask.get("size") or 0), int(mask.get("keep_first") or 0)
+    if window < 0 or keep < 0 or (mask and not window):
+        raise ValueError(f"attention mask {mask!r} is not a window")
+    kv_from = m.get("kv_from")
+    return GroupedMixer(**_ints(m, "heads", "kv_heads", "dim", "vdim"), scale=float(m["scale"]), head_norms=False,
+                        conv=int(m.get("conv") or 0), rot=_rotary(m.get("rot"), int(m["dim"])), window=window,
+                        keep_first=keep, kv_from=None if kv_from is None else int(kv_from))
+
+
+def _kadavik_mlp(mixer: Mixer, mlp: dict[str, Any] | None) -> LayerSpec:
+    if mlp is None:
+        return LayerSpec(mixer)
+    if mlp["kind"] == "dense":
+        return LayerSpec(mixer, int(mlp["ff"]), gelu=True)
+    if mlp["kind"] != "moe":
+        raise ValueError(f"unsupported feed-forward kind {mlp['kind']!r}")
+    r, shared = mlp["router"], mlp.get("shared")
+    moe = MoeSpec(int(r["experts"]), int(r["top"]), int(mlp["expert"]["ff"]), int(r.get("identity") or 0), float(r["scale"]),
+                  int(shared["ff"]) if shared else 0)
+    if not 0 < moe.top <= min(moe.routed, 32) or moe.routed > 256 or moe.experts < 1:
+        raise ValueError(f"a router of {moe.routed} outputs that takes {moe.top} is not supported (at most 32 of 256)")
+    return LayerSpec(mixer, moe=moe)
+
+
+def kadavik_config(cfg: dict[str, Any], name: str = "") -> ModelConfig:
+    """Kadavik: norms before and behind every sublayer, matrix memories (mlstm) and windowed grouped-query attention with short
+    convolutions in any order, attention layers that read another layer's keys and values, gelu or routed FFNs, and a second
+    token embedding that every layer adds through a gate; its ``config.json`` lists every layer."""
+    specs: list[LayerSpec] = []
+    for i, l in enumerate(cfg["layers"]):
+        m = l["mixer"]
+        if l["type"] == "mlstm":
+            mixer: Mixer = MemoryMixer(**_ints(m, "heads", "dim", "vdim"), gate_cap=float(m["gate_cap"]))
+            if not mixer.gate_cap > 0:
+                raise ValueError(f"gate cap {mixer.gate_cap} is not positive")
+        elif l["type"] == "attention":
+            mixer = _kadavik_attention(m)
+            if mixer.kv_from is not None:
+                src = specs[mixer.kv_from].mixer if 0 <= mixer.kv_from < i else None
+                if not isinstance(src, GroupedMixer) or src.kv_from is not None or \
+                        (src.kv_heads, src.dim, src.vdim) != (mixer.kv_heads, mixer.dim, mixer.vdim):
+                    raise ValueError(f"layer {i} cannot read the keys and values of layer {mixer.kv_from}")
+        else:
+            raise ValueError(f"unsupported mixer {l['type']!r}")
+        specs.append(_kadavik_mlp(mixer, l.get("mlp")))
+    first = specs[0].mixer
+    side = cfg.get("token_side")
+    return ModelConfig(
+        name=name or cfg["architecture"], architecture=cfg["architecture"], hidden_size=int(cfg["width"]), num_layers=len(specs),
+        num_q_heads=first.heads, num_kv_heads=getattr(first, "kv_heads", first.heads), head_dim=first.dim,
+        intermediate_size=max(s.moe.ff if s.moe else s.ff for s in specs), vocab_size=int(cfg["vocab"]),
+        rms_norm_eps=float(cfg["norm"]["eps"]), qk_norm=False, tie_word_embeddings=True, hidden_act="gelu_pytorch_tanh",
+        max_position_embeddings=1 << 30, layer_specs=tuple(specs), output_norm=True, input_norm=True,
+        token_side=int(side["dim"]) if side else 0, embed_scale=float((cfg.get("embedding") or {}).get("scale", 1.0)),
+        logit_scale=float(cfg.get("logit_scale", 1.0)))
+
+
+LAYERED_CONFIGS = {"Segirax": segirax_config, "Saninex": saninex_config, "Kadavik": kadavik_config}
 
 
 def from_hf_config(cfg: dict[str, Any], name: str = "") -> ModelConfig:

@@ -15,20 +15,21 @@ from typing import Callable
 import torch
 
 from ..ops.mixers import DeltaWeights, NormParams, decay_powers, expanded_shape
-from .config import DeltaMixer, GatedLinearMixer, GroupedMixer, LatentMixer, LayerSpec, LinearMixer, ModelConfig, ParallelMixer, ceil8
+from .config import (DeltaMixer, GatedLinearMixer, GroupedMixer, LatentMixer, LayerSpec, LinearMixer, MemoryMixer, ModelConfig,
+                     ParallelMixer, RotarySpec, ceil8)
 
 # get(name, shape): the checkpoint tensor (or a random one) of that name; a size of 0 is whatever the checkpoint has
 Getter = Callable[[str, tuple[int, ...]], torch.Tensor]
 
 
 def pad_pitch(w: torch.Tensor) -> torch.Tensor:
-    """``[n, k]`` with a row pitch of whole 16-byte units (zeros behind the k columns)."""
-    n, k = w.shape
+    """``[..., n, k]`` with a row pitch of whole 16-byte units (zeros behind the k columns)."""
+    *lead, k = w.shape
     if k % 8 == 0:
         return w.contiguous()
-    out = torch.zeros(n, ceil8(k), dtype=w.dtype, device=w.device)
-    out[:, :k] = w
-    return out[:, :k]
+    out = torch.zeros(*lead, ceil8(k), dtype=w.dtype, device=w.device)
+    out[..., :k] = w
+    return out[..., :k]
 
 
 @dataclass
@@ -47,6 +48,12 @@ class LayeredLayerWeights:
     rg2: torch.Tensor | None = None         # residual gate of the FFN
     rg2_bias: torch.Tensor | None = None
     silu_cols: int = 0                      # leading columns of the product that are stored through silu
+    norm1b: NormParams | None = None        # behind the mixer, where norm1 stands in front of it (ModelConfig.input_norm)
+    norm2b: NormParams | None = None        # ... behind the FFN
+    fp32_from: int = 0                      # columns of the product from here on are wanted in fp32 (0: none are)
+    side_gate: torch.Tensor | None = None   # token side: [dim, hidden], [hidden, dim], its norm
+    side_proj: torch.Tensor | None = None
+    side_norm: NormParams | None = None
 
 
 def _fuse(sections: list[tuple[str, torch.Tensor]]) -> tuple[torch.Tensor, dict[str, int]]:
@@ -70,6 +77,18 @@ def _norm(get: Getter, name: str, cfg: ModelConfig) -> NormParams:
 
 def rotary_frequencies(dims: int, base: float) -> torch.Tensor:
     return float(base) ** (-2.0 * torch.arange(dims // 2, dtype=torch.float64) / dims)
+
+
+def rotary_table(rot: RotarySpec, positions: int, device) -> torch.Tensor:
+    """cos and sin of every position's angles, fp32 ``[positions, dims / 2, 2]`` rounded from double."""
+    f = rotary_frequencies(rot.dims, rot.base).to(device)
+    sc = rot.scaling
+    if sc is not None:
+        turns = sc.original * f / (2 * torch.pi)             # of the original context: original / wavelength
+        blend = ((turns - sc.low) / (sc.high - sc.low)).clamp(0, 1) if sc.high > sc.low else (turns >= sc.low).double()
+        f = f * (blend + (1 - blend) / sc.factor)
+    a = torch.arange(positions, dtype=torch.float64, device=device)[:, None] * f
+    return torch.stack([a.cos(), a.sin()], -1).float().contiguous()
 
 
 def _latent(m: LatentMixer, get: Getter, p: str, hidden: int, dtype: torch.dtype, device) -> tuple[list, dict]:
@@ -123,6 +142,50 @@ def _delta(m: DeltaMixer, get: Getter, p: str, hidden: int) -> tuple[list, dict]
     return [(n, get(p + n, (r, hidden))) for n, r in rows.items()], {"delta": w}
 
 
+def _windowed(m: GroupedMixer, get: Getter, p: str, hidden: int) -> tuple[list, dict]:
+    """Grouped-query attention without head norms; a layer that reads another layer's keys and values has queries only."""
+    rows = {"q": m.heads * m.dim}
+    if m.kv_from is None:
+        rows.update(k=m.kv_heads * m.dim, v=m.kv_heads * m.vdim)
+    mix = {"conv": torch.cat([get(f"{p}{n}.conv", (r, m.conv)).float() for n, r in rows.items()], 0).t().contiguous() if m.conv else None}
+    return [(n, get(p + n, (r, hidden))) for n, r in {**rows, "g": m.out_features}.items()], mix
+
+
+def _memory(m: MemoryMixer, get: Getter, p: str, hidden: int) -> tuple[list, dict, dict]:
+    rows = {"q": m.heads * m.dim, "k": m.heads * m.dim, "v": m.out_features, "g": m.out_features, "i": m.heads, "f": m.heads}
+    return ([(n, get(p + n, (r, hidden))) for n, r in rows.items()], {n: get(f"{p}{n}.b", (m.heads,)).float() for n in "if"},
+            {"norm": get(p + "norm", (m.out_features,)).float().contiguous()})
+
+
+def _plain_norm(get: Getter, name: str, cfg: ModelConfig) -> NormParams:
+    return NormParams("rmsnorm", get(name, (cfg.hidden_size,)).float().contiguous(), eps=cfg.rms_norm_eps)
+
+
+def _input_output_norm_layer(cfg: ModelConfig, i: int, spec: LayerSpec, get: Getter, device) -> LayeredLayerWeights:
+    """A layer with a norm in front of and behind each sublayer, and perhaps a token side."""
+    h, m, p = cfg.hidden_size, spec.mixer, f"l{i}."
+    biases: dict = {}
+    if isinstance(m, MemoryMixer):
+        sections, biases, mix = _memory(m, get, p + "mix.", h)
+    else:
+        sections, mix = _windowed(m, get, p + "mix.", h)
+    proj, offs = _fuse(sections)
+    bias = None
+    if biases:
+        bias = torch.zeros(offs["end"], dtype=torch.float32, device=device)
+        for n, b in biases.items():
+            bias[offs[n]:offs[n] + b.shape[0]] = b
+    lw = LayeredLayerWeights(spec, _plain_norm(get, p + "norm1", cfg), proj, bias, offs, pad_pitch(get(p + "mix.o", (h, m.out_features))), mix,
+                             norm1b=_plain_norm(get, p + "norm1b", cfg), fp32_from=offs.get("i", 0))
+    if spec.has_ffn:
+        lw.norm2, lw.norm2b = (_plain_norm(get, p + n, cfg) for n in ("norm2", "norm2b"))
+    if cfg.token_side:
+        lw.side_gate = pad_pitch(get(p + "side.gate", (cfg.token_side, h)))
+        lw.side_proj = pad_pitch(get(p + "side.proj", (h, cfg.token_side)))
+        lw.side_norm = _plain_norm(get, p + "side.norm", cfg)
+    return lw
+
+
 def _centred_norm(get: Getter, name: str, cfg: ModelConfig) -> NormParams:
     """An RMS norm whose weight is stored as its distance from one."""
     return NormParams("rmsnorm", 1.0 + get(name, (cfg.hidden_size,)).float(), eps=cfg.rms_norm_eps)
@@ -162,6 +225,9 @@ def layered_attention_weights(cfg: ModelConfig, get: Getter, device, dtype: torc
     h = cfg.hidden_size
     layers = []
     for i, spec in enumerate(cfg.layer_specs):
+        if cfg.input_norm:
+            layers.append(_input_output_norm_layer(cfg, i, spec, get, device))
+            continue
         if cfg.output_norm:
             layers.append(_output_norm_layer(cfg, i, spec, get, device))
             continue
@@ -183,8 +249,11 @@ def layered_attention_weights(cfg: ModelConfig, get: Getter, device, dtype: torc
             lw.silu_cols = offs["g"]            # q, k and v
         layers.append(lw)
     embed = get("embed", (cfg.vocab_size, h)).contiguous()
-    final = (_centred_norm if cfg.output_norm else _norm)(get, "final.norm", cfg)
-    return AttentionWeights(embed, layers, final, pad_pitch(embed))
+    final = (_plain_norm if cfg.input_norm else _centred_norm if cfg.output_norm else _norm)(get, "final.norm", cfg)
+    w = AttentionWeights(embed, layers, final, pad_pitch(embed))
+    if cfg.token_side:
+        w.extra["side_embed"] = get("side.embed", (cfg.vocab_size, cfg.num_layers * cfg.token_side)).contiguous()
+    return w
 
 
 # stored around zero: norms behind sublayers; biases and decays of random models are zero too

@@ -17,7 +17,7 @@ from pathlib import Path
 
 import torch
 
-from .config import GLU_ALPHA, ModelConfig
+from .config import GELU_ALPHA, GELU_CUBIC, GLU_ALPHA, ModelConfig
 from ..utils.dtype import decode_dtype
 
 FFN_KEY = re.compile(r"^model\.layers\.(\d+)\.mlp\.")
@@ -100,7 +100,7 @@ def random_attention_weights(cfg: ModelConfig, seed: int = 0, device="cpu", dtyp
     if cfg.layered:
         from .layered import layered_attention_weights, random_getter
 
-        return layered_attention_weights(cfg, random_getter(gen, dt, device, cfg.output_norm), device, dt)
+        return layered_attention_weights(cfg, random_getter(gen, dt, device, cfg.output_norm and not cfg.input_norm), device, dt)
     embed = _randn(gen, (cfg.vocab_size, cfg.hidden_size), dt, device)
     layers = []
     if not cfg.gpu_attention_supported:
@@ -225,9 +225,24 @@ def random_ffn_layer(cfg: ModelConfig, layer: int, seed: int = 0, device="cpu", 
                 w.router = w.extra["router_fp32"].to(dt)
         return w
     if cfg.layered:
-        inter, limit = cfg.layer_specs[layer].ff, cfg.layer_specs[layer].gate_limit
+        spec = cfg.layer_specs[layer]
+        inter, limit = spec.ff, spec.gate_limit
         if tp_size > 1:
             raise NotImplementedError("the FFNs of layered decoders run whole on one GPU (FFN TP 1)")
+        if spec.moe is not None:
+            m = spec.moe
+            w = FfnLayerWeights(_randn(gen, (m.experts, 2 * m.ff, h), dt, device), _randn(gen, (m.experts, h, m.ff), dt, device),
+                                router=_randn(gen, (m.routed, h), dt, device))
+            if m.shared_ff:
+                w.shared_gate_up, w.shared_down = _randn(gen, (2 * m.shared_ff, h), dt, device), _randn(gen, (h, m.shared_ff), dt, device)
+                w.extra["shared_scale"] = _randn(gen, (1, h), dt, device)
+            w.extra.update(correction_bias=torch.zeros(m.routed, dtype=torch.float32, device=device), experts=(0, m.experts),
+                           router_precision="fp32_logits")
+            return w
+        if spec.gelu:
+            w = FfnLayerWeights(_randn(gen, (2 * inter, h), dt, device), _randn(gen, (h, inter), dt, device))
+            w.extra.update(gated=True, gate_transform=(0.0, 0.0, GELU_ALPHA, GELU_CUBIC))
+            return w
         if limit > 0:
             w = FfnLayerWeights(_randn(gen, (2 * inter, h), dt, device), _randn(gen, (h, inter), dt, device))
             w.extra.update(gated=True, gate_transform=(limit, 1.0, GLU_ALPHA))
@@ -260,7 +275,7 @@ def quantize_ffn_layer_fp8(w: FfnLayerWeights) -> FfnLayerWeights:
 def random_ffn_weights(cfg: ModelConfig, seed: int = 0, device="cpu", dtype: torch.dtype | None = None,
                        tp_rank: int = 0, tp_size: int = 1) -> list[FfnLayerWeights | None]:
     """One entry per layer; None for the layers of a layered decoder that have no FFN."""
-    return [None if cfg.layered and not cfg.layer_specs[l].ff else random_ffn_layer(cfg, l, seed, device, dtype, tp_rank, tp_size)
+    return [None if cfg.layered and not cfg.layer_specs[l].has_ffn else random_ffn_layer(cfg, l, seed, device, dtype, tp_rank, tp_size)
             for l in range(cfg.num_layers)]
 
 

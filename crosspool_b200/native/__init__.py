@@ -15,7 +15,7 @@ import ctypes as C
 import functools
 from pathlib import Path
 
-EXPECTED_ABI = 23
+EXPECTED_ABI = 24
 HERE = Path(__file__).resolve().parent
 
 
@@ -68,6 +68,12 @@ class GemmArgs(C.Structure):
         ("out_group_stride", C.c_int),
         ("out_scale", C.c_float),
         ("silu_cols", C.c_int),
+        ("act_cubic", C.c_float),
+        ("ids_limit", C.c_int),
+        ("ids", C.c_void_p),
+        ("tail", C.c_void_p),
+        ("tail_from", C.c_int),
+        ("ld_tail", C.c_int),
     ]
 
 
@@ -234,6 +240,9 @@ class DecodeRowsArgs(C.Structure):
         ("ld_out", C.c_int),
         ("ld_gate", C.c_int),
         ("softcap", C.c_float),
+        ("window", C.c_int),
+        ("keep_first", C.c_int),
+        ("gate_elems", C.c_int),
     ]
 
 
@@ -268,6 +277,9 @@ class PrefillAttnArgs(C.Structure):
         ("p_pair", C.c_int),
         ("group_valid", C.c_int),
         ("softcap", C.c_float),
+        ("window", C.c_int),
+        ("keep_first", C.c_int),
+        ("gate_elems", C.c_int),
     ]
 
 
@@ -287,15 +299,20 @@ PolyNormArgs = _struct("PolyNormArgs", "XpPolyNormArgs", a_ptr="z coef out", b_i
 GatedRmsArgs = _struct("GatedRmsArgs", "XpGatedRmsArgs", a_ptr="o weight gate out", b_int="rows cols ld_o ld_gate ld_out", c_float="eps",
                        d_int="f32")
 PostNormArgs = _struct("PostNormArgs", "XpPostNormArgs", a_ptr="resid", b_ptr2="branches branch_w", c_ptr="ids table sel weight out_weight out",
-                       d_int="rows hidden nbranches", e_int2="ld_branch", f_int="ld_out vocab", g_float="eps", h_int="f32")
+                       d_int="rows hidden nbranches", e_int2="ld_branch", f_int="ld_out vocab", g_float="eps embed_scale", h_int="f32")
 HeadGateArgs = _struct("HeadGateArgs", "XpHeadGateArgs", a_ptr="o weight gate out", b_int="rows heads dim ld_o ld_gate ld_out", c_float="eps",
-                       d_int="f32")
-GluArgs = _struct("GluArgs", "XpGluArgs", a_ptr="z out", b_int="rows cols ld_z ld_out", c_float="limit up_add alpha")
+                       d_int="f32 per_head_weight sigmoid_gate")
+GluArgs = _struct("GluArgs", "XpGluArgs", a_ptr="z out", b_int="rows cols ld_z ld_out", c_float="limit up_add alpha cubic")
+TokenGateArgs = _struct("TokenGateArgs", "XpTokenGateArgs", a_ptr="z table ids out", b_int="rows cols ld_z ld_table ld_out vocab", c_float="alpha cubic")
 GroupedPrepArgs = _struct("GroupedPrepArgs", "XpGroupedPrepArgs", a_ptr="proj q_norm k_norm slots k_cache v_cache q_out",
                           b_int="rows heads kv_heads group_pad dim vdim dq dv ld_proj q_off k_off v_off", c_float="eps", d_int="f32")
 GroupedAttnArgs = _struct("GroupedAttnArgs", "XpGroupedAttnArgs", a_ptr="q k_cache v_cache out gate row_seq positions slots block_table",
                           b_int="rows heads kv_heads group_pad dim vdim dq dv ld_gate ld_out page_size max_blocks", c_float="scale softcap",
-                          d_int="f32")
+                          d_int="f32 window keep_first gate_elems")
+ConvRopeArgs = _struct("ConvRopeArgs", "XpConvRopeArgs",
+                       a_ptr="proj conv_w ring rot positions slots state_slots q_starts q_lens k_cache v_cache q_out",
+                       b_int="rows seqs max_q heads kv_heads group_pad dim vdim dq dv own_kv ld_proj q_off k_off v_off taps rot_pairs rot_positions "
+                             "row_floats f32")
 GatedLinearArgs = _struct("GatedLinearArgs", "XpGatedLinearArgs",
                           a_ptr="proj z a2 a2_bias norm state out positions slots state_slots q_starts q_lens ws records",
                           b_int="rows seqs max_q heads dim vdim ld_proj ld_out q_off k_off v_off g_off a_off rank ld_a2 segs seg_tokens force_sequential",
@@ -304,6 +321,10 @@ DeltaArgs = _struct("DeltaArgs", "XpDeltaArgs",
                     a_ptr="proj conv_w conv_state neg_a dt_bias norm state out qkv qk_scale beta_g ws positions slots state_slots q_starts q_lens",
                     b_int="rows seqs max_q heads kv_heads dim vdim taps ld_proj ld_out q_off k_off v_off g_off b_off a_off force_sequential",
                     c_float="qscale eps", d_int="f32")
+MemoryArgs = _struct("MemoryArgs", "XpMemoryArgs", a_ptr="proj gates norm state out planes before ws positions slots state_slots q_starts q_lens",
+                     b_int="rows seqs max_q heads dim vdim head_state ld_proj ld_gates ld_out q_off k_off v_off g_off i_off f_off segs seg_tokens "
+                           "force_sequential",
+                     c_float="qscale cap eps", d_int="f32")
 LatentPrepArgs = _struct("LatentPrepArgs", "XpLatentPrepArgs", a_ptr="proj norm_w freq positions slots cache q_plain q_abs q_exp",
                          b_int="rows heads dim rot rot_dims kv_rank ld_proj q_off kv_off ld_cache qp_rows dim_p ld_abs dq_pad abs_rows",
                          c_float="eps", d_int="f32")
@@ -321,15 +342,17 @@ def _declare_mixers(lib: C.CDLL) -> None:
     for fn, args in (("xp_resid_norm", ResidNormArgs), ("xp_polynorm", PolyNormArgs), ("xp_gated_rms", GatedRmsArgs),
                      ("xp_latent_prep", LatentPrepArgs), ("xp_latent_attn", LatentAttnArgs), ("xp_latent_gather", LatentGatherArgs),
                      ("xp_linear_attn_decode", LinearAttnArgs), ("xp_linear_attn_prefill", LinearAttnArgs),
-                     ("xp_post_norm", PostNormArgs), ("xp_head_gate", HeadGateArgs), ("xp_glu_f32", GluArgs),
-                     ("xp_grouped_prep", GroupedPrepArgs), ("xp_grouped_attn", GroupedAttnArgs),
+                     ("xp_post_norm", PostNormArgs), ("xp_head_gate", HeadGateArgs), ("xp_glu_f32", GluArgs), ("xp_token_gate_f32", TokenGateArgs),
+                     ("xp_grouped_prep", GroupedPrepArgs), ("xp_conv_rope_decode", ConvRopeArgs), ("xp_conv_rope_prefill", ConvRopeArgs), ("xp_grouped_attn", GroupedAttnArgs),
                      ("xp_gated_linear_decode", GatedLinearArgs), ("xp_gated_linear_prefill", GatedLinearArgs),
-                     ("xp_delta_decode", DeltaArgs), ("xp_delta_prep", DeltaArgs), ("xp_delta_prefill", DeltaArgs)):
+                     ("xp_memory_decode", MemoryArgs), ("xp_memory_prefill", MemoryArgs), ("xp_delta_decode", DeltaArgs), ("xp_delta_prep", DeltaArgs), ("xp_delta_prefill", DeltaArgs)):
         getattr(lib, fn).restype = C.c_int
         getattr(lib, fn).argtypes = [C.POINTER(args), C.c_void_p]
     for fn in ("xp_delta_ws_bytes", "xp_gated_linear_record_bytes"):
         getattr(lib, fn).restype = C.c_size_t
         getattr(lib, fn).argtypes = [C.c_int] * 3
+    lib.xp_gemm_f32_grouped.restype = C.c_int
+    lib.xp_gemm_f32_grouped.argtypes = [C.c_void_p] * 5 + [C.c_int] * 7 + [C.c_void_p]
     lib.xp_gemm_f32.restype = C.c_int
     lib.xp_gemm_f32.argtypes = [C.c_void_p] * 4 + [C.c_int] * 7 + [C.c_int64] * 3 + [C.c_float, C.c_int, C.c_void_p]
 
@@ -485,8 +508,14 @@ class RouteArgs(C.Structure):
     ]
 
 
+MoeMixArgs = _struct("MoeMixArgs", "XpMoeMixArgs", a_ptr="y x shared shared_gate topk_ids route_pos weights out",
+                     b_int="rows top_k hidden experts ld_y ld_x ld_shared ld_gate ld_out f32")
+
+
 def _declare_moe(lib: C.CDLL) -> None:
     sig = {
+        "xp_moe_mix": [C.POINTER(MoeMixArgs), C.c_void_p],
+        "xp_moe_topk_route": [C.POINTER(RouterArgs), C.POINTER(RouteArgs), C.c_void_p],
         "xp_debug_options_set": [C.POINTER(C.c_uint32)],
         "xp_debug_options_get": [C.POINTER(C.c_uint32)],
         "xp_router_topk": [C.POINTER(RouterArgs), C.c_void_p],

@@ -29,6 +29,7 @@ EPI_STORE = 0
 EPI_SWIGLU = 1
 EPI_RESIDUAL = 2
 EPI_STORE_F32 = 3
+EPI_TOKEN_GATE = 4
 
 _WS_BYTES = 96 << 20
 _COUNTER_WORDS = 1 << 16
@@ -120,7 +121,7 @@ def tile_weight(w: torch.Tensor) -> TiledWeight:
 
 
 def _args(x, w, out, *, n_out, rows, epilogue, dual=0, up_offset=0, bias=None, resid=None, splits=0, bn=0,
-          num_sms=0, evict_first=None, gate_limit=0.0, up_add=0.0, act_alpha=0.0, out_scale=0.0, silu_cols=0) -> native.GemmArgs:
+          num_sms=0, evict_first=None, gate_limit=0.0, up_add=0.0, act_alpha=0.0, out_scale=0.0, silu_cols=0, act_cubic=0.0) -> native.GemmArgs:
     tiled = isinstance(w, TiledWeight)
     assert x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16
     assert x.stride(-1) == 1 and out.stride(-1) == 1 and (tiled or w.stride(-1) == 1)
@@ -159,6 +160,7 @@ def _args(x, w, out, *, n_out, rows, epilogue, dual=0, up_offset=0, bias=None, r
     a.gate_limit = gate_limit
     a.up_add = up_add
     a.act_alpha = act_alpha
+    a.act_cubic = act_cubic
     a.out_scale = out_scale
     a.silu_cols = silu_cols
     # decode-size calls leave room for a second kernel on the SM (the co-located Instance's attention)
@@ -184,9 +186,11 @@ def plan_shape(n_out: int, k: int, rows: int, dual: int = 0, num_sms: int = 148,
 
 def linear(x: torch.Tensor, w: torch.Tensor, *, out: torch.Tensor | None = None, bias: torch.Tensor | None = None,
            resid: torch.Tensor | None = None, out_fp32: bool = False, splits: int = 0, bn: int = 0,
-           num_sms: int = 0, evict_first: bool | None = None, out_scale: float = 0.0, silu_cols: int = 0) -> torch.Tensor:
+           num_sms: int = 0, evict_first: bool | None = None, out_scale: float = 0.0, silu_cols: int = 0,
+           tail: torch.Tensor | None = None) -> torch.Tensor:
     """``x[rows, k] @ w[n, k].T`` (* ``out_scale`` unless 0) (+ fp32 ``bias``) (+ ``resid``) on the tcgen05 kernel; fp32
-    operands run the plain fp32 kernel. The first ``silu_cols`` features are stored as ``silu(value)``. Any ``n`` and ``k``; bf16 row pitches must be multiples of 16 bytes."""
+    operands run the plain fp32 kernel. The first ``silu_cols`` features are stored as ``silu(value)``. Any ``n`` and ``k``; bf16 row pitches must be multiples of 16 bytes.
+    ``tail``: the last ``tail.shape[1]`` features go to this fp32 tensor instead (bf16 products)."""
     x2 = x if x.dim() == 2 else x.reshape(-1, x.shape[-1])   # reshape would forget the row pitch of a single row
     rows, n = x2.shape[0], w.shape[0]
     if x.dtype == torch.float32:
@@ -201,6 +205,9 @@ def linear(x: torch.Tensor, w: torch.Tensor, *, out: torch.Tensor | None = None,
     epi = EPI_STORE_F32 if out.dtype == torch.float32 else (EPI_RESIDUAL if resid is not None else EPI_STORE)
     a = _args(x2, w, out, n_out=n, rows=rows, epilogue=epi, bias=bias, resid=resid, splits=splits, bn=bn,
               num_sms=num_sms, evict_first=evict_first, out_scale=out_scale, silu_cols=silu_cols)
+    if tail is not None:
+        assert tail.dtype == torch.float32 and tail.shape[0] == rows and tail.stride(1) == 1
+        a.tail, a.tail_from, a.ld_tail = tail.data_ptr(), n - tail.shape[1], tail.stride(0)
     native.check(native.kernels().xp_gemm(C.byref(a)), "xp_gemm")
     return out.reshape(*x.shape[:-1], n) if x.dim() != 2 else out
 
@@ -230,17 +237,28 @@ def linear_batched(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, out_grou
     return out
 
 
+def linear_token_gate(x: torch.Tensor, w: torch.Tensor, table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor, alpha: float,
+                      cubic: float) -> torch.Tensor:
+    """``act(x @ w.T) * table[ids]`` in bf16, ``act(g) = g sigmoid(alpha g (1 + cubic g^2))``; ``ids`` int32, one per row."""
+    assert table.dtype == torch.bfloat16 and table.stride(1) == 1 and ids.dtype == torch.int32 and table.shape[1] == w.shape[0]
+    a = _args(x, w, out, n_out=w.shape[0], rows=x.shape[0], epilogue=EPI_TOKEN_GATE, resid=table, act_alpha=alpha, act_cubic=cubic)
+    a.ids, a.ids_limit = ids.data_ptr(), table.shape[0]
+    native.check(native.kernels().xp_gemm(C.byref(a)), "xp_gemm(token gate)")
+    return out
+
+
 def gateup_swiglu(x: torch.Tensor, w_gate_up: torch.Tensor, *, out: torch.Tensor | None = None,
                   bias: torch.Tensor | None = None, gate_limit: float = 0.0, up_add: float = 0.0,
-                  act_alpha: float = 0.0, splits: int = 0, bn: int = 0, num_sms: int = 0) -> torch.Tensor:
-    """``silu(x @ Wg.T) * (x @ Wu.T)`` with ``w_gate_up = cat([Wg, Wu])`` of shape ``[2*I, k]``."""
+                  act_alpha: float = 0.0, act_cubic: float = 0.0, splits: int = 0, bn: int = 0, num_sms: int = 0) -> torch.Tensor:
+    """``silu(x @ Wg.T) * (x @ Wu.T)`` with ``w_gate_up = cat([Wg, Wu])`` of shape ``[2*I, k]`` (another activation
+    ``g sigmoid(act_alpha g (1 + act_cubic g^2))`` where those are given)."""
     x2 = x if x.dim() == 2 else x.reshape(-1, x.shape[-1])
     rows = x2.shape[0]
     inter = w_gate_up.shape[0] // 2
     if out is None:
         out = torch.empty(rows, inter, dtype=torch.bfloat16, device=x.device)
     a = _args(x2, w_gate_up, out, n_out=inter, rows=rows, epilogue=EPI_SWIGLU, dual=1, up_offset=inter, bias=bias,
-              splits=splits, bn=bn, num_sms=num_sms, gate_limit=gate_limit, up_add=up_add, act_alpha=act_alpha)
+              splits=splits, bn=bn, num_sms=num_sms, gate_limit=gate_limit, up_add=up_add, act_alpha=act_alpha, act_cubic=act_cubic)
     native.check(native.kernels().xp_gemm(C.byref(a)), "xp_gemm(swiglu)")
     return out
 

@@ -14,7 +14,8 @@ from typing import Sequence
 import torch
 
 from .. import native
-from ..models.config import attention_shape
+from ..models.config import GELU_ALPHA, GELU_CUBIC, attention_shape
+from . import gemm
 
 NORM_KINDS = {"rmsnorm": 0, "layernorm": 1, "dyt": 2}
 # Rows of a recurrence computed with one set of matrix products (decay powers are tabulated up to this).
@@ -75,9 +76,10 @@ def resid_norm(resid: torch.Tensor, norm: NormParams | None, out: torch.Tensor |
 
 def post_norm(resid: torch.Tensor, out: torch.Tensor | None, *, norm: NormParams | None = None, branches: Sequence[torch.Tensor] = (),
               branch_norms: Sequence[NormParams] = (), ids: torch.Tensor | None = None, table: torch.Tensor | None = None,
-              out_norm: NormParams | None = None, sel: torch.Tensor | None = None, rows: int | None = None, eps: float = 1e-6) -> None:
-    """``resid += norm(branch)`` (``branch_norms``: of the mean of the normed branches; ``ids``: ``resid = table[ids]``) in
-    fp32, then ``out = resid``, or ``out_norm(resid)``. All norms are RMS norms with ``eps``. With ``sel`` (int32) only the
+              out_norm: NormParams | None = None, sel: torch.Tensor | None = None, rows: int | None = None, eps: float = 1e-6,
+              embed_scale: float = 1.0) -> None:
+    """``resid += norm(branch)`` (``branch_norms``: of the mean of the normed branches; ``ids``: ``resid = table[ids] *
+    embed_scale``) in fp32, then ``out = resid``, or ``out_norm(resid)``. All norms are RMS norms with ``eps``. With ``sel`` (int32) only the
     selected rows are computed and the residual is left alone."""
     a = native.PostNormArgs()
     act = branches[0] if branches else table
@@ -95,28 +97,44 @@ def post_norm(resid: torch.Tensor, out: torch.Tensor | None, *, norm: NormParams
     a.hidden, a.nbranches = resid.shape[1], len(branches)
     a.ld_out = out.stride(0) if out is not None else 0
     a.vocab = table.shape[0] if table is not None else 0
-    a.eps, a.f32 = norm.eps if norm is not None else eps, _f32(act)
+    a.eps, a.f32, a.embed_scale = norm.eps if norm is not None else out_norm.eps if out_norm is not None else eps, _f32(act), embed_scale
     native.check(native.kernels().xp_post_norm(C.byref(a), _stream(resid)), "xp_post_norm")
 
 
-def head_gate(o: torch.Tensor, weight: torch.Tensor, gate: torch.Tensor, eps: float, out: torch.Tensor) -> torch.Tensor:
-    """``rmsnorm(o) * weight * silu(gate)`` with the norm over every head of ``len(weight)`` columns; ``o`` fp32."""
+def head_gate(o: torch.Tensor, weight: torch.Tensor, gate: torch.Tensor, eps: float, out: torch.Tensor, heads: int = 0) -> torch.Tensor:
+    """``rmsnorm(o) * weight * silu(gate)`` with the norm over every head of ``len(weight)`` columns; ``o`` fp32. With
+    ``heads`` the weight covers all heads and the gate is a sigmoid."""
     assert o.dtype == torch.float32 and weight.dtype == torch.float32 and gate.dtype == out.dtype
     a = native.HeadGateArgs()
     a.o, a.weight, a.gate, a.out = o.data_ptr(), weight.data_ptr(), gate.data_ptr(), out.data_ptr()
-    a.rows, a.heads, a.dim = o.shape[0], o.shape[1] // weight.numel(), weight.numel()
+    dim = weight.numel() // heads if heads else weight.numel()
+    a.rows, a.heads, a.dim, a.per_head_weight, a.sigmoid_gate = o.shape[0], o.shape[1] // dim, dim, int(heads > 0), int(heads > 0)
     a.ld_o, a.ld_gate, a.ld_out, a.eps, a.f32 = o.stride(0), gate.stride(0), out.stride(0), eps, _f32(out)
     native.check(native.kernels().xp_head_gate(C.byref(a), _stream(o)), "xp_head_gate")
     return out
 
 
-def glu_f32(z: torch.Tensor, limit: float, up_add: float, alpha: float, out: torch.Tensor) -> torch.Tensor:
-    """Clamped gated activation of fp32 rows ``[g, u]`` (the bf16 product applies it in its epilogue)."""
+def glu_f32(z: torch.Tensor, limit: float, up_add: float, alpha: float, out: torch.Tensor, cubic: float = 0.0) -> torch.Tensor:
+    """Gated activation of fp32 rows ``[g, u]`` (the bf16 product applies it in its epilogue)."""
     assert z.dtype == out.dtype == torch.float32
     a = native.GluArgs()
     a.z, a.out, a.rows, a.cols, a.ld_z, a.ld_out = z.data_ptr(), out.data_ptr(), z.shape[0], z.shape[1] // 2, z.stride(0), out.stride(0)
-    a.limit, a.up_add, a.alpha = limit, up_add, alpha
+    a.limit, a.up_add, a.alpha, a.cubic = limit, up_add, alpha, cubic
     native.check(native.kernels().xp_glu_f32(C.byref(a), _stream(z)), "xp_glu_f32")
+    return out
+
+
+def token_gate(x: torch.Tensor, w: torch.Tensor, table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor, z: torch.Tensor) -> torch.Tensor:
+    """``gelu_tanh(x @ w.T) * table[ids]``; ``table`` ``[vocab, n]`` may be a column range of a wider one. bf16: one product
+    with the gate in its epilogue; fp32: product into ``z``, then a row kernel."""
+    if x.dtype == torch.bfloat16:
+        return gemm.linear_token_gate(x, w, table, ids, out, GELU_ALPHA, GELU_CUBIC)
+    gemm.linear(x, w, out=z)
+    a = native.TokenGateArgs()
+    a.z, a.table, a.ids, a.out = z.data_ptr(), table.data_ptr(), ids.data_ptr(), out.data_ptr()
+    a.rows, a.cols, a.ld_z, a.ld_table, a.ld_out, a.vocab = x.shape[0], w.shape[0], z.stride(0), table.stride(0), out.stride(0), table.shape[0]
+    a.alpha, a.cubic = GELU_ALPHA, GELU_CUBIC
+    native.check(native.kernels().xp_token_gate_f32(C.byref(a), _stream(x)), "xp_token_gate_f32")
     return out
 
 
@@ -195,9 +213,7 @@ def latent_attn(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, block_t
     a.page_size, a.max_blocks, a.num_splits, a.chunk_tokens = cache.shape[1], block_table.stride(0), num_splits, chunk_tokens
     assert num_splits == 1 or ws.numel() >= rows * heads * num_splits * (kv_rank + 2)
     a.scale, a.f32, a.force_simt = scale, _f32(q), int(force_simt)
-    from .gemm import status_words
-
-    a.status = status_words(q.device).data_ptr()
+    a.status = gemm.status_words(q.device).data_ptr()
     native.check(native.kernels().xp_latent_attn(C.byref(a), _stream(q)), "xp_latent_attn", 2 if num_splits > 1 else 1)
     return out
 
@@ -224,8 +240,6 @@ def expanded_prefill(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, out: tor
     """Causal attention of chunk queries ``q`` ``[rows, heads, dq]`` over dense per-head keys ``k`` ``[tokens, heads, dq]``
     and values ``v`` ``[tokens, heads, dv]`` (sequence i's tokens start at row ``starts[i]``, a multiple of 64); ``out``
     ``[rows, heads * vdim]``, head h multiplied by ``sigmoid(gate[:, h])``."""
-    from .gemm import status_words
-
     a = native.PrefillAttnArgs()
     a.q, a.k_cache, a.v_cache, a.out = q.data_ptr(), k.data_ptr(), v.data_ptr(), out.data_ptr()
     a.q_starts, a.q_lens, a.ctx_lens, a.seq_starts = q_starts.data_ptr(), q_lens.data_ptr(), ctx_lens.data_ptr(), starts.data_ptr()
@@ -235,7 +249,7 @@ def expanded_prefill(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, out: tor
     a.scale, a.total_q, a.p_pair = scale, q.shape[0], 1
     a.gate = _ptr(gate)
     a.ld_gate = gate.stride(0) if gate is not None else 0
-    a.status = status_words(q.device).data_ptr()
+    a.status = gemm.status_words(q.device).data_ptr()
     lib = native.kernels()
     native.check(lib.xp_prefill_attn_umma(C.byref(a), _stream(q)), "xp_prefill_attn_umma")
 
@@ -328,11 +342,50 @@ def grouped_prep(proj: torch.Tensor, q_norm: torch.Tensor | None, k_norm: torch.
     native.check(native.kernels().xp_grouped_prep(C.byref(a), _stream(proj)), "xp_grouped_prep")
 
 
+def _gate_elems(gate: torch.Tensor | None, heads: int, vdim: int) -> int:
+    """Whether a gate has one logit per output element (of a single-column head either reading is the same)."""
+    if gate is None or gate.shape[1] == heads:
+        return 0
+    assert gate.shape[1] == heads * vdim
+    return 1
+
+
+def conv_rope(proj: torch.Tensor, conv_w: torch.Tensor | None, ring: torch.Tensor | None, rot: torch.Tensor | None, positions: torch.Tensor,
+              slots: torch.Tensor, state_slots: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, q_out: torch.Tensor, *, heads: int,
+              dim: int, vdim: int, offs: tuple[int, ...], q_starts: torch.Tensor | None = None, q_lens: torch.Tensor | None = None,
+              max_q: int = 0) -> None:
+    """Convolution over time (``conv_w`` fp32 ``[taps, channels]``, inputs behind every sequence in ``ring`` ``[slots, taps,
+    channels]``), rotation (``rot`` fp32 ``[positions, pairs, 2]``), cache write and the padded query layout ``q_out`` ``[rows,
+    kv_heads, group_pad, dq]``. ``offs``: columns of q, k, v in ``proj``, or of q alone (nothing is cached). One token per row,
+    or with ``q_lens`` the portions that start at rows ``q_starts``."""
+    a = native.ConvRopeArgs()
+    assert k_cache.dtype == proj.dtype == q_out.dtype and (rot is None or rot.dtype == torch.float32)
+    a.proj, a.conv_w, a.ring, a.rot = proj.data_ptr(), _ptr(conv_w), _ptr(ring), _ptr(rot)
+    a.positions, a.slots, a.state_slots = positions.data_ptr(), slots.data_ptr(), state_slots.data_ptr()
+    a.k_cache, a.v_cache, a.q_out = k_cache.data_ptr(), v_cache.data_ptr(), q_out.data_ptr()
+    a.rows, a.heads, a.kv_heads, a.group_pad = proj.shape[0], heads, k_cache.shape[2], q_out.shape[2]
+    a.dim, a.vdim, a.dq, a.dv, a.ld_proj, a.own_kv = dim, vdim, k_cache.shape[3], v_cache.shape[3], proj.stride(0), int(len(offs) == 3)
+    a.q_off, a.k_off, a.v_off = offs if len(offs) == 3 else (offs[0], 0, 0)
+    if conv_w is not None:
+        assert conv_w.dtype == torch.float32 and conv_w.is_contiguous() and ring.dtype == proj.dtype and tuple(conv_w.shape) == tuple(ring.shape[1:])
+        a.taps = conv_w.shape[0]
+    if rot is not None:
+        a.rot_positions, a.rot_pairs = rot.shape[0], rot.shape[1]
+    a.f32 = _f32(proj)
+    lib = native.kernels()
+    if q_lens is None:
+        native.check(lib.xp_conv_rope_decode(C.byref(a), _stream(proj)), "xp_conv_rope_decode")
+        return
+    a.q_starts, a.q_lens, a.seqs, a.max_q = q_starts.data_ptr(), q_lens.data_ptr(), q_lens.shape[0], max_q
+    native.check(lib.xp_conv_rope_prefill(C.byref(a), _stream(proj)), "xp_conv_rope_prefill")
+
+
 def grouped_attn(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, out: torch.Tensor, block_table: torch.Tensor,
                  positions: torch.Tensor, slots: torch.Tensor, *, heads: int, dim: int, vdim: int, scale: float, softcap: float = 0.0,
-                 gate: torch.Tensor | None = None, row_seq: torch.Tensor | None = None) -> torch.Tensor:
+                 gate: torch.Tensor | None = None, row_seq: torch.Tensor | None = None, window: int = 0, keep_first: int = 0) -> torch.Tensor:
     """Rows of queries ``[rows, kv_heads, group_pad, dq]`` against the first ``positions[r] + 1`` cached tokens of their
-    sequences, any sizes and types; ``out`` ``[rows, heads * vdim]``, head h multiplied by ``sigmoid(gate[:, h])``."""
+    sequences (``window`` > 0: the last ``window`` of those and the first ``keep_first``), any sizes and types; ``out`` ``[rows,
+    heads * vdim]``, multiplied by the sigmoid of ``gate``, which has one column per head or one per output."""
     step = 32768
     for lo in range(0, q.shape[0], step):
         n = min(step, q.shape[0] - lo)
@@ -345,6 +398,7 @@ def grouped_attn(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, 
         a.rows, a.heads, a.kv_heads, a.group_pad, a.dim, a.vdim = n, heads, q.shape[1], q.shape[2], dim, vdim
         a.dq, a.dv, a.ld_gate, a.ld_out = q.shape[3], v_cache.shape[3], gate.stride(0) if gate is not None else 0, out.stride(0)
         a.page_size, a.max_blocks, a.scale, a.softcap, a.f32 = k_cache.shape[1], block_table.stride(0), scale, softcap, _f32(q)
+        a.window, a.keep_first, a.gate_elems = window, keep_first, _gate_elems(gate, heads, vdim)
         native.check(native.kernels().xp_grouped_attn(C.byref(a), _stream(q)), "xp_grouped_attn")
     return out
 
@@ -352,32 +406,29 @@ def grouped_attn(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, 
 def grouped_decode(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, out: torch.Tensor, block_table: torch.Tensor,
                    positions: torch.Tensor, slots: torch.Tensor, *, heads: int, dim: int, vdim: int, scale: float, softcap: float = 0.0,
                    gate: torch.Tensor | None = None, row_seq: torch.Tensor | None = None, num_splits: int = 1, chunk_tokens: int = 0,
-                   ws: torch.Tensor | None = None) -> torch.Tensor:
+                   ws: torch.Tensor | None = None, window: int = 0, keep_first: int = 0) -> torch.Tensor:
     """:func:`grouped_attn` on the tensor cores (bf16, widths of ``ATTENTION_SHAPES``, at most 16 query heads per key head).
     ``ws``: fp32, ``rows * heads * num_splits * (dv + 2)`` elements when ``num_splits`` > 1."""
-    from .gemm import status_words
-
     r = native.DecodeRowsArgs()
     a = r.a
     a.q, a.k_cache, a.v_cache, a.out, a.ws = q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), out.data_ptr(), _ptr(ws)
     assert q.dtype == out.dtype == torch.bfloat16 and (num_splits == 1 or ws.numel() >= q.shape[0] * heads * num_splits * (v_cache.shape[3] + 2))
     a.block_table, a.batch, a.q_heads, a.kv_heads, a.head_dim = block_table.data_ptr(), q.shape[0], heads, q.shape[1], q.shape[3]
     a.page_size, a.max_blocks, a.num_splits, a.chunk_tokens, a.num_pages = k_cache.shape[1], block_table.stride(0), num_splits, chunk_tokens, k_cache.shape[0]
-    a.scale, a.status = scale, status_words(q.device).data_ptr()
+    a.scale, a.status = scale, gemm.status_words(q.device).data_ptr()
     r.row_seq, r.positions, r.slots, r.gate = _ptr(row_seq), positions.data_ptr(), slots.data_ptr(), _ptr(gate)
     r.group_pad, r.v_dim, r.v_valid, r.ld_out, r.softcap = q.shape[2], v_cache.shape[3], vdim, out.stride(0), softcap
     r.ld_gate = gate.stride(0) if gate is not None else 0
+    r.window, r.keep_first, r.gate_elems = window, keep_first, _gate_elems(gate, heads, vdim)
     native.check(native.kernels().xp_decode_rows(C.byref(r), _stream(q)), "xp_decode_rows", 2 if num_splits > 1 else 1)
     return out
 
 
 def grouped_prefill(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, out: torch.Tensor, block_table: torch.Tensor,
                     q_starts: torch.Tensor, q_lens: torch.Tensor, ctx_lens: torch.Tensor, max_q: int, *, heads: int, vdim: int, scale: float,
-                    softcap: float = 0.0, gate: torch.Tensor | None = None) -> torch.Tensor:
+                    softcap: float = 0.0, gate: torch.Tensor | None = None, window: int = 0, keep_first: int = 0) -> torch.Tensor:
     """Causal attention of portions (rows of ``q`` ``[rows, kv_heads, group_pad, dq]``) over the paged cache, which holds the
     portions' own tokens already, on tcgen05; ``out`` ``[rows, heads * vdim]``."""
-    from .gemm import status_words
-
     a = native.PrefillAttnArgs()
     a.q, a.k_cache, a.v_cache, a.out, a.block_table = (t.data_ptr() for t in (q, k_cache, v_cache, out, block_table))
     a.q_starts, a.q_lens, a.ctx_lens = q_starts.data_ptr(), q_lens.data_ptr(), ctx_lens.data_ptr()
@@ -386,7 +437,8 @@ def grouped_prefill(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
     a.page_size, a.max_blocks, a.num_pages = k_cache.shape[1], block_table.stride(0), k_cache.shape[0]
     a.scale, a.total_q, a.p_pair, a.group_valid, a.softcap = scale, q.shape[0], 1, heads // q.shape[1], softcap
     a.gate, a.ld_gate = _ptr(gate), gate.stride(0) if gate is not None else 0
-    a.status = status_words(q.device).data_ptr()
+    a.window, a.keep_first, a.gate_elems = window, keep_first, _gate_elems(gate, heads, vdim)
+    a.status = gemm.status_words(q.device).data_ptr()
     native.check(native.kernels().xp_prefill_attn_umma(C.byref(a), _stream(q)), "xp_prefill_attn_umma")
     return out
 
@@ -460,6 +512,57 @@ def gated_linear_prefill(proj, z, state, out, positions, slots, state_slots, q_s
         assert segs <= 1 or scratch.ws.numel() >= q_lens.shape[0] * heads * segs * dim * (vdim + 1)
         n = 4 if segs > 1 else 2
     native.check(native.kernels().xp_gated_linear_prefill(C.byref(a), _stream(proj)), "xp_gated_linear_prefill", n)
+
+
+@dataclass
+class MemoryScratch:
+    """What the prefill kernels hand on: the gates of every (token, head), key sums and maxima before every portion, states
+    between segments."""
+
+    planes: torch.Tensor
+    before: torch.Tensor
+    ws: torch.Tensor
+
+    @classmethod
+    def for_rows(cls, rows: int, seqs: int, heads: int, dim: int, vdim: int, device) -> "MemoryScratch":
+        """For batches of at most ``rows`` rows in ``seqs`` portions; any plan of :func:`linear_attn_plan` fits."""
+        return cls(*(torch.zeros(n, dtype=torch.float32, device=device)
+                     for n in (3 * heads * rows, seqs * heads * (dim + 1), 2 * 148 * (dim * (vdim + 1) + 4))))
+
+
+def _memory(proj, gates, state, out, positions, slots, state_slots, heads, dim, vdim, offs, cap) -> "native.MemoryArgs":
+    assert gates.dtype == torch.float32 and state.shape[1] == heads and state.is_contiguous()
+    a = _recurrent(native.MemoryArgs(), proj, state, out, positions, slots, state_slots, heads, dim, vdim)
+    a.gates, a.ld_gates, a.head_state, a.cap, a.qscale = gates.data_ptr(), gates.stride(0), state.shape[2], cap, dim ** -0.5
+    a.q_off, a.k_off, a.v_off, a.g_off, a.i_off, a.f_off = offs
+    return a
+
+
+def memory_decode(proj, gates, state, norm, out, positions, slots, state_slots, *, heads: int, dim: int, vdim: int,
+                  offs: tuple[int, int, int, int, int, int], cap: float, eps: float) -> None:
+    """One token per row from the projection (q, k, v, output gate in ``proj``, input and forget gate in the fp32 rows of
+    ``gates``, at ``offs``) to the normed and gated heads ``out``; row r updates state slot ``state_slots[r]``."""
+    a = _memory(proj, gates, state, out, positions, slots, state_slots, heads, dim, vdim, offs, cap)
+    assert out.dtype == proj.dtype and norm.dtype == torch.float32 and norm.numel() == heads * vdim
+    a.norm, a.eps = norm.data_ptr(), eps
+    native.check(native.kernels().xp_memory_decode(C.byref(a), _stream(proj)), "xp_memory_decode")
+
+
+def memory_prefill(proj, gates, state, out, positions, slots, state_slots, q_starts, q_lens, max_q: int, scratch: MemoryScratch, *, heads: int,
+                   dim: int, vdim: int, offs: tuple[int, int, int, int, int, int], cap: float, segs: int = 1, seg_tokens: int = 0,
+                   force_sequential: bool = False) -> None:
+    """Portions of sequences (the longest has ``max_q`` rows) continue state ``state_slots[i]``; ``out`` fp32 ``[rows, heads *
+    vdim]``. bf16 rows with widths in multiples of 8 and at most 256 key dimensions run the chunked tensor-core kernel, with
+    ``segs`` and ``seg_tokens`` as planned for the longest portion (:func:`linear_attn_plan`)."""
+    a = _memory(proj, gates, state, out, positions, slots, state_slots, heads, dim, vdim, offs, cap)
+    n = q_lens.shape[0]
+    assert out.dtype == torch.float32 and scratch.planes.numel() >= 3 * heads * proj.shape[0] and scratch.before.numel() >= n * heads * (dim + 1)
+    a.planes, a.before, a.ws = scratch.planes.data_ptr(), scratch.before.data_ptr(), scratch.ws.data_ptr()
+    a.q_starts, a.q_lens, a.seqs, a.max_q, a.force_sequential = q_starts.data_ptr(), q_lens.data_ptr(), n, max_q, int(force_sequential)
+    if segs > 1 and not a.f32 and not force_sequential:
+        assert scratch.ws.numel() >= n * heads * segs * state.shape[2]
+        a.segs, a.seg_tokens = segs, seg_tokens
+    native.check(native.kernels().xp_memory_prefill(C.byref(a), _stream(proj)), "xp_memory_prefill", 4 if a.segs > 1 else 2)
 
 
 @dataclass

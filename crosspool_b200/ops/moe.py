@@ -19,7 +19,8 @@ from dataclasses import dataclass
 import torch
 
 from .. import native
-from ..models.config import ModelConfig
+from ..models.config import ModelConfig, MoeSpec, ceil8
+from ..models.layered import pad_pitch
 from ..models.weights import FfnLayerWeights
 from . import gemm
 
@@ -116,10 +117,9 @@ def _stream(dev) -> int:
     return torch.cuda.current_stream(dev).cuda_stream
 
 
-def router_topk(logits: torch.Tensor, num_experts: int, top_k: int, *, out_ids: torch.Tensor, out_weights: torch.Tensor,
-                sigmoid: bool = False, renormalize: bool = True, scale: float = 1.0,
-                logit_bias: torch.Tensor | None = None, correction_bias: torch.Tensor | None = None,
-                round_weights_bf16: bool = False) -> None:
+def _router_args(logits: torch.Tensor, num_experts: int, top_k: int, out_ids: torch.Tensor, out_weights: torch.Tensor, sigmoid: bool = False,
+                 renormalize: bool = True, scale: float = 1.0, logit_bias: torch.Tensor | None = None,
+                 correction_bias: torch.Tensor | None = None, round_weights_bf16: bool = False) -> "native.RouterArgs":
     a = native.RouterArgs()
     a.logits = logits.data_ptr()
     a.logit_bias = logit_bias.data_ptr() if logit_bias is not None else None
@@ -128,6 +128,13 @@ def router_topk(logits: torch.Tensor, num_experts: int, top_k: int, *, out_ids: 
     a.rows, a.num_experts, a.top_k, a.ld_logits = logits.shape[0], num_experts, top_k, logits.stride(0)
     a.logits_fp32 = int(logits.dtype == torch.float32)
     a.sigmoid, a.renormalize, a.round_weights_bf16, a.scale = int(sigmoid), int(renormalize), int(round_weights_bf16), scale
+    return a
+
+
+def router_topk(logits: torch.Tensor, num_experts: int, top_k: int, *, out_ids: torch.Tensor, out_weights: torch.Tensor, **kw) -> None:
+    """Scores (softmax, or ``sigmoid=True``), the ``top_k`` largest after ``correction_bias``, their weights (``renormalize``,
+    ``scale``)."""
+    a = _router_args(logits, num_experts, top_k, out_ids, out_weights, **kw)
     native.check(native.kernels().xp_router_topk(C.byref(a), _stream(logits.device)), "xp_router_topk")
 
 
@@ -146,6 +153,18 @@ def _grouped(x, w2d, out, *, n_out, rows_cap, bn, dual, up_offset, tiles, n_tile
                    bias=bias, gate_limit=transform[0], up_add=transform[1], act_alpha=transform[2])
     a.tile_table, a.n_tiles, a.w_rows_per_group = tiles.data_ptr(), n_tiles.data_ptr(), rows_per_group
     native.check(native.kernels().xp_gemm(C.byref(a)), "xp_gemm(grouped)")
+
+
+def _route_args(ws: "MoeWorkspace | RoutedWorkspace", rows: int, k: int, lo: int, hi: int, gateup_features: int, down_features: int,
+                bn: int) -> "native.RouteArgs":
+    r = native.RouteArgs()
+    r.topk_ids, r.counts, r.offsets = ws.ids.data_ptr(), ws.counts.data_ptr(), ws.offsets.data_ptr()
+    r.perm_token, r.route_pos = ws.perm_token.data_ptr(), ws.route_pos.data_ptr()
+    r.tiles_gateup, r.tiles_down = ws.tiles_gu.data_ptr(), ws.tiles_dn.data_ptr()
+    r.n_tiles_gateup, r.n_tiles_down = ws.n_tiles.data_ptr(), ws.n_tiles.data_ptr() + 4
+    r.rows, r.top_k, r.expert_lo, r.expert_hi = rows, k, lo, hi
+    r.tm_gateup, r.bn_gateup, r.tm_down, r.bn_down = (gateup_features + 127) // 128, bn, (down_features + 127) // 128, bn
+    return r
 
 
 def moe_forward(x: torch.Tensor, w: FfnLayerWeights, cfg: ModelConfig, out: torch.Tensor | None = None,
@@ -176,13 +195,7 @@ def moe_forward(x: torch.Tensor, w: FfnLayerWeights, cfg: ModelConfig, out: torc
                 round_weights_bf16=bool(w.extra.get("round_topk_weights")))
     # 2. order the routes of the local experts, build the tile tables
     bn = _tile_width(rows, k, n_local)
-    r = native.RouteArgs()
-    r.topk_ids, r.counts, r.offsets = ws.ids.data_ptr(), ws.counts.data_ptr(), ws.offsets.data_ptr()
-    r.perm_token, r.route_pos = ws.perm_token.data_ptr(), ws.route_pos.data_ptr()
-    r.tiles_gateup, r.tiles_down = ws.tiles_gu.data_ptr(), ws.tiles_dn.data_ptr()
-    r.n_tiles_gateup, r.n_tiles_down = ws.n_tiles.data_ptr(), ws.n_tiles.data_ptr() + 4
-    r.rows, r.top_k, r.expert_lo, r.expert_hi = rows, k, lo, hi
-    r.tm_gateup, r.bn_gateup, r.tm_down, r.bn_down = inter // 128, bn, h // 128, bn
+    r = _route_args(ws, rows, k, lo, hi, inter, h, bn)
     native.check(lib.xp_moe_route(C.byref(r), s), "xp_moe_route", 3)
     # 3. gather rows into expert order
     routes = rows * k
@@ -201,4 +214,122 @@ def moe_forward(x: torch.Tensor, w: FfnLayerWeights, cfg: ModelConfig, out: torc
     if w.shared_gate_up is not None and (expert_range is None or lo == 0):
         sh = gemm.linear(gemm.gateup_swiglu(x, w.shared_gate_up), w.shared_down)
         out += sh
+    return out
+
+
+# ------------------------------------------------------------------------------------------ layered decoders
+
+@dataclass
+class RoutedWorkspace:
+    """Scratch of :func:`routed_ffn`, sized for the widest routed layer of a model and ``cap`` rows."""
+
+    ids: torch.Tensor
+    weights: torch.Tensor
+    counts: torch.Tensor
+    offsets: torch.Tensor
+    perm_token: torch.Tensor
+    route_pos: torch.Tensor
+    tiles_gu: torch.Tensor
+    tiles_dn: torch.Tensor
+    n_tiles: torch.Tensor
+    logits: torch.Tensor          # fp32
+    xp: torch.Tensor              # the others: activations
+    act: torch.Tensor
+    yp: torch.Tensor
+    shared: torch.Tensor
+    z: torch.Tensor | None = None # fp32 models: gate and up columns in front of their activation
+
+    @classmethod
+    def for_layers(cls, specs: list[MoeSpec], hidden: int, cap: int, dtype: torch.dtype, device) -> "RoutedWorkspace":
+        def buf(n, dt=torch.int32):
+            return torch.zeros(n, dtype=dt, device=device)
+
+        top, experts, ff = max(s.top for s in specs), max(s.experts for s in specs), ceil8(max(max(s.ff, s.shared_ff) for s in specs))
+        routes, wide = cap * top, (max(2 * ff, hidden) + 127) // 128
+        tiles = wide * (routes // 16 + experts + 1)
+        f32 = dtype == torch.float32
+        return cls(buf(routes), buf(routes, torch.float32), buf(experts), buf(experts + 1), buf(routes), buf(routes), buf(4 * tiles),
+                   buf(4 * tiles), buf(2), buf(cap * (ceil8(max(s.routed for s in specs) + 1)), torch.float32), buf(routes * ceil8(hidden), dtype),
+                   buf(routes * ff, dtype), buf(routes * ceil8(hidden), dtype), buf(cap * ceil8(hidden), dtype),
+                   buf(max(routes, cap) * 2 * ff, dtype) if f32 else None)
+
+
+def prepare_routed(w: FfnLayerWeights) -> None:
+    """Puts a layer's weights in the layout of :func:`routed_ffn` (in place): the gate of the shared expert joins the router's
+    rows, row pitches become whole 16-byte units."""
+    w.gate_up, w.down = pad_pitch(w.gate_up), pad_pitch(w.down)
+    scale = w.extra.get("shared_scale")
+    w.extra["router_rows"] = pad_pitch(w.router if scale is None else torch.cat([w.router, scale.to(w.router.dtype)], 0))
+    if w.shared_gate_up is not None:
+        w.shared_gate_up, w.shared_down = pad_pitch(w.shared_gate_up), pad_pitch(w.shared_down)
+
+
+def _grouped_f32(x, w, out, *, n, tiles, n_tiles, max_tiles) -> None:
+    native.check(native.kernels().xp_gemm_f32_grouped(x.data_ptr(), w.data_ptr(), out.data_ptr(), tiles.data_ptr(), n_tiles.data_ptr(), max_tiles, n,
+                                                      w.shape[2], x.stride(0), w.stride(1), out.stride(0), w.shape[1], _stream(x.device)),
+                 "xp_gemm_f32_grouped")
+
+
+def _gated_rows(x: torch.Tensor, w_gate_up: torch.Tensor, act: torch.Tensor, z: torch.Tensor | None) -> torch.Tensor:
+    """``silu(gate) * up`` of plain rows in the rows' element type."""
+    if x.dtype == torch.float32:
+        from . import mixers
+
+        z = z[:x.shape[0] * w_gate_up.shape[0]].view(x.shape[0], w_gate_up.shape[0])
+        gemm.linear(x, w_gate_up, out=z)
+        return mixers.glu_f32(z, 0.0, 0.0, 1.0, act)
+    return gemm.gateup_swiglu(x, w_gate_up, out=act)
+
+
+def routed_ffn(x: torch.Tensor, w: FfnLayerWeights, spec: MoeSpec, out: torch.Tensor, ws: RoutedWorkspace) -> torch.Tensor:
+    """Routed FFN of ``x`` ``[rows, hidden]`` (any width, bf16 or fp32): fp32 router logits of one product (the shared
+    expert's gate is its last column), routes ordered by expert, two grouped products, and one kernel that adds up the
+    chosen experts, the identity experts and the shared expert. Few rows choose and order in one launch."""
+    rows, h = x.shape
+    f32, lib, s = x.dtype == torch.float32, native.kernels(), _stream(x.device)
+    hp, ffp, E, k = ceil8(h), ceil8(spec.ff), spec.experts, spec.top
+    router = w.extra["router_rows"]
+    ld = ceil8(router.shape[0])
+    logits = ws.logits[:rows * ld].view(rows, ld)[:, :router.shape[0]]
+    gemm.linear(x, router, out=logits)
+    bn = 64 if f32 else _tile_width(rows, k, E)
+    n_gu = 2 * spec.ff if f32 else spec.ff
+    ids, wts = ws.ids[:rows * k].view(rows, k), ws.weights[:rows * k].view(rows, k)
+    a = _router_args(logits, spec.routed, k, ids, wts, scale=spec.scale, correction_bias=w.extra["correction_bias"])
+    r = _route_args(ws, rows, k, 0, E, n_gu, h, bn)
+    if rows <= 128:
+        native.check(lib.xp_moe_topk_route(C.byref(a), C.byref(r), s), "xp_moe_topk_route")
+    else:
+        native.check(lib.xp_router_topk(C.byref(a), s), "xp_router_topk")
+        native.check(lib.xp_moe_route(C.byref(r), s), "xp_moe_route", 3)
+    routes = rows * k
+    xp, yp = (t[:routes * hp].view(routes, hp)[:, :h] for t in (ws.xp, ws.yp))
+    act = ws.act[:routes * ffp].view(routes, ffp)[:, :spec.ff]
+    words = 2 if f32 else 1                               # the gather counts in 16-bit elements
+    native.check(lib.xp_moe_gather(x.data_ptr(), ws.perm_token.data_ptr(), ws.offsets.data_ptr() + 4 * E, xp.data_ptr(), routes, hp * words,
+                                   x.stride(0) * words, s), "xp_moe_gather")
+    if f32:
+        from . import mixers
+
+        most = routes // bn + E
+        z = ws.z[:routes * 2 * spec.ff].view(routes, 2 * spec.ff)
+        _grouped_f32(xp, w.gate_up, z, n=2 * spec.ff, tiles=ws.tiles_gu, n_tiles=ws.n_tiles[0:1], max_tiles=most * r.tm_gateup)
+        mixers.glu_f32(z, 0.0, 0.0, 1.0, act)
+        _grouped_f32(act, w.down, yp, n=h, tiles=ws.tiles_dn, n_tiles=ws.n_tiles[1:2], max_tiles=most * r.tm_down)
+    else:
+        _grouped(xp, w.gate_up.flatten(0, 1), act, n_out=spec.ff, rows_cap=routes, bn=bn, dual=1, up_offset=spec.ff, tiles=ws.tiles_gu,
+                 n_tiles=ws.n_tiles[0:1], rows_per_group=2 * spec.ff, epilogue=gemm.EPI_SWIGLU)
+        _grouped(act, w.down.flatten(0, 1), yp, n_out=h, rows_cap=routes, bn=bn, dual=0, up_offset=0, tiles=ws.tiles_dn,
+                 n_tiles=ws.n_tiles[1:2], rows_per_group=h, epilogue=gemm.EPI_STORE)
+    m = native.MoeMixArgs()
+    if spec.shared_ff:
+        # the experts' products are done with these rows
+        sact = ws.act[:rows * ceil8(spec.shared_ff)].view(rows, ceil8(spec.shared_ff))[:, :spec.shared_ff]
+        _gated_rows(x, w.shared_gate_up, sact, ws.z)
+        shared = ws.shared[:rows * hp].view(rows, hp)[:, :h]
+        gemm.linear(sact, w.shared_down, out=shared)
+        m.shared, m.ld_shared, m.shared_gate, m.ld_gate = shared.data_ptr(), shared.stride(0), logits[:, spec.routed:].data_ptr(), ld
+    m.y, m.x, m.topk_ids, m.route_pos, m.weights, m.out = (t.data_ptr() for t in (yp, x, ws.ids, ws.route_pos, ws.weights, out))
+    m.rows, m.top_k, m.hidden, m.experts, m.ld_y, m.ld_x, m.ld_out, m.f32 = rows, k, h, E, hp, x.stride(0), out.stride(0), int(f32)
+    native.check(lib.xp_moe_mix(C.byref(m), s), "xp_moe_mix")
     return out
