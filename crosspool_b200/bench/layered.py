@@ -1,5 +1,6 @@
-"""Layered decoders beside the closest classic model of equal size on one GPU: ``bench.py --layered`` (Segirax) and
-``--layered saninex`` (also beside Segirax; its sizes and kernels are in ``layered_saninex.py``).
+"""Layered decoders beside the closest classic model of equal size on one GPU: ``bench.py --layered`` (Segirax),
+``--layered saninex`` and ``--layered kadavik`` (also beside Segirax; their sizes and kernels are in ``layered_saninex.py`` and
+``layered_kadavik.py``).
 
 Two sizes whose layers resemble a real model's (random weights, a few layers): latent attention and decayed linear attention
 alternate, each with a PolyNorm FFN that holds as many weights as the gated FFN of the classic model. For both models, in
@@ -222,7 +223,7 @@ def kernel_table(classic: ModelConfig, cfg: ModelConfig, timer: Timer, batch: in
 
 
 def run(steps: int = 20, warmup: int = 5, layers: int = 8, sizes=tuple(SIZES), design: str = "segirax") -> dict:
-    from . import layered_saninex
+    from . import layered_kadavik, layered_saninex
     from .decode_bench import ClockSampler
 
     torch.cuda.set_device(0)
@@ -235,16 +236,17 @@ def run(steps: int = 20, warmup: int = 5, layers: int = 8, sizes=tuple(SIZES), d
         name, heads = SIZES[size]
         classic = mc_preset(name).with_layers(layers)
         segirax = layered_twin(classic, heads, layers)
-        cfg = segirax if design == "segirax" else layered_saninex.twin(classic, heads, layers)
+        other = {"saninex": layered_saninex, "kadavik": layered_kadavik}.get(design)
+        cfg = segirax if other is None else other.twin(classic, heads, layers)
         res = {"classic": name, "layered": throughput(cfg, steps, warmup), "classic_rates": throughput(classic, steps, warmup)}
         torch.cuda.empty_cache()
         timer = Timer(max(10, steps), max(3, warmup), True)
-        if design == "segirax":
+        if other is None:
             res["kernels"] = kernel_table(classic, cfg, timer)
         else:
             res["segirax_rates"] = throughput(segirax, steps, warmup)
             torch.cuda.empty_cache()
-            res["kernels"] = layered_saninex.kernel_table(classic, cfg, timer, CONTEXT, CHUNK, _row)
+            res["kernels"] = other.kernel_table(classic, cfg, timer, CONTEXT, CHUNK, _row)
         torch.cuda.empty_cache()
         out["sizes"][size] = res
     out["clocks"] = sampler.stop()

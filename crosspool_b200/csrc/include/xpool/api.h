@@ -31,7 +31,7 @@ typedef struct XpGemmArgs {
   int k;               /* row pitches are multiples of 16 bytes (multiple of 64 elements in the forms above) */
   int rows;
   int ldw, ldx, ld_out, ld_resid; /* element strides; 0 = dense */
-  int epilogue;        /* 0 store bf16, 1 swiglu (dual), 2 residual add, 3 store fp32, 4 act(value) * resid[ids[row]] */
+  int epilogue;        /* 0 store bf16, 1 swiglu (dual), 2 residual add, 3 store fp32, 4 act(value) * resid */
   int dual;
   int up_offset;       /* first weight row of the up projection */
   int splits;          /* 0 = choose */
@@ -56,10 +56,9 @@ typedef struct XpGemmArgs {
   float out_scale;     /* multiplies the accumulator of epilogues 0 and 3; 0 = 1 */
   int silu_cols;       /* epilogues 0 and 3: features below this are stored as silu(value) */
   float act_cubic;     /* the activation of epilogues 1 and 4: g sigmoid(act_alpha g (1 + act_cubic g^2)) */
-  int ids_limit;       /* epilogue 4: rows of the table; ids outside read row 0 */
-  const int* ids;      /* epilogue 4: [rows] */
-  float* tail;         /* epilogue 0: features from tail_from on are stored here in fp32 instead, [rows, ld_tail] */
-  int tail_from, ld_tail;
+  int tail_from;       /* epilogue 0: features from here on are stored to tail in fp32 instead, [rows, ld_tail] */
+  float* tail;
+  int ld_tail;
 } XpGemmArgs;
 
 typedef struct XpGemmPlan {

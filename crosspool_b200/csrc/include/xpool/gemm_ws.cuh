@@ -38,7 +38,7 @@ enum Epilogue : int {
   kEpiSwiglu = 1,    // dual: out = silu(round(g)) * round(u)
   kEpiResidual = 2,  // out = round(acc) + resid
   kEpiStoreF32 = 3,  // fp32 out = acc (+ bias)
-  kEpiTokenGate = 4, // out = act(acc) * table[ids[row], f], resid being the table
+  kEpiGateMul = 4,   // out = act(round(acc)) * resid
 };
 
 enum Status : uint32_t {
@@ -99,8 +99,6 @@ struct Problem {
   int silu_cols;           // plain stores: features below this are stored as silu(value)
   float out_scale;         // multiplies the accumulator of the two plain store epilogues; 0 = 1
   float act_cubic;         // the activation is g * sigmoid(alpha * g * (1 + cubic * g^2))
-  const int* ids;          // token of every row (kEpiTokenGate), below ids_limit
-  int ids_limit;
   float* tail;             // kEpiStore: features from tail_from on go here in fp32, row r at r * ld_tail
   int tail_from;
   int ld_tail;
@@ -470,25 +468,26 @@ __device__ __forceinline__ void epilogue_store16(const Problem& p, int f, int fb
         v[j] = __fdividef(gg, 1.f + __expf(-a * gg)) * (uu + p.up_add);
       }
     }
-  } else if (p.epilogue == kEpiTokenGate) {
-    const __nv_bfloat16* table = reinterpret_cast<const __nv_bfloat16*>(p.resid) + f;
+  } else if (p.epilogue == kEpiResidual || p.epilogue == kEpiGateMul) {
+    // sixteen loads in flight: no branch around any of them (rows and features that are not stored repeat ones that are)
+    const __nv_bfloat16* r = reinterpret_cast<const __nv_bfloat16*>(p.resid) + static_cast<size_t>(n_first) * p.ld_resid + (live ? f : 0);
+    const int last = valid > 0 ? valid - 1 : 0;
+    uint16_t raw[16];
 #pragma unroll
-    for (int j = 0; j < 16; ++j) {
-      v[j] = 0.f;
-      if (j < valid) {
-        const int id = p.ids[n_first + j];
-        const float e = __bfloat162float(table[static_cast<size_t>(id >= 0 && id < p.ids_limit ? id : 0) * p.ld_resid]);
-        const float gg = round_bf16(g[j] + bias);
-        v[j] = __fdividef(gg, 1.f + __expf(-p.act_alpha * gg * fmaf(p.act_cubic * gg, gg, 1.f))) * e;
-      }
-    }
-  } else if (p.epilogue == kEpiResidual) {
-    const __nv_bfloat16* r = reinterpret_cast<const __nv_bfloat16*>(p.resid) + static_cast<size_t>(n_first) * p.ld_resid + f;
+    for (int j = 0; j < 16; ++j)
+      asm volatile("ld.global.u16 %0, [%1];" : "=h"(raw[j]) : "l"(r + static_cast<size_t>(j < last ? j : last) * p.ld_resid));
     float rr[16];
 #pragma unroll
-    for (int j = 0; j < 16; ++j) rr[j] = j < valid ? __bfloat162float(r[static_cast<size_t>(j) * p.ld_resid]) : 0.f;
+    for (int j = 0; j < 16; ++j) rr[j] = __uint_as_float(static_cast<uint32_t>(raw[j]) << 16);
 #pragma unroll
-    for (int j = 0; j < 16; ++j) v[j] = round_bf16(g[j] + bias) + rr[j];
+    for (int j = 0; j < 16; ++j) v[j] = round_bf16(g[j] + bias);
+    if (p.epilogue == kEpiResidual) {
+#pragma unroll
+      for (int j = 0; j < 16; ++j) v[j] += rr[j];
+    } else {
+#pragma unroll
+      for (int j = 0; j < 16; ++j) v[j] = __fdividef(v[j], 1.f + __expf(-p.act_alpha * v[j] * fmaf(p.act_cubic * v[j], v[j], 1.f))) * rr[j];
+    }
   } else {
     const float sc = p.out_scale == 0.f ? 1.f : p.out_scale;
 #pragma unroll

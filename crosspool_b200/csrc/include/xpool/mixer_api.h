@@ -96,15 +96,14 @@ typedef struct XpGluArgs {
   float limit, up_add, alpha, cubic;
 } XpGluArgs;
 
-/* out = act(z) * table[ids[row]], act as above, in fp32. */
-typedef struct XpTokenGateArgs {
+/* out = act(z) * e, act as above, in fp32; out may be z. */
+typedef struct XpGateMulArgs {
   const float* z;        /* [rows, ld_z] */
-  const float* table;    /* [vocab, ld_table] */
-  const int* ids;        /* [rows] */
+  const float* e;        /* [rows, ld_e] */
   float* out;            /* [rows, ld_out] */
-  int rows, cols, ld_z, ld_table, ld_out, vocab;
+  int rows, cols, ld_z, ld_e, ld_out;
   float alpha, cubic;
-} XpTokenGateArgs;
+} XpGateMulArgs;
 
 /* Grouped-query attention without rotation, per token row: RMS norm of query and key heads, queries laid out
  * [rows, kv_heads, group_pad, dq], keys and values written to the cache row of the token, everything zero-padded. */
@@ -313,7 +312,7 @@ int xp_gated_rms(const XpGatedRmsArgs* a, void* stream);
 int xp_post_norm(const XpPostNormArgs* a, void* stream);
 int xp_head_gate(const XpHeadGateArgs* a, void* stream);
 int xp_glu_f32(const XpGluArgs* a, void* stream);
-int xp_token_gate_f32(const XpTokenGateArgs* a, void* stream);
+int xp_gate_mul_f32(const XpGateMulArgs* a, void* stream);
 int xp_grouped_prep(const XpGroupedPrepArgs* a, void* stream);
 int xp_conv_rope_decode(const XpConvRopeArgs* a, void* stream);
 int xp_conv_rope_prefill(const XpConvRopeArgs* a, void* stream);

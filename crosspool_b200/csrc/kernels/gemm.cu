@@ -287,8 +287,7 @@ extern "C" int xp_gemm_plan(const XpGemmArgs* a, XpGemmPlan* plan) {
   if (whole && (a->n_out % gemm::kTileM != 0 || a->k % kblk != 0)) return -10;
   const int batch = a->batch > 1 ? a->batch : 1;
   if (batch > 1 && (whole || a->tile_table != nullptr || a->dual || a->epilogue == gemm::kEpiResidual || a->bias != nullptr || a->x_group_rows < a->rows)) return -16;
-  if (a->epilogue == gemm::kEpiTokenGate && (a->dual || batch > 1 || a->tile_table != nullptr || a->ids == nullptr || a->resid == nullptr || a->ids_limit <= 0))
-    return -17;
+  if (a->epilogue == gemm::kEpiGateMul && (a->dual || batch > 1 || a->tile_table != nullptr || a->resid == nullptr)) return -17;
   if (a->tail != nullptr && (a->epilogue != gemm::kEpiStore || batch > 1 || a->tile_table != nullptr)) return -18;
   if (a->fp8 && (a->dual || a->w_tiled || a->tile_table != nullptr || a->w_scale == nullptr || a->x_scale == nullptr ||
                  a->ld_xscale % 4 != 0 || a->bn > gemm::kMaxBnF8))
@@ -398,8 +397,6 @@ extern "C" int xp_gemm(const XpGemmArgs* a) {
   p.out_scale = a->out_scale;
   p.silu_cols = a->silu_cols;
   p.act_cubic = a->act_cubic;
-  p.ids = a->ids;
-  p.ids_limit = a->ids_limit;
   p.tail = a->tail;
   p.tail_from = a->tail_from;
   p.ld_tail = a->ld_tail;

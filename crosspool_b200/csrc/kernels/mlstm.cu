@@ -158,7 +158,9 @@ struct Step {
 __device__ __forceinline__ Step then(const Step& x, const Step& y) { return {x.f + y.f, fmaxf(x.top + y.f, y.top)}; }
 
 // CTA = (head, portion); a warp takes a chunk at a time, two tokens per lane.
-__global__ void __launch_bounds__(kThreads)
+constexpr int kGateThreads = 1024;
+
+__global__ void __launch_bounds__(kGateThreads)
 memory_gates_kernel(XpMemoryArgs a) {
   extern __shared__ float sm[];            // per chunk: step (f, top), then the maximum before it
   const int h = blockIdx.x, seq = blockIdx.y, n = a.q_lens[seq];
@@ -169,11 +171,11 @@ memory_gates_kernel(XpMemoryArgs a) {
   const bool fresh = a.positions[r0] == 0;
   const float* n_p = a.state + (static_cast<size_t>(a.state_slots[seq]) * a.heads + h) * a.head_state + static_cast<size_t>(a.dim) * a.vdim;
   float* before = a.before + (static_cast<size_t>(seq) * a.heads + h) * (a.dim + 1);
-  for (int c = threadIdx.x; c <= a.dim; c += kThreads) before[c] = fresh ? 0.f : n_p[c];
+  for (int c = threadIdx.x; c <= a.dim; c += kGateThreads) before[c] = fresh ? 0.f : n_p[c];
   float* pa = plane(a, kA, h) + r0;
   float* pr = plane(a, kR, h) + r0;
   float* pm = plane(a, kM, h) + r0;
-  for (int c = warp; c < chunks; c += kThreads / 32) {
+  for (int c = warp; c < chunks; c += kGateThreads / 32) {
     const int t = c * kChunk + lane * 2;
     float i[2], f[2];
 #pragma unroll
@@ -219,7 +221,7 @@ memory_gates_kernel(XpMemoryArgs a) {
     }
   }
   __syncthreads();
-  for (int t = threadIdx.x; t < n; t += kThreads) {
+  for (int t = threadIdx.x; t < n; t += kGateThreads) {
     const float top = fmaxf(steps[t / kChunk].x, pr[t]);
     pa[t] *= kLog2e;
     pr[t] = -top * kLog2e;
@@ -646,23 +648,38 @@ memory_scan_kernel(XpMemoryArgs a) {
   if (total <= 0) return;
   const size_t matrix = static_cast<size_t>(a.dim) * a.vdim;
   const size_t i = blockIdx.x * 256ull + threadIdx.x;
-  if (i >= matrix + a.dim) return;
+  __shared__ float factor[64];                       // what a whole segment leaves of the state before it
   const int r0 = a.q_starts[seq];
   const float* before = a.before + (static_cast<size_t>(seq) * a.heads + h) * (a.dim + 1);
   const float* pr = plane(a, kR, h) + r0;
   const float* pm = plane(a, kM, h) + r0;
+  const int segs = (total + a.seg_tokens - 1) / a.seg_tokens;              // at most 64
+  for (int s = threadIdx.x >> 5; s + 1 < segs; s += 8) {                   // the last segment adds to nobody
+    float f = 0.f;
+    for (int c = threadIdx.x & 31; c < a.seg_tokens / kChunk; c += 32) {
+      const int t = s * a.seg_tokens + c * kChunk;
+      f += (t == 0 ? before[a.dim] : pm[t - 1]) * kLog2e + pr[t + kChunk - 1];
+    }
+    f = elem::warp_sum(f);
+    if ((threadIdx.x & 31) == 0) factor[s] = ex2_approx(f);
+  }
+  __syncthreads();
+  if (i >= matrix + a.dim) return;
   float* mid = a.ws + (static_cast<size_t>(seq) * a.heads + h) * a.segs * a.head_state + i;
   float x;
   if (i >= matrix) x = before[i - matrix];
   else x = a.positions[r0] == 0 ? 0.f : a.state[(static_cast<size_t>(a.state_slots[seq]) * a.heads + h) * a.head_state + i];
-  for (int s = 0; s * a.seg_tokens < total; ++s) {
-    const bool tail = (s + 1) * a.seg_tokens >= total;                     // the last segment adds to nobody
-    float f = 0.f;
-    for (int t = s * a.seg_tokens; t < (s + 1) * a.seg_tokens && !tail; t += kChunk)
-      f += (t == 0 ? before[a.dim] : pm[t - 1]) * kLog2e + pr[t + kChunk - 1];
-    const float add = tail ? 0.f : mid[static_cast<size_t>(s) * a.head_state];
-    mid[static_cast<size_t>(s) * a.head_state] = x;
-    x = fmaf(ex2_approx(f), x, add);
+  constexpr int kAhead = 8;                          // loads in flight before the first store
+  for (int s0 = 0; s0 < segs; s0 += kAhead) {
+    float add[kAhead];
+#pragma unroll
+    for (int u = 0; u < kAhead; ++u) add[u] = s0 + u + 1 < segs ? mid[static_cast<size_t>(s0 + u) * a.head_state] : 0.f;
+#pragma unroll
+    for (int u = 0; u < kAhead; ++u) {
+      if (s0 + u >= segs) break;
+      mid[static_cast<size_t>(s0 + u) * a.head_state] = x;
+      if (s0 + u + 1 < segs) x = fmaf(factor[s0 + u], x, add[u]);
+    }
   }
 }
 
@@ -726,7 +743,7 @@ int launch_chunked(const XpMemoryArgs& a, cudaStream_t s) {
   if (b.segs <= 1) {
     b.segs = 1;
     b.seg_tokens = 0x40000000;
-  } else if (b.ws == nullptr || b.seg_tokens <= 0 || b.seg_tokens % kChunk != 0) {
+  } else if (b.ws == nullptr || b.segs > 64 || b.seg_tokens <= 0 || b.seg_tokens % kChunk != 0) {
     return -13;
   }
   const dim3 grid((a.vdim + VS - 1) / VS * b.segs, a.heads, a.seqs);
@@ -773,7 +790,7 @@ extern "C" int xp_memory_prefill(const XpMemoryArgs* a, void* stream) {
   const size_t sm = static_cast<size_t>((a->max_q + kChunk - 1) / kChunk) * 8;
   int rc = big_smem(memory_gates_kernel, sm);
   if (rc != 0) return rc;
-  memory_gates_kernel<<<dim3(a->heads, a->seqs), kThreads, sm, s>>>(*a);
+  memory_gates_kernel<<<dim3(a->heads, a->seqs), kGateThreads, sm, s>>>(*a);
   if (a->f32) return sequential_any<float>(*a, s);
   const bool chunked = !a->force_sequential && a->dim <= 256 && a->dim % 8 == 0 && a->vdim % 8 == 0 && a->ld_proj % 8 == 0 && a->q_off % 8 == 0 &&
                        a->k_off % 8 == 0 && a->v_off % 8 == 0 && a->ld_out % 2 == 0 && a->head_state % 2 == 0 && aligned(a->proj, 16) &&

@@ -177,34 +177,40 @@ route_offsets_tiles_kernel(const int* __restrict__ counts, int n_experts, int* _
   }
 }
 
-// Stable placement: routes of an expert keep their (token, k) order.
-__global__ void __launch_bounds__(256)
+// Stable placement: routes of an expert keep their (token, k) order. A thread takes kPlaceRun consecutive routes.
+constexpr int kPlaceThreads = 512, kPlaceRun = 8;
+
+__global__ void __launch_bounds__(kPlaceThreads)
 route_place_kernel(const int* __restrict__ ids, int n_routes, int top_k, int lo, const int* __restrict__ offsets,
                    int* __restrict__ perm_token, int* __restrict__ route_pos) {
-  __shared__ int warp_tot[8];
-  __shared__ int base;
-  const int e = lo + blockIdx.x;
-  if (threadIdx.x == 0) base = offsets[blockIdx.x];
-  __syncthreads();
-  for (int start = 0; start < n_routes; start += 256) {
-    const int i = start + threadIdx.x;
-    const int hit = (i < n_routes && ids[i] == e) ? 1 : 0;
-    const unsigned ballot = __ballot_sync(0xffffffffu, hit);
-    const int lane = threadIdx.x & 31, w = threadIdx.x >> 5;
-    if (lane == 0) warp_tot[w] = __popc(ballot);
+  __shared__ int warp_tot[kPlaceThreads / 32];
+  const int e = lo + blockIdx.x, lane = threadIdx.x & 31, w = threadIdx.x >> 5;
+  int base = offsets[blockIdx.x];
+  for (int start = 0; start < n_routes; start += kPlaceThreads * kPlaceRun) {
+    const int first = start + threadIdx.x * kPlaceRun;
+    unsigned hits = 0;
+#pragma unroll
+    for (int u = 0; u < kPlaceRun; ++u)
+      if (first + u < n_routes && ids[first + u] == e) hits |= 1u << u;
+    int before = __popc(hits);
+#pragma unroll
+    for (int d = 1; d < 32; d <<= 1) {
+      const int x = __shfl_up_sync(0xffffffffu, before, d);
+      if (lane >= d) before += x;
+    }
+    if (lane == 31) warp_tot[w] = before;
     __syncthreads();
-    int before = __popc(ballot & ((1u << lane) - 1));
-    for (int j = 0; j < w; ++j) before += warp_tot[j];
-    if (hit) {
-      const int pos = base + before;
+    int pos = base + before - __popc(hits);
+#pragma unroll
+    for (int j = 0; j < kPlaceThreads / 32; ++j) {
+      const int t = warp_tot[j];
+      pos += j < w ? t : 0;
+      base += t;
+    }
+    for (; hits != 0; hits &= hits - 1, ++pos) {
+      const int i = first + __ffs(hits) - 1;
       perm_token[pos] = i / top_k;
       route_pos[i] = pos;
-    }
-    __syncthreads();
-    if (threadIdx.x == 0) {
-      int t = 0;
-      for (int j = 0; j < 8; ++j) t += warp_tot[j];
-      base += t;
     }
     __syncthreads();
   }
@@ -566,7 +572,7 @@ extern "C" int xp_moe_route(const XpRouteArgs* a, void* stream) {
   route_offsets_tiles_kernel<<<1, 1024, 0, s>>>(a->counts, n_local, a->offsets, a->tm_gateup, a->bn_gateup,
                                                 reinterpret_cast<int4*>(a->tiles_gateup), a->n_tiles_gateup, a->tm_down,
                                                 a->bn_down, reinterpret_cast<int4*>(a->tiles_down), a->n_tiles_down);
-  route_place_kernel<<<n_local, 256, 0, s>>>(a->topk_ids, n_routes, a->top_k, a->expert_lo, a->offsets, a->perm_token,
+  route_place_kernel<<<n_local, kPlaceThreads, 0, s>>>(a->topk_ids, n_routes, a->top_k, a->expert_lo, a->offsets, a->perm_token,
                                              a->route_pos);
   return last_error();
 }

@@ -27,7 +27,7 @@ from ..models.config import (DeltaMixer, GatedLinearMixer, GroupedMixer, LatentM
 from ..models.layered import LayeredLayerWeights, rotary_table
 from ..ops import gemm
 from ..ops import mixers as M
-from ..ops.attention import decode_plan
+from ..ops.attention import decode_plan, embedding
 
 # Portions of at most this many tokens run as single rows (latent attention: in the absorbed form, expanding the whole context
 # costs more).
@@ -134,7 +134,7 @@ class LayeredForward:
         self.tails = buf(cap * max((lw.offs["end"] - lw.fp32_from for lw in layers if lw.fp32_from), default=0), torch.float32)
         if cfg.token_side:
             self.side = torch.zeros(cap, ceil8(cfg.token_side), dtype=dt, device=dev)[:, :cfg.token_side]
-            self.side_z = self.side if dt == torch.float32 else None
+            self.side_e = torch.zeros(cap, engine.w.extra["side_embed"].shape[1], dtype=dt, device=dev)
         if lin or gla or delta or mem:
             self.o_lin = buf(cap * max(m.out_features for m in lin + gla + delta + mem), torch.float32)
         if lin:
@@ -328,6 +328,8 @@ class LayeredForward:
         pending: dict = dict(ids=ids, table=self.e.w.embed)
         if cfg.embed_scale != 1.0:
             pending["embed_scale"] = cfg.embed_scale
+        if cfg.token_side:
+            embedding(ids, self.e.w.extra["side_embed"], out=self.side_e[:rows])
         for l, lw in enumerate(self.layers):
             self._enter(resid, lw.norm1, x, pending)
             proj, ys = self._mix(l, lw, x, b)
@@ -344,17 +346,17 @@ class LayeredForward:
                     gemm.linear(x2, lw.rg2, out=rg2, bias=lw.rg2_bias)
                     pending = dict(parts=self.e.port.run(l, x2, rows, mode), gate=rg2)
             if lw.side_gate is not None:
-                pending = self._token_side(l, lw, resid, x, ids, pending)
+                pending = self._token_side(l, lw, resid, x, pending)
             self.tap(l, rows, pending)
         self._pending = pending
 
-    def _token_side(self, l: int, lw: LayeredLayerWeights, resid: torch.Tensor, x: torch.Tensor, ids: torch.Tensor, pending: dict) -> dict:
+    def _token_side(self, l: int, lw: LayeredLayerWeights, resid: torch.Tensor, x: torch.Tensor, pending: dict) -> dict:
         """``gelu_tanh(side_gate x)`` times the layer's part of the token's second embedding, mapped back to the model width;
         ``x`` is the residual itself."""
         rows, n = x.shape[0], self.e.cfg.token_side
         M.post_norm(resid, x, **pending)
         e = self.side[:rows]
-        M.token_gate(x, lw.side_gate, self.e.w.extra["side_embed"][:, l * n:(l + 1) * n], ids, e, self.side_z[:rows] if self.side_z is not None else None)
+        M.gelu_gate(x, lw.side_gate, self.side_e[:rows, l * n:(l + 1) * n], e)
         gemm.linear(e, lw.side_proj, out=self.y[:rows])
         return dict(branches=[self.y[:rows]], norm=lw.side_norm)
 

@@ -252,7 +252,9 @@ def layered_attention_weights(cfg: ModelConfig, get: Getter, device, dtype: torc
     final = (_plain_norm if cfg.input_norm else _centred_norm if cfg.output_norm else _norm)(get, "final.norm", cfg)
     w = AttentionWeights(embed, layers, final, pad_pitch(embed))
     if cfg.token_side:
-        w.extra["side_embed"] = get("side.embed", (cfg.vocab_size, cfg.num_layers * cfg.token_side)).contiguous()
+        # rows of whole 16-byte units, gathered for all layers at once
+        n = cfg.num_layers * cfg.token_side
+        w.extra["side_embed"] = torch.nn.functional.pad(get("side.embed", (cfg.vocab_size, n)), (0, ceil8(n) - n)).contiguous()
     return w
 
 

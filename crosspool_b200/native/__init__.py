@@ -69,10 +69,8 @@ class GemmArgs(C.Structure):
         ("out_scale", C.c_float),
         ("silu_cols", C.c_int),
         ("act_cubic", C.c_float),
-        ("ids_limit", C.c_int),
-        ("ids", C.c_void_p),
-        ("tail", C.c_void_p),
         ("tail_from", C.c_int),
+        ("tail", C.c_void_p),
         ("ld_tail", C.c_int),
     ]
 
@@ -303,7 +301,7 @@ PostNormArgs = _struct("PostNormArgs", "XpPostNormArgs", a_ptr="resid", b_ptr2="
 HeadGateArgs = _struct("HeadGateArgs", "XpHeadGateArgs", a_ptr="o weight gate out", b_int="rows heads dim ld_o ld_gate ld_out", c_float="eps",
                        d_int="f32 per_head_weight sigmoid_gate")
 GluArgs = _struct("GluArgs", "XpGluArgs", a_ptr="z out", b_int="rows cols ld_z ld_out", c_float="limit up_add alpha cubic")
-TokenGateArgs = _struct("TokenGateArgs", "XpTokenGateArgs", a_ptr="z table ids out", b_int="rows cols ld_z ld_table ld_out vocab", c_float="alpha cubic")
+GateMulArgs = _struct("GateMulArgs", "XpGateMulArgs", a_ptr="z e out", b_int="rows cols ld_z ld_e ld_out", c_float="alpha cubic")
 GroupedPrepArgs = _struct("GroupedPrepArgs", "XpGroupedPrepArgs", a_ptr="proj q_norm k_norm slots k_cache v_cache q_out",
                           b_int="rows heads kv_heads group_pad dim vdim dq dv ld_proj q_off k_off v_off", c_float="eps", d_int="f32")
 GroupedAttnArgs = _struct("GroupedAttnArgs", "XpGroupedAttnArgs", a_ptr="q k_cache v_cache out gate row_seq positions slots block_table",
@@ -342,7 +340,7 @@ def _declare_mixers(lib: C.CDLL) -> None:
     for fn, args in (("xp_resid_norm", ResidNormArgs), ("xp_polynorm", PolyNormArgs), ("xp_gated_rms", GatedRmsArgs),
                      ("xp_latent_prep", LatentPrepArgs), ("xp_latent_attn", LatentAttnArgs), ("xp_latent_gather", LatentGatherArgs),
                      ("xp_linear_attn_decode", LinearAttnArgs), ("xp_linear_attn_prefill", LinearAttnArgs),
-                     ("xp_post_norm", PostNormArgs), ("xp_head_gate", HeadGateArgs), ("xp_glu_f32", GluArgs), ("xp_token_gate_f32", TokenGateArgs),
+                     ("xp_post_norm", PostNormArgs), ("xp_head_gate", HeadGateArgs), ("xp_glu_f32", GluArgs), ("xp_gate_mul_f32", GateMulArgs),
                      ("xp_grouped_prep", GroupedPrepArgs), ("xp_conv_rope_decode", ConvRopeArgs), ("xp_conv_rope_prefill", ConvRopeArgs), ("xp_grouped_attn", GroupedAttnArgs),
                      ("xp_gated_linear_decode", GatedLinearArgs), ("xp_gated_linear_prefill", GatedLinearArgs),
                      ("xp_memory_decode", MemoryArgs), ("xp_memory_prefill", MemoryArgs), ("xp_delta_decode", DeltaArgs), ("xp_delta_prep", DeltaArgs), ("xp_delta_prefill", DeltaArgs)):

@@ -137,6 +137,7 @@ def embedding(ids: torch.Tensor, table: torch.Tensor, out: torch.Tensor | None =
     rows, hidden = ids.shape[0], table.shape[1]
     if out is None:
         out = torch.empty(rows, hidden, dtype=table.dtype, device=table.device)
+    hidden = hidden * table.element_size() // 2          # rows are copied as they are, counted in 16-bit elements
     native.check(native.kernels().xp_embedding(ids.data_ptr(), table.data_ptr(), out.data_ptr(), rows, hidden,
                                                table.shape[0], _stream(table.device)), "xp_embedding")
     return out

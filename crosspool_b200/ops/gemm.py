@@ -29,7 +29,7 @@ EPI_STORE = 0
 EPI_SWIGLU = 1
 EPI_RESIDUAL = 2
 EPI_STORE_F32 = 3
-EPI_TOKEN_GATE = 4
+EPI_GATE_MUL = 4
 
 _WS_BYTES = 96 << 20
 _COUNTER_WORDS = 1 << 16
@@ -237,13 +237,12 @@ def linear_batched(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, out_grou
     return out
 
 
-def linear_token_gate(x: torch.Tensor, w: torch.Tensor, table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor, alpha: float,
-                      cubic: float) -> torch.Tensor:
-    """``act(x @ w.T) * table[ids]`` in bf16, ``act(g) = g sigmoid(alpha g (1 + cubic g^2))``; ``ids`` int32, one per row."""
-    assert table.dtype == torch.bfloat16 and table.stride(1) == 1 and ids.dtype == torch.int32 and table.shape[1] == w.shape[0]
-    a = _args(x, w, out, n_out=w.shape[0], rows=x.shape[0], epilogue=EPI_TOKEN_GATE, resid=table, act_alpha=alpha, act_cubic=cubic)
-    a.ids, a.ids_limit = ids.data_ptr(), table.shape[0]
-    native.check(native.kernels().xp_gemm(C.byref(a)), "xp_gemm(token gate)")
+def linear_gate_mul(x: torch.Tensor, w: torch.Tensor, e: torch.Tensor, out: torch.Tensor, alpha: float, cubic: float, splits: int = 0,
+                    bn: int = 0) -> torch.Tensor:
+    """``act(x @ w.T) * e`` in bf16, ``act(g) = g sigmoid(alpha g (1 + cubic g^2))``."""
+    assert e.dtype == torch.bfloat16 and e.stride(1) == 1 and tuple(e.shape) == (x.shape[0], w.shape[0])
+    a = _args(x, w, out, n_out=w.shape[0], rows=x.shape[0], epilogue=EPI_GATE_MUL, resid=e, act_alpha=alpha, act_cubic=cubic, splits=splits, bn=bn)
+    native.check(native.kernels().xp_gemm(C.byref(a)), "xp_gemm(gate)")
     return out
 
 

@@ -124,17 +124,16 @@ def glu_f32(z: torch.Tensor, limit: float, up_add: float, alpha: float, out: tor
     return out
 
 
-def token_gate(x: torch.Tensor, w: torch.Tensor, table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor, z: torch.Tensor) -> torch.Tensor:
-    """``gelu_tanh(x @ w.T) * table[ids]``; ``table`` ``[vocab, n]`` may be a column range of a wider one. bf16: one product
-    with the gate in its epilogue; fp32: product into ``z``, then a row kernel."""
+def gelu_gate(x: torch.Tensor, w: torch.Tensor, e: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+    """``gelu_tanh(x @ w.T) * e``. bf16: one product with the gate in its epilogue; fp32: product, then a row kernel."""
     if x.dtype == torch.bfloat16:
-        return gemm.linear_token_gate(x, w, table, ids, out, GELU_ALPHA, GELU_CUBIC)
-    gemm.linear(x, w, out=z)
-    a = native.TokenGateArgs()
-    a.z, a.table, a.ids, a.out = z.data_ptr(), table.data_ptr(), ids.data_ptr(), out.data_ptr()
-    a.rows, a.cols, a.ld_z, a.ld_table, a.ld_out, a.vocab = x.shape[0], w.shape[0], z.stride(0), table.stride(0), out.stride(0), table.shape[0]
+        return gemm.linear_gate_mul(x, w, e, out, GELU_ALPHA, GELU_CUBIC)
+    gemm.linear(x, w, out=out)
+    a = native.GateMulArgs()
+    a.z, a.e, a.out = out.data_ptr(), e.data_ptr(), out.data_ptr()
+    a.rows, a.cols, a.ld_z, a.ld_e, a.ld_out = x.shape[0], w.shape[0], out.stride(0), e.stride(0), out.stride(0)
     a.alpha, a.cubic = GELU_ALPHA, GELU_CUBIC
-    native.check(native.kernels().xp_token_gate_f32(C.byref(a), _stream(x)), "xp_token_gate_f32")
+    native.check(native.kernels().xp_gate_mul_f32(C.byref(a), _stream(x)), "xp_gate_mul_f32")
     return out
 
 

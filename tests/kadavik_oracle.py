@@ -126,17 +126,21 @@ def dense(h, t, act):
     return (act(h @ t("gate").T) * (h @ t("up").T)) @ t("down").T
 
 
-def routing(z, correction, top, scale):
-    """Logits ``[T, n]`` -> weights ``[T, n]``, zero where an expert is not chosen."""
+def routing(z, correction, top, scale, margins=None):
+    """Logits ``[T, n]`` -> weights ``[T, n]``, zero where an expert is not chosen. ``margins``: a list that receives how far
+    every token's last choice was from the first expert it left out."""
     s = z.softmax(-1)
-    chosen = (s + correction).topk(top, -1).indices
+    order = (s + correction).sort(-1, descending=True)
+    if margins is not None and top < z.shape[-1]:
+        margins.append(order.values[:, top - 1] - order.values[:, top])
+    chosen = order.indices[:, :top]
     w = s.gather(-1, chosen)
     return torch.zeros_like(s).scatter(-1, chosen, w / (w.sum(-1, keepdim=True) + 1e-20) * scale)
 
 
-def experts(h, m, t):
+def experts(h, m, t, margins=None):
     r = m["router"]
-    w = routing(h @ t("router").T, t("correction"), r["top"], r["scale"])
+    w = routing(h @ t("router").T, t("correction"), r["top"], r["scale"], margins)
     y = torch.zeros_like(h)
     for e in range(r["experts"]):
         y = y + w[:, e:e + 1] * dense(h, lambda n: t(f"e{e}.{n}"), silu)
@@ -147,16 +151,17 @@ def experts(h, m, t):
     return y
 
 
-def feed_forward(h, m, t):
-    return dense(h, t, gelu_tanh) if m["kind"] == "dense" else experts(h, m, t)
+def feed_forward(h, m, t, margins=None):
+    return dense(h, t, gelu_tanh) if m["kind"] == "dense" else experts(h, m, t, margins)
 
 
 def token_side(x, e, t, eps):
     return rms((gelu_tanh(x @ t("gate").T) * e) @ t("proj").T, eps) * t("norm")
 
 
-def forward(config, tensors, ids, dtype=torch.float64, layer_outputs=None):
-    """Logits ``[T, vocab]`` of one sequence; ``layer_outputs``: a list that receives the residual after every layer."""
+def forward(config, tensors, ids, dtype=torch.float64, layer_outputs=None, margins=None):
+    """Logits ``[T, vocab]`` of one sequence; ``layer_outputs``: a list that receives the residual after every layer;
+    ``margins``: see :func:`routing`."""
     w = {k: v.to(dtype) for k, v in tensors.items()}
     eps, ids = config["norm"]["eps"], torch.as_tensor(ids)
     x = w["embed"][ids] * config["embedding"]["scale"]
@@ -174,7 +179,7 @@ def forward(config, tensors, ids, dtype=torch.float64, layer_outputs=None):
             y, kv[i] = attention(h, m, mix, eps, kv[m["kv_from"]] if m.get("kv_from") is not None else None)
         x = x + rms(y, eps) * w[p + ".norm1b"]
         if layer["mlp"] is not None:
-            y = feed_forward(rms(x, eps) * w[p + ".norm2"], layer["mlp"], lambda n: w[f"{p}.mlp.{n}"])
+            y = feed_forward(rms(x, eps) * w[p + ".norm2"], layer["mlp"], lambda n: w[f"{p}.mlp.{n}"], margins)
             x = x + rms(y, eps) * w[p + ".norm2b"]
         if config.get("token_side"):
             n = config["token_side"]["dim"]
@@ -182,3 +187,63 @@ def forward(config, tensors, ids, dtype=torch.float64, layer_outputs=None):
         if layer_outputs is not None:
             layer_outputs.append(x)
     return (rms(x, eps) * w["final.norm"]) @ w["embed"].T * config["logit_scale"]
+
+
+def random_tensors(config, seed):
+    """Random bf16 tensors under the checkpoint's names, sized so that every term matters. Memories' queries resemble their keys:
+    a first token reads (q . k) v, which is normed, so that its sign would be a matter of rounding where q and k happen to be
+    orthogonal."""
+    g = torch.Generator().manual_seed(seed)
+    W, V = config["width"], config["vocab"]
+
+    def lin(o, i, gain=1.0):
+        return (torch.randn(o, i, generator=g) * gain / math.sqrt(i)).bfloat16()
+
+    def vec(n, mean=1.0, std=0.3):
+        return (mean + std * torch.randn(n, generator=g)).bfloat16()
+
+    def alike(w):
+        return (0.8 * w.float() + 0.6 * torch.randn(w.shape, generator=g) * w.float().std()).bfloat16()
+
+    def gated(p, ff):
+        t[p + "gate"], t[p + "up"], t[p + "down"] = lin(ff, W), lin(ff, W), lin(W, ff)
+
+    t = {"embed": (torch.randn(V, W, generator=g) / config["embedding"]["scale"]).bfloat16()}
+    for i, layer in enumerate(config["layers"]):
+        m, mlp, q = layer["mixer"], layer["mlp"], f"l{i}.mix."
+        names = ["norm1", "norm1b"] + (["norm2", "norm2b"] if mlp else [])
+        for n in names:
+            t[f"l{i}.{n}"] = vec(W, 0.6 if n.endswith("b") else 1.0)
+        H, d, e = m["heads"], m["dim"], m["vdim"]
+        if layer["type"] == "mlstm":
+            t[q + "q"], t[q + "v"], t[q + "g"], t[q + "o"] = lin(H * d, W), lin(H * e, W), lin(H * e, W), lin(W, H * e)
+            t[q + "k"], t[q + "norm"] = alike(t[q + "q"]), vec(H * e)
+            t[q + "i"], t[q + "i.b"], t[q + "f"], t[q + "f.b"] = lin(H, W, 2.0), vec(H, -0.5, 1.5), lin(H, W, 2.0), vec(H, 2.5, 2.0)
+        else:
+            rows = {"q": H * d}
+            if m.get("kv_from") is None:
+                rows.update(k=m["kv_heads"] * d, v=m["kv_heads"] * e)
+            for n, r in rows.items():
+                t[q + n] = lin(r, W, 1.2)
+                if m.get("conv"):
+                    t[q + n + ".conv"] = lin(r, m["conv"], 1.2)
+            t[q + "g"], t[q + "o"] = lin(H * e, W), lin(W, H * e)
+        p = f"l{i}.mlp."
+        if mlp and mlp["kind"] == "dense":
+            gated(p, mlp["ff"])
+        elif mlp:
+            r = mlp["router"]
+            n = r["experts"] + (r.get("identity") or 0)
+            t[p + "router"], t[p + "correction"] = lin(n, W), vec(n, 0.0, 0.1)
+            for x in range(r["experts"]):
+                gated(f"{p}e{x}.", mlp["expert"]["ff"])
+            if mlp.get("shared"):
+                gated(p + "shared.", mlp["shared"]["ff"])
+                t[p + "shared.sg"] = lin(1, W)
+        if config.get("token_side"):
+            n = config["token_side"]["dim"]
+            t[f"l{i}.side.gate"], t[f"l{i}.side.proj"], t[f"l{i}.side.norm"] = lin(n, W), lin(W, n), vec(W, 0.5)
+    if config.get("token_side"):
+        t["side.embed"] = torch.randn(V, len(config["layers"]) * config["token_side"]["dim"], generator=g).bfloat16()
+    t["final.norm"] = vec(W)
+    return t
