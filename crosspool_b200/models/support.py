@@ -45,7 +45,19 @@ _SANINEX_PROBE = {
                 "mixer": {"left": {"heads": 2, "kv_heads": 1, "dim": 16, "vdim": 16, "scale": 0.2, "softcap": 30.0},
                           "right": {"heads": 1, "dim": 16, "vdim": 16, "tau": 8.0}}}]}
 
+_KADAVIK_PROBE = {
+    "architecture": "Kadavik", "vocab": 256, "width": 64, "norm": {"eps": 1e-6}, "embedding": {"scale": 8.0}, "logit_scale": 1.0,
+    "token_side": {"dim": 16},
+    "layers": [{"type": "mlstm", "mixer": {"heads": 2, "dim": 16, "vdim": 16, "gate_cap": 15.0}, "mlp": {"kind": "dense", "ff": 128}},
+               {"type": "attention", "mlp": {"kind": "moe", "expert": {"ff": 32}, "shared": {"ff": 32},
+                                             "router": {"experts": 4, "identity": 1, "top": 2, "scale": 1.0}},
+                "mixer": {"heads": 2, "kv_heads": 1, "dim": 16, "vdim": 16, "scale": 0.25, "conv": 3, "rot": {"dims": 8, "base": 1e4},
+                          "mask": {"size": 32, "keep_first": 4}}}]}
+
 _LAYERED = {
+    "Kadavik": (_KADAVIK_PROBE, "per layer: matrix memory with exponential gates (mLSTM) or grouped-query attention (short convolutions, scaled "
+                                "rotary, sliding window with kept first tokens, gate per output, keys and values of another layer); norms before "
+                                "and behind the sublayers, a second token embedding per layer"),
     "Segirax": (_SEGIRAX_PROBE, "per layer: latent attention (rotate-half rotary, output gate) or decayed linear attention; dynamic tanh "
                                 "norms, gated fp32 residual"),
     "Saninex": (_SANINEX_PROBE, "per layer: gated delta rule (short convolutions) or, side by side, grouped-query attention (q/k RMSNorm, "
@@ -101,7 +113,9 @@ def _ffn_features(spec) -> str:
             if l.correction_bias_key:
                 out.append("selection bias")
             if l.num_shared_experts:
-                out.append("shared experts")
+                out.append("gated shared expert" if l.shared_scale_key else "shared experts")
+            if l.identity_experts:
+                out.append("identity experts")
             if l.routed_scaling_factor != 1.0 or "Deepseek" in spec.architecture or "Glm4" in spec.architecture:
                 out.append("routed scaling")
             if l.experts.gate_bias_key:

@@ -342,11 +342,8 @@ def grouped_prep(proj: torch.Tensor, q_norm: torch.Tensor | None, k_norm: torch.
 
 
 def _gate_elems(gate: torch.Tensor | None, heads: int, vdim: int) -> int:
-    """Whether a gate has one logit per output element (of a single-column head either reading is the same)."""
-    if gate is None or gate.shape[1] == heads:
-        return 0
-    assert gate.shape[1] == heads * vdim
-    return 1
+    """Whether a gate has one logit per output element: as many columns as the output, and more than heads."""
+    return int(gate is not None and vdim > 1 and gate.shape[1] == heads * vdim)
 
 
 def conv_rope(proj: torch.Tensor, conv_w: torch.Tensor | None, ring: torch.Tensor | None, rot: torch.Tensor | None, positions: torch.Tensor,
