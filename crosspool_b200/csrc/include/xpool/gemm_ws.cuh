@@ -442,6 +442,10 @@ __device__ __forceinline__ void epi_bar_sync() {
 // but the warp's own independent work: the 16 values are computed as 16
 // independent chains (fully unrolled, no early exit) and stored with
 // predicates, the epilogue kind is tested once per call.
+//
+// kWide: the forms with a cubic activation, a gating operand or fp32 features. They are a kernel of their own, because one
+// warp per scheduler feels every instruction that the common forms would have to skip.
+template <bool kWide>
 __device__ __forceinline__ void epilogue_store16(const Problem& p, int f, int fb, int n_first, int row_end,
                                                  const float* g, const float* u, int64_t out_off = 0) {
   const bool live = f < p.n_out;        // false in the padding rows of a last partial weight tile
@@ -453,7 +457,7 @@ __device__ __forceinline__ void epilogue_store16(const Problem& p, int f, int fb
     const float bias_u = (p.bias != nullptr && p.dual && live) ? p.bias[p.up_offset + fb] : 0.f;
     const float lim = p.gate_limit > 0.f ? p.gate_limit : 3.0e38f;
     const float a = p.act_alpha == 0.f ? 1.f : p.act_alpha;
-    if (p.act_cubic != 0.f) {
+    if (kWide && p.act_cubic != 0.f) {
 #pragma unroll
       for (int j = 0; j < 16; ++j) {
         const float gg = fminf(round_bf16(g[j] + bias), lim);
@@ -468,7 +472,7 @@ __device__ __forceinline__ void epilogue_store16(const Problem& p, int f, int fb
         v[j] = __fdividef(gg, 1.f + __expf(-a * gg)) * (uu + p.up_add);
       }
     }
-  } else if (p.epilogue == kEpiResidual || p.epilogue == kEpiGateMul) {
+  } else if (p.epilogue == kEpiResidual || (kWide && p.epilogue == kEpiGateMul)) {
     // sixteen loads in flight: no branch around any of them (rows and features that are not stored repeat ones that are)
     const __nv_bfloat16* r = reinterpret_cast<const __nv_bfloat16*>(p.resid) + static_cast<size_t>(n_first) * p.ld_resid + (live ? f : 0);
     const int last = valid > 0 ? valid - 1 : 0;
@@ -481,7 +485,7 @@ __device__ __forceinline__ void epilogue_store16(const Problem& p, int f, int fb
     for (int j = 0; j < 16; ++j) rr[j] = __uint_as_float(static_cast<uint32_t>(raw[j]) << 16);
 #pragma unroll
     for (int j = 0; j < 16; ++j) v[j] = round_bf16(g[j] + bias);
-    if (p.epilogue == kEpiResidual) {
+    if (!kWide || p.epilogue == kEpiResidual) {
 #pragma unroll
       for (int j = 0; j < 16; ++j) v[j] += rr[j];
     } else {
@@ -502,7 +506,7 @@ __device__ __forceinline__ void epilogue_store16(const Problem& p, int f, int fb
 #pragma unroll
     for (int j = 0; j < 16; ++j)
       if (j < valid) o[static_cast<size_t>(j) * p.ld_out] = v[j];
-  } else if (p.tail != nullptr && f >= p.tail_from) {
+  } else if (kWide && p.tail != nullptr && f >= p.tail_from) {
     float* o = p.tail + static_cast<int64_t>(n_first) * p.ld_tail + (f - p.tail_from);
 #pragma unroll
     for (int j = 0; j < 16; ++j)
@@ -516,6 +520,7 @@ __device__ __forceinline__ void epilogue_store16(const Problem& p, int f, int fb
 }
 
 // Runs on the 128 epilogue threads. `ew` is the warp's TMEM lane quarter.
+template <bool kWide>
 __device__ __forceinline__ bool epilogue_tile(const Problem& p, const TileCoord& c, Barriers* bar,
                                               PipeState& st, int nacc, int ew, int lane,
                                               uint64_t deadline) {
@@ -590,7 +595,7 @@ __device__ __forceinline__ bool epilogue_tile(const Problem& p, const TileCoord&
     if (p.splits == 1) {
 #pragma unroll
       for (int cc = 0; cc < kMaxBnF8 / 16; ++cc)
-        if (cc * 16 < p.bn && c.n0 + cc * 16 < c.row_end) epilogue_store16(p, f, fb, c.n0 + cc * 16, c.row_end, &acc[cc * 16], u);
+        if (cc * 16 < p.bn && c.n0 + cc * 16 < c.row_end) epilogue_store16<kWide>(p, f, fb, c.n0 + cc * 16, c.row_end, &acc[cc * 16], u);
     } else {
       float* ws = p.ws + (static_cast<size_t>(c.mn) * p.splits + c.split) * acc_cols * kTileM;
 #pragma unroll
@@ -619,7 +624,7 @@ __device__ __forceinline__ bool epilogue_tile(const Problem& p, const TileCoord&
         g[j] = __uint_as_float(ga[j]);
         u[j] = __uint_as_float(ua[j]);
       }
-      epilogue_store16(p, f, fb, c.n0 + col, c.row_end, g, u, c.out_off);
+      epilogue_store16<kWide>(p, f, fb, c.n0 + col, c.row_end, g, u, c.out_off);
       if (more) {
         sm100::tmem_ld_wait32(gb, ub);
         if (col + 32 < ncol) {
@@ -631,7 +636,7 @@ __device__ __forceinline__ bool epilogue_tile(const Problem& p, const TileCoord&
           g[j] = __uint_as_float(gb[j]);
           u[j] = __uint_as_float(ub[j]);
         }
-        epilogue_store16(p, f, fb, c.n0 + col + 16, c.row_end, g, u, c.out_off);
+        epilogue_store16<kWide>(p, f, fb, c.n0 + col + 16, c.row_end, g, u, c.out_off);
       }
     }
   } else {
@@ -689,7 +694,7 @@ __device__ __forceinline__ bool epilogue_tile(const Problem& p, const TileCoord&
             }
           }
         }
-        epilogue_store16(p, f, fb, c.n0 + col, c.row_end, g, u);
+        epilogue_store16<kWide>(p, f, fb, c.n0 + col, c.row_end, g, u);
       }
       if (ew == 0 && lane == 0) p.counters[c.mn] = 0;  // ready for the next call
     }

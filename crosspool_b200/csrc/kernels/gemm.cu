@@ -12,6 +12,7 @@ namespace gemm {
 
 // Body shared by the stream-launched kernel and the Lane kernel: every CTA loops
 // over the tiles assigned to it.
+template <bool kWide>
 __device__ __forceinline__ void run_tiles(const Problem& p, int nacc, int smem_budget, uint32_t* status) {
   extern __shared__ uint8_t smem_raw[];
   const int warp = threadIdx.x >> 5;
@@ -53,7 +54,7 @@ __device__ __forceinline__ void run_tiles(const Problem& p, int nacc, int smem_b
     const int ew = warp & 3;
     for (int t = blockIdx.x; t < ntiles; t += gridDim.x) {
       const uint64_t deadline = sm100::global_timer_ns() + sm100::kPipelineWaitNs;
-      if (!epilogue_tile(p, tile_coord(p, t), bar, st, nacc, ew, lane, deadline)) {
+      if (!epilogue_tile<kWide>(p, tile_coord(p, t), bar, st, nacc, ew, lane, deadline)) {
         record_status(status, kTimeoutEpilogue);
         break;
       }
@@ -65,13 +66,14 @@ __device__ __forceinline__ void run_tiles(const Problem& p, int nacc, int smem_b
 // At most 208 registers: 192 threads x 208 leave room on the SM for one decode-attention CTA of another
 // stream (128 threads x 192 registers), which is how decode GEMMs hide behind the co-located Instance's
 // attention.
+template <bool kWide>
 __global__ void __maxnreg__(208)
 gemm_ws_kernel(const __grid_constant__ CUtensorMap tmap_w,
                const __grid_constant__ CUtensorMap tmap_x, Problem p, int nacc, int smem_budget,
                uint32_t* status) {
   p.tmap_w = &tmap_w;
   p.tmap_x = &tmap_x;
-  run_tiles(p, nacc, smem_budget, status);
+  run_tiles<kWide>(p, nacc, smem_budget, status);
 }
 
 // Lane form: the problem is assembled on the device from the descriptor table
@@ -205,7 +207,7 @@ gemm_lane_kernel(const lane::InstanceSlot* slots, const lane::LaneCur* cur, int 
   p.ld_resid = p.ld_out;
   const int nacc = p.bn * (p.dual ? 2 : 1) * 2 <= 512 ? 2 : 1;
   if (threadIdx.x == 0 && (phase == 0 || phase == 2 || phase == 3)) sm100::fence_proxy_async();  // payload arrived through peer stores
-  run_tiles(p, nacc, smem_budget, status);
+  run_tiles<false>(p, nacc, smem_budget, status);
 }
 
 // Estimated duration (microseconds) of one launch for a tile width and split-K factor, fitted to
@@ -413,14 +415,14 @@ extern "C" int xp_gemm(const XpGemmArgs* a) {
   int dev = 0;
   cudaGetDevice(&dev);
   if (dev < 64 && !attr_set[dev]) {
-    cudaError_t e = cudaFuncSetAttribute(gemm::gemm_ws_kernel,
-                                         cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
-    if (e != cudaSuccess) return -30;
+    if (cudaFuncSetAttribute(gemm::gemm_ws_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024) != cudaSuccess ||
+        cudaFuncSetAttribute(gemm::gemm_ws_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024) != cudaSuccess)
+      return -30;
     attr_set[dev] = true;
   }
-  gemm::gemm_ws_kernel<<<plan.grid, gemm::kThreads, plan.smem_bytes,
-                         reinterpret_cast<cudaStream_t>(a->stream)>>>(
-      tw, tx, p, plan.nacc, plan.smem_budget, a->status);
+  const bool wide = p.act_cubic != 0.f || p.epilogue == gemm::kEpiGateMul || p.tail != nullptr;
+  auto kernel = wide ? gemm::gemm_ws_kernel<true> : gemm::gemm_ws_kernel<false>;
+  kernel<<<plan.grid, gemm::kThreads, plan.smem_bytes, reinterpret_cast<cudaStream_t>(a->stream)>>>(tw, tx, p, plan.nacc, plan.smem_budget, a->status);
   cudaError_t e = cudaGetLastError();
   return e == cudaSuccess ? 0 : -100 - static_cast<int>(e);
 }
