@@ -70,7 +70,7 @@ def kernel_table(classic: ModelConfig, cfg: ModelConfig, timer, context: int, ch
     kc, vc, q = rnd(batch * blocks, 64, hk, d), rnd(batch * blocks, 64, hk, d), rnd(batch, hk, G, d)
     o, gate, lens = torch.empty(batch, no, dtype=bf, device=dev), rnd(T, no), i32([context] * batch)
     seen = att.visible(context)
-    sp, ck = A.decode_plan(batch, hk, min(context, seen + 32))
+    sp, ck = A.window_plan(batch, hk, seen + 32)
     ws = torch.empty(max(1, batch * hq * sp * (d + 2)), device=dev)
     kw = dict(heads=hq, vdim=d, scale=att.scale, window=WINDOW, keep_first=KEEP)
     add(f"windowed decode b{batch}", lambda: M.grouped_decode(q, kc, vc, o, table, pos, slots, dim=d, gate=gate[:batch], num_splits=sp, chunk_tokens=ck,

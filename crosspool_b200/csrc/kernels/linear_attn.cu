@@ -453,10 +453,18 @@ linear_scan_kernel(XpLinearAttnArgs a) {
   const float p64 = a.decay_pow[h * (kChunk + 1) + kChunk];
   float f = 1.f;                                     // decay over one whole segment
   for (int c = 0; c < a.seg_tokens / kChunk; ++c) f *= p64;
-  for (int s = 0; s * a.seg_tokens < total; ++s) {
-    const float add = (s + 1) * a.seg_tokens < total ? mid[s * state_elems] : 0.f;   // the last segment adds to nobody
-    mid[s * state_elems] = x;
-    x = fmaf(f, x, add);
+  const int segs = (total + a.seg_tokens - 1) / a.seg_tokens;
+  constexpr int kAhead = 8;                          // loads in flight before the first store
+  for (int s0 = 0; s0 < segs; s0 += kAhead) {
+    float add[kAhead];
+#pragma unroll
+    for (int u = 0; u < kAhead; ++u) add[u] = s0 + u + 1 < segs ? mid[(s0 + u) * state_elems] : 0.f;   // the last segment adds to nobody
+#pragma unroll
+    for (int u = 0; u < kAhead; ++u) {
+      if (s0 + u >= segs) break;
+      mid[(s0 + u) * state_elems] = x;
+      x = fmaf(f, x, add[u]);
+    }
   }
 }
 

@@ -16,6 +16,7 @@
 #include "xpool/api.h"
 #include "xpool/elem.cuh"
 #include "xpool/lane.cuh"
+#include "xpool/recurrence.cuh"
 #include "xpool/sm100.cuh"
 
 namespace xpool {
@@ -260,34 +261,51 @@ combine_kernel(const __nv_bfloat16* __restrict__ y, const int* __restrict__ rout
   combine_token(y, route_pos, weights, out, top_k, hidden, ld_out, blockIdx.x);
 }
 
-// Weighted experts, identity experts and the gated shared expert of one token.
+// Weighted experts, identity experts and the gated shared expert of one token: a list of rows and weights, then their sum with
+// kAhead rows in flight.
+constexpr int kMixThreads = 256;
+
 template <typename T, int N>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(kMixThreads)
 mix_kernel(XpMoeMixArgs a) {
-  const int t = blockIdx.x;
-  const T* x = reinterpret_cast<const T*>(a.x) + static_cast<size_t>(t) * a.ld_x;
-  const T* sh = a.shared != nullptr ? reinterpret_cast<const T*>(a.shared) + static_cast<size_t>(t) * a.ld_shared : nullptr;
-  const float sg = sh != nullptr ? elem::sigmoid(a.shared_gate[static_cast<size_t>(t) * a.ld_gate]) : 0.f;
+  constexpr int kAhead = 5;
+  __shared__ const T* rows[33 + kAhead];
+  __shared__ float weights[33 + kAhead];
+  const int t = blockIdx.x, n = a.top_k + (a.shared != nullptr ? 1 : 0), k = threadIdx.x;
+  if (k < n + kAhead) {                              // what is missing counts the token's own row with weight zero: no load is skipped
+    const T* row = reinterpret_cast<const T*>(a.x) + static_cast<size_t>(t) * a.ld_x;
+    float w = 0.f;
+    if (k < a.top_k) {
+      const int pos = a.route_pos[t * a.top_k + k], id = a.topk_ids[t * a.top_k + k];
+      if (pos >= 0) row = reinterpret_cast<const T*>(a.y) + static_cast<size_t>(pos) * a.ld_y;
+      if (pos >= 0 || id >= a.experts) w = a.weights[t * a.top_k + k];
+    } else if (k < n) {
+      row = reinterpret_cast<const T*>(a.shared) + static_cast<size_t>(t) * a.ld_shared;
+      w = elem::sigmoid(a.shared_gate[static_cast<size_t>(t) * a.ld_gate]);
+    }
+    rows[k] = row, weights[k] = w;
+  }
+  __syncthreads();
   T* out = reinterpret_cast<T*>(a.out) + static_cast<size_t>(t) * a.ld_out;
-  for (int c = threadIdx.x * N; c < a.hidden; c += 128 * N) {
-    float acc[N], v[N];
+  for (int c = threadIdx.x * N; c < a.hidden; c += kMixThreads * N) {
+    float acc[N];
 #pragma unroll
     for (int j = 0; j < N; ++j) acc[j] = 0.f;
-    for (int k = 0; k < a.top_k; ++k) {
-      const int pos = a.route_pos[t * a.top_k + k];
-      const float w = a.weights[t * a.top_k + k];
-      if (pos >= 0) elem::ldv<N>(reinterpret_cast<const T*>(a.y) + static_cast<size_t>(pos) * a.ld_y + c, v);
-      else if (a.topk_ids[t * a.top_k + k] >= a.experts) elem::ldv<N>(x + c, v);
-      else continue;
+    for (int k0 = 0; k0 < n; k0 += kAhead) {
+      T raw[kAhead][N];
 #pragma unroll
-      for (int j = 0; j < N; ++j) acc[j] = fmaf(w, v[j], acc[j]);
-    }
-    if (sh != nullptr) {
-      elem::ldv<N>(sh + c, v);
+      for (int u = 0; u < kAhead; ++u) recur::ldr<N>(rows[k0 + u] + c, raw[u]);
 #pragma unroll
-      for (int j = 0; j < N; ++j) acc[j] = fmaf(sg, v[j], acc[j]);
+      for (int u = 0; u < kAhead; ++u) {
+        const float w = weights[k0 + u];
+#pragma unroll
+        for (int j = 0; j < N; ++j) acc[j] = fmaf(w, elem::ld(&raw[u][j]), acc[j]);
+      }
     }
-    elem::stv<N>(out + c, acc);
+    T res[N];
+#pragma unroll
+    for (int j = 0; j < N; ++j) elem::st(&res[j], acc[j]);
+    recur::stx<N>(out + c, res);
   }
 }
 
@@ -354,6 +372,7 @@ __device__ __forceinline__ int block_exclusive_scan(int v, int* warp_sums, int* 
 __global__ void __launch_bounds__(1024)
 topk_route_kernel(XpRouterArgs a, XpRouteArgs r) {
   __shared__ int hist[1024], cursor[1024], warp_sums[32];
+  __shared__ int4 seg[256];                          // per expert: first row, rows, first tile of either table
   const int e = threadIdx.x, lo = r.expert_lo, n_local = r.expert_hi - r.expert_lo;
   hist[e] = 0;
   for (int row = e >> 5; row < a.rows; row += 32) router_topk_row(a, row, e & 31);
@@ -373,7 +392,7 @@ topk_route_kernel(XpRouterArgs a, XpRouteArgs r) {
   const int t_dn = block_exclusive_scan(r.tm_down * b_dn, warp_sums, &total_dn);
   cursor[e] = off;
   if (e <= n_local) r.offsets[e] = off;
-  if (e < n_local) r.counts[e] = c;
+  if (e < n_local) r.counts[e] = c, seg[e] = make_int4(off, c, t_gu, t_dn);
   if (e == 0) *r.n_tiles_gateup = total_gu, *r.n_tiles_down = total_dn;
   __syncthreads();
   for (int i = e; i < n_routes; i += 1024) {
@@ -384,13 +403,13 @@ topk_route_kernel(XpRouterArgs a, XpRouteArgs r) {
       r.route_pos[i] = pos;
     }
   }
-  if (e < n_local) {
-    int idx = t_gu;
-    for (int m = 0; m < r.tm_gateup; ++m)
-      for (int p = off; p < off + c; p += r.bn_gateup) reinterpret_cast<int4*>(r.tiles_gateup)[idx++] = make_int4(e, m * 128, p, off + c);
-    idx = t_dn;
-    for (int m = 0; m < r.tm_down; ++m)
-      for (int p = off; p < off + c; p += r.bn_down) reinterpret_cast<int4*>(r.tiles_down)[idx++] = make_int4(e, m * 128, p, off + c);
+  for (int x = e >> 5; x < n_local; x += 32) {       // a warp per expert, a lane per tile
+    const int4 s = seg[x];
+    const int ng = (s.y + r.bn_gateup - 1) / r.bn_gateup, nd = (s.y + r.bn_down - 1) / r.bn_down;
+    for (int i = e & 31; i < r.tm_gateup * ng; i += 32)
+      reinterpret_cast<int4*>(r.tiles_gateup)[s.z + i] = make_int4(x, i / ng * 128, s.x + i % ng * r.bn_gateup, s.x + s.y);
+    for (int i = e & 31; i < r.tm_down * nd; i += 32)
+      reinterpret_cast<int4*>(r.tiles_down)[s.w + i] = make_int4(x, i / nd * 128, s.x + i % nd * r.bn_down, s.x + s.y);
   }
 }
 
@@ -580,7 +599,7 @@ extern "C" int xp_moe_route(const XpRouteArgs* a, void* stream) {
 extern "C" int xp_moe_topk_route(const XpRouterArgs* a, const XpRouteArgs* r, void* stream) {
   if (a->rows <= 0) return 0;
   const int n_local = r->expert_hi - r->expert_lo;
-  if (a->num_experts > 32 * kMaxPerLane || a->top_k > 32 || a->top_k > a->num_experts || n_local < 1 || n_local > 1023 || a->rows > 128 ||
+  if (a->num_experts > 32 * kMaxPerLane || a->top_k > 32 || a->top_k > a->num_experts || n_local < 1 || n_local > 256 || a->rows > 128 ||
       a->rows != r->rows || a->top_k != r->top_k || a->topk_ids != r->topk_ids)
     return -10;
   topk_route_kernel<<<1, 1024, 0, reinterpret_cast<cudaStream_t>(stream)>>>(*a, *r);
@@ -589,17 +608,17 @@ extern "C" int xp_moe_topk_route(const XpRouterArgs* a, const XpRouteArgs* r, vo
 
 extern "C" int xp_moe_mix(const XpMoeMixArgs* a, void* stream) {
   if (a->rows <= 0) return 0;
-  if (a->hidden <= 0 || a->top_k <= 0 || (a->shared != nullptr && a->shared_gate == nullptr)) return -10;
-  const int eb = a->f32 ? 4 : 2;
-  auto fits = [&](const void* p, int ld) { return p == nullptr || (reinterpret_cast<uintptr_t>(p) % (4 * eb) == 0 && ld % 4 == 0); };
-  const bool v = a->hidden % 4 == 0 && fits(a->y, a->ld_y) && fits(a->x, a->ld_x) && fits(a->shared, a->ld_shared) && fits(a->out, a->ld_out);
+  if (a->hidden <= 0 || a->top_k <= 0 || a->top_k > 32 || (a->shared != nullptr && a->shared_gate == nullptr)) return -10;
+  const int n = a->f32 ? 4 : 8;                      // elements of 16 bytes
+  auto fits = [&](const void* p, int ld) { return p == nullptr || (reinterpret_cast<uintptr_t>(p) % 16 == 0 && ld % n == 0); };
+  const bool v = a->hidden % n == 0 && fits(a->y, a->ld_y) && fits(a->x, a->ld_x) && fits(a->shared, a->ld_shared) && fits(a->out, a->ld_out);
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   if (a->f32) {
-    if (v) mix_kernel<float, 4><<<a->rows, 128, 0, s>>>(*a);
-    else mix_kernel<float, 1><<<a->rows, 128, 0, s>>>(*a);
+    if (v) mix_kernel<float, 4><<<a->rows, kMixThreads, 0, s>>>(*a);
+    else mix_kernel<float, 1><<<a->rows, kMixThreads, 0, s>>>(*a);
   } else {
-    if (v) mix_kernel<__nv_bfloat16, 4><<<a->rows, 128, 0, s>>>(*a);
-    else mix_kernel<__nv_bfloat16, 1><<<a->rows, 128, 0, s>>>(*a);
+    if (v) mix_kernel<__nv_bfloat16, 8><<<a->rows, kMixThreads, 0, s>>>(*a);
+    else mix_kernel<__nv_bfloat16, 1><<<a->rows, kMixThreads, 0, s>>>(*a);
   }
   return last_error();
 }

@@ -27,7 +27,7 @@ from ..models.config import (DeltaMixer, GatedLinearMixer, GroupedMixer, LatentM
 from ..models.layered import LayeredLayerWeights, rotary_table
 from ..ops import gemm
 from ..ops import mixers as M
-from ..ops.attention import decode_plan, embedding
+from ..ops.attention import decode_plan, embedding, window_plan
 
 # Portions of at most this many tokens run as single rows (latent attention: in the absorbed form, expanding the whole context
 # costs more).
@@ -116,7 +116,7 @@ class LayeredForward:
         self.rot_tables = {rot: rotary_table(rot, engine.ecfg.max_seq_len, dev) for rot in {m.rot for m in grp if m.rot is not None}}
         if grp:
             self.q_grp = buf(cap * max(m.kv_heads * M.group_pad(m.heads, m.kv_heads) * m.row_shapes[0][1] for m in grp))
-            need = max(b * m.heads * decode_plan(b, m.kv_heads, engine.ecfg.max_seq_len)[0] * (m.row_shapes[1][1] + 2)
+            need = max(b * m.heads * self._splits(m, b, engine.ecfg.max_seq_len)[0] * (m.row_shapes[1][1] + 2)
                        for b in engine._buckets for m in grp)
             self.grp_ws = buf(max(need, 1 << 20), torch.float32)
         if gla:
@@ -198,6 +198,11 @@ class LayeredForward:
         return (self.dtype == torch.bfloat16 and shape is not None and m.heads // m.kv_heads <= 16 and page & (page - 1) == 0
                 and page >= (16 if shape[0] == shape[1] else 64))
 
+    @staticmethod
+    def _splits(m: GroupedMixer, rows: int, max_len: int) -> tuple[int, int]:
+        seen = m.visible(max_len)
+        return window_plan(rows, m.kv_heads, seen + 32) if seen < max_len else decode_plan(rows, m.kv_heads, max_len)   # edges lie inside tiles
+
     def _grouped(self, l: int, lw: LayeredLayerWeights, m: GroupedMixer, proj: torch.Tensor, out: torch.Tensor, b: RowBatch) -> None:
         rows, o, kv = b.rows, lw.offs, self.e.kv
         k, v = kv.k[l], kv.v[l]
@@ -216,7 +221,7 @@ class LayeredForward:
             return
         n = b.n_abs
         if n:
-            splits, chunk = decode_plan(n, m.kv_heads, min(b.max_len, m.visible(b.max_len) + 32))   # a window's edges lie inside tiles
+            splits, chunk = self._splits(m, n, b.max_len)
             if splits > 1 and n * m.heads * splits * (v.shape[3] + 2) > self.grp_ws.numel():
                 splits, chunk = 1, 0
             M.grouped_decode(q[:n], k, v, out[:n], b.table, b.positions, b.slots, dim=m.dim, gate=gate, row_seq=b.row_seq, num_splits=splits,

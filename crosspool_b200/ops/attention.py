@@ -66,6 +66,14 @@ def decode_plan(batch: int, kv_heads: int, max_len: int) -> tuple[int, int]:
     return (max_len + chunk - 1) // chunk, chunk
 
 
+def window_plan(batch: int, kv_heads: int, seen: int) -> tuple[int, int]:
+    """(num_splits, chunk_tokens) for rows that see a window of ``seen`` tokens at most (first tokens and the edges of 16-token
+    tiles included): slices of equal length, and only while (row, head) pairs leave SMs idle. Measured on B200 with 8 KV heads
+    and 1104 tokens: one slice from 64 rows on, four for 1 and 8 rows."""
+    splits = min(max(1, 256 // (batch * kv_heads)), (seen + 287) // 288)
+    return (splits, (seen + splits * 16 - 1) // (splits * 16) * 16) if splits > 1 else (1, 0)
+
+
 def paged_decode(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, block_table: torch.Tensor,
                  seq_lens: torch.Tensor, *, out: torch.Tensor | None = None, num_splits: int = 0,
                  ws: torch.Tensor | None = None, scale: float | None = None, max_len: int | None = None,
