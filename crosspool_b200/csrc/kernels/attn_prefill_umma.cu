@@ -163,14 +163,14 @@ prefill_attn_umma_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gri
   const int kv_end = ctx + min(q_len, q0 + 2 * np);            // causal bound of the CTA
   // tiles [0, head) and those from head + skip on are read
   int head = 0, skip = 0;
-  if (a.window > 0 && ctx + q0 >= a.window) {
+  if (kPair && a.window > 0 && ctx + q0 >= a.window) {
     const int lo_tile = (ctx + q0 - a.window + 1) / kBN;       // of the first query's window
     head = min((a.keep_first + kBN - 1) / kBN, lo_tile);
     skip = lo_tile - head;
   }
   const int n_tiles = (kv_end + kBN - 1) / kBN - skip;
   const int n_a = min(n_tiles, (ctx + min(q_len, q0 + np) + kBN - 1) / kBN - skip);   // tiles that tile A can see
-  auto tile_token = [&](int t) { return (t < head ? t : t + skip) * kBN; };           // first token of a tile
+  auto tile_token = [&](int t) { return (kPair && t >= head ? t + skip : t) * kBN; }; // first token of a tile
 
   if (threadIdx.x == 0) {
     sm100::mbar_init(&bars.q_full, 1);
@@ -331,7 +331,7 @@ prefill_attn_umma_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gri
     const bool tile_on = x == 0 || act_b;
     const int my_tiles = x == 0 ? n_a : n_tiles;
     const int limit = min(ctx + pos, kv_end - 1);     // last visible cache position of this row
-    const int win_lo = a.window > 0 ? ctx + pos - a.window + 1 : 0;   // first of its window
+    const int win_lo = kPair && a.window > 0 ? ctx + pos - a.window + 1 : 0;   // first of its window
     const uint32_t lane_off = static_cast<uint32_t>((warp & 3) * 32) << 16;
     const uint32_t o_t = tmem + lane_off + kOCol + static_cast<uint32_t>(x * DV);
     const uint32_t p_row = p_s + x * kPTile + row * 128;
@@ -365,7 +365,7 @@ prefill_attn_umma_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gri
             if (j >= nvis) sv[j] = 0xff800000u;       // -inf: selected, never computed with (the slot may hold NaN)
         }
         const int below = win_lo - tok0, kept = a.keep_first - tok0;   // tokens [kept, below) of the tile are behind the window
-        if (below > 0 && kept < kBN) {
+        if (kPair && below > 0 && kept < kBN) {
 #pragma unroll
           for (int j = 0; j < kBN; ++j)
             if (j >= kept && j < below) sv[j] = 0xff800000u;
@@ -461,42 +461,68 @@ prefill_attn_umma_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gri
         __syncwarp();
         if (lane == 0) sm100::mbar_arrive(&bars.p_full[x]);
       }
+      // a gate per element: the row's logits are requested before the wait for the last product
+      uint4 gate_row[DV / 8];
+      if (kPair && a.gate_elems) {
+        const __nv_bfloat16* ge = reinterpret_cast<const __nv_bfloat16*>(a.gate) + static_cast<size_t>(q_base + (stored ? pos : 0)) * a.ld_gate +
+                                  (stored ? hq : 0) * a.v_valid;
+#pragma unroll
+        for (int i = 0; i < DV / 8; ++i)
+          asm volatile("ld.global.nc.v4.u32 {%0, %1, %2, %3}, [%4];"
+                       : "=r"(gate_row[i].x), "=r"(gate_row[i].y), "=r"(gate_row[i].z), "=r"(gate_row[i].w)
+                       : "l"(ge + min(i * 8, a.v_valid - 8)));
+      }
       if (ok && my_tiles > 0) ok = __all_sync(0xffffffffu, wait_bar(&bars.pv_done[x], (my_tiles - 1) & 1, &bars, 11));
       if (ok) {
         sm100::tc_fence_after_sync();
         float inv = l > 0.f ? 1.f / l : 0.f;
-        const __nv_bfloat16* ge = nullptr;                // one gate per element
-        if (a.gate_elems && stored)
-          ge = reinterpret_cast<const __nv_bfloat16*>(a.gate) + static_cast<size_t>(q_base + pos) * a.ld_gate + hq * a.v_valid;
-        else if (a.gate != nullptr && stored)
+        if (a.gate != nullptr && !a.gate_elems && stored)
           inv *= 1.f / (1.f + expf(-__bfloat162float(reinterpret_cast<const __nv_bfloat16*>(a.gate)[static_cast<size_t>(q_base + pos) * a.ld_gate + hq])));
         const int v_valid = a.v_valid;                    // stored columns of a head (a multiple of 8)
         __nv_bfloat16* og = reinterpret_cast<__nv_bfloat16*>(a.out) + static_cast<size_t>(q_base + pos) * a.ld_out + hq * v_valid;
-#pragma unroll 1
-        for (int c = 0; c < DV; c += 32) {
-          uint32_t ov[32];
-          sm100::tmem_ld32_issue(o_t + c, ov);
-          sm100::tmem_ld_wait_all(ov);
-          if (stored) {
+        if (kPair && a.gate_elems) {
+#pragma unroll
+          for (int c = 0; c < DV; c += 32) {
+            uint32_t ov[32];
+            sm100::tmem_ld32_issue(o_t + c, ov);
+            sm100::tmem_ld_wait_all(ov);
 #pragma unroll
             for (int j = 0; j < 32; j += 8) {
-              if (c + j >= v_valid) break;
-              if (ge != nullptr) {
-                const uint4 gr = *reinterpret_cast<const uint4*>(ge + c + j);
-                const uint32_t gw[4] = {gr.x, gr.y, gr.z, gr.w};
+              const uint4 gr = gate_row[(c + j) / 8];
+              const uint32_t gw[4] = {gr.x, gr.y, gr.z, gr.w};
 #pragma unroll
-                for (int i = 0; i < 4; ++i) {
-                  const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&gw[i]));
-                  ov[j + 2 * i] = __float_as_uint(__uint_as_float(ov[j + 2 * i]) * (1.f / (1.f + __expf(-f.x))));
-                  ov[j + 2 * i + 1] = __float_as_uint(__uint_as_float(ov[j + 2 * i + 1]) * (1.f / (1.f + __expf(-f.y))));
-                }
+              for (int i = 0; i < 4; ++i) {
+                const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&gw[i]));
+                ov[j + 2 * i] = __float_as_uint(__fdividef(__uint_as_float(ov[j + 2 * i]), 1.f + __expf(-f.x)));
+                ov[j + 2 * i + 1] = __float_as_uint(__fdividef(__uint_as_float(ov[j + 2 * i + 1]), 1.f + __expf(-f.y)));
               }
-              uint4 v;
-              v.x = pack2(__uint_as_float(ov[j]) * inv, __uint_as_float(ov[j + 1]) * inv);
-              v.y = pack2(__uint_as_float(ov[j + 2]) * inv, __uint_as_float(ov[j + 3]) * inv);
-              v.z = pack2(__uint_as_float(ov[j + 4]) * inv, __uint_as_float(ov[j + 5]) * inv);
-              v.w = pack2(__uint_as_float(ov[j + 6]) * inv, __uint_as_float(ov[j + 7]) * inv);
-              *reinterpret_cast<uint4*>(og + c + j) = v;
+              if (stored && c + j < v_valid) {
+                uint4 v;
+                v.x = pack2(__uint_as_float(ov[j]) * inv, __uint_as_float(ov[j + 1]) * inv);
+                v.y = pack2(__uint_as_float(ov[j + 2]) * inv, __uint_as_float(ov[j + 3]) * inv);
+                v.z = pack2(__uint_as_float(ov[j + 4]) * inv, __uint_as_float(ov[j + 5]) * inv);
+                v.w = pack2(__uint_as_float(ov[j + 6]) * inv, __uint_as_float(ov[j + 7]) * inv);
+                *reinterpret_cast<uint4*>(og + c + j) = v;
+              }
+            }
+          }
+        } else {
+#pragma unroll 1
+          for (int c = 0; c < DV; c += 32) {
+            uint32_t ov[32];
+            sm100::tmem_ld32_issue(o_t + c, ov);
+            sm100::tmem_ld_wait_all(ov);
+            if (stored) {
+#pragma unroll
+              for (int j = 0; j < 32; j += 8) {
+                if (c + j >= v_valid) break;
+                uint4 v;
+                v.x = pack2(__uint_as_float(ov[j]) * inv, __uint_as_float(ov[j + 1]) * inv);
+                v.y = pack2(__uint_as_float(ov[j + 2]) * inv, __uint_as_float(ov[j + 3]) * inv);
+                v.z = pack2(__uint_as_float(ov[j + 4]) * inv, __uint_as_float(ov[j + 5]) * inv);
+                v.w = pack2(__uint_as_float(ov[j + 6]) * inv, __uint_as_float(ov[j + 7]) * inv);
+                *reinterpret_cast<uint4*>(og + c + j) = v;
+              }
             }
           }
         }
@@ -588,7 +614,7 @@ extern "C" int xp_prefill_attn_umma(const XpPrefillAttnArgs* a, void* stream) {
     if (a->head_dim == 192 && dv == 128) return launch_pair<192, 128>(*a, G, s);
     return 1;
   }
-  if (dv != a->head_dim || a->softcap > 0.f) return 1;
+  if (dv != a->head_dim || a->softcap > 0.f || a->gate_elems || a->window > 0) return 1;   // the forms of layered decoders only
   if (a->head_dim == 128) return ts ? launch<128, 128, true, false>(*a, G, s) : launch<128, 128, false, false>(*a, G, s);
   if (a->head_dim == 64) return ts ? launch<64, 64, true, false>(*a, G, s) : launch<64, 64, false, false>(*a, G, s);
   return 1;
