@@ -26,7 +26,7 @@ when an SLO is missed or the correctness gate (logits against an oracle engine) 
 broadcast / reduce, cuBLAS GEMMs, unfused SwiGLU). ``--impl reference`` reports why the reference itself cannot
 run here. ``--decode-only`` runs the steady-state decode replay benchmark instead (every Instance at a full
 running batch, no arrivals), a kernel-level figure. ``--layered`` measures layered decoders (per-layer mixers:
-latent attention, decayed linear attention) beside the closest classic model of equal size.
+latent and windowed attention, recurrences) beside the closest classic model of equal size.
 """
 
 from __future__ import annotations

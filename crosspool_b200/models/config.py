@@ -625,7 +625,7 @@ def saninex_config(cfg: dict[str, Any], name: str = "") -> ModelConfig:
 
 
 def _rotary(r: dict[str, Any] | None, dim: int) -> RotarySpec | None:
-    if not r:
+    if not r or not int(r["dims"]):
         return None
     sc = r.get("scaling")
     rot = RotarySpec(int(r["dims"]), float(r["base"]),
@@ -655,7 +655,7 @@ def _kadavik_mlp(mixer: Mixer, mlp: dict[str, Any] | None) -> LayerSpec:
     if mlp["kind"] != "moe":
         raise ValueError(f"unsupported feed-forward kind {mlp['kind']!r}")
     r, shared = mlp["router"], mlp.get("shared")
-    moe = MoeSpec(int(r["experts"]), int(r["top"]), int(mlp["expert"]["ff"]), int(r.get("identity") or 0), float(r["scale"]),
+    moe = MoeSpec(int(r["experts"]), int(r["top"]), int(mlp["expert"]["ff"]), int(r.get("identity") or 0), float(r.get("scale", 1.0)),
                   int(shared["ff"]) if shared else 0)
     if not 0 < moe.top <= min(moe.routed, 32) or moe.routed > 256 or moe.experts < 1:
         raise ValueError(f"a router of {moe.routed} outputs that takes {moe.top} is not supported (at most 32 of 256)")
