@@ -8,7 +8,7 @@
 #include <stddef.h>
 #include <stdint.h>
 
-#define XP_ABI_VERSION 24
+#define XP_ABI_VERSION 25
 
 #ifdef __cplusplus
 extern "C" {
@@ -31,7 +31,8 @@ typedef struct XpGemmArgs {
   int k;               /* row pitches are multiples of 16 bytes (multiple of 64 elements in the forms above) */
   int rows;
   int ldw, ldx, ld_out, ld_resid; /* element strides; 0 = dense */
-  int epilogue;        /* 0 store bf16, 1 swiglu (dual), 2 residual add, 3 store fp32, 4 act(value) * resid */
+  int epilogue;        /* 0 store bf16, 1 swiglu (dual), 2 residual add, 3 store fp32, 4 act(value) * resid,
+                          5 value * sigmoid(resid) (batched: resid is laid out like out, with its own pitch) */
   int dual;
   int up_offset;       /* first weight row of the up projection */
   int splits;          /* 0 = choose */
@@ -59,6 +60,7 @@ typedef struct XpGemmArgs {
   int tail_from;       /* epilogue 0: features from here on are stored to tail in fp32 instead, [rows, ld_tail] */
   float* tail;
   int ld_tail;
+  int relu2;           /* epilogue 0: values are stored as max(value, 0)^2 */
 } XpGemmArgs;
 
 typedef struct XpGemmPlan {
@@ -211,7 +213,9 @@ typedef struct XpRouterArgs {
   int* topk_ids;                /* [rows, top_k] */
   float* topk_weights;          /* [rows, top_k] */
   int rows, num_experts, top_k, ld_logits;
-  int logits_fp32, sigmoid, renormalize, round_weights_bf16;
+  int logits_fp32;
+  int sigmoid;                  /* scores: 0 softmax over all experts, 1 sigmoid, 2 softmax over the chosen logits (no correction) */
+  int renormalize, round_weights_bf16;
   float scale;
 } XpRouterArgs;
 
@@ -230,12 +234,12 @@ typedef struct XpRouteArgs {
 } XpRouteArgs;
 
 /* out[t] = sum over k (in order) of weights[t, k] * (y[route_pos[t, k]], or x[t] where topk_ids[t, k] >= experts)
- *          + sigmoid(shared_gate[t]) * shared[t] */
+ *          + sigmoid(shared_gate[t]) * shared[t] (without shared_gate: + shared[t]) */
 typedef struct XpMoeMixArgs {
   const void* y;                /* [routes, ld_y] expert outputs in route order */
   const void* x;                /* [rows, ld_x] the layer's input */
   const void* shared;           /* optional [rows, ld_shared] */
-  const float* shared_gate;     /* logits, row t at t * ld_gate */
+  const float* shared_gate;     /* optional logits, row t at t * ld_gate */
   const int* topk_ids;          /* [rows, top_k] */
   const int* route_pos;         /* [rows, top_k], -1: not an expert */
   const float* weights;         /* [rows, top_k] */
@@ -314,6 +318,14 @@ typedef struct XpDecodeRowsArgs {
   int window;                 /* > 0: a row sees the last `window` of its tokens, and the first `keep_first` */
   int keep_first;
   int gate_elems;             /* the gate has one logit per output element: [rows, heads * v_valid] */
+  const float* sink;          /* optional [q_heads]: exp(sink) joins the softmax's sum and has no value */
+  /* sigmoid_bias [q_heads]: no softmax, a token's weight is sigmoid(score + bias). Beside its window a row may then see one key
+   * and value per block of `pool` tokens that lies wholly behind the window: block b is row b % pool_page of page
+   * block_table[b / pool_page] of k_pool, v_pool ([pages, pool_page, kv_heads, width], pool_page a power of two >= 8). */
+  const float* sigmoid_bias;
+  const void* k_pool;
+  const void* v_pool;
+  int pool, pool_page;
 } XpDecodeRowsArgs;
 
 typedef struct XpPrefillAttnArgs {
@@ -338,7 +350,8 @@ typedef struct XpPrefillAttnArgs {
   int v_dim;                  /* value width; 0: head_dim */
   int v_valid;                /* columns of a head stored to out (multiple of 8); 0: v_dim */
   int ld_out;                 /* elements of an out row (multiple of 8); 0: q_heads * v_valid */
-  const int* seq_starts;      /* [num_seqs] first K/V row of each sequence when its rows lie densely (no block table) */
+  const int* seq_starts;      /* [num_seqs] first K/V row of each sequence when its rows lie densely (no block table); with a
+                                 window the rows begin at the 64-token boundary at or before the first query's window */
   const void* gate;           /* optional bf16 [total_q, ld_gate] logits: head h's output is multiplied by sigmoid */
   int ld_gate;
   int p_pair;                 /* probabilities as a bf16 pair in the second product */
@@ -347,6 +360,11 @@ typedef struct XpPrefillAttnArgs {
   int window;                 /* > 0: a token sees the `window` tokens that end with itself, and the first `keep_first` */
   int keep_first;
   int gate_elems;             /* the gate has one logit per output element: [rows, heads * v_valid], rows of 16-byte units */
+  const float* sink;          /* as in XpDecodeRowsArgs */
+  const float* sigmoid_bias;
+  const void* k_pool;
+  const void* v_pool;
+  int pool, pool_page;
 } XpPrefillAttnArgs;
 
 int xp_rope_kv(const XpRopeArgs* a, void* stream);

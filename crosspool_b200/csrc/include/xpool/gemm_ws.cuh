@@ -39,6 +39,7 @@ enum Epilogue : int {
   kEpiResidual = 2,  // out = round(acc) + resid
   kEpiStoreF32 = 3,  // fp32 out = acc (+ bias)
   kEpiGateMul = 4,   // out = act(round(acc)) * resid
+  kEpiSigmoid = 5,   // out = acc * sigmoid(resid)
 };
 
 enum Status : uint32_t {
@@ -102,6 +103,7 @@ struct Problem {
   float* tail;             // kEpiStore: features from tail_from on go here in fp32, row r at r * ld_tail
   int tail_from;
   int ld_tail;
+  int relu2;               // kEpiStore: features are stored as max(value, 0)^2
 };
 
 struct SmemLayout {
@@ -443,7 +445,7 @@ __device__ __forceinline__ void epi_bar_sync() {
 // independent chains (fully unrolled, no early exit) and stored with
 // predicates, the epilogue kind is tested once per call.
 //
-// kWide: the forms with a cubic activation, a gating operand or fp32 features. They are a kernel of their own, because one
+// kWide: the forms with a cubic or squared activation, a gating operand or fp32 features. They are a kernel of their own, because one
 // warp per scheduler feels every instruction that the common forms would have to skip.
 template <bool kWide>
 __device__ __forceinline__ void epilogue_store16(const Problem& p, int f, int fb, int n_first, int row_end,
@@ -472,9 +474,13 @@ __device__ __forceinline__ void epilogue_store16(const Problem& p, int f, int fb
         v[j] = __fdividef(gg, 1.f + __expf(-a * gg)) * (uu + p.up_add);
       }
     }
-  } else if (p.epilogue == kEpiResidual || (kWide && p.epilogue == kEpiGateMul)) {
+  } else if (p.epilogue == kEpiResidual || (kWide && (p.epilogue == kEpiGateMul || p.epilogue == kEpiSigmoid))) {
     // sixteen loads in flight: no branch around any of them (rows and features that are not stored repeat ones that are)
     const __nv_bfloat16* r = reinterpret_cast<const __nv_bfloat16*>(p.resid) + static_cast<size_t>(n_first) * p.ld_resid + (live ? f : 0);
+    if (kWide && p.batch > 1) {
+      const int64_t group = n_first / p.x_group_rows;
+      r += group * (p.out_group_stride - static_cast<int64_t>(p.x_group_rows) * p.ld_resid);
+    }
     const int last = valid > 0 ? valid - 1 : 0;
     uint16_t raw[16];
 #pragma unroll
@@ -483,12 +489,17 @@ __device__ __forceinline__ void epilogue_store16(const Problem& p, int f, int fb
     float rr[16];
 #pragma unroll
     for (int j = 0; j < 16; ++j) rr[j] = __uint_as_float(static_cast<uint32_t>(raw[j]) << 16);
+    if (kWide && p.epilogue == kEpiSigmoid) {
 #pragma unroll
-    for (int j = 0; j < 16; ++j) v[j] = round_bf16(g[j] + bias);
+      for (int j = 0; j < 16; ++j) v[j] = __fdividef(g[j] + bias, 1.f + __expf(-rr[j]));
+    } else {
+#pragma unroll
+      for (int j = 0; j < 16; ++j) v[j] = round_bf16(g[j] + bias);
+    }
     if (!kWide || p.epilogue == kEpiResidual) {
 #pragma unroll
       for (int j = 0; j < 16; ++j) v[j] += rr[j];
-    } else {
+    } else if (p.epilogue == kEpiGateMul) {
 #pragma unroll
       for (int j = 0; j < 16; ++j) v[j] = __fdividef(v[j], 1.f + __expf(-p.act_alpha * v[j] * fmaf(p.act_cubic * v[j], v[j], 1.f))) * rr[j];
     }
@@ -499,6 +510,10 @@ __device__ __forceinline__ void epilogue_store16(const Problem& p, int f, int fb
     if (f < p.silu_cols) {
 #pragma unroll
       for (int j = 0; j < 16; ++j) v[j] = __fdividef(v[j], 1.f + __expf(-v[j]));
+    }
+    if (kWide && p.relu2) {
+#pragma unroll
+      for (int j = 0; j < 16; ++j) v[j] = fmaxf(v[j], 0.f) * fmaxf(v[j], 0.f);
     }
   }
   if (p.epilogue == kEpiStoreF32) {

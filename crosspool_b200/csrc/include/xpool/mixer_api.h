@@ -96,20 +96,24 @@ typedef struct XpGluArgs {
   float limit, up_add, alpha, cubic;
 } XpGluArgs;
 
-/* out = act(z) * e, act as above, in fp32; out may be z. */
+/* Elementwise, in fp32; out may be z. kind 0: out = act(z) * e, act as above; 1: out = z * sigmoid(e); 2: out = max(z, 0)^2. */
 typedef struct XpGateMulArgs {
   const float* z;        /* [rows, ld_z] */
-  const float* e;        /* [rows, ld_e] */
+  const float* e;        /* [rows, ld_e], kinds 0 and 1 */
   float* out;            /* [rows, ld_out] */
   int rows, cols, ld_z, ld_e, ld_out;
   float alpha, cubic;
+  int kind;
 } XpGateMulArgs;
 
-/* Grouped-query attention without rotation, per token row: RMS norm of query and key heads, queries laid out
- * [rows, kv_heads, group_pad, dq], keys and values written to the cache row of the token, everything zero-padded. */
+/* Between the projection and grouped-query attention, per token row: RMS norm of query and key heads, rotation of their first
+ * 2 rot_pairs channels (the order of the two does not matter for a norm without a weight; one with a weight comes first),
+ * queries laid out [rows, kv_heads, group_pad, dq], keys and values written to the cache row of the token, everything
+ * zero-padded. Values may be the projected keys (v_off = k_off). With pool > 0 the first pool_rows rows (row r of table row r)
+ * also store the means of the blocks that they complete (XpBlockMeanArgs). */
 typedef struct XpGroupedPrepArgs {
   const void* proj;      /* [rows, ld_proj]: q (heads x dim), k (kv_heads x dim), v (kv_heads x vdim) at the offsets */
-  const float* q_norm;   /* [dim], or null: no norm */
+  const float* q_norm;   /* [dim], or null: no weight */
   const float* k_norm;
   const int* slots;      /* [rows] cache row, -1: none */
   void* k_cache;         /* [tokens, kv_heads, dq] */
@@ -118,7 +122,32 @@ typedef struct XpGroupedPrepArgs {
   int rows, heads, kv_heads, group_pad, dim, vdim, dq, dv, ld_proj, q_off, k_off, v_off;
   float eps;
   int f32;
+  int norm;              /* queries and keys are divided by their root mean square */
+  int rot_pairs;         /* 0: no rotation */
+  int rot_positions;
+  int interleaved;       /* pairs (2 i, 2 i + 1) instead of (i, i + rot_pairs) */
+  const float* rot;      /* [rot_positions, rot_pairs, 2]: cos, sin */
+  const int* positions;  /* [rows], rotation and pooling */
+  const int* block_table;/* pooling */
+  void* k_pool;          /* [pages, pool_page, kv_heads, dq] */
+  void* v_pool;
+  int pool, pool_page, pool_rows, page_size, max_blocks;
 } XpGroupedPrepArgs;
+
+/* Means over blocks of `pool` cached tokens: every row whose position completes block b stores the mean of the block's keys and
+ * values in row b % pool_page of page block_table[b / pool_page] of k_pool and v_pool. */
+typedef struct XpBlockMeanArgs {
+  const void* k_cache;   /* [pages, page_size, kv_heads, dq] */
+  const void* v_cache;
+  void* k_pool;
+  void* v_pool;
+  const int* row_seq;    /* [rows] table row, or null: row r uses table row r */
+  const int* positions;  /* [rows] */
+  const int* slots;      /* [rows] < 0: padding row */
+  const int* block_table;
+  int rows, kv_heads, dq, dv, page_size, max_blocks, pool, pool_page;
+  int f32;
+} XpBlockMeanArgs;
 
 /* Between the projection and grouped-query attention: causal convolution over time of every query, key and value channel
  * (conv_w null: none), rotary positions on the first 2 rot_pairs channels of queries and keys (pairs (i, i + rot_pairs)),
@@ -159,6 +188,11 @@ typedef struct XpGroupedAttnArgs {
   float scale, softcap;
   int f32;
   int window, keep_first, gate_elems;
+  const float* sink;         /* [heads], or null: exp(sink) joins the softmax's sum */
+  const float* sigmoid_bias; /* [heads]: weights are sigmoid(score + bias), not normalised (null: softmax) */
+  const void* k_pool;        /* pool > 0: keys and values of the blocks behind the window, seen beside it */
+  const void* v_pool;
+  int pool, pool_page;
 } XpGroupedAttnArgs;
 
 /* Linear attention with a decay per key channel: S = diag(alpha) S + k v^T, o = S^T q qscale, log alpha = -softplus(-z) / tau.
@@ -238,7 +272,8 @@ typedef struct XpMemoryArgs {
 
 /* Latent attention, per token row: normalise the latent, rotate the shared key part, write both to the cache row of the
  * token; rotate the rotary part of every query head and lay the queries out for the absorbed form
- * (q_plain head-major, q_abs columns [kv_rank, +rot)) and/or the expanded form (q_exp). */
+ * (q_plain head-major, q_abs columns [kv_rank, +rot)) and/or the expanded form (q_exp). Queries may come from a buffer of
+ * their own (q), as a map of the q_rank projected columns at ql_off that still lacks the division by their root mean square. */
 typedef struct XpLatentPrepArgs {
   const void* proj;      /* [rows, ld_proj]: q at q_off (heads x (dim + rot)), latent + key at kv_off (kv_rank + rot) */
   const float* norm_w;   /* [kv_rank] */
@@ -253,6 +288,9 @@ typedef struct XpLatentPrepArgs {
   int abs_rows;          /* rows < abs_rows are laid out for the absorbed form, the others for the expanded one */
   float eps;
   int f32;
+  const void* q;         /* optional [rows, ld_q]: heads x (dim + rot), instead of the columns at q_off */
+  int ld_q, q_rank, ql_off;
+  int interleaved;       /* pairs (2 i, 2 i + 1) instead of (i, i + rot_dims / 2) */
 } XpLatentPrepArgs;
 
 /* Attention of single rows against the latent cache (keys: the first kv_rank + rot columns of a cache row shared by
@@ -273,9 +311,11 @@ typedef struct XpLatentAttnArgs {
   float scale;
   int f32;
   int force_simt;        /* plain kernel */
+  int window;            /* > 0: rows see the last `window` of their tokens; slices count over those */
 } XpLatentAttnArgs;
 
-/* Copies the cached latents of each sequence to a dense workspace: sequence i's ctx + q tokens start at row starts[i]. */
+/* Copies the cached latents of each sequence to a dense workspace: sequence i's ctx + q tokens start at row starts[i]. With a
+ * window the copy begins at the 64-token boundary at or before the first token that the first query sees. */
 typedef struct XpLatentGatherArgs {
   const void* cache;
   void* out;             /* [*, ld_cache] */
@@ -283,7 +323,7 @@ typedef struct XpLatentGatherArgs {
   const int* ctx_lens;
   const int* q_lens;
   const int* starts;     /* [n_seqs] first workspace row */
-  int n_seqs, max_len, page_size, max_blocks, ld_cache, elem_bytes;
+  int n_seqs, max_len, page_size, max_blocks, ld_cache, elem_bytes, window;
 } XpLatentGatherArgs;
 
 /* Decayed linear attention S = decay S + k v^T, o = S^T q; the state of sequence slot s is
@@ -314,6 +354,7 @@ int xp_head_gate(const XpHeadGateArgs* a, void* stream);
 int xp_glu_f32(const XpGluArgs* a, void* stream);
 int xp_gate_mul_f32(const XpGateMulArgs* a, void* stream);
 int xp_grouped_prep(const XpGroupedPrepArgs* a, void* stream);
+int xp_block_mean(const XpBlockMeanArgs* a, void* stream);
 int xp_conv_rope_decode(const XpConvRopeArgs* a, void* stream);
 int xp_conv_rope_prefill(const XpConvRopeArgs* a, void* stream);
 int xp_grouped_attn(const XpGroupedAttnArgs* a, void* stream);

@@ -276,8 +276,11 @@ decode_attn_kernel(XpDecodeAttnArgs a) {
 //
 // kRows: the form of layered decoders (XpDecodeRowsArgs): rows name their sequence, query groups are padded, keys and values
 // differ in width, scores may be capped, rows may see a window of their tokens and the first ones only (the tiles between are
-// left out: slices and tiles count over what remains), outputs gated, and the probabilities enter the second product as a bf16 pair (high
-// and low part), so that they keep 16 mantissa bits.
+// left out: slices and tiles count over what remains), outputs gated, a number per head may join the softmax's sum, and the
+// probabilities enter the second product as a bf16 pair (high and low part), so that they keep 16 mantissa bits.
+//
+// kSig: weights are sigmoids of the scores (no maximum, no sum), and the tiles may begin with the means of the blocks behind the
+// window, which come from a paged cache of their own in two boxes of eight rows.
 constexpr int kTcStages = 3;
 
 __device__ __forceinline__ void tma_load_kv(uint32_t dst, const CUtensorMap* m, uint32_t bar, int d0, int head, int token) {
@@ -318,20 +321,21 @@ __device__ __forceinline__ const XpDecodeAttnArgs& base_of(const XpDecodeRowsArg
 __device__ __forceinline__ const XpDecodeAttnArgs& base_of(const XpDecodeAttnArgs& a) { return a; }
 
 // What a row reads of its sequence: tokens [0, head) and [head + skip, len + skip), head and skip whole 16-token tiles. `len`
-// counts both; lo is the first token of the window.
+// counts both; lo is the first token of the window. With pooled blocks the first `blocks` of [0, head) are those.
 struct Span {
-  int len, head, skip, lo;
+  int len, head, skip, lo, blocks;
   __device__ __forceinline__ int token(int v) const { return v < head ? v : v + skip; }
 };
 
 template <typename A>
 __device__ __forceinline__ Span row_span(const A& args, int b) {
-  Span s{0, 0, 0, 0};
+  Span s{0, 0, 0, 0, 0};
   if constexpr (std::is_same<A, XpDecodeRowsArgs>::value) {
     s.len = args.slots[b] < 0 ? 0 : args.positions[b] + 1;
     if (args.window > 0 && s.len > args.window) {
       s.lo = s.len - args.window;
-      s.head = min((args.keep_first + 15) & ~15, s.lo & ~15);
+      s.blocks = args.pool > 0 ? s.lo / args.pool : 0;
+      s.head = args.pool > 0 ? (s.blocks + 15) & ~15 : min((args.keep_first + 15) & ~15, s.lo & ~15);
       s.skip = (s.lo & ~15) - s.head;
       s.len -= s.skip;
     }
@@ -356,10 +360,26 @@ __device__ __forceinline__ void store_out(const A& args, int b, int hq, int d, f
   }
 }
 
-template <int DQ, int DV, typename A>
+// Final value of an output element from its sum of weighted values, the sum of weights and their scale (log2 domain).
+template <bool kSig, typename A>
+__device__ __forceinline__ float finish_out(const A& args, int hq, float av, float ll, float mm) {
+  if constexpr (kSig) return av;
+  if constexpr (std::is_same<A, XpDecodeRowsArgs>::value) {
+    if (args.sink != nullptr) {
+      const float sink = args.sink[hq] * 1.4426950408889634f, top = fmaxf(mm, sink);
+      const float c = mm == -CUDART_INF_F ? 0.f : exp2f(mm - top);
+      av *= c, ll = ll * c + exp2f(sink - top);
+    }
+  }
+  return ll > 0.f ? av / ll : 0.f;
+}
+
+template <int DQ, int DV, typename A, bool kSig = false>
 __global__ void __launch_bounds__(kDecodeThreads, 2)
-decode_attn_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constant__ CUtensorMap tmap_v, A args) {
+decode_attn_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constant__ CUtensorMap tmap_v,
+                      const __grid_constant__ CUtensorMap tmap_kp, const __grid_constant__ CUtensorMap tmap_vp, A args) {
   constexpr bool kRows = std::is_same<A, XpDecodeRowsArgs>::value;
+  static_assert(kRows || !kSig, "sigmoid weights are a form of single rows");
   const XpDecodeAttnArgs& a = base_of(args);
   constexpr int kHalves = DQ / 64;             // 64-dim boxes per key row
   constexpr int kVHalves = DV / 64;            // ... per value row
@@ -405,18 +425,42 @@ decode_attn_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_c
     if (args.row_seq != nullptr) table_row = args.row_seq[b];
   }
   const int* table = a.block_table + static_cast<size_t>(table_row) * a.max_blocks;
-  // lane i looks up the cache position of the tile of iteration (base + i)
-  auto lookup = [&](int it) -> int {
+  // lane i looks up the cache position of the tile of iteration (base + i); pooled tiles: of its first (part 0) or last eight rows
+  auto lookup = [&](int it, int part = 0) -> int {
     if (it >= n_it) return 0;
-    const int ts = span.token(t0 + ((it * 4 + warp) << 4));
+    const int v = t0 + ((it * 4 + warp) << 4);
+    if constexpr (kSig) {
+      if (v < span.head) {
+        const int b = v + part * 8 < span.blocks ? v + part * 8 : v;
+        return table[b / args.pool_page] * args.pool_page + b % args.pool_page;
+      }
+      if (part) return 0;
+    }
+    const int ts = span.token(v);
     return (table[ts >> page_shift] << page_shift) + (ts & page_mask);
   };
-  int my_tok = lookup(lane);
-  auto issue = [&](int it, int tok) {  // lane 0 only
+  int my_tok = lookup(lane), my_tok2 = 0;
+  if constexpr (kSig) my_tok2 = lookup(lane, 1);
+  auto issue = [&](int it, int tok, int tok2) {  // lane 0 only
     const int s = it % kTcStages;
     const uint32_t bar = sm100::smem_u32(&full[warp][s]);
     const uint32_t dst = ring + s * kStage;
     sm100::mbar_arrive_expect_tx(&full[warp][s], kStage);
+    if constexpr (kSig) {
+      if (t0 + ((it * 4 + warp) << 4) < span.head) {
+#pragma unroll
+        for (int h = 0; h < kHalves; ++h) {
+          tma_load_kv(dst + h * kBox, &tmap_kp, bar, h * 64, hk, tok);
+          tma_load_kv(dst + h * kBox + kBox / 2, &tmap_kp, bar, h * 64, hk, tok2);
+        }
+#pragma unroll
+        for (int h = 0; h < kVHalves; ++h) {
+          tma_load_kv(dst + (kHalves + h) * kBox, &tmap_vp, bar, h * 64, hk, tok);
+          tma_load_kv(dst + (kHalves + h) * kBox + kBox / 2, &tmap_vp, bar, h * 64, hk, tok2);
+        }
+        return;
+      }
+    }
 #pragma unroll
     for (int h = 0; h < (kHalves > kVHalves ? kHalves : kVHalves); ++h) {
       if (h < kHalves) tma_load_kv(dst + h * kBox, &tmap_k, bar, h * 64, hk, tok);
@@ -426,7 +470,8 @@ decode_attn_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_c
 #pragma unroll
   for (int i = 0; i < kTcStages; ++i) {
     const int tok = __shfl_sync(0xffffffffu, my_tok, i);
-    if (lane == 0 && i < n_it) issue(i, tok);
+    const int tok2 = kSig ? __shfl_sync(0xffffffffu, my_tok2, i) : 0;
+    if (lane == 0 && i < n_it) issue(i, tok, tok2);
   }
 
   // Q fragments (A operand), unscaled; rows >= G are zero
@@ -449,7 +494,12 @@ decode_attn_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_c
   if constexpr (kRows) {
     if (args.softcap > 0.f) cap2 = args.softcap * 1.4426950408889634f, capx = 2.f * sscale / args.softcap;
   }
-  float m0 = -CUDART_INF_F, m1 = -CUDART_INF_F, l0 = 0.f, l1 = 0.f;
+  float m0 = kSig ? 0.f : -CUDART_INF_F, m1 = m0, l0 = 0.f, l1 = 0.f;
+  float b0 = 0.f, b1 = 0.f;                            // biases of rows g and g + 8, log2 domain
+  if constexpr (kSig) {
+    if (g < G) b0 = args.sigmoid_bias[hk * G + g] * 1.4426950408889634f;
+    if (g + 8 < G) b1 = args.sigmoid_bias[hk * G + g + 8] * 1.4426950408889634f;
+  }
   float acc[DV / 8][4];
 #pragma unroll
   for (int j = 0; j < DV / 8; ++j)
@@ -467,12 +517,15 @@ decode_attn_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_c
       break;
     }
     const int tbase = t0 + ((it * 4 + warp) << 4);
-    const int nvalid = min(16, t1 - tbase);
+    const bool pooled = kSig && tbase < span.head;
+    const int nvalid = min(16, (pooled ? span.blocks : t1) - tbase);
     // tokens [unseen, below) of the tile lie between the first tokens and the window
     int unseen = 0, below = 0;
-    if constexpr (kRows) {
+    if (kRows && !pooled) {
       const int first = span.token(tbase);
-      if (first < span.lo) unseen = max(0, args.keep_first - first), below = span.lo - first;
+      if constexpr (kRows) {
+        if (first < span.lo) unseen = max(0, args.keep_first - first), below = span.lo - first;
+      }
     }
     if (nvalid < 16) {
       // cache slots past the sequence end hold whatever was there: zero those V rows so that a
@@ -501,7 +554,19 @@ decode_attn_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_c
         mma_bf16_16816(sc[nt], qf[2 * j + 1], kb[2], kb[3]);
       }
     }
+    if constexpr (kSig) {
+      // ---- sigmoid weights on rows g and g + 8
+#pragma unroll
+      for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int col = nt * 8 + q4 * 2 + (e & 1);
+          const float v = __frcp_rn(1.f + exp2f(-fmaf(sc[nt][e], sscale, e < 2 ? b0 : b1)));
+          sc[nt][e] = col >= nvalid || (col >= unseen && col < below) ? 0.f : v;
+        }
+    }
     // ---- online softmax on rows g and g + 8
+    if constexpr (!kSig) {
     float mx0 = -CUDART_INF_F, mx1 = -CUDART_INF_F;
 #pragma unroll
     for (int nt = 0; nt < 2; ++nt)
@@ -536,10 +601,12 @@ decode_attn_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_c
       m0 = n0;
       m1 = n1;
     }
+    }
     uint32_t pf[4], pl[4];
     {
-      const float p00 = exp2f(sc[0][0] - m0), p01 = exp2f(sc[0][1] - m0), p02 = exp2f(sc[0][2] - m1), p03 = exp2f(sc[0][3] - m1);
-      const float p10 = exp2f(sc[1][0] - m0), p11 = exp2f(sc[1][1] - m0), p12 = exp2f(sc[1][2] - m1), p13 = exp2f(sc[1][3] - m1);
+      auto weight = [&](float v, float m) { return kSig ? v : exp2f(v - m); };
+      const float p00 = weight(sc[0][0], m0), p01 = weight(sc[0][1], m0), p02 = weight(sc[0][2], m1), p03 = weight(sc[0][3], m1);
+      const float p10 = weight(sc[1][0], m0), p11 = weight(sc[1][1], m0), p12 = weight(sc[1][2], m1), p13 = weight(sc[1][3], m1);
       l0 += p00 + p01 + p10 + p11;
       l1 += p02 + p03 + p12 + p13;
       pf[0] = pack_bf16(p00, p01);  // (row g,     tokens 2 q4 ..)
@@ -570,11 +637,15 @@ decode_attn_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_c
     }
     __syncwarp();  // every lane has consumed the stage
     const int nxt = it + kTcStages;
-    if ((nxt & 31) == 0) my_tok = lookup(nxt + lane);
+    if ((nxt & 31) == 0) {
+      my_tok = lookup(nxt + lane);
+      if constexpr (kSig) my_tok2 = lookup(nxt + lane, 1);
+    }
     const int tok = __shfl_sync(0xffffffffu, my_tok, nxt & 31);
+    const int tok2 = kSig ? __shfl_sync(0xffffffffu, my_tok2, nxt & 31) : 0;
     if (lane == 0 && nxt < n_it) {
       sm100::fence_proxy_async_smem();
-      issue(nxt, tok);
+      issue(nxt, tok, tok2);
     }
   }
   if (timed_out) {
@@ -622,7 +693,7 @@ decode_attn_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_c
     }
     const int hq = hk * G + gg;
     if (nsplit == 1) {
-      store_out<DV>(args, b, hq, d, ll > 0.f ? av / ll : 0.f);
+      store_out<DV>(args, b, hq, d, finish_out<kSig>(args, hq, av, ll, mm));
     } else {
       float* ws = a.ws + ((static_cast<size_t>(b) * a.q_heads + hq) * nsplit + split) * (DV + 2);
       ws[d] = av;
@@ -634,7 +705,7 @@ decode_attn_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_c
   }
 }
 
-template <int D, typename A>
+template <int D, bool kSig = false, typename A>
 __global__ void decode_combine_kernel(A args, int nsplit) {
   const XpDecodeAttnArgs& a = base_of(args);
   const int hq = blockIdx.x, b = blockIdx.y, d = threadIdx.x;
@@ -652,7 +723,7 @@ __global__ void decode_combine_kernel(A args, int nsplit) {
     ll += ws[s * (D + 2) + D + 1] * c;
     av += ws[s * (D + 2) + d] * c;
   }
-  store_out<D>(args, b, hq, d, ll > 0.f ? av / ll : 0.f);
+  store_out<D>(args, b, hq, d, finish_out<kSig>(args, hq, av, ll, mm));
 }
 
 template <int D, int GMAX>
@@ -670,24 +741,32 @@ static int launch_decode(const XpDecodeAttnArgs& a, int nsplit, cudaStream_t s) 
   return e == cudaSuccess ? 0 : -100 - static_cast<int>(e);
 }
 
-template <int DQ, int DV, typename A>
+template <int DQ, int DV, bool kSig = false, typename A>
 static int launch_decode_tc(const A& args, int nsplit, cudaStream_t s) {
   const XpDecodeAttnArgs& a = reinterpret_cast<const XpDecodeAttnArgs&>(args);   // the first member of the wider form
-  CUtensorMap mk, mv;
+  CUtensorMap mk, mv, mkp, mvp;
   const uint64_t tokens = static_cast<uint64_t>(a.num_pages) * a.page_size;
   if (tmap::cache().get_kv(&mk, a.k_cache, tokens, a.kv_heads, DQ) != 0) return -20;
   if (tmap::cache().get_kv(&mv, a.v_cache, tokens, a.kv_heads, DV) != 0) return -20;
+  mkp = mk, mvp = mv;
+  if constexpr (kSig) {
+    if (args.pool > 0) {
+      const uint64_t rows = static_cast<uint64_t>(a.num_pages) * args.pool_page;
+      if (tmap::cache().get_kv(&mkp, args.k_pool, rows, a.kv_heads, DQ, 8) != 0) return -20;
+      if (tmap::cache().get_kv(&mvp, args.v_pool, rows, a.kv_heads, DV, 8) != 0) return -20;
+    }
+  }
   constexpr int kStage = ((DQ + DV) / 64) * 16 * 128;
   constexpr int kSmem = 4 * kTcStages * kStage + 1024;  // rings of four warps + alignment slack
   static_assert(4 * 16 * (DV + 2) * 4 <= 4 * kTcStages * kStage, "merge scratch must fit in the rings");
   static bool attr_set = false;
   if (!attr_set) {
-    if (cudaFuncSetAttribute(decode_attn_tc_kernel<DQ, DV, A>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem) != cudaSuccess) return -21;
+    if (cudaFuncSetAttribute(decode_attn_tc_kernel<DQ, DV, A, kSig>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem) != cudaSuccess) return -21;
     attr_set = true;
   }
   dim3 grid(nsplit, a.kv_heads, a.batch);
-  decode_attn_tc_kernel<DQ, DV, A><<<grid, kDecodeThreads, kSmem, s>>>(mk, mv, args);
-  if (nsplit > 1) decode_combine_kernel<DV><<<dim3(a.q_heads, a.batch), DV, 0, s>>>(args, nsplit);
+  decode_attn_tc_kernel<DQ, DV, A, kSig><<<grid, kDecodeThreads, kSmem, s>>>(mk, mv, mkp, mvp, args);
+  if (nsplit > 1) decode_combine_kernel<DV, kSig><<<dim3(a.q_heads, a.batch), DV, 0, s>>>(args, nsplit);
   cudaError_t e = cudaGetLastError();
   return e == cudaSuccess ? 0 : -100 - static_cast<int>(e);
 }
@@ -742,6 +821,15 @@ extern "C" int xp_decode_rows(const XpDecodeRowsArgs* r, void* stream) {
       a->chunk_tokens % 16 != 0 || (reinterpret_cast<uintptr_t>(a->q) & 3) != 0 || a->batch > 65535)
     return -12;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  if (r->pool > 0 && (r->sigmoid_bias == nullptr || r->window <= 0 || r->keep_first > 0 || r->k_pool == nullptr || r->v_pool == nullptr ||
+                      r->pool_page < 8 || (r->pool_page & (r->pool_page - 1)) != 0))
+    return -14;
+  if (r->sigmoid_bias != nullptr) {
+    if (r->softcap > 0.f || r->sink != nullptr || r->keep_first > 0) return -15;
+    if (a->head_dim == 64 && r->v_dim == 64) return launch_decode_tc<64, 64, true>(*r, nsplit, s);
+    if (a->head_dim == 128 && r->v_dim == 128) return launch_decode_tc<128, 128, true>(*r, nsplit, s);
+    return -13;
+  }
   if (a->head_dim == 64 && r->v_dim == 64) return launch_decode_tc<64, 64>(*r, nsplit, s);
   if (a->head_dim == 128 && r->v_dim == 64) return launch_decode_tc<128, 64>(*r, nsplit, s);
   if (a->head_dim == 128 && r->v_dim == 128) return launch_decode_tc<128, 128>(*r, nsplit, s);

@@ -25,7 +25,12 @@
 // number of query heads is no power of two come padded (their padding is computed and not stored). Scores may be capped,
 // cap tanh(s / cap): in a tile whose scores are all far below the cap by a polynomial on the FMA pipe, otherwise through
 // 2 ** x and a reciprocal. Queries may see a window of tokens and the first ones of the sequence only: the K/V tiles between
-// are left out (the roles count over the tiles that remain), the edges are masked per row.
+// are left out (the roles count over the tiles that remain), the edges are masked per row. A number per head may join the
+// softmax's sum (a sink). Dense rows of a windowed layer begin at the tile in which the first query's window does.
+//
+// kSig: weights are sigmoids of the scores plus a number per head (no maximum, no sum, no rescaling), and the tiles may begin with
+// the means of the blocks behind the window, copied from a paged cache of their own in boxes of eight rows; which of them a row
+// sees is masked per row.
 //
 // V is used where it lands (token-major rows of 64 dims) through an MN-major operand descriptor; no transpose.
 // Tensor memory: S buffers 4 x 64 columns, O 2 x D columns (512 columns with D = 128).
@@ -127,13 +132,28 @@ __device__ __forceinline__ void cap_scores(uint32_t (&sv)[kBN], float scale, flo
   }
 }
 
-template <int DQ, int DV, bool kTS, bool kPair, bool kCap>
+// Scores of one row (raw products) -> sigmoid(s + bias), scale and bias in log2 units. Two elements share a reciprocal; scores
+// below -60 count as -60, -inf (masked) becomes zero.
+__device__ __forceinline__ void sigmoid_scores(uint32_t (&sv)[kBN], float scale2, float bias2) {
+#pragma unroll
+  for (int j = 0; j < kBN; j += 2) {
+    const float x = fmaf(__uint_as_float(sv[j]), scale2, bias2), y = fmaf(__uint_as_float(sv[j + 1]), scale2, bias2);
+    const float a = 1.f + sm100::ex2_approx(fminf(-x, 60.f)), b = 1.f + sm100::ex2_approx(fminf(-y, 60.f));
+    float r;
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(a * b));
+    sv[j] = sv[j] == 0xff800000u ? 0u : __float_as_uint(r * b);
+    sv[j + 1] = sv[j + 1] == 0xff800000u ? 0u : __float_as_uint(r * a);
+  }
+}
+
+template <int DQ, int DV, bool kTS, bool kPair, bool kCap, bool kSig>
 __global__ void __launch_bounds__(kThreads, 1)
 prefill_attn_umma_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
                          const __grid_constant__ CUtensorMap tmap_v, const __grid_constant__ CUtensorMap tmap_k3,
-                         const __grid_constant__ CUtensorMap tmap_v3, XpPrefillAttnArgs a, int G, int g_shift,
-                         int box_tokens) {
+                         const __grid_constant__ CUtensorMap tmap_v3, const __grid_constant__ CUtensorMap tmap_kp,
+                         const __grid_constant__ CUtensorMap tmap_vp, XpPrefillAttnArgs a, int G, int g_shift, int box_tokens) {
   static_assert(kTS || !kPair, "the low parts live beside the high parts in tensor memory");
+  static_assert(!kSig || (kPair && !kCap), "a form of layered decoders");
   constexpr int kHalves = DQ / 64;                // 64-dim (128-byte) column blocks of a query or key row
   constexpr int kVHalves = DV / 64;               // ... of a value row
   constexpr int kQHalf = kRows * 128;             // one 64-dim block of a query tile
@@ -154,7 +174,8 @@ prefill_attn_umma_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gri
   const int q_len = a.q_lens[seq];
   const int q0 = qt * 2 * np;                     // first position of the CTA (longest tiles are dispatched first)
   if (q0 >= q_len) return;
-  const int ctx = a.ctx_lens[seq];
+  int ctx = a.ctx_lens[seq];
+  if (kPair && a.seq_starts != nullptr && a.window > 0) ctx -= max(0, ctx - a.window + 1) & ~(kBN - 1);   // the rows begin there
   const int q_base = a.q_starts[seq];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const uint32_t base = (sm100::smem_u32(smem_dyn) + 1023u) & ~1023u;
@@ -162,8 +183,13 @@ prefill_attn_umma_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gri
   const bool act_b = q0 + np < q_len;             // tile B holds at least one real row
   const int kv_end = ctx + min(q_len, q0 + 2 * np);            // causal bound of the CTA
   // tiles [0, head) and those from head + skip on are read
-  int head = 0, skip = 0;
-  if (kPair && a.window > 0 && ctx + q0 >= a.window) {
+  // (kSig: tiles [0, head) hold the means of the first `blocks` blocks, the others start where the window does)
+  int head = 0, skip = 0, blocks = 0;
+  if (kSig && a.pool > 0) {
+    blocks = max(0, kv_end - a.window) / a.pool;               // that the last query sees
+    head = (blocks + kBN - 1) / kBN;
+    skip = max(0, ctx + q0 - a.window + 1) / kBN - head;
+  } else if (kPair && a.window > 0 && ctx + q0 >= a.window) {
     const int lo_tile = (ctx + q0 - a.window + 1) / kBN;       // of the first query's window
     head = min((a.keep_first + kBN - 1) / kBN, lo_tile);
     skip = lo_tile - head;
@@ -225,7 +251,18 @@ prefill_attn_umma_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gri
       if (t >= kStages && !__all_sync(0xffffffffu, wait_bar(&bars.kv_empty[s], ((t / kStages) - 1) & 1, &bars, 1))) break;
       if (lane == 0) sm100::mbar_arrive_expect_tx(&bars.kv_full[s], kStage);
       __syncwarp();
-      if (boxes == 1) {
+      if (kSig && a.pool > 0 && t < head) {
+        for (int i = lane; i < 8 * (kHalves + kVHalves); i += 32) {
+          const int j = i & 7, h = i >> 3;           // eight rows, 64 dims of keys, then of values
+          int b = t * kBN + j * 8;
+          if (b >= blocks) b = (blocks - 1) & ~7;    // rows past the end repeat valid ones (masked)
+          const int tok = table[b / a.pool_page] * a.pool_page + (b & (a.pool_page - 1));
+          const bool is_v = h >= kHalves;
+          const int hh = is_v ? h - kHalves : h;
+          sm100::tma_load_3d_addr(kv_s + s * kStage + (is_v ? kKTile : 0) + hh * kKVHalf + j * 1024, is_v ? &tmap_vp : &tmap_kp,
+                                  sm100::smem_u32(&bars.kv_full[s]), hh * 64, hk, tok);
+        }
+      } else if (boxes == 1) {
         if (lane < 2) {
           int tk = tile_token(t);
           if (tk >= kv_end) tk = (kv_end - 1) & ~(kBN - 1);
@@ -336,6 +373,10 @@ prefill_attn_umma_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gri
     const uint32_t o_t = tmem + lane_off + kOCol + static_cast<uint32_t>(x * DV);
     const uint32_t p_row = p_s + x * kPTile + row * 128;
     const float sc2 = kCap ? 1.f : a.scale * 1.4426950408889634f;
+    const bool pooling = kSig && a.pool > 0;
+    const int my_blocks = pooling ? max(0, ctx + pos - a.window + 1) / a.pool : 0;
+    float bias2 = 0.f;
+    if constexpr (kSig) bias2 = a.sigmoid_bias[min(hq, a.kv_heads * heads - 1)] * 1.4426950408889634f;
     float m_used = -CUDART_INF_F, l = 0.f;
     bool ok = true;
     if (tile_on) {
@@ -357,50 +398,62 @@ prefill_attn_umma_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gri
         }
 
         if constexpr (kCap) cap_scores(sv, a.scale, a.softcap);
-        const int tok0 = tile_token(t);
-        const int nvis = min(kBN, max(0, limit - tok0 + 1));      // visible tokens of this tile for this row
+        const bool pooled = kSig && pooling && t < head;
+        const int tok0 = pooled ? t * kBN : tile_token(t);
+        const int nvis = min(kBN, max(0, (pooled ? my_blocks : limit + 1) - tok0));      // visible tokens of this tile for this row
         if (nvis < kBN) {
 #pragma unroll
           for (int j = 0; j < kBN; ++j)
             if (j >= nvis) sv[j] = 0xff800000u;       // -inf: selected, never computed with (the slot may hold NaN)
         }
-        const int below = win_lo - tok0, kept = a.keep_first - tok0;   // tokens [kept, below) of the tile are behind the window
+        const int below = pooled ? 0 : win_lo - tok0, kept = a.keep_first - tok0;   // tokens [kept, below) of the tile are behind the window
         if (kPair && below > 0 && kept < kBN) {
 #pragma unroll
           for (int j = 0; j < kBN; ++j)
             if (j >= kept && j < below) sv[j] = 0xff800000u;
         }
-        // four independent chains of three-input maxima: a serial chain over 64 values costs its latency 64 times
-        float mx4[4] = {-CUDART_INF_F, -CUDART_INF_F, -CUDART_INF_F, -CUDART_INF_F};
-#pragma unroll
-        for (int j = 0; j < kBN; j += 8) {
-#pragma unroll
-          for (int c = 0; c < 4; ++c) mx4[c] = max3(mx4[c], __uint_as_float(sv[j + 2 * c]), __uint_as_float(sv[j + 2 * c + 1]));
-        }
-        const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
-        const float m_new = mx * sc2;
         float factor = 1.f;
-        if (m_new > m_used + kRescaleStep || m_used == -CUDART_INF_F) {
-          if (m_new != -CUDART_INF_F) {
-            factor = m_used == -CUDART_INF_F ? 0.f : sm100::ex2_approx(m_used - m_new);
-            m_used = m_new;
-          }
-        }
-        const float m_sub = m_used == -CUDART_INF_F ? 0.f : m_used;
-        float sum4[4] = {0.f, 0.f, 0.f, 0.f};
         uint32_t pk[kBN / 2];
+        if constexpr (kSig) {
+          sigmoid_scores(sv, sc2, bias2);
 #pragma unroll
-        for (int j = 0; j < kBN; j += 2) {
-          const float p0 = sm100::ex2_approx(fmaf(__uint_as_float(sv[j]), sc2, -m_sub));
-          const float p1 = sm100::ex2_approx(fmaf(__uint_as_float(sv[j + 1]), sc2, -m_sub));
-          sum4[(j >> 1) & 3] += p0 + p1;
-          pk[j >> 1] = pack2(p0, p1);
-          if constexpr (kPair) {
+          for (int j = 0; j < kBN; j += 2) {
+            const float p0 = __uint_as_float(sv[j]), p1 = __uint_as_float(sv[j + 1]);
+            pk[j >> 1] = pack2(p0, p1);
             const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&pk[j >> 1]));
-            sv[j >> 1] = pack2(p0 - hi.x, p1 - hi.y);     // over scores already consumed
+            sv[j >> 1] = pack2(p0 - hi.x, p1 - hi.y);
           }
+        } else {
+          // four independent chains of three-input maxima: a serial chain over 64 values costs its latency 64 times
+          float mx4[4] = {-CUDART_INF_F, -CUDART_INF_F, -CUDART_INF_F, -CUDART_INF_F};
+#pragma unroll
+          for (int j = 0; j < kBN; j += 8) {
+#pragma unroll
+            for (int c = 0; c < 4; ++c) mx4[c] = max3(mx4[c], __uint_as_float(sv[j + 2 * c]), __uint_as_float(sv[j + 2 * c + 1]));
+          }
+          const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
+          const float m_new = mx * sc2;
+          if (m_new > m_used + kRescaleStep || m_used == -CUDART_INF_F) {
+            if (m_new != -CUDART_INF_F) {
+              factor = m_used == -CUDART_INF_F ? 0.f : sm100::ex2_approx(m_used - m_new);
+              m_used = m_new;
+            }
+          }
+          const float m_sub = m_used == -CUDART_INF_F ? 0.f : m_used;
+          float sum4[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+          for (int j = 0; j < kBN; j += 2) {
+            const float p0 = sm100::ex2_approx(fmaf(__uint_as_float(sv[j]), sc2, -m_sub));
+            const float p1 = sm100::ex2_approx(fmaf(__uint_as_float(sv[j + 1]), sc2, -m_sub));
+            sum4[(j >> 1) & 3] += p0 + p1;
+            pk[j >> 1] = pack2(p0, p1);
+            if constexpr (kPair) {
+              const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&pk[j >> 1]));
+              sv[j >> 1] = pack2(p0 - hi.x, p1 - hi.y);     // over scores already consumed
+            }
+          }
+          l = l * factor + ((sum4[0] + sum4[1]) + (sum4[2] + sum4[3]));
         }
-        l = l * factor + ((sum4[0] + sum4[1]) + (sum4[2] + sum4[3]));
         const bool rescale = __any_sync(0xffffffffu, factor != 1.f);
         if (t > 0 && (!kTS || rescale)) {
           // the previous PV product must have retired: it accumulates into O (and reads the shared-memory P buffer)
@@ -433,13 +486,14 @@ prefill_attn_umma_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gri
                        "r"(pk[c * 4 + 1]), "r"(pk[c * 4 + 2]), "r"(pk[c * 4 + 3])
                        : "memory");
         }
-        const bool v_tail = (x == 0 || t >= n_a) && tok0 + kBN > kv_end;
+        const int v_end = pooled ? blocks : kv_end;
+        const bool v_tail = (x == 0 || t >= n_a) && tok0 + kBN > v_end;
         if (v_tail) {
           // cache slots past the sequence end may hold anything: zero those V rows (probability 0 x NaN).
           // Tile A's PV product is issued before tile B's and both read this stage, so tile A's threads do it
           // on the tiles that tile A visits, tile B's on the rest.
           const uint32_t v_s = kv_s + (t % kStages) * kStage + kKTile;
-          const int first = kv_end - tok0;
+          const int first = v_end - tok0;
           for (int i = row; i < (kBN - first) * (DV / 8); i += kRows) {
             const int R = first + i / (DV / 8), cc = i % (DV / 8);
             const uint32_t off = (cc >> 3) * kKVHalf + R * 128 + (((cc & 7) ^ (R & 7)) << 4);
@@ -475,7 +529,8 @@ prefill_attn_umma_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gri
       if (ok && my_tiles > 0) ok = __all_sync(0xffffffffu, wait_bar(&bars.pv_done[x], (my_tiles - 1) & 1, &bars, 11));
       if (ok) {
         sm100::tc_fence_after_sync();
-        float inv = l > 0.f ? 1.f / l : 0.f;
+        if (kPair && a.sink != nullptr && stored) l += sm100::ex2_approx(fmaf(a.sink[hq], 1.4426950408889634f, -m_used));
+        float inv = kSig ? 1.f : l > 0.f ? 1.f / l : 0.f;
         if (a.gate != nullptr && !a.gate_elems && stored)
           inv *= 1.f / (1.f + expf(-__bfloat162float(reinterpret_cast<const __nv_bfloat16*>(a.gate)[static_cast<size_t>(q_base + pos) * a.ld_gate + hq])));
         const int v_valid = a.v_valid;                    // stored columns of a head (a multiple of 8)
@@ -547,9 +602,9 @@ prefill_attn_umma_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gri
   }
 }
 
-template <int DQ, int DV, bool kTS, bool kPair, bool kCap = false>
+template <int DQ, int DV, bool kTS, bool kPair, bool kCap = false, bool kSig = false>
 static int launch(const XpPrefillAttnArgs& a, int G, cudaStream_t s) {
-  CUtensorMap mq, mk, mv, mk3, mv3;
+  CUtensorMap mq, mk, mv, mk3, mv3, mkp, mvp;
   const uint64_t tokens = static_cast<uint64_t>(a.num_pages) * a.page_size;
   int g_shift = 0;
   while ((1 << g_shift) < G) ++g_shift;
@@ -563,12 +618,18 @@ static int launch(const XpPrefillAttnArgs& a, int G, cudaStream_t s) {
   if (tmap::cache().get_kv(&mk3, a.k_cache, tokens, a.kv_heads, DQ) != 0) return -20;
   if (tmap::cache().get_kv(&mv3, a.v_cache, tokens, a.kv_heads, DV) != 0) return -20;
   if (tmap::cache().get_q(&mq, a.q, static_cast<uint64_t>(a.total_q), a.q_heads, DQ, G, np) != 0) return -20;
+  mkp = mk3, mvp = mv3;
+  if (kSig && a.pool > 0) {
+    const uint64_t rows = static_cast<uint64_t>(a.num_pages) * a.pool_page;
+    if (tmap::cache().get_kv(&mkp, a.k_pool, rows, a.kv_heads, DQ, 8) != 0) return -20;
+    if (tmap::cache().get_kv(&mvp, a.v_pool, rows, a.kv_heads, DV, 8) != 0) return -20;
+  }
   // the shared-memory tiles of the probabilities exist only in the form that stages them there
   constexpr int kSmem = 2 * (DQ / 64) * kRows * 128 + kStages * ((DQ + DV) / 64) * kBN * 128 + (kTS ? 0 : 2 * kRows * 128) + 1024;
   static_assert(kSmem <= 227 * 1024, "tiles exceed the shared memory of an SM");
   static bool attr_set = false;
   if (!attr_set) {
-    if (cudaFuncSetAttribute(prefill_attn_umma_kernel<DQ, DV, kTS, kPair, kCap>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem) != cudaSuccess)
+    if (cudaFuncSetAttribute(prefill_attn_umma_kernel<DQ, DV, kTS, kPair, kCap, kSig>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem) != cudaSuccess)
       return -21;
     attr_set = true;
   }
@@ -577,7 +638,7 @@ static int launch(const XpPrefillAttnArgs& a, int G, cudaStream_t s) {
   if (b.ld_out <= 0) b.ld_out = b.q_heads * b.v_valid;
   if (b.group_valid <= 0) b.group_valid = G;
   dim3 grid(b.kv_heads, b.num_seqs, (b.max_q_len + 2 * np - 1) / (2 * np));
-  prefill_attn_umma_kernel<DQ, DV, kTS, kPair, kCap><<<grid, kThreads, kSmem, s>>>(mq, mk, mv, mk3, mv3, b, G, g_shift, box_tokens);
+  prefill_attn_umma_kernel<DQ, DV, kTS, kPair, kCap, kSig><<<grid, kThreads, kSmem, s>>>(mq, mk, mv, mk3, mv3, mkp, mvp, b, G, g_shift, box_tokens);
   cudaError_t e = cudaGetLastError();
   return e == cudaSuccess ? 0 : -100 - static_cast<int>(e);
 }
@@ -607,6 +668,15 @@ extern "C" int xp_prefill_attn_umma(const XpPrefillAttnArgs* a, void* stream) {
   const bool ts = ((a->force_simple >> 8) & 1) != kDefaultTS;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   const int dv = a->v_dim > 0 ? a->v_dim : a->head_dim;
+  if (a->pool > 0 && (a->sigmoid_bias == nullptr || a->window <= 0 || a->keep_first > 0 || a->seq_starts != nullptr || a->k_pool == nullptr ||
+                      a->v_pool == nullptr || a->pool_page < 8 || (a->pool_page & (a->pool_page - 1)) != 0))
+    return 1;
+  if (a->sigmoid_bias != nullptr) {
+    if (!a->p_pair || a->softcap > 0.f || a->sink != nullptr || a->keep_first > 0) return 1;
+    if (a->head_dim == 64 && dv == 64) return launch<64, 64, true, true, false, true>(*a, G, s);
+    if (a->head_dim == 128 && dv == 128) return launch<128, 128, true, true, false, true>(*a, G, s);
+    return 1;
+  }
   if (a->p_pair) {
     if (a->head_dim == 64 && dv == 64) return launch_pair<64, 64>(*a, G, s);
     if (a->head_dim == 128 && dv == 64) return launch_pair<128, 64>(*a, G, s);
@@ -614,7 +684,7 @@ extern "C" int xp_prefill_attn_umma(const XpPrefillAttnArgs* a, void* stream) {
     if (a->head_dim == 192 && dv == 128) return launch_pair<192, 128>(*a, G, s);
     return 1;
   }
-  if (dv != a->head_dim || a->softcap > 0.f || a->gate_elems || a->window > 0) return 1;   // the forms of layered decoders only
+  if (dv != a->head_dim || a->softcap > 0.f || a->gate_elems || a->window > 0 || a->sink != nullptr) return 1;   // the forms of layered decoders only
   if (a->head_dim == 128) return ts ? launch<128, 128, true, false>(*a, G, s) : launch<128, 128, false, false>(*a, G, s);
   if (a->head_dim == 64) return ts ? launch<64, 64, true, false>(*a, G, s) : launch<64, 64, false, false>(*a, G, s);
   return 1;

@@ -290,6 +290,8 @@ extern "C" int xp_gemm_plan(const XpGemmArgs* a, XpGemmPlan* plan) {
   const int batch = a->batch > 1 ? a->batch : 1;
   if (batch > 1 && (whole || a->tile_table != nullptr || a->dual || a->epilogue == gemm::kEpiResidual || a->bias != nullptr || a->x_group_rows < a->rows)) return -16;
   if (a->epilogue == gemm::kEpiGateMul && (a->dual || batch > 1 || a->tile_table != nullptr || a->resid == nullptr)) return -17;
+  if (a->epilogue == gemm::kEpiSigmoid && (a->dual || a->tile_table != nullptr || a->resid == nullptr)) return -17;
+  if (a->relu2 && a->epilogue != gemm::kEpiStore) return -19;
   if (a->tail != nullptr && (a->epilogue != gemm::kEpiStore || batch > 1 || a->tile_table != nullptr)) return -18;
   if (a->fp8 && (a->dual || a->w_tiled || a->tile_table != nullptr || a->w_scale == nullptr || a->x_scale == nullptr ||
                  a->ld_xscale % 4 != 0 || a->bn > gemm::kMaxBnF8))
@@ -402,6 +404,7 @@ extern "C" int xp_gemm(const XpGemmArgs* a) {
   p.tail = a->tail;
   p.tail_from = a->tail_from;
   p.ld_tail = a->ld_tail;
+  p.relu2 = a->relu2;
   if (a->tile_table != nullptr) {
     if (plan.splits != 1) return -13;
     plan.grid = plan.smem_bytes > 0 ? 148 : 148;
@@ -420,7 +423,7 @@ extern "C" int xp_gemm(const XpGemmArgs* a) {
       return -30;
     attr_set[dev] = true;
   }
-  const bool wide = p.act_cubic != 0.f || p.epilogue == gemm::kEpiGateMul || p.tail != nullptr;
+  const bool wide = p.act_cubic != 0.f || p.epilogue == gemm::kEpiGateMul || p.epilogue == gemm::kEpiSigmoid || p.tail != nullptr || p.relu2 != 0;
   auto kernel = wide ? gemm::gemm_ws_kernel<true> : gemm::gemm_ws_kernel<false>;
   kernel<<<plan.grid, gemm::kThreads, plan.smem_bytes, reinterpret_cast<cudaStream_t>(a->stream)>>>(tw, tx, p, plan.nacc, plan.smem_budget, a->status);
   cudaError_t e = cudaGetLastError();

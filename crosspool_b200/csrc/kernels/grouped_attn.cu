@@ -1,5 +1,6 @@
-// Grouped-query attention: the row kernel of the form without positions between the projection and the attention kernels, and the plain
-// attention kernel for sizes and types that the tensor-core kernels (attn_decode.cu, attn_prefill_umma.cu) do not cover.
+// Grouped-query attention: the row kernel between the projection and the attention kernels (norms, rotation, cache rows, query
+// layout), the means of pooled blocks, and the plain attention kernel for sizes and types that the tensor-core kernels
+// (attn_decode.cu, attn_prefill_umma.cu) do not cover.
 #include <math_constants.h>
 
 #include "xpool/elem.cuh"
@@ -14,53 +15,188 @@ using elem::st;
 constexpr int kPrepThreads = 256;
 constexpr int kAttnWarps = 4;
 
-// One warp per head slot of a row: padded query heads, then keys, then values.
-template <typename T>
+// N elements at a time: 16 bytes where the layouts allow it, else one.
+template <int N, typename T>
+__device__ __forceinline__ void load_n(const T* p, float (&v)[N]) {
+  if constexpr (N == 8) {
+    float lo[4], hi[4];
+    const uint4 x = *reinterpret_cast<const uint4*>(p);
+    const uint2 h[2] = {make_uint2(x.x, x.y), make_uint2(x.z, x.w)};
+    elem::ldv<4>(reinterpret_cast<const T*>(&h[0]), lo);
+    elem::ldv<4>(reinterpret_cast<const T*>(&h[1]), hi);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) v[j] = lo[j], v[4 + j] = hi[j];
+  } else {
+    elem::ldv<N>(p, v);
+  }
+}
+template <int N, typename T>
+__device__ __forceinline__ void store_n(T* p, const float (&v)[N]) {
+  if constexpr (N == 8) {
+    float lo[4], hi[4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) lo[j] = v[j], hi[j] = v[4 + j];
+    uint2 h[2];
+    elem::stv<4>(reinterpret_cast<T*>(&h[0]), lo);
+    elem::stv<4>(reinterpret_cast<T*>(&h[1]), hi);
+    *reinterpret_cast<uint4*>(p) = make_uint4(h[0].x, h[0].y, h[1].x, h[1].y);
+  } else {
+    elem::stv<N>(p, v);
+  }
+}
+
+// Row of a paged cache of `heads` heads of `width` elements.
+__device__ __forceinline__ size_t paged_row(const int* table, int t, int page_size, int heads, int h, int width) {
+  return ((static_cast<size_t>(table[t / page_size]) * page_size + t % page_size) * heads + h) * width;
+}
+
+// Mean of the `pool` cached rows that end with token `last`, elements c .. c + N - 1 of head h. `own`, where given, is what the
+// cache holds for the last token.
+template <int N, typename T>
+__device__ __forceinline__ void block_mean(const T* cache, const int* table, int last, int pool, int page_size, int heads, int h, int width, int c,
+                                           const float* own, float (&mean)[N]) {
+#pragma unroll
+  for (int j = 0; j < N; ++j) mean[j] = 0.f;
+  const int stop = own != nullptr ? last : last + 1;
+  for (int t = last + 1 - pool; t < stop; t += 4) {  // four rows in flight
+    float v[4][N];
+#pragma unroll
+    for (int u = 0; u < 4; ++u) load_n<N>(cache + paged_row(table, min(t + u, stop - 1), page_size, heads, h, width) + c, v[u]);
+#pragma unroll
+    for (int u = 0; u < 4; ++u)
+#pragma unroll
+      for (int j = 0; j < N; ++j) mean[j] += t + u < stop ? v[u][j] : 0.f;
+  }
+#pragma unroll
+  for (int j = 0; j < N; ++j) mean[j] = (own != nullptr ? mean[j] + own[j] : mean[j]) / static_cast<float>(pool);
+}
+
+// L lanes per head slot of a row: padded query heads, then keys, then values. A lane takes N elements at a time.
+template <typename T, int N, int L>
 __global__ void __launch_bounds__(kPrepThreads)
 grouped_prep_kernel(XpGroupedPrepArgs a) {
   const int per_row = a.kv_heads * (a.group_pad + 2);
-  const int64_t unit = static_cast<int64_t>(blockIdx.x) * (kPrepThreads / 32) + (threadIdx.x >> 5);
-  const int lane = threadIdx.x & 31;
-  if (unit >= static_cast<int64_t>(a.rows) * per_row) return;
-  const int row = static_cast<int>(unit / per_row), u = static_cast<int>(unit % per_row);
+  const int64_t unit = (static_cast<int64_t>(blockIdx.x) * kPrepThreads + threadIdx.x) / L;
+  const int lane = threadIdx.x % L;
+  const bool on = unit < static_cast<int64_t>(a.rows) * per_row;
+  const int row = on ? static_cast<int>(unit / per_row) : 0, u = on ? static_cast<int>(unit % per_row) : 0;
   const int nq = a.kv_heads * a.group_pad;
   const T* proj = reinterpret_cast<const T*>(a.proj) + static_cast<size_t>(row) * a.ld_proj;
   const T* src = nullptr;
-  T* dst;
-  const float* norm = nullptr;
-  int n, width;
+  T* dst = nullptr;
+  const T* cache = nullptr;                          // of a key or value head
+  const float* weight = nullptr;
+  bool query_or_key = true;
+  int n, width, h = 0;
   if (u < nq) {
     const int group = a.heads / a.kv_heads, g = u % a.group_pad;
     if (g < group) src = proj + a.q_off + (u / a.group_pad * group + g) * a.dim;
     dst = reinterpret_cast<T*>(a.q_out) + (static_cast<size_t>(row) * nq + u) * a.dq;
-    norm = a.q_norm, n = a.dim, width = a.dq;
+    weight = a.q_norm, n = a.dim, width = a.dq;
   } else {
     const int slot = a.slots[row];
-    if (slot < 0) return;
-    const bool is_k = u < nq + a.kv_heads;
-    const int h = u - nq - (is_k ? 0 : a.kv_heads);
-    n = is_k ? a.dim : a.vdim;
-    width = is_k ? a.dq : a.dv;
-    src = proj + (is_k ? a.k_off : a.v_off) + h * n;
-    dst = reinterpret_cast<T*>(is_k ? a.k_cache : a.v_cache) + (static_cast<size_t>(slot) * a.kv_heads + h) * width;
-    if (is_k) norm = a.k_norm;
+    query_or_key = u < nq + a.kv_heads;
+    h = u - nq - (query_or_key ? 0 : a.kv_heads);
+    n = query_or_key ? a.dim : a.vdim;
+    width = query_or_key ? a.dq : a.dv;
+    src = proj + (query_or_key ? a.k_off : a.v_off) + h * n;
+    cache = reinterpret_cast<const T*>(query_or_key ? a.k_cache : a.v_cache);
+    if (slot >= 0) dst = const_cast<T*>(cache) + (static_cast<size_t>(slot) * a.kv_heads + h) * width;
+    if (query_or_key) weight = a.k_norm;
   }
+  const bool work = on && dst != nullptr, read = work && src != nullptr;
+  const int c0 = lane * N;
+  float first[N];
+#pragma unroll
+  for (int j = 0; j < N; ++j) first[j] = 0.f;
+  if (read && c0 < n) load_n<N>(src + c0, first);
+  auto get = [&](int c, float (&x)[N]) {
+    if (c == c0) {
+#pragma unroll
+      for (int j = 0; j < N; ++j) x[j] = first[j];
+    } else {
+      load_n<N>(src + c, x);
+    }
+  };
   float inv = 1.f;
-  if (src != nullptr && norm != nullptr) {
+  if (a.norm) {
     float ss = 0.f;
-    for (int c = lane; c < n; c += 32) {
-      const float x = ld(src + c);
-      ss += x * x;
-    }
-    inv = rsqrtf(elem::warp_sum(ss) / static_cast<float>(n) + a.eps);
+    if (read && query_or_key)
+      for (int c = c0; c < n; c += L * N) {
+        float x[N];
+        get(c, x);
+#pragma unroll
+        for (int j = 0; j < N; ++j) ss += x[j] * x[j];
+      }
+#pragma unroll
+    for (int o = L / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    if (query_or_key) inv = rsqrtf(ss / static_cast<float>(n) + a.eps);
   }
-  for (int c = lane; c < width; c += 32) {
-    float x = 0.f;
+  if (!work) return;
+  const int rotated = query_or_key ? 2 * a.rot_pairs : 0;
+  const int pos = a.positions != nullptr ? a.positions[row] : 0;
+  const float2* turn = reinterpret_cast<const float2*>(a.rot) + static_cast<size_t>(pos < a.rot_positions ? pos : 0) * a.rot_pairs;
+  const bool means = cache != nullptr && a.pool > 0 && row < a.pool_rows && (pos + 1) % a.pool == 0;
+  for (int c = c0; c < width; c += L * N) {
+    float x[N];
+#pragma unroll
+    for (int j = 0; j < N; ++j) x[j] = 0.f;
     if (src != nullptr && c < n) {
-      x = ld(src + c);
-      if (norm != nullptr) x *= inv * norm[c];
+      get(c, x);
+      if (query_or_key) {
+#pragma unroll
+        for (int j = 0; j < N; ++j) x[j] *= weight != nullptr ? inv * weight[c + j] : inv;
+        if (c < rotated) {
+          float y[N];
+#pragma unroll
+          for (int j = 0; j < N; ++j) {
+            const int e = c + j;
+            y[j] = x[j];
+            if (e >= rotated) continue;
+            const bool second = a.interleaved ? e & 1 : e >= a.rot_pairs;
+            const int pair = a.interleaved ? e >> 1 : second ? e - a.rot_pairs : e;
+            float other;
+            if (a.interleaved && N > 1) {
+              other = x[j ^ (N > 1 ? 1 : 0)];
+            } else {
+              const int o = a.interleaved ? e ^ 1 : second ? e - a.rot_pairs : e + a.rot_pairs;
+              other = ld(src + o) * (weight != nullptr ? inv * weight[o] : inv);
+            }
+            const float2 t = turn[pair];
+            y[j] = second ? x[j] * t.x + other * t.y : x[j] * t.x - other * t.y;
+          }
+#pragma unroll
+          for (int j = 0; j < N; ++j) x[j] = y[j];
+        }
+      }
     }
-    st(dst + c, x);
+    store_n<N>(dst + c, x);
+    if (means) {
+      float own[N], mean[N];
+      T held[N];
+#pragma unroll
+      for (int j = 0; j < N; ++j) st(&held[j], x[j]), own[j] = ld(&held[j]);
+      const int* table = a.block_table + static_cast<size_t>(row) * a.max_blocks;
+      block_mean<N>(cache, table, pos, a.pool, a.page_size, a.kv_heads, h, width, c, own, mean);
+      store_n<N>(reinterpret_cast<T*>(query_or_key ? a.k_pool : a.v_pool) + paged_row(table, pos / a.pool, a.pool_page, a.kv_heads, h, width) + c, mean);
+    }
+  }
+}
+
+// One CTA per row; most rows complete no block.
+template <typename T, int N>
+__global__ void __launch_bounds__(128)
+block_mean_kernel(XpBlockMeanArgs a) {
+  const int row = blockIdx.x, pos = a.positions[row];
+  if (a.slots[row] < 0 || (pos + 1) % a.pool != 0) return;
+  const int* table = a.block_table + static_cast<size_t>(a.row_seq != nullptr ? a.row_seq[row] : row) * a.max_blocks;
+  const int nk = a.kv_heads * a.dq, total = nk + a.kv_heads * a.dv;
+  for (int i = threadIdx.x * N; i < total; i += 128 * N) {
+    const bool is_k = i < nk;
+    const int width = is_k ? a.dq : a.dv, e = is_k ? i : i - nk, h = e / width, c = e % width;
+    float mean[N];
+    block_mean<N>(reinterpret_cast<const T*>(is_k ? a.k_cache : a.v_cache), table, pos, a.pool, a.page_size, a.kv_heads, h, width, c, nullptr, mean);
+    store_n<N>(reinterpret_cast<T*>(is_k ? a.k_pool : a.v_pool) + paged_row(table, pos / a.pool, a.pool_page, a.kv_heads, h, width) + c, mean);
   }
 }
 
@@ -87,16 +223,21 @@ grouped_attn_kernel(XpGroupedAttnArgs a) {
   const int len = a.positions[row] + 1;
   const T* kc = reinterpret_cast<const T*>(a.k_cache);
   const T* vc = reinterpret_cast<const T*>(a.v_cache);
-  // the kept first tokens in whole steps of 32, then the step in which the window begins and those behind it
+  // the kept first tokens (or the pooled blocks) in whole steps of 32, then the step in which the window begins and those behind it
   const int lo = a.window > 0 && len > a.window ? len - a.window : 0;
-  const int head = min((a.keep_first + 31) / 32, lo / 32) * 32, skip = lo / 32 * 32 - head;
-  float m = -CUDART_INF_F, l = 0.f;
+  const int blocks = a.pool > 0 ? lo / a.pool : 0;
+  const int head = a.pool > 0 ? (blocks + 31) / 32 * 32 : min((a.keep_first + 31) / 32, lo / 32) * 32, skip = lo / 32 * 32 - head;
+  const bool sig = a.sigmoid_bias != nullptr;
+  const float bias = sig ? a.sigmoid_bias[h] : 0.f;
+  float m = sig ? 0.f : -CUDART_INF_F, l = 0.f;
   for (int v0 = warp * 32; v0 + (v0 < head ? 0 : skip) < len; v0 += kAttnWarps * 32) {
-    const int t0 = v0 + (v0 < head ? 0 : skip), t = t0 + lane;
-    const bool on = t < len && (t >= lo || t < a.keep_first);
-    const int tt = t < len ? t : t0;
-    const size_t tok = (static_cast<size_t>(table[tt / a.page_size]) * a.page_size + tt % a.page_size) * a.kv_heads + hk;
-    const T* k = kc + tok * a.dq;
+    const bool pooled = a.pool > 0 && v0 < head;
+    const int t0 = v0 + (v0 < head ? 0 : skip), t = t0 + lane, stop = pooled ? blocks : len;
+    const bool on = t < stop && (pooled || t >= lo || t < a.keep_first);
+    const int tt = t < stop ? t : t0;
+    const size_t tok = paged_row(table, tt, pooled ? a.pool_page : a.page_size, a.kv_heads, hk, 1);
+    const T* k = (pooled ? reinterpret_cast<const T*>(a.k_pool) : kc) + tok * a.dq;
+    const T* vals = pooled ? reinterpret_cast<const T*>(a.v_pool) : vc;
     float s = 0.f;
     for (int c = 0; c < a.dim; ++c) s = fmaf(q_s[c], ld(k + c), s);
     if (a.softcap > 0.f) s = a.softcap * tanhf(s / a.softcap);
@@ -104,17 +245,17 @@ grouped_attn_kernel(XpGroupedAttnArgs a) {
     float mx = s;
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
-    const float mn = fmaxf(m, mx), corr = m == -CUDART_INF_F ? 0.f : expf(m - mn);
-    const float p = on ? expf(s - mn) : 0.f;
+    const float mn = sig ? 0.f : fmaxf(m, mx), corr = sig ? 1.f : m == -CUDART_INF_F ? 0.f : expf(m - mn);
+    const float p = !on ? 0.f : sig ? elem::sigmoid(s + bias) : expf(s - mn);
     l = l * corr + elem::warp_sum(p);
     m = mn;
-    const int live = min(32, len - t0);
+    const int live = min(32, stop - t0);
     for (int c = lane; c - lane < a.vdim; c += 32) {       // every lane takes part in the shuffles
       float v = c < a.vdim ? acc_s[c] * corr : 0.f;
       for (int j = 0; j < live; ++j) {
         const float pj = __shfl_sync(0xffffffffu, p, j);
         const size_t tj = __shfl_sync(0xffffffffu, static_cast<unsigned long long>(tok), j);
-        if (c < a.vdim) v = fmaf(pj, ld(vc + tj * a.dv + c), v);
+        if (c < a.vdim) v = fmaf(pj, ld(vals + tj * a.dv + c), v);
       }
       if (c < a.vdim) acc_s[c] = v;
     }
@@ -129,7 +270,12 @@ grouped_attn_kernel(XpGroupedAttnArgs a) {
     const float mw = all[w * step + a.vdim];
     if (mw != -CUDART_INF_F) ll += all[w * step + a.vdim + 1] * expf(mw - mm);
   }
-  float f = 1.f / ll;
+  if (a.sink != nullptr) {
+    const float top = fmaxf(mm, a.sink[h]);
+    ll = ll * expf(mm - top) + expf(a.sink[h] - top);
+    mm = top;
+  }
+  float f = sig ? 1.f : 1.f / ll;
   const T* gate = a.gate != nullptr ? reinterpret_cast<const T*>(a.gate) + static_cast<size_t>(row) * a.ld_gate : nullptr;
   if (gate != nullptr && !a.gate_elems) f *= elem::sigmoid(ld(gate + h));
   for (int c = threadIdx.x; c < a.vdim; c += kAttnWarps * 32) {
@@ -156,17 +302,53 @@ using namespace xpool::grouped;
 extern "C" int xp_grouped_prep(const XpGroupedPrepArgs* a, void* stream) {
   if (a->rows <= 0) return 0;
   if (a->kv_heads <= 0 || a->heads % a->kv_heads != 0 || a->group_pad < a->heads / a->kv_heads || a->dq < a->dim || a->dv < a->vdim) return -10;
-  const int64_t units = static_cast<int64_t>(a->rows) * a->kv_heads * (a->group_pad + 2);
-  const unsigned grid = static_cast<unsigned>((units + kPrepThreads / 32 - 1) / (kPrepThreads / 32));
+  if (a->rot_pairs < 0 || 2 * a->rot_pairs > a->dim || (a->rot_pairs > 0 && (a->rot == nullptr || a->rot_positions <= 0 || a->positions == nullptr))) return -12;
+  if (a->pool > 0 && (a->pool_rows > a->rows || a->positions == nullptr || a->block_table == nullptr || a->k_pool == nullptr || a->v_pool == nullptr ||
+                      a->pool_page <= 0 || a->page_size <= 0))
+    return -13;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
-  if (a->f32) grouped_prep_kernel<float><<<grid, kPrepThreads, 0, s>>>(*a);
-  else grouped_prep_kernel<__nv_bfloat16><<<grid, kPrepThreads, 0, s>>>(*a);
+  auto al = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
+  const int n = a->f32 ? 4 : 8;
+  const bool v = a->dim % n == 0 && a->vdim % n == 0 && a->dq % n == 0 && a->dv % n == 0 && a->ld_proj % n == 0 && a->q_off % n == 0 && a->k_off % n == 0 &&
+                 a->v_off % n == 0 && al(a->proj) && al(a->k_cache) && al(a->v_cache) && al(a->q_out) && al(a->k_pool) && al(a->v_pool);
+  const int widest = a->dq > a->dv ? a->dq : a->dv;
+  const int64_t units = static_cast<int64_t>(a->rows) * a->kv_heads * (a->group_pad + 2);
+  auto run = [&](auto kernel, int lanes) {
+    kernel<<<static_cast<unsigned>((units * lanes + kPrepThreads - 1) / kPrepThreads), kPrepThreads, 0, s>>>(*a);
+  };
+  if (a->f32) {
+    if (!v) run(grouped_prep_kernel<float, 1, 32>, 32);
+    else if (widest <= 64) run(grouped_prep_kernel<float, 4, 16>, 16);
+    else run(grouped_prep_kernel<float, 4, 32>, 32);
+  } else {
+    if (!v) run(grouped_prep_kernel<__nv_bfloat16, 1, 32>, 32);
+    else if (widest <= 64) run(grouped_prep_kernel<__nv_bfloat16, 8, 8>, 8);
+    else run(grouped_prep_kernel<__nv_bfloat16, 8, 16>, 16);
+  }
+  return done();
+}
+
+extern "C" int xp_block_mean(const XpBlockMeanArgs* a, void* stream) {
+  if (a->rows <= 0) return 0;
+  if (a->pool <= 0 || a->pool_page <= 0 || a->page_size <= 0 || a->kv_heads <= 0) return -10;
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  auto al = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
+  const int n = a->f32 ? 4 : 8;
+  const bool v = a->dq % n == 0 && a->dv % n == 0 && al(a->k_cache) && al(a->v_cache) && al(a->k_pool) && al(a->v_pool);
+  if (a->f32) {
+    if (v) block_mean_kernel<float, 4><<<a->rows, 128, 0, s>>>(*a);
+    else block_mean_kernel<float, 1><<<a->rows, 128, 0, s>>>(*a);
+  } else {
+    if (v) block_mean_kernel<__nv_bfloat16, 8><<<a->rows, 128, 0, s>>>(*a);
+    else block_mean_kernel<__nv_bfloat16, 1><<<a->rows, 128, 0, s>>>(*a);
+  }
   return done();
 }
 
 extern "C" int xp_grouped_attn(const XpGroupedAttnArgs* a, void* stream) {
   if (a->rows <= 0) return 0;
   if (a->kv_heads <= 0 || a->heads % a->kv_heads != 0 || a->rows > 65535) return -10;
+  if (a->pool > 0 && (a->window <= 0 || a->keep_first > 0 || a->pool_page <= 0 || a->k_pool == nullptr || a->v_pool == nullptr)) return -12;
   const size_t smem = static_cast<size_t>(a->dim + kAttnWarps * (a->vdim + 2)) * 4;
   if (smem > 48 * 1024) return -11;
   const dim3 grid(a->heads, a->rows);

@@ -45,14 +45,26 @@ latent_prep_kernel(XpLatentPrepArgs a) {
     cs[half + i] = s;
   }
   __syncthreads();
-  // element j of a vector x whose first rot_dims elements are rotated in pairs (j, j + half)
+  // element j of a vector x whose first rot_dims elements are rotated in pairs (j, j + half), or of neighbours
   auto rotated = [&](const T* x, int j) -> float {
     const float v = elem::ld(x + j);
     if (j >= a.rot_dims) return v;
-    const int i = j < half ? j : j - half;
-    const float o = elem::ld(x + (j < half ? j + half : i));
-    return j < half ? v * cs[i] - o * cs[half + i] : v * cs[i] + o * cs[half + i];
+    const bool first = a.interleaved ? (j & 1) == 0 : j < half;
+    const int i = a.interleaved ? j >> 1 : first ? j : j - half;
+    const float o = elem::ld(x + (a.interleaved ? j ^ 1 : first ? j + half : i));
+    return first ? v * cs[i] - o * cs[half + i] : v * cs[i] + o * cs[half + i];
   };
+  float q_inv = 1.f;                        // queries made from a latent lack its norm
+  if (a.q_rank > 0) {
+    float ss = 0.f;
+    for (int c = threadIdx.x * VEC; c < a.q_rank; c += kPrepThreads * VEC) {
+      float v[VEC];
+      elem::ldv<VEC>(proj + a.ql_off + c, v);
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) ss += v[j] * v[j];
+    }
+    q_inv = rsqrtf(elem::block_sum<kPrepThreads>(ss, red) / static_cast<float>(a.q_rank) + a.eps);
+  }
 
   const int slot = a.slots[row];
   if (slot >= 0 && blockIdx.y == 0) {
@@ -76,7 +88,7 @@ latent_prep_kernel(XpLatentPrepArgs a) {
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int dh = a.dim + a.rot;
   for (int h = blockIdx.y * kPrepHeads + warp; h < min(a.heads, static_cast<int>(blockIdx.y + 1) * kPrepHeads); h += kPrepThreads / 32) {
-    const T* q = proj + a.q_off + h * dh;
+    const T* q = (a.q != nullptr ? reinterpret_cast<const T*>(a.q) + static_cast<size_t>(row) * a.ld_q : proj + a.q_off) + h * dh;
     T *plain, *rot;
     int plain_end, rot_end;                 // columns past the vector's own hold zeros
     if (row < a.abs_rows) {
@@ -95,13 +107,15 @@ latent_prep_kernel(XpLatentPrepArgs a) {
       for (int c = lane * 4; c < a.dim; c += 128) {
         float v[4];
         elem::ldv<4>(q + c, v);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) v[j] *= q_inv;
         elem::stv<4>(plain + c, v);
       }
       for (int c = a.dim + lane; c < plain_end; c += 32) elem::st(plain + c, 0.f);
     } else {
-      for (int c = lane; c < plain_end; c += 32) elem::st(plain + c, c < a.dim ? elem::ld(q + c) : 0.f);
+      for (int c = lane; c < plain_end; c += 32) elem::st(plain + c, c < a.dim ? elem::ld(q + c) * q_inv : 0.f);
     }
-    for (int c = lane; c < rot_end; c += 32) elem::st(rot + c, c < a.rot ? rotated(q + a.dim, c) : 0.f);
+    for (int c = lane; c < rot_end; c += 32) elem::st(rot + c, c < a.rot ? rotated(q + a.dim, c) * q_inv : 0.f);
   }
 }
 
@@ -109,6 +123,9 @@ latent_prep_kernel(XpLatentPrepArgs a) {
 constexpr int kSimtThreads = 128;
 constexpr int kSimtTile = 32;
 constexpr int kSimtAcc = 8;              // latent columns per thread: kv_rank <= 1024
+
+// First token that a row at the end of len tokens sees.
+__device__ __forceinline__ int window_start(const XpLatentAttnArgs& a, int len) { return a.window > 0 ? max(0, len - a.window) : 0; }
 
 template <typename T>
 __global__ void __launch_bounds__(kSimtThreads)
@@ -135,7 +152,7 @@ latent_attn_simt_kernel(XpLatentAttnArgs a) {
   float m = -CUDART_INF_F, l = 0.f, acc[kSimtAcc];
 #pragma unroll
   for (int j = 0; j < kSimtAcc; ++j) acc[j] = 0.f;
-  for (int t0 = 0; t0 < len; t0 += kSimtTile) {
+  for (int t0 = window_start(a, len); t0 < len; t0 += kSimtTile) {
     const int n = min(kSimtTile, len - t0);
     for (int j = warp; j < n; j += kSimtThreads / 32) {
       const T* k = token_row(t0 + j);
@@ -274,7 +291,7 @@ latent_attn_tc_kernel(XpLatentAttnArgs a) {
   const bool pad = a.slots[row] < 0;
   const int len = pad ? 0 : a.positions[row] + 1;
   const int chunk = a.chunk_tokens > 0 ? a.chunk_tokens : len;
-  const int t0 = split * chunk, t1 = a.num_splits > 1 ? min(len, t0 + chunk) : len;
+  const int t0 = window_start(a, len) + split * chunk, t1 = a.num_splits > 1 ? min(len, t0 + chunk) : len;
   if (a.num_splits > 1 && t0 >= len) return;         // the merge kernel skips this slice
   const int tiles = (t1 - t0 + kTile - 1) / kTile;
   const int* table = a.block_table + static_cast<size_t>(a.row_seq != nullptr ? a.row_seq[row] : row) * a.max_blocks;
@@ -523,7 +540,7 @@ latent_merge_kernel(XpLatentAttnArgs a) {
   const int h = blockIdx.x, row = blockIdx.y;
   const bool pad = a.slots[row] < 0;
   const int len = pad ? 0 : a.positions[row] + 1;
-  const int n = min(a.num_splits, (len + a.chunk_tokens - 1) / a.chunk_tokens);
+  const int n = min(a.num_splits, (len - window_start(a, len) + a.chunk_tokens - 1) / a.chunk_tokens);
   const float* w = a.ws + (static_cast<size_t>(row) * a.heads + h) * a.num_splits * (a.kv_rank + 2);
   float m = -CUDART_INF_F, l = 0.f;
   for (int s = 0; s < n; ++s) m = fmaxf(m, w[s * (a.kv_rank + 2) + a.kv_rank]);
@@ -545,7 +562,8 @@ constexpr int kGatherTokens = 4;
 __global__ void __launch_bounds__(128)
 latent_gather_kernel(XpLatentGatherArgs a) {
   const int seq = blockIdx.y;
-  const int len = a.ctx_lens[seq] + a.q_lens[seq];
+  const int ctx = a.ctx_lens[seq], base = a.window > 0 ? max(0, ctx - a.window + 1) & ~63 : 0;
+  const int len = ctx + a.q_lens[seq] - base;
   const int row_bytes = a.ld_cache * a.elem_bytes;   // a multiple of 16
   const int* table = a.block_table + static_cast<size_t>(seq) * a.max_blocks;
   const uint8_t* cache = static_cast<const uint8_t*>(a.cache);
@@ -553,8 +571,8 @@ latent_gather_kernel(XpLatentGatherArgs a) {
   const int per = row_bytes / 16;
   const int t0 = blockIdx.x * kGatherTokens, n = min(kGatherTokens, len - t0);
   for (int u = threadIdx.x; u < n * per; u += 128) {
-    const int t = t0 + u / per, c = u % per;
-    const size_t src = (static_cast<size_t>(table[t / a.page_size]) * a.page_size + t % a.page_size) * row_bytes;
+    const int t = t0 + u / per, c = u % per, from = base + t;
+    const size_t src = (static_cast<size_t>(table[from / a.page_size]) * a.page_size + from % a.page_size) * row_bytes;
     *reinterpret_cast<uint4*>(out + static_cast<size_t>(t) * row_bytes + c * 16) =
         __ldg(reinterpret_cast<const uint4*>(cache + src + c * 16));
   }
@@ -591,6 +609,7 @@ extern "C" int xp_latent_prep(const XpLatentPrepArgs* a, void* stream) {
   if (a->abs_rows > 0 && (a->q_plain == nullptr || a->q_abs == nullptr || a->ld_abs < a->kv_rank + a->rot || a->abs_rows > a->qp_rows ||
                           a->dim_p < a->dim))
     return -11;
+  if (a->q == nullptr ? a->q_rank > 0 : a->ld_q < a->heads * (a->dim + a->rot)) return -13;
   if (a->abs_rows < a->rows && (a->q_exp == nullptr || a->dq_pad < a->dim + a->rot)) return -12;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   const size_t sm = static_cast<size_t>(a->rot_dims > 0 ? a->rot_dims : 1) * 4;
@@ -598,7 +617,7 @@ extern "C" int xp_latent_prep(const XpLatentPrepArgs* a, void* stream) {
   const int eb = a->f32 ? 4 : 2;
   auto al = [&](const void* p) { return reinterpret_cast<uintptr_t>(p) % (4 * eb) == 0; };
   const bool v = a->dim % 4 == 0 && a->rot % 4 == 0 && a->ld_proj % 4 == 0 && a->q_off % 4 == 0 && a->dim_p % 4 == 0 && a->dq_pad % 4 == 0 &&
-                 al(a->proj) && al(a->q_plain) && al(a->q_exp);
+                 al(a->proj) && al(a->q_plain) && al(a->q_exp) && al(a->q) && a->ld_q % 4 == 0 && a->q_rank % 4 == 0 && a->ql_off % 4 == 0;
   dim3 grid(a->rows, (a->heads + kPrepHeads - 1) / kPrepHeads);
   if (a->f32) {
     if (v) latent_prep_kernel<float, 4><<<grid, kPrepThreads, sm, s>>>(*a);

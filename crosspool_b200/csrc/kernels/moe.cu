@@ -41,7 +41,10 @@ __device__ __forceinline__ void router_topk_row(const XpRouterArgs& a, int row, 
     score[j] = v;
     mx = fmaxf(mx, v);
   }
-  if (a.sigmoid) {
+  if (a.sigmoid == 2) {
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+  } else if (a.sigmoid) {
 #pragma unroll
     for (int j = 0; j < kMaxPerLane; ++j) score[j] = (lane + 32 * j < E) ? 1.f / (1.f + __expf(-score[j])) : -CUDART_INF_F;
   } else {
@@ -64,6 +67,10 @@ __device__ __forceinline__ void router_topk_row(const XpRouterArgs& a, int row, 
     const int e = lane + 32 * j;
     sel[j] = (e < E) ? score[j] + (a.correction_bias != nullptr ? a.correction_bias[e] : 0.f) : -CUDART_INF_F;
   }
+  if (a.sigmoid == 2) {                              // chosen by their logits; scores on the scale of the largest
+#pragma unroll
+    for (int j = 0; j < kMaxPerLane; ++j) score[j] = (lane + 32 * j < E) ? expf(score[j] - mx) : 0.f;
+  }
   float wsum = 0.f;
   float my_w = 0.f;
   int my_id = -1;
@@ -74,7 +81,7 @@ __device__ __forceinline__ void router_topk_row(const XpRouterArgs& a, int row, 
 #pragma unroll
     for (int j = 0; j < kMaxPerLane; ++j) {
       const int e = lane + 32 * j;
-      const bool better = sel[j] > bv || (sel[j] == bv && be >= 0 && (a.sigmoid ? e > be : e < be));
+      const bool better = sel[j] > bv || (sel[j] == bv && be >= 0 && (a.sigmoid == 1 ? e > be : e < be));
       if (e < E && better) {
         bv = sel[j];
         be = e;
@@ -86,7 +93,7 @@ __device__ __forceinline__ void router_topk_row(const XpRouterArgs& a, int row, 
       const float ov = __shfl_xor_sync(0xffffffffu, bv, o);
       const int oe = __shfl_xor_sync(0xffffffffu, be, o);
       const float os = __shfl_xor_sync(0xffffffffu, bs, o);
-      const bool better = oe >= 0 && (be < 0 || ov > bv || (ov == bv && (a.sigmoid ? oe > be : oe < be)));
+      const bool better = oe >= 0 && (be < 0 || ov > bv || (ov == bv && (a.sigmoid == 1 ? oe > be : oe < be)));
       if (better) {
         bv = ov;
         be = oe;
@@ -281,7 +288,7 @@ mix_kernel(XpMoeMixArgs a) {
       if (pos >= 0 || id >= a.experts) w = a.weights[t * a.top_k + k];
     } else if (k < n) {
       row = reinterpret_cast<const T*>(a.shared) + static_cast<size_t>(t) * a.ld_shared;
-      w = elem::sigmoid(a.shared_gate[static_cast<size_t>(t) * a.ld_gate]);
+      w = a.shared_gate != nullptr ? elem::sigmoid(a.shared_gate[static_cast<size_t>(t) * a.ld_gate]) : 1.f;
     }
     rows[k] = row, weights[k] = w;
   }
@@ -608,7 +615,7 @@ extern "C" int xp_moe_topk_route(const XpRouterArgs* a, const XpRouteArgs* r, vo
 
 extern "C" int xp_moe_mix(const XpMoeMixArgs* a, void* stream) {
   if (a->rows <= 0) return 0;
-  if (a->hidden <= 0 || a->top_k <= 0 || a->top_k > 32 || (a->shared != nullptr && a->shared_gate == nullptr)) return -10;
+  if (a->hidden <= 0 || a->top_k <= 0 || a->top_k > 32) return -10;
   const int n = a->f32 ? 4 : 8;                      // elements of 16 bytes
   auto fits = [&](const void* p, int ld) { return p == nullptr || (reinterpret_cast<uintptr_t>(p) % 16 == 0 && ld % n == 0); };
   const bool v = a->hidden % n == 0 && fits(a->y, a->ld_y) && fits(a->x, a->ld_x) && fits(a->shared, a->ld_shared) && fits(a->out, a->ld_out);

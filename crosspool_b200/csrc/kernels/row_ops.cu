@@ -5,7 +5,7 @@
 //   post_norm    residual += rmsnorm(sublayer output, or the mean of normed branches) * w [-> norm] -> activation row
 //   head_gate    rmsnorm per head * w * silu(gate) or sigmoid(gate), one warp per head
 //   glu_f32      gated activation of fp32 models (bf16 has it in the product's epilogue)
-//   gate_mul     activation times another row, fp32 models (bf16: the product's epilogue)
+//   gate_mul     activation times another row, row times sigmoid, squared relu; fp32 models (bf16: the product's epilogue)
 // Rows whose pitches allow it are moved four elements at a time.
 #include "xpool/elem.cuh"
 #include "xpool/mixer_api.h"
@@ -336,8 +336,10 @@ __global__ void __launch_bounds__(kThreads)
 gate_mul_f32_kernel(XpGateMulArgs a) {
   const int c = blockIdx.x * kThreads + threadIdx.x;
   if (c >= a.cols) return;
-  for (int r = blockIdx.y; r < a.rows; r += gridDim.y)
-    a.out[static_cast<size_t>(r) * a.ld_out + c] = gated(a.z[static_cast<size_t>(r) * a.ld_z + c], a.alpha, a.cubic) * a.e[static_cast<size_t>(r) * a.ld_e + c];
+  for (int r = blockIdx.y; r < a.rows; r += gridDim.y) {
+    const float z = a.z[static_cast<size_t>(r) * a.ld_z + c], e = a.kind == 2 ? 0.f : a.e[static_cast<size_t>(r) * a.ld_e + c];
+    a.out[static_cast<size_t>(r) * a.ld_out + c] = a.kind == 2 ? fmaxf(z, 0.f) * fmaxf(z, 0.f) : a.kind == 1 ? z * sigmoid(e) : gated(z, a.alpha, a.cubic) * e;
+  }
 }
 
 inline bool vec4(const void* p, int64_t ld, int elem_bytes) {
@@ -461,7 +463,7 @@ extern "C" int xp_glu_f32(const XpGluArgs* a, void* stream) {
 
 extern "C" int xp_gate_mul_f32(const XpGateMulArgs* a, void* stream) {
   if (a->rows <= 0) return 0;
-  if (a->cols <= 0) return -10;
+  if (a->cols <= 0 || a->kind < 0 || a->kind > 2 || (a->kind != 2 && a->e == nullptr)) return -10;
   const dim3 grid((a->cols + kThreads - 1) / kThreads, a->rows < 65535 ? a->rows : 65535);
   gate_mul_f32_kernel<<<grid, kThreads, 0, reinterpret_cast<cudaStream_t>(stream)>>>(*a);
   return done();

@@ -448,13 +448,13 @@ class AttentionEngine:
         while start < n and room:
             used, i = 0, start
             while i < n:
-                need = (chosen[i][0].computed + chosen[i][1] + 63) // 64 * 64
+                need = self.body.expand_rows(chosen[i][0].computed, chosen[i][1])
                 if used + need > room:
                     break
                 used += need
                 i += 1
             part = chosen[start:i]
-            groups.append(ExpandGroup(start, i - start, max(s.computed + c for s, c in part), max(c for _, c in part), used))
+            groups.append(ExpandGroup(start, i - start, max(self.body.expand_rows(s.computed, c) for s, c in part), max(c for _, c in part), used))
             start = i
         batch = RowBatch(
             rows, n, n_dec, n_abs, len(short), max((c for _, c in chosen[n_dec:]), default=0),
@@ -475,7 +475,7 @@ class AttentionEngine:
             row += n
             hv[r + P + i] = self.kv.seq_slots.get(s.seq_id, 0)
             if n > SHORT_PORTION:
-                need = (s.computed + n + 63) // 64 * 64
+                need = self.body.expand_rows(s.computed, n)
                 if used + need > self.body.ws_tokens:
                     used = 0                       # the next group reuses the workspace from its start
                 hv[r + P + S + i] = used

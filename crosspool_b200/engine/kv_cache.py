@@ -15,11 +15,12 @@ sequence (:class:`StateSlots`) in those with a recurrence (a layer can have both
 
 from __future__ import annotations
 
+import math
 from dataclasses import dataclass, field
 
 import torch
 
-from ..models.config import ModelConfig, sub_mixers
+from ..models.config import GroupedMixer, ModelConfig, sub_mixers
 
 
 class OutOfPages(RuntimeError):
@@ -133,6 +134,7 @@ class KvLayout:
     num_layers: int
     elem_bytes: int = 2
     row_widths: tuple[int, ...] = ()   # layered decoders: elements of one token's row per layer (0: the layer caches none)
+    pool_elems: int = 0                # block means beside one page, all layers
 
     @property
     def page_bytes_per_buffer(self) -> int:
@@ -145,7 +147,7 @@ class KvLayout:
     @property
     def bytes_per_page_all_layers(self) -> int:
         if self.row_widths:
-            return self.page_size * sum(self.row_widths) * self.elem_bytes
+            return (self.page_size * sum(self.row_widths) + self.pool_elems) * self.elem_bytes
         return 2 * self.num_layers * self.page_bytes_per_buffer
 
 
@@ -161,6 +163,10 @@ class PagedKvCache:
     states: list[torch.Tensor | None] = field(default_factory=list)
     # convolution inputs behind every live sequence, [slots, taps, channels] per layer: the input at position p is entry p % taps
     conv: list[torch.Tensor | None] = field(default_factory=list)
+    # layers that pool: means of keys and of values of whole token blocks, [pages, rows beside a page, kv heads, head]; the blocks of
+    # a sequence fill the rows beside its pages in order
+    k_pool: list[torch.Tensor | None] = field(default_factory=list)
+    v_pool: list[torch.Tensor | None] = field(default_factory=list)
     slots: StateSlots | None = None
     seq_slots: dict[int, int] = field(default_factory=dict)
 
@@ -178,10 +184,12 @@ class PagedKvCache:
     @classmethod
     def _layered(cls, cfg: ModelConfig, num_pages: int, page_size: int, device, dtype: torch.dtype, state_slots: int) -> "PagedKvCache":
         """Pages hold a key row and a value row per token in the layers that cache any (or one latent row that is both); a layer
-        may read another one's instead. Recurrent mixers hold one state per slot, and mixers with a convolution its latest
-        inputs."""
+        may read another one's instead, and layers that pool hold the means of token blocks beside them. Recurrent mixers hold one
+        state per slot, and mixers with a convolution its latest inputs."""
         mixers = [s.mixer for s in cfg.layer_specs]
-        lay = KvLayout(page_size, num_pages, 1, 0, cfg.num_layers, dtype.itemsize, tuple(m.cache_width for m in mixers))
+        pools = [m.pool_shapes(page_size) if isinstance(m, GroupedMixer) else () for m in mixers]
+        lay = KvLayout(page_size, num_pages, 1, 0, cfg.num_layers, dtype.itemsize, tuple(m.cache_width for m in mixers),
+                       sum(math.prod(shape) for p in pools for shape in p))
 
         def rows(m, i: int) -> torch.Tensor | None:
             if len(m.cache_rows) <= i:
@@ -199,7 +207,8 @@ class PagedKvCache:
         for l, m in enumerate(mixers):
             if getattr(m, "kv_from", None) is not None:
                 k[l], v[l] = k[m.kv_from], v[m.kv_from]
-        return cls(lay, k, v, PageAllocator(num_pages), states=states, conv=conv,
+        k_pool, v_pool = ([torch.zeros(num_pages, *p[i], dtype=dtype, device=device) if p else None for p in pools] for i in (0, 1))
+        return cls(lay, k, v, PageAllocator(num_pages), states=states, conv=conv, k_pool=k_pool, v_pool=v_pool,
                    slots=StateSlots(state_slots) if cfg.recurrent else None)
 
     # -- per-sequence page tables --------------------------------------------------------------

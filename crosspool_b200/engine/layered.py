@@ -5,8 +5,9 @@ over all rows together; a mixer splits the rows where its decode and prefill ker
 
 * latent attention: decoded tokens and short portions run in the absorbed form (queries multiplied into the latent space,
   one pass over the cached rows); long portions in the expanded form (the sequence's latents are expanded to per-head keys
-  and values with one product each, then the tcgen05 prefill kernel);
-* grouped-query attention: decoded tokens and short portions as single rows, long portions in the tcgen05 prefill kernel;
+  and values with one product each, then the tcgen05 prefill kernel; of a windowed layer only what the portion sees);
+* grouped-query attention: decoded tokens and short portions as single rows, long portions in the tcgen05 prefill kernel; a layer
+  that pools stores the means of the blocks that the batch completes before it attends;
 * recurrences (decayed linear attention, gated linear attention, gated delta rule, matrix memory): one kernel advances the
   states of the decoded tokens, others those of the portions;
 * a parallel pair runs both of its sides on the columns of one projection.
@@ -40,7 +41,7 @@ class ExpandGroup:
 
     seq0: int
     n: int
-    max_len: int
+    max_len: int      # bound on the workspace rows of a sequence
     max_q: int
     tokens: int       # workspace rows, every sequence starting on a multiple of 64
 
@@ -100,10 +101,14 @@ class LayeredForward:
             self.q_abs = buf(cap * max(m.heads * m.cache_width for m in lat))
             self.o_lat = buf(cap * max(m.heads * ceil8(m.kv_rank) for m in lat))
             buckets = engine._buckets
-            need = max(b * M.latent_attn_plan(b, m.heads, engine.ecfg.max_seq_len, m.cache_width)[0] * m.heads * (m.kv_rank + 2)
+            need = max(b * M.latent_attn_plan(b, m.heads, m.visible(engine.ecfg.max_seq_len), m.cache_width)[0] * m.heads * (m.kv_rank + 2)
                        for b in buckets for m in lat)
             self.attn_ws = buf(max(need, 1 << 20), torch.float32)
+            if any(m.q_rank for m in lat):
+                self.q_lat = buf(cap * max(ceil8(m.heads * (m.dim + m.rot_dim)) for m in lat if m.q_rank))
         self.ws_tokens = 0
+        # tokens that the widest latent layer sees (0: all of them)
+        self.latent_window = 0 if any(not m.window for m in lat) else max((m.window for m in lat), default=0)
         if any(self.expands):
             shapes = [(m.heads, *M.expanded_shape(m.dim, m.rot_dim, m.vdim), m.cache_width)
                       for m, ex in ((lw.spec.mixer, ex) for lw, ex in zip(layers, self.expands)) if ex]
@@ -140,6 +145,13 @@ class LayeredForward:
         if lin:
             self.lin_ws = buf(max(M.linear_attn_ws_elems(m.dim, m.vdim) for m in lin) if dt == torch.bfloat16 else 1, torch.float32)
 
+    def expand_rows(self, computed: int, n: int) -> int:
+        """Workspace rows in which the expanded form holds what a portion of ``n`` tokens behind ``computed`` ones sees."""
+        behind = computed
+        if self.latent_window:
+            behind -= max(0, computed - self.latent_window + 1) // 64 * 64
+        return (behind + n + 63) // 64 * 64
+
     # ------------------------------------------------------------------ mixers
     def _latent(self, l: int, lw: LayeredLayerWeights, m: LatentMixer, proj: torch.Tensor, out: torch.Tensor, b: RowBatch) -> None:
         rows, H, R, W = b.rows, m.heads, m.kv_rank, m.cache_width
@@ -152,31 +164,37 @@ class LayeredForward:
         if n_abs < rows:
             dq, dv = M.expanded_shape(m.dim, m.rot_dim, m.vdim)
             q_exp = self.q_exp[:rows * H * dq].view(rows, H, dq)
-        gate = proj[:, lw.offs["g"]:lw.offs["g"] + H]
+        gate = proj[:, lw.offs["g"]:lw.offs["g"] + m.gate_features]
+        q, q_off = None, lw.offs["q"]
+        if m.q_rank:
+            n = m.heads * (m.dim + m.rot_dim)
+            q = self.q_lat[:rows * ceil8(n)].view(rows, ceil8(n))[:, :n]
+            gemm.linear(proj[:, q_off:q_off + m.q_rank], lw.mix["uq"], out=q)
         M.latent_prep(proj, lw.mix["norm"], lw.mix["freq"], b.positions, b.slots, cache, heads=H, dim=m.dim, rot=m.rot_dim, kv_rank=R,
-                      q_off=lw.offs["q"], kv_off=lw.offs["kv"], eps=self.e.cfg.rms_norm_eps, abs_rows=n_abs, q_plain=q_plain,
-                      q_abs=q_abs, q_exp=q_exp)
+                      q_off=q_off, kv_off=lw.offs["kv"], eps=self.e.cfg.rms_norm_eps, abs_rows=n_abs, q_plain=q_plain,
+                      q_abs=q_abs, q_exp=q_exp, q=q, q_rank=m.q_rank, interleaved=m.rot.interleaved)
         if n_abs:
             gemm.linear_batched(q_plain[:, :, :m.dim], lw.mix["uk_t"], q_abs, n_abs * W)
-            splits, chunk = M.latent_attn_plan(n_abs, H, b.max_len, W)
+            splits, chunk = M.latent_attn_plan(n_abs, H, m.visible(b.max_len), W)
             if splits > 1 and n_abs * H * splits * (R + 2) > self.attn_ws.numel():
                 splits, chunk = 1, 0
             o_lat = self.o_lat[:H * n_abs * rp].view(H, n_abs, rp)
-            M.latent_attn(q_abs, cache, o_lat, b.table, b.positions, b.slots, kv_rank=R, rot=m.rot_dim, scale=m.scale, gate=gate,
-                          row_seq=b.row_seq, num_splits=splits, chunk_tokens=chunk, ws=self.attn_ws)
-            gemm.linear_batched(o_lat[:, :, :R], lw.mix["uv"], out[:n_abs], m.vdim)
+            M.latent_attn(q_abs, cache, o_lat, b.table, b.positions, b.slots, kv_rank=R, rot=m.rot_dim, scale=m.scale,
+                          gate=None if m.gate_elems else gate, row_seq=b.row_seq, num_splits=splits, chunk_tokens=chunk, ws=self.attn_ws,
+                          window=m.window)
+            gemm.linear_batched(o_lat[:, :, :R], lw.mix["uv"], out[:n_abs], m.vdim, gate=gate[:n_abs] if m.gate_elems else None)
         if n_abs < rows:
             for g in b.groups:
                 s = slice(g.seq0, g.seq0 + g.n)
                 starts = b.starts[s]
                 lat = self.lat_ws[:g.tokens * W].view(g.tokens, W)
-                M.latent_gather(cache, lat, b.table[s], b.ctx_lens[s], b.q_lens[s], starts, g.max_len)
+                M.latent_gather(cache, lat, b.table[s], b.ctx_lens[s], b.q_lens[s], starts, g.max_len, m.window)
                 k = self.k_exp[:g.tokens * H * dq].view(g.tokens, H, dq)
                 v = self.v_exp[:g.tokens * H * dv].view(g.tokens, H, dv)
                 gemm.linear(lat[:, :R + m.rot_dim], lw.mix["exp_k"], out=k.view(g.tokens, H * dq))
                 gemm.linear(lat[:, :R], lw.mix["exp_v"], out=v.view(g.tokens, H * dv))
                 M.expanded_prefill(q_exp, k, v, out, b.q_starts[s], b.q_lens[s], b.ctx_lens[s], starts, g.max_q, scale=m.scale,
-                                   vdim=m.vdim, gate=gate)
+                                   vdim=m.vdim, gate=gate, window=m.window)
 
     def _linear(self, l: int, lw: LayeredLayerWeights, m: LinearMixer, proj: torch.Tensor, out: torch.Tensor, b: RowBatch) -> None:
         n = m.out_features
@@ -196,7 +214,7 @@ class LayeredForward:
         """Whether the tensor-core attention kernels cover the mixer."""
         shape, page = attention_shape(m.dim, m.vdim), self.e.ecfg.page_size
         return (self.dtype == torch.bfloat16 and shape is not None and m.heads // m.kv_heads <= 16 and page & (page - 1) == 0
-                and page >= (16 if shape[0] == shape[1] else 64))
+                and page >= (16 if shape[0] == shape[1] else 64) and (not m.sigmoid or shape[0] == shape[1]) and (m.sigmoid or not m.pool))
 
     @staticmethod
     def _splits(m: GroupedMixer, rows: int, max_len: int) -> tuple[int, int]:
@@ -208,14 +226,21 @@ class LayeredForward:
         k, v = kv.k[l], kv.v[l]
         gp = M.group_pad(m.heads, m.kv_heads)
         q = self.q_grp[:rows * m.kv_heads * gp * k.shape[3]].view(rows, m.kv_heads, gp, k.shape[3])
-        if m.head_norms:
-            M.grouped_prep(proj, lw.mix["q_norm"], lw.mix["k_norm"], b.slots, k, v, q, heads=m.heads, dim=m.dim, vdim=m.vdim,
-                           offs=(o["q"], o["k"], o["v"]), eps=self.e.cfg.rms_norm_eps)
-            gate = proj[:, o["hg"]:o["hg"] + m.heads]
+        pool = M.BlockMeans(kv.k_pool[l], kv.v_pool[l], m.pool) if m.pool else None
+        if m.norm:
+            rot = self.rot_tables.get(m.rot)
+            M.grouped_prep(proj, lw.mix.get("q_norm"), lw.mix.get("k_norm"), b.slots, k, v, q, heads=m.heads, dim=m.dim, vdim=m.vdim,
+                           offs=(o["q"], o["k"], o["v"]), eps=self.e.cfg.rms_norm_eps, rot=rot, interleaved=rot is not None and m.rot.interleaved,
+                           positions=b.positions, pool=pool, pool_rows=b.n_dec, block_table=b.table)
         else:
             self._conv_rope(l, lw, m, proj, q, b)
-            gate = proj[:, o["g"]:o["g"] + m.out_features]
-        kw = dict(heads=m.heads, vdim=m.vdim, scale=m.scale, softcap=m.softcap, window=m.window, keep_first=m.keep_first)
+        if pool is not None and b.n_dec < rows:
+            s = slice(b.n_dec, rows)
+            M.block_means(k, v, pool, b.table, b.positions[s], b.slots[s], b.row_seq[s])
+        g_at = o["hg" if m.gate == "head" else "g"] if m.gate else 0
+        gate = proj[:, g_at:g_at + m.gate_features] if m.gate else None
+        kw = dict(heads=m.heads, vdim=m.vdim, scale=m.scale, softcap=m.softcap, window=m.window, keep_first=m.keep_first,
+                  sink=lw.mix.get("sink"), sigmoid_bias=lw.mix.get("bias"), pool=pool)
         if not self._tiled(m):
             M.grouped_attn(q, k, v, out, b.table, b.positions, b.slots, dim=m.dim, gate=gate, row_seq=b.row_seq, **kw)
             return
@@ -341,11 +366,13 @@ class LayeredForward:
             if post:
                 pending = dict(branches=ys, branch_norms=lw.branch_norms, norm=lw.norm1b or lw.norm1)
             else:
-                pending = dict(parts=ys, gate=proj[:, lw.offs["rg"]:lw.offs["rg"] + hid])
+                pending = dict(parts=ys, gate=proj[:, lw.offs["rg"]:lw.offs["rg"] + hid] if cfg.residual_gate else None)
             if lw.norm2 is not None:
                 self._enter(resid, lw.norm2, x2, pending)
                 if post:
                     pending = dict(branches=self.e.port.run(l, x2, rows, mode), norm=lw.norm2b or lw.norm2)
+                elif not cfg.residual_gate:
+                    pending = dict(parts=self.e.port.run(l, x2, rows, mode))
                 else:
                     rg2 = self.rg2[:rows]
                     gemm.linear(x2, lw.rg2, out=rg2, bias=lw.rg2_bias)

@@ -227,7 +227,8 @@ def _moe_reads(l: MoeFfnSpec, rank: int, size: int, experts: range, packed_weigh
         if not packed_weights:
             continue
         if ex.per_expert:
-            reads[f"gate{e}"] = TensorRead(ex.gate_key.format(expert=e), rows=rows)
+            if ex.gate_key:
+                reads[f"gate{e}"] = TensorRead(ex.gate_key.format(expert=e), rows=rows)
             reads[f"up{e}"] = TensorRead(ex.up_key.format(expert=e), rows=rows)
             reads[f"down{e}"] = TensorRead(ex.down_key.format(expert=e), cols=rows)
         else:
@@ -242,7 +243,8 @@ def _moe_reads(l: MoeFfnSpec, rank: int, size: int, experts: range, packed_weigh
             reads[f"down{e}"] = TensorRead(ex.down_key, cols=rows, expert=e, transposed=ex.input_major)
     if l.num_shared_experts:
         srows = _local(l.shared_intermediate_size, rank, size)
-        reads["shared_gate"] = TensorRead(l.shared_gate_key, rows=srows)
+        if l.shared_gate_key:
+            reads["shared_gate"] = TensorRead(l.shared_gate_key, rows=srows)
         reads["shared_up"] = TensorRead(l.shared_up_key, rows=srows)
         reads["shared_down"] = TensorRead(l.shared_down_key, cols=srows)
     if l.shared_scale_key:
@@ -292,7 +294,8 @@ def materialize_layer_weights(spec: FfnModelSpec, view: CheckpointKeyView, layer
         if t is not None and not t.plain:
             w.extra["gate_transform"] = t.constants()
         return w
-    gate_up = torch.stack([torch.cat([got[f"gate{e}"], got[f"up{e}"]], 0) for e in experts])
+    gated = f"gate{experts[0]}" in got
+    gate_up = torch.stack([torch.cat([got[f"gate{e}"], got[f"up{e}"]], 0) if gated else got[f"up{e}"] for e in experts])
     down = torch.stack([got[f"down{e}"] for e in experts])
     w = FfnLayerWeights(gate_up, down, router=got["router"])
     if f"gate_bias{experts[0]}" in got:
@@ -302,8 +305,8 @@ def materialize_layer_weights(spec: FfnModelSpec, view: CheckpointKeyView, layer
     t = l.gate_transform
     if t is not None and not t.plain:
         w.extra["gate_transform"] = t.constants()
-    if "shared_gate" in got:
-        w.shared_gate_up = torch.cat([got["shared_gate"], got["shared_up"]], 0)
+    if "shared_up" in got:
+        w.shared_gate_up = torch.cat([got["shared_gate"], got["shared_up"]], 0) if "shared_gate" in got else got["shared_up"]
         w.shared_down = got["shared_down"]
     for k in ("router_bias", "correction_bias", "shared_scale"):
         if k in got:

@@ -19,6 +19,7 @@ class ActivationKind(str, Enum):
     SILU = "silu"
     RELU = "relu"
     GELU = "gelu"
+    RELU2 = "relu2"                # max(z, 0)^2
     POLYNORM = "polynorm"          # a N(z) + b N(z^2) + c N(z^3) + e, N = row RMS normalisation: needs the whole row
 
 

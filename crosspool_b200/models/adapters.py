@@ -1,7 +1,7 @@
 """Architecture adapters: Hugging Face ``config.json`` + checkpoint keys → :class:`FfnModelSpec`.
 
 One adapter per supported architecture, discovered by ``architectures[0]`` (``architecture`` in the
-configuration files of layered decoders) — Kadavik, Saninex, Segirax and the same eight families the reference serves (src/xpool/runtime/ffnagent/models/*.py, discovery in
+configuration files of layered decoders) — Dofevik, Kadavik, Saninex, Segirax and the same eight families the reference serves (src/xpool/runtime/ffnagent/models/*.py, discovery in
 src/xpool/runtime/ffnagent/architecture.py:175-215): Qwen2, Qwen3, Qwen3-MoE, Llama, OPT,
 DeepSeek-V2, GLM-4 MoE Lite and GPT-OSS. Adapters only read the configuration and the *names* of
 checkpoint tensors; no weight is opened here.
@@ -265,6 +265,23 @@ def _kadavik(model_id: str, src: FfnSourceConfig, keys: Iterable[str]) -> FfnMod
     return FfnModelSpec(model_id, src.architecture, src.payload_dtype, c.hidden_size, src.quantization, tuple(layers))
 
 
+def _dofevik(model_id: str, src: FfnSourceConfig, keys: Iterable[str]) -> FfnModelSpec:
+    from .config import dofevik_config
+
+    c = dofevik_config(dict(src.cfg), model_id)
+    layers = []
+    for i, s in enumerate(c.layer_specs):
+        p, m = f"l{i}.mlp", s.moe
+        if m is not None:
+            layers.append(MoeFfnSpec(
+                i, c.hidden_size, m.ff, m.experts, m.top, ActivationKind.RELU2,
+                ExpertSource(True, None, p + ".e{expert}.up", None, p + ".e{expert}.down"), router_weight_key=f"{p}.router",
+                router_bias_key=f"{p}.router.b", router_precision=RouterProjectionPrecision.FP32_LOGITS,
+                num_shared_experts=int(m.shared_ff > 0), shared_intermediate_size=m.shared_ff,
+                shared_up_key=f"{p}.shared.up" if m.shared_ff else None, shared_down_key=f"{p}.shared.down" if m.shared_ff else None))
+    return FfnModelSpec(model_id, src.architecture, src.payload_dtype, c.hidden_size, src.quantization, tuple(layers))
+
+
 ADAPTERS: dict[str, Callable[[str, FfnSourceConfig, Iterable[str]], FfnModelSpec]] = {
     "Qwen2ForCausalLM": _llama_like,
     "Qwen3ForCausalLM": _llama_like,
@@ -275,6 +292,7 @@ ADAPTERS: dict[str, Callable[[str, FfnSourceConfig, Iterable[str]], FfnModelSpec
     "DeepseekV2ForCausalLM": lambda m, s, k: _deepseek_like(m, s, k, sigmoid=False),
     "Glm4MoeLiteForCausalLM": lambda m, s, k: _deepseek_like(m, s, k, sigmoid=True),
     "GptOssForCausalLM": _gpt_oss,
+    "Dofevik": _dofevik,
     "Kadavik": _kadavik,
     "Saninex": _saninex,
     "Segirax": _segirax,

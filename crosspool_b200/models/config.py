@@ -36,22 +36,25 @@ class MlaShape:
 @dataclass(frozen=True)
 class RotaryScaling:
     """Rotary frequencies for contexts beyond ``original`` tokens: wavelengths above ``original / low`` are stretched by
-    ``factor``, those below ``original / high`` are kept, the ones between blend linearly in ``original / wavelength``."""
+    ``factor``, those below ``original / high`` are kept, the ones between blend linearly in ``original / wavelength``.
+    ``original`` = 0: all of them are stretched by ``factor``."""
 
     factor: float
-    low: float
-    high: float
-    original: float
+    low: float = 0.0
+    high: float = 0.0
+    original: float = 0.0
 
 
 @dataclass(frozen=True)
 class RotarySpec:
-    """Rotary positions on the first ``dims`` dimensions of a vector, paired (i, i + dims / 2): the pair at position p
-    turns by ``p * f_i``, ``f_i = base ** (-2 i / dims)``, scaled where there is a ``scaling``."""
+    """Rotary positions on the first ``dims`` dimensions of a vector, paired (i, i + dims / 2), or (2 i, 2 i + 1) with
+    ``interleaved``: the pair at position p turns by ``p * f_i``, ``f_i = base ** (-2 i / dims)``, scaled where there is a
+    ``scaling``."""
 
     dims: int
     base: float
     scaling: RotaryScaling | None = None
+    interleaved: bool = False
 
 
 def ceil8(n: int) -> int:
@@ -75,7 +78,9 @@ def attention_shape(dim: int, vdim: int) -> tuple[int, int] | None:
 @dataclass(frozen=True)
 class LatentMixer:
     """Latent attention as a layer's mixer: per-head keys and values are linear maps of one cached ``kv_rank`` latent,
-    plus one rotary key part of ``rot_dim`` shared by the heads. The output of every head is gated by a sigmoid."""
+    plus one rotary key part of ``rot_dim`` shared by the heads. The output is gated by a sigmoid, one number per head or, with
+    ``gate_elems``, per element. ``q_rank`` > 0: queries come from a normed latent of their own of that size. ``window`` > 0: a
+    token sees itself and the ``window - 1`` tokens before it."""
 
     heads: int
     dim: int                    # unrotated query/key dimensions per head
@@ -84,6 +89,9 @@ class LatentMixer:
     kv_rank: int
     rot: RotarySpec
     scale: float
+    q_rank: int = 0
+    window: int = 0
+    gate_elems: bool = False
     kind: str = "latent_attention"
 
     @property
@@ -103,9 +111,18 @@ class LatentMixer:
     def out_features(self) -> int:
         return self.heads * self.vdim
 
+    @property
+    def gate_features(self) -> int:
+        return self.out_features if self.gate_elems else self.heads
+
+    def visible(self, length: int) -> int:
+        """Bound on the tokens a query at the end of ``length`` tokens sees."""
+        return min(length, self.window) if self.window else length
+
     def param_count(self, hidden: int) -> int:
         q = self.heads * (self.dim + self.rot_dim)
-        return (hidden * (q + self.kv_rank + self.rot_dim + self.heads + self.out_features) + self.kv_rank
+        q = self.q_rank * (hidden + 1 + q) if self.q_rank else hidden * q
+        return (q + hidden * (self.kv_rank + self.rot_dim + self.gate_features + self.out_features) + self.kv_rank
                 + self.kv_rank * self.heads * (self.dim + self.vdim))
 
 
@@ -148,14 +165,17 @@ class LinearMixer(_RecurrentMixer):
 
 @dataclass(frozen=True)
 class GroupedMixer:
-    """Grouped-query softmax attention: ``heads`` query heads share ``kv_heads`` cached keys and values, scores saturate at
-    +-``softcap`` (0: they do not), and a sigmoid gates the output.
+    """Grouped-query attention: ``heads`` query heads share ``kv_heads`` cached keys and values, scores saturate at +-``softcap``
+    (0: they do not).
 
-    ``head_norms``: projections have biases, queries and keys are RMS-normed per head, the gate is one number per head.
-    Without: none of these, and the gate is one number per output element. ``conv``: queries, keys and values pass a causal
-    convolution of that many taps before anything else (0: none). ``window``: a token sees itself and the ``window - 1``
-    tokens before it, and the first ``keep_first`` tokens of the sequence (0: all before it). ``kv_from``: the layer has no
-    keys and values of its own and reads those that layer caches."""
+    ``norm``: queries and keys are RMS-normed per head, with a ``"weight"`` or as ``"unit"`` vectors of root mean square one
+    (``""``: not at all). ``biases``: of the projections. ``gate``: a sigmoid gates the output, one number per ``"head"`` or
+    ``"element"`` (``""``: none). ``conv``: queries, keys and values pass a causal convolution of that many taps before anything
+    else (0: none). ``window``: a token sees itself and the ``window - 1`` tokens before it, and the first ``keep_first`` tokens
+    of the sequence (0: all before it). ``kv_from``: the layer has no keys and values of its own and reads those that layer
+    caches. ``sink``: a number per head joins the softmax's sum and has no value. ``sigmoid``: no softmax, a token's weight is
+    the sigmoid of its score plus a number per head. ``pool`` > 0: beside its window a token sees the mean key and value of
+    every block of that many tokens that lies wholly behind the window. ``tied``: values are the projected keys."""
 
     heads: int
     kv_heads: int
@@ -163,13 +183,40 @@ class GroupedMixer:
     vdim: int
     scale: float
     softcap: float = 0.0
-    head_norms: bool = True
+    norm: str = "weight"
+    biases: bool = True
+    gate: str = "head"
     conv: int = 0
     rot: RotarySpec | None = None
     window: int = 0
     keep_first: int = 0
     kv_from: int | None = None
+    sink: bool = False
+    sigmoid: bool = False
+    pool: int = 0
+    tied: bool = False
     kind: str = "grouped_attention"
+
+    @property
+    def head_norms(self) -> bool:
+        return bool(self.norm)
+
+    @property
+    def gate_features(self) -> int:
+        return {"head": self.heads, "element": self.out_features, "": 0}[self.gate]
+
+    def pool_page(self, page_size: int) -> int:
+        """Rows for block means beside every page of ``page_size`` tokens: at least as many as blocks end in it, so that block b
+        lies beside page ``b // pool_page`` of its sequence; a power of two of at least eight (the copies of the tensor-core
+        kernels bring eight rows)."""
+        n = 8
+        while n * self.pool < page_size:
+            n *= 2
+        return n
+
+    def pool_shapes(self, page_size: int) -> tuple[tuple[int, int, int], ...]:
+        """Block means beside one page, keys and values: (rows, heads, elements per head)."""
+        return tuple((self.pool_page(page_size), *r) for r in self.row_shapes) if self.pool else ()
 
     @property
     def row_shapes(self) -> tuple[tuple[int, int], ...]:
@@ -204,13 +251,16 @@ class GroupedMixer:
 
     def visible(self, length: int) -> int:
         """Bound on the tokens a query at the end of ``length`` tokens sees."""
-        return min(length, self.window + self.keep_first) if self.window else length
+        blocks = max(0, length - self.window) // self.pool if self.pool else 0
+        return min(length, self.window + self.keep_first) + blocks if self.window else length
 
     def param_count(self, hidden: int) -> int:
-        if not self.head_norms:
-            return hidden * (self.conv_channels + 2 * self.out_features) + self.conv_state_elems
-        kv = self.kv_heads * (self.dim + self.vdim)
-        return ((hidden + 1) * (self.heads * self.dim + kv) + 2 * self.dim + hidden * (self.heads + self.out_features + 1))
+        rows = self.heads * self.dim
+        if self.kv_from is None:
+            rows += self.kv_heads * (self.dim + (0 if self.tied else self.vdim))
+        n = rows * (hidden + int(self.biases)) + hidden * (self.gate_features + self.out_features) + self.conv_state_elems
+        n += self.heads * (int(self.sink) + int(self.sigmoid)) + (2 * self.dim if self.norm == "weight" else 0)
+        return n + (hidden if self.biases and self.gate == "head" else 0)        # (with a bias behind the output map as well)
 
 
 @dataclass(frozen=True)
@@ -331,7 +381,9 @@ GELU_CUBIC = 0.044715
 class MoeSpec:
     """Routed FFN of a layered decoder: ``experts`` gated (silu) FFNs of ``ff`` features and ``identity`` experts that return
     their input; a token takes ``top`` of them by softmax score plus a correction, weighted by their scores normalised to
-    ``scale``. ``shared_ff`` > 0: one more expert for every token, its output times a sigmoid per token."""
+    ``scale``. ``shared_ff`` > 0: one more expert for every token, its output times a sigmoid per token with ``shared_gate``.
+    ``relu2``: experts are ungated, ``down(max(up x, 0)^2)``. ``logit_choice``: the router has biases, its largest logits are
+    chosen and their softmax weighs them (no correction)."""
 
     experts: int
     top: int
@@ -339,6 +391,19 @@ class MoeSpec:
     identity: int = 0
     scale: float = 1.0
     shared_ff: int = 0
+    shared_gate: bool = True
+    relu2: bool = False
+    logit_choice: bool = False
+
+    @property
+    def maps(self) -> int:
+        """Matrices of an expert."""
+        return 2 if self.relu2 else 3
+
+    @property
+    def in_features(self) -> int:
+        """Rows of an expert's input map."""
+        return self.ff * (self.maps - 1)
 
     @property
     def routed(self) -> int:
@@ -371,8 +436,8 @@ class LayerSpec:
         m = self.moe
         if m is None:
             return self.ffn_maps * hidden * self.ff
-        shared = hidden * (3 * m.shared_ff + 1) if m.shared_ff else 0
-        return 3 * m.experts * hidden * m.ff + m.routed * (hidden + 1) + shared
+        shared = hidden * (m.maps * m.shared_ff + int(m.shared_gate)) if m.shared_ff else 0
+        return m.maps * m.experts * hidden * m.ff + m.routed * (hidden + 1) + shared
 
 
 @dataclass(frozen=True)
@@ -413,8 +478,8 @@ class ModelConfig:
     attention_sinks: bool = False    # one learned logit per head joins every softmax and takes no value: GPT-OSS
     o_bias: bool = False
     mla: MlaShape | None = None
-    # Layered decoders: every layer names its own mixer and FFN. norm "dyt" is dynamic tanh (elementwise, no statistics);
-    # ``residual_gate``: each sublayer's result is multiplied by sigmoid(W h + b) of its input and summed in fp32.
+    # Layered decoders: every layer names its own mixer and FFN. norm "dyt" is dynamic tanh (elementwise, no statistics), "scalar"
+    # an RMS norm with one weight for all coordinates; ``residual_gate``: each sublayer's result is multiplied by sigmoid(W h + b) of its input and summed in fp32.
     # ``output_norm``: sublayers' results are normed before they are added to the residual, which the sublayers read as it
     # is, or with ``input_norm`` through a norm of their own.
     # ``token_side`` > 0: behind the FFN every layer adds a small gated map of the residual and of a second embedding of its
@@ -469,7 +534,7 @@ class ModelConfig:
 
     def attention_param_bytes(self) -> int:
         if self.layered:
-            norm = 2 * self.hidden_size + 1 if self.norm == "dyt" else self.hidden_size
+            norm = {"dyt": 2 * self.hidden_size + 1, "scalar": 1}.get(self.norm, self.hidden_size)
             n = self.hidden_size * self.vocab_size * (1 if self.tie_word_embeddings else 2) + norm
             if self.token_side:
                 n += self.num_layers * (self.token_side * (self.vocab_size + 2 * self.hidden_size) + norm)
@@ -496,7 +561,7 @@ class ModelConfig:
 
     def kv_bytes_per_token(self) -> int:
         if self.layered:
-            return 2 * sum(s.mixer.cache_width for s in self.layer_specs)
+            return 2 * sum(s.mixer.cache_width for s in self.layer_specs)        # (without the block means of pooling layers)
         return 2 * self.num_layers * self.kv_size * 2
 
     def state_bytes_per_sequence(self) -> int:
@@ -624,12 +689,12 @@ def saninex_config(cfg: dict[str, Any], name: str = "") -> ModelConfig:
         hidden_act="clamped_glu", max_position_embeddings=1 << 30, norm="rmsnorm", layer_specs=tuple(specs), output_norm=True)
 
 
-def _rotary(r: dict[str, Any] | None, dim: int) -> RotarySpec | None:
+def _rotary(r: dict[str, Any] | None, dim: int, interleaved: bool = False) -> RotarySpec | None:
     if not r or not int(r["dims"]):
         return None
     sc = r.get("scaling")
     rot = RotarySpec(int(r["dims"]), float(r["base"]),
-                     RotaryScaling(*(float(sc[n]) for n in ("factor", "low", "high", "original"))) if sc else None)
+                     RotaryScaling(*(float(sc[n]) for n in ("factor", "low", "high", "original") if n in sc)) if sc else None, interleaved)
     if rot.dims % 2 or not 0 < rot.dims <= dim:
         raise ValueError(f"rotary dims {rot.dims} do not fit a head of {dim}")
     return rot
@@ -642,7 +707,7 @@ def _kadavik_attention(m: dict[str, Any]) -> GroupedMixer:
     if window < 0 or keep < 0 or (mask and not window):
         raise ValueError(f"attention mask {mask!r} is not a window")
     kv_from = m.get("kv_from")
-    return GroupedMixer(**_ints(m, "heads", "kv_heads", "dim", "vdim"), scale=float(m["scale"]), head_norms=False,
+    return GroupedMixer(**_ints(m, "heads", "kv_heads", "dim", "vdim"), scale=float(m["scale"]), norm="", biases=False, gate="element",
                         conv=int(m.get("conv") or 0), rot=_rotary(m.get("rot"), int(m["dim"])), window=window,
                         keep_first=keep, kv_from=None if kv_from is None else int(kv_from))
 
@@ -695,7 +760,65 @@ def kadavik_config(cfg: dict[str, Any], name: str = "") -> ModelConfig:
         logit_scale=float(cfg.get("logit_scale", 1.0)))
 
 
-LAYERED_CONFIGS = {"Segirax": segirax_config, "Saninex": saninex_config, "Kadavik": kadavik_config}
+def _window(m: dict[str, Any]) -> int:
+    """Tokens a layer sees, itself included (0: all of them)."""
+    mask = m.get("mask") or {}
+    window = int(mask.get("size") or 0)
+    if window < 0 or (mask and not window):
+        raise ValueError(f"attention mask {mask!r} is not a window")
+    return window
+
+
+def _dofevik_mixer(kind: str, m: dict[str, Any]) -> Mixer:
+    if kind == "attention":
+        _grouped_heads(m)
+        return GroupedMixer(**_ints(m, "heads", "kv_heads", "dim", "vdim"), scale=float(m["scale"]), norm="unit", gate="", window=_window(m),
+                            rot=_rotary(m.get("rot"), int(m["dim"]), interleaved=True), sink=True)
+    if kind == "attention_2":
+        _grouped_heads(m)
+        if int(m.get("vdim", m["dim"])) != int(m["dim"]):
+            raise ValueError(f"values of {m['vdim']} dimensions cannot be keys of {m['dim']}")
+        window, pool = _window(m), int((m.get("mask") or {}).get("pool") or 0)
+        if pool < 0:
+            raise ValueError(f"blocks of {pool} tokens")
+        return GroupedMixer(**_ints(m, "heads", "kv_heads", "dim"), vdim=int(m["dim"]), scale=float(m["scale"]), biases=False, gate="",
+                            window=window, sigmoid=True, pool=pool, tied=True)
+    if kind == "latent_attention":
+        mixer = LatentMixer(**_ints(m, "heads", "dim", "rot_dim", "vdim", "kv_rank"), rot=_rotary(m["rot"], int(m["rot_dim"])),
+                            scale=float(m["scale"]), q_rank=int(m["q_rank"]), window=_window(m), gate_elems=True)
+        if mixer.q_rank < 1:
+            raise ValueError(f"a query latent of {mixer.q_rank} dimensions")
+        return mixer
+    raise ValueError(f"unsupported mixer {kind!r}")
+
+
+def _dofevik_mlp(mixer: Mixer, mlp: dict[str, Any] | None) -> LayerSpec:
+    if mlp is None:
+        return LayerSpec(mixer)
+    if mlp.get("kind", "moe") != "moe":
+        raise ValueError(f"unsupported feed-forward kind {mlp['kind']!r}")
+    r, shared = mlp["router"], mlp.get("shared")
+    moe = MoeSpec(int(r["experts"]), int(r["top"]), int(mlp["expert"]["ff"]), shared_ff=int(shared["ff"]) if shared else 0, shared_gate=False,
+                  relu2=True, logit_choice=True)
+    if not 0 < moe.top <= min(moe.experts, 32) or moe.experts > 256:
+        raise ValueError(f"a router of {moe.experts} outputs that takes {moe.top} is not supported (at most 32 of 256)")
+    return LayerSpec(mixer, moe=moe)
+
+
+def dofevik_config(cfg: dict[str, Any], name: str = "") -> ModelConfig:
+    """Dofevik: RMS norms with one weight in front of every sublayer; windowed attention with unit queries and keys and a sink,
+    attention with sigmoid weights over a window and the means of the blocks behind it, and windowed latent attention whose queries
+    come from a latent, in any order; routed FFNs of squared-relu experts; its ``config.json`` lists every layer."""
+    specs = tuple(_dofevik_mlp(_dofevik_mixer(l["type"], l["mixer"]), l.get("mlp")) for l in cfg["layers"])
+    first = specs[0].mixer
+    return ModelConfig(
+        name=name or cfg["architecture"], architecture=cfg["architecture"], hidden_size=int(cfg["width"]), num_layers=len(specs),
+        num_q_heads=first.heads, num_kv_heads=getattr(first, "kv_heads", first.heads), head_dim=first.dim,
+        intermediate_size=max(s.moe.ff if s.moe else 0 for s in specs), vocab_size=int(cfg["vocab"]), rms_norm_eps=float(cfg["norm"]["eps"]),
+        qk_norm=False, hidden_act="relu2", max_position_embeddings=1 << 30, norm="scalar", layer_specs=specs)
+
+
+LAYERED_CONFIGS = {"Segirax": segirax_config, "Saninex": saninex_config, "Kadavik": kadavik_config, "Dofevik": dofevik_config}
 
 
 def from_hf_config(cfg: dict[str, Any], name: str = "") -> ModelConfig:

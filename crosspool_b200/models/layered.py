@@ -79,23 +79,36 @@ def rotary_frequencies(dims: int, base: float) -> torch.Tensor:
     return float(base) ** (-2.0 * torch.arange(dims // 2, dtype=torch.float64) / dims)
 
 
+def scaled_frequencies(rot: RotarySpec) -> torch.Tensor:
+    """Turns per position (radians) of every pair, double."""
+    f, sc = rotary_frequencies(rot.dims, rot.base), rot.scaling
+    if sc is None:
+        return f
+    if not sc.original:
+        return f / sc.factor
+    turns = sc.original * f / (2 * torch.pi)                 # of the original context: original / wavelength
+    blend = ((turns - sc.low) / (sc.high - sc.low)).clamp(0, 1) if sc.high > sc.low else (turns >= sc.low).double()
+    return f * (blend + (1 - blend) / sc.factor)
+
+
 def rotary_table(rot: RotarySpec, positions: int, device) -> torch.Tensor:
     """cos and sin of every position's angles, fp32 ``[positions, dims / 2, 2]`` rounded from double."""
-    f = rotary_frequencies(rot.dims, rot.base).to(device)
-    sc = rot.scaling
-    if sc is not None:
-        turns = sc.original * f / (2 * torch.pi)             # of the original context: original / wavelength
-        blend = ((turns - sc.low) / (sc.high - sc.low)).clamp(0, 1) if sc.high > sc.low else (turns >= sc.low).double()
-        f = f * (blend + (1 - blend) / sc.factor)
-    a = torch.arange(positions, dtype=torch.float64, device=device)[:, None] * f
+    a = torch.arange(positions, dtype=torch.float64, device=device)[:, None] * scaled_frequencies(rot).to(device)
     return torch.stack([a.cos(), a.sin()], -1).float().contiguous()
 
 
 def _latent(m: LatentMixer, get: Getter, p: str, hidden: int, dtype: torch.dtype, device) -> tuple[list, dict]:
     H, R, d, r, vd = m.heads, m.kv_rank, m.dim, m.rot_dim, m.vdim
-    q, dkv, g = get(p + "q", (H * (d + r), hidden)), get(p + "dkv", (R + r, hidden)), get(p + "g", (H, hidden))
+    dkv, g = get(p + "dkv", (R + r, hidden)), get(p + "g", (m.gate_features, hidden))
+    mix = {}
+    if m.q_rank:
+        # the latent's norm weight is folded into the map behind it, its division follows the product (a number per row)
+        q, uq = get(p + "dq", (m.q_rank, hidden)), get(p + "uq", (H * (d + r), m.q_rank))
+        mix["uq"] = pad_pitch((uq.float() * get(p + "dq.norm", (m.q_rank,)).float()).to(dtype))
+    else:
+        q = get(p + "q", (H * (d + r), hidden))
     uk, uv = get(p + "uk", (H * d, R)), get(p + "uv", (H * vd, R))
-    mix = {"norm": get(p + "dkv.norm", (R,)).float().contiguous(), "freq": rotary_frequencies(m.rot.dims, m.rot.base).to(device),
+    mix |= {"norm": get(p + "dkv.norm", (R,)).float().contiguous(), "freq": scaled_frequencies(m.rot).to(device),
            "uk_t": pad_pitch(uk.view(H, d, R).transpose(1, 2).reshape(H * R, d)), "uv": pad_pitch(uv)}
     shape = expanded_shape(d, r, vd) if dtype == torch.bfloat16 else None
     if shape is not None:
@@ -151,6 +164,17 @@ def _windowed(m: GroupedMixer, get: Getter, p: str, hidden: int) -> tuple[list, 
     return [(n, get(p + n, (r, hidden))) for n, r in {**rows, "g": m.out_features}.items()], mix
 
 
+def _scored(m: GroupedMixer, get: Getter, p: str, hidden: int) -> tuple[list, dict, dict]:
+    """Grouped-query attention whose scores come from normed queries and keys, with a number per head beside them."""
+    rows = {"q": m.heads * m.dim, "k": m.kv_heads * m.dim}
+    if not m.tied:
+        rows["v"] = m.kv_heads * m.vdim
+    mix = {n: get(p + name, (m.heads,)).float().contiguous() for n, name, on in (("sink", "sink", m.sink), ("bias", "pb", m.sigmoid)) if on}
+    if m.norm == "weight":
+        mix |= {n: get(f"{p}{n[0]}.norm", (m.dim,)).float().contiguous() for n in ("q_norm", "k_norm")}
+    return [(n, get(p + n, (r, hidden))) for n, r in rows.items()], {n: get(f"{p}{n}.b", (r,)).float() for n, r in rows.items() if m.biases}, mix
+
+
 def _memory(m: MemoryMixer, get: Getter, p: str, hidden: int) -> tuple[list, dict, dict]:
     rows = {"q": m.heads * m.dim, "k": m.heads * m.dim, "v": m.out_features, "g": m.out_features, "i": m.heads, "f": m.heads}
     return ([(n, get(p + n, (r, hidden))) for n, r in rows.items()], {n: get(f"{p}{n}.b", (m.heads,)).float() for n in "if"},
@@ -184,6 +208,29 @@ def _input_output_norm_layer(cfg: ModelConfig, i: int, spec: LayerSpec, get: Get
         lw.side_proj = pad_pitch(get(p + "side.proj", (h, cfg.token_side)))
         lw.side_norm = _plain_norm(get, p + "side.norm", cfg)
     return lw
+
+
+def _scalar_norm(get: Getter, name: str, cfg: ModelConfig) -> NormParams:
+    """An RMS norm with one weight for all coordinates."""
+    return NormParams("rmsnorm", get(name, ()).float().expand(cfg.hidden_size).contiguous(), eps=cfg.rms_norm_eps)
+
+
+def _input_norm_layer(cfg: ModelConfig, i: int, spec: LayerSpec, get: Getter, device, dtype: torch.dtype) -> LayeredLayerWeights:
+    """A layer with norms in front of its sublayers only, whose results are added as they are."""
+    h, m, p = cfg.hidden_size, spec.mixer, f"l{i}."
+    biases: dict = {}
+    if isinstance(m, LatentMixer):
+        sections, mix = _latent(m, get, p + "mix.", h, dtype, device)
+    else:
+        sections, biases, mix = _scored(m, get, p + "mix.", h)
+    proj, offs = _fuse(sections)
+    if "v" not in offs and "k" in offs:
+        offs["v"] = offs["k"]                            # values are the projected keys
+    bias = torch.zeros(offs["end"], dtype=torch.float32, device=device) if biases else None
+    for n, b in biases.items():
+        bias[offs[n]:offs[n] + b.shape[0]] = b
+    return LayeredLayerWeights(spec, _scalar_norm(get, p + "norm1", cfg), proj, bias, offs, pad_pitch(get(p + "mix.o", (h, m.out_features))), mix,
+                               norm2=_scalar_norm(get, p + "norm2", cfg) if spec.has_ffn else None)
 
 
 def _centred_norm(get: Getter, name: str, cfg: ModelConfig) -> NormParams:
@@ -231,6 +278,9 @@ def layered_attention_weights(cfg: ModelConfig, get: Getter, device, dtype: torc
         if cfg.output_norm:
             layers.append(_output_norm_layer(cfg, i, spec, get, device))
             continue
+        if cfg.norm == "scalar":
+            layers.append(_input_norm_layer(cfg, i, spec, get, device, dtype))
+            continue
         p, m = f"l{i}", spec.mixer
         if isinstance(m, LatentMixer):
             sections, mix = _latent(m, get, p + ".mix.", h, dtype, device)
@@ -249,8 +299,9 @@ def layered_attention_weights(cfg: ModelConfig, get: Getter, device, dtype: torc
             lw.silu_cols = offs["g"]            # q, k and v
         layers.append(lw)
     embed = get("embed", (cfg.vocab_size, h)).contiguous()
-    final = (_plain_norm if cfg.input_norm else _centred_norm if cfg.output_norm else _norm)(get, "final.norm", cfg)
-    w = AttentionWeights(embed, layers, final, pad_pitch(embed))
+    norm = _scalar_norm if cfg.norm == "scalar" else _plain_norm if cfg.input_norm else _centred_norm if cfg.output_norm else _norm
+    head = embed if cfg.tie_word_embeddings else get("head", (cfg.vocab_size, h))
+    w = AttentionWeights(embed, layers, norm(get, "final.norm", cfg), pad_pitch(head))
     if cfg.token_side:
         # rows of whole 16-byte units, gathered for all layers at once
         n = cfg.num_layers * cfg.token_side
@@ -259,7 +310,7 @@ def layered_attention_weights(cfg: ModelConfig, get: Getter, device, dtype: torc
 
 
 # stored around zero: norms behind sublayers; biases and decays of random models are zero too
-_ZERO = (".b", "A_log", "dt_bias")
+_ZERO = (".b", "A_log", "dt_bias", ".pb")
 
 
 def random_getter(gen: torch.Generator, dtype: torch.dtype, device, centred_norms: bool = False) -> Getter:

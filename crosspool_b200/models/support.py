@@ -54,7 +54,20 @@ _KADAVIK_PROBE = {
                 "mixer": {"heads": 2, "kv_heads": 1, "dim": 16, "vdim": 16, "scale": 0.25, "conv": 3, "rot": {"dims": 8, "base": 1e4},
                           "mask": {"size": 32, "keep_first": 4}}}]}
 
+_DOFEVIK_PROBE = {
+    "architecture": "Dofevik", "vocab": 256, "width": 64, "norm": {"eps": 1e-6},
+    "layers": [{"type": "attention", "mlp": None, "mixer": {"heads": 2, "kv_heads": 1, "dim": 16, "vdim": 16, "scale": 0.25, "mask": {"size": 32},
+                                                            "rot": {"dims": 8, "base": 1e4, "scaling": {"factor": 4.0}}}},
+               {"type": "attention_2", "mlp": None, "mixer": {"heads": 2, "kv_heads": 1, "dim": 16, "vdim": 16, "scale": 0.25,
+                                                              "mask": {"size": 32, "pool": 8}}},
+               {"type": "latent_attention", "mlp": {"kind": "moe", "expert": {"ff": 32}, "shared": {"ff": 32}, "router": {"experts": 4, "top": 2}},
+                "mixer": {"heads": 2, "dim": 16, "rot_dim": 8, "vdim": 16, "q_rank": 24, "kv_rank": 32, "scale": 0.2, "mask": {"size": 32},
+                          "rot": {"dims": 8, "base": 1e4}}}]}
+
 _LAYERED = {
+    "Dofevik": (_DOFEVIK_PROBE, "per layer: grouped-query attention over a window (scaled interleaved rotary, unit queries and keys, sinks), attention "
+                                "with sigmoid weights over a window and pooled blocks (q/k RMSNorm, values are the keys), or latent attention over "
+                                "a window (queries from a latent, gate per output); RMS norms with one weight, untied head"),
     "Kadavik": (_KADAVIK_PROBE, "per layer: matrix memory with exponential gates (mLSTM) or grouped-query attention (short convolutions, scaled "
                                 "rotary, sliding window with kept first tokens, gate per output, keys and values of another layer); norms before "
                                 "and behind the sublayers, a second token embedding per layer"),
@@ -107,6 +120,8 @@ def _ffn_features(spec) -> str:
             if l.gate_transform.limit > 0:
                 out.append("clamped activation")
         elif isinstance(l, MoeFfnSpec):
+            if l.experts.gate_key is None and l.experts.packed_key is None:
+                out.append(f"ungated {l.activation.value} experts")
             out.append(f"top-k {'sigmoid' if l.router_algorithm == RouterAlgorithm.SIGMOID else 'softmax'} router")
             if l.router_precision != RouterProjectionPrecision.PAYLOAD:
                 out.append(f"{l.router_precision.value} router projection")

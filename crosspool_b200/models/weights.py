@@ -231,13 +231,15 @@ def random_ffn_layer(cfg: ModelConfig, layer: int, seed: int = 0, device="cpu", 
             raise NotImplementedError("the FFNs of layered decoders run whole on one GPU (FFN TP 1)")
         if spec.moe is not None:
             m = spec.moe
-            w = FfnLayerWeights(_randn(gen, (m.experts, 2 * m.ff, h), dt, device), _randn(gen, (m.experts, h, m.ff), dt, device),
+            w = FfnLayerWeights(_randn(gen, (m.experts, m.in_features, h), dt, device), _randn(gen, (m.experts, h, m.ff), dt, device),
                                 router=_randn(gen, (m.routed, h), dt, device))
             if m.shared_ff:
-                w.shared_gate_up, w.shared_down = _randn(gen, (2 * m.shared_ff, h), dt, device), _randn(gen, (h, m.shared_ff), dt, device)
-                w.extra["shared_scale"] = _randn(gen, (1, h), dt, device)
-            w.extra.update(correction_bias=torch.zeros(m.routed, dtype=torch.float32, device=device), experts=(0, m.experts),
-                           router_precision="fp32_logits")
+                w.shared_gate_up = _randn(gen, ((m.maps - 1) * m.shared_ff, h), dt, device)
+                w.shared_down = _randn(gen, (h, m.shared_ff), dt, device)
+                if m.shared_gate:
+                    w.extra["shared_scale"] = _randn(gen, (1, h), dt, device)
+            bias = "router_bias" if m.logit_choice else "correction_bias"
+            w.extra.update({bias: torch.zeros(m.routed, dtype=torch.float32, device=device)}, experts=(0, m.experts), router_precision="fp32_logits")
             return w
         if spec.gelu:
             w = FfnLayerWeights(_randn(gen, (2 * inter, h), dt, device), _randn(gen, (h, inter), dt, device))

@@ -15,7 +15,7 @@ import ctypes as C
 import functools
 from pathlib import Path
 
-EXPECTED_ABI = 24
+EXPECTED_ABI = 25
 HERE = Path(__file__).resolve().parent
 
 
@@ -72,6 +72,7 @@ class GemmArgs(C.Structure):
         ("tail_from", C.c_int),
         ("tail", C.c_void_p),
         ("ld_tail", C.c_int),
+        ("relu2", C.c_int),
     ]
 
 
@@ -241,6 +242,12 @@ class DecodeRowsArgs(C.Structure):
         ("window", C.c_int),
         ("keep_first", C.c_int),
         ("gate_elems", C.c_int),
+        ("sink", C.c_void_p),
+        ("sigmoid_bias", C.c_void_p),
+        ("k_pool", C.c_void_p),
+        ("v_pool", C.c_void_p),
+        ("pool", C.c_int),
+        ("pool_page", C.c_int),
     ]
 
 
@@ -278,6 +285,12 @@ class PrefillAttnArgs(C.Structure):
         ("window", C.c_int),
         ("keep_first", C.c_int),
         ("gate_elems", C.c_int),
+        ("sink", C.c_void_p),
+        ("sigmoid_bias", C.c_void_p),
+        ("k_pool", C.c_void_p),
+        ("v_pool", C.c_void_p),
+        ("pool", C.c_int),
+        ("pool_page", C.c_int),
     ]
 
 
@@ -301,12 +314,16 @@ PostNormArgs = _struct("PostNormArgs", "XpPostNormArgs", a_ptr="resid", b_ptr2="
 HeadGateArgs = _struct("HeadGateArgs", "XpHeadGateArgs", a_ptr="o weight gate out", b_int="rows heads dim ld_o ld_gate ld_out", c_float="eps",
                        d_int="f32 per_head_weight sigmoid_gate")
 GluArgs = _struct("GluArgs", "XpGluArgs", a_ptr="z out", b_int="rows cols ld_z ld_out", c_float="limit up_add alpha cubic")
-GateMulArgs = _struct("GateMulArgs", "XpGateMulArgs", a_ptr="z e out", b_int="rows cols ld_z ld_e ld_out", c_float="alpha cubic")
+GateMulArgs = _struct("GateMulArgs", "XpGateMulArgs", a_ptr="z e out", b_int="rows cols ld_z ld_e ld_out", c_float="alpha cubic", d_int="kind")
 GroupedPrepArgs = _struct("GroupedPrepArgs", "XpGroupedPrepArgs", a_ptr="proj q_norm k_norm slots k_cache v_cache q_out",
-                          b_int="rows heads kv_heads group_pad dim vdim dq dv ld_proj q_off k_off v_off", c_float="eps", d_int="f32")
+                          b_int="rows heads kv_heads group_pad dim vdim dq dv ld_proj q_off k_off v_off", c_float="eps",
+                          d_int="f32 norm rot_pairs rot_positions interleaved", e_ptr="rot positions block_table k_pool v_pool",
+                          f_int="pool pool_page pool_rows page_size max_blocks")
+BlockMeanArgs = _struct("BlockMeanArgs", "XpBlockMeanArgs", a_ptr="k_cache v_cache k_pool v_pool row_seq positions slots block_table",
+                        b_int="rows kv_heads dq dv page_size max_blocks pool pool_page f32")
 GroupedAttnArgs = _struct("GroupedAttnArgs", "XpGroupedAttnArgs", a_ptr="q k_cache v_cache out gate row_seq positions slots block_table",
                           b_int="rows heads kv_heads group_pad dim vdim dq dv ld_gate ld_out page_size max_blocks", c_float="scale softcap",
-                          d_int="f32 window keep_first gate_elems")
+                          d_int="f32 window keep_first gate_elems", e_ptr="sink sigmoid_bias k_pool v_pool", f_int="pool pool_page")
 ConvRopeArgs = _struct("ConvRopeArgs", "XpConvRopeArgs",
                        a_ptr="proj conv_w ring rot positions slots state_slots q_starts q_lens k_cache v_cache q_out",
                        b_int="rows seqs max_q heads kv_heads group_pad dim vdim dq dv own_kv ld_proj q_off k_off v_off taps rot_pairs rot_positions "
@@ -325,12 +342,12 @@ MemoryArgs = _struct("MemoryArgs", "XpMemoryArgs", a_ptr="proj gates norm state 
                      c_float="qscale cap eps", d_int="f32")
 LatentPrepArgs = _struct("LatentPrepArgs", "XpLatentPrepArgs", a_ptr="proj norm_w freq positions slots cache q_plain q_abs q_exp",
                          b_int="rows heads dim rot rot_dims kv_rank ld_proj q_off kv_off ld_cache qp_rows dim_p ld_abs dq_pad abs_rows",
-                         c_float="eps", d_int="f32")
+                         c_float="eps", d_int="f32", e_ptr="q", f_int="ld_q q_rank ql_off interleaved")
 LatentAttnArgs = _struct("LatentAttnArgs", "XpLatentAttnArgs", a_ptr="q cache out gate row_seq positions slots block_table ws status",
                          b_int="rows heads kv_rank rot q_rows ld_q ld_cache ld_out ld_gate page_size max_blocks num_splits chunk_tokens",
-                         c_float="scale", d_int="f32 force_simt")
+                         c_float="scale", d_int="f32 force_simt window")
 LatentGatherArgs = _struct("LatentGatherArgs", "XpLatentGatherArgs", a_ptr="cache out block_table ctx_lens q_lens starts",
-                           b_int="n_seqs max_len page_size max_blocks ld_cache elem_bytes")
+                           b_int="n_seqs max_len page_size max_blocks ld_cache elem_bytes window")
 LinearAttnArgs = _struct("LinearAttnArgs", "XpLinearAttnArgs",
                          a_ptr="proj state decay decay_pow out positions slots state_slots q_starts q_lens ws",
                          b_int="rows seqs heads dim vdim ld_proj q_off k_off v_off force_sequential segs seg_tokens f32")
@@ -341,7 +358,7 @@ def _declare_mixers(lib: C.CDLL) -> None:
                      ("xp_latent_prep", LatentPrepArgs), ("xp_latent_attn", LatentAttnArgs), ("xp_latent_gather", LatentGatherArgs),
                      ("xp_linear_attn_decode", LinearAttnArgs), ("xp_linear_attn_prefill", LinearAttnArgs),
                      ("xp_post_norm", PostNormArgs), ("xp_head_gate", HeadGateArgs), ("xp_glu_f32", GluArgs), ("xp_gate_mul_f32", GateMulArgs),
-                     ("xp_grouped_prep", GroupedPrepArgs), ("xp_conv_rope_decode", ConvRopeArgs), ("xp_conv_rope_prefill", ConvRopeArgs), ("xp_grouped_attn", GroupedAttnArgs),
+                     ("xp_grouped_prep", GroupedPrepArgs), ("xp_block_mean", BlockMeanArgs), ("xp_conv_rope_decode", ConvRopeArgs), ("xp_conv_rope_prefill", ConvRopeArgs), ("xp_grouped_attn", GroupedAttnArgs),
                      ("xp_gated_linear_decode", GatedLinearArgs), ("xp_gated_linear_prefill", GatedLinearArgs),
                      ("xp_memory_decode", MemoryArgs), ("xp_memory_prefill", MemoryArgs), ("xp_delta_decode", DeltaArgs), ("xp_delta_prep", DeltaArgs), ("xp_delta_prefill", DeltaArgs)):
         getattr(lib, fn).restype = C.c_int

@@ -30,6 +30,7 @@ EPI_SWIGLU = 1
 EPI_RESIDUAL = 2
 EPI_STORE_F32 = 3
 EPI_GATE_MUL = 4
+EPI_SIGMOID = 5
 
 _WS_BYTES = 96 << 20
 _COUNTER_WORDS = 1 << 16
@@ -220,20 +221,39 @@ def _linear_f32(x, w, out, bias, out_scale=0.0, silu_cols=0, rows=None, n=None, 
         batch, sx, sw, so, out_scale, silu_cols, torch.cuda.current_stream(x.device).cuda_stream), "xp_gemm_f32")
 
 
-def linear_batched(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, out_group_stride: int) -> torch.Tensor:
+def linear_batched(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, out_group_stride: int, gate: torch.Tensor | None = None) -> torch.Tensor:
     """One small product per group (an attention head): ``x`` ``[groups, rows, k]`` with contiguous groups, ``w``
     ``[groups * n, k]``; row ``r`` of group ``g`` goes to ``out`` at element ``g * out_group_stride + r * out.stride(-2)``
-    (``out`` is a view whose last dimension is at least ``n`` wide)."""
+    (``out`` is a view whose last dimension is at least ``n`` wide). ``gate``: logits laid out like ``out`` (a pitch of their
+    own); the result is multiplied by their sigmoid."""
     groups, rows, k = x.shape
     n = w.shape[0] // groups
     assert x.stride(0) == rows * x.stride(1)
     if x.dtype == torch.float32:
         _linear_f32(x, w, out, None, rows=rows, n=n, batch=groups, sx=x.stride(0), sw=n * w.stride(0), so=out_group_stride)
+        if gate is not None:
+            from . import mixers
+
+            assert out.dim() == 2 and out.shape == gate.shape
+            mixers.sigmoid_mul_f32(out, gate, out)
         return out
-    a = _args(x[0], w, out, n_out=n, rows=rows, epilogue=EPI_STORE)
+    a = _args(x[0], w, out, n_out=n, rows=rows, epilogue=EPI_STORE if gate is None else EPI_SIGMOID, resid=gate)
     a.batch, a.x_group_rows, a.w_rows_per_group, a.out_group_stride = groups, rows, n, out_group_stride
     a.ld_out = out.stride(-2)
     native.check(native.kernels().xp_gemm(C.byref(a)), "xp_gemm(batched)")
+    return out
+
+
+def linear_relu2(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+    """``max(x @ w.T, 0)^2``; bf16 in the product's epilogue, fp32 by a row kernel behind it."""
+    if x.dtype == torch.float32:
+        from . import mixers
+
+        linear(x, w, out=out)
+        return mixers.relu2_f32(out, out)
+    a = _args(x, w, out, n_out=w.shape[0], rows=x.shape[0], epilogue=EPI_STORE)
+    a.relu2 = 1
+    native.check(native.kernels().xp_gemm(C.byref(a)), "xp_gemm(relu2)")
     return out
 
 

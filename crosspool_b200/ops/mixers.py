@@ -137,6 +137,25 @@ def gelu_gate(x: torch.Tensor, w: torch.Tensor, e: torch.Tensor, out: torch.Tens
     return out
 
 
+def sigmoid_mul_f32(z: torch.Tensor, e: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+    """``z * sigmoid(e)`` of fp32 rows (the bf16 product applies it in its epilogue); ``out`` may be ``z``."""
+    return _elementwise(z, e, out, 1)
+
+
+def relu2_f32(z: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+    """``max(z, 0)^2`` of fp32 rows (the bf16 product applies it in its epilogue); ``out`` may be ``z``."""
+    return _elementwise(z, None, out, 2)
+
+
+def _elementwise(z, e, out, kind: int) -> torch.Tensor:
+    assert z.dtype == out.dtype == torch.float32 and z.stride(1) == out.stride(1) == 1
+    a = native.GateMulArgs()
+    a.z, a.e, a.out, a.kind = z.data_ptr(), _ptr(e), out.data_ptr(), kind
+    a.rows, a.cols, a.ld_z, a.ld_e, a.ld_out = z.shape[0], z.shape[1], z.stride(0), e.stride(0) if e is not None else 0, out.stride(0)
+    native.check(native.kernels().xp_gate_mul_f32(C.byref(a), _stream(z)), "xp_gate_mul_f32")
+    return out
+
+
 def polynorm(z: torch.Tensor, coef: torch.Tensor, eps: float, out: torch.Tensor) -> torch.Tensor:
     """``c0 N(z) + c1 N(z^2) + c2 N(z^3) + c3`` per row, ``N`` dividing by the root mean square; ``out`` may be ``z``."""
     assert coef.dtype == torch.float32 and coef.numel() == 4 and out.dtype == z.dtype
@@ -162,9 +181,11 @@ def gated_rms(o: torch.Tensor, weight: torch.Tensor, gate: torch.Tensor, eps: fl
 
 def latent_prep(proj: torch.Tensor, norm_w: torch.Tensor, freq: torch.Tensor, positions: torch.Tensor, slots: torch.Tensor,
                 cache: torch.Tensor, *, heads: int, dim: int, rot: int, kv_rank: int, q_off: int, kv_off: int, eps: float,
-                abs_rows: int, q_plain: torch.Tensor | None, q_abs: torch.Tensor | None, q_exp: torch.Tensor | None) -> None:
+                abs_rows: int, q_plain: torch.Tensor | None, q_abs: torch.Tensor | None, q_exp: torch.Tensor | None,
+                q: torch.Tensor | None = None, q_rank: int = 0, interleaved: bool = False) -> None:
     """Latent norm, rotary positions, cache write and query layouts of ``proj`` ``[rows, ...]``. ``cache`` ``[pages, page,
-    1, width]``. Rows below ``abs_rows`` go to ``q_plain`` ``[heads, abs_rows, dim_p]`` and the rotary columns of ``q_abs``
+    1, width]``. Queries are the columns at ``q_off``, or ``q`` ``[rows, heads * (dim + rot)]``, a map of the ``q_rank`` columns at
+    ``q_off`` that is divided by their root mean square here. Rows below ``abs_rows`` go to ``q_plain`` ``[heads, abs_rows, dim_p]`` and the rotary columns of ``q_abs``
     ``[heads, abs_rows, width]``; the others to ``q_exp`` ``[rows, heads, dq]`` (zero-padded)."""
     a = native.LatentPrepArgs()
     assert freq.dtype == torch.float64 and norm_w.dtype == torch.float32 and cache.dtype == proj.dtype
@@ -175,7 +196,9 @@ def latent_prep(proj: torch.Tensor, norm_w: torch.Tensor, freq: torch.Tensor, po
     if q_plain is not None:
         a.qp_rows, a.dim_p, a.ld_abs = q_plain.shape[1], q_plain.shape[2], q_abs.shape[2]
     a.dq_pad = q_exp.shape[2] if q_exp is not None else 0
-    a.abs_rows, a.eps, a.f32 = abs_rows, eps, _f32(proj)
+    a.abs_rows, a.eps, a.f32, a.interleaved = abs_rows, eps, _f32(proj), int(interleaved)
+    if q is not None:
+        a.q, a.ld_q, a.q_rank, a.ql_off = q.data_ptr(), q.stride(0), q_rank, q_off
     native.check(native.kernels().xp_latent_prep(C.byref(a), _stream(proj)), "xp_latent_prep")
 
 
@@ -199,9 +222,10 @@ def latent_attn_plan(rows: int, heads: int, max_len: int, width: int = 576) -> t
 def latent_attn(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, block_table: torch.Tensor, positions: torch.Tensor,
                 slots: torch.Tensor, *, kv_rank: int, rot: int, scale: float, gate: torch.Tensor | None = None,
                 row_seq: torch.Tensor | None = None, num_splits: int = 1, chunk_tokens: int = 0, ws: torch.Tensor | None = None,
-                force_simt: bool = False) -> torch.Tensor:
+                force_simt: bool = False, window: int = 0) -> torch.Tensor:
     """Rows of latent-space queries ``q`` ``[heads, rows, width]`` against the latent cache; ``out`` ``[heads, rows, >= kv_rank]``.
-    Row ``r`` attends to the first ``positions[r] + 1`` tokens of its sequence. ``force_simt`` selects the plain kernel."""
+    Row ``r`` attends to the first ``positions[r] + 1`` tokens of its sequence (``window`` > 0: to the last ``window`` of those).
+    ``force_simt`` selects the plain kernel."""
     a = native.LatentAttnArgs()
     heads, rows = q.shape[0], q.shape[1]
     a.q, a.cache, a.out, a.gate, a.row_seq = q.data_ptr(), cache.data_ptr(), out.data_ptr(), _ptr(gate), _ptr(row_seq)
@@ -211,20 +235,22 @@ def latent_attn(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, block_t
     a.ld_gate = gate.stride(0) if gate is not None else 0
     a.page_size, a.max_blocks, a.num_splits, a.chunk_tokens = cache.shape[1], block_table.stride(0), num_splits, chunk_tokens
     assert num_splits == 1 or ws.numel() >= rows * heads * num_splits * (kv_rank + 2)
-    a.scale, a.f32, a.force_simt = scale, _f32(q), int(force_simt)
+    a.scale, a.f32, a.force_simt, a.window = scale, _f32(q), int(force_simt), window
     a.status = gemm.status_words(q.device).data_ptr()
     native.check(native.kernels().xp_latent_attn(C.byref(a), _stream(q)), "xp_latent_attn", 2 if num_splits > 1 else 1)
     return out
 
 
 def latent_gather(cache: torch.Tensor, out: torch.Tensor, block_table: torch.Tensor, ctx_lens: torch.Tensor, q_lens: torch.Tensor,
-                  starts: torch.Tensor, max_len: int) -> None:
-    """Dense copies of the sequences' cached rows: sequence i's tokens start at row ``starts[i]`` of ``out``."""
+                  starts: torch.Tensor, max_len: int, window: int = 0) -> None:
+    """Dense copies of the sequences' cached rows: sequence i's tokens start at row ``starts[i]`` of ``out``. With a ``window`` only
+    those from the 64-token boundary at or before the first token that the first query sees; ``max_len`` bounds the rows of a
+    sequence."""
     a = native.LatentGatherArgs()
     a.cache, a.out, a.block_table = cache.data_ptr(), out.data_ptr(), block_table.data_ptr()
     a.ctx_lens, a.q_lens, a.starts = ctx_lens.data_ptr(), q_lens.data_ptr(), starts.data_ptr()
     a.n_seqs, a.max_len, a.page_size, a.max_blocks = q_lens.shape[0], max_len, cache.shape[1], block_table.stride(0)
-    a.ld_cache, a.elem_bytes = cache.shape[-1], cache.element_size()
+    a.ld_cache, a.elem_bytes, a.window = cache.shape[-1], cache.element_size(), window
     native.check(native.kernels().xp_latent_gather(C.byref(a), _stream(cache)), "xp_latent_gather")
 
 
@@ -235,10 +261,11 @@ def expanded_shape(dim: int, rot: int, vdim: int) -> tuple[int, int] | None:
 
 def expanded_prefill(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, out: torch.Tensor, q_starts: torch.Tensor, q_lens: torch.Tensor,
                      ctx_lens: torch.Tensor, starts: torch.Tensor, max_q: int, *, scale: float, vdim: int,
-                     gate: torch.Tensor | None = None) -> None:
+                     gate: torch.Tensor | None = None, window: int = 0) -> None:
     """Causal attention of chunk queries ``q`` ``[rows, heads, dq]`` over dense per-head keys ``k`` ``[tokens, heads, dq]``
-    and values ``v`` ``[tokens, heads, dv]`` (sequence i's tokens start at row ``starts[i]``, a multiple of 64); ``out``
-    ``[rows, heads * vdim]``, head h multiplied by ``sigmoid(gate[:, h])``."""
+    and values ``v`` ``[tokens, heads, dv]`` (sequence i's tokens start at row ``starts[i]``, a multiple of 64; with a ``window``
+    those that :func:`latent_gather` leaves); ``out`` ``[rows, heads * vdim]``, multiplied by the sigmoid of ``gate``, which has
+    one column per head or one per output."""
     a = native.PrefillAttnArgs()
     a.q, a.k_cache, a.v_cache, a.out = q.data_ptr(), k.data_ptr(), v.data_ptr(), out.data_ptr()
     a.q_starts, a.q_lens, a.ctx_lens, a.seq_starts = q_starts.data_ptr(), q_lens.data_ptr(), ctx_lens.data_ptr(), starts.data_ptr()
@@ -246,7 +273,7 @@ def expanded_prefill(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, out: tor
     a.head_dim, a.v_dim, a.v_valid, a.ld_out = q.shape[2], v.shape[2], vdim, out.stride(0)
     a.page_size, a.max_blocks, a.num_pages = 64, 0, k.shape[0] // 64
     a.scale, a.total_q, a.p_pair = scale, q.shape[0], 1
-    a.gate = _ptr(gate)
+    a.gate, a.window, a.gate_elems = _ptr(gate), window, _gate_elems(gate, a.q_heads, vdim)
     a.ld_gate = gate.stride(0) if gate is not None else 0
     a.status = gemm.status_words(q.device).data_ptr()
     lib = native.kernels()
@@ -326,10 +353,26 @@ def group_pad(heads: int, kv_heads: int) -> int:
     return n
 
 
+@dataclass
+class BlockMeans:
+    """Means of whole blocks of ``size`` cached tokens, keys and values ``[pages, rows beside a page, kv_heads, width]``: block b of a
+    sequence is row ``b % rows`` beside page ``b // rows`` of its table."""
+
+    k: torch.Tensor
+    v: torch.Tensor
+    size: int
+
+    def put(self, a) -> None:
+        a.k_pool, a.v_pool, a.pool, a.pool_page = self.k.data_ptr(), self.v.data_ptr(), self.size, self.k.shape[1]
+
+
 def grouped_prep(proj: torch.Tensor, q_norm: torch.Tensor | None, k_norm: torch.Tensor | None, slots: torch.Tensor, k_cache: torch.Tensor,
-                 v_cache: torch.Tensor, q_out: torch.Tensor, *, heads: int, dim: int, vdim: int, offs: tuple[int, int, int], eps: float) -> None:
-    """Query and key norms, cache write and the padded query layout ``q_out`` ``[rows, kv_heads, group_pad, dq]``; caches
-    ``[pages, page, kv_heads, dq]`` and ``[..., dv]``."""
+                 v_cache: torch.Tensor, q_out: torch.Tensor, *, heads: int, dim: int, vdim: int, offs: tuple[int, int, int], eps: float,
+                 norm: bool = True, rot: torch.Tensor | None = None, interleaved: bool = False, positions: torch.Tensor | None = None,
+                 pool: BlockMeans | None = None, pool_rows: int = 0, block_table: torch.Tensor | None = None) -> None:
+    """Query and key norms (``norm``; with weights where there are any), rotation (``rot`` fp32 ``[positions, pairs, 2]``), cache
+    write and the padded query layout ``q_out`` ``[rows, kv_heads, group_pad, dq]``; caches ``[pages, page, kv_heads, dq]`` and
+    ``[..., dv]``. The first ``pool_rows`` rows (row r is sequence r) store the block means that they complete."""
     assert k_cache.dtype == proj.dtype == q_out.dtype and (q_norm is None or q_norm.dtype == torch.float32)
     a = native.GroupedPrepArgs()
     a.proj, a.q_norm, a.k_norm, a.slots = proj.data_ptr(), _ptr(q_norm), _ptr(k_norm), slots.data_ptr()
@@ -337,8 +380,33 @@ def grouped_prep(proj: torch.Tensor, q_norm: torch.Tensor | None, k_norm: torch.
     a.rows, a.heads, a.kv_heads, a.group_pad = proj.shape[0], heads, k_cache.shape[2], q_out.shape[2]
     a.dim, a.vdim, a.dq, a.dv, a.ld_proj = dim, vdim, k_cache.shape[3], v_cache.shape[3], proj.stride(0)
     a.q_off, a.k_off, a.v_off = offs
-    a.eps, a.f32 = eps, _f32(proj)
+    a.eps, a.f32, a.norm, a.interleaved, a.positions = eps, _f32(proj), int(norm), int(interleaved), _ptr(positions)
+    if rot is not None:
+        assert rot.dtype == torch.float32
+        a.rot, a.rot_positions, a.rot_pairs = rot.data_ptr(), rot.shape[0], rot.shape[1]
+    if pool is not None and pool_rows:
+        pool.put(a)
+        a.pool_rows, a.block_table, a.page_size, a.max_blocks = pool_rows, block_table.data_ptr(), k_cache.shape[1], block_table.stride(0)
     native.check(native.kernels().xp_grouped_prep(C.byref(a), _stream(proj)), "xp_grouped_prep")
+
+
+def block_means(k_cache: torch.Tensor, v_cache: torch.Tensor, pool: BlockMeans, block_table: torch.Tensor, positions: torch.Tensor,
+                slots: torch.Tensor, row_seq: torch.Tensor | None = None) -> None:
+    """Every row whose position completes a block stores the means of the block's cached keys and values."""
+    a = native.BlockMeanArgs()
+    a.k_cache, a.v_cache, a.row_seq, a.positions, a.slots = k_cache.data_ptr(), v_cache.data_ptr(), _ptr(row_seq), positions.data_ptr(), slots.data_ptr()
+    a.block_table, a.rows, a.kv_heads, a.dq, a.dv = block_table.data_ptr(), positions.shape[0], k_cache.shape[2], k_cache.shape[3], v_cache.shape[3]
+    a.page_size, a.max_blocks, a.f32 = k_cache.shape[1], block_table.stride(0), _f32(k_cache)
+    pool.put(a)
+    native.check(native.kernels().xp_block_mean(C.byref(a), _stream(k_cache)), "xp_block_mean")
+
+
+def _score_forms(a, heads: int, sink: torch.Tensor | None, sigmoid_bias: torch.Tensor | None, pool: BlockMeans | None) -> None:
+    for t in (sink, sigmoid_bias):
+        assert t is None or t.dtype == torch.float32 and t.numel() == heads
+    a.sink, a.sigmoid_bias = _ptr(sink), _ptr(sigmoid_bias)
+    if pool is not None:
+        pool.put(a)
 
 
 def _gate_elems(gate: torch.Tensor | None, heads: int, vdim: int) -> int:
@@ -378,10 +446,13 @@ def conv_rope(proj: torch.Tensor, conv_w: torch.Tensor | None, ring: torch.Tenso
 
 def grouped_attn(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, out: torch.Tensor, block_table: torch.Tensor,
                  positions: torch.Tensor, slots: torch.Tensor, *, heads: int, dim: int, vdim: int, scale: float, softcap: float = 0.0,
-                 gate: torch.Tensor | None = None, row_seq: torch.Tensor | None = None, window: int = 0, keep_first: int = 0) -> torch.Tensor:
+                 gate: torch.Tensor | None = None, row_seq: torch.Tensor | None = None, window: int = 0, keep_first: int = 0,
+                 sink: torch.Tensor | None = None, sigmoid_bias: torch.Tensor | None = None, pool: BlockMeans | None = None) -> torch.Tensor:
     """Rows of queries ``[rows, kv_heads, group_pad, dq]`` against the first ``positions[r] + 1`` cached tokens of their
-    sequences (``window`` > 0: the last ``window`` of those and the first ``keep_first``), any sizes and types; ``out`` ``[rows,
-    heads * vdim]``, multiplied by the sigmoid of ``gate``, which has one column per head or one per output."""
+    sequences (``window`` > 0: the last ``window`` of those and the first ``keep_first``, or with ``pool`` the means of the blocks
+    behind the window), any sizes and types; ``out`` ``[rows, heads * vdim]``, multiplied by the sigmoid of ``gate``, which has one
+    column per head or one per output. ``sink``: a number per head that joins the softmax's sum; ``sigmoid_bias``: weights are
+    ``sigmoid(score + bias)``, not normalised."""
     step = 32768
     for lo in range(0, q.shape[0], step):
         n = min(step, q.shape[0] - lo)
@@ -395,6 +466,7 @@ def grouped_attn(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, 
         a.dq, a.dv, a.ld_gate, a.ld_out = q.shape[3], v_cache.shape[3], gate.stride(0) if gate is not None else 0, out.stride(0)
         a.page_size, a.max_blocks, a.scale, a.softcap, a.f32 = k_cache.shape[1], block_table.stride(0), scale, softcap, _f32(q)
         a.window, a.keep_first, a.gate_elems = window, keep_first, _gate_elems(gate, heads, vdim)
+        _score_forms(a, heads, sink, sigmoid_bias, pool)
         native.check(native.kernels().xp_grouped_attn(C.byref(a), _stream(q)), "xp_grouped_attn")
     return out
 
@@ -402,7 +474,8 @@ def grouped_attn(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, 
 def grouped_decode(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, out: torch.Tensor, block_table: torch.Tensor,
                    positions: torch.Tensor, slots: torch.Tensor, *, heads: int, dim: int, vdim: int, scale: float, softcap: float = 0.0,
                    gate: torch.Tensor | None = None, row_seq: torch.Tensor | None = None, num_splits: int = 1, chunk_tokens: int = 0,
-                   ws: torch.Tensor | None = None, window: int = 0, keep_first: int = 0) -> torch.Tensor:
+                   ws: torch.Tensor | None = None, window: int = 0, keep_first: int = 0, sink: torch.Tensor | None = None,
+                   sigmoid_bias: torch.Tensor | None = None, pool: BlockMeans | None = None) -> torch.Tensor:
     """:func:`grouped_attn` on the tensor cores (bf16, widths of ``ATTENTION_SHAPES``, at most 16 query heads per key head).
     ``ws``: fp32, ``rows * heads * num_splits * (dv + 2)`` elements when ``num_splits`` > 1."""
     r = native.DecodeRowsArgs()
@@ -416,13 +489,15 @@ def grouped_decode(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor
     r.group_pad, r.v_dim, r.v_valid, r.ld_out, r.softcap = q.shape[2], v_cache.shape[3], vdim, out.stride(0), softcap
     r.ld_gate = gate.stride(0) if gate is not None else 0
     r.window, r.keep_first, r.gate_elems = window, keep_first, _gate_elems(gate, heads, vdim)
+    _score_forms(r, heads, sink, sigmoid_bias, pool)
     native.check(native.kernels().xp_decode_rows(C.byref(r), _stream(q)), "xp_decode_rows", 2 if num_splits > 1 else 1)
     return out
 
 
 def grouped_prefill(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, out: torch.Tensor, block_table: torch.Tensor,
                     q_starts: torch.Tensor, q_lens: torch.Tensor, ctx_lens: torch.Tensor, max_q: int, *, heads: int, vdim: int, scale: float,
-                    softcap: float = 0.0, gate: torch.Tensor | None = None, window: int = 0, keep_first: int = 0) -> torch.Tensor:
+                    softcap: float = 0.0, gate: torch.Tensor | None = None, window: int = 0, keep_first: int = 0, sink: torch.Tensor | None = None,
+                    sigmoid_bias: torch.Tensor | None = None, pool: BlockMeans | None = None) -> torch.Tensor:
     """Causal attention of portions (rows of ``q`` ``[rows, kv_heads, group_pad, dq]``) over the paged cache, which holds the
     portions' own tokens already, on tcgen05; ``out`` ``[rows, heads * vdim]``."""
     a = native.PrefillAttnArgs()
@@ -434,6 +509,7 @@ def grouped_prefill(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
     a.scale, a.total_q, a.p_pair, a.group_valid, a.softcap = scale, q.shape[0], 1, heads // q.shape[1], softcap
     a.gate, a.ld_gate = _ptr(gate), gate.stride(0) if gate is not None else 0
     a.window, a.keep_first, a.gate_elems = window, keep_first, _gate_elems(gate, heads, vdim)
+    _score_forms(a, heads, sink, sigmoid_bias, pool)
     a.status = gemm.status_words(q.device).data_ptr()
     native.check(native.kernels().xp_prefill_attn_umma(C.byref(a), _stream(q)), "xp_prefill_attn_umma")
     return out

@@ -117,7 +117,7 @@ def _stream(dev) -> int:
     return torch.cuda.current_stream(dev).cuda_stream
 
 
-def _router_args(logits: torch.Tensor, num_experts: int, top_k: int, out_ids: torch.Tensor, out_weights: torch.Tensor, sigmoid: bool = False,
+def _router_args(logits: torch.Tensor, num_experts: int, top_k: int, out_ids: torch.Tensor, out_weights: torch.Tensor, sigmoid: int = False,
                  renormalize: bool = True, scale: float = 1.0, logit_bias: torch.Tensor | None = None,
                  correction_bias: torch.Tensor | None = None, round_weights_bf16: bool = False) -> "native.RouterArgs":
     a = native.RouterArgs()
@@ -132,7 +132,7 @@ def _router_args(logits: torch.Tensor, num_experts: int, top_k: int, out_ids: to
 
 
 def router_topk(logits: torch.Tensor, num_experts: int, top_k: int, *, out_ids: torch.Tensor, out_weights: torch.Tensor, **kw) -> None:
-    """Scores (softmax, or ``sigmoid=True``), the ``top_k`` largest after ``correction_bias``, their weights (``renormalize``,
+    """Scores (softmax, or ``sigmoid=True``; 2: the choice by logits, softmax over the chosen), the ``top_k`` largest after ``correction_bias``, their weights (``renormalize``,
     ``scale``)."""
     a = _router_args(logits, num_experts, top_k, out_ids, out_weights, **kw)
     native.check(native.kernels().xp_router_topk(C.byref(a), _stream(logits.device)), "xp_router_topk")
@@ -147,10 +147,11 @@ def _tile_width(rows: int, top_k: int, n_local: int) -> int:
 
 
 def _grouped(x, w2d, out, *, n_out, rows_cap, bn, dual, up_offset, tiles, n_tiles, rows_per_group, epilogue, bias=None,
-             transform=(0.0, 0.0, 0.0)):
+             transform=(0.0, 0.0, 0.0), relu2=0):
     """``bias``: fp32 ``[experts, rows_per_group]``, indexed by the weight row of the stacked tensor."""
     a = gemm._args(x, w2d, out, n_out=n_out, rows=rows_cap, epilogue=epilogue, dual=dual, up_offset=up_offset, splits=1, bn=bn,
                    bias=bias, gate_limit=transform[0], up_add=transform[1], act_alpha=transform[2])
+    a.relu2 = relu2
     a.tile_table, a.n_tiles, a.w_rows_per_group = tiles.data_ptr(), n_tiles.data_ptr(), rows_per_group
     native.check(native.kernels().xp_gemm(C.byref(a)), "xp_gemm(grouped)")
 
@@ -245,7 +246,7 @@ class RoutedWorkspace:
             return torch.zeros(n, dtype=dt, device=device)
 
         top, experts, ff = max(s.top for s in specs), max(s.experts for s in specs), ceil8(max(max(s.ff, s.shared_ff) for s in specs))
-        routes, wide = cap * top, (max(2 * ff, hidden) + 127) // 128
+        routes, wide = cap * top, (max(2 * ff, hidden) + 127) // 128    # (ungated experts need half the tiles)
         tiles = wide * (routes // 16 + experts + 1)
         f32 = dtype == torch.float32
         return cls(buf(routes), buf(routes, torch.float32), buf(experts), buf(experts + 1), buf(routes), buf(routes), buf(4 * tiles),
@@ -270,8 +271,10 @@ def _grouped_f32(x, w, out, *, n, tiles, n_tiles, max_tiles) -> None:
                  "xp_gemm_f32_grouped")
 
 
-def _gated_rows(x: torch.Tensor, w_gate_up: torch.Tensor, act: torch.Tensor, z: torch.Tensor | None) -> torch.Tensor:
-    """``silu(gate) * up`` of plain rows in the rows' element type."""
+def _hidden_rows(x: torch.Tensor, w_gate_up: torch.Tensor, act: torch.Tensor, z: torch.Tensor | None, relu2: bool) -> torch.Tensor:
+    """``silu(gate) * up`` (or ``max(up, 0)^2``) of plain rows in the rows' element type."""
+    if relu2:
+        return gemm.linear_relu2(x, w_gate_up, act)
     if x.dtype == torch.float32:
         from . import mixers
 
@@ -293,9 +296,10 @@ def routed_ffn(x: torch.Tensor, w: FfnLayerWeights, spec: MoeSpec, out: torch.Te
     logits = ws.logits[:rows * ld].view(rows, ld)[:, :router.shape[0]]
     gemm.linear(x, router, out=logits)
     bn = 64 if f32 else _tile_width(rows, k, E)
-    n_gu = 2 * spec.ff if f32 else spec.ff
+    n_gu = spec.in_features if f32 else spec.ff
     ids, wts = ws.ids[:rows * k].view(rows, k), ws.weights[:rows * k].view(rows, k)
-    a = _router_args(logits, spec.routed, k, ids, wts, scale=spec.scale, correction_bias=w.extra["correction_bias"])
+    a = _router_args(logits, spec.routed, k, ids, wts, sigmoid=2 if spec.logit_choice else 0, scale=spec.scale,
+                     logit_bias=w.extra.get("router_bias"), correction_bias=w.extra.get("correction_bias"))
     r = _route_args(ws, rows, k, 0, E, n_gu, h, bn)
     if rows <= 128:
         native.check(lib.xp_moe_topk_route(C.byref(a), C.byref(r), s), "xp_moe_topk_route")
@@ -312,23 +316,29 @@ def routed_ffn(x: torch.Tensor, w: FfnLayerWeights, spec: MoeSpec, out: torch.Te
         from . import mixers
 
         most = routes // bn + E
-        z = ws.z[:routes * 2 * spec.ff].view(routes, 2 * spec.ff)
-        _grouped_f32(xp, w.gate_up, z, n=2 * spec.ff, tiles=ws.tiles_gu, n_tiles=ws.n_tiles[0:1], max_tiles=most * r.tm_gateup)
-        mixers.glu_f32(z, 0.0, 0.0, 1.0, act)
+        z = ws.z[:routes * n_gu].view(routes, n_gu)
+        _grouped_f32(xp, w.gate_up, z, n=n_gu, tiles=ws.tiles_gu, n_tiles=ws.n_tiles[0:1], max_tiles=most * r.tm_gateup)
+        if spec.relu2:
+            mixers.relu2_f32(z, act)
+        else:
+            mixers.glu_f32(z, 0.0, 0.0, 1.0, act)
         _grouped_f32(act, w.down, yp, n=h, tiles=ws.tiles_dn, n_tiles=ws.n_tiles[1:2], max_tiles=most * r.tm_down)
     else:
-        _grouped(xp, w.gate_up.flatten(0, 1), act, n_out=spec.ff, rows_cap=routes, bn=bn, dual=1, up_offset=spec.ff, tiles=ws.tiles_gu,
-                 n_tiles=ws.n_tiles[0:1], rows_per_group=2 * spec.ff, epilogue=gemm.EPI_SWIGLU)
+        _grouped(xp, w.gate_up.flatten(0, 1), act, n_out=spec.ff, rows_cap=routes, bn=bn, dual=int(not spec.relu2),
+                 up_offset=0 if spec.relu2 else spec.ff, tiles=ws.tiles_gu, n_tiles=ws.n_tiles[0:1], rows_per_group=spec.in_features,
+                 epilogue=gemm.EPI_STORE if spec.relu2 else gemm.EPI_SWIGLU, relu2=int(spec.relu2))
         _grouped(act, w.down.flatten(0, 1), yp, n_out=h, rows_cap=routes, bn=bn, dual=0, up_offset=0, tiles=ws.tiles_dn,
                  n_tiles=ws.n_tiles[1:2], rows_per_group=h, epilogue=gemm.EPI_STORE)
     m = native.MoeMixArgs()
     if spec.shared_ff:
         # the experts' products are done with these rows
         sact = ws.act[:rows * ceil8(spec.shared_ff)].view(rows, ceil8(spec.shared_ff))[:, :spec.shared_ff]
-        _gated_rows(x, w.shared_gate_up, sact, ws.z)
+        _hidden_rows(x, w.shared_gate_up, sact, ws.z, spec.relu2)
         shared = ws.shared[:rows * hp].view(rows, hp)[:, :h]
         gemm.linear(sact, w.shared_down, out=shared)
-        m.shared, m.ld_shared, m.shared_gate, m.ld_gate = shared.data_ptr(), shared.stride(0), logits[:, spec.routed:].data_ptr(), ld
+        m.shared, m.ld_shared = shared.data_ptr(), shared.stride(0)
+        if spec.shared_gate:
+            m.shared_gate, m.ld_gate = logits[:, spec.routed:].data_ptr(), ld
     m.y, m.x, m.topk_ids, m.route_pos, m.weights, m.out = (t.data_ptr() for t in (yp, x, ws.ids, ws.route_pos, ws.weights, out))
     m.rows, m.top_k, m.hidden, m.experts, m.ld_y, m.ld_x, m.ld_out, m.f32 = rows, k, h, E, hp, x.stride(0), out.stride(0), int(f32)
     native.check(lib.xp_moe_mix(C.byref(m), s), "xp_moe_mix")
