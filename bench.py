@@ -55,7 +55,7 @@ def parse_args(argv=None):
     ap.add_argument("--layers", type=int, default=0, help="debug only: truncate the models (marks the result invalid)")
     ap.add_argument("--lanes", type=int, default=2, help="Executor Lanes per FFN device (multi-GPU only)")
     ap.add_argument("--policy", default="fifo", choices=["fifo", "random", "slo"], help="Lane scheduling policy")
-    ap.add_argument("--layered", nargs="?", const="segirax", default="", choices=["segirax", "saninex", "kadavik"],
+    ap.add_argument("--layered", nargs="?", const="segirax", default="", choices=["segirax", "saninex", "kadavik", "dofevik"],
                     help="a layered decoder beside the closest classic model of equal size, rates and kernels (one GPU)")
     # steady-state decode replay (kernel-level)
     ap.add_argument("--decode-only", action="store_true")

@@ -1,6 +1,6 @@
 """Layered decoders beside the closest classic model of equal size on one GPU: ``bench.py --layered`` (Segirax),
-``--layered saninex`` and ``--layered kadavik`` (also beside Segirax; their sizes and kernels are in ``layered_saninex.py`` and
-``layered_kadavik.py``).
+``--layered saninex`` and ``--layered kadavik`` (also beside Segirax), ``--layered dofevik`` (also beside Kadavik); their sizes and
+kernels are in ``layered_saninex.py``, ``layered_kadavik.py`` and ``layered_dofevik.py``.
 
 Two sizes whose layers resemble a real model's (random weights, a few layers): latent attention and decayed linear attention
 alternate, each with a PolyNorm FFN that holds as many weights as the gated FFN of the classic model. For both models, in
@@ -223,7 +223,7 @@ def kernel_table(classic: ModelConfig, cfg: ModelConfig, timer: Timer, batch: in
 
 
 def run(steps: int = 20, warmup: int = 5, layers: int = 8, sizes=tuple(SIZES), design: str = "segirax") -> dict:
-    from . import layered_kadavik, layered_saninex
+    from . import layered_dofevik, layered_kadavik, layered_saninex
     from .decode_bench import ClockSampler
 
     torch.cuda.set_device(0)
@@ -236,15 +236,16 @@ def run(steps: int = 20, warmup: int = 5, layers: int = 8, sizes=tuple(SIZES), d
         name, heads = SIZES[size]
         classic = mc_preset(name).with_layers(layers)
         segirax = layered_twin(classic, heads, layers)
-        other = {"saninex": layered_saninex, "kadavik": layered_kadavik}.get(design)
+        other = {"saninex": layered_saninex, "kadavik": layered_kadavik, "dofevik": layered_dofevik}.get(design)
         cfg = segirax if other is None else other.twin(classic, heads, layers)
+        beside = ("kadavik", layered_kadavik.twin(classic, heads, layers)) if design == "dofevik" else ("segirax", segirax)
         res = {"classic": name, "layered": throughput(cfg, steps, warmup), "classic_rates": throughput(classic, steps, warmup)}
         torch.cuda.empty_cache()
         timer = Timer(max(10, steps), max(3, warmup), True)
         if other is None:
             res["kernels"] = kernel_table(classic, cfg, timer)
         else:
-            res["segirax_rates"] = throughput(segirax, steps, warmup)
+            res[beside[0] + "_rates"] = throughput(beside[1], steps, warmup)
             torch.cuda.empty_cache()
             res["kernels"] = other.kernel_table(classic, cfg, timer, CONTEXT, CHUNK, _row)
         torch.cuda.empty_cache()

@@ -150,6 +150,8 @@ class AttentionEngine:
                 raise UnsupportedAttention(f"{cfg.architecture}: layered decoders run their FFNs in-stream (LocalFfnPort), without attention TP")
             if e.prefix_cache and cfg.recurrent:
                 raise ValueError("prefix sharing needs a cache of pages; this model carries a recurrent state per sequence")
+            if e.prefix_cache and not cfg.pages_shareable(e.page_size):
+                raise ValueError(f"prefix sharing needs whole blocks per page; this model pools blocks that do not fill {e.page_size} tokens in eights")
         elif e.dtype != "bfloat16":
             raise ValueError(f"{cfg.architecture} runs in bfloat16 on the GPU engine")
         self.cfg, self.w, self.port = cfg, weights, port

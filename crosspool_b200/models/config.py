@@ -503,6 +503,12 @@ class ModelConfig:
         a cache page."""
         return any(s.mixer.state_elems or getattr(s.mixer, "conv_state_elems", 0) for s in self.layer_specs)
 
+    def pages_shareable(self, page_size: int) -> bool:
+        """Whether a page holds nothing but what its own tokens say: no state beside the pages, and no mean of a block that ends
+        behind its page."""
+        pools = [s.mixer for s in self.layer_specs if getattr(s.mixer, "pool", 0)]
+        return not self.recurrent and all(m.pool_page(page_size) * m.pool == page_size for m in pools)
+
     @property
     def gpu_attention_supported(self) -> bool:
         if self.layered:

@@ -149,6 +149,15 @@ def test_block_means_fit_beside_their_pages():
                 assert blocks == 0 or (blocks - 1) // n < pages
 
 
+def test_pages_that_hold_whole_blocks_can_be_shared():
+    from crosspool_b200.models import config as mc
+
+    for page, pool, ok in ((16, 2, True), (64, 8, True), (64, 4, True), (64, 7, False), (64, 16, False), (128, 16, True), (16, 8, False)):
+        c = mc.from_hf_config(dc.model(32, 40, [(dc.pooled(2, 1, 16, 9, pool), None)]))
+        assert c.pages_shareable(page) == ok, (page, pool)
+    assert mc.from_hf_config(dc.model(32, 40, [(dc.attention(2, 1, 16, 16, 9), None)])).pages_shareable(64)
+
+
 def test_parameter_counts_match_the_checkpoint():
     for name in dc.CASES:
         t, c = dc.tensors(name), _cfg(name)
