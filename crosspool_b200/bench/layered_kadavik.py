@@ -24,7 +24,7 @@ def twin(classic: ModelConfig, heads: int, layers: int) -> ModelConfig:
     ff = classic.intermediate_size
     memory = MemoryMixer(heads, DIM, DIM, 15.0)
     att = dict(heads=classic.num_q_heads, kv_heads=classic.num_kv_heads, dim=classic.head_dim, vdim=classic.head_dim, scale=classic.head_dim ** -0.5,
-               head_norms=False, conv=TAPS, rot=RotarySpec(64, 5e5, RotaryScaling(8.0, 1.0, 4.0, 8192)), window=WINDOW, keep_first=KEEP)
+               norm="", biases=False, gate="element", conv=TAPS, rot=RotarySpec(64, 5e5, RotaryScaling(8.0, 1.0, 4.0, 8192)), window=WINDOW, keep_first=KEEP)
     moe = MoeSpec(EXPERTS, TOP, ff // 4, IDENTITY, 2.5, ff // 4)
     specs = []
     for i in range(layers):
