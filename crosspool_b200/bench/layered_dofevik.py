@@ -126,7 +126,7 @@ def kernel_table(classic: ModelConfig, cfg: ModelConfig, timer, context: int, ch
         ab = n if dec else 0
         ps, sl, tb = (pos, slots, table) if dec else (p0, p0, tp)
         add(f"unit norm + rope + kv write {n}", lambda: M.grouped_prep(qkv[:n], None, None, sl, kc, vc, qp[:n], heads=hq, dim=d, vdim=d,
-                                                                      offs=(0, hq * d, (hq + hk) * d), eps=1e-6, rot=rot, interleaved=True, positions=ps),
+                                                                      offs=(0, hq * d, (hq + hk) * d), eps=1e-6, unit=True, rot=rot, interleaved=True, positions=ps),
             4 * n * (hq + 2 * hk) * d, 0.0, "rope + kv write")
         add(f"norm + kv write, tied{', block means' if dec else ''} {n}",
             lambda: M.grouped_prep(qkv[:n], ones, ones, sl, kc, vc, qp[:n], heads=hq, dim=d, vdim=d, offs=(0, hq * d, hq * d), eps=1e-6, positions=ps,
@@ -161,7 +161,7 @@ def kernel_table(classic: ModelConfig, cfg: ModelConfig, timer, context: int, ch
         if sp.shared_gate:
             w.extra["shared_scale"] = rnd(1, W, scale=0.02)
         w.extra["router_bias" if sp.logit_choice else "correction_bias"] = torch.zeros(E, device=dev)
-        moe.prepare_routed(w)
+        moe.prepare_routed(w, sp)
         rws = moe.RoutedWorkspace.for_layers([sp], W, T, bf, dev)
         for n in (batch, T):
             use, per = min(E, n * k), 2.0 * sp.maps * W * f

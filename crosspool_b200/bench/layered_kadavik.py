@@ -150,7 +150,7 @@ def kernel_table(classic: ModelConfig, cfg: ModelConfig, timer, context: int, ch
     plain = FfnLayerWeights(w.gate_up, w.down, router=w.router[:E].contiguous())
     w.shared_gate_up, w.shared_down, w.extra["shared_scale"] = rnd(2 * f, W, scale=0.02), rnd(W, f, scale=0.02), rnd(1, W, scale=0.02)
     w.extra["correction_bias"] = torch.zeros(spec.routed, device=dev)
-    moe.prepare_routed(w)
+    moe.prepare_routed(w, spec)
     rws = moe.RoutedWorkspace.for_layers([spec], W, T, bf, dev)
     cws = moe.workspace(dev, T, shape, f, E)
     for r in (batch, T):

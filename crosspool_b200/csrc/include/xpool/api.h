@@ -217,6 +217,7 @@ typedef struct XpRouterArgs {
   int sigmoid;                  /* scores: 0 softmax over all experts, 1 sigmoid, 2 softmax over the chosen logits (no correction) */
   int renormalize, round_weights_bf16;
   float scale;
+  int always;                   /* 1: every token also takes expert num_experts with weight 1, behind its top_k (rows of top_k + 1) */
 } XpRouterArgs;
 
 typedef struct XpRouteArgs {

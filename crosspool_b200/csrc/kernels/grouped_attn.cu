@@ -3,6 +3,8 @@
 // (attn_decode.cu, attn_prefill_umma.cu) do not cover.
 #include <math_constants.h>
 
+#include <type_traits>
+
 #include "xpool/elem.cuh"
 #include "xpool/mixer_api.h"
 
@@ -45,25 +47,31 @@ __device__ __forceinline__ void store_n(T* p, const float (&v)[N]) {
   }
 }
 
+// N elements as they lie in memory.
+template <typename T, int N>
+struct alignas(N * sizeof(T)) Raw {
+  T v[N];
+};
+
 // Row of a paged cache of `heads` heads of `width` elements.
 __device__ __forceinline__ size_t paged_row(const int* table, int t, int page_size, int heads, int h, int width) {
   return ((static_cast<size_t>(table[t / page_size]) * page_size + t % page_size) * heads + h) * width;
 }
 
 // Mean of the `pool` cached rows that end with token `last`, elements c .. c + N - 1 of head h. `own`, where given, is what the
-// cache holds for the last token.
-template <int N, typename T>
+// cache holds for the last token. kFlight rows are in flight.
+template <int N, int kFlight, typename T>
 __device__ __forceinline__ void block_mean(const T* cache, const int* table, int last, int pool, int page_size, int heads, int h, int width, int c,
                                            const float* own, float (&mean)[N]) {
 #pragma unroll
   for (int j = 0; j < N; ++j) mean[j] = 0.f;
   const int stop = own != nullptr ? last : last + 1;
-  for (int t = last + 1 - pool; t < stop; t += 4) {  // four rows in flight
-    float v[4][N];
+  for (int t = last + 1 - pool; t < stop; t += kFlight) {
+    float v[kFlight][N];
 #pragma unroll
-    for (int u = 0; u < 4; ++u) load_n<N>(cache + paged_row(table, min(t + u, stop - 1), page_size, heads, h, width) + c, v[u]);
+    for (int u = 0; u < kFlight; ++u) load_n<N>(cache + paged_row(table, min(t + u, stop - 1), page_size, heads, h, width) + c, v[u]);
 #pragma unroll
-    for (int u = 0; u < 4; ++u)
+    for (int u = 0; u < kFlight; ++u)
 #pragma unroll
       for (int j = 0; j < N; ++j) mean[j] += t + u < stop ? v[u][j] : 0.f;
   }
@@ -71,131 +79,137 @@ __device__ __forceinline__ void block_mean(const T* cache, const int* table, int
   for (int j = 0; j < N; ++j) mean[j] = (own != nullptr ? mean[j] + own[j] : mean[j]) / static_cast<float>(pool);
 }
 
-// L lanes per head slot of a row: padded query heads, then keys, then values. A lane takes N elements at a time.
-template <typename T, int N, int L>
+// One CTA per row, L lanes per head slot: padded query heads, then keys, then values. A lane takes N elements at a time and the
+// same columns of every slot it serves, so that it looks up their turns once; kAhead slots are in flight. kMeans: rows may complete
+// blocks.
+template <typename T, int N, int L, bool kMeans>
 __global__ void __launch_bounds__(kPrepThreads)
 grouped_prep_kernel(XpGroupedPrepArgs a) {
-  const int per_row = a.kv_heads * (a.group_pad + 2);
-  const int64_t unit = (static_cast<int64_t>(blockIdx.x) * kPrepThreads + threadIdx.x) / L;
-  const int lane = threadIdx.x % L;
-  const bool on = unit < static_cast<int64_t>(a.rows) * per_row;
-  const int row = on ? static_cast<int>(unit / per_row) : 0, u = on ? static_cast<int>(unit % per_row) : 0;
-  const int nq = a.kv_heads * a.group_pad;
+  constexpr int kAhead = N == 1 ? 1 : kMeans ? 2 : 4;
+  const int per_row = a.kv_heads * (a.group_pad + 2), nq = a.kv_heads * a.group_pad, group = a.heads / a.kv_heads;
+  const int row = blockIdx.x, lane = threadIdx.x % L, slots = blockDim.x / L;
   const T* proj = reinterpret_cast<const T*>(a.proj) + static_cast<size_t>(row) * a.ld_proj;
-  const T* src = nullptr;
-  T* dst = nullptr;
-  const T* cache = nullptr;                          // of a key or value head
-  const float* weight = nullptr;
-  bool query_or_key = true;
-  int n, width, h = 0;
-  if (u < nq) {
-    const int group = a.heads / a.kv_heads, g = u % a.group_pad;
-    if (g < group) src = proj + a.q_off + (u / a.group_pad * group + g) * a.dim;
-    dst = reinterpret_cast<T*>(a.q_out) + (static_cast<size_t>(row) * nq + u) * a.dq;
-    weight = a.q_norm, n = a.dim, width = a.dq;
-  } else {
-    const int slot = a.slots[row];
-    query_or_key = u < nq + a.kv_heads;
-    h = u - nq - (query_or_key ? 0 : a.kv_heads);
-    n = query_or_key ? a.dim : a.vdim;
-    width = query_or_key ? a.dq : a.dv;
-    src = proj + (query_or_key ? a.k_off : a.v_off) + h * n;
-    cache = reinterpret_cast<const T*>(query_or_key ? a.k_cache : a.v_cache);
-    if (slot >= 0) dst = const_cast<T*>(cache) + (static_cast<size_t>(slot) * a.kv_heads + h) * width;
-    if (query_or_key) weight = a.k_norm;
-  }
-  const bool work = on && dst != nullptr, read = work && src != nullptr;
-  const int c0 = lane * N;
-  float first[N];
-#pragma unroll
-  for (int j = 0; j < N; ++j) first[j] = 0.f;
-  if (read && c0 < n) load_n<N>(src + c0, first);
-  auto get = [&](int c, float (&x)[N]) {
-    if (c == c0) {
-#pragma unroll
-      for (int j = 0; j < N; ++j) x[j] = first[j];
-    } else {
-      load_n<N>(src + c, x);
-    }
-  };
-  float inv = 1.f;
-  if (a.norm) {
-    float ss = 0.f;
-    if (read && query_or_key)
-      for (int c = c0; c < n; c += L * N) {
-        float x[N];
-        get(c, x);
-#pragma unroll
-        for (int j = 0; j < N; ++j) ss += x[j] * x[j];
-      }
-#pragma unroll
-    for (int o = L / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-    if (query_or_key) inv = rsqrtf(ss / static_cast<float>(n) + a.eps);
-  }
-  if (!work) return;
-  const int rotated = query_or_key ? 2 * a.rot_pairs : 0;
+  const int cache_row = a.slots[row];
+  const int c0 = lane * N, rotated = 2 * a.rot_pairs;
   const int pos = a.positions != nullptr ? a.positions[row] : 0;
   const float2* turn = reinterpret_cast<const float2*>(a.rot) + static_cast<size_t>(pos < a.rot_positions ? pos : 0) * a.rot_pairs;
-  const bool means = cache != nullptr && a.pool > 0 && row < a.pool_rows && (pos + 1) % a.pool == 0;
-  for (int c = c0; c < width; c += L * N) {
-    float x[N];
+  auto pair_of = [&](int e) { return a.interleaved ? e >> 1 : e >= a.rot_pairs ? e - a.rot_pairs : e; };
+  float2 own_turn[N];
 #pragma unroll
-    for (int j = 0; j < N; ++j) x[j] = 0.f;
-    if (src != nullptr && c < n) {
-      get(c, x);
-      if (query_or_key) {
+  for (int j = 0; j < N; ++j) own_turn[j] = c0 + j < rotated ? turn[pair_of(c0 + j)] : make_float2(1.f, 0.f);
+  const bool means = kMeans && row < a.pool_rows && (pos + 1) % a.pool == 0;
+
+  for (int u0 = threadIdx.x / L; u0 < per_row + slots; u0 += slots * kAhead) {    // every lane of a warp takes part in the shuffles
+    if (__all_sync(0xffffffffu, u0 >= per_row)) break;
+    const T* src[kAhead];
+    T* dst[kAhead];
+    Raw<T, N> raw[kAhead];                           // the lane's first columns of every slot
 #pragma unroll
-        for (int j = 0; j < N; ++j) x[j] *= weight != nullptr ? inv * weight[c + j] : inv;
-        if (c < rotated) {
-          float y[N];
+    for (int k = 0; k < kAhead; ++k) {
+      const int u = u0 + k * slots;
+      src[k] = nullptr, dst[k] = nullptr;
+      if (u < nq) {
+        const int g = u % a.group_pad;
+        if (g < group) src[k] = proj + a.q_off + (u / a.group_pad * group + g) * a.dim;
+        dst[k] = reinterpret_cast<T*>(a.q_out) + (static_cast<size_t>(row) * nq + u) * a.dq;
+      } else if (u < per_row && cache_row >= 0) {
+        const bool is_k = u < nq + a.kv_heads;
+        const int h = u - nq - (is_k ? 0 : a.kv_heads);
+        src[k] = proj + (is_k ? a.k_off + h * a.dim : a.v_off + h * a.vdim);
+        dst[k] = is_k ? reinterpret_cast<T*>(a.k_cache) + (static_cast<size_t>(cache_row) * a.kv_heads + h) * a.dq
+                      : reinterpret_cast<T*>(a.v_cache) + (static_cast<size_t>(cache_row) * a.kv_heads + h) * a.dv;
+      }
+      const bool some = src[k] != nullptr && c0 < (u < nq + a.kv_heads ? a.dim : a.vdim);
+      raw[k] = *reinterpret_cast<const Raw<T, N>*>(some ? src[k] + c0 : proj + a.q_off);      // no branch around the load
+      if (!some) raw[k] = Raw<T, N>{};
+    }
 #pragma unroll
-          for (int j = 0; j < N; ++j) {
-            const int e = c + j;
-            y[j] = x[j];
-            if (e >= rotated) continue;
-            const bool second = a.interleaved ? e & 1 : e >= a.rot_pairs;
-            const int pair = a.interleaved ? e >> 1 : second ? e - a.rot_pairs : e;
-            float other;
-            if (a.interleaved && N > 1) {
-              other = x[j ^ (N > 1 ? 1 : 0)];
-            } else {
-              const int o = a.interleaved ? e ^ 1 : second ? e - a.rot_pairs : e + a.rot_pairs;
-              other = ld(src + o) * (weight != nullptr ? inv * weight[o] : inv);
-            }
-            const float2 t = turn[pair];
-            y[j] = second ? x[j] * t.x + other * t.y : x[j] * t.x - other * t.y;
+    for (int k = 0; k < kAhead; ++k) {
+      const int u = u0 + k * slots;
+      const bool qk = u < nq + a.kv_heads;
+      const int n = qk ? a.dim : a.vdim, width = qk ? a.dq : a.dv;
+      const float* weight = u < nq ? a.q_norm : a.k_norm;
+      float inv = 1.f, x0[N];
+#pragma unroll
+      for (int j = 0; j < N; ++j) x0[j] = ld(&raw[k].v[j]);
+      if (a.norm) {
+        float ss = 0.f;
+        if (src[k] != nullptr && qk) {
+#pragma unroll
+          for (int j = 0; j < N; ++j) ss += x0[j] * x0[j];
+          for (int c = c0 + L * N; c < n; c += L * N) {
+            float x[N];
+            load_n<N>(src[k] + c, x);
+#pragma unroll
+            for (int j = 0; j < N; ++j) ss += x[j] * x[j];
           }
+        }
 #pragma unroll
-          for (int j = 0; j < N; ++j) x[j] = y[j];
+        for (int o = L / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+        if (qk) inv = rsqrtf(ss / static_cast<float>(n) + a.eps);
+      }
+      if (dst[k] == nullptr) continue;
+      for (int c = c0; c < width; c += L * N) {
+        float x[N];
+#pragma unroll
+        for (int j = 0; j < N; ++j) x[j] = c == c0 ? x0[j] : 0.f;
+        if (src[k] != nullptr && c < n) {
+          if (c != c0) load_n<N>(src[k] + c, x);
+          if (qk) {
+#pragma unroll
+            for (int j = 0; j < N; ++j) x[j] *= weight != nullptr ? inv * weight[c + j] : inv;
+            if (c < rotated) {
+              float y[N];
+#pragma unroll
+              for (int j = 0; j < N; ++j) {
+                const int e = c + j;
+                y[j] = x[j];
+                if (e >= rotated) continue;
+                const bool second = a.interleaved ? e & 1 : e >= a.rot_pairs;
+                float other;
+                if (a.interleaved && N > 1) {
+                  other = x[j ^ (N > 1 ? 1 : 0)];
+                } else {
+                  const int o = a.interleaved ? e ^ 1 : second ? e - a.rot_pairs : e + a.rot_pairs;
+                  other = ld(src[k] + o) * (weight != nullptr ? inv * weight[o] : inv);
+                }
+                const float2 t = c == c0 ? own_turn[j] : turn[pair_of(e)];
+                y[j] = second ? x[j] * t.x + other * t.y : x[j] * t.x - other * t.y;
+              }
+#pragma unroll
+              for (int j = 0; j < N; ++j) x[j] = y[j];
+            }
+          }
+        }
+        store_n<N>(dst[k] + c, x);
+        if (kMeans && means && u >= nq) {
+          const int* table = a.block_table + static_cast<size_t>(row) * a.max_blocks;
+          const int h = u - nq - (qk ? 0 : a.kv_heads);
+          float own[N], mean[N];
+          T held[N];
+#pragma unroll
+          for (int j = 0; j < N; ++j) st(&held[j], x[j]), own[j] = ld(&held[j]);
+          block_mean<N, 4>(reinterpret_cast<const T*>(qk ? a.k_cache : a.v_cache), table, pos, a.pool, a.page_size, a.kv_heads, h, width, c, own, mean);
+          store_n<N>(reinterpret_cast<T*>(qk ? a.k_pool : a.v_pool) + paged_row(table, pos / a.pool, a.pool_page, a.kv_heads, h, width) + c, mean);
         }
       }
-    }
-    store_n<N>(dst + c, x);
-    if (means) {
-      float own[N], mean[N];
-      T held[N];
-#pragma unroll
-      for (int j = 0; j < N; ++j) st(&held[j], x[j]), own[j] = ld(&held[j]);
-      const int* table = a.block_table + static_cast<size_t>(row) * a.max_blocks;
-      block_mean<N>(cache, table, pos, a.pool, a.page_size, a.kv_heads, h, width, c, own, mean);
-      store_n<N>(reinterpret_cast<T*>(query_or_key ? a.k_pool : a.v_pool) + paged_row(table, pos / a.pool, a.pool_page, a.kv_heads, h, width) + c, mean);
     }
   }
 }
 
 // One CTA per row; most rows complete no block.
 template <typename T, int N>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(kPrepThreads)
 block_mean_kernel(XpBlockMeanArgs a) {
   const int row = blockIdx.x, pos = a.positions[row];
   if (a.slots[row] < 0 || (pos + 1) % a.pool != 0) return;
   const int* table = a.block_table + static_cast<size_t>(a.row_seq != nullptr ? a.row_seq[row] : row) * a.max_blocks;
   const int nk = a.kv_heads * a.dq, total = nk + a.kv_heads * a.dv;
-  for (int i = threadIdx.x * N; i < total; i += 128 * N) {
+  for (int i = threadIdx.x * N; i < total; i += kPrepThreads * N) {
     const bool is_k = i < nk;
     const int width = is_k ? a.dq : a.dv, e = is_k ? i : i - nk, h = e / width, c = e % width;
     float mean[N];
-    block_mean<N>(reinterpret_cast<const T*>(is_k ? a.k_cache : a.v_cache), table, pos, a.pool, a.page_size, a.kv_heads, h, width, c, nullptr, mean);
+    block_mean<N, 8>(reinterpret_cast<const T*>(is_k ? a.k_cache : a.v_cache), table, pos, a.pool, a.page_size, a.kv_heads, h, width, c, nullptr, mean);
     store_n<N>(reinterpret_cast<T*>(is_k ? a.k_pool : a.v_pool) + paged_row(table, pos / a.pool, a.pool_page, a.kv_heads, h, width) + c, mean);
   }
 }
@@ -312,19 +326,26 @@ extern "C" int xp_grouped_prep(const XpGroupedPrepArgs* a, void* stream) {
   const bool v = a->dim % n == 0 && a->vdim % n == 0 && a->dq % n == 0 && a->dv % n == 0 && a->ld_proj % n == 0 && a->q_off % n == 0 && a->k_off % n == 0 &&
                  a->v_off % n == 0 && al(a->proj) && al(a->k_cache) && al(a->v_cache) && al(a->q_out) && al(a->k_pool) && al(a->v_pool);
   const int widest = a->dq > a->dv ? a->dq : a->dv;
-  const int64_t units = static_cast<int64_t>(a->rows) * a->kv_heads * (a->group_pad + 2);
-  auto run = [&](auto kernel, int lanes) {
-    kernel<<<static_cast<unsigned>((units * lanes + kPrepThreads - 1) / kPrepThreads), kPrepThreads, 0, s>>>(*a);
+  const int units = a->kv_heads * (a->group_pad + 2);
+  auto run = [&](auto kernel, int lanes) {               // few rows: as many slots at a time as fit; many: four slots per thread
+    int threads = a->rows <= 512 ? units * lanes : (units * lanes + 3) / 4;
+    threads = (threads + 31) / 32 * 32;
+    kernel<<<a->rows, threads < kPrepThreads ? threads : kPrepThreads, 0, s>>>(*a);
   };
-  if (a->f32) {
-    if (!v) run(grouped_prep_kernel<float, 1, 32>, 32);
-    else if (widest <= 64) run(grouped_prep_kernel<float, 4, 16>, 16);
-    else run(grouped_prep_kernel<float, 4, 32>, 32);
-  } else {
-    if (!v) run(grouped_prep_kernel<__nv_bfloat16, 1, 32>, 32);
-    else if (widest <= 64) run(grouped_prep_kernel<__nv_bfloat16, 8, 8>, 8);
-    else run(grouped_prep_kernel<__nv_bfloat16, 8, 16>, 16);
-  }
+  auto pick = [&](auto means) {
+    constexpr bool M = decltype(means)::value;
+    if (a->f32) {
+      if (!v) run(grouped_prep_kernel<float, 1, 32, M>, 32);
+      else if (widest <= 64) run(grouped_prep_kernel<float, 4, 16, M>, 16);
+      else run(grouped_prep_kernel<float, 4, 32, M>, 32);
+    } else {
+      if (!v) run(grouped_prep_kernel<__nv_bfloat16, 1, 32, M>, 32);
+      else if (widest <= 64) run(grouped_prep_kernel<__nv_bfloat16, 8, 8, M>, 8);
+      else run(grouped_prep_kernel<__nv_bfloat16, 8, 16, M>, 16);
+    }
+  };
+  if (a->pool > 0 && a->pool_rows > 0) pick(std::true_type{});
+  else pick(std::false_type{});
   return done();
 }
 
@@ -336,11 +357,11 @@ extern "C" int xp_block_mean(const XpBlockMeanArgs* a, void* stream) {
   const int n = a->f32 ? 4 : 8;
   const bool v = a->dq % n == 0 && a->dv % n == 0 && al(a->k_cache) && al(a->v_cache) && al(a->k_pool) && al(a->v_pool);
   if (a->f32) {
-    if (v) block_mean_kernel<float, 4><<<a->rows, 128, 0, s>>>(*a);
-    else block_mean_kernel<float, 1><<<a->rows, 128, 0, s>>>(*a);
+    if (v) block_mean_kernel<float, 4><<<a->rows, kPrepThreads, 0, s>>>(*a);
+    else block_mean_kernel<float, 1><<<a->rows, kPrepThreads, 0, s>>>(*a);
   } else {
-    if (v) block_mean_kernel<__nv_bfloat16, 8><<<a->rows, 128, 0, s>>>(*a);
-    else block_mean_kernel<__nv_bfloat16, 1><<<a->rows, 128, 0, s>>>(*a);
+    if (v) block_mean_kernel<__nv_bfloat16, 8><<<a->rows, kPrepThreads, 0, s>>>(*a);
+    else block_mean_kernel<__nv_bfloat16, 1><<<a->rows, kPrepThreads, 0, s>>>(*a);
   }
   return done();
 }

@@ -534,6 +534,8 @@ latent_attn_tc_kernel(XpLatentAttnArgs a) {
     }
 }
 
+constexpr int kMaxSlices = 64;
+
 // One CTA per (head, row): folds the slices in order.
 __global__ void __launch_bounds__(128)
 latent_merge_kernel(XpLatentAttnArgs a) {
@@ -541,17 +543,42 @@ latent_merge_kernel(XpLatentAttnArgs a) {
   const bool pad = a.slots[row] < 0;
   const int len = pad ? 0 : a.positions[row] + 1;
   const int n = min(a.num_splits, (len - window_start(a, len) + a.chunk_tokens - 1) / a.chunk_tokens);
-  const float* w = a.ws + (static_cast<size_t>(row) * a.heads + h) * a.num_splits * (a.kv_rank + 2);
-  float m = -CUDART_INF_F, l = 0.f;
-  for (int s = 0; s < n; ++s) m = fmaxf(m, w[s * (a.kv_rank + 2) + a.kv_rank]);
-  for (int s = 0; s < n; ++s) l += w[s * (a.kv_rank + 2) + a.kv_rank + 1] * exp2f(w[s * (a.kv_rank + 2) + a.kv_rank] - m);
+  const int step = a.kv_rank + 2;
+  const float* w = a.ws + (static_cast<size_t>(row) * a.heads + h) * a.num_splits * step;
+  // the slices' maxima and sums, a slice per lane; every warp computes the same factors
+  __shared__ float scale_s[kMaxSlices];
+  const int lane = threadIdx.x & 31;
+  float ms[kMaxSlices / 32], ls[kMaxSlices / 32], m = -CUDART_INF_F, l = 0.f;
+#pragma unroll
+  for (int i = 0; i < kMaxSlices / 32; ++i) {
+    const int s = lane + 32 * i;
+    ms[i] = s < n ? w[s * step + a.kv_rank] : -CUDART_INF_F;
+    ls[i] = s < n ? w[s * step + a.kv_rank + 1] : 0.f;
+    m = fmaxf(m, ms[i]);
+  }
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
+#pragma unroll
+  for (int i = 0; i < kMaxSlices / 32; ++i) {
+    const float c = ms[i] == -CUDART_INF_F ? 0.f : exp2f(ms[i] - m);
+    l += ls[i] * c;
+    if (threadIdx.x < 32) scale_s[lane + 32 * i] = c;
+  }
+  l = elem::warp_sum(l);
   float f = pad ? 0.f : 1.f / l;
+  __syncthreads();
   if (a.gate != nullptr)
     f *= elem::sigmoid(elem::ld(reinterpret_cast<const __nv_bfloat16*>(a.gate) + static_cast<size_t>(row) * a.ld_gate + h));
   __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(a.out) + (static_cast<size_t>(h) * a.q_rows + row) * a.ld_out;
   for (int c = threadIdx.x; c < a.kv_rank; c += 128) {
     float v = 0.f;
-    for (int s = 0; s < n; ++s) v += w[s * (a.kv_rank + 2) + c] * exp2f(w[s * (a.kv_rank + 2) + a.kv_rank] - m);
+    for (int s0 = 0; s0 < n; s0 += 8) {              // eight slices in flight
+      float x[8];
+#pragma unroll
+      for (int u = 0; u < 8; ++u) x[u] = w[min(s0 + u, n - 1) * step + c];
+#pragma unroll
+      for (int u = 0; u < 8; ++u) v += s0 + u < n ? x[u] * scale_s[s0 + u] : 0.f;
+    }
     out[c] = __float2bfloat16_rn(v * f);
   }
 }
@@ -632,7 +659,7 @@ extern "C" int xp_latent_prep(const XpLatentPrepArgs* a, void* stream) {
 extern "C" int xp_latent_attn(const XpLatentAttnArgs* a, void* stream) {
   if (a->rows <= 0) return 0;
   if (a->heads <= 0 || a->kv_rank <= 0 || a->page_size <= 0 || a->rows > a->q_rows || a->ld_q < a->kv_rank + a->rot) return -10;
-  if (a->num_splits > 1 && (a->ws == nullptr || a->chunk_tokens <= 0)) return -11;
+  if (a->num_splits > 1 && (a->ws == nullptr || a->chunk_tokens <= 0 || a->num_splits > kMaxSlices)) return -11;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   if (!a->f32 && !a->force_simt && a->kv_rank <= 512 && a->ld_cache % 16 == 0 && a->ld_q % 8 == 0 && a->ld_q >= a->ld_cache) {
     int rc;

@@ -110,13 +110,17 @@ __device__ __forceinline__ void router_topk_row(const XpRouterArgs& a, int row, 
       my_id = be;
     }
   }
+  const size_t at = static_cast<size_t>(row) * (a.top_k + a.always) + lane;
   if (lane < a.top_k) {
     float w = my_w;
     if (a.renormalize && wsum > 0.f) w = w / wsum;
     w *= a.scale;
     if (a.round_weights_bf16) w = __bfloat162float(__float2bfloat16_rn(w));
-    a.topk_ids[static_cast<size_t>(row) * a.top_k + lane] = my_id;
-    a.topk_weights[static_cast<size_t>(row) * a.top_k + lane] = w;
+    a.topk_ids[at] = my_id;
+    a.topk_weights[at] = w;
+  } else if (lane == a.top_k && a.always) {
+    a.topk_ids[at] = E;
+    a.topk_weights[at] = 1.f;
   }
 }
 
@@ -342,6 +346,7 @@ moe_lane_topk_kernel(const lane::InstanceSlot* slots, const lane::LaneCur* cur, 
   a.ld_logits = m->e_pad;
   a.logits_fp32 = m->router_precision != 0;
   a.sigmoid = m->sigmoid;
+  a.always = 0;
   a.renormalize = m->renormalize;
   a.round_weights_bf16 = 0;
   a.scale = m->scale;
@@ -384,7 +389,7 @@ topk_route_kernel(XpRouterArgs a, XpRouteArgs r) {
   hist[e] = 0;
   for (int row = e >> 5; row < a.rows; row += 32) router_topk_row(a, row, e & 31);
   __syncthreads();                                   // the ids below were written by this CTA
-  const int n_routes = a.rows * a.top_k;
+  const int n_routes = a.rows * r.top_k;
   for (int i = e; i < n_routes; i += 1024) {
     const int x = a.topk_ids[i] - lo;
     if (x >= 0 && x < n_local) atomicAdd(&hist[x], 1);
@@ -583,7 +588,7 @@ extern "C" int xp_router_fp32(const void* x, int ldx, const void* w, int w_fp32,
 
 extern "C" int xp_router_topk(const XpRouterArgs* a, void* stream) {
   if (a->rows <= 0) return 0;
-  if (a->num_experts > 32 * kMaxPerLane || a->top_k > 32 || a->top_k > a->num_experts) return -10;
+  if (a->num_experts > 32 * kMaxPerLane || a->top_k + a->always > 32 || a->top_k > a->num_experts) return -10;
   router_topk_kernel<<<(a->rows + 3) / 4, 128, 0, reinterpret_cast<cudaStream_t>(stream)>>>(*a);
   return last_error();
 }
@@ -606,8 +611,8 @@ extern "C" int xp_moe_route(const XpRouteArgs* a, void* stream) {
 extern "C" int xp_moe_topk_route(const XpRouterArgs* a, const XpRouteArgs* r, void* stream) {
   if (a->rows <= 0) return 0;
   const int n_local = r->expert_hi - r->expert_lo;
-  if (a->num_experts > 32 * kMaxPerLane || a->top_k > 32 || a->top_k > a->num_experts || n_local < 1 || n_local > 256 || a->rows > 128 ||
-      a->rows != r->rows || a->top_k != r->top_k || a->topk_ids != r->topk_ids)
+  if (a->num_experts > 32 * kMaxPerLane || a->top_k + a->always > 32 || a->top_k > a->num_experts || n_local < 1 || n_local > 256 || a->rows > 128 ||
+      a->rows != r->rows || a->top_k + a->always != r->top_k || a->topk_ids != r->topk_ids)
     return -10;
   topk_route_kernel<<<1, 1024, 0, reinterpret_cast<cudaStream_t>(stream)>>>(*a, *r);
   return last_error();

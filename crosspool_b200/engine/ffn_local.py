@@ -49,9 +49,9 @@ class LocalFfnPort(FfnPort):
         if routed:
             from ..ops import moe
 
-            for w in self.weights:
+            for w, s in zip(self.weights, self.cfg.layer_specs):
                 if w is not None and w.is_moe:
-                    moe.prepare_routed(w)
+                    moe.prepare_routed(w, s.moe)
             self.moe_ws = moe.RoutedWorkspace.for_layers(routed, self.cfg.hidden_size, engine.cap, engine.dtype, engine.device)
         self.act = torch.zeros(engine.cap * inter, dtype=engine.dtype, device=engine.device)
         self.y = torch.zeros(engine.cap, ceil8(self.cfg.hidden_size), dtype=engine.dtype, device=engine.device)[:, :self.cfg.hidden_size]

@@ -230,7 +230,7 @@ class LayeredForward:
         if m.norm:
             rot = self.rot_tables.get(m.rot)
             M.grouped_prep(proj, lw.mix.get("q_norm"), lw.mix.get("k_norm"), b.slots, k, v, q, heads=m.heads, dim=m.dim, vdim=m.vdim,
-                           offs=(o["q"], o["k"], o["v"]), eps=self.e.cfg.rms_norm_eps, rot=rot, interleaved=rot is not None and m.rot.interleaved,
+                           offs=(o["q"], o["k"], o["v"]), eps=self.e.cfg.rms_norm_eps, unit=m.norm == "unit", rot=rot, interleaved=rot is not None and m.rot.interleaved,
                            positions=b.positions, pool=pool, pool_rows=b.n_dec, block_table=b.table)
         else:
             self._conv_rope(l, lw, m, proj, q, b)

@@ -401,6 +401,13 @@ class MoeSpec:
         return 2 if self.relu2 else 3
 
     @property
+    def folds_shared(self) -> bool:
+        """The shared expert runs as one more routed expert that every token takes: it has the experts' form and about their
+        width, and no gate."""
+        return (self.relu2 and not self.shared_gate and self.ff <= 2 * self.shared_ff <= 2 * self.ff and self.identity == 0 and self.top < 32
+                and self.experts < 256)
+
+    @property
     def in_features(self) -> int:
         """Rows of an expert's input map."""
         return self.ff * (self.maps - 1)

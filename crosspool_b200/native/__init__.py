@@ -509,7 +509,7 @@ class RouterArgs(C.Structure):
         ("topk_ids", C.c_void_p), ("topk_weights", C.c_void_p),
         ("rows", C.c_int), ("num_experts", C.c_int), ("top_k", C.c_int), ("ld_logits", C.c_int),
         ("logits_fp32", C.c_int), ("sigmoid", C.c_int), ("renormalize", C.c_int), ("round_weights_bf16", C.c_int),
-        ("scale", C.c_float),
+        ("scale", C.c_float), ("always", C.c_int),
     ]
 
 

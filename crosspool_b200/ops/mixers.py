@@ -368,9 +368,9 @@ class BlockMeans:
 
 def grouped_prep(proj: torch.Tensor, q_norm: torch.Tensor | None, k_norm: torch.Tensor | None, slots: torch.Tensor, k_cache: torch.Tensor,
                  v_cache: torch.Tensor, q_out: torch.Tensor, *, heads: int, dim: int, vdim: int, offs: tuple[int, int, int], eps: float,
-                 norm: bool = True, rot: torch.Tensor | None = None, interleaved: bool = False, positions: torch.Tensor | None = None,
+                 unit: bool = False, rot: torch.Tensor | None = None, interleaved: bool = False, positions: torch.Tensor | None = None,
                  pool: BlockMeans | None = None, pool_rows: int = 0, block_table: torch.Tensor | None = None) -> None:
-    """Query and key norms (``norm``; with weights where there are any), rotation (``rot`` fp32 ``[positions, pairs, 2]``), cache
+    """Query and key norms (with weights, or ``unit`` without any), rotation (``rot`` fp32 ``[positions, pairs, 2]``), cache
     write and the padded query layout ``q_out`` ``[rows, kv_heads, group_pad, dq]``; caches ``[pages, page, kv_heads, dq]`` and
     ``[..., dv]``. The first ``pool_rows`` rows (row r is sequence r) store the block means that they complete."""
     assert k_cache.dtype == proj.dtype == q_out.dtype and (q_norm is None or q_norm.dtype == torch.float32)
@@ -380,7 +380,7 @@ def grouped_prep(proj: torch.Tensor, q_norm: torch.Tensor | None, k_norm: torch.
     a.rows, a.heads, a.kv_heads, a.group_pad = proj.shape[0], heads, k_cache.shape[2], q_out.shape[2]
     a.dim, a.vdim, a.dq, a.dv, a.ld_proj = dim, vdim, k_cache.shape[3], v_cache.shape[3], proj.stride(0)
     a.q_off, a.k_off, a.v_off = offs
-    a.eps, a.f32, a.norm, a.interleaved, a.positions = eps, _f32(proj), int(norm), int(interleaved), _ptr(positions)
+    a.eps, a.f32, a.norm, a.interleaved, a.positions = eps, _f32(proj), int(unit or q_norm is not None), int(interleaved), _ptr(positions)
     if rot is not None:
         assert rot.dtype == torch.float32
         a.rot, a.rot_positions, a.rot_pairs = rot.data_ptr(), rot.shape[0], rot.shape[1]

@@ -138,10 +138,10 @@ def router_topk(logits: torch.Tensor, num_experts: int, top_k: int, *, out_ids: 
     native.check(native.kernels().xp_router_topk(C.byref(a), _stream(logits.device)), "xp_router_topk")
 
 
-def _tile_width(rows: int, top_k: int, n_local: int) -> int:
+def _tile_width(rows: int, top_k: int, n_local: int, widest: int = 128) -> int:
     avg = max(1, rows * top_k // max(1, n_local))
     bn = 16
-    while bn < avg and bn < 128:
+    while bn < avg and bn < widest:
         bn <<= 1
     return bn
 
@@ -245,7 +245,7 @@ class RoutedWorkspace:
         def buf(n, dt=torch.int32):
             return torch.zeros(n, dtype=dt, device=device)
 
-        top, experts, ff = max(s.top for s in specs), max(s.experts for s in specs), ceil8(max(max(s.ff, s.shared_ff) for s in specs))
+        top, experts, ff = max(s.top + s.folds_shared for s in specs), max(s.experts + s.folds_shared for s in specs), ceil8(max(max(s.ff, s.shared_ff) for s in specs))
         routes, wide = cap * top, (max(2 * ff, hidden) + 127) // 128    # (ungated experts need half the tiles)
         tiles = wide * (routes // 16 + experts + 1)
         f32 = dtype == torch.float32
@@ -255,9 +255,14 @@ class RoutedWorkspace:
                    buf(max(routes, cap) * 2 * ff, dtype) if f32 else None)
 
 
-def prepare_routed(w: FfnLayerWeights) -> None:
+def prepare_routed(w: FfnLayerWeights, spec: MoeSpec) -> None:
     """Puts a layer's weights in the layout of :func:`routed_ffn` (in place): the gate of the shared expert joins the router's
-    rows, row pitches become whole 16-byte units."""
+    rows, or the shared expert the routed ones; row pitches become whole 16-byte units."""
+    if spec.folds_shared:
+        pad = spec.ff - spec.shared_ff
+        w.gate_up = torch.cat([w.gate_up, torch.nn.functional.pad(w.shared_gate_up, (0, 0, 0, pad))[None]])
+        w.down = torch.cat([w.down, torch.nn.functional.pad(w.shared_down, (0, pad))[None]])
+        w.shared_gate_up = w.shared_down = None
     w.gate_up, w.down = pad_pitch(w.gate_up), pad_pitch(w.down)
     scale = w.extra.get("shared_scale")
     w.extra["router_rows"] = pad_pitch(w.router if scale is None else torch.cat([w.router, scale.to(w.router.dtype)], 0))
@@ -287,20 +292,25 @@ def _hidden_rows(x: torch.Tensor, w_gate_up: torch.Tensor, act: torch.Tensor, z:
 def routed_ffn(x: torch.Tensor, w: FfnLayerWeights, spec: MoeSpec, out: torch.Tensor, ws: RoutedWorkspace) -> torch.Tensor:
     """Routed FFN of ``x`` ``[rows, hidden]`` (any width, bf16 or fp32): fp32 router logits of one product (the shared
     expert's gate is its last column), routes ordered by expert, two grouped products, and one kernel that adds up the
-    chosen experts, the identity experts and the shared expert. Few rows choose and order in one launch."""
+    chosen experts, the identity experts and the shared expert (which may be one more of the former). Few rows choose and order
+    in one launch."""
     rows, h = x.shape
     f32, lib, s = x.dtype == torch.float32, native.kernels(), _stream(x.device)
-    hp, ffp, E, k = ceil8(h), ceil8(spec.ff), spec.experts, spec.top
+    hp, ffp, fold = ceil8(h), ceil8(spec.ff), spec.folds_shared
+    E, k = spec.experts + fold, spec.top + fold
     router = w.extra["router_rows"]
     ld = ceil8(router.shape[0])
     logits = ws.logits[:rows * ld].view(rows, ld)[:, :router.shape[0]]
     gemm.linear(x, router, out=logits)
-    bn = 64 if f32 else _tile_width(rows, k, E)
+    bn = 64 if f32 else _tile_width(rows, k, E, 256)
+    bn_gu = min(bn, 256 if spec.relu2 else 128)            # a gated tile holds two accumulators
     n_gu = spec.in_features if f32 else spec.ff
     ids, wts = ws.ids[:rows * k].view(rows, k), ws.weights[:rows * k].view(rows, k)
-    a = _router_args(logits, spec.routed, k, ids, wts, sigmoid=2 if spec.logit_choice else 0, scale=spec.scale,
+    a = _router_args(logits, spec.routed, spec.top, ids, wts, sigmoid=2 if spec.logit_choice else 0, scale=spec.scale,
                      logit_bias=w.extra.get("router_bias"), correction_bias=w.extra.get("correction_bias"))
+    a.always = int(fold)
     r = _route_args(ws, rows, k, 0, E, n_gu, h, bn)
+    r.bn_gateup = bn_gu
     if rows <= 128:
         native.check(lib.xp_moe_topk_route(C.byref(a), C.byref(r), s), "xp_moe_topk_route")
     else:
@@ -324,13 +334,13 @@ def routed_ffn(x: torch.Tensor, w: FfnLayerWeights, spec: MoeSpec, out: torch.Te
             mixers.glu_f32(z, 0.0, 0.0, 1.0, act)
         _grouped_f32(act, w.down, yp, n=h, tiles=ws.tiles_dn, n_tiles=ws.n_tiles[1:2], max_tiles=most * r.tm_down)
     else:
-        _grouped(xp, w.gate_up.flatten(0, 1), act, n_out=spec.ff, rows_cap=routes, bn=bn, dual=int(not spec.relu2),
+        _grouped(xp, w.gate_up.flatten(0, 1), act, n_out=spec.ff, rows_cap=routes, bn=bn_gu, dual=int(not spec.relu2),
                  up_offset=0 if spec.relu2 else spec.ff, tiles=ws.tiles_gu, n_tiles=ws.n_tiles[0:1], rows_per_group=spec.in_features,
                  epilogue=gemm.EPI_STORE if spec.relu2 else gemm.EPI_SWIGLU, relu2=int(spec.relu2))
         _grouped(act, w.down.flatten(0, 1), yp, n_out=h, rows_cap=routes, bn=bn, dual=0, up_offset=0, tiles=ws.tiles_dn,
                  n_tiles=ws.n_tiles[1:2], rows_per_group=h, epilogue=gemm.EPI_STORE)
     m = native.MoeMixArgs()
-    if spec.shared_ff:
+    if spec.shared_ff and not fold:
         # the experts' products are done with these rows
         sact = ws.act[:rows * ceil8(spec.shared_ff)].view(rows, ceil8(spec.shared_ff))[:, :spec.shared_ff]
         _hidden_rows(x, w.shared_gate_up, sact, ws.z, spec.relu2)

@@ -99,7 +99,7 @@ def test_routed_ffn_of_squared_relu_experts(rows, h, E, top, ff, shared, dtype):
     if shared:
         t.update({"shared.up": _rnd(shared, h, seed=6, dtype=bf, scale=h ** -0.5), "shared.down": _rnd(h, shared, seed=7, dtype=bf, scale=shared ** -0.5)})
         w.shared_gate_up, w.shared_down = t["shared.up"].to(dtype), t["shared.down"].to(dtype)
-    moe.prepare_routed(w)
+    moe.prepare_routed(w, spec)
     x = _pitched(rows, h, dtype, 3)
     ws = moe.RoutedWorkspace.for_layers([spec, MoeSpec(2, 1, 8, **kw)], h, 400, dtype, torch.device("cuda"))
     out = torch.full((rows, (h + 7) // 8 * 8), 7.0, dtype=dtype, device="cuda")
@@ -181,7 +181,7 @@ def test_norms_rotation_cache_rows_and_block_means(H, G, d, e, pairs, form, dtyp
     bm, _ = _blocks([h[:n - 1] for h, n in zip(hist[0], lens)], [h[:n - 1] for h, n in zip(hist[1], lens)], G, dq, dv, pool, table, [n - 1 for n in lens], page, dtype, 9.0)
     before = bm.k.clone(), bm.v.clone()
     q = torch.full((rows + 1, G, M.group_pad(H, G), dq), 9.0, dtype=dtype, device="cuda")
-    M.grouped_prep(proj, qn, kn, slots, kc, vc, q, heads=H, dim=d, vdim=e, offs=(off_q, off_k, off_v), eps=1e-3, rot=rot, interleaved=neighbours and pairs > 0,
+    M.grouped_prep(proj, qn, kn, slots, kc, vc, q, heads=H, dim=d, vdim=e, offs=(off_q, off_k, off_v), eps=1e-3, unit=form == "unit", rot=rot, interleaved=neighbours and pairs > 0,
                    positions=pos, pool=bm, pool_rows=rows, block_table=table)
     x = _cpu(proj)
 

@@ -156,7 +156,7 @@ def test_routed_ffn(rows, h, E, top, ff, ident, shared, dtype):
                   "shared.down": _rnd(h, shared, seed=7, dtype=torch.bfloat16, scale=shared ** -0.5), "shared.sg": _rnd(1, h, seed=8, dtype=torch.bfloat16)})
         w.shared_gate_up, w.shared_down = torch.cat([t["shared.gate"], t["shared.up"]]).to(dtype), t["shared.down"].to(dtype)
         w.extra["shared_scale"] = t["shared.sg"].to(dtype)
-    moe.prepare_routed(w)
+    moe.prepare_routed(w, spec)
     x = _pitched(rows, h, torch.bfloat16, 3).to(dtype)
     if x.stride(0) % 8:
         x = _pitched(rows, h, dtype, 3).copy_(x)
