@@ -79,109 +79,116 @@ __device__ __forceinline__ void block_mean(const T* cache, const int* table, int
   for (int j = 0; j < N; ++j) mean[j] = (own != nullptr ? mean[j] + own[j] : mean[j]) / static_cast<float>(pool);
 }
 
-// One CTA per row, L lanes per head slot: padded query heads, then keys, then values. A lane takes N elements at a time and the
-// same columns of every slot it serves, so that it looks up their turns once; kAhead slots are in flight. kMeans: rows may complete
-// blocks.
-template <typename T, int N, int L, bool kMeans>
-__global__ void __launch_bounds__(kPrepThreads)
+// A CTA (or several, grid y) per row, L lanes per head slot: padded query heads, then keys, then values. A lane takes N elements at a time and the
+// same columns of every slot it serves, so that it looks up their turns once; kAhead slots are in flight, and registers are kept
+// for four CTAs of 256 threads. kInter: pairs of neighbours turn. kMeans: rows may complete blocks.
+template <typename T, int N, int L, bool kInter, bool kMeans>
+__global__ void __launch_bounds__(kPrepThreads, kMeans ? 2 : 4)
 grouped_prep_kernel(XpGroupedPrepArgs a) {
   constexpr int kAhead = N == 1 ? 1 : kMeans ? 2 : 4;
+  constexpr int kTurns = kInter && N > 1 ? N / 2 : N;
   const int per_row = a.kv_heads * (a.group_pad + 2), nq = a.kv_heads * a.group_pad, group = a.heads / a.kv_heads;
-  const int row = blockIdx.x, lane = threadIdx.x % L, slots = blockDim.x / L;
+  const int row = blockIdx.x, lane = threadIdx.x % L, slots = blockDim.x / L * gridDim.y;   // slots at a time
   const T* proj = reinterpret_cast<const T*>(a.proj) + static_cast<size_t>(row) * a.ld_proj;
-  const int cache_row = a.slots[row];
   const int c0 = lane * N, rotated = 2 * a.rot_pairs;
+  // first column of a slot in the row, -1: padding of a group
+  auto column = [&](int u) {
+    if (u < nq) {
+      const int q = u / a.group_pad, g = u - q * a.group_pad;
+      return g < group ? a.q_off + (q * group + g) * a.dim : -1;
+    }
+    const int h = u - nq;
+    return h < a.kv_heads ? a.k_off + h * a.dim : a.v_off + (h - a.kv_heads) * a.vdim;
+  };
+  const int cache_row = a.slots[row];
   const int pos = a.positions != nullptr ? a.positions[row] : 0;
   const float2* turn = reinterpret_cast<const float2*>(a.rot) + static_cast<size_t>(pos < a.rot_positions ? pos : 0) * a.rot_pairs;
-  auto pair_of = [&](int e) { return a.interleaved ? e >> 1 : e >= a.rot_pairs ? e - a.rot_pairs : e; };
-  float2 own_turn[N];
+  auto pair_of = [&](int e) { return kInter ? e >> 1 : e >= a.rot_pairs ? e - a.rot_pairs : e; };
+  float2 own_turn[kTurns];
 #pragma unroll
-  for (int j = 0; j < N; ++j) own_turn[j] = c0 + j < rotated ? turn[pair_of(c0 + j)] : make_float2(1.f, 0.f);
+  for (int j = 0; j < kTurns; ++j) {
+    const int e = c0 + j * (N / kTurns);
+    own_turn[j] = e < rotated ? turn[pair_of(e)] : make_float2(1.f, 0.f);
+  }
   const bool means = kMeans && row < a.pool_rows && (pos + 1) % a.pool == 0;
 
-  for (int u0 = threadIdx.x / L; u0 < per_row + slots; u0 += slots * kAhead) {    // every lane of a warp takes part in the shuffles
+  for (int u0 = blockIdx.y * (blockDim.x / L) + threadIdx.x / L; u0 < per_row + slots; u0 += slots * kAhead) {    // every lane of a warp takes part in the shuffles
     if (__all_sync(0xffffffffu, u0 >= per_row)) break;
-    const T* src[kAhead];
-    T* dst[kAhead];
     Raw<T, N> raw[kAhead];                           // the lane's first columns of every slot
 #pragma unroll
     for (int k = 0; k < kAhead; ++k) {
       const int u = u0 + k * slots;
-      src[k] = nullptr, dst[k] = nullptr;
-      if (u < nq) {
-        const int g = u % a.group_pad;
-        if (g < group) src[k] = proj + a.q_off + (u / a.group_pad * group + g) * a.dim;
-        dst[k] = reinterpret_cast<T*>(a.q_out) + (static_cast<size_t>(row) * nq + u) * a.dq;
-      } else if (u < per_row && cache_row >= 0) {
-        const bool is_k = u < nq + a.kv_heads;
-        const int h = u - nq - (is_k ? 0 : a.kv_heads);
-        src[k] = proj + (is_k ? a.k_off + h * a.dim : a.v_off + h * a.vdim);
-        dst[k] = is_k ? reinterpret_cast<T*>(a.k_cache) + (static_cast<size_t>(cache_row) * a.kv_heads + h) * a.dq
-                      : reinterpret_cast<T*>(a.v_cache) + (static_cast<size_t>(cache_row) * a.kv_heads + h) * a.dv;
-      }
-      const bool some = src[k] != nullptr && c0 < (u < nq + a.kv_heads ? a.dim : a.vdim);
-      raw[k] = *reinterpret_cast<const Raw<T, N>*>(some ? src[k] + c0 : proj + a.q_off);      // no branch around the load
+      const int at = u < per_row ? column(u) : -1;
+      const bool some = at >= 0 && c0 < (u < nq + a.kv_heads ? a.dim : a.vdim);
+      raw[k] = *reinterpret_cast<const Raw<T, N>*>(proj + (some ? at + c0 : a.q_off));      // no branch around the load
       if (!some) raw[k] = Raw<T, N>{};
     }
 #pragma unroll
     for (int k = 0; k < kAhead; ++k) {
       const int u = u0 + k * slots;
       const bool qk = u < nq + a.kv_heads;
-      const int n = qk ? a.dim : a.vdim, width = qk ? a.dq : a.dv;
+      const int at = u < per_row ? column(u) : -1;
+      const T* src = proj + at;
+      const int n = at < 0 ? 0 : qk ? a.dim : a.vdim, width = qk ? a.dq : a.dv;
       const float* weight = u < nq ? a.q_norm : a.k_norm;
-      float inv = 1.f, x0[N];
+      float inv = 1.f, x[N];
 #pragma unroll
-      for (int j = 0; j < N; ++j) x0[j] = ld(&raw[k].v[j]);
+      for (int j = 0; j < N; ++j) x[j] = ld(&raw[k].v[j]);
       if (a.norm) {
         float ss = 0.f;
-        if (src[k] != nullptr && qk) {
 #pragma unroll
-          for (int j = 0; j < N; ++j) ss += x0[j] * x0[j];
-          for (int c = c0 + L * N; c < n; c += L * N) {
-            float x[N];
-            load_n<N>(src[k] + c, x);
+        for (int j = 0; j < N; ++j) ss += x[j] * x[j];
+        for (int c = c0 + L * N; c < n; c += L * N) {
+          float y[N];
+          load_n<N>(src + c, y);
 #pragma unroll
-            for (int j = 0; j < N; ++j) ss += x[j] * x[j];
-          }
+          for (int j = 0; j < N; ++j) ss += y[j] * y[j];
         }
 #pragma unroll
         for (int o = L / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-        if (qk) inv = rsqrtf(ss / static_cast<float>(n) + a.eps);
+        if (qk && n > 0) inv = rsqrtf(ss / static_cast<float>(n) + a.eps);
       }
-      if (dst[k] == nullptr) continue;
+      if (u >= per_row || (u >= nq && cache_row < 0)) continue;
+      T* dst;
+      if (u < nq) {
+        dst = reinterpret_cast<T*>(a.q_out) + (static_cast<size_t>(row) * nq + u) * a.dq;
+      } else {
+        const int h = u - nq - (qk ? 0 : a.kv_heads);
+        dst = (qk ? reinterpret_cast<T*>(a.k_cache) : reinterpret_cast<T*>(a.v_cache)) + (static_cast<size_t>(cache_row) * a.kv_heads + h) * width;
+      }
       for (int c = c0; c < width; c += L * N) {
-        float x[N];
+        if (c != c0) {
 #pragma unroll
-        for (int j = 0; j < N; ++j) x[j] = c == c0 ? x0[j] : 0.f;
-        if (src[k] != nullptr && c < n) {
-          if (c != c0) load_n<N>(src[k] + c, x);
-          if (qk) {
+          for (int j = 0; j < N; ++j) x[j] = 0.f;
+          if (c < n) load_n<N>(src + c, x);
+        }
+        if (qk && c < n) {
 #pragma unroll
-            for (int j = 0; j < N; ++j) x[j] *= weight != nullptr ? inv * weight[c + j] : inv;
-            if (c < rotated) {
-              float y[N];
+          for (int j = 0; j < N; ++j) x[j] *= weight != nullptr ? inv * weight[c + j] : inv;
+          if (c < rotated) {
+            if constexpr (kInter && N > 1) {
+#pragma unroll
+              for (int j = 0; j < N; j += 2) {
+                if (c + j >= rotated) continue;
+                const float2 t = c == c0 ? own_turn[j / 2] : turn[(c + j) >> 1];
+                const float v = x[j], w = x[j + 1];
+                x[j] = v * t.x - w * t.y, x[j + 1] = w * t.x + v * t.y;
+              }
+            } else {
 #pragma unroll
               for (int j = 0; j < N; ++j) {
                 const int e = c + j;
-                y[j] = x[j];
                 if (e >= rotated) continue;
-                const bool second = a.interleaved ? e & 1 : e >= a.rot_pairs;
-                float other;
-                if (a.interleaved && N > 1) {
-                  other = x[j ^ (N > 1 ? 1 : 0)];
-                } else {
-                  const int o = a.interleaved ? e ^ 1 : second ? e - a.rot_pairs : e + a.rot_pairs;
-                  other = ld(src[k] + o) * (weight != nullptr ? inv * weight[o] : inv);
-                }
+                const bool second = kInter ? e & 1 : e >= a.rot_pairs;
+                const int o = kInter ? e ^ 1 : second ? e - a.rot_pairs : e + a.rot_pairs;
+                const float other = ld(src + o) * (weight != nullptr ? inv * weight[o] : inv);
                 const float2 t = c == c0 ? own_turn[j] : turn[pair_of(e)];
-                y[j] = second ? x[j] * t.x + other * t.y : x[j] * t.x - other * t.y;
+                x[j] = second ? x[j] * t.x + other * t.y : x[j] * t.x - other * t.y;
               }
-#pragma unroll
-              for (int j = 0; j < N; ++j) x[j] = y[j];
             }
           }
         }
-        store_n<N>(dst[k] + c, x);
+        store_n<N>(dst + c, x);
         if (kMeans && means && u >= nq) {
           const int* table = a.block_table + static_cast<size_t>(row) * a.max_blocks;
           const int h = u - nq - (qk ? 0 : a.kv_heads);
@@ -197,20 +204,28 @@ grouped_prep_kernel(XpGroupedPrepArgs a) {
   }
 }
 
-// One CTA per row; most rows complete no block.
+// A CTA looks at kMeanRows rows, few of which complete a block.
+constexpr int kMeanRows = 16;
+
 template <typename T, int N>
 __global__ void __launch_bounds__(kPrepThreads)
 block_mean_kernel(XpBlockMeanArgs a) {
-  const int row = blockIdx.x, pos = a.positions[row];
-  if (a.slots[row] < 0 || (pos + 1) % a.pool != 0) return;
-  const int* table = a.block_table + static_cast<size_t>(a.row_seq != nullptr ? a.row_seq[row] : row) * a.max_blocks;
+  const int first = blockIdx.x * kMeanRows, lane = threadIdx.x & 31;
+  const int mine = first + (lane < kMeanRows ? lane : 0);
+  const int my_pos = mine < a.rows ? a.positions[mine] : -1;
+  const int my_seq = mine < a.rows && a.row_seq != nullptr ? a.row_seq[mine] : mine;
+  const bool completes = lane < kMeanRows && my_pos >= 0 && a.slots[mine] >= 0 && (my_pos + 1) % a.pool == 0;
   const int nk = a.kv_heads * a.dq, total = nk + a.kv_heads * a.dv;
-  for (int i = threadIdx.x * N; i < total; i += kPrepThreads * N) {
-    const bool is_k = i < nk;
-    const int width = is_k ? a.dq : a.dv, e = is_k ? i : i - nk, h = e / width, c = e % width;
-    float mean[N];
-    block_mean<N, 8>(reinterpret_cast<const T*>(is_k ? a.k_cache : a.v_cache), table, pos, a.pool, a.page_size, a.kv_heads, h, width, c, nullptr, mean);
-    store_n<N>(reinterpret_cast<T*>(is_k ? a.k_pool : a.v_pool) + paged_row(table, pos / a.pool, a.pool_page, a.kv_heads, h, width) + c, mean);
+  for (uint32_t left = __ballot_sync(0xffffffffu, completes); left != 0; left &= left - 1) {
+    const int from = __ffs(left) - 1, pos = __shfl_sync(0xffffffffu, my_pos, from), seq = __shfl_sync(0xffffffffu, my_seq, from);
+    const int* table = a.block_table + static_cast<size_t>(seq) * a.max_blocks;
+    for (int i = threadIdx.x * N; i < total; i += kPrepThreads * N) {
+      const bool is_k = i < nk;
+      const int width = is_k ? a.dq : a.dv, e = is_k ? i : i - nk, h = e / width, c = e % width;
+      float mean[N];
+      block_mean<N, 8>(reinterpret_cast<const T*>(is_k ? a.k_cache : a.v_cache), table, pos, a.pool, a.page_size, a.kv_heads, h, width, c, nullptr, mean);
+      store_n<N>(reinterpret_cast<T*>(is_k ? a.k_pool : a.v_pool) + paged_row(table, pos / a.pool, a.pool_page, a.kv_heads, h, width) + c, mean);
+    }
   }
 }
 
@@ -327,25 +342,27 @@ extern "C" int xp_grouped_prep(const XpGroupedPrepArgs* a, void* stream) {
                  a->v_off % n == 0 && al(a->proj) && al(a->k_cache) && al(a->v_cache) && al(a->q_out) && al(a->k_pool) && al(a->v_pool);
   const int widest = a->dq > a->dv ? a->dq : a->dv;
   const int units = a->kv_heads * (a->group_pad + 2);
-  auto run = [&](auto kernel, int lanes) {               // few rows: as many slots at a time as fit; many: four slots per thread
-    int threads = a->rows <= 512 ? units * lanes : (units * lanes + 3) / 4;
-    threads = (threads + 31) / 32 * 32;
-    kernel<<<a->rows, threads < kPrepThreads ? threads : kPrepThreads, 0, s>>>(*a);
+  auto run = [&](auto kernel, int lanes) {               // few rows: a slot per thread, four CTAs or more per row; many: four slots per thread
+    const bool few = a->rows <= 512;
+    const int want = few ? units * lanes : (units * lanes + 3) / 4, most = few ? 128 : kPrepThreads;
+    const int threads = want < most ? (want + 31) / 32 * 32 : most;
+    kernel<<<dim3(a->rows, few ? (want + threads - 1) / threads : 1), threads, 0, s>>>(*a);
   };
-  auto pick = [&](auto means) {
-    constexpr bool M = decltype(means)::value;
+  auto pick = [&](auto inter, auto means) {
+    constexpr bool I = decltype(inter)::value, M = decltype(means)::value;
     if (a->f32) {
-      if (!v) run(grouped_prep_kernel<float, 1, 32, M>, 32);
-      else if (widest <= 64) run(grouped_prep_kernel<float, 4, 16, M>, 16);
-      else run(grouped_prep_kernel<float, 4, 32, M>, 32);
+      if (!v) run(grouped_prep_kernel<float, 1, 32, I, M>, 32);
+      else if (widest <= 64) run(grouped_prep_kernel<float, 4, 16, I, M>, 16);
+      else run(grouped_prep_kernel<float, 4, 32, I, M>, 32);
     } else {
-      if (!v) run(grouped_prep_kernel<__nv_bfloat16, 1, 32, M>, 32);
-      else if (widest <= 64) run(grouped_prep_kernel<__nv_bfloat16, 8, 8, M>, 8);
-      else run(grouped_prep_kernel<__nv_bfloat16, 8, 16, M>, 16);
+      if (!v) run(grouped_prep_kernel<__nv_bfloat16, 1, 32, I, M>, 32);
+      else if (widest <= 64) run(grouped_prep_kernel<__nv_bfloat16, 8, 8, I, M>, 8);
+      else run(grouped_prep_kernel<__nv_bfloat16, 8, 16, I, M>, 16);
     }
   };
-  if (a->pool > 0 && a->pool_rows > 0) pick(std::true_type{});
-  else pick(std::false_type{});
+  const bool pooling = a->pool > 0 && a->pool_rows > 0;
+  if (a->interleaved) pooling ? pick(std::true_type{}, std::true_type{}) : pick(std::true_type{}, std::false_type{});
+  else pooling ? pick(std::false_type{}, std::true_type{}) : pick(std::false_type{}, std::false_type{});
   return done();
 }
 
@@ -355,13 +372,14 @@ extern "C" int xp_block_mean(const XpBlockMeanArgs* a, void* stream) {
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   auto al = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
   const int n = a->f32 ? 4 : 8;
+  const int blocks = (a->rows + kMeanRows - 1) / kMeanRows;
   const bool v = a->dq % n == 0 && a->dv % n == 0 && al(a->k_cache) && al(a->v_cache) && al(a->k_pool) && al(a->v_pool);
   if (a->f32) {
-    if (v) block_mean_kernel<float, 4><<<a->rows, kPrepThreads, 0, s>>>(*a);
-    else block_mean_kernel<float, 1><<<a->rows, kPrepThreads, 0, s>>>(*a);
+    if (v) block_mean_kernel<float, 4><<<blocks, kPrepThreads, 0, s>>>(*a);
+    else block_mean_kernel<float, 1><<<blocks, kPrepThreads, 0, s>>>(*a);
   } else {
-    if (v) block_mean_kernel<__nv_bfloat16, 8><<<a->rows, kPrepThreads, 0, s>>>(*a);
-    else block_mean_kernel<__nv_bfloat16, 1><<<a->rows, kPrepThreads, 0, s>>>(*a);
+    if (v) block_mean_kernel<__nv_bfloat16, 8><<<blocks, kPrepThreads, 0, s>>>(*a);
+    else block_mean_kernel<__nv_bfloat16, 1><<<blocks, kPrepThreads, 0, s>>>(*a);
   }
   return done();
 }
