@@ -147,7 +147,8 @@ def kernel_table(classic: ModelConfig, cfg: ModelConfig, timer, context: int, ch
             w1, x1, o1 = rnd(no_, k), rnd(n, k), torch.empty(n, no_, dtype=bf, device=dev)
             add(f"{name} {n}", lambda: gemm.linear(x1, w1, out=o1), 2 * (w1.numel() + n * (k + no_)), 2.0 * n * w1.numel(), "" if name == "o product" else "o product")
             del w1, x1, o1
-    add(f"block means {T}", lambda: M.block_means(kc, vc, means, tp, p0, p0, torch.zeros_like(p0)), 2 * 2 * T * hk * d * (1 + 1 / POOL), 0.0, "rope + kv write")
+    seq = torch.zeros_like(p0)
+    add(f"block means {T}", lambda: M.block_means(kc, vc, means, tp, p0, p0, seq), 2 * 2 * T * hk * d * (1 + 1 / POOL), 0.0, "rope + kv write")
     lat_d = rnd(T, lat.cache_width)
     wek, kx = rnd(H * dq, R + r), torch.empty(T, H * dq, dtype=bf, device=dev)
     add(f"expand keys {T} (as Segirax)", lambda: gemm.linear(lat_d[:, :R + r], wek, out=kx), 2 * (wek.numel() + T * (R + r + H * dq)), 2.0 * T * wek.numel())

@@ -4,7 +4,8 @@ Every layer's linear maps of the same input become one matrix: the mixer's input
 parallel pair) and the residual gate (``[projections | gate | residual gate]``), each section padded to eight rows so that its
 columns in the product start on a 16-byte boundary. Latent attention keeps its up-projections twice: per head for the absorbed form (decode), and with the
 shared rotary key folded in as identity rows for the expanded form (prefill), so that one product writes complete per-head
-keys. Norm parameters, gates' biases and decays are fp32.
+keys; where queries come from a latent of their own, its norm's weight is part of the map behind it. Norm parameters, gates' biases,
+sinks and decays are fp32.
 """
 
 from __future__ import annotations
